@@ -24,29 +24,17 @@ from __future__ import annotations
 
 import os
 import time
-from collections import deque
 
 import numpy as np
-from dataclasses import dataclass, field
-from typing import Deque, Dict, List, Optional
+from typing import Dict, List, Optional
 
 import torch
 
 from .. import _native, ops
 from .._native import check, lib, stream_ptr
-from ..models.llama import GenerateConfig, LlamaModel
+from ..models.llama import LlamaModel
 from ..models.scheduler import EngineConfig
-from ..nn.kv_cache import BlockAllocator
-
-P, I, L, F = _native.P, _native.I, _native.L, _native.F
-_native.register_signatures({
-    "tsb_argmax_rows": [P, P, I, I, L, I, P],
-    "tsb_argmax_rows_pack": [P, P, I, I, L, I, I, P],
-    "tsb_argmax_rows_unpack": [P, P, I, I, I, P],
-    "tsb_sample_top_p_rows": [P, P, I, I, L, F, F, _native.ctypes.c_ulonglong, _native.ctypes.c_ulonglong, I, P],
-    "tsb_sample_rows": [P, P, I, I, L, F, I, F, _native.ctypes.c_ulonglong, _native.ctypes.c_ulonglong, P, I, P],
-    "tsb_repetition_penalty_rows": [P, I, I, L, P, L, P, F, I, P],
-})
+from .core import EngineCore, _Req, argmax_rows, repetition_penalty_rows_, sample_rows, sample_top_p_rows  # noqa: F401
 
 
 class _Weight:
@@ -64,28 +52,6 @@ class _Weight:
         if self.w is not None:
             return self.w.numel() * self.w.element_size()
         return self.q.numel() + self.s.numel() * 4      # (the scale atoms of the prompt-sized GEMM are 1 / 32 more)
-
-
-@dataclass
-class _Req:
-    id: int
-    gen: GenerateConfig
-    tokens: List[int]
-    prompt_len: int
-    generated: int = 0
-    finished: bool = False
-    blocks: List[int] = field(default_factory=list)
-    slot: int = -1                 # row of the engine's host-side state arrays while the request holds KV blocks
-    t_submit: float = 0.0
-    t_first: float = 0.0
-    t_done: float = 0.0
-
-
-def argmax_rows(logits: torch.Tensor) -> torch.Tensor:
-    out = torch.empty(logits.shape[0], dtype=torch.int32, device=logits.device)
-    check(lib().tsb_argmax_rows(logits.data_ptr(), out.data_ptr(), logits.shape[0], logits.shape[1], logits.stride(0),
-                                _native.dtype_code(logits.dtype), stream_ptr(logits.device)), "tsb_argmax_rows")
-    return out
 
 
 def argmax_rows_pack(logits: torch.Tensor, packed: torch.Tensor, rank: int, world: int) -> None:
@@ -111,37 +77,6 @@ def vocab_shard_rows(vocab: int, world: int) -> int:
     return shard if (world - 1) * shard < vocab else 0
 
 
-def sample_rows(logits: torch.Tensor, temperature: float, top_k: int, top_p: float, seed: int, step: int = 0,
-                step_counter: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Temperature -> top-k (0 = off) -> top-p -> one draw per row, on the device. With ``step_counter`` (an int64
-    device tensor of one element) the step is read from it when the kernel runs, so the launch can be captured in a
-    CUDA graph; the caller advances the counter."""
-    out = torch.empty(logits.shape[0], dtype=torch.int32, device=logits.device)
-    check(lib().tsb_sample_rows(logits.data_ptr(), out.data_ptr(), logits.shape[0], logits.shape[1], logits.stride(0),
-                                float(temperature), int(top_k), float(top_p), seed, step,
-                                step_counter.data_ptr() if step_counter is not None else None,
-                                _native.dtype_code(logits.dtype), stream_ptr(logits.device)), "tsb_sample_rows")
-    return out
-
-
-def repetition_penalty_rows_(logits: torch.Tensor, history: torch.Tensor, hist_len: torch.Tensor, penalty: float) -> None:
-    """In place: every occurrence of a token in ``history[row, :hist_len[row]]`` (int32) divides its positive logit
-    by ``penalty`` or multiplies its non-positive logit by it (src/models/Sampler.cpp:29-50)."""
-    check(lib().tsb_repetition_penalty_rows(logits.data_ptr(), logits.shape[0], logits.shape[1], logits.stride(0),
-                                            history.data_ptr(), history.stride(0), hist_len.data_ptr(), float(penalty),
-                                            _native.dtype_code(logits.dtype), stream_ptr(logits.device)),
-          "tsb_repetition_penalty_rows")
-
-
-def sample_top_p_rows(logits: torch.Tensor, temperature: float, top_p: float, seed: int, step: int) -> torch.Tensor:
-    out = torch.empty(logits.shape[0], dtype=torch.int32, device=logits.device)
-    check(lib().tsb_sample_top_p_rows(logits.data_ptr(), out.data_ptr(), logits.shape[0], logits.shape[1],
-                                      logits.stride(0), float(temperature), float(top_p), seed, step,
-                                      _native.dtype_code(logits.dtype), stream_ptr(logits.device)),
-          "tsb_sample_top_p_rows")
-    return out
-
-
 class TPServe:
     """Tensor-parallel context of a serving engine: process group, this rank, and the peer-memory all-reduce."""
 
@@ -162,14 +97,12 @@ class TPServe:
         return x
 
 
-class ServingEngine:
-    BUCKETS = (1, 2, 4, 8, 16, 32, 64, 128, 256, 512)
-
+class ServingEngine(EngineCore):
     def __init__(self, model: LlamaModel, cfg: Optional[EngineConfig] = None, use_cuda_graph: bool = True,
                  temperature: float = 0.0, top_p: float = 1.0, seed: int = 0, tp: Optional[TPServe] = None,
                  max_prefill_tokens: int = 0, fp8_prefill: bool = False, weights: str = "bf16", top_k: int = 0,
                  repetition_penalty: float = 1.0):
-        self.model, self.cfg = model, cfg or EngineConfig()
+        self.model = model
         self.tp = tp
         # weights="fp8": every layer projection and the LM head are held as E4M3 with 128 x 128 block scales (half the
         # bytes a decode step streams), the scales rounded up to powers of two. Decode-sized batches quantise the
@@ -179,7 +112,6 @@ class ServingEngine:
         if weights not in ("bf16", "fp8"):
             raise ValueError("ServingEngine: weights must be 'bf16' or 'fp8'")
         self.weights = weights
-        self.top_k, self.repetition_penalty = int(top_k), float(repetition_penalty)
         # fp8_prefill: the layer GEMMs of prefill-sized batches (more than 512 rows) run on E4M3 copies of the weights
         # with one scale per tensor and a per-call activation scale (about 2 x the bf16 GEMM rate); decode-sized
         # batches and the LM head stay bf16. Off by default: it changes the numerics of the prompt pass.
@@ -195,19 +127,19 @@ class ServingEngine:
         self.pdl = os.environ.get("TESSERACT_PDL", "1") == "1"
         self.stream_rows = 256       # batches up to this many rows count as decode-sized
         self.decode_gemm = os.environ.get("TESSERACT_SERVE_DECODE_GEMM", "auto")   # auto | mx | stream | splitk | fp8gemm (A/B runs)
-        c, mc = self.cfg, model.config
-        self.device = model._device()
-        if self.device.type != "cuda" or mc.dtype not in (torch.bfloat16, torch.float16):
+        mc = model.config
+        device = model._device()
+        if device.type != "cuda" or mc.dtype not in (torch.bfloat16, torch.float16):
             raise ValueError("ServingEngine needs a bf16 / fp16 model on a CUDA device "
                              "(use ContinuousBatchingScheduler for CPU or fp32 models)")
+        self._init_core(cfg, mc.vocab_size, device, temperature, top_p, seed, top_k, repetition_penalty)
+        c = self.cfg
         self.H, self.Hkv, self.D = mc.num_attention_heads, mc.kv_heads(), mc.head_dim
         if tp is not None:
             if self.H % tp.world or self.Hkv % tp.world or mc.intermediate_size % tp.world:
                 raise ValueError("ServingEngine: heads, KV heads and FFN width must divide over the TP ranks")
             self.H, self.Hkv = self.H // tp.world, self.Hkv // tp.world
         self.L = len(model.layers)
-        self.temperature, self.top_p, self.seed = temperature, top_p, seed
-        self.greedy = temperature <= 1e-6
         kv_dtype = torch.int8 if c.kv_int8 else mc.dtype
         shape = (self.L, c.num_blocks, self.Hkv, c.block_size, self.D)
         self.k_pool = torch.zeros(shape, dtype=kv_dtype, device=self.device)
@@ -216,8 +148,6 @@ class ServingEngine:
         if c.kv_int8:
             self.k_scale = torch.ones(shape[:-1], dtype=torch.float32, device=self.device)
             self.v_scale = torch.ones(shape[:-1], dtype=torch.float32, device=self.device)
-        self.allocator = BlockAllocator(c.num_blocks)
-        self.max_blocks = (c.max_seq_len + c.block_size - 1) // c.block_size
         self._fuse_weights()
         if self.fp8_prefill and self.weights == "bf16":
             from ..ops import fp8
@@ -225,25 +155,9 @@ class ServingEngine:
                 for W in ws:
                     if W.w is not None and W.w.dtype == torch.bfloat16 and W.shape[1] % 128 == 0:
                         self._w8[id(W)] = fp8.quantize_tensor(W.w)
-        self._step_dev = torch.zeros(1, dtype=torch.int64, device=self.device)   # sampling step counter (graph-safe)
-        self.waiting: Deque[_Req] = deque()
-        self.running: List[_Req] = []
-        self.requests: Dict[int, _Req] = {}
-        self._next_id = 0
-        self.steps = 0
         self.use_cuda_graph = use_cuda_graph
         self._graphs: Dict[int, dict] = {}
         self._host_inputs: Dict[int, torch.Tensor] = {}
-        # Host-side state of the resident requests as arrays indexed by a stable slot (block table, block count, last
-        # token, length): a decode step packs its inputs with a few gathers instead of a Python loop over requests.
-        cap = self.cfg.max_batch_size
-        self._tab = np.zeros((cap, self.max_blocks), dtype=np.int32)
-        self._nblk = np.zeros(cap, dtype=np.int32)
-        self._last = np.zeros(cap, dtype=np.int32)
-        self._len = np.zeros(cap, dtype=np.int32)
-        self._free_slots = list(range(cap - 1, -1, -1))
-        self.stats = {"prefill_tokens": 0, "decode_tokens": 0, "prefill_s": 0.0, "decode_s": 0.0, "decode_gpu_s": 0.0,
-                      "decode_steps": 0}
         self._step_events = (torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True))
 
     # ------------------------------------------------------------------ weights
@@ -350,71 +264,6 @@ class ServingEngine:
             q, sf, h = fp8.rms_norm_quant_mx(x, norm.weight, norm.eps, residual=res)
             return (q, sf), h
         return self._norm(x, res, norm, rows)
-
-    # ------------------------------------------------------------------ requests
-    def add_request(self, prompt_ids, gen: Optional[GenerateConfig] = None) -> int:
-        gen = gen or GenerateConfig()
-        prompt = [int(t) for t in prompt_ids]
-        if not prompt:
-            raise ValueError("add_request: empty prompt")
-        V = self.model.config.vocab_size
-        if any(t < 0 or t >= V for t in prompt):
-            raise ValueError("add_request: prompt id outside [0, vocab_size)")
-        if gen.max_new_tokens < 0 or len(prompt) + gen.max_new_tokens > self.cfg.max_seq_len:
-            raise ValueError("add_request: prompt + max_new_tokens exceeds max_seq_len")
-        r = _Req(self._next_id, gen, prompt, len(prompt), t_submit=time.perf_counter())
-        self._next_id += 1
-        self.waiting.append(r)
-        self.requests[r.id] = r
-        return r.id
-
-    def has_pending(self) -> bool:
-        return bool(self.waiting) or bool(self.running)
-
-    def num_running(self) -> int:
-        return len(self.running)
-
-    def num_waiting(self) -> int:
-        return len(self.waiting)
-
-    def free_blocks(self) -> int:
-        return self.allocator.num_free()
-
-    def allocated_blocks(self) -> int:
-        return self.allocator.num_used()
-
-    def is_finished(self, rid: int) -> bool:
-        return self.requests[rid].finished
-
-    def result(self, rid: int) -> List[int]:
-        r = self.requests[rid]
-        if not r.finished:
-            raise KeyError(f"request {rid} is not finished")
-        return list(r.tokens)
-
-    def _blocks_for(self, n: int) -> int:
-        return (n + self.cfg.block_size - 1) // self.cfg.block_size
-
-    def _grow(self, r: _Req, new_len: int) -> None:
-        if r.slot < 0:
-            r.slot = self._free_slots.pop()
-            self._tab[r.slot] = 0
-            self._nblk[r.slot] = 0
-        while len(r.blocks) < self._blocks_for(new_len):
-            b = self.allocator.allocate()
-            self._tab[r.slot, len(r.blocks)] = b
-            r.blocks.append(b)
-        self._nblk[r.slot] = len(r.blocks)
-
-    def _retire(self, r: _Req) -> None:
-        for b in r.blocks:
-            self.allocator.free(b)
-        r.blocks = []
-        if r.slot >= 0:
-            self._free_slots.append(r.slot)
-            r.slot = -1
-        r.finished = True
-        r.t_done = time.perf_counter()
 
     # ------------------------------------------------------------------ model pieces
     def _layer(self, li: int, x, res, positions, slots, tables, lens, prefill_bounds=None):
@@ -532,17 +381,7 @@ class ServingEngine:
         return self._mm(h.contiguous(), self.w_head)
 
     def _pick(self, logits: torch.Tensor, reqs: Optional[List[_Req]] = None) -> torch.Tensor:
-        """Next token per row, on the device. Greedy: arg-max. Otherwise the device sampler; its step comes from a
-        device counter that is advanced right after, so the pair can sit in a captured graph."""
-        if self.repetition_penalty != 1.0 and reqs is not None:
-            n = len(reqs)
-            width = max(len(r.tokens) for r in reqs)
-            hist = torch.zeros((logits.shape[0], width), dtype=torch.int32)
-            lens = torch.zeros(logits.shape[0], dtype=torch.int32)
-            for i, r in enumerate(reqs):
-                hist[i, :len(r.tokens)] = torch.tensor(r.tokens, dtype=torch.int32)
-                lens[i] = len(r.tokens)
-            repetition_penalty_rows_(logits, hist.to(logits.device), lens.to(logits.device), self.repetition_penalty)
+        """``EngineCore._pick``; greedy tensor-parallel serving picks from the shards of a vocabulary-parallel head."""
         if self.greedy and self.vocab_shard:
             tp, T = self.tp, logits.shape[0]
             if T > tp.max_rows:
@@ -551,11 +390,7 @@ class ServingEngine:
             argmax_rows_pack(logits, tp.head_ar.input_view(T, 4 * tp.world), tp.rank, tp.world)
             summed = tp.head_ar.reduce(T, 4 * tp.world)
             return argmax_rows_unpack(summed, tp.world, self.vocab_shard)
-        if self.greedy:
-            return argmax_rows(logits)
-        out = sample_rows(logits, self.temperature, self.top_k, self.top_p, self.seed, step_counter=self._step_dev)
-        self._step_dev.add_(1)
-        return out
+        return super()._pick(logits, reqs)
 
     # ------------------------------------------------------------------ scheduling
     def _admit(self) -> List[_Req]:
@@ -602,24 +437,6 @@ class ServingEngine:
             self._emit(r, int(t))
         self.stats["prefill_tokens"] += off
         self.stats["prefill_s"] += now - t0
-
-    def _emit(self, r: _Req, tok: int) -> None:
-        if r.gen.max_new_tokens == 0:
-            self._retire(r)
-            return
-        r.tokens.append(tok)
-        r.generated += 1
-        if r.slot >= 0:
-            self._last[r.slot] = tok
-            self._len[r.slot] = len(r.tokens)
-        if (r.gen.eos_token_id >= 0 and tok == r.gen.eos_token_id) or r.generated >= r.gen.max_new_tokens:
-            self._retire(r)
-
-    def _bucket(self, n: int) -> int:
-        for b in self.BUCKETS:
-            if b >= n:
-                return b
-        return n
 
     def _decode_inputs(self, reqs: List[_Req], A: int) -> torch.Tensor:
         """Packed int32 step inputs [A, 4 + max_blocks]: token, position, cache slot, length after the append,
@@ -718,26 +535,6 @@ class ServingEngine:
         self._graphs[A] = g
         return g
 
-    def instrument(self, metrics=None, watchdog=None, nvtx_ranges: Optional[bool] = None) -> "ServingEngine":
-        """Attach a ``utils.metrics.MetricsLogger`` (``run`` writes one summary record; every ``log_every`` steps a
-        progress record), a ``utils.watchdog.RankWatchdog`` (tensor-parallel serving: every step beats and checks the
-        peers on the host before it launches a collective) and / or NVTX ranges around prefill and decode (default:
-        the ``TESSERACT_NVTX`` environment variable)."""
-        import os
-        if metrics is not None:
-            self.metrics_logger = metrics
-        if watchdog is not None:
-            self.watchdog = watchdog
-        self.nvtx = bool(nvtx_ranges) if nvtx_ranges is not None else os.environ.get("TESSERACT_NVTX", "0") == "1"
-        return self
-
-    def _range(self, name: str):
-        import contextlib
-        if not getattr(self, "nvtx", False):
-            return contextlib.nullcontext()
-        from ..utils import nvtx
-        return nvtx.range_(name)
-
     def step(self) -> bool:
         wd = getattr(self, "watchdog", None)
         if wd is not None:
@@ -758,34 +555,3 @@ class ServingEngine:
             ml.log(event="serve_progress", step=self.steps, running=len(self.running), waiting=len(self.waiting),
                    decode_tokens=self.stats["decode_tokens"], prefill_tokens=self.stats["prefill_tokens"])
         return self.has_pending()
-
-    log_every = 100
-
-    def run(self) -> None:
-        try:
-            while self.has_pending():
-                self.step()
-        except Exception as e:
-            wd = getattr(self, "watchdog", None)
-            if wd is not None:
-                wd.report_failure(f"{type(e).__name__}: {e}")
-            raise
-        ml = getattr(self, "metrics_logger", None)
-        if ml is not None:
-            ml.log(event="serve_summary", **self.metrics())
-
-    # ------------------------------------------------------------------ metrics
-    def metrics(self) -> dict:
-        done = [r for r in self.requests.values() if r.finished and r.t_first > 0]
-        ttft = sorted((r.t_first - r.t_submit) * 1e3 for r in done)
-        s = self.stats
-        return {
-            "requests": len(done),
-            "prefill_tok_s": s["prefill_tokens"] / s["prefill_s"] if s["prefill_s"] > 0 else 0.0,
-            "decode_tok_s": s["decode_tokens"] / s["decode_s"] if s["decode_s"] > 0 else 0.0,
-            "ttft_p50_ms": ttft[len(ttft) // 2] if ttft else 0.0,
-            "steps": self.steps,
-            # wall time of a decode step against the device time of its captured graph: the difference is host work
-            "decode_ms_per_step": 1e3 * s["decode_s"] / max(1, s["decode_steps"]),
-            "decode_gpu_ms_per_step": 1e3 * s["decode_gpu_s"] / max(1, s["decode_steps"]),
-        }
