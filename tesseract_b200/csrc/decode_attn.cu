@@ -26,7 +26,7 @@ namespace tsb {
 
 int paged_decode_mma_dispatch(const void* q, const void* k_pool, const void* v_pool, const float* k_scale,
                               const float* v_scale, const int* tables, const int* lens, void* out, float* part_o, float* part_ml, int A, int H, int Hkv, int D, int bs, int nb,
-                              int max_logical, int splits, int gh, float scale_log2, int dtype, cudaStream_t s);
+                              int max_logical, int splits, int gh, float scale_log2, int chunk, int dtype, cudaStream_t s);
 
 namespace {
 
@@ -498,10 +498,9 @@ TSB_EXPORT long long tsb_paged_decode_scratch_floats(int A, int H, int D, int ma
 // out[a, h, :] = attention of query q[a, h, :] over the first lens[a] pooled tokens of request a.
 //   dtype: 1 = bf16, 2 = fp16 (q, out, and the pool unless k_scale != NULL, in which case the pool is INT8).
 //   max_len: upper bound of lens (sizes the key split); scratch: tsb_paged_decode_scratch_floats() floats.
-TSB_EXPORT int tsb_paged_decode(const void* q, const void* k_pool, const void* v_pool, const float* k_scale,
-                                const float* v_scale, const int* tables, const int* lens, void* out, float* scratch,
-                                int A, int H, int Hkv, int D, int bs, int nb, int max_logical, float scale,
-                                int max_len, int dtype, void* stream) {
+static int paged_decode(const void* q, const void* k_pool, const void* v_pool, const float* k_scale, const float* v_scale,
+                        const int* tables, const int* lens, void* out, float* scratch, int A, int H, int Hkv, int D, int bs,
+                        int nb, int max_logical, float scale, int max_len, int chunk, int dtype, void* stream) {
   using namespace tsb;
   if (A <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || (D != 64 && D != 128) || bs <= 0) return -2;
   const int G = H / Hkv;
@@ -513,7 +512,7 @@ TSB_EXPORT int tsb_paged_decode(const void* q, const void* k_pool, const void* v
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   {
     int rc = paged_decode_mma_dispatch(q, k_pool, v_pool, k_scale, v_scale, tables, lens, out, part_o, part_ml, A, H, Hkv, D, bs, nb,
-                                       max_logical, splits, gh, scale * 1.4426950408889634f, dtype, s);
+                                       max_logical, splits, gh, scale * 1.4426950408889634f, chunk, dtype, s);
     if (rc != -100) {
       if (rc != 0 || splits == 1) return rc;
       if (dtype == 1) {
@@ -528,6 +527,7 @@ TSB_EXPORT int tsb_paged_decode(const void* q, const void* k_pool, const void* v
       return static_cast<int>(cudaGetLastError());
     }
   }
+  if (chunk > 0) return -2;   // the CUDA-core kernel knows no chunk mask
   DecParams p;
   p.q = q; p.k_pool = k_pool; p.v_pool = v_pool; p.k_scale = k_scale; p.v_scale = v_scale;
   p.tables = tables; p.lens = lens; p.out = out;
@@ -545,6 +545,24 @@ TSB_EXPORT int tsb_paged_decode(const void* q, const void* k_pool, const void* v
     return i8 ? launch_decode<__half, true, 64>(p, G, s) : launch_decode<__half, false, 64>(p, G, s);
   }
   return -2;
+}
+
+TSB_EXPORT int tsb_paged_decode(const void* q, const void* k_pool, const void* v_pool, const float* k_scale,
+                                const float* v_scale, const int* tables, const int* lens, void* out, float* scratch,
+                                int A, int H, int Hkv, int D, int bs, int nb, int max_logical, float scale,
+                                int max_len, int dtype, void* stream) {
+  return paged_decode(q, k_pool, v_pool, k_scale, v_scale, tables, lens, out, scratch, A, H, Hkv, D, bs, nb, max_logical, scale,
+                      max_len, 0, dtype, stream);
+}
+
+// The same under a chunk mask: the newest token (position lens[a] - 1) sees only the keys of its own run of `chunk`
+// positions. max_len bounds lens as above (the key split is planned for min(max_len, chunk) keys); bf16 / fp16 pools.
+TSB_EXPORT int tsb_paged_decode_chunked(const void* q, const void* k_pool, const void* v_pool, const int* tables,
+                                        const int* lens, void* out, float* scratch, int A, int H, int Hkv, int D, int bs, int nb,
+                                        int max_logical, float scale, int max_len, int chunk, int dtype, void* stream) {
+  if (chunk <= 0) return -2;
+  return paged_decode(q, k_pool, v_pool, nullptr, nullptr, tables, lens, out, scratch, A, H, Hkv, D, bs, nb, max_logical, scale,
+                      max_len < chunk ? max_len : chunk, chunk, dtype, stream);
 }
 
 extern "C" int tsb_quant_act_mx_layout(const void* X, long long ldx, void* Xq, void* sf, int M, int K, int atoms,
@@ -568,7 +586,7 @@ TSB_EXPORT int tsb_paged_decode_mx(const void* q, const void* k_pool, const void
     float* part_o = scratch;
     float* part_ml = scratch + static_cast<long long>(A) * H * splits * D;
     const int rc = paged_decode_mma_dispatch(q, k_pool, v_pool, k_scale, v_scale, tables, lens, out, part_o, part_ml, A, H,
-                                             Hkv, D, bs, nb, max_logical, splits, gh, scale * 1.4426950408889634f,
+                                             Hkv, D, bs, nb, max_logical, splits, gh, scale * 1.4426950408889634f, 0,
                                              dtype, s);
     if (rc == 0) {
       launch_pdl(decode_merge_quant_mx_kernel, dim3(A * H), dim3(128), 0, s, pdl_all_enabled(), part_o, part_ml,

@@ -88,6 +88,7 @@ struct MmaDecParams {
   float* part_ml;
   int A, H, Hkv, bs, nb, max_logical, splits, gh;  // gh = query heads per CTA (<= 8)
   float scale_log2;
+  int chunk;             // > 0: the newest token sees only the keys of its own run of `chunk` positions
   int* status;           // device status word: a block-table entry outside the pool is reported there
 };
 
@@ -127,9 +128,10 @@ paged_decode_mma_kernel(MmaDecParams p) {
   const int g = lane >> 2, t4 = lane & 3;
 
   const int len = p.lens[a];
-  const int chunk = ((len + p.splits - 1) / p.splits + 15) & ~15;
-  const int t_begin = split * chunk;
-  const int t_end = min(len, t_begin + chunk);
+  const int first = p.chunk > 0 && len > 0 ? (len - 1) / p.chunk * p.chunk : 0;
+  const int share = ((len - first + p.splits - 1) / p.splits + 15) & ~15;
+  const int t_begin = first + split * share;
+  const int t_end = min(len, t_begin + share);
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + kTile - 1) / kTile : 0;
 
   uint8_t* wsmem = smem + warp * kWarpBytes;
@@ -449,7 +451,7 @@ int launch_mma(const MmaDecParams& p, cudaStream_t s) {
 int paged_decode_mma_dispatch(const void* q, const void* k_pool, const void* v_pool, const float* k_scale,
                               const float* v_scale, const int* tables, const int* lens,
                               void* out, float* part_o, float* part_ml, int A, int H, int Hkv, int D, int bs, int nb,
-                              int max_logical, int splits, int gh, float scale_log2, int dtype, cudaStream_t s) {
+                              int max_logical, int splits, int gh, float scale_log2, int chunk, int dtype, cudaStream_t s) {
   if (gh > 8 || (D != 64 && D != 128)) return -100;
   MmaDecParams p;
   p.q = q; p.k_pool = k_pool; p.v_pool = v_pool; p.k_scale = k_scale; p.v_scale = v_scale;
@@ -457,6 +459,7 @@ int paged_decode_mma_dispatch(const void* q, const void* k_pool, const void* v_p
   p.part_o = part_o; p.part_ml = part_ml;
   p.A = A; p.H = H; p.Hkv = Hkv; p.bs = bs; p.nb = nb; p.max_logical = max_logical; p.splits = splits; p.gh = gh;
   p.scale_log2 = scale_log2;
+  p.chunk = chunk;
   p.status = device_status_word();
   const bool i8 = k_scale != nullptr;
   if (dtype == 1) {

@@ -44,6 +44,7 @@ struct FaParams {
   int B, Sq, Sk, H, Hkv;
   long long o_sb, o_ss, o_sh;
   const int* cu_seqlens;  // varlen: int32 [B + 1] row offsets of the sequences in the packed token axis, else null
+  const int* cu_keys;     // varlen: row offsets of the sequences' keys on a key axis of their own, null: the token axis
   float scale_log2;  // softmax scale * log2(e)
   float scale;
   int causal;
@@ -75,11 +76,17 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   // block z handles sequence z, whose rows start at cu_seqlens[z]. Tiles that reach past its end read rows of the
   // next sequence (or the zero fill) and the length mask below discards them.
   FaParams p = p_in;
-  int row0 = 0;
+  // With `cu_keys` the keys of a sequence are rows of a second axis and may outnumber the queries: the queries are then
+  // the last Sq of its Sk positions.
+  int row0 = 0, krow0 = 0;
   int bb = blockIdx.z;
   if (p_in.cu_seqlens) {
-    row0 = p_in.cu_seqlens[blockIdx.z];
+    row0 = krow0 = p_in.cu_seqlens[blockIdx.z];
     p.Sq = p.Sk = p_in.cu_seqlens[blockIdx.z + 1] - row0;
+    if (p_in.cu_keys) {
+      krow0 = p_in.cu_keys[blockIdx.z];
+      p.Sk = p_in.cu_keys[blockIdx.z + 1] - krow0;
+    }
     bb = 0;
     if (static_cast<int>(gridDim.x - 1 - blockIdx.x) * BQ >= p.Sq) return;  // no query rows: the whole CTA leaves
   }
@@ -151,12 +158,12 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         mbar_expect_tx(&k_full[st], Cfg::kTileBytes);
 #pragma unroll
         for (int hf = 0; hf < Cfg::kHalves; ++hf)
-          tma_load_4d(sK + st * Cfg::kTileBytes + hf * 16384, &tmK, &k_full[st], hf * 64, j * BKV + row0, hk, bb);
+          tma_load_4d(sK + st * Cfg::kTileBytes + hf * 16384, &tmK, &k_full[st], hf * 64, j * BKV + krow0, hk, bb);
         if (!mbar_wait(&v_empty[st], par, &cta_abort, p.status)) break;
         mbar_expect_tx(&v_full[st], Cfg::kTileBytes);
 #pragma unroll
         for (int hf = 0; hf < Cfg::kHalves; ++hf)
-          tma_load_4d(sV + st * Cfg::kTileBytes + hf * 16384, &tmV, &v_full[st], hf * 64, j * BKV + row0, hk, bb);
+          tma_load_4d(sV + st * Cfg::kTileBytes + hf * 16384, &tmV, &v_full[st], hf * 64, j * BKV + krow0, hk, bb);
       }
     }
   } else if (warp == 5) {
@@ -554,7 +561,7 @@ TSB_EXPORT int tsb_flash_fwd(const void* q, const void* k, const void* v, void* 
   FaParams p;
   p.o = static_cast<__nv_bfloat16*>(o);
   p.lse = lse;
-  p.cu_seqlens = nullptr;
+  p.cu_seqlens = p.cu_keys = nullptr;
   p.B = B; p.Sq = Sq; p.Sk = Sk; p.H = H; p.Hkv = Hkv;
   p.o_sb = o_sb; p.o_ss = o_ss; p.o_sh = o_sh;
   p.scale = scale;
@@ -588,12 +595,12 @@ TSB_EXPORT int tsb_flash_fwd(const void* q, const void* k, const void* v, void* 
 // different lengths in ONE launch): q [T, H, D], k / v [T, Hkv, D], o [T, H, D] bf16 with token / head strides in
 // elements (unit stride in D, multiples of 8, 16-byte aligned bases); cu_seqlens int32 [n_seqs + 1] on the device,
 // cu_seqlens[0] = 0, cu_seqlens[n_seqs] = T; max_len >= the longest sequence. D is 64 or 128.
-TSB_EXPORT int tsb_flash_fwd_varlen(const void* q, const void* k, const void* v, void* o, const int* cu_seqlens,
-                                    int n_seqs, int max_len, int T, int H, int Hkv, int D, long long q_ss, long long q_sh,
-                                    long long k_ss, long long k_sh, long long v_ss, long long v_sh, long long o_ss,
-                                    long long o_sh, float scale, void* stream) {
+static int flash_fwd_varlen(const void* q, const void* k, const void* v, void* o, const int* cu_seqlens, const int* cu_keys,
+                            int n_seqs, int max_len, int T, int TK, int H, int Hkv, int D, long long q_ss, long long q_sh,
+                            long long k_ss, long long k_sh, long long v_ss, long long v_sh, long long o_ss,
+                            long long o_sh, float scale, void* stream) {
   using namespace tsb;
-  if (n_seqs <= 0 || max_len <= 0 || T <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || (D != 64 && D != 128) || !cu_seqlens)
+  if (n_seqs <= 0 || max_len <= 0 || T <= 0 || TK <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || (D != 64 && D != 128) || !cu_seqlens)
     return -2;
   const long long strides[] = {q_ss, q_sh, k_ss, k_sh, v_ss, v_sh, o_ss, o_sh};
   for (long long st : strides)
@@ -602,14 +609,15 @@ TSB_EXPORT int tsb_flash_fwd_varlen(const void* q, const void* k, const void* v,
        reinterpret_cast<uintptr_t>(o)) & 15)
     return -2;
   CUtensorMap tq, tk, tv;
-  const long long big = static_cast<long long>(T) * std::max({q_ss, k_ss, v_ss});  // batch stride of the single batch
+  const long long big = static_cast<long long>(std::max(T, TK)) * std::max({q_ss, k_ss, v_ss});  // batch stride of the single batch
   if (!make_bshd_tmap(&tq, q, 1, T, H, D, big, q_ss, q_sh, 128)) return -3;
-  if (!make_bshd_tmap(&tk, k, 1, T, Hkv, D, big, k_ss, k_sh, 128)) return -3;
-  if (!make_bshd_tmap(&tv, v, 1, T, Hkv, D, big, v_ss, v_sh, 128)) return -3;
+  if (!make_bshd_tmap(&tk, k, 1, TK, Hkv, D, big, k_ss, k_sh, 128)) return -3;
+  if (!make_bshd_tmap(&tv, v, 1, TK, Hkv, D, big, v_ss, v_sh, 128)) return -3;
   FaParams p;
   p.o = static_cast<__nv_bfloat16*>(o);
   p.lse = nullptr;
   p.cu_seqlens = cu_seqlens;
+  p.cu_keys = cu_keys;
   p.B = n_seqs; p.Sq = max_len; p.Sk = max_len; p.H = H; p.Hkv = Hkv;
   p.o_sb = 0; p.o_ss = o_ss; p.o_sh = o_sh;
   p.scale = scale;
@@ -628,4 +636,24 @@ TSB_EXPORT int tsb_flash_fwd_varlen(const void* q, const void* k, const void* v,
                             : launch(flash_fwd_kernel<64, false>, FaCfg<64>::kSmemBytes);
   if (rc) return rc;
   return static_cast<int>(cudaGetLastError());
+}
+
+TSB_EXPORT int tsb_flash_fwd_varlen(const void* q, const void* k, const void* v, void* o, const int* cu_seqlens,
+                                    int n_seqs, int max_len, int T, int H, int Hkv, int D, long long q_ss, long long q_sh,
+                                    long long k_ss, long long k_sh, long long v_ss, long long v_sh, long long o_ss,
+                                    long long o_sh, float scale, void* stream) {
+  return flash_fwd_varlen(q, k, v, o, cu_seqlens, nullptr, n_seqs, max_len, T, T, H, Hkv, D, q_ss, q_sh, k_ss, k_sh, v_ss,
+                          v_sh, o_ss, o_sh, scale, stream);
+}
+
+// The same with the keys on an axis of their own (k / v [TK, Hkv, D], cu_keys int32 [n_seqs + 1], cu_keys[n_seqs] = TK):
+// the queries of sequence i are its last Sq positions and see every key before them. Used for portions of prompts
+// (keys of earlier portions, then the portion's own) and for chunked masks (one "sequence" per chunk).
+TSB_EXPORT int tsb_flash_fwd_varlen_keys(const void* q, const void* k, const void* v, void* o, const int* cu_seqlens,
+                                         const int* cu_keys, int n_seqs, int max_len, int T, int TK, int H, int Hkv, int D,
+                                         long long q_ss, long long q_sh, long long k_ss, long long k_sh, long long v_ss,
+                                         long long v_sh, long long o_ss, long long o_sh, float scale, void* stream) {
+  if (!cu_keys) return -2;
+  return flash_fwd_varlen(q, k, v, o, cu_seqlens, cu_keys, n_seqs, max_len, T, TK, H, Hkv, D, q_ss, q_sh, k_ss, k_sh, v_ss,
+                          v_sh, o_ss, o_sh, scale, stream);
 }
