@@ -75,6 +75,14 @@ def cuda_lib_path() -> Path:
     return _CUDA_LIB_PATH
 
 
+def use_library(path) -> None:
+    """Loads this library instead of the full one (``build.ensure`` built the part of it that a program needs)."""
+    global _CUDA_LIB_PATH
+    if _lib is not None and Path(path) != _CUDA_LIB_PATH:
+        raise RuntimeError("use_library: a CUDA library is loaded already")
+    _CUDA_LIB_PATH = Path(path)
+
+
 def available() -> bool:
     """True when the built CUDA library exists on disk (it may still need a GPU to run)."""
     return _CUDA_LIB_PATH.exists()

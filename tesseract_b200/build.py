@@ -9,7 +9,8 @@ Two artefacts, both placed inside the package so that they travel with a source 
 * ``tesseract_b200/_lib/_tsb_host*.so`` -- the host runtime (safetensors reads, BPE merge loop, sampler, regex
   compiler and token mask, block allocator, CPU GEMV and GEMM), a pybind11 module built from ``csrc/host``.
 
-``python -m tesseract_b200.build`` rebuilds whatever is out of date (``--force`` rebuilds everything).
+``python -m tesseract_b200.build`` rebuilds whatever is out of date (``--force`` rebuilds everything). Programs that serve
+one model family from a fresh checkout call ``ensure(group)``, which compiles only that family's translation units.
 """
 from __future__ import annotations
 
@@ -29,6 +30,12 @@ LIB_DIR = PKG / "_lib"
 OBJ_DIR = PKG.parent / "build" / "obj"
 
 CUDA_LIB = LIB_DIR / "libtesseract_b200_cuda.so"
+
+# translation units of one model family: what its kernels are in and what those link against
+GROUPS = {
+    "hybrid": ("runtime", "gemm_tcgen05", "gemm_decode_wq", "gemm_decode_mx", "decode_attn", "decode_attn_mma", "flash_attn_fwd",
+               "ragged_attn", "delta_rule", "dyn_tanh", "sampling"),
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -68,12 +75,18 @@ def _run(cmd, verbose):
     return r.stdout + r.stderr
 
 
-def build_cuda(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
-    """Compile csrc/*.cu for sm_100a and link libtesseract_b200_cuda.so. Returns its path."""
+def group_lib(group: str) -> Path:
+    return LIB_DIR / f"libtesseract_b200_cuda.{group}.so"
+
+
+def build_cuda(force: bool = False, verbose: bool = False, ptxas_info: bool = False, group: str = "") -> Path:
+    """Compile csrc/*.cu for sm_100a and link libtesseract_b200_cuda.so -- or, with ``group``, only that group's units into
+    a library of their own. Returns its path."""
+    lib = group_lib(group) if group else CUDA_LIB
     nvcc = _nvcc()
     LIB_DIR.mkdir(parents=True, exist_ok=True)
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
-    sources = sorted(CSRC.glob("*.cu"))
+    sources = [CSRC / f"{n}.cu" for n in GROUPS[group]] if group else sorted(CSRC.glob("*.cu"))
     headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
     flags = NVCC_FLAGS + (["-Xptxas", "-v"] if ptxas_info else [])
     hdr_digest = _digest(headers, flags)
@@ -98,12 +111,27 @@ def build_cuda(force: bool = False, verbose: bool = False, ptxas_info: bool = Fa
             for name, out in ex.map(compile_one, jobs):
                 if ptxas_info and out:
                     print(f"== {name}\n{out}")
-    link_stamp = OBJ_DIR / "link.stamp"
+    link_stamp = OBJ_DIR / (f"link.{group}.stamp" if group else "link.stamp")
     want_link = hashlib.sha256("".join((OBJ_DIR / (s.stem + ".stamp")).read_text() for s in sources).encode()).hexdigest()
-    if jobs or not CUDA_LIB.exists() or not link_stamp.exists() or link_stamp.read_text() != want_link:
-        _run([nvcc, "-shared", "-o", str(CUDA_LIB), *map(str, objs), "-Xcompiler", "-fPIC", "-lcudart"], verbose)
+    if jobs or not lib.exists() or not link_stamp.exists() or link_stamp.read_text() != want_link:
+        part = lib.with_suffix(".part")
+        _run([nvcc, "-shared", "-o", str(part), *map(str, objs), "-Xcompiler", "-fPIC", "-lcudart"], verbose)
+        os.replace(part, lib)      # (a process that has the old file loaded keeps it)
         link_stamp.write_text(want_link)
-    return CUDA_LIB
+    return lib
+
+
+def ensure(group: str) -> Path:
+    """The library to load for ``group``: the full one if it is there, else the group's own, compiled now if it is missing
+    or older than its sources. Concurrent callers wait for one another."""
+    import fcntl
+
+    if CUDA_LIB.exists():
+        return CUDA_LIB
+    LIB_DIR.mkdir(parents=True, exist_ok=True)
+    with open(LIB_DIR / f".{group}.lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build_cuda(group=group)
 
 
 def build_host(force: bool = False, verbose: bool = False) -> Path:

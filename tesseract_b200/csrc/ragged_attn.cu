@@ -1,9 +1,9 @@
 // Paged attention pieces for ragged batches: portions of prompts beside single decoded tokens, with an optional chunk
 // mask (token i sees the tokens j <= i of its own run of `chunk` positions, counted from position 0).
 //
-//   ragged_append_kernel   adds the projection biases to a packed [q | k | v] row, leaves q in place, and stores k and v
-//                          in the pool slot of the token and, for prompt rows, in the contiguous key axis that the
-//                          tcgen05 attention kernel reads (`stage`).
+//   ragged_append_kernel   adds the projection biases to a packed [q | k | v] row, writes q to a buffer of its own, and
+//                          stores k and v in the pool slot of the token and, for prompt rows, in the contiguous key axis
+//                          that the tcgen05 attention kernel reads (`stage`).
 //   stage_gather_kernel    copies keys and values that earlier portions left in the pool to the key axis.
 //   ragged_attn_kernel     attention of each row over the pool: one warp per (row, head), fp32 arithmetic. Serves fp32
 //                          models and head sizes that the tensor-core kernels do not take.
@@ -35,7 +35,7 @@ __device__ __forceinline__ uint4 pack16(const float (&f)[kVec<T>]) {
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-ragged_append_kernel(T* qkv, long long ld, const float* bias, const int* slots, T* k_pool, T* v_pool, T* stage,
+ragged_append_kernel(const T* qkv, long long ld, const float* bias, const int* slots, T* q_out, T* k_pool, T* v_pool, T* stage,
                      const int* stage_rows, int stage_from, int rows, int H, int Hkv, int D, int bs) {
   pdl_trigger();
   pdl_grid_wait();
@@ -46,7 +46,7 @@ ragged_append_kernel(T* qkv, long long ld, const float* bias, const int* slots, 
   const int row = static_cast<int>(idx / vpr), w = static_cast<int>(idx % vpr);
   if (row >= rows) return;
   const int head = w / vph, d = (w % vph) * V;
-  T* src = qkv + row * ld + head * D + d;
+  const T* src = qkv + row * ld + head * D + d;
   float f[V];
   load16<T>(src, f);
   if (bias) {
@@ -55,7 +55,7 @@ ragged_append_kernel(T* qkv, long long ld, const float* bias, const int* slots, 
   }
   const uint4 val = pack16<T>(f);
   if (head < H) {
-    if (bias) *reinterpret_cast<uint4*>(src) = val;
+    *reinterpret_cast<uint4*>(q_out + (static_cast<long long>(row) * H + head) * D + d) = val;
     return;
   }
   const int hk = (head - H) % Hkv;
@@ -182,9 +182,9 @@ int launch_ragged_attn(const RaggedAttnParams& p, int D, cudaStream_t s) {
 }  // namespace tsb
 
 // qkv [rows, ld] = packed [q: H heads | k: Hkv | v: Hkv] of D, bf16 (dtype 1) or fp32 (0); bias fp32 [(H + 2 Hkv) D] or
-// null. Pools [blocks, Hkv, bs, D]; slots[row] = block * bs + offset (-1: no slot). Rows from stage_from on also go to
+// null; q_out [rows, H, D]. Pools [blocks, Hkv, bs, D]; slots[row] = block * bs + offset (-1: no slot). Rows from stage_from on also go to
 // stage [*, 2 Hkv, D] at stage_rows[row - stage_from] when stage is given. D % 8 == 0, 16-byte aligned bases and rows.
-TSB_EXPORT int tsb_ragged_append(void* qkv, long long ld, const float* bias, const int* slots, void* k_pool, void* v_pool,
+TSB_EXPORT int tsb_ragged_append(const void* qkv, long long ld, const float* bias, const int* slots, void* q_out, void* k_pool, void* v_pool,
                                  void* stage, const int* stage_rows, int stage_from, int rows, int H, int Hkv, int D, int bs,
                                  int dtype, void* stream) {
   using namespace tsb;
@@ -194,12 +194,12 @@ TSB_EXPORT int tsb_ragged_append(void* qkv, long long ld, const float* bias, con
   if (vecs > 0x7fffffffLL) return -2;
   const dim3 grid(static_cast<unsigned>((vecs + 255) / 256));
   if (dtype == 1)
-    launch_pdl(ragged_append_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl_all_enabled(), static_cast<__nv_bfloat16*>(qkv), ld,
-               bias, slots, static_cast<__nv_bfloat16*>(k_pool), static_cast<__nv_bfloat16*>(v_pool),
+    launch_pdl(ragged_append_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl_all_enabled(), static_cast<const __nv_bfloat16*>(qkv), ld,
+               bias, slots, static_cast<__nv_bfloat16*>(q_out), static_cast<__nv_bfloat16*>(k_pool), static_cast<__nv_bfloat16*>(v_pool),
                static_cast<__nv_bfloat16*>(stage), stage_rows, stage_from, rows, H, Hkv, D, bs);
   else if (dtype == 0)
-    launch_pdl(ragged_append_kernel<float>, grid, dim3(256), 0, s, pdl_all_enabled(), static_cast<float*>(qkv), ld, bias, slots,
-               static_cast<float*>(k_pool), static_cast<float*>(v_pool), static_cast<float*>(stage), stage_rows, stage_from, rows,
+    launch_pdl(ragged_append_kernel<float>, grid, dim3(256), 0, s, pdl_all_enabled(), static_cast<const float*>(qkv), ld, bias, slots,
+               static_cast<float*>(q_out), static_cast<float*>(k_pool), static_cast<float*>(v_pool), static_cast<float*>(stage), stage_rows, stage_from, rows,
                H, Hkv, D, bs);
   else
     return -2;

@@ -53,8 +53,10 @@ class ContinuousBatchingScheduler:
         c = self.cfg
         if c.block_size <= 0 or c.num_blocks <= 0 or c.max_batch_size <= 0:
             raise ValueError("EngineConfig: block_size, num_blocks and max_batch_size must be positive")
+        # models with recurrent state also need a slot per sequence
+        extra = {"max_sequences": c.max_batch_size, "max_len": c.max_seq_len} if hasattr(model, "make_cache") else {}
         self.pools = (model.make_quantized_layer_pools(c.num_blocks, c.block_size) if c.kv_int8
-                      else model.make_layer_pools(c.num_blocks, c.block_size))
+                      else model.make_layer_pools(c.num_blocks, c.block_size, **extra))
         self.waiting: Deque[_Request] = deque()
         self.running: List[int] = []
         self.requests: Dict[int, _Request] = {}

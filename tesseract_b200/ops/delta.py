@@ -1,0 +1,170 @@
+"""Gated delta rule over ragged batches (``csrc/delta_rule.cu``): per value head a state S [dim, vdim] with
+
+    S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+
+fed by short causal convolutions of a packed projection and read out through a per-head RMS norm and a SiLU gate.
+``gated_delta`` takes the projection of a ragged batch (decoded rows first, then portions of prompts), advances the
+slots of a state pool and returns the gated read-outs. CPU tensors run the torch restatement below.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+
+import torch
+
+from .. import _native
+from .._native import check, dtype_code, lib, stream_ptr
+
+P, I, L, F = _native.P, _native.I, _native.L, _native.F
+_native.register_signatures({
+    "tsb_delta_prefill": [P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, F, I, P],
+    "tsb_delta_step": [P, L, P, P, P, P, P, P, P, P, P, P, L, I, I, I, F, I, P],
+})
+
+MAX_TAPS = 8
+MAX_DIM = 256
+
+
+def _up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+@dataclass(frozen=True)
+class DeltaGeometry:
+    """Sizes of one mixer and the layout of its packed projection row: [q | k | v | gate | b | a], every section padded to
+    a multiple of 8 columns."""
+    kv_heads: int
+    heads: int
+    dim: int
+    vdim: int
+    taps: int
+
+    def __post_init__(self):
+        if min(self.kv_heads, self.heads, self.dim, self.vdim, self.taps) < 1 or self.heads % self.kv_heads:
+            raise ValueError("delta rule: positive sizes, and heads a multiple of kv_heads")
+        if self.dim > MAX_DIM or self.taps > MAX_TAPS:
+            raise ValueError(f"delta rule: dim <= {MAX_DIM} and at most {MAX_TAPS} convolution taps")
+
+    @property
+    def dim_pad(self) -> int:
+        return next(d for d in (32, 64, 128, 256) if d >= self.dim)
+
+    @property
+    def vdim_pad(self) -> int:
+        return _up(self.vdim, 4)
+
+    @property
+    def off_k(self) -> int:
+        return _up(self.kv_heads * self.dim, 8)
+
+    @property
+    def off_v(self) -> int:
+        return 2 * self.off_k
+
+    @property
+    def off_gate(self) -> int:
+        return self.off_v + _up(self.heads * self.vdim, 8)
+
+    conv_cols = off_gate
+
+    @property
+    def off_b(self) -> int:
+        return self.off_gate + _up(self.heads * self.vdim, 8)
+
+    @property
+    def off_a(self) -> int:
+        return self.off_b + _up(self.heads, 8)
+
+    @property
+    def cols(self) -> int:
+        return self.off_a + _up(self.heads, 8)
+
+    @property
+    def out_cols(self) -> int:
+        return _up(self.heads * self.vdim, 16)
+
+    def as_ints(self):
+        v = (self.kv_heads, self.heads, self.dim, self.vdim, self.dim_pad, self.vdim_pad, self.off_k, self.off_v,
+             self.off_gate, self.off_b, self.off_a, self.conv_cols)
+        return (ctypes.c_int * len(v))(*v)
+
+
+@dataclass
+class DeltaWeights:
+    """fp32 parameters of the mixer besides its projections: convolution taps [taps, conv_cols], A_log and dt_bias [heads],
+    norm [vdim]."""
+    conv: torch.Tensor
+    a_log: torch.Tensor
+    dt_bias: torch.Tensor
+    norm: torch.Tensor
+    eps: float
+
+
+def gated_delta(proj: torch.Tensor, geo: DeltaGeometry, w: DeltaWeights, conv_state: torch.Tensor, state: torch.Tensor,
+                batch) -> torch.Tensor:
+    """proj [T, geo.cols] of a ragged batch -> [T, geo.out_cols]. ``conv_state`` [slots, taps - 1, conv_cols] (projection
+    dtype) and ``state`` [slots, heads, dim, vdim_pad] (fp32) are advanced in place for the batch's sequences; a sequence
+    whose first row is at position 0 starts from zeros whatever its slot holds."""
+    T = proj.shape[0]
+    y = torch.empty((T, geo.out_cols), device=proj.device, dtype=proj.dtype)
+    if T == 0:
+        return y
+    if not proj.is_cuda:
+        return _gated_delta_torch(proj, geo, w, conv_state, state, batch, y)
+    nd = batch.n_decode
+    g = geo.as_ints()
+    dt, st = dtype_code(proj.dtype), stream_ptr(proj.device)
+    if nd:
+        check(lib().tsb_delta_step(proj.data_ptr(), proj.stride(0), g, w.conv.data_ptr(), w.a_log.data_ptr(), w.dt_bias.data_ptr(),
+                                   w.norm.data_ptr(), conv_state.data_ptr(), state.data_ptr(), batch.state_slots.data_ptr(),
+                                   batch.positions.data_ptr(), y.data_ptr(), y.stride(0), geo.out_cols, nd, geo.taps,
+                                   float(w.eps), dt, st), "tsb_delta_step")
+    n = T - nd
+    if n:
+        H, dev = geo.heads, proj.device
+        kq = torch.empty((n, geo.kv_heads, 2, geo.dim_pad), device=dev, dtype=torch.float32)
+        v = torch.empty((n, H, geo.vdim_pad), device=dev, dtype=torch.float32)
+        gates = torch.empty((n, H, 4), device=dev, dtype=torch.float32)
+        o = torch.empty((n, H, geo.vdim_pad), device=dev, dtype=torch.float32)
+        pr = proj[nd:]
+        check(lib().tsb_delta_prefill(pr.data_ptr(), pr.stride(0), g, w.conv.data_ptr(), w.a_log.data_ptr(), w.dt_bias.data_ptr(),
+                                      w.norm.data_ptr(), conv_state.data_ptr(), state.data_ptr(), batch.cu.data_ptr(),
+                                      batch.state_slots[nd:].data_ptr(), batch.pos0.data_ptr(), batch.prompt_seq.data_ptr(),
+                                      kq.data_ptr(), v.data_ptr(), gates.data_ptr(), o.data_ptr(), y[nd:].data_ptr(), y.stride(0),
+                                      geo.out_cols, n, batch.n_prompts, geo.taps, float(w.eps), dt, st), "tsb_delta_prefill")
+        _native.add_launches(3 if geo.taps > 1 else 2)
+    return y
+
+
+def _gated_delta_torch(proj, geo, w, conv_state, state, batch, y):
+    H, G, D, E, K = geo.heads, geo.kv_heads, geo.dim, geo.vdim, geo.taps
+    y.zero_()
+    for row0, n, slot, pos0 in batch.spans():
+        if slot < 0:
+            continue
+        p = proj[row0:row0 + n].float()
+        past = conv_state[slot].float() if pos0 > 0 else torch.zeros(K - 1, geo.conv_cols)
+        x = torch.cat([past, p[:, :geo.conv_cols]], dim=0)
+        c = torch.nn.functional.silu(sum(w.conv[j] * x[j:j + n] for j in range(K)))
+        conv_state[slot] = x[n:].to(conv_state.dtype)
+        q, k = (c[:, o:o + G * D].view(n, G, D) for o in (0, geo.off_k))
+        q = q / torch.sqrt((q * q).sum(-1, keepdim=True) + 1e-6) * D ** -0.5
+        k = k / torch.sqrt((k * k).sum(-1, keepdim=True) + 1e-6)
+        q, k = (t.repeat_interleave(H // G, dim=1) for t in (q, k))
+        v = c[:, geo.off_v:geo.off_v + H * E].view(n, H, E)
+        beta = torch.sigmoid(p[:, geo.off_b:geo.off_b + H])
+        a = torch.nn.functional.softplus(p[:, geo.off_a:geo.off_a + H] + w.dt_bias, threshold=1e9)
+        decay = torch.exp(-torch.exp(w.a_log) * a)
+        S = state[slot, :, :, :E].clone() if pos0 > 0 else torch.zeros(H, D, E)
+        o = torch.empty(n, H, E)
+        for t in range(n):
+            S = S * decay[t, :, None, None]
+            u = beta[t, :, None] * (v[t] - torch.einsum("hde,hd->he", S, k[t]))
+            S = S + k[t, :, :, None] * u[:, None, :]
+            o[t] = torch.einsum("hde,hd->he", S, q[t])
+        state[slot, :, :, :E] = S
+        gate = p[:, geo.off_gate:geo.off_gate + H * E].view(n, H, E)
+        o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + w.eps) * w.norm * torch.nn.functional.silu(gate)
+        y[row0:row0 + n, :H * E] = o.reshape(n, H * E).to(y.dtype)
+    return y

@@ -374,3 +374,85 @@ def cross_entropy(logits: torch.Tensor, targets: torch.Tensor) -> torch.Tensor:
     if _native_ok(logits):
         return _CrossEntropyFn.apply(logits.contiguous(), targets.contiguous())
     return cross_entropy_ref(logits, targets)
+
+
+# --------------------------------------------------------------------------------------- Dynamic Tanh, clamped GLU
+_P, _I, _L, _F = _native.P, _native.I, _native.L, _native.F
+_native.register_signatures({
+    "tsb_dyn_tanh_residual": [_P, _I, _I, _P, _L, _P, _F, _P, _P, _P, _P, _L, _F, _I, _I, _P, _F, _P, _P, _P, _L, _I, _I, _P],
+    "tsb_clamped_glu": [_P, _L, _P, _P, _L, _I, _I, _F, _F, _I, _P],
+})
+_EMBED_MODES = {None: 0, "set": 1, "add": 2}
+
+
+def _ptr(t):
+    return t.data_ptr() if t is not None else None
+
+
+def dyn_tanh_residual(x, y=None, y_bias=None, post=None, tokens=None, table=None, scale=1.0, embed=None, step=None,
+                      next_norm=None, out_cols=0, out_dtype=None):
+    """One step of an fp32 residual stream ``x`` [T, W] (updated in place) between two matrix products; norms are
+    (alpha, weight, bias) triples meaning tanh(alpha z) * weight + bias, all in fp32:
+
+        x  = table[tokens] * scale                 (embed="set")
+        x += post(y + y_bias)                      (y given)
+        x += table[tokens] * scale                 (embed="add")
+        x += step                                  (step given)
+        return next_norm(x)                        (next_norm given: [T, out_cols], zero past W, ``out_dtype``)
+    """
+    T, W = x.shape
+    h = None
+    if next_norm is not None:
+        h = torch.empty((T, out_cols or W), device=x.device, dtype=out_dtype or (y.dtype if y is not None else table.dtype))
+    if T == 0:
+        return h
+    if x.is_cuda:
+        act = next(t for t in (h, y, table) if t is not None)
+        for t in (y, table, h):
+            if t is not None and (t.dtype != act.dtype or t.stride(-1) != 1):
+                raise ValueError("dyn_tanh_residual: y, table and the result share one dtype and have contiguous rows")
+        pa, pw, pb = post if post is not None else (0.0, None, None)
+        na, nw, nb = next_norm if next_norm is not None else (0.0, None, None)
+        check(lib().tsb_dyn_tanh_residual(
+            x.data_ptr(), T, W, _ptr(y), y.stride(0) if y is not None else 0, _ptr(y_bias), float(pa), _ptr(pw), _ptr(pb),
+            _ptr(tokens), _ptr(table), table.stride(0) if table is not None else 0, float(scale), _EMBED_MODES[embed],
+            table.shape[0] if table is not None else 0, _ptr(step), float(na), _ptr(nw), _ptr(nb), _ptr(h),
+            h.stride(0) if h is not None else 0, h.shape[1] if h is not None else 0, dtype_code(act.dtype),
+            stream_ptr(x.device)), "tsb_dyn_tanh_residual")
+        return h
+    e = table[tokens.long(), :W].float() * scale if embed is not None else None
+    if embed == "set":
+        x.copy_(e)
+    if y is not None:
+        z = y[:, :W].float()
+        if y_bias is not None:
+            z = z + y_bias
+        x.add_(torch.tanh(post[0] * z) * post[1] + post[2])
+    if embed == "add":
+        x.add_(e)
+    if step is not None:
+        x.add_(step)
+    if h is not None:
+        h[:, W:] = 0
+        h[:, :W] = torch.tanh(next_norm[0] * x) * next_norm[1] + next_norm[2]
+    return h
+
+
+def clamped_glu(gate_up, bias, limit, slope=1.702):
+    """gate_up [T, 2 F] (gate, then up; ``bias`` fp32 [2 F] or None is added first) -> g sigmoid(slope g) (u + 1) with
+    g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    T, F2 = gate_up.shape
+    F = F2 // 2
+    out = torch.empty((T, F), device=gate_up.device, dtype=gate_up.dtype)
+    if T == 0:
+        return out
+    if gate_up.is_cuda:
+        check(lib().tsb_clamped_glu(gate_up.data_ptr(), gate_up.stride(0), _ptr(bias), out.data_ptr(), out.stride(0), T, F,
+                                    float(limit), float(slope), dtype_code(gate_up.dtype), stream_ptr(gate_up.device)),
+              "tsb_clamped_glu")
+        return out
+    z = gate_up.float()
+    if bias is not None:
+        z = z + bias
+    g, u = z[:, :F].clamp(max=limit), z[:, F:].clamp(-limit, limit)
+    return out.copy_(g * torch.sigmoid(slope * g) * (u + 1.0))

@@ -278,3 +278,22 @@ class _AccumLinearFn(torch.autograd.Function):
         ctx.wgrad_buf.add_((dy2.t() @ x2).to(ctx.wgrad_buf.dtype))
         db = dy2.sum(0) if ctx.has_bias else None
         return dx, None, db, None
+
+
+def project(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None, pdl: bool = True) -> torch.Tensor:
+    """x [M, K] @ w [N, K]^T for inference, whatever M is: decode-sized bf16 batches stream the weights
+    (``csrc/gemm_decode_wq.cu``), larger ones (and fp32 results) run on the persistent tcgen05 GEMM; fp32 tensors are
+    multiplied in true fp32. K is a multiple of 16."""
+    if _use_native(x):
+        if out_dtype in (None, torch.bfloat16) and x.shape[0] <= 256:
+            return stream_linear(x, w, pdl=pdl)
+        return gemm_bf16(x, w, out_dtype=out_dtype)
+    if x.is_cuda and torch.backends.cuda.matmul.allow_tf32:
+        torch.backends.cuda.matmul.allow_tf32 = False
+        try:
+            return (x @ w.t()).to(out_dtype or x.dtype)
+        finally:
+            torch.backends.cuda.matmul.allow_tf32 = True
+    if x.is_cuda:
+        return (x @ w.t()).to(out_dtype or x.dtype)
+    return (x.float() @ w.float().t()).to(out_dtype or x.dtype)

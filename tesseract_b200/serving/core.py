@@ -41,6 +41,10 @@ class _Req:
     t_submit: float = 0.0
     t_first: float = 0.0
     t_done: float = 0.0
+    # engines whose steps cut prompts: the sequence's share of the cache, tokens fed so far, host sampler
+    seq: object = None
+    fed: int = 0
+    sampler: object = None
 
 
 def argmax_rows(logits: torch.Tensor) -> torch.Tensor:
