@@ -49,9 +49,10 @@ class HybridEngine(EngineCore):
         seq.reset()
 
     @torch.no_grad()
-    def execute(self, entries: Sequence, want: Sequence) -> Optional[torch.Tensor]:
+    def execute(self, entries: Sequence, want: Sequence, keep: bool = True) -> Optional[torch.Tensor]:
         """entries: (sequence, token ids) with each sequence at most once; want[i]: places among entry i's tokens. Returns fp32
-        logits [wanted, vocab] on the device in the order of the entries and of their wanted places, or None."""
+        logits [wanted, vocab] on the device in the order of the entries and of their wanted places, or None. ``keep=False``
+        may return a buffer that the next step overwrites."""
         V = self.vocab_size
         for _, toks in entries:
             if any(t < 0 or t >= V for t in toks):
@@ -64,7 +65,9 @@ class HybridEngine(EngineCore):
             rows = [i for i, w in enumerate(want) for _ in w]
             if not rows:
                 return None
-            return logits[:len(entries)] if rows == list(range(len(entries))) else logits[rows]
+            if rows != list(range(len(entries))):
+                return logits[rows]
+            return logits[:len(entries)].clone() if keep else logits[:len(entries)]
         batch = self.model.make_batch(self.cache, entries, want)
         logits = self.model.forward_ragged(batch, self.cache)
         batch.commit()
@@ -195,7 +198,8 @@ class HybridEngine(EngineCore):
         ends = [r.fed + len(t) >= r.prompt_len for r, t in plan]
         with self._range(f"step[{len(plan)} requests, {new} tokens]"):
             before = sum(len(r.seq.blocks) for r, _ in plan)
-            logits = self.execute([(r.seq, t) for r, t in plan], [[len(t) - 1] if e else [] for (r, t), e in zip(plan, ends)])
+            logits = self.execute([(r.seq, t) for r, t in plan], [[len(t) - 1] if e else [] for (r, t), e in zip(plan, ends)],
+                                  keep=False)
             self._promised -= sum(len(r.seq.blocks) for r, _ in plan) - before
             for r, t in plan:
                 r.fed += len(t)

@@ -24,7 +24,10 @@ from tesseract_b200.serving import HybridEngine, make_engine
 DEVICES = ["cpu", pytest.param("cuda", marks=pytest.mark.gpu)]
 KINDS = [("cpu", "float32"), ("cpu", "bfloat16"), pytest.param(("cuda", "float32"), marks=pytest.mark.gpu),
          pytest.param(("cuda", "bfloat16"), marks=pytest.mark.gpu)]
-TOL = {torch.float32: 1e-4, torch.bfloat16: 0.05}
+# relative error of a row of logits: bf16 rounding alone reaches 0.04 in single rows of the deepest configuration and
+# 0.01 on average; a mechanism that is off by one token or factor shows as 0.3 and more
+TOL = {torch.float32: 1e-4, torch.bfloat16: 0.1}
+MEAN_TOL = {torch.float32: 5e-5, torch.bfloat16: 0.03}
 
 
 def attn(heads, kv, dim, vdim, scale, size, ff=None, limit=1.0):
@@ -108,6 +111,8 @@ def check(got, want, kind, what=""):
     e = row_error(got, want)
     tol = TOL[getattr(torch, kind[1])]
     assert float(e.max()) < tol, f"{what}: worst row {int(e.argmax())} of {len(e)}: {float(e.max()):.2e} (limit {tol})"
+    if len(e) >= 8:
+        assert float(e.mean()) < MEAN_TOL[getattr(torch, kind[1])], f"{what}: mean {float(e.mean()):.2e}"
 
 
 _reference = {}
