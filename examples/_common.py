@@ -36,7 +36,20 @@ def preset(name: str, dtype: torch.dtype, max_pos: int) -> LlamaConfig:
         cfg = LlamaConfig.llama_3_2_1b()
         cfg.dtype, cfg.max_position_embeddings = dtype, max_pos
         return cfg
-    raise SystemExit(f"error: unknown --model '{name}' (tiny | small | llama3.2-1b | llama3-8b)")
+    if name.startswith("fozelix-"):
+        from tesseract_b200.models import fozelix
+        try:
+            return fozelix.preset(name[len("fozelix-"):], dtype)
+        except ValueError as e:
+            raise SystemExit(f"error: --model: {e}") from None
+    raise SystemExit(f"error: unknown --model '{name}' (tiny | small | llama3.2-1b | llama3-8b | fozelix-tiny | fozelix-small)")
+
+
+def random_model(cfg, device, seed: int):
+    """A random-weight model of whatever family the configuration belongs to."""
+    from tesseract_b200.models import HybridConfig, HybridModel, LlamaModel
+    cls = HybridModel if isinstance(cfg, HybridConfig) else LlamaModel
+    return cls(cfg, device=device, init_std=0.02, seed=seed)
 
 
 class ByteTokenizer:

@@ -1,10 +1,11 @@
 #!/usr/bin/env python
-"""Text generation from a Hugging Face Llama directory or a random-weight preset (the reference's
-examples/llama_generate.cpp, same flags).
+"""Text generation from a model directory (config.json + model.safetensors; the model registry picks the family: Hugging
+Face Llama, Fozelix) or a random-weight preset (the reference's examples/llama_generate.cpp, same flags).
 
     python examples/llama_generate.py --model-dir /path/to/Llama-3.2-1B --prompt "Hello" --max-new-tokens 64
     python examples/llama_generate.py --config c.json --safetensors m.safetensors --tokenizer tokenizer.json --prompt hi
     python examples/llama_generate.py --model small --prompt abc --sample --top-p 0.9 --temperature 0.8 --kv-int8
+    python examples/llama_generate.py --model fozelix-small --device cuda --prompt abc
     python examples/llama_generate.py --model small --prompt 12 --grammar-regex "[0-9]+"
 """
 from __future__ import annotations
@@ -13,7 +14,7 @@ import argparse
 import os
 import sys
 
-from _common import load_tokenizer, pick_device, preset, torch
+from _common import load_tokenizer, pick_device, preset, random_model, torch
 
 
 def main() -> int:
@@ -22,7 +23,7 @@ def main() -> int:
     ap.add_argument("--config", default="")
     ap.add_argument("--safetensors", default="")
     ap.add_argument("--tokenizer", default="")
-    ap.add_argument("--model", default="", help="random-weight preset instead of files: tiny | small | llama3-8b")
+    ap.add_argument("--model", default="", help="random-weight preset instead of files: tiny | small | llama3-8b | fozelix-tiny | fozelix-small")
     ap.add_argument("--prompt", default="Hello")
     ap.add_argument("--device", default="cpu")
     ap.add_argument("--max-new-tokens", type=int, default=32)
@@ -38,21 +39,21 @@ def main() -> int:
     ap.add_argument("--no-stream", action="store_true")
     a = ap.parse_args()
 
-    from tesseract_b200.models import GenerateConfig, LlamaConfig, LlamaModel
+    from tesseract_b200.models import GenerateConfig, load_model
     from tesseract_b200.models.sampler import SamplingParams
     dev = pick_device(a.device)
     dtype = torch.bfloat16 if dev.type == "cuda" else torch.float32
     if a.model_dir:
         a.config = a.config or os.path.join(a.model_dir, "config.json")
         a.safetensors = a.safetensors or os.path.join(a.model_dir, "model.safetensors")
-        a.tokenizer = a.tokenizer or os.path.join(a.model_dir, "tokenizer.json")
+        tok_file = os.path.join(a.model_dir, "tokenizer.json")
+        a.tokenizer = a.tokenizer or (tok_file if os.path.exists(tok_file) else "")
     if a.config and a.safetensors:
-        cfg = LlamaConfig.from_json(open(a.config).read())
-        cfg.dtype = dtype
-        model = LlamaModel.from_pretrained(a.safetensors, cfg, device=dev)
+        model = load_model(a.config, a.safetensors, dtype, dev)
+        cfg = model.config
     elif a.model:
         cfg = preset(a.model, dtype, 2048)
-        model = LlamaModel(cfg, device=dev, init_std=0.02, seed=a.seed)
+        model = random_model(cfg, dev, a.seed)
     else:
         print("error: pass --model-dir, or --config with --safetensors, or a --model preset. See --help.", file=sys.stderr)
         return 1

@@ -5,6 +5,7 @@ examples/llama_infer.cpp:118-298, same flags).
 
     python examples/llama_infer.py --synthetic --vocab 512 --hidden 64 --layers 2 --heads 4 --kv-heads 2 --ff 128
     python examples/llama_infer.py --synthetic --prompt "hello" --generate --max-new-tokens 8 --sample --top-k 20
+    python examples/llama_infer.py --model-dir DIR --batch 2 --seq 16       # config.json picks the family
     python examples/llama_infer.py --safetensors m.safetensors --tokenizer tokenizer.json --prompt "Hi" --generate
 """
 from __future__ import annotations
@@ -19,6 +20,7 @@ def main(argv=None) -> int:
     ap.add_argument("--device", default="cpu")
     ap.add_argument("--synthetic", action="store_true")
     ap.add_argument("--safetensors", default="")
+    ap.add_argument("--model-dir", default="", help="folder with config.json and model.safetensors")
     ap.add_argument("--tokenizer", default="")
     ap.add_argument("--prompt", default="")
     ap.add_argument("--generate", action="store_true")
@@ -42,27 +44,33 @@ def main(argv=None) -> int:
     ap.add_argument("--seq", type=int, default=8)
     ap.add_argument("--topk", type=int, default=5)
     a = ap.parse_args(argv)
-    if not a.synthetic and not a.safetensors:
-        raise SystemExit("error: pass --synthetic or --safetensors PATH. See --help.")
+    if not a.synthetic and not a.safetensors and not a.model_dir:
+        raise SystemExit("error: pass --synthetic, --safetensors PATH or --model-dir DIR. See --help.")
 
-    from tesseract_b200.models import GenerateConfig, LlamaConfig, LlamaModel
+    from tesseract_b200.models import GenerateConfig, LlamaConfig, LlamaModel, load_pretrained
     from tesseract_b200.models.sampler import SamplingParams
     dev = pick_device(a.device)
     dtype = torch.bfloat16 if dev.type == "cuda" else torch.float32
-    cfg = LlamaConfig(vocab_size=a.vocab, hidden_size=a.hidden, num_hidden_layers=a.layers,
-                      num_attention_heads=a.heads, num_key_value_heads=a.kv_heads, intermediate_size=a.ff,
-                      max_position_embeddings=a.max_seq, rope_theta=a.rope_theta,
-                      tie_word_embeddings=(a.tie != "false"), dtype=dtype)
-    print(f"[llama_infer] config:\n  vocab={cfg.vocab_size} hidden={cfg.hidden_size} layers={cfg.num_hidden_layers} "
-          f"heads={cfg.num_attention_heads} kv_heads={cfg.num_key_value_heads} ff={cfg.intermediate_size} "
-          f"max_seq={cfg.max_position_embeddings} tie={cfg.tie_word_embeddings} device={dev} dtype={dtype}")
-    if a.synthetic:
-        print("[llama_infer] using synthetic (random-init) weights")
-        model = LlamaModel(cfg, device=dev, init_std=0.02, seed=a.seed)
-    else:
-        print(f"[llama_infer] loading {a.safetensors}")
-        model = LlamaModel.from_pretrained(a.safetensors, cfg, device=dev)
+    if a.model_dir:
+        print(f"[llama_infer] loading {a.model_dir}")
+        model = load_pretrained(a.model_dir, dtype, dev)
+        cfg = model.config
         print(f"[llama_infer] loaded {sum(p.numel() for p in model.parameters())} parameters")
+    else:
+        cfg = LlamaConfig(vocab_size=a.vocab, hidden_size=a.hidden, num_hidden_layers=a.layers,
+                          num_attention_heads=a.heads, num_key_value_heads=a.kv_heads, intermediate_size=a.ff,
+                          max_position_embeddings=a.max_seq, rope_theta=a.rope_theta,
+                          tie_word_embeddings=(a.tie != "false"), dtype=dtype)
+        print(f"[llama_infer] config:\n  vocab={cfg.vocab_size} hidden={cfg.hidden_size} layers={cfg.num_hidden_layers} "
+              f"heads={cfg.num_attention_heads} kv_heads={cfg.num_key_value_heads} ff={cfg.intermediate_size} "
+              f"max_seq={cfg.max_position_embeddings} tie={cfg.tie_word_embeddings} device={dev} dtype={dtype}")
+        if a.synthetic:
+            print("[llama_infer] using synthetic (random-init) weights")
+            model = LlamaModel(cfg, device=dev, init_std=0.02, seed=a.seed)
+        else:
+            print(f"[llama_infer] loading {a.safetensors}")
+            model = LlamaModel.from_pretrained(a.safetensors, cfg, device=dev)
+            print(f"[llama_infer] loaded {sum(p.numel() for p in model.parameters())} parameters")
     model.eval()
     tok = load_tokenizer(a.tokenizer)
 

@@ -4,6 +4,7 @@ are queued on one engine, decoded together step by step over a paged KV cache, a
 
     python examples/llama_serve.py --synthetic --prompts "alpha|beta|gamma" --max-new-tokens 16 --max-batch 4
     python examples/llama_serve.py --device cuda --model small --sample --temperature 0.8 --seed 7
+    python examples/llama_serve.py --device cuda --model-dir DIR        # config.json + model.safetensors, any registered family
 """
 from __future__ import annotations
 
@@ -11,7 +12,7 @@ import argparse
 import sys
 import time
 
-from _common import load_tokenizer, pick_device, preset, torch
+from _common import load_tokenizer, pick_device, preset, random_model, torch
 
 
 def main() -> int:
@@ -26,25 +27,30 @@ def main() -> int:
     ap.add_argument("--seed", type=int, default=0)
     ap.add_argument("--synthetic", action="store_true", help="random weights (the default, as in the reference)")
     ap.add_argument("--model", default="small")
+    ap.add_argument("--model-dir", default="", help="serve this model instead of a random-weight preset")
     ap.add_argument("--kv-int8", action="store_true")
     ap.add_argument("--engine", default="auto", help="auto | scheduler (reference semantics) | batched (device-resident engine)")
     a = ap.parse_args()
 
-    from tesseract_b200.models import GenerateConfig, LlamaModel
+    from tesseract_b200.models import GenerateConfig, load_pretrained
     from tesseract_b200.models.sampler import SamplingParams
     from tesseract_b200.models.scheduler import ContinuousBatchingScheduler, EngineConfig
     dev = pick_device(a.device)
     dtype = torch.bfloat16 if dev.type == "cuda" else torch.float32
-    cfg = preset(a.model, dtype, 2048)
-    model = LlamaModel(cfg, device=dev, init_std=0.02, seed=a.seed)
+    if a.model_dir:
+        model = load_pretrained(a.model_dir, dtype, dev)
+        cfg = model.config
+    else:
+        cfg = preset(a.model, dtype, 2048)
+        model = random_model(cfg, dev, a.seed)
     model.eval()
     tok = load_tokenizer(a.tokenizer)
     ecfg = EngineConfig(block_size=16, num_blocks=1024, max_seq_len=2048, max_batch_size=a.max_batch, kv_int8=a.kv_int8)
     use_batched = a.engine == "batched" or (a.engine == "auto" and dev.type == "cuda")
     if use_batched:
-        from tesseract_b200.serving.engine import ServingEngine
+        from tesseract_b200.serving import make_engine
         from tesseract_b200.parallel.launch import job_metrics
-        engine = ServingEngine(model, ecfg).instrument(metrics=job_metrics())    # TESSERACT_METRICS_FILE / TESSERACT_NVTX
+        engine = make_engine(model, ecfg).instrument(metrics=job_metrics())    # TESSERACT_METRICS_FILE / TESSERACT_NVTX
     else:
         engine = ContinuousBatchingScheduler(model, ecfg)
     prompts = [p for p in a.prompts.split("|") if p]

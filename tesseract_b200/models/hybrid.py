@@ -313,6 +313,15 @@ class HybridModel:
         batch.commit()
         return logits.view(A, S, -1)
 
+    def forward(self, tokens: torch.Tensor) -> torch.Tensor:
+        """Logits [B, S, V] of B whole sequences, run as one ragged batch."""
+        B, S = tokens.shape
+        bs = 16
+        cache = self.make_cache(B * ((S + bs - 1) // bs), bs, B, S)
+        return self.forward_step_batched(tokens, [[HybridSequence(cache)] for _ in range(B)])
+
+    __call__ = forward
+
     def generate(self, prompt_ids, cfg: Optional[GenerateConfig] = None) -> list:
         """Prompt + generated ids, through the serving engine with one request."""
         from ..models.scheduler import EngineConfig
