@@ -406,11 +406,94 @@ def case_ag_gemm_emul(b: Bench):
            note="multiply half of rank 0 of 2 after both ranks' push halves; push_ms = one rank's push half alone")
 
 
+# ---- hybrid decoders: 4096-wide layers, 16 key / 32 value heads of 128 x 128 (delta), 32 / 8 heads of 128 (attention)
+class _Step:
+    """A ragged batch of ``n`` sequences bringing ``rows`` tokens each, after ``past`` tokens."""
+
+    def __init__(self, b, run, n, rows, past=0, chunks=(), block=16):
+        from tesseract_b200.nn.ragged import HybridCache, HybridSequence, RaggedBatch
+        blocks = n * ((past + rows + block - 1) // block)
+        self.cache = HybridCache([run], blocks, block, n, past + rows + block, torch.bfloat16, b.dev)
+        seqs = [HybridSequence(self.cache) for _ in range(n)]
+        for s in seqs:
+            if past:
+                s.reserve(past)
+                s.advance(past)
+        self.batch = RaggedBatch(self.cache, [(s, [0] * rows) for s in seqs], None, chunks)
+
+
+def _delta_case(b, n, rows, past):
+    from tesseract_b200.nn.ragged import StateRun
+    from tesseract_b200.ops.delta import DeltaGeometry, DeltaWeights, gated_delta
+    g = DeltaGeometry(16, 32, 128, 128, 4)
+    st = _Step(b, StateRun((g.heads, g.dim, g.vdim_pad), (g.taps - 1, g.conv_cols)), n, rows, past)
+    proj = b.randn(n * rows, g.cols)
+    f = lambda *sh: torch.randn(*sh, device=b.dev, generator=b.gen)   # noqa: E731
+    w = DeltaWeights(f(g.taps, g.conv_cols), f(g.heads), f(g.heads), f(g.vdim), 1e-5)
+    ms = b.time(lambda: gated_delta(proj, g, w, *st.cache.runs[0], st.batch))
+    return g, ms
+
+
+def case_delta_prefill(b: Bench):
+    """All four launches; bound by the fp32 multiply-adds of the recurrence (8 flops per state element and token)."""
+    for n, rows in ((4, 4096), (1, 4096), (32, 512)):
+        g, ms = _delta_case(b, n, rows, 0)
+        fl = 8.0 * g.heads * g.dim * g.vdim * n * rows
+        peak = 148 * 128 * 2 * 1.965e9 / 1e12
+        print(json.dumps({"case": "delta_prefill", "ms": round(ms, 4), "fp32_tflops": round(fl / ms / 1e9, 2),
+                          "frac_of_nominal_fp32": round(fl / ms / 1e9 / peak, 3), "ns_per_token": round(ms * 1e6 / (n * rows), 1),
+                          "shape": [n, rows]}))
+
+
+def case_delta_step(b: Bench):
+    for n in (256, 32):
+        g, ms = _delta_case(b, n, 1, 7)
+        report("delta_step", ms, bytes_=n * (2.0 * g.heads * g.dim * g.vdim * 4 + 2 * (2 * g.taps - 1) * g.conv_cols), shape=[n])
+
+
+def _chunk_attn(b, n, rows, past, chunk):
+    from tesseract_b200 import ops
+    from tesseract_b200.nn.ragged import PagedRun
+    H, G, D = 32, 8, 128
+    st = _Step(b, PagedRun(G, D), n, rows, past, (chunk,))
+    qkv, bias = b.randn(n * rows, (H + 2 * G) * D), torch.zeros((H + 2 * G) * D, device=b.dev)
+    return b.time(lambda: ops.ragged_attention(qkv, bias, *st.cache.runs[0], st.batch, H, G, D ** -0.5, chunk))
+
+
+def case_chunk_attn(b: Bench):
+    """Append + attention. Prompts: two sequences of 4096 in chunks of 4096 (the flash_fwd case) and of 1024; decode: 256
+    sequences at 1400 tokens of one chunk (the decode case)."""
+    for chunk in (4096, 1024):
+        ms = _chunk_attn(b, 2, 4096, 0, chunk)
+        report("chunk_attn_prefill", ms, flops=2 * 4096 * chunk * 32 * 128 * 2.0, shape=[2, 4096, chunk])
+    ms = _chunk_attn(b, 256, 1, 1399, 4096)
+    report("chunk_attn_decode", ms, bytes_=256 * 1400 * 8 * 128 * 2 * 2, shape=[256, 1400])
+
+
+def case_dyn_tanh(b: Bench):
+    from tesseract_b200 import ops
+    T, W = 16384, 4096
+    x, y = torch.randn(T, W, device=b.dev, generator=b.gen), b.randn(T, W)
+    v = lambda: torch.randn(W, device=b.dev, generator=b.gen)   # noqa: E731
+    post, nxt = (0.5, v(), v()), (0.5, v() * 0.01, v() * 0.01)
+    ms = b.time(lambda: ops.dyn_tanh_residual(x, y, None, post, next_norm=nxt))
+    report("dyn_tanh_residual", ms, bytes_=T * W * 12, shape=[T, W])
+
+
+def case_clamped_glu(b: Bench):
+    from tesseract_b200 import ops
+    x, bias = b.randn(16384, 2 * 14336), torch.zeros(2 * 14336, device=b.dev)
+    ms = b.time(lambda: ops.clamped_glu(x, bias, 7.0))
+    report("clamped_glu", ms, bytes_=x.numel() * 2 * 1.5, shape=list(x.shape))
+
+
 CASES = {"gemm": case_gemm, "gemm_fp8": case_gemm_fp8, "gemm_fp8_pertensor": case_gemm_fp8_pertensor, "decode_gemm": case_decode_gemm, "gemm_wgrad": case_gemm_wgrad, "grouped_gemm": case_grouped_gemm,
          "flash_fwd": case_flash_fwd, "flash_bwd": case_flash_bwd, "decode": case_decode,
          "decode_int8": case_decode_int8, "rmsnorm": case_rmsnorm, "swiglu": case_swiglu, "swiglu_bwd": case_swiglu_bwd, "adam": case_adam,
          "ce_stats": case_ce, "selective_scan": case_scan, "gemv_w8": case_gemv, "gemm_rs_emul": case_gemm_rs_emul,
-         "ag_gemm_emul": case_ag_gemm_emul, "stream_linear": case_stream_linear, "mx_linear": case_mx_linear, "gemm_mx": case_gemm_mx}
+         "ag_gemm_emul": case_ag_gemm_emul, "stream_linear": case_stream_linear, "mx_linear": case_mx_linear, "gemm_mx": case_gemm_mx,
+         "delta_prefill": case_delta_prefill, "delta_step": case_delta_step, "chunk_attn": case_chunk_attn,
+         "dyn_tanh": case_dyn_tanh, "clamped_glu": case_clamped_glu}
 
 
 def main():

@@ -12,10 +12,12 @@
 // streaming the state through registers once.
 //
 // The columns of S do not talk to each other, so the recurrence is split over value columns. In the scan eight lanes
-// share a column (each holds dim / 8 rows of it in registers) and a warp walks 4 * CT columns. Both products with
-// the OLD state are formed in one sweep, since S_new^T q = g (S_old^T q) + (k . q) u; that leaves two fused
-// multiply-adds per element for the products and two instructions for the update, issued on register pairs
-// (fma.rn.f32x2). Everything of the recurrence is fp32; nothing here uses the tensor cores.
+// share a column (each holds dim / 8 rows of it in registers), and four tokens are taken at once: the products of the
+// state with their k and q are formed from the state before the block, the tokens' influence on one another is a 4 x 4
+// triangle of scalars that the prepare kernel has computed, and the state is updated once. That is 3.25 multiply-adds
+// per element and token instead of 4, and one reduction latency per four tokens; they are issued on register pairs
+// (fma.rn.f32x2). The one-token kernel uses the same identity: S_new^T q = g (S_old^T q) + (k . q) u, so the state is
+// read once. Everything of the recurrence is fp32; nothing here uses the tensor cores.
 //
 // Packed projection row (element offsets, sections padded to multiples of 8):
 //   [ q: Hk * dim | k: Hk * dim | v: H * vdim | gate: H * vdim | b: H | a: H ]
@@ -23,6 +25,8 @@
 #include "common.cuh"
 
 #include <algorithm>
+#include <cstdlib>
+#include <type_traits>
 
 namespace tsb {
 namespace {
@@ -35,9 +39,57 @@ struct DeltaGeom {
   long long ldp;             // projection row stride
 };
 
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+constexpr int kBlk = 4;          // tokens the recurrence takes at once
+constexpr int kCoef = 36;        // coefficients per (block, value head), see delta_prepare_kernel
+
+template <bool FAST = false>
+__device__ __forceinline__ float silu_f(float x) {
+  if constexpr (FAST) return __fdividef(x, 1.f + __expf(-x));
+  return x / (1.f + expf(-x));
+}
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+
+// N consecutive channels starting at p, of which `valid` exist; vector loads when the caller knows p to be aligned.
+template <typename T, int N>
+__device__ __forceinline__ void load_ch(const T* p, int valid, bool vec, float (&f)[N]) {
+  if (vec && valid >= N) {
+    constexpr int kBytes = N * sizeof(T);
+    if constexpr (kBytes == 2) {
+      f[0] = to_f32<T>(p[0]);
+    } else if constexpr (kBytes == 4) {
+      const uint32_t r = *reinterpret_cast<const uint32_t*>(p);
+#pragma unroll
+      for (int i = 0; i < N; ++i) f[i] = to_f32<T>(reinterpret_cast<const T*>(&r)[i]);
+    } else if constexpr (kBytes == 8) {
+      const uint2 r = *reinterpret_cast<const uint2*>(p);
+#pragma unroll
+      for (int i = 0; i < N; ++i) f[i] = to_f32<T>(reinterpret_cast<const T*>(&r)[i]);
+    } else {
+#pragma unroll
+      for (int v = 0; v < kBytes / 16; ++v) {
+        const uint4 r = reinterpret_cast<const uint4*>(p)[v];
+        constexpr int kPer = 16 / sizeof(T);
+#pragma unroll
+        for (int i = 0; i < kPer; ++i) f[v * kPer + i] = to_f32<T>(reinterpret_cast<const T*>(&r)[i]);
+      }
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) f[i] = i < valid ? to_f32<T>(p[i]) : 0.f;
+  }
+}
+template <int N>
+__device__ __forceinline__ void store_f32(float* p, int valid, bool vec, const float (&f)[N]) {
+  if (vec && valid >= N && N % 4 == 0) {
+#pragma unroll
+    for (int v = 0; v < N / 4; ++v) reinterpret_cast<float4*>(p)[v] = make_float4(f[4 * v], f[4 * v + 1], f[4 * v + 2], f[4 * v + 3]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      if (i < valid) p[i] = f[i];
+  }
+}
 
 // ------------------------------------------------------------------ prompt rows: convolution, unit vectors, gates
 struct DeltaPrepParams {
@@ -50,92 +102,179 @@ struct DeltaPrepParams {
   const int* cu;             // [nseq + 1] row offsets of the sequences
   const int* slots;          // [nseq]
   const int* pos0;           // [nseq] position of the first row (0: the sequence starts here)
-  const int* seq_of;         // [rows]
+  const int* blk_seq;        // [blocks] sequence of a block of kBlk tokens
+  const int* blk0;           // [nseq + 1] first block of a sequence
   float* kq;                 // [rows, Hk, 2, dkp]: k, then q
   float* v;                  // [rows, H, vp]
-  float4* gates;             // [rows, H]: (g, beta, k . q, 0)
-  int rows;
+  float* coef;               // [blocks, H, kCoef]
+  int blocks;
 };
 
-template <typename T, int TAPS>
-__device__ __forceinline__ float conv_at(const DeltaPrepParams& p, const T* proj, int row, int row0, long long state_row,
-                                         bool has_state, int c) {
-  float acc = 0.f;
+// N consecutive channels as stored, in registers.
+template <typename T, int N>
+struct alignas(N * sizeof(T) >= 16 ? 16 : N * sizeof(T)) Packed {
+  T v[N];
+};
+
+// Convolution and SiLU of N channels of a block's tokens. Every input row is requested before the first is used; rows
+// past the end of the portion repeat its last one (their results are dropped).
+template <typename T, int TAPS, int N>
+__device__ __forceinline__ void conv_block(const DeltaPrepParams& p, int row0, int first, int cnt, long long state_row,
+                                           bool has_state, int c, int valid, bool vec, float (&y)[kBlk][N]) {
+  constexpr int R = TAPS - 1 + kBlk;
+  Packed<T, N> x[R];
+  const bool whole = vec && valid >= N;
 #pragma unroll
-  for (int j = 0; j < TAPS; ++j) {
-    const int r = row - (TAPS - 1) + j;
-    float x = 0.f;
-    if (r >= row0) x = to_f32<T>(proj[static_cast<long long>(r) * p.g.ldp + c]);
-    else if (has_state)
-      x = to_f32<T>(static_cast<const T*>(p.conv_state)[(state_row + (TAPS - 1) + r - row0) * p.g.conv_c + c]);
-    acc = fmaf(p.conv_w[static_cast<long long>(j) * p.g.conv_c + c], x, acc);
+  for (int r = 0; r < R; ++r) {
+    const int t = min(first + r - (TAPS - 1), first + cnt - 1);      // token of this portion, negative: before it
+    const T* src = t >= 0 ? static_cast<const T*>(p.proj) + static_cast<long long>(row0 + t) * p.g.ldp + c
+                          : static_cast<const T*>(p.conv_state) + (state_row + (TAPS - 1) + t) * p.g.conv_c + c;
+    const bool there = t >= 0 || has_state;
+#pragma unroll
+    for (int i = 0; i < N; ++i) x[r].v[i] = from_f32<T>(0.f);
+    if (whole) {
+      if (there) x[r] = *reinterpret_cast<const Packed<T, N>*>(src);
+    } else {
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+        if (there && i < valid) x[r].v[i] = src[i];
+    }
   }
-  return silu_f(acc);
+  float w[TAPS][N];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j)
+    load_ch<float, N>(p.conv_w + static_cast<long long>(j) * p.g.conv_c + c, valid, vec, w[j]);
+#pragma unroll
+  for (int t = 0; t < kBlk; ++t)
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j][i], to_f32<T>(x[t + j].v[i]), acc);
+      y[t][i] = t < cnt ? silu_f<sizeof(T) == 2>(acc) : 0.f;
+    }
 }
 
-// One warp per (row, unit). Units: the Hk key heads (q and k of the head together with its heads' gates), then blocks
-// of 128 value channels.
-template <typename T, int TAPS>
-__global__ void __launch_bounds__(256)
+// One warp per (block of kBlk tokens, unit). Units: the Hk key heads (q and k of the head, and the coefficients of its
+// value heads), then blocks of 256 value channels. EPL = dkp / 32 channels of a key head per lane.
+//
+// Taking tokens 0 .. 3 of a block at once, with d_j = S^T k_j and e_j = S^T q_j formed from the state before the block:
+//   u_j = beta_j (v_j - G_j d_j - sum_{i < j} A_ji u_i),  o_j = G_j e_j + sum_{i <= j} W_ji u_i,
+//   S <- G_3 S + sum_j c_j k_j u_j^T,
+//   G_j = g_0 .. g_j,  c_j = g_{j+1} .. g_3,  A_ji = (g_{i+1} .. g_j)(k_i . k_j),  W_ji = (g_{i+1} .. g_j)(k_i . q_j).
+// Coefficients as stored: G (4), beta (4), A (10, 20, 21, 30, 31, 32, 0, 0), c (4), W (4 rows of 4, zero above the
+// diagonal). Tokens past the end of the portion get g = 1, beta = 0, k = q = 0: they change nothing.
+template <typename T, int TAPS, int EPL>
+__global__ void __launch_bounds__(128, TAPS <= 4 && EPL <= 4 ? 5 : 1)
 delta_prepare_kernel(DeltaPrepParams p) {
   pdl_trigger();
   pdl_grid_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int row = blockIdx.y * 8 + warp;
-  if (row >= p.rows) return;
+  const int blk = blockIdx.y * 4 + warp;
+  if (blk >= p.blocks) return;
   const DeltaGeom& g = p.g;
-  const int seq = p.seq_of[row];
-  const int row0 = p.cu[seq];
+  const int seq = p.blk_seq[blk];
+  const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
+  const int first = (blk - p.blk0[seq]) * kBlk;
+  const int cnt = min(kBlk, n - first);
   const bool has_state = p.pos0[seq] > 0;
   const long long state_row = static_cast<long long>(p.slots[seq]) * (TAPS - 1);
-  const T* proj = static_cast<const T*>(p.proj);
   const int unit = blockIdx.x;
   if (unit < g.Hk) {
-    constexpr int kMax = 8;                 // dim <= 256
-    float qv[kMax], kv[kMax];
-    float sqq = 0.f, skk = 0.f, sqk = 0.f;
+    const int d0 = lane * EPL;
+    const int valid = min(EPL, g.dim - d0);
+    const bool vec = g.dim % EPL == 0;
+    float qv[kBlk][EPL], kv[kBlk][EPL];
+    conv_block<T, TAPS, EPL>(p, row0, first, cnt, state_row, has_state, unit * g.dim + d0, valid, vec, qv);
+    conv_block<T, TAPS, EPL>(p, row0, first, cnt, state_row, has_state, g.off_k + unit * g.dim + d0, valid, vec, kv);
+    const float rsqrt_dim = rsqrtf(static_cast<float>(g.dim));
+    float* out = p.kq + (static_cast<long long>(row0 + first) * g.Hk + unit) * 2 * g.dkp + d0;
 #pragma unroll
-    for (int i = 0; i < kMax; ++i) {
-      const int d = lane + 32 * i;
-      qv[i] = kv[i] = 0.f;
-      if (d < g.dim) {
-        qv[i] = conv_at<T, TAPS>(p, proj, row, row0, state_row, has_state, unit * g.dim + d);
-        kv[i] = conv_at<T, TAPS>(p, proj, row, row0, state_row, has_state, g.off_k + unit * g.dim + d);
-      }
-      sqq = fmaf(qv[i], qv[i], sqq);
-      skk = fmaf(kv[i], kv[i], skk);
-      sqk = fmaf(qv[i], kv[i], sqk);
-    }
-    sqq = warp_sum(sqq);
-    skk = warp_sum(skk);
-    sqk = warp_sum(sqk);
-    const float rq = 1.f / (sqrtf(sqq + 1e-6f) * sqrtf(static_cast<float>(g.dim)));
-    const float rk = 1.f / sqrtf(skk + 1e-6f);
-    float* out = p.kq + (static_cast<long long>(row) * g.Hk + unit) * 2 * g.dkp;
+    for (int t = 0; t < kBlk; ++t) {
+      float sq = 0.f, sk = 0.f;
 #pragma unroll
-    for (int i = 0; i < kMax; ++i) {
-      const int d = lane + 32 * i;
-      if (d < g.dkp) {
-        out[d] = kv[i] * rk;
-        out[g.dkp + d] = qv[i] * rq;
+      for (int i = 0; i < EPL; ++i) {
+        sq = fmaf(qv[t][i], qv[t][i], sq);
+        sk = fmaf(kv[t][i], kv[t][i], sk);
+      }
+      const float rq = rsqrtf(warp_sum(sq) + 1e-6f) * rsqrt_dim;
+      const float rk = rsqrtf(warp_sum(sk) + 1e-6f);
+#pragma unroll
+      for (int i = 0; i < EPL; ++i) {
+        qv[t][i] *= rq;
+        kv[t][i] *= rk;
+      }
+      if (t < cnt) {
+        float* o = out + static_cast<long long>(t) * g.Hk * 2 * g.dkp;
+        store_f32<EPL>(o, EPL, true, kv[t]);
+        store_f32<EPL>(o + g.dkp, EPL, true, qv[t]);
       }
     }
+    float kk[kBlk][kBlk], kqd[kBlk][kBlk];          // [j][i]: k_i . k_j (i < j) and k_i . q_j (i <= j)
+#pragma unroll
+    for (int j = 0; j < kBlk; ++j)
+#pragma unroll
+      for (int i = 0; i < kBlk; ++i) {
+        kk[j][i] = kqd[j][i] = 0.f;
+        if (i <= j) {
+          float a = 0.f, b = 0.f;
+#pragma unroll
+          for (int e = 0; e < EPL; ++e) {
+            a = fmaf(kv[i][e], kv[j][e], a);
+            b = fmaf(kv[i][e], qv[j][e], b);
+          }
+          if (i < j) kk[j][i] = warp_sum(a);
+          kqd[j][i] = warp_sum(b);
+        }
+      }
     const int per = g.H / g.Hk;
-    for (int i = lane; i < per; i += 32) {
-      const int h = unit * per + i;
-      const float b = to_f32<T>(proj[static_cast<long long>(row) * g.ldp + g.off_b + h]);
-      const float a = to_f32<T>(proj[static_cast<long long>(row) * g.ldp + g.off_a + h]);
-      const float decay = expf(-expf(p.a_log[h]) * softplus_f(a + p.dt_bias[h]));
-      p.gates[static_cast<long long>(row) * g.H + h] = make_float4(decay, sigmoid_f(b), sqk * rq * rk, 0.f);
+    const T* proj = static_cast<const T*>(p.proj);
+    // eight heads at a time: lane = token * 8 + head works out one pair of gates, then lanes 0 .. 7 collect their head's
+    for (int h0 = 0; h0 < per; h0 += 8) {
+      const int hh = h0 + (lane & 7), tok = lane >> 3;
+      const int h = unit * per + min(hh, per - 1);
+      float gate = 1.f, beta = 0.f;
+      if (tok < cnt) {
+        const T* pr = proj + static_cast<long long>(row0 + first + tok) * g.ldp;
+        gate = expf(-expf(p.a_log[h]) * softplus_f(to_f32<T>(pr[g.off_a + h]) + p.dt_bias[h]));
+        beta = sigmoid_f(to_f32<T>(pr[g.off_b + h]));
+      }
+      float gd[kBlk], be[kBlk];
+#pragma unroll
+      for (int t = 0; t < kBlk; ++t) {
+        gd[t] = __shfl_sync(0xffffffffu, gate, t * 8 + (lane & 7));
+        be[t] = __shfl_sync(0xffffffffu, beta, t * 8 + (lane & 7));
+      }
+      if (lane >= 8 || hh >= per) continue;
+      float4* o = reinterpret_cast<float4*>(p.coef + (static_cast<long long>(blk) * g.H + h) * kCoef);
+      const float g10 = gd[1], g21 = gd[2], g32 = gd[3], g20 = g10 * g21, g31 = g21 * g32, g30 = g20 * g32;
+      o[0] = make_float4(gd[0], gd[0] * g10, gd[0] * g20, gd[0] * g30);
+      o[1] = make_float4(be[0], be[1], be[2], be[3]);
+      o[2] = make_float4(g10 * kk[1][0], g20 * kk[2][0], g21 * kk[2][1], g30 * kk[3][0]);
+      o[3] = make_float4(g31 * kk[3][1], g32 * kk[3][2], 0.f, 0.f);
+      o[4] = make_float4(g30, g31, g32, 1.f);
+      o[5] = make_float4(kqd[0][0], 0.f, 0.f, 0.f);
+      o[6] = make_float4(g10 * kqd[1][0], kqd[1][1], 0.f, 0.f);
+      o[7] = make_float4(g20 * kqd[2][0], g21 * kqd[2][1], kqd[2][2], 0.f);
+      o[8] = make_float4(g30 * kqd[3][0], g31 * kqd[3][1], g32 * kqd[3][2], kqd[3][3]);
     }
   } else {
-    const int c0 = (unit - g.Hk) * 128;
+    const int c = (unit - g.Hk) * 256 + lane * 8, total = g.H * g.vdim;
+    if (c >= total) return;
+    const int valid = min(8, total - c);
+    float y[kBlk][8];
+    conv_block<T, TAPS, 8>(p, row0, first, cnt, state_row, has_state, g.off_v + c, valid, true, y);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int c = c0 + lane + 32 * i;
-      if (c < g.H * g.vdim)
-        p.v[(static_cast<long long>(row) * g.H + c / g.vdim) * g.vp + c % g.vdim] =
-            conv_at<T, TAPS>(p, proj, row, row0, state_row, has_state, g.off_v + c);
+    for (int t = 0; t < kBlk; ++t) {
+      if (t >= cnt) break;
+      float* vr = p.v + static_cast<long long>(row0 + first + t) * g.H * g.vp;
+      if (g.vp == g.vdim) {
+        store_f32<8>(vr + c, valid, true, y[t]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          if (i < valid) vr[static_cast<long long>((c + i) / g.vdim) * g.vp + (c + i) % g.vdim] = y[t][i];
+      }
     }
   }
 }
@@ -188,39 +327,46 @@ struct DeltaScanParams {
   DeltaGeom g;
   const float* kq;           // [rows, Hk, 2, dkp]
   const float* v;            // [rows, H, vp]
-  const float4* gates;       // [rows, H]
+  const float* coef;         // [blocks, H, kCoef]
   float* state;              // [slots, H, dim, vp]
   float* o;                  // [rows, H, vp]
   const int* cu;
   const int* slots;
   const int* pos0;
+  const int* blk0;
 };
 
 constexpr int kScanWarps = 4;
 constexpr int kScanTile = 16;    // tokens per shared-memory stage
-constexpr int CT = 2;            // columns per lane
-constexpr int kScanCols = kScanWarps * 4 * CT;
 
-template <int KT>
+template <int KT, int CT>
 struct ScanCfg {
   static constexpr int DK = 8 * KT;
-  static constexpr int kStageFloats = kScanTile * (2 * DK + kScanCols + 4);
+  static constexpr int kCols = kScanWarps * 4 * CT;                   // value columns per CTA
+  static constexpr int kV = kScanTile * 2 * DK;                       // float offsets within a stage
+  static constexpr int kC = kV + kScanTile * kCols;
+  static constexpr int kStageFloats = kC + kScanTile / kBlk * kCoef;
   static constexpr int kSmemBytes = 2 * kStageFloats * 4;
 };
 
-template <int KT>
-__global__ void __launch_bounds__(kScanWarps * 32)
+// Eight lanes share CT columns of S (lane kl of the eight holds rows {32 i + 4 kl .. + 3}); a warp walks 4 * CT columns,
+// kBlk tokens at a time. The sums d_j, e_j over the eight lanes are exchanged so that lane j ends up with d_j and lane
+// 4 + j with e_j of its columns; every lane then solves for u itself, and lanes 4 .. 7 write the read-outs. A float of k or
+// q loaded from shared memory feeds CT columns: with CT = 2 the kernel is bound by those loads, with CT = 4 by the
+// multiply-adds; small batches take fewer columns per lane and more warps.
+template <int KT, int CT>
+__global__ void __launch_bounds__(kScanWarps * 32, 2)
 delta_scan_kernel(DeltaScanParams p) {
-  pdl_trigger();
   pdl_grid_wait();
-  using Cfg = ScanCfg<KT>;
-  constexpr int DK = Cfg::DK;
+  using Cfg = ScanCfg<KT, CT>;
+  constexpr int DK = Cfg::DK, kScanCols = Cfg::kCols;
   extern __shared__ __align__(16) float sm[];
   const DeltaGeom& g = p.g;
   const int seq = blockIdx.z, head = blockIdx.y;
   const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
   const int slot = p.slots[seq];
   if (n <= 0 || slot < 0) return;
+  const int blk0 = p.blk0[seq], n_blk = (n + kBlk - 1) / kBlk;
   const int hk = head / (g.H / g.Hk);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int kl = lane & 7, cg = lane >> 3;
@@ -246,96 +392,147 @@ delta_scan_kernel(DeltaScanParams p) {
     float* base = sm + (tile & 1) * Cfg::kStageFloats;
     const int t0 = tile * kScanTile;
     const int cnt = min(kScanTile, n - t0);
+    const int full = (cnt + kBlk - 1) / kBlk * kBlk;     // tokens past the end of the last block are zeros
     constexpr int kRowVec = 2 * DK / 4;
-    for (int i = threadIdx.x; i < cnt * kRowVec; i += kScanWarps * 32) {
+    for (int i = threadIdx.x; i < full * kRowVec; i += kScanWarps * 32) {
       const int t = i / kRowVec, w = i % kRowVec;
-      cp16(smem_u32(base + t * 2 * DK + w * 4), p.kq + (static_cast<long long>(row0 + t0 + t) * g.Hk + hk) * 2 * DK + w * 4, 16);
+      const int ts = min(t, cnt - 1);
+      cp16(smem_u32(base + t * 2 * DK + w * 4), p.kq + (static_cast<long long>(row0 + t0 + ts) * g.Hk + hk) * 2 * DK + w * 4,
+           t < cnt ? 16 : 0);
     }
-    float* bv = base + kScanTile * 2 * DK;
     constexpr int kColVec = kScanCols / 4;
-    for (int i = threadIdx.x; i < cnt * kColVec; i += kScanWarps * 32) {
+    for (int i = threadIdx.x; i < full * kColVec; i += kScanWarps * 32) {
       const int t = i / kColVec, w = i % kColVec;
+      const int ts = min(t, cnt - 1);
       const int col = slice0 + w * 4;
       const bool ok = col < g.vp;
-      cp16(smem_u32(bv + t * kScanCols + w * 4),
-           p.v + (static_cast<long long>(row0 + t0 + t) * g.H + head) * g.vp + (ok ? col : 0), ok ? 16 : 0);
+      cp16(smem_u32(base + Cfg::kV + t * kScanCols + w * 4),
+           p.v + (static_cast<long long>(row0 + t0 + ts) * g.H + head) * g.vp + (ok ? col : 0), ok && t < cnt ? 16 : 0);
     }
-    float* bg = bv + kScanTile * kScanCols;
-    if (threadIdx.x < cnt)
-      cp16(smem_u32(bg + threadIdx.x * 4), p.gates + static_cast<long long>(row0 + t0 + threadIdx.x) * g.H + head, 16);
+    constexpr int kCoefVec = kCoef / 4;
+    if (threadIdx.x < full / kBlk * kCoefVec) {
+      const int bi = threadIdx.x / kCoefVec, w = threadIdx.x % kCoefVec;
+      cp16(smem_u32(base + Cfg::kC + bi * kCoef + w * 4),
+           p.coef + (static_cast<long long>(blk0 + tile * (kScanTile / kBlk) + bi) * g.H + head) * kCoef + w * 4, 16);
+    }
   };
   issue(0);
   asm volatile("cp.async.commit_group;" ::: "memory");
 
-  // which of the four sums (dk0, dk1, dq0, dq1) this lane ends up with after the exchange below
-  const int own = ((lane & 4) ? 2 : 0) + ((lane & 2) ? 1 : 0);
-  const int src_base = lane & ~7;
+  const int src0 = lane & ~7;
   for (int tile = 0; tile < n_tiles; ++tile) {
     if (tile + 1 < n_tiles) issue(tile + 1);
     asm volatile("cp.async.commit_group;" ::: "memory");
     asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
     const float* base = sm + (tile & 1) * Cfg::kStageFloats;
-    const float* bv = base + kScanTile * 2 * DK;
-    const float* bg = bv + kScanTile * kScanCols;
-    const int t0 = tile * kScanTile;
-    const int cnt = min(kScanTile, n - t0);
-#pragma unroll 2
-    for (int t = 0; t < cnt; ++t) {
-      const float4* kr = reinterpret_cast<const float4*>(base + t * 2 * DK);
-      const float4* qr = kr + DK / 4;
-      const float4 gt = *reinterpret_cast<const float4*>(bg + t * 4);
-      const float2 vv = *reinterpret_cast<const float2*>(bv + t * kScanCols + lcol);
-      float2 k2[KT / 2];
-      float2 dk[CT], dq[CT];
+    const int nb = min(kScanTile / kBlk, n_blk - tile * (kScanTile / kBlk));
+    for (int bi = 0; bi < nb; ++bi) {
+      const float* kqb = base + bi * kBlk * 2 * DK;
+      const float4* cf = reinterpret_cast<const float4*>(base + Cfg::kC + bi * kCoef);
+      float2 k2[kBlk][KT / 2];
+      float a[2 * kBlk][CT];                       // d_0 .. d_3, e_0 .. e_3 per column
 #pragma unroll
-      for (int c = 0; c < CT; ++c) dk[c] = dq[c] = make_float2(0.f, 0.f);
+      for (int j = 0; j < kBlk; ++j) {
+        const float4* kr = reinterpret_cast<const float4*>(kqb + j * 2 * DK);
+        const float4* qr = kr + DK / 4;
+        float2 dk[CT], dq[CT];
 #pragma unroll
-      for (int i = 0; i < KT / 4; ++i) {
-        const float4 kk = kr[i * 8 + kl];
-        const float4 qq = qr[i * 8 + kl];
-        k2[2 * i] = make_float2(kk.x, kk.y);
-        k2[2 * i + 1] = make_float2(kk.z, kk.w);
-        const float2 q0 = make_float2(qq.x, qq.y), q1 = make_float2(qq.z, qq.w);
+        for (int c = 0; c < CT; ++c) dk[c] = dq[c] = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < KT / 4; ++i) {
+          const float4 kk = kr[i * 8 + kl], qq = qr[i * 8 + kl];
+          k2[j][2 * i] = make_float2(kk.x, kk.y);
+          k2[j][2 * i + 1] = make_float2(kk.z, kk.w);
+          const float2 q0 = make_float2(qq.x, qq.y), q1 = make_float2(qq.z, qq.w);
+#pragma unroll
+          for (int c = 0; c < CT; ++c) {
+            dk[c] = fma2(S[c][2 * i], k2[j][2 * i], dk[c]);
+            dq[c] = fma2(S[c][2 * i], q0, dq[c]);
+            dk[c] = fma2(S[c][2 * i + 1], k2[j][2 * i + 1], dk[c]);
+            dq[c] = fma2(S[c][2 * i + 1], q1, dq[c]);
+          }
+        }
 #pragma unroll
         for (int c = 0; c < CT; ++c) {
-          dk[c] = fma2(S[c][2 * i], k2[2 * i], dk[c]);
-          dq[c] = fma2(S[c][2 * i], q0, dq[c]);
-          dk[c] = fma2(S[c][2 * i + 1], k2[2 * i + 1], dk[c]);
-          dq[c] = fma2(S[c][2 * i + 1], q1, dq[c]);
+          a[j][c] = dk[c].x + dk[c].y;
+          a[kBlk + j][c] = dq[c].x + dq[c].y;
         }
       }
-      float a0 = dk[0].x + dk[0].y, a1 = dk[1].x + dk[1].y, a2 = dq[0].x + dq[0].y, a3 = dq[1].x + dq[1].y;
-      // sum over the eight lanes of the column group: halve the number of values held per lane at each exchange
-      {
-        const bool hi = lane & 4;
-        const float s0 = hi ? a0 : a2, s1 = hi ? a1 : a3;
-        const float k0 = hi ? a2 : a0, k1 = hi ? a3 : a1;
-        a0 = k0 + __shfl_xor_sync(0xffffffffu, s0, 4);
-        a1 = k1 + __shfl_xor_sync(0xffffffffu, s1, 4);
-      }
-      {
-        const bool hi = lane & 2;
-        const float s0 = hi ? a0 : a1, k0 = hi ? a1 : a0;
-        a0 = k0 + __shfl_xor_sync(0xffffffffu, s0, 2);
-      }
-      a0 += __shfl_xor_sync(0xffffffffu, a0, 1);
-      const float dk0 = __shfl_sync(0xffffffffu, a0, src_base);
-      const float dk1 = __shfl_sync(0xffffffffu, a0, src_base + 2);
-      const float u0 = gt.y * (vv.x - gt.x * dk0);
-      const float u1 = gt.y * (vv.y - gt.x * dk1);
-      const float2 g2 = make_float2(gt.x, gt.x);
-      const float2 uu0 = make_float2(u0, u0), uu1 = make_float2(u1, u1);
+      // halve the number of sums held per lane at each exchange
+      float r4[4][CT], r2[2][CT], r1[CT];
 #pragma unroll
-      for (int i = 0; i < KT / 2; ++i) {
-        S[0][i] = fma2(S[0][i], g2, mul2(k2[i], uu0));
-        S[1][i] = fma2(S[1][i], g2, mul2(k2[i], uu1));
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int c = 0; c < CT; ++c) {
+          const float keep = (lane & 4) ? a[4 + i][c] : a[i][c], give = (lane & 4) ? a[i][c] : a[4 + i][c];
+          r4[i][c] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+        }
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int c = 0; c < CT; ++c) {
+          const float keep = (lane & 2) ? r4[2 + i][c] : r4[i][c], give = (lane & 2) ? r4[i][c] : r4[2 + i][c];
+          r2[i][c] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+        }
+#pragma unroll
+      for (int c = 0; c < CT; ++c) {
+        const float keep = (lane & 1) ? r2[1][c] : r2[0][c], give = (lane & 1) ? r2[0][c] : r2[1][c];
+        r1[c] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
       }
-      if ((lane & 5) == 4) {               // lanes 4 and 6 of each group hold the two read-outs
-        const int c = own - 2;
-        if (col0 + c < g.vdim)
-          p.o[(static_cast<long long>(row0 + t0 + t) * g.H + head) * g.vp + col0 + c] =
-              fmaf(gt.x, a0, gt.z * (c ? u1 : u0));
+      const float4 G = cf[0], be = cf[1], A0 = cf[2], A1 = cf[3], cc = cf[4];
+      float vals[kBlk][CT];
+#pragma unroll
+      for (int j = 0; j < kBlk; ++j) {
+        const float* vr = base + Cfg::kV + (bi * kBlk + j) * kScanCols + lcol;
+        if constexpr (CT == 4) {
+          const float4 t = *reinterpret_cast<const float4*>(vr);
+          vals[j][0] = t.x; vals[j][1] = t.y; vals[j][2] = t.z; vals[j][3] = t.w;
+        } else {
+#pragma unroll
+          for (int c = 0; c < CT; ++c) vals[j][c] = vr[c];
+        }
+      }
+      float u[kBlk][CT];
+#pragma unroll
+      for (int c = 0; c < CT; ++c) {
+        float d[kBlk], vv[kBlk];
+#pragma unroll
+        for (int j = 0; j < kBlk; ++j) {
+          d[j] = __shfl_sync(0xffffffffu, r1[c], src0 + j);
+          vv[j] = vals[j][c];
+        }
+        u[0][c] = be.x * fmaf(-G.x, d[0], vv[0]);
+        u[1][c] = be.y * fmaf(-A0.x, u[0][c], fmaf(-G.y, d[1], vv[1]));
+        u[2][c] = be.z * fmaf(-A0.z, u[1][c], fmaf(-A0.y, u[0][c], fmaf(-G.z, d[2], vv[2])));
+        u[3][c] = be.w * fmaf(-A1.y, u[2][c], fmaf(-A1.x, u[1][c], fmaf(-A0.w, u[0][c], fmaf(-G.w, d[3], vv[3]))));
+      }
+      if (kl >= 4) {
+        const int j = kl - 4, t = tile * kScanTile + bi * kBlk + j;
+        const float4 W = cf[5 + j];
+        const float Gj = base[Cfg::kC + bi * kCoef + j];
+        if (t < n) {
+          float* orow = p.o + (static_cast<long long>(row0 + t) * g.H + head) * g.vp + col0;
+#pragma unroll
+          for (int c = 0; c < CT; ++c)
+            if (col0 + c < g.vdim)
+              orow[c] = fmaf(Gj, r1[c], fmaf(W.x, u[0][c], fmaf(W.y, u[1][c], fmaf(W.z, u[2][c], W.w * u[3][c]))));
+        }
+      }
+      const float2 g2 = make_float2(G.w, G.w);
+      const float cs[kBlk] = {cc.x, cc.y, cc.z, cc.w};
+#pragma unroll
+      for (int c = 0; c < CT; ++c) {
+        float2 uu[kBlk];
+#pragma unroll
+        for (int j = 0; j < kBlk; ++j) uu[j] = make_float2(cs[j] * u[j][c], cs[j] * u[j][c]);
+#pragma unroll
+        for (int i = 0; i < KT / 2; ++i) {
+          float2 acc = mul2(S[c][i], g2);
+#pragma unroll
+          for (int j = 0; j < kBlk; ++j) acc = fma2(k2[j][i], uu[j], acc);
+          S[c][i] = acc;
+        }
       }
     }
     __syncthreads();
@@ -351,28 +548,78 @@ delta_scan_kernel(DeltaScanParams p) {
 }
 
 // ------------------------------------------------------------------ read-out norm and gate
-// One warp per (row, head): y = o / rms(o) * weight * silu(gate), in the projection's type; columns past H * vdim of
-// the output row are zeroed by the last head's warp.
-template <typename T>
+// y = o / rms(o) * weight * silu(gate) per (row, head), in the projection's type; columns past H * vdim of the output row
+// are zeroed by the last head's warp. A warp takes one head of kNormRows rows; heads of up to 128 columns are read once,
+// all rows at a time, wider ones are read twice.
+constexpr int kNormRows = 4;
+
+template <typename T, bool NARROW>
 __global__ void __launch_bounds__(256)
 delta_gate_norm_kernel(DeltaGeom g, const float* o, const T* proj, const float* weight, T* y, long long ldy, int y_cols,
                        int rows, float eps) {
   pdl_trigger();
   pdl_grid_wait();
-  const long long w = blockIdx.x * 8ll + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (w >= static_cast<long long>(rows) * g.H) return;
-  const int row = static_cast<int>(w / g.H), h = static_cast<int>(w % g.H);
-  const float* orow = o + w * g.vp;
-  const T* gate = proj + static_cast<long long>(row) * g.ldp + g.off_g + h * g.vdim;
-  T* yr = y + row * ldy + h * g.vdim;
-  float ss = 0.f;
-  for (int c = lane; c < g.vdim; c += 32) ss = fmaf(orow[c], orow[c], ss);
-  ss = warp_sum(ss);
-  const float r = 1.f / sqrtf(ss / static_cast<float>(g.vdim) + eps);
-  for (int c = lane; c < g.vdim; c += 32) yr[c] = from_f32<T>(orow[c] * r * weight[c] * silu_f(to_f32<T>(gate[c])));
+  const int h = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= g.H) return;
+  constexpr bool kFast = sizeof(T) == 2;
+  const bool vec = g.vdim % 4 == 0 && ldy % 4 == 0;
+  const int row_a = blockIdx.y * kNormRows, cnt = min(kNormRows, rows - row_a);
+  const float inv_n = 1.f / static_cast<float>(g.vdim);
+  const float* o0 = o + (static_cast<long long>(row_a) * g.H + h) * g.vp;
+  const T* g0 = proj + static_cast<long long>(row_a) * g.ldp + g.off_g + h * g.vdim;
+  T* y0 = y + row_a * ldy + h * g.vdim;
+  const long long so = static_cast<long long>(g.H) * g.vp;
+  auto store = [&](T* dst, int c, const float (&f)[4]) {
+    if (vec) {
+      if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+      else *reinterpret_cast<float4*>(dst + c) = make_float4(f[0], f[1], f[2], f[3]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (c + e < g.vdim) dst[c + e] = from_f32<T>(f[e]);
+    }
+  };
+  if constexpr (NARROW) {
+    const int c = lane * 4, valid = g.vdim - c;
+    float f[kNormRows][4], gt[kNormRows][4], wt[4];
+#pragma unroll
+    for (int r = 0; r < kNormRows; ++r) {
+      const int rr = min(r, cnt - 1);
+      load_ch<float, 4>(o0 + rr * so + c, valid, true, f[r]);
+      load_ch<T, 4>(g0 + rr * g.ldp + c, valid, vec, gt[r]);
+    }
+    load_ch<float, 4>(weight + c, valid, true, wt);
+#pragma unroll
+    for (int r = 0; r < kNormRows; ++r) {
+      const float ss = warp_sum(f[r][0] * f[r][0] + f[r][1] * f[r][1] + f[r][2] * f[r][2] + f[r][3] * f[r][3]);
+      const float rs = rsqrtf(fmaf(ss, inv_n, eps));
+#pragma unroll
+      for (int e = 0; e < 4; ++e) f[r][e] *= rs * wt[e] * silu_f<kFast>(gt[r][e]);
+      if (r < cnt && valid > 0) store(y0 + r * ldy, c, f[r]);
+    }
+  } else {
+    for (int r = 0; r < cnt; ++r) {
+      float ss = 0.f;
+      for (int c = lane * 4; c < g.vdim; c += 128) {
+        float f[4];
+        load_ch<float, 4>(o0 + r * so + c, g.vdim - c, true, f);
+        ss += f[0] * f[0] + f[1] * f[1] + f[2] * f[2] + f[3] * f[3];
+      }
+      const float rs = rsqrtf(fmaf(warp_sum(ss), inv_n, eps));
+      for (int c = lane * 4; c < g.vdim; c += 128) {
+        float f[4], gt[4], wt[4];
+        load_ch<float, 4>(o0 + r * so + c, g.vdim - c, true, f);
+        load_ch<T, 4>(g0 + r * g.ldp + c, g.vdim - c, vec, gt);
+        load_ch<float, 4>(weight + c, g.vdim - c, true, wt);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) f[e] *= rs * wt[e] * silu_f<kFast>(gt[e]);
+        store(y0 + r * ldy, c, f);
+      }
+    }
+  }
   if (h == g.H - 1)
-    for (int c = g.H * g.vdim + lane; c < y_cols; c += 32) y[row * ldy + c] = from_f32<T>(0.f);
+    for (int r = 0; r < cnt; ++r)
+      for (int c = g.H * g.vdim + lane; c < y_cols; c += 32) y[(row_a + r) * ldy + c] = from_f32<T>(0.f);
 }
 
 // ------------------------------------------------------------------ decoded rows: one token per sequence, one launch
@@ -399,7 +646,7 @@ constexpr int kStepWarps = kStepThreads / 32;
 // CTA = (sequence, key head): it owns the head's q / k channels and all value heads that read them. A warp holds RPW
 // rows of a 128-column block of S: dim / 8 rounded up.
 template <typename T, int RPW>
-__global__ void __launch_bounds__(kStepThreads)
+__global__ void __launch_bounds__(kStepThreads, RPW <= 16 ? 2 : 1)
 delta_step_kernel(DeltaStepParams p) {
   pdl_trigger();
   pdl_grid_wait();
@@ -426,23 +673,70 @@ delta_step_kernel(DeltaStepParams p) {
   const T* proj = static_cast<const T*>(p.proj) + row * g.ldp;
   const int tail = p.taps - 1;
   T* cs = static_cast<T*>(p.conv_state) + static_cast<long long>(slot) * tail * g.conv_c;
-  auto conv = [&](int c) -> float {
-    float acc = 0.f;
-    for (int j = 0; j < tail; ++j) {
-      float x = has_state ? to_f32<T>(cs[static_cast<long long>(j) * g.conv_c + c]) : 0.f;
-      acc = fmaf(p.conv_w[static_cast<long long>(j) * g.conv_c + c], x, acc);
-      if (j > 0) cs[static_cast<long long>(j - 1) * g.conv_c + c] = from_f32<T>(x);
-    }
-    const T cur = proj[c];
-    if (tail > 0) cs[static_cast<long long>(tail - 1) * g.conv_c + c] = cur;
-    return silu_f(fmaf(p.conv_w[static_cast<long long>(tail) * g.conv_c + c], to_f32<T>(cur), acc));
+  // The state streams through registers one (head, 128-column block) at a time; the first block is requested before the
+  // convolution, every later one as soon as its predecessor has been stored.
+  const int col_blocks = (g.vp + 127) / 128, steps = per * col_blocks;
+  float4 S[RPW];
+  auto state_at = [&](int it) {
+    return p.state + (static_cast<long long>(slot) * g.H + hk * per + it / col_blocks) * g.dim * g.vp + (it % col_blocks) * 128 +
+           lane * 4;
   };
-  for (int d = tid; d < g.dkp; d += kStepThreads) {
-    sq[d] = d < g.dim ? conv(hk * g.dim + d) : 0.f;
-    sk[d] = d < g.dim ? conv(g.off_k + hk * g.dim + d) : 0.f;
+  auto fetch = [&](int it) {
+    const float* st = state_at(it);
+    const bool ok = has_state && (it % col_blocks) * 128 + lane * 4 < g.vp;
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) {
+      const int k = warp + kStepWarps * i;
+      S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (ok && k < g.dim) S[i] = __ldcs(reinterpret_cast<const float4*>(st + static_cast<long long>(k) * g.vp));
+    }
+  };
+  fetch(0);
+  // channel i of this CTA (its q, its k, then the v of its heads): column in the projection, place in shared memory
+  const int n_ch = 2 * g.dim + per * g.vdim;
+  auto channel = [&](int i, int* c) -> float* {
+    if (i < g.dim) {
+      *c = hk * g.dim + i;
+      return sq + i;
+    }
+    if (i < 2 * g.dim) {
+      *c = g.off_k + hk * g.dim + i - g.dim;
+      return sk + i - g.dim;
+    }
+    const int v = i - 2 * g.dim;
+    *c = g.off_v + hk * per * g.vdim + v;
+    return sv + (v / g.vdim) * g.vp + v % g.vdim;
+  };
+  for (int i0 = tid; i0 < n_ch; i0 += 2 * kStepThreads) {
+    float x[2][8], w[2][8];               // both channels' inputs are requested before anything is written
+    int c[2];
+    float* dst[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int i = i0 + h * kStepThreads;
+      dst[h] = i < n_ch ? channel(i, &c[h]) : nullptr;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        x[h][j] = w[h][j] = 0.f;
+        if (dst[h] && j <= tail) {
+          w[h][j] = p.conv_w[static_cast<long long>(j) * g.conv_c + c[h]];
+          if (j == tail) x[h][j] = to_f32<T>(proj[c[h]]);
+          else if (has_state) x[h][j] = to_f32<T>(cs[static_cast<long long>(j) * g.conv_c + c[h]]);
+        }
+      }
+    }
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      if (!dst[h]) continue;
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        acc = fmaf(w[h][j], x[h][j], acc);
+        if (j > 0 && j <= tail) cs[static_cast<long long>(j - 1) * g.conv_c + c[h]] = from_f32<T>(x[h][j]);
+      }
+      *dst[h] = silu_f<sizeof(T) == 2>(acc);
+    }
   }
-  for (int c = tid; c < per * g.vdim; c += kStepThreads)
-    sv[(c / g.vdim) * g.vp + c % g.vdim] = conv(g.off_v + hk * per * g.vdim + c);
   __syncthreads();
   float sqq = 0.f, skk = 0.f, sqk = 0.f;
   for (int d = tid; d < g.dim; d += kStepThreads) {
@@ -470,22 +764,17 @@ delta_step_kernel(DeltaStepParams p) {
   const float rk = 1.f / sqrtf(skk + 1e-6f);
   const float kq = sqk * rq * rk;
 
-  for (int hh = 0; hh < per; ++hh) {
-    const int h = hk * per + hh;
-    const float bb = to_f32<T>(proj[g.off_b + h]), aa = to_f32<T>(proj[g.off_a + h]);
-    const float decay = expf(-expf(p.a_log[h]) * softplus_f(aa + p.dt_bias[h]));
-    const float beta = sigmoid_f(bb);
-    float* st = p.state + (static_cast<long long>(slot) * g.H + h) * g.dim * g.vp;
-    for (int cb = 0; cb < g.vp; cb += 128) {
-      const int col = cb + lane * 4;
+  float decay = 0.f, beta = 0.f;
+  for (int it = 0; it < steps; ++it) {
+    const int hh = it / col_blocks, h = hk * per + hh;
+    if (it % col_blocks == 0) {
+      decay = expf(-expf(p.a_log[h]) * softplus_f(to_f32<T>(proj[g.off_a + h]) + p.dt_bias[h]));
+      beta = sigmoid_f(to_f32<T>(proj[g.off_b + h]));
+    }
+    float* st = state_at(it);
+    {
+      const int col = (it % col_blocks) * 128 + lane * 4;
       const bool col_ok = col < g.vp;
-      float4 S[RPW];
-#pragma unroll
-      for (int i = 0; i < RPW; ++i) {
-        const int k = warp + kStepWarps * i;
-        S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (has_state && col_ok && k < g.dim) S[i] = *reinterpret_cast<const float4*>(st + static_cast<long long>(k) * g.vp + col);
-      }
       float4 dk = make_float4(0.f, 0.f, 0.f, 0.f), dq = dk;
 #pragma unroll
       for (int i = 0; i < RPW; ++i) {
@@ -535,10 +824,11 @@ delta_step_kernel(DeltaStepParams p) {
             s.y = fmaf(s.y, decay, kk * u.y);
             s.z = fmaf(s.z, decay, kk * u.z);
             s.w = fmaf(s.w, decay, kk * u.w);
-            *reinterpret_cast<float4*>(st + static_cast<long long>(k) * g.vp + col) = s;
+            __stcs(reinterpret_cast<float4*>(st + static_cast<long long>(k) * g.vp), s);
           }
         }
       }
+      if (it + 1 < steps) fetch(it + 1);
       __syncthreads();
     }
   }
@@ -562,35 +852,66 @@ bool read_geom(const int* v, long long ldp, DeltaGeom* g) {
   g->ldp = ldp;
   const bool dk_ok = g->dkp == 32 || g->dkp == 64 || g->dkp == 128 || g->dkp == 256;
   return g->Hk > 0 && g->H > 0 && g->H % g->Hk == 0 && g->dim > 0 && g->vdim > 0 && dk_ok && g->dim <= g->dkp &&
-         g->vp >= g->vdim && g->vp % 4 == 0 && g->conv_c > 0 && ldp >= g->off_a + g->H;
+         g->vp >= g->vdim && g->vp % 4 == 0 && g->conv_c > 0 && ldp >= g->off_a + g->H && ldp % 8 == 0 && g->off_k % 8 == 0 &&
+         g->off_v % 8 == 0 && g->off_g % 8 == 0 && g->conv_c % 8 == 0;
+}
+
+template <typename T, int TAPS>
+int launch_prepare_taps(const DeltaPrepParams& p, cudaStream_t s) {
+  const DeltaGeom& g = p.g;
+  const dim3 grid(g.Hk + (g.H * g.vdim + 255) / 256, (p.blocks + 3) / 4);
+  const bool pdl = pdl_all_enabled();
+  switch (g.dkp) {
+    case 32: launch_pdl(delta_prepare_kernel<T, TAPS, 1>, grid, dim3(128), 0, s, pdl, p); break;
+    case 64: launch_pdl(delta_prepare_kernel<T, TAPS, 2>, grid, dim3(128), 0, s, pdl, p); break;
+    case 128: launch_pdl(delta_prepare_kernel<T, TAPS, 4>, grid, dim3(128), 0, s, pdl, p); break;
+    default: launch_pdl(delta_prepare_kernel<T, TAPS, 8>, grid, dim3(128), 0, s, pdl, p); break;
+  }
+  return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T>
 int launch_prepare(const DeltaPrepParams& p, int taps, cudaStream_t s) {
-  const DeltaGeom& g = p.g;
-  const dim3 grid(g.Hk + (g.H * g.vdim + 127) / 128, (p.rows + 7) / 8);
-  const bool pdl = pdl_all_enabled();
-#define TSB_PREP(N) case N: launch_pdl(delta_prepare_kernel<T, N>, grid, dim3(256), 0, s, pdl, p); break
   switch (taps) {
-    TSB_PREP(1); TSB_PREP(2); TSB_PREP(3); TSB_PREP(4); TSB_PREP(5); TSB_PREP(6); TSB_PREP(7); TSB_PREP(8);
+    case 1: return launch_prepare_taps<T, 1>(p, s);
+    case 2: return launch_prepare_taps<T, 2>(p, s);
+    case 3: return launch_prepare_taps<T, 3>(p, s);
+    case 4: return launch_prepare_taps<T, 4>(p, s);
+    case 5: return launch_prepare_taps<T, 5>(p, s);
+    case 6: return launch_prepare_taps<T, 6>(p, s);
+    case 7: return launch_prepare_taps<T, 7>(p, s);
+    case 8: return launch_prepare_taps<T, 8>(p, s);
     default: return -2;
   }
-#undef TSB_PREP
+}
+
+template <int KT, int CT>
+int launch_scan_cols(const DeltaScanParams& p, int nseq, cudaStream_t s) {
+  using Cfg = ScanCfg<KT, CT>;
+  auto kern = delta_scan_kernel<KT, CT>;
+  static PerDeviceFlag attr;
+  if (attr.unset()) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    attr.set();
+  }
+  const dim3 grid((p.g.vdim + Cfg::kCols - 1) / Cfg::kCols, p.g.H, nseq);
+  // launched after its predecessor has left: CTAs that start early land on whatever SMs drain first and stay there for
+  // the whole scan, several on one SM while others idle
+  launch_pdl(kern, grid, dim3(kScanWarps * 32), Cfg::kSmemBytes, s, false, p);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <int KT>
 int launch_scan(const DeltaScanParams& p, int nseq, cudaStream_t s) {
-  auto kern = delta_scan_kernel<KT>;
-  static PerDeviceFlag attr;
-  if (attr.unset()) {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, ScanCfg<KT>::kSmemBytes);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    attr.set();
-  }
-  const dim3 grid((p.g.vdim + kScanCols - 1) / kScanCols, p.g.H, nseq);
-  launch_pdl(kern, grid, dim3(kScanWarps * 32), ScanCfg<KT>::kSmemBytes, s, pdl_all_enabled(), p);
-  return static_cast<int>(cudaGetLastError());
+  static const int forced = [] { const char* e = getenv("TESSERACT_DELTA_COLS"); return e ? atoi(e) : 0; }();
+  // columns of the whole launch against what one warp per scheduler covers
+  const long long cols = static_cast<long long>(nseq) * p.g.H * p.g.vdim, one = 4ll * sm_count() * 4;
+  int ct = forced ? forced : (cols >= 5 * one ? 4 : (cols >= one ? 2 : 1));
+  if (KT > 16 && ct > 2) ct = 2;
+  if constexpr (KT <= 16)
+    if (ct == 4) return launch_scan_cols<KT, 4>(p, nseq, s);
+  return ct >= 2 ? launch_scan_cols<KT, 2>(p, nseq, s) : launch_scan_cols<KT, 1>(p, nseq, s);
 }
 
 template <typename T, int RPW>
@@ -612,22 +933,22 @@ int launch_step(const DeltaStepParams& p, int rows, cudaStream_t s) {
 }  // namespace
 }  // namespace tsb
 
-// Prompt rows [rows, ldp] of nseq sequences. dtype: 0 = fp32, 1 = bf16 (projection, convolution state, y). `kq`, `v`,
-// `gates`, `o` are fp32 scratch of rows * Hk * 2 * dkp, rows * H * vp, rows * H * 4 and rows * H * vp elements (16-byte
-// aligned; the padding columns of v must be zero). See the structures above for the rest.
+// Prompt rows [rows, ldp] of nseq sequences, cut into blocks of 4 tokens from each sequence's first row (blk_seq [blocks],
+// blk0 [nseq + 1]). dtype: 0 = fp32, 1 = bf16 (projection, convolution state, y). `kq`, `v`, `coef`, `o` are fp32 scratch
+// of rows * Hk * 2 * dkp, rows * H * vp, blocks * H * 36 and rows * H * vp elements (16-byte aligned). See the
+// structures above for the rest.
 TSB_EXPORT int tsb_delta_prefill(const void* proj, long long ldp, const int* geom, const float* conv_w, const float* a_log,
                                  const float* dt_bias, const float* norm_w, void* conv_state, float* state, const int* cu,
-                                 const int* slots, const int* pos0, const int* seq_of, float* kq, float* v, float* gates,
-                                 float* o, void* y, long long ldy, int y_cols, int rows, int nseq, int taps, float eps,
-                                 int dtype, void* stream) {
+                                 const int* slots, const int* pos0, const int* blk_seq, const int* blk0, float* kq, float* v,
+                                 float* coef, float* o, void* y, long long ldy, int y_cols, int rows, int blocks, int nseq,
+                                 int taps, float eps, int dtype, void* stream) {
   using namespace tsb;
   DeltaGeom g;
-  if (!read_geom(geom, ldp, &g) || rows <= 0 || nseq <= 0 || nseq > 65535 || taps < 1 || taps > 8 || (rows + 7) / 8 > 65535 ||
-      (dtype != 0 && dtype != 1) || y_cols < g.H * g.vdim)
+  if (!read_geom(geom, ldp, &g) || rows <= 0 || blocks <= 0 || nseq <= 0 || nseq > 65535 || taps < 1 || taps > 8 ||
+      (blocks + 3) / 4 > 65535 || (rows + kNormRows - 1) / kNormRows > 65535 || (dtype != 0 && dtype != 1) || y_cols < g.H * g.vdim)
     return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  DeltaPrepParams pp{g, proj, conv_w, a_log, dt_bias, conv_state, cu, slots, pos0, seq_of, kq, v,
-                     reinterpret_cast<float4*>(gates), rows};
+  DeltaPrepParams pp{g, proj, conv_w, a_log, dt_bias, conv_state, cu, slots, pos0, blk_seq, blk0, kq, v, coef, blocks};
   int rc = dtype == 1 ? launch_prepare<__nv_bfloat16>(pp, taps, s) : launch_prepare<float>(pp, taps, s);
   if (rc) return rc;
   const bool pdl = pdl_all_enabled();
@@ -642,7 +963,7 @@ TSB_EXPORT int tsb_delta_prefill(const void* proj, long long ldp, const int* geo
     rc = static_cast<int>(cudaGetLastError());
     if (rc) return rc;
   }
-  DeltaScanParams sp{g, kq, v, reinterpret_cast<const float4*>(gates), state, o, cu, slots, pos0};
+  DeltaScanParams sp{g, kq, v, coef, state, o, cu, slots, pos0, blk0};
   switch (g.dkp) {
     case 32: rc = launch_scan<4>(sp, nseq, s); break;
     case 64: rc = launch_scan<8>(sp, nseq, s); break;
@@ -650,13 +971,15 @@ TSB_EXPORT int tsb_delta_prefill(const void* proj, long long ldp, const int* geo
     default: rc = launch_scan<32>(sp, nseq, s); break;
   }
   if (rc) return rc;
-  const unsigned blocks = static_cast<unsigned>((static_cast<long long>(rows) * g.H + 7) / 8);
-  if (dtype == 1)
-    launch_pdl(delta_gate_norm_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, s, pdl, g, o,
-               static_cast<const __nv_bfloat16*>(proj), norm_w, static_cast<__nv_bfloat16*>(y), ldy, y_cols, rows, eps);
-  else
-    launch_pdl(delta_gate_norm_kernel<float>, dim3(blocks), dim3(256), 0, s, pdl, g, o, static_cast<const float*>(proj), norm_w,
-               static_cast<float*>(y), ldy, y_cols, rows, eps);
+  const dim3 ngrid((g.H + 7) / 8, (rows + kNormRows - 1) / kNormRows);
+  auto norm = [&](auto tag, auto narrow) {
+    using T = decltype(tag);
+    launch_pdl(delta_gate_norm_kernel<T, decltype(narrow)::value>, ngrid, dim3(256), 0, s, pdl, g, o, static_cast<const T*>(proj),
+               norm_w, static_cast<T*>(y), ldy, y_cols, rows, eps);
+  };
+  const bool narrow = g.vdim <= 128;
+  if (dtype == 1) narrow ? norm(__nv_bfloat16{}, std::true_type{}) : norm(__nv_bfloat16{}, std::false_type{});
+  else narrow ? norm(float{}, std::true_type{}) : norm(float{}, std::false_type{});
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -667,7 +990,7 @@ TSB_EXPORT int tsb_delta_step(const void* proj, long long ldp, const int* geom, 
                               void* stream) {
   using namespace tsb;
   DeltaGeom g;
-  if (!read_geom(geom, ldp, &g) || rows <= 0 || g.Hk > 65535 || taps < 1 || (dtype != 0 && dtype != 1) ||
+  if (!read_geom(geom, ldp, &g) || rows <= 0 || g.Hk > 65535 || taps < 1 || taps > 8 || (dtype != 0 && dtype != 1) ||
       y_cols < g.H * g.vdim)
     return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

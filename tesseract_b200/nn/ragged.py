@@ -215,10 +215,11 @@ class RaggedBatch:
                 return cache.tables[pslots[i], p // bs] * bs + p % bs
             for c in chunks:
                 segs[c] = cut_segments(list(zip(pos0[nd:].tolist(), n[nd:].tolist())), c, slot_of)
+        nblk = (n[nd:] + 3) // 4                  # the recurrence takes four tokens of a portion at once
         fields = {
             "tokens": np.concatenate(toks), "positions": positions, "slots": pool_slots, "seq_of": seq_of, "tables": tables,
             "state_slots": slot, "lens": pos0[:nd] + 1, "cu": row0[nd:] - row0[nd], "pos0": pos0[nd:],
-            "prompt_seq": seq_of[nd:] - nd, "want": np.asarray(rows, dtype=np.int64),
+            "blk_seq": np.repeat(np.arange(self.n_prompts), nblk), "blk0": np.concatenate([[0], np.cumsum(nblk)]), "want": np.asarray(rows, dtype=np.int64),
         }
         for c, sg in segs.items():
             for name, a in zip(("cu_q", "cu_k", "stage_rows", "gather_dst", "gather_src"), sg.host):

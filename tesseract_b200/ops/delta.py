@@ -18,7 +18,7 @@ from .._native import check, dtype_code, lib, stream_ptr
 
 P, I, L, F = _native.P, _native.I, _native.L, _native.F
 _native.register_signatures({
-    "tsb_delta_prefill": [P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, F, I, P],
+    "tsb_delta_prefill": [P, L] + [P] * 17 + [L, I, I, I, I, I, F, I, P],
     "tsb_delta_step": [P, L, P, P, P, P, P, P, P, P, P, P, L, I, I, I, F, I, P],
 })
 
@@ -125,14 +125,15 @@ def gated_delta(proj: torch.Tensor, geo: DeltaGeometry, w: DeltaWeights, conv_st
         H, dev = geo.heads, proj.device
         kq = torch.empty((n, geo.kv_heads, 2, geo.dim_pad), device=dev, dtype=torch.float32)
         v = torch.empty((n, H, geo.vdim_pad), device=dev, dtype=torch.float32)
-        gates = torch.empty((n, H, 4), device=dev, dtype=torch.float32)
+        blocks = batch.blk_seq.shape[0]
+        coef = torch.empty((blocks, H, 36), device=dev, dtype=torch.float32)
         o = torch.empty((n, H, geo.vdim_pad), device=dev, dtype=torch.float32)
         pr = proj[nd:]
         check(lib().tsb_delta_prefill(pr.data_ptr(), pr.stride(0), g, w.conv.data_ptr(), w.a_log.data_ptr(), w.dt_bias.data_ptr(),
                                       w.norm.data_ptr(), conv_state.data_ptr(), state.data_ptr(), batch.cu.data_ptr(),
-                                      batch.state_slots[nd:].data_ptr(), batch.pos0.data_ptr(), batch.prompt_seq.data_ptr(),
-                                      kq.data_ptr(), v.data_ptr(), gates.data_ptr(), o.data_ptr(), y[nd:].data_ptr(), y.stride(0),
-                                      geo.out_cols, n, batch.n_prompts, geo.taps, float(w.eps), dt, st), "tsb_delta_prefill")
+                                      batch.state_slots[nd:].data_ptr(), batch.pos0.data_ptr(), batch.blk_seq.data_ptr(),
+                                      batch.blk0.data_ptr(), kq.data_ptr(), v.data_ptr(), coef.data_ptr(), o.data_ptr(),
+                                      y[nd:].data_ptr(), y.stride(0), geo.out_cols, n, blocks, batch.n_prompts, geo.taps, float(w.eps), dt, st), "tsb_delta_prefill")
         _native.add_launches(3 if geo.taps > 1 else 2)
     return y
 

@@ -197,8 +197,8 @@ def test_clamped_glu_cuts_gate_above_only_and_up_on_both_sides(kind):
     got = ops.clamped_glu(gu.to(dev), b.to(dev), limit).cpu().double()
     assert (got - want).abs().max() < (1e-5 if dt == torch.float32 else 0.02)
     # a gate far below -limit still passes (it is not cut from below), one far above is cut; up likewise on both sides
-    row = torch.tensor([[-2.0, 9.0, 0.5, 0.5, 1.0, 1.0, -9.0, 9.0]]).to(dt)
-    want = oracle.clamped_glu(row[:, :4].double(), row[:, 4:].double(), limit)
+    row = torch.tensor([[-2.0, 9.0, 0.5, 0.5] * 2 + [1.0, 1.0, -9.0, 9.0] * 2]).to(dt)
+    want = oracle.clamped_glu(row[:, :8].double(), row[:, 8:].double(), limit)
     assert abs(float(want[0, 0])) > 0.1
     assert (ops.clamped_glu(row.to(dev), None, limit).cpu().double() - want).abs().max() < 0.01
 
