@@ -110,6 +110,9 @@ def parse_args():
                     help="auto | dp | tp | tpK (tensor parallel over K ranks, data parallel over the rest) | a comma list: "
                          "every mesh listed is measured and `value` is the fastest")
     ap.add_argument("--no-e2e", action="store_true")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="instead of the headline: prefill and decode throughput of the hybrid decoder (gated delta rule + chunked "
+                         "attention) beside Llama at equal sizes, one GPU (benchmarks/bench_hybrid.py)")
     ap.add_argument("--ref-time-budget", type=float, default=float(os.environ.get("TESSERACT_REF_TIME_BUDGET", 780)),
                     help="(--impl reference) seconds the whole reference arm may take; the timed step count shrinks to fit")
     return ap.parse_args()
@@ -288,6 +291,15 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         return run_reference(args)
+    if args.hybrid:
+        sys.path.insert(0, os.path.join(REPO_ROOT, "benchmarks"))
+        from bench_hybrid import run
+        sampler = ClockSampler(0)
+        sampler.start()
+        sizes = run()
+        print(json.dumps({"benchmark": "hybrid decoder serving beside Llama at equal size", "n_gpus": 1, "dtype": "bf16",
+                          "data": "synthetic random token ids; random-init weights", "sizes": sizes, "clocks": sampler.stop()}))
+        return 0
 
     import gc
 

@@ -463,9 +463,15 @@ def _chunk_attn(b, n, rows, past, chunk):
 def case_chunk_attn(b: Bench):
     """Append + attention. Prompts: two sequences of 4096 in chunks of 4096 (the flash_fwd case) and of 1024; decode: 256
     sequences at 1400 tokens of one chunk (the decode case)."""
+    from tesseract_b200 import ops
     for chunk in (4096, 1024):
         ms = _chunk_attn(b, 2, 4096, 0, chunk)
         report("chunk_attn_prefill", ms, flops=2 * 4096 * chunk * 32 * 128 * 2.0, shape=[2, 4096, chunk])
+        n = 2 * 4096 // chunk                       # the plain kernel over as many sequences of the chunk's length
+        qkv = b.randn(n, chunk, 48, 128)
+        with torch.no_grad():
+            ms = b.time(lambda: ops.flash_attention_packed(qkv, 32, 8))
+        report("flash_fwd_same_lengths", ms, flops=2 * 4096 * chunk * 32 * 128 * 2.0, shape=[n, chunk])
     ms = _chunk_attn(b, 256, 1, 1399, 4096)
     report("chunk_attn_decode", ms, bytes_=256 * 1400 * 8 * 128 * 2 * 2, shape=[256, 1400])
 

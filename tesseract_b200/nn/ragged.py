@@ -97,6 +97,14 @@ class HybridSequence:
             c.tables[self.slot, len(self.blocks)] = b
             self.blocks.append(b)
 
+    def release_to(self, blocks: int, slot: int) -> None:
+        """Undoes a ``reserve`` that found ``blocks`` pages and this slot."""
+        while len(self.blocks) > blocks:
+            self.cache.allocator.free(self.blocks.pop())
+        if slot < 0 and self.slot >= 0:
+            self.cache.slot_allocator.free(self.slot)
+            self.slot = -1
+
     def advance(self, n: int) -> None:
         self.length += n
 
@@ -173,11 +181,7 @@ class RaggedBatch:
                 taken.append((s, before))
         except Exception:
             for s, (nb, slot) in taken:        # a step that does not fit leaves no trace
-                while len(s.blocks) > nb:
-                    cache.allocator.free(s.blocks.pop())
-                if slot < 0 and s.slot >= 0:
-                    cache.slot_allocator.free(s.slot)
-                    s.slot = -1
+                s.release_to(nb, slot)
             raise
         order = sorted(range(len(entries)), key=lambda i: len(entries[i][1]) > 1)
         self.entries = entries

@@ -54,14 +54,16 @@ class HybridEngine(EngineCore):
         logits [wanted, vocab] on the device in the order of the entries and of their wanted places, or None. ``keep=False``
         may return a buffer that the next step overwrites."""
         V = self.vocab_size
-        for _, toks in entries:
-            if any(t < 0 or t >= V for t in toks):
-                raise ValueError("execute: token id outside [0, vocab_size)")
+        if any(len(t) and (min(t) < 0 or max(t) >= V) for _, t in entries):
+            raise ValueError("execute: token id outside [0, vocab_size)")
         if not entries:
             return None
         # a position's place in a captured launch is bounded by the tables, so every sequence of the engine fits a graph
-        if self.use_cuda_graph and all(len(t) == 1 for _, t in entries) and len(entries) <= self.BUCKETS[-1]:
-            logits = self._execute_captured(entries)
+        if self.use_cuda_graph and len(entries) <= self.BUCKETS[-1] and all(len(t) == 1 for _, t in entries):
+            seqs = [s for s, _ in entries]
+            if len(set(map(id, seqs))) != len(seqs):
+                raise ValueError("execute: a sequence appears twice")
+            logits = self._execute_captured(seqs, [t[0] for _, t in entries])
             rows = [i for i, w in enumerate(want) for _ in w]
             if not rows:
                 return None
@@ -73,32 +75,29 @@ class HybridEngine(EngineCore):
         batch.commit()
         return logits
 
-    def _execute_captured(self, entries) -> torch.Tensor:
-        done = []
+    def _execute_captured(self, seqs, tokens) -> torch.Tensor:
+        bs, done = self.cfg.block_size, []
         try:
-            for s, _ in entries:
-                before = (len(s.blocks), s.slot)
-                s.reserve(1)
-                done.append((s, before))
+            for s in seqs:
+                if s.slot < 0 or s.length >= len(s.blocks) * bs:      # (most tokens land in a page the sequence has)
+                    before = (s, len(s.blocks), s.slot)
+                    s.reserve(1)
+                    done.append(before)
         except Exception:
-            for s, (nb, slot) in done:
-                while len(s.blocks) > nb:
-                    self.allocator.free(s.blocks.pop())
-                if slot < 0 and s.slot >= 0:
-                    self.cache.slot_allocator.free(s.slot)
-                    s.slot = -1
+            for s, nb, slot in done:               # a step that does not fit leaves no trace
+                s.release_to(nb, slot)
             raise
-        A = self._bucket(len(entries))
+        A = self._bucket(len(seqs))
         g = self._graphs.get(A) or self._capture(A)
         if g["copied"] is not None:
             g["copied"].synchronize()            # the host buffer is free again
-        DecodeBatch.fill(g["host"].numpy(), self.cache, [s for s, _ in entries], [t[0] for _, t in entries])
+        DecodeBatch.fill(g["host_np"], self.cache, seqs, tokens)
         g["inp"].copy_(g["host"], non_blocking=True)
         g["copied"] = g["copied"] or torch.cuda.Event()
         g["copied"].record()
         g["graph"].replay()
-        for s, _ in entries:
-            s.advance(1)
+        for s in seqs:
+            s.length += 1
         return g["logits"]
 
     def _capture(self, A: int) -> dict:
@@ -106,7 +105,7 @@ class HybridEngine(EngineCore):
         dev = self.device
         host = torch.zeros((A, DecodeBatch.HEAD + self.max_blocks), dtype=torch.int32).pin_memory()
         DecodeBatch.fill(host.numpy(), self.cache, [], [])
-        g = {"host": host, "inp": host.to(dev), "copied": None}
+        g = {"host": host, "host_np": host.numpy(), "inp": host.to(dev), "copied": None}
 
         def run():
             return self.model.forward_ragged(DecodeBatch(g["inp"], self.cache.max_len).unpack(), self.cache)
