@@ -128,8 +128,8 @@ def ensure(group: str) -> Path:
 
     if CUDA_LIB.exists():
         return CUDA_LIB
-    LIB_DIR.mkdir(parents=True, exist_ok=True)
-    with open(LIB_DIR / f".{group}.lock", "w") as lock:
+    OBJ_DIR.mkdir(parents=True, exist_ok=True)
+    with open(OBJ_DIR / f"{group}.lock", "w") as lock:
         fcntl.flock(lock, fcntl.LOCK_EX)
         return build_cuda(group=group)
 
