@@ -6,7 +6,7 @@ the trace asks for are written out. Nothing is sampled.
 DIR holds config.json and model.safetensors; the model class comes from the registry. Steps are read from standard input,
 one JSON object a line:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["b"]}
+    {"step": 4, "entries": [{"id": "q7", "tokens": [11, 2], "want": [1]}, {"id": "q9", "tokens": [8], "want": []}], "end": ["q7"]}
 
 All entries of a step are one batch. ``want`` lists places among an entry's tokens; their logits go to OUT/<step>.f32
 (little-endian fp32 [wanted, vocab], entry order). A request is admitted at its first entry and gives back its pages and
