@@ -32,9 +32,10 @@ OBJ_DIR = PKG.parent / "build" / "obj"
 CUDA_LIB = LIB_DIR / "libtesseract_b200_cuda.so"
 
 # translation units of one model family: what its kernels are in and what those link against
+_HYBRID = ("runtime", "gemm_tcgen05", "gemm_decode_wq", "gemm_decode_mx", "flash_attn_fwd", "dyn_tanh", "sampling")
 GROUPS = {
-    "hybrid": ("runtime", "gemm_tcgen05", "gemm_decode_wq", "gemm_decode_mx", "decode_attn", "decode_attn_mma", "flash_attn_fwd",
-               "ragged_attn", "delta_rule", "dyn_tanh", "sampling"),
+    "fozelix": _HYBRID + ("decode_attn", "decode_attn_mma", "ragged_attn", "delta_rule"),
+    "polosun": _HYBRID + ("depth_residual", "latent_attn", "retention", "rglru"),
 }
 
 NVCC_FLAGS = [

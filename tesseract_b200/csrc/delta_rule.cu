@@ -7,7 +7,7 @@
 // divided by its root mean square over vdim, scaled by a weight and by SiLU of a gate projection.
 //
 // Prompt rows take four launches: `delta_prepare_kernel` (convolution, unit vectors, gates; every token in parallel),
-// `delta_conv_state_kernel` (the convolution's tail of each sequence goes to its slot), `delta_scan_kernel` (the
+// `conv_state_kernel` (the convolution's tail of each sequence goes to its slot), `delta_scan_kernel` (the
 // recurrence) and `delta_gate_norm_kernel`. Decoded rows take one: `delta_step_kernel` does all of it for one token,
 // streaming the state through registers once.
 //
@@ -22,7 +22,7 @@
 // Packed projection row (element offsets, sections padded to multiples of 8):
 //   [ q: Hk * dim | k: Hk * dim | v: H * vdim | gate: H * vdim | b: H | a: H ]
 // A slot's convolution state holds the last taps - 1 rows of the first three sections, in the projection's type.
-#include "common.cuh"
+#include "ragged_conv.cuh"
 
 #include <algorithm>
 #include <cstdlib>
@@ -276,30 +276,6 @@ delta_prepare_kernel(DeltaPrepParams p) {
           if (i < valid) vr[static_cast<long long>((c + i) / g.vdim) * g.vp + (c + i) % g.vdim] = y[t][i];
       }
     }
-  }
-}
-
-// The last taps - 1 inputs of every sequence -> its slot. Runs after the prepare kernel has read the old contents; one
-// thread owns one channel of one sequence, and walks up, so a short portion may shift the slot in place.
-template <typename T>
-__global__ void __launch_bounds__(256)
-delta_conv_state_kernel(DeltaGeom g, const T* proj, T* conv_state, const int* cu, const int* slots, const int* pos0, int tail) {
-  pdl_trigger();
-  pdl_grid_wait();
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  const int seq = blockIdx.y;
-  if (c >= g.conv_c) return;
-  const int row0 = cu[seq], n = cu[seq + 1] - row0;
-  const int slot = slots[seq];
-  if (slot < 0 || n <= 0) return;
-  const bool has_state = pos0[seq] > 0;
-  T* st = conv_state + static_cast<long long>(slot) * tail * g.conv_c + c;
-  for (int j = 0; j < tail; ++j) {
-    const int i = n - tail + j;            // token of this portion whose input belongs in place j
-    T val = from_f32<T>(0.f);
-    if (i >= 0) val = proj[static_cast<long long>(row0 + i) * g.ldp + c];
-    else if (has_state) val = st[static_cast<long long>(j + n) * g.conv_c];
-    st[static_cast<long long>(j) * g.conv_c] = val;
   }
 }
 
@@ -955,10 +931,10 @@ TSB_EXPORT int tsb_delta_prefill(const void* proj, long long ldp, const int* geo
   if (taps > 1) {
     const dim3 grid((g.conv_c + 255) / 256, nseq);
     if (dtype == 1)
-      launch_pdl(delta_conv_state_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl, g, static_cast<const __nv_bfloat16*>(proj),
+      launch_pdl(conv_state_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl, static_cast<const __nv_bfloat16*>(proj), g.ldp, g.conv_c,
                  static_cast<__nv_bfloat16*>(conv_state), cu, slots, pos0, taps - 1);
     else
-      launch_pdl(delta_conv_state_kernel<float>, grid, dim3(256), 0, s, pdl, g, static_cast<const float*>(proj),
+      launch_pdl(conv_state_kernel<float>, grid, dim3(256), 0, s, pdl, static_cast<const float*>(proj), g.ldp, g.conv_c,
                  static_cast<float*>(conv_state), cu, slots, pos0, taps - 1);
     rc = static_cast<int>(cudaGetLastError());
     if (rc) return rc;

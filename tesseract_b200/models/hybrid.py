@@ -1,6 +1,14 @@
 """Decoders that mix recurrent and attention layers, described by a list: every layer has a mixer and, optionally, a
-feed-forward, both normed before and after; a range of layers may run several times in a row with the same weights and
-separate caches ("loop"). Embedding and output share one table.
+feed-forward. Two forms of layer:
+
+* ``sandwich``: mixer, then feed-forward, each normed before and after by Dynamic Tanh; a range of layers may run several
+  times in a row with the same weights and separate caches ("loop");
+* ``parallel``: mixer and feed-forward of the same x side by side, x + m (mixer(norm1 x) + ff(norm2 x)), normed by RMS with one
+  gain. The gains ride on the sublayers (``in_scale``), so one normed row feeds one product for both, and one product takes
+  both results back. Optionally every layer hands on a weighted sum of the embedding output and all layers' results so far
+  ("depth average").
+
+Embedding and output share one table, or the output has its own.
 
 ``HybridModel`` runs ragged batches (``forward_ragged``: any mix of prompt portions and decoded tokens) over a
 ``HybridCache``. The serving engine drives that step; ``forward_step`` / ``forward_step_batched`` give it the interface
@@ -14,8 +22,10 @@ from typing import Callable, Dict, List, Optional, Union
 import torch
 
 from .. import ops
-from ..nn.hybrid import ChunkedAttention, ClampedGLU, DynamicTanh, GatedDelta, pad_to
+from ..nn.hybrid import (RGLRU, ChunkedAttention, ClampedGLU, DynamicTanh, GatedDelta, LatentAttention, Retention, ScalarRMSNorm,
+                         SiluGLU, pad_to)
 from ..nn.ragged import HybridCache, HybridSequence, RaggedBatch
+from ..ops.rotary import Rotary, Yarn
 from .llama import GenerateConfig, pick_next_token
 
 
@@ -39,15 +49,47 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
+class LatentSpec:
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rotary: Rotary
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+    rotary: Rotary
+
+
+@dataclass(frozen=True)
+class RGLRUSpec:
+    width: int
+    blocks: int
+    conv: int
+
+
+@dataclass(frozen=True)
 class GLUSpec:
     ff: int
     limit: float
 
 
 @dataclass(frozen=True)
+class SiluGLUSpec:
+    ff: int
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, DeltaSpec]
-    mlp: Optional[GLUSpec] = None
+    mixer: Union[AttentionSpec, DeltaSpec, LatentSpec, RetentionSpec, RGLRUSpec]
+    mlp: Union[GLUSpec, SiluGLUSpec, None] = None
 
 
 @dataclass(frozen=True)
@@ -68,8 +110,12 @@ class HybridConfig:
     dtype: torch.dtype = torch.bfloat16
     bos_token_id: int = -1
     eos_token_id: int = -1
-    max_position_embeddings: int = 1 << 20     # no positions enter the model: a bound for caches only
+    max_position_embeddings: int = 1 << 20     # a bound for caches only
     architecture: str = ""
+    form: str = "sandwich"                     # or "parallel"
+    residual_mult: float = 1.0                 # (parallel)
+    depth_average: bool = False                # (parallel)
+    tied: bool = True                          # the output product uses the embedding table
 
     def __post_init__(self):
         if self.vocab_size < 1 or self.width < 1 or not self.layers:
@@ -79,6 +125,12 @@ class HybridConfig:
             raise ValueError("HybridConfig: loop must name a range of layers and run at least once")
         if self.dtype not in (torch.bfloat16, torch.float32):
             raise ValueError("HybridConfig: dtype is bfloat16 or float32")
+        if self.form not in ("sandwich", "parallel"):
+            raise ValueError(f"HybridConfig: unknown form {self.form!r}")
+        if self.form == "parallel" and (lp is not None or self.embedding_scale != 1.0):
+            raise ValueError("HybridConfig: parallel layers take no loop and no embedding scale")
+        if self.form == "sandwich" and (self.residual_mult != 1.0 or self.depth_average):
+            raise ValueError("HybridConfig: a residual multiplier and depth averaging belong to parallel layers")
 
     def runs(self):
         """[(layer, pass)] in the order they run; pass is -1 outside the loop."""
@@ -90,18 +142,35 @@ class HybridConfig:
                 + [(i, -1) for i in range(lp.stop, n)])
 
 
-class _Layer:
-    def __init__(self, spec: LayerSpec, c: HybridConfig, device):
-        m, W, dt = spec.mixer, c.width, c.dtype
-        if isinstance(m, AttentionSpec):
-            self.mixer = ChunkedAttention(W, m.heads, m.kv_heads, m.dim, m.vdim, m.scale, m.chunk, dt, device)
-        else:
-            self.mixer = GatedDelta(W, m.heads, m.kv_heads, m.dim, m.vdim, m.conv, c.eps, dt, device)
-        self.norm1, self.norm1b = DynamicTanh(W, dt, device), DynamicTanh(W, dt, device)
-        self.mlp = self.norm2 = self.norm2b = None
-        if spec.mlp is not None:
-            self.mlp = ClampedGLU(W, spec.mlp.ff, spec.mlp.limit, dt, device)
-            self.norm2, self.norm2b = DynamicTanh(W, dt, device), DynamicTanh(W, dt, device)
+def _make_mixer(m, c: HybridConfig, device):
+    W, dt = c.width, c.dtype
+    if isinstance(m, AttentionSpec):
+        return ChunkedAttention(W, m.heads, m.kv_heads, m.dim, m.vdim, m.scale, m.chunk, dt, device)
+    if isinstance(m, DeltaSpec):
+        return GatedDelta(W, m.heads, m.kv_heads, m.dim, m.vdim, m.conv, c.eps, dt, device)
+    if isinstance(m, LatentSpec):
+        return LatentAttention(W, m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.scale, m.rotary, c.eps, dt, device)
+    if isinstance(m, RetentionSpec):
+        return Retention(W, m.heads, m.dim, m.vdim, m.decay, m.rotary, c.eps, dt, device)
+    if isinstance(m, RGLRUSpec):
+        return RGLRU(W, m.width, m.blocks, m.conv, dt, device)
+    raise ValueError(f"HybridConfig: unknown mixer {m!r}")
+
+
+def _make_mlp(m, c: HybridConfig, device):
+    if m is None:
+        return None
+    if isinstance(m, SiluGLUSpec):
+        return SiluGLU(c.width, m.ff, c.dtype, device)
+    return ClampedGLU(c.width, m.ff, m.limit, c.dtype, device)
+
+
+class _SandwichLayer:
+    def __init__(self, spec: LayerSpec, c: HybridConfig, index: int, device):
+        norm = lambda: DynamicTanh(c.width, c.dtype, device)   # noqa: E731
+        self.mixer, self.mlp = _make_mixer(spec.mixer, c, device), _make_mlp(spec.mlp, c, device)
+        self.norm1, self.norm1b = norm(), norm()
+        self.norm2, self.norm2b = (norm(), norm()) if spec.mlp is not None else (None, None)
 
     def parts(self):
         out = [("norm1", self.norm1), ("norm1b", self.norm1b), ("mix.", self.mixer)]
@@ -109,19 +178,73 @@ class _Layer:
             out += [("norm2", self.norm2), ("norm2b", self.norm2b), ("mlp.", self.mlp)]
         return out
 
+    extra = {}
+
+
+class _ParallelLayer:
+    """One input matrix (rows of the mixer, then of the feed-forward) and one output matrix (columns likewise)."""
+
+    def __init__(self, spec: LayerSpec, c: HybridConfig, index: int, device):
+        self.mixer, self.mlp = _make_mixer(spec.mixer, c, device), _make_mlp(spec.mlp, c, device)
+        self.norm1 = ScalarRMSNorm(c.eps, c.dtype, device)
+        self.norm2 = ScalarRMSNorm(c.eps, c.dtype, device) if spec.mlp is not None else None
+        subs = [s for s in (self.mixer, self.mlp) if s is not None]
+        for s in subs:
+            if not s.takes_in_scale or s.out_bias is not None:
+                raise ValueError(f"HybridConfig: {type(s).__name__} does not run in parallel layers")
+        self.in_cut, self.out_cut = self.mixer.cols, self.mixer.out_cols
+        if self.mlp is None:
+            self.w_in, self.w_out = self.mixer.w_in, self.mixer.w_out
+        else:
+            new = lambda *shape: torch.zeros(shape, dtype=c.dtype, device=device)   # noqa: E731
+            self.w_in = new(sum(s.cols for s in subs), self.mixer.w_in.shape[1])
+            self.w_out = new(c.width, sum(s.out_cols for s in subs))
+            self.mixer.place(self.w_in[:self.in_cut], self.w_out[:, :self.out_cut])
+            self.mlp.place(self.w_in[self.in_cut:], self.w_out[:, self.out_cut:])
+        self.average = torch.zeros(index + 2, dtype=torch.float32, device=device) if c.depth_average else None
+        self.extra = {"dwa": self.average} if c.depth_average else {}
+
+    def parts(self):
+        out = [("norm1", self.norm1), ("mix.", self.mixer)]
+        if self.mlp is not None:
+            out += [("norm2", self.norm2), ("mlp.", self.mlp)]
+        return out
+
+    def set_gains(self) -> None:
+        self.mixer.in_scale = self.norm1.gain
+        if self.mlp is not None:
+            self.mlp.in_scale = self.norm2.gain
+
+    def forward(self, h, storage, batch):
+        """h: the normed row without a gain."""
+        p = ops.project(h, self.w_in)
+        if self.mlp is None:
+            return ops.project(self.mixer.core(p, storage, batch), self.w_out)
+        z = torch.empty((h.shape[0], self.w_out.shape[1]), device=h.device, dtype=h.dtype)
+        self.mixer.core(p[:, :self.in_cut], storage, batch, out=z[:, :self.out_cut])
+        self.mlp.core(p[:, self.in_cut:], out=z[:, self.out_cut:])
+        return ops.project(z, self.w_out)
+
 
 class HybridModel:
     def __init__(self, config: HybridConfig, device=None, init_std: Optional[float] = None, seed: int = 0):
         self.config = c = config
         self.device = torch.device(device) if device is not None else torch.device("cpu")
-        # one table for the embedding and the output product; its rows are padded like every matrix the GEMMs read
+        # one table for the embedding and, unless it has its own, the output product; rows are padded like every matrix the
+        # GEMMs read
         self.embed = torch.zeros(c.vocab_size, pad_to(c.width), dtype=c.dtype, device=self.device)
-        self.layers = [_Layer(s, c, self.device) for s in c.layers]
-        self.final_norm = DynamicTanh(c.width, c.dtype, self.device)
+        self.head = self.embed if c.tied else torch.zeros_like(self.embed)
+        layer = _SandwichLayer if c.form == "sandwich" else _ParallelLayer
+        self.layers = [layer(s, c, i, self.device) for i, s in enumerate(c.layers)]
+        self.final_norm = (DynamicTanh(c.width, c.dtype, self.device) if c.form == "sandwich"
+                           else ScalarRMSNorm(c.eps, c.dtype, self.device))
         self.loop_step = (torch.zeros(c.loop.times, c.width, dtype=torch.float32, device=self.device)
                           if c.loop is not None else None)
         self.runs = c.runs()
-        self.chunks = sorted({s.mixer.chunk for s in c.layers if isinstance(s.mixer, AttentionSpec)})
+        # what the mixers ask a batch for: masks of prompt attention, sizes of prompt tiles
+        self.chunks = sorted({s.mixer.chunk if isinstance(s.mixer, AttentionSpec) else 0
+                              for s in c.layers if isinstance(s.mixer, (AttentionSpec, LatentSpec))})
+        self.tiles = sorted({l.mixer.tile for l in self.layers if l.mixer.tile})
         if init_std is not None:
             self.init_weights(init_std, seed)
 
@@ -133,9 +256,8 @@ class HybridModel:
         return self
 
     def parameters(self):
-        yield self.embed
-        if self.loop_step is not None:
-            yield self.loop_step
+        for _, t in self._tables():
+            yield t
         for _, part in self._parts():
             yield from part.tensors()
 
@@ -153,11 +275,22 @@ class HybridModel:
                 yield f"l{i}.{name}", part
         yield "final.norm", self.final_norm
 
+    def _tables(self):
+        """Tensors of the model itself: (name, packed tensor; its first columns are the logical ones)."""
+        yield "embed", self.embed
+        if not self.config.tied:
+            yield "head", self.head
+        if self.loop_step is not None:
+            yield "loop.step", self.loop_step
+        for i, l in enumerate(self.layers):
+            for name, t in l.extra.items():
+                yield f"l{i}.{name}", t
+
+    def _logical(self, t: torch.Tensor) -> torch.Tensor:
+        return t[:, :self.config.width] if t.dim() == 2 else t
+
     def logical_shapes(self) -> Dict[str, tuple]:
-        c = self.config
-        out = {"embed": (c.vocab_size, c.width)}
-        if c.loop is not None:
-            out["loop.step"] = (c.loop.times, c.width)
+        out = {name: tuple(self._logical(t).shape) for name, t in self._tables()}
         for name, part in self._parts():
             out.update({name + k: tuple(v) for k, v in part.logical_shapes().items()})
         return out
@@ -165,28 +298,25 @@ class HybridModel:
     @torch.no_grad()
     def load_tensors(self, sd: Dict[str, torch.Tensor]) -> list:
         """Packs a dict of logical tensors; returns the names in it that the model does not have."""
-        c = self.config
         known = self.logical_shapes()
-        for name in ("embed", "loop.step"):
-            if name in known:
-                if name not in sd:
-                    raise KeyError(f"load: required tensor {name!r} is missing")
-                if tuple(sd[name].shape) != known[name]:
-                    raise ValueError(f"load: shape of {name!r} is {tuple(sd[name].shape)}, expected {known[name]}")
-        self.embed[:, :c.width].copy_(sd["embed"])
-        if self.loop_step is not None:
-            self.loop_step.copy_(sd["loop.step"])
+        for name, t in self._tables():
+            if name not in sd:
+                raise KeyError(f"load: required tensor {name!r} is missing")
+            if tuple(sd[name].shape) != known[name]:
+                raise ValueError(f"load: shape of {name!r} is {tuple(sd[name].shape)}, expected {known[name]}")
+            self._logical(t).copy_(sd[name])
         for name, part in self._parts():
             try:
                 part.load({k: sd[name + k] for k in part.logical_shapes() if name + k in sd})
             except (KeyError, ValueError, TypeError) as e:
                 raise type(e)(f"{name}: {e.args[0]}") from None
+        if self.config.form == "parallel":
+            for l in self.layers:
+                l.set_gains()
         return [k for k in sd if k not in known]
 
     def state_tensors(self) -> Dict[str, torch.Tensor]:
-        out = {"embed": self.embed[:, :self.config.width].contiguous()}
-        if self.loop_step is not None:
-            out["loop.step"] = self.loop_step.to(self.config.dtype)
+        out = {name: self._logical(t).to(self.config.dtype).contiguous() for name, t in self._tables()}
         for name, part in self._parts():
             out.update({name + k: v for k, v in part.unpack().items()})
         return out
@@ -202,14 +332,23 @@ class HybridModel:
 
     @torch.no_grad()
     def init_weights(self, std: float = 0.02, seed: int = 0) -> None:
-        """N(0, std) matrices from a fixed seed; norms start as tanh(x), decays between slow and fast."""
+        """N(0, std) matrices from a fixed seed; norms start with unit gains, decays between slow and fast, and a depth average
+        passes the newest result on."""
         gen = torch.Generator(device=self.device)
         gen.manual_seed(seed)
 
         def draw(name, shape):
             last = name.rsplit(".", 1)[-1]
-            if last == "alpha":
+            if last == "alpha" or shape == ():
                 return torch.tensor(1.0)
+            if last == "dwa":
+                return torch.eye(shape[0])[-1]
+            if len(shape) == 3:
+                return torch.randn(shape, generator=gen, device=self.device) * shape[-1] ** -0.5
+            if last == "lam":
+                return torch.rand(shape, generator=gen, device=self.device) * 3.0 - 4.0
+            if last == "b":
+                return torch.zeros(shape)
             if len(shape) == 2:
                 s = 0.5 if last == "conv" else std
                 return torch.randn(shape, generator=gen, device=self.device) * s
@@ -217,8 +356,6 @@ class HybridModel:
                 return torch.rand(shape, generator=gen, device=self.device) * 2.0 - 2.0
             if last == "dt_bias":
                 return torch.rand(shape, generator=gen, device=self.device) - 3.0
-            if last == "b":
-                return torch.zeros(shape)
             return torch.ones(shape)
         self.load_tensors({n: draw(n, s) for n, s in self.logical_shapes().items()})
 
@@ -229,12 +366,21 @@ class HybridModel:
         return HybridCache(specs, num_blocks, block_size, max_sequences, max_len, self.config.dtype, self.device)
 
     def make_batch(self, cache: HybridCache, entries, want=None, max_len: int = 0) -> RaggedBatch:
-        return RaggedBatch(cache, entries, want, self.chunks, max_len)
+        return RaggedBatch(cache, entries, want, self.chunks, max_len, self.tiles)
 
     @torch.no_grad()
     def forward_ragged(self, batch, cache: HybridCache, on_layer: Optional[Callable] = None) -> Optional[torch.Tensor]:
         """Runs one step over the cache; fp32 logits [wanted rows, vocab] (None when nothing is wanted). ``on_layer`` is
         called with (run, residual) after every layer run, before what comes ahead of the next pass."""
+        run = self._run_sandwich if self.config.form == "sandwich" else self._run_parallel
+        h = run(batch, cache, on_layer)
+        if batch.n_want == 0:
+            return None
+        if batch.want is not None:
+            h = h.index_select(0, batch.want)
+        return ops.project(h, self.head, out_dtype=torch.float32)
+
+    def _run_sandwich(self, batch, cache: HybridCache, on_layer) -> torch.Tensor:
         c = self.config
         x = torch.empty((batch.rows, c.width), device=self.device, dtype=torch.float32)
         Kp, emb = pad_to(c.width), dict(tokens=batch.tokens, table=self.embed, scale=c.embedding_scale)
@@ -270,11 +416,23 @@ class HybridModel:
                 on_layer(r, x)
                 y = bias = post = None
             h = step(y, bias, post, add, norm)
-        if batch.n_want == 0:
-            return None
-        if batch.want is not None:
-            h = h.index_select(0, batch.want)
-        return ops.project(h, self.embed, out_dtype=torch.float32)
+        return h
+
+    def _run_parallel(self, batch, cache: HybridCache, on_layer) -> torch.Tensor:
+        c = self.config
+        n = len(self.layers)
+        form = dict(out_cols=pad_to(c.width), out_dtype=c.dtype, eps=c.eps)
+        # what the depth average looks back on: the embedding output and every layer's result
+        history = (torch.empty((n, batch.rows, c.width), device=self.device, dtype=torch.float32) if c.depth_average else None)
+        x, h = ops.depth_residual(tokens=batch.tokens, table=self.embed, width=c.width, history=history, **form)
+        for r, l in enumerate(self.layers):
+            y = l.forward(h, cache.runs[r], batch)
+            last = r == n - 1
+            x, h = ops.depth_residual(x, y, c.residual_mult, history=history, depth=r + 1, average=l.average, store=not last,
+                                      gain=self.final_norm.gain if last else 1.0, **form)
+            if on_layer is not None:
+                on_layer(r, x)
+        return h
 
     # ------------------------------------------------------------------ interface of the per-request schedulers
     def make_layer_pools(self, num_blocks: int, block_size: int, max_sequences: int = 16, max_len: int = 0) -> list:
@@ -337,4 +495,5 @@ class HybridModel:
         return eng.result(rid)
 
 
-__all__ = ["AttentionSpec", "DeltaSpec", "GLUSpec", "LayerSpec", "LoopSpec", "HybridConfig", "HybridModel", "pick_next_token"]
+__all__ = ["AttentionSpec", "DeltaSpec", "GLUSpec", "HybridConfig", "HybridModel", "LatentSpec", "LayerSpec", "LoopSpec", "RGLRUSpec",
+           "RetentionSpec", "Rotary", "SiluGLUSpec", "Yarn", "pick_next_token"]

@@ -20,6 +20,7 @@ class Architecture:
     matches: Callable[[dict], bool]
     config: Callable          # (parsed config, dtype) -> configuration object
     build: Callable           # (configuration object, device) -> model with load_safetensors
+    kernels: str = ""         # group of translation units that serves it (build.GROUPS); empty: the whole library
 
 
 _REGISTRY: List[Architecture] = []
@@ -99,5 +100,18 @@ def _fozelix_build(cfg, device):
     return fozelix.build(cfg, device)
 
 
+def _polosun_config(obj: dict, dtype: torch.dtype):
+    from . import polosun
+    return polosun.config_from_dict(obj, dtype)
+
+
+def _polosun_build(cfg, device):
+    from . import polosun
+    return polosun.build(cfg, device)
+
+
 register(Architecture("Llama", _is_llama, _llama_config, _llama_build))
-register(Architecture("Fozelix", lambda o: o.get("architecture") == "Fozelix", _fozelix_config, _fozelix_build))
+register(Architecture("Fozelix", lambda o: o.get("architecture") == "Fozelix", _fozelix_config, _fozelix_build,
+                      kernels="fozelix"))
+register(Architecture("Polosun", lambda o: o.get("architecture") == "Polosun", _polosun_config, _polosun_build,
+                      kernels="polosun"))

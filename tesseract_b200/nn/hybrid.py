@@ -1,5 +1,10 @@
-"""Building blocks of hybrid decoders for inference over ragged batches: Dynamic Tanh norms, chunked attention, the gated
-delta rule and the clamped GLU feed-forward.
+"""Building blocks of hybrid decoders for inference over ragged batches: norms (Dynamic Tanh, RMS with one gain), mixers
+(chunked attention, latent attention, the gated delta rule, retention, the real-gated linear recurrence) and gated
+feed-forwards (clamped, SiLU).
+
+A mixer or feed-forward is two matrix products around a ``core``: rows of ``w_in`` make its packed input, ``w_out`` takes what
+the core leaves. Layers whose sublayers run side by side lay several of them into one matrix (``place``) and call the cores on
+columns of the shared product.
 
 A block holds its parameters packed for the kernels (adjacent projections in one matrix, sections and heads padded with
 zeros, everything that the kernels use in fp32 already widened) and translates to and from its logical tensors:
@@ -13,8 +18,12 @@ import torch
 
 from .. import ops
 from ..ops.delta import DeltaGeometry, DeltaWeights, gated_delta
+from ..ops.latent import LatentGeometry, LatentWeights, latent_attention
 from ..ops.ragged import padded_head_dim, ragged_attention
-from .ragged import PagedRun, StateRun
+from ..ops.retention import SPAN, RetentionGeometry, log2_decays, retention
+from ..ops.rglru import CHUNK, RGLRUGeometry, RGLRUWeights, rglru
+from ..ops.rotary import Rotary
+from .ragged import LatentRun, PagedRun, StateRun
 
 
 def pad_to(n: int, m: int = 16) -> int:
@@ -40,6 +49,56 @@ class _Packed:
             if not t[name].is_floating_point():
                 raise TypeError(f"load: {name!r} is not a floating-point tensor")
         self._pack(t)
+
+
+class _Sublayer(_Packed):
+    """Two products around a core. ``in_scale`` multiplies the packed input inside the core: the gain of a norm that has only
+    one, where the layer leaves it to the sublayers. ``tile``: size of the prompt tiles that the core asks the batch for."""
+    out_bias = None
+    in_scale = 1.0
+    takes_in_scale = False
+    tile = 0
+
+    @property
+    def cols(self) -> int:
+        return self.w_in.shape[0]
+
+    @property
+    def out_cols(self) -> int:
+        return self.w_out.shape[1]
+
+    def place(self, w_in: torch.Tensor, w_out: torch.Tensor) -> None:
+        """Moves the two matrices into rows and columns of larger ones."""
+        w_in.copy_(self.w_in)
+        w_out.copy_(self.w_out)
+        self.w_in, self.w_out = w_in, w_out
+
+
+class _Mixer(_Sublayer):
+    def forward(self, h, storage, batch):
+        return ops.project(self.core(ops.project(h, self.w_in), storage, batch), self.w_out)
+
+
+class _FeedForward(_Sublayer):
+    def forward(self, h):
+        return ops.project(self.core(ops.project(h, self.w_in)), self.w_out)
+
+
+class ScalarRMSNorm(_Packed):
+    """x / sqrt(mean(x^2) + eps) * gain with one gain for all channels."""
+
+    def __init__(self, eps: float, dtype, device):
+        super().__init__(dtype, device)
+        self.eps, self.gain = float(eps), 1.0
+
+    def logical_shapes(self):
+        return {"": ()}
+
+    def _pack(self, t):
+        self.gain = float(t[""])
+
+    def unpack(self):
+        return {"": torch.tensor(self.gain, dtype=self.dtype, device=self.device)}
 
 
 class DynamicTanh(_Packed):
@@ -68,7 +127,7 @@ class DynamicTanh(_Packed):
         return self.alpha, self.weight, self.bias
 
 
-class ChunkedAttention(_Packed):
+class ChunkedAttention(_Mixer):
     """Grouped-query attention without positions whose mask is causal inside runs of ``chunk`` positions (0: causal over
     everything); biases on q, k and v. Query / key heads are ``dim`` wide, value heads ``vdim``."""
 
@@ -82,8 +141,6 @@ class ChunkedAttention(_Packed):
         self.w_in = self._zeros((heads + 2 * kv_heads) * self.D, pad_to(width))
         self.b_in = self._zeros((heads + 2 * kv_heads) * self.D, dtype=torch.float32)
         self.w_out = self._zeros(width, heads * self.D)
-
-    out_bias = None
 
     def run_spec(self) -> PagedRun:
         return PagedRun(self.kv_heads, self.D)
@@ -121,13 +178,11 @@ class ChunkedAttention(_Packed):
         out["o"] = self.w_out.view(self.width, self.heads, self.D)[:, :, :self.vdim].reshape(self.width, -1)
         return out
 
-    def forward(self, h, storage, batch):
-        qkv = ops.project(h, self.w_in)
-        o = ragged_attention(qkv, self.b_in, storage[0], storage[1], batch, self.heads, self.kv_heads, self.scale, self.chunk)
-        return ops.project(o, self.w_out)
+    def core(self, qkv, storage, batch):
+        return ragged_attention(qkv, self.b_in, storage[0], storage[1], batch, self.heads, self.kv_heads, self.scale, self.chunk)
 
 
-class GatedDelta(_Packed):
+class GatedDelta(_Mixer):
     """The gated delta rule with short convolutions (see ``ops.delta``)."""
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, conv: int, eps: float, dtype, device):
@@ -139,8 +194,6 @@ class GatedDelta(_Packed):
         f32 = torch.float32
         self.w = DeltaWeights(self._zeros(conv, g.conv_cols, dtype=f32), self._zeros(heads, dtype=f32),
                               self._zeros(heads, dtype=f32), self._zeros(vdim, dtype=f32), float(eps))
-
-    out_bias = None
 
     def tensors(self):
         return super().tensors() + [self.w.conv, self.w.a_log, self.w.dt_bias, self.w.norm]
@@ -185,12 +238,11 @@ class GatedDelta(_Packed):
                     "norm": self.w.norm.to(self.dtype), "o": self.w_out[:, :self.geo.heads * self.geo.vdim].contiguous()})
         return out
 
-    def forward(self, h, storage, batch):
-        y = gated_delta(ops.project(h, self.w_in), self.geo, self.w, storage[0], storage[1], batch)
-        return ops.project(y, self.w_out)
+    def core(self, proj, storage, batch):
+        return gated_delta(proj, self.geo, self.w, storage[0], storage[1], batch)
 
 
-class ClampedGLU(_Packed):
+class ClampedGLU(_FeedForward):
     """g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit); W_down (g sigmoid(slope g) (u + 1)), biases on all three.
     The bias of the last product is left to the residual step (``out_bias``)."""
 
@@ -222,5 +274,225 @@ class ClampedGLU(_Packed):
         out["down"], out["down.b"] = self.w_out[:, :self.ff].contiguous(), self.out_bias.to(self.dtype)
         return out
 
-    def forward(self, h):
-        return ops.project(ops.clamped_glu(ops.project(h, self.w_in), self.b_in, self.limit, self.slope), self.w_out)
+    def core(self, gate_up, out=None):
+        return ops.clamped_glu(gate_up, self.b_in, self.limit, self.slope, out=out)
+
+
+class SiluGLU(_FeedForward):
+    """W_down (silu(W_gate h) * (W_up h)) without biases."""
+    takes_in_scale = True
+
+    def __init__(self, width: int, ff: int, dtype, device):
+        super().__init__(dtype, device)
+        if ff < 1:
+            raise ValueError("feed-forward: ff must be positive")
+        self.width, self.ff = width, ff
+        self.F = F = pad_to(ff)
+        self.w_in, self.w_out = self._zeros(2 * F, pad_to(width)), self._zeros(width, F)
+
+    def logical_shapes(self):
+        return {"gate": (self.ff, self.width), "up": (self.ff, self.width), "down": (self.width, self.ff)}
+
+    def _pack(self, t):
+        for name, at in (("gate", 0), ("up", self.F)):
+            self.w_in[at:at + self.ff, :self.width].copy_(t[name])
+        self.w_out[:, :self.ff].copy_(t["down"])
+
+    def unpack(self):
+        out = {name: self.w_in[at:at + self.ff, :self.width].contiguous() for name, at in (("gate", 0), ("up", self.F))}
+        out["down"] = self.w_out[:, :self.ff].contiguous()
+        return out
+
+    def core(self, gate_up, out=None):
+        return ops.silu_glu(gate_up, self.in_scale, out)
+
+
+def _head_rows(at: int, heads: int, stride: int, columns: torch.Tensor) -> torch.Tensor:
+    """Packed row of every coordinate of a section of heads: ``columns`` places a head's coordinates inside its ``stride``."""
+    return (at + torch.arange(heads)[:, None] * stride + columns[None, :]).reshape(-1)
+
+
+class _RowPacked(_Mixer):
+    """A mixer whose projections are rows of ``w_in`` at places given by index (``_rows``: name -> packed row of every logical
+    row), and whose output product reads columns ``_out_columns()``."""
+
+    def _pack_rows(self, t):
+        for name, rows in self._rows().items():
+            self.w_in[rows.to(self.device), :self.width] = t[name].to(self.device, self.dtype)
+        self.w_out[:, self._out_columns().to(self.device)] = t["o"].to(self.device, self.dtype)
+
+    def _unpack_rows(self):
+        out = {name: self.w_in[rows.to(self.device), :self.width] for name, rows in self._rows().items()}
+        out["o"] = self.w_out[:, self._out_columns().to(self.device)]
+        return out
+
+    def _row_shapes(self):
+        out = {name: (len(rows), self.width) for name, rows in self._rows().items()}
+        out["o"] = (self.width, len(self._out_columns()))
+        return out
+
+
+class LatentAttention(_RowPacked):
+    """Attention whose keys and values are products of a cached latent, with a rotated key part shared by all heads and a
+    sigmoid gate on the heads (see ``ops.latent``)."""
+    takes_in_scale = True
+
+    def __init__(self, width: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float, rotary: Rotary, eps: float,
+                 dtype, device):
+        super().__init__(dtype, device)
+        self.width = width
+        self.geo = g = LatentGeometry(heads, dim, rot_dim, vdim, kv_rank, rotary)
+        self.w_in, self.w_out = self._zeros(g.cols, pad_to(width)), self._zeros(width, g.out_cols)
+        self.w = LatentWeights(self._zeros(g.cp, dtype=torch.float32), self._zeros(2 * heads * g.D, g.row),
+                               self._zeros(heads, g.cp, pad_to(dim)), float(eps), float(scale))
+        # the rows that copy the rotated part of a cached row into every head's key
+        up = self.w.w_up[:heads * g.D].view(heads, g.D, g.row)
+        for j in range(2 * rotary.hp):
+            up[:, g.np + j, g.cp + j] = 1.0
+
+    def tensors(self):
+        return super().tensors() + [self.w.norm, self.w.w_up, self.w.w_absorb]
+
+    def run_spec(self) -> LatentRun:
+        return LatentRun(self.geo.row, self.geo.rotary)
+
+    def _rows(self):
+        g = self.geo
+        rot = g.rotary.columns(g.rot_dim)
+        head = torch.cat([torch.arange(g.dim), g.np + rot])
+        down = torch.cat([torch.arange(g.kv_rank), pad_to(g.kv_rank, 8) + rot])
+        return {"q": _head_rows(0, g.heads, g.q_cols, head), "dkv": g.off_c + down,
+                "g": _head_rows(g.off_gate, g.heads, g.vp, torch.arange(g.vdim))}
+
+    def _out_columns(self):
+        return _head_rows(0, self.geo.heads, self.geo.vp, torch.arange(self.geo.vdim))
+
+    def logical_shapes(self):
+        g = self.geo
+        return {**self._row_shapes(), "dkv.norm": (g.kv_rank,), "uk": (g.heads * g.dim, g.kv_rank), "uv": (g.heads * g.vdim, g.kv_rank)}
+
+    def _up_views(self):
+        g = self.geo
+        up = self.w.w_up.view(2, g.heads, g.D, g.row)
+        return up[0, :, :g.dim, :g.kv_rank], up[1, :, :g.vdim, :g.kv_rank]
+
+    def _pack(self, t):
+        g = self.geo
+        self._pack_rows(t)
+        self.w.norm[:g.kv_rank].copy_(t["dkv.norm"])
+        k, v = self._up_views()
+        k.copy_(t["uk"].view(g.heads, g.dim, g.kv_rank))
+        v.copy_(t["uv"].view(g.heads, g.vdim, g.kv_rank))
+        self.w.w_absorb[:, :g.kv_rank, :g.dim].copy_(t["uk"].view(g.heads, g.dim, g.kv_rank).transpose(1, 2))
+
+    def unpack(self):
+        g = self.geo
+        k, v = self._up_views()
+        return {**self._unpack_rows(), "dkv.norm": self.w.norm[:g.kv_rank].to(self.dtype), "uk": k.reshape(-1, g.kv_rank),
+                "uv": v.reshape(-1, g.kv_rank)}
+
+    def core(self, proj, storage, batch, out=None):
+        return latent_attention(proj, self.geo, self.w, storage[0], storage[1], batch, self.in_scale, out)
+
+
+class Retention(_RowPacked):
+    """Linear attention with a fixed decay per head (see ``ops.retention``)."""
+    takes_in_scale = True
+    tile = SPAN
+
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, decay, rotary: Rotary, eps: float, dtype, device):
+        super().__init__(dtype, device)
+        if len(decay) != heads:
+            raise ValueError("retention: one decay per head")
+        self.width, self.eps = width, float(eps)
+        self.geo = g = RetentionGeometry(heads, dim, vdim, rotary)
+        self.w_in, self.w_out = self._zeros(g.cols, pad_to(width)), self._zeros(width, g.out_cols)
+        self.log2_decay = log2_decays(decay).to(self.device)
+
+    def run_spec(self) -> StateRun:
+        g = self.geo
+        return StateRun((g.heads, g.dp, g.vp), rotary=g.rotary)
+
+    def _rows(self):
+        g = self.geo
+        qk, v = g.rotary.columns(g.dim), torch.arange(g.vdim)
+        return {"q": _head_rows(0, g.heads, g.dp, qk), "k": _head_rows(g.off_k, g.heads, g.dp, qk),
+                "v": _head_rows(g.off_v, g.heads, g.vp, v), "g": _head_rows(g.off_gate, g.heads, g.vp, v)}
+
+    def _out_columns(self):
+        return _head_rows(0, self.geo.heads, self.geo.vp, torch.arange(self.geo.vdim))
+
+    def logical_shapes(self):
+        return self._row_shapes()
+
+    def _pack(self, t):
+        self._pack_rows(t)
+
+    def unpack(self):
+        return self._unpack_rows()
+
+    def core(self, proj, storage, batch, out=None):
+        return retention(proj, self.geo, self.log2_decay, self.eps, storage[0], storage[1], batch, self.in_scale, out)
+
+
+class RGLRU(_RowPacked):
+    """A short convolution and a real-gated linear recurrence, times a GELU branch (see ``ops.rglru``)."""
+    takes_in_scale = True
+    tile = CHUNK
+    _vectors = ("x_bias", "y_bias", "conv_b", "ra_b", "ri_b", "decay")
+
+    def __init__(self, width: int, channels: int, blocks: int, conv: int, dtype, device):
+        super().__init__(dtype, device)
+        self.width = width
+        self.geo = g = RGLRUGeometry(channels, blocks, conv)
+        self.w_in, self.w_out = self._zeros(g.cols, pad_to(width)), self._zeros(width, g.out_cols)
+        vec = {n: self._zeros(g.channels, dtype=torch.float32) for n in self._vectors}
+        self.w = RGLRUWeights(conv=self._zeros(conv, g.channels, dtype=torch.float32), ra=self._zeros(blocks, g.kp, g.kp),
+                              ri=self._zeros(blocks, g.kp, g.kp), **vec)
+        self.lam = self._zeros(channels, dtype=torch.float32)
+
+    def tensors(self):
+        return super().tensors() + [t for t in vars(self.w).values()]
+
+    def run_spec(self) -> StateRun:
+        g = self.geo
+        return StateRun((g.channels,), (g.taps - 1, g.channels))
+
+    def _rows(self):
+        c = self.geo.columns()
+        return {"x": c, "y": self.geo.channels + c}
+
+    def _out_columns(self):
+        return self.geo.columns()
+
+    def logical_shapes(self):
+        g = self.geo
+        return {**self._row_shapes(), "x.b": (g.width,), "y.b": (g.width,), "conv": (g.width, g.taps), "conv.b": (g.width,),
+                "ra": (g.blocks, g.k, g.k), "ra.b": (g.blocks, g.k), "ri": (g.blocks, g.k, g.k), "ri.b": (g.blocks, g.k),
+                "lam": (g.width,)}
+
+    def _pack(self, t):
+        g, w = self.geo, self.w
+        self._pack_rows(t)
+        c = g.columns().to(self.device)
+        put = lambda dst, src: dst.__setitem__(c, src.to(self.device).float().reshape(-1))   # noqa: E731
+        put(w.x_bias, t["x.b"])
+        put(w.y_bias, t["y.b"])
+        put(w.conv_b, t["conv.b"])
+        put(w.ra_b, t["ra.b"])
+        put(w.ri_b, t["ri.b"])
+        put(w.decay, 8.0 * torch.nn.functional.softplus(t["lam"].double(), threshold=700.0))
+        w.conv[:, c] = t["conv"].to(self.device).float().t()
+        w.ra[:, :g.k, :g.k].copy_(t["ra"])
+        w.ri[:, :g.k, :g.k].copy_(t["ri"])
+        self.lam.copy_(t["lam"])
+
+    def unpack(self):
+        g, w, c = self.geo, self.w, self.geo.columns().to(self.device)
+        get = lambda v: v[c].to(self.dtype)   # noqa: E731
+        return {**self._unpack_rows(), "x.b": get(w.x_bias), "y.b": get(w.y_bias), "conv": w.conv[:, c].t().contiguous().to(self.dtype),
+                "conv.b": get(w.conv_b), "ra": w.ra[:, :g.k, :g.k].contiguous(), "ra.b": get(w.ra_b).view(g.blocks, g.k),
+                "ri": w.ri[:, :g.k, :g.k].contiguous(), "ri.b": get(w.ri_b).view(g.blocks, g.k), "lam": self.lam.to(self.dtype)}
+
+    def core(self, proj, storage, batch, out=None):
+        return rglru(proj, self.geo, self.w, storage[0], storage[1], batch, self.in_scale, out)

@@ -1,7 +1,8 @@
 """Cache manager and batch layout of decoders that mix paged attention with recurrent state.
 
-``HybridCache`` owns, for every layer run of a model, either a K / V pool (pages addressed through ONE block table per
-sequence, shared by all attention runs) or slot-indexed recurrent state, and hands out pages and slots.
+``HybridCache`` owns, for every layer run of a model, what its run spec allocates: a K / V pool or a pool of latents (pages
+addressed through ONE block table per sequence, shared by all attention runs) or slot-indexed recurrent state; it hands out
+pages and slots.
 ``HybridSequence`` is one request's share of it. ``RaggedBatch`` describes one step: for every sequence the tokens it
 brings, single decoded tokens first, then portions of prompts; all index arrays travel in one host-to-device copy.
 """
@@ -13,6 +14,7 @@ from typing import Dict, List, Optional, Sequence
 import numpy as np
 import torch
 
+from ..ops.rotary import Rotary
 from .kv_cache import BlockAllocator
 
 
@@ -22,13 +24,37 @@ class PagedRun:
     kv_heads: int
     head_dim: int
 
+    def allocate(self, c: "HybridCache") -> tuple:
+        shape = (c.num_blocks, self.kv_heads, c.block_size, self.head_dim)
+        return tuple(torch.zeros(shape, dtype=c.dtype, device=c.device) for _ in range(2))
+
+
+@dataclass(frozen=True)
+class LatentRun:
+    """Storage of one latent attention run: pages of one ``width``-column row per token, and the angles of its positions."""
+    width: int
+    rotary: Rotary
+
+    def allocate(self, c: "HybridCache") -> tuple:
+        return torch.zeros((c.num_blocks, c.block_size, self.width), dtype=c.dtype, device=c.device), c.angles(self.rotary)
+
 
 @dataclass(frozen=True)
 class StateRun:
-    """Storage of one recurrent run: per slot a recurrent state (fp32) and the tail of its convolution's inputs (the model's
-    dtype)."""
+    """Storage of one recurrent run: per slot the tail of its convolution's inputs (the model's dtype; absent without a
+    convolution) and a recurrent state (fp32); the angles of its positions where it rotates anything."""
     state: tuple
-    conv: tuple
+    conv: Optional[tuple] = None
+    rotary: Optional[Rotary] = None
+
+    def allocate(self, c: "HybridCache") -> tuple:
+        out = []
+        if self.conv is not None:
+            out.append(torch.zeros((c.max_sequences, *self.conv), dtype=c.dtype, device=c.device))
+        out.append(torch.zeros((c.max_sequences, *self.state), dtype=torch.float32, device=c.device))
+        if self.rotary is not None:
+            out.append(c.angles(self.rotary))
+        return tuple(out)
 
 
 class HybridCache:
@@ -43,17 +69,18 @@ class HybridCache:
         self.allocator = BlockAllocator(num_blocks)
         self.slot_allocator = BlockAllocator(max_sequences)
         self.tables = np.zeros((max_sequences, self.max_blocks), dtype=np.int32)   # row = the sequence's slot
-        self.runs: List[tuple] = []
-        for r in runs:
-            if isinstance(r, PagedRun):
-                shape = (num_blocks, r.kv_heads, block_size, r.head_dim)
-                self.runs.append((torch.zeros(shape, dtype=dtype, device=device), torch.zeros(shape, dtype=dtype, device=device)))
-            else:
-                self.runs.append((torch.zeros((max_sequences, *r.conv), dtype=dtype, device=device),
-                                  torch.zeros((max_sequences, *r.state), dtype=torch.float32, device=device)))
+        self._angles: Dict[Rotary, torch.Tensor] = {}
+        self.runs: List[tuple] = [r.allocate(self) for r in runs]
+
+    def angles(self, rotary: Rotary) -> torch.Tensor:
+        """(cos, sin) of every position the cache can hold; one table for all runs that rotate alike."""
+        if rotary not in self._angles:
+            self._angles[rotary] = rotary.table(self.max_len, self.device)
+        return self._angles[rotary]
 
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for r in self.runs for t in r)
+        unique = {t.data_ptr(): t for r in self.runs for t in r if t.numel()}
+        return sum(t.numel() * t.element_size() for t in unique.values())
 
     def can_admit(self) -> bool:
         """A slot is free (pages are the caller's business)."""
@@ -160,12 +187,23 @@ def cut_segments(portions, chunk: int, slot_of) -> Segments:
     return Segments(len(cu_q) - 1, int(np.diff(q).max()) if len(q) > 1 else 0, key, len(host[3]), host)
 
 
+@dataclass
+class Tiles:
+    """A step's prompt portions cut into tiles of a fixed number of tokens, each portion from its first row: the portion of
+    every tile, and the first tile of every portion."""
+    n: int
+    seq: Optional[torch.Tensor] = None
+    first: Optional[torch.Tensor] = None
+
+
 class RaggedBatch:
     """One step. ``entries``: (sequence, token ids); the sequences' pages are reserved here and their lengths advanced by
     ``commit`` once the step has been launched. Rows are ordered with single tokens first; ``row_of[i]`` is the first row
-    of entry i. ``want`` [i]: places among entry i's tokens whose logits are asked for, answered in entry order."""
+    of entry i. ``want`` [i]: places among entry i's tokens whose logits are asked for, answered in entry order. ``chunks``:
+    attention masks, ``tiles``: tile sizes that the model's mixers ask for (``segments``, ``tiles``)."""
 
-    def __init__(self, cache: HybridCache, entries, want=None, chunks: Sequence[int] = (), max_len: int = 0):
+    def __init__(self, cache: HybridCache, entries, want=None, chunks: Sequence[int] = (), max_len: int = 0,
+                 tiles: Sequence[int] = ()):
         self.cache = cache
         entries = [(s, np.asarray(t, dtype=np.int32)) for s, t in entries]
         if any(len(t) == 0 for _, t in entries):
@@ -225,6 +263,13 @@ class RaggedBatch:
             "state_slots": slot, "lens": pos0[:nd] + 1, "cu": row0[nd:] - row0[nd], "pos0": pos0[nd:],
             "blk_seq": np.repeat(np.arange(self.n_prompts), nblk), "blk0": np.concatenate([[0], np.cumsum(nblk)]), "want": np.asarray(rows, dtype=np.int64),
         }
+        self._tiles: Dict[int, Tiles] = {}
+        if self.n_prompts:
+            for size in tiles:
+                per = -(-n[nd:] // size)
+                self._tiles[size] = Tiles(int(per.sum()))
+                fields[f"seq:{size}"] = np.repeat(np.arange(self.n_prompts), per)
+                fields[f"first:{size}"] = np.concatenate([[0], np.cumsum(per)])
         for c, sg in segs.items():
             for name, a in zip(("cu_q", "cu_k", "stage_rows", "gather_dst", "gather_src"), sg.host):
                 fields[f"{name}:{c}"] = a
@@ -240,13 +285,16 @@ class RaggedBatch:
             at += a.size
             if ":" in name:
                 f, c = name.split(":")
-                setattr(segs[int(c)], f, t)
+                setattr(self._tiles[int(c)] if f in ("seq", "first") else segs[int(c)], f, t)
             else:
                 setattr(self, name, t)
         self._segs = segs
 
     def segments(self, chunk: int) -> Segments:
         return self._segs[chunk]
+
+    def tiles(self, size: int) -> Tiles:
+        return self._tiles[size]
 
     def spans(self):
         """(first row, rows, slot, position of the first row) of every sequence, in row order."""

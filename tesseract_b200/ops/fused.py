@@ -9,6 +9,8 @@ src/nn/RotaryEmbedding.cpp:35-57), mean cross-entropy with int64 targets (src/op
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from .. import _native
@@ -376,11 +378,12 @@ def cross_entropy(logits: torch.Tensor, targets: torch.Tensor) -> torch.Tensor:
     return cross_entropy_ref(logits, targets)
 
 
-# --------------------------------------------------------------------------------------- Dynamic Tanh, clamped GLU
+# --------------------------------------------------------------------------------------- residual steps, clamped GLU
 _P, _I, _L, _F = _native.P, _native.I, _native.L, _native.F
 _native.register_signatures({
     "tsb_dyn_tanh_residual": [_P, _I, _I, _P, _L, _P, _F, _P, _P, _P, _P, _L, _F, _I, _I, _P, _F, _P, _P, _P, _L, _I, _I, _P],
-    "tsb_clamped_glu": [_P, _L, _P, _P, _L, _I, _I, _F, _F, _I, _P],
+    "tsb_clamped_glu": [_P, _L, _P, _P, _L, _I, _I, _F, _F, _F, _F, _I, _P],
+    "tsb_depth_residual": [_P, _P, _P, _L, _P, _I, _I, _P, _L, _F, _P, _P, _L, _I, _P, _L, _I, _I, _I, _F, _F, _I, _P],
 })
 _EMBED_MODES = {None: 0, "set": 1, "add": 2}
 
@@ -438,21 +441,70 @@ def dyn_tanh_residual(x, y=None, y_bias=None, post=None, tokens=None, table=None
     return h
 
 
-def clamped_glu(gate_up, bias, limit, slope=1.702):
-    """gate_up [T, 2 F] (gate, then up; ``bias`` fp32 [2 F] or None is added first) -> g sigmoid(slope g) (u + 1) with
-    g = min(gate, limit), u = clamp(up, -limit, limit)."""
+def clamped_glu(gate_up, bias, limit, slope=1.702, shift=1.0, in_scale=1.0, out=None):
+    """gate_up [T, 2 F] (gate, then up; times ``in_scale``, plus ``bias`` fp32 [2 F] if given) -> g sigmoid(slope g) (u + shift)
+    with g = min(gate, limit), u = clamp(up, -limit, limit). ``out`` may be columns of a wider matrix."""
     T, F2 = gate_up.shape
     F = F2 // 2
-    out = torch.empty((T, F), device=gate_up.device, dtype=gate_up.dtype)
+    if out is None:
+        out = torch.empty((T, F), device=gate_up.device, dtype=gate_up.dtype)
     if T == 0:
         return out
     if gate_up.is_cuda:
         check(lib().tsb_clamped_glu(gate_up.data_ptr(), gate_up.stride(0), _ptr(bias), out.data_ptr(), out.stride(0), T, F,
-                                    float(limit), float(slope), dtype_code(gate_up.dtype), stream_ptr(gate_up.device)),
-              "tsb_clamped_glu")
+                                    float(limit), float(slope), float(shift), float(in_scale), dtype_code(gate_up.dtype),
+                                    stream_ptr(gate_up.device)), "tsb_clamped_glu")
         return out
-    z = gate_up.float()
+    z = gate_up.float() * in_scale
     if bias is not None:
         z = z + bias
     g, u = z[:, :F].clamp(max=limit), z[:, F:].clamp(-limit, limit)
-    return out.copy_(g * torch.sigmoid(slope * g) * (u + 1.0))
+    return out.copy_(g * torch.sigmoid(slope * g) * (u + shift))
+
+
+def silu_glu(gate_up, in_scale=1.0, out=None):
+    """SiLU(gate) * up of the two halves of a row, both times ``in_scale`` first."""
+    return clamped_glu(gate_up, None, math.inf, 1.0, 0.0, in_scale, out)
+
+
+def depth_residual(x_in=None, y=None, mult=1.0, tokens=None, table=None, width=0, history=None, depth=0, average=None, store=True,
+                   gain=1.0, eps=0.0, out_cols=0, out_dtype=None, want_h=True):
+    """One step of an fp32 residual stream between two matrix products, with depth averaging and an RMS norm of one gain:
+
+        X = table[tokens]  or  x_in + mult * y
+        x = sum_j average[j] history[j] + average[depth] X, j < depth    (average given; else x = X)
+        h = x / sqrt(mean(x^2) + eps) * gain
+
+    ``history`` [entries, T, width] (fp32) receives X as entry ``depth`` when ``store``. Returns (x, h [T, out_cols] in
+    ``out_dtype`` with zeros past the width, or None); at the start of the model x is the stored entry itself."""
+    start = tokens is not None
+    T, W = (tokens.shape[0], width) if start else x_in.shape
+    dev = table.device if start else x_in.device
+    src = table if start else y
+    h = torch.empty((T, out_cols or W), device=dev, dtype=out_dtype or src.dtype) if want_h else None
+    store = store and history is not None
+    alias = start and store and average is None
+    x = history[depth] if alias else torch.empty((T, W), device=dev, dtype=torch.float32)
+    if T == 0:
+        return x, h
+    if x.is_cuda:
+        if h is not None and h.dtype != src.dtype:
+            raise ValueError("depth_residual: the input and the result share one dtype")
+        check(lib().tsb_depth_residual(_ptr(x_in), None if alias else x.data_ptr(), _ptr(history),
+                                       history.stride(0) if history is not None else 0, _ptr(average), depth, int(store),
+                                       _ptr(y), y.stride(0) if y is not None else 0, float(mult), _ptr(tokens), _ptr(table),
+                                       table.stride(0) if start else 0, table.shape[0] if start else 0, _ptr(h),
+                                       h.stride(0) if h is not None else 0, h.shape[1] if h is not None else 0, T, W, float(gain), float(eps),
+                                       dtype_code(src.dtype), stream_ptr(dev)), "tsb_depth_residual")
+        return x, h
+    new = table[tokens.long(), :W].float() if start else x_in + mult * y[:, :W].float()
+    if store:
+        history[depth].copy_(new)
+    if average is not None:
+        new = average[depth] * new + (average[:depth, None, None] * history[:depth]).sum(0)
+    if not alias:
+        x.copy_(new)
+    if h is not None:
+        h[:, W:] = 0
+        h[:, :W] = new / torch.sqrt((new * new).mean(-1, keepdim=True) + eps) * gain
+    return x, h

@@ -85,10 +85,12 @@ def main(argv=None) -> int:
     import torch
 
     from .. import _native, build
+    from ..models.registry import read_config, resolve
     if not torch.cuda.is_available():
         print("trace_run: no CUDA GPU is visible", file=sys.stderr)
         return 1
-    _native.use_library(build.ensure("hybrid"))
+    kernels = resolve(read_config(os.path.join(a.model, "config.json"))).kernels
+    _native.use_library(build.ensure(kernels) if kernels else build.build_cuda())
     torch.backends.cuda.matmul.allow_tf32 = False
     torch.cuda.set_device(0)
     rep = make_replay(a.model, getattr(torch, a.dtype), torch.device("cuda", 0), a.max_tokens)
