@@ -110,9 +110,10 @@ def parse_args():
                     help="auto | dp | tp | tpK (tensor parallel over K ranks, data parallel over the rest) | a comma list: "
                          "every mesh listed is measured and `value` is the fastest")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--hybrid", action="store_true",
-                    help="instead of the headline: prefill and decode throughput of the hybrid decoder (gated delta rule + chunked "
-                         "attention) beside Llama at equal sizes, one GPU (benchmarks/bench_hybrid.py)")
+    ap.add_argument("--hybrid", nargs="?", const="fozelix", default="", choices=["fozelix", "polosun"],
+                    help="instead of the headline: prefill and decode throughput of a hybrid decoder at the sizes of real layers, one "
+                         "GPU (benchmarks/bench_hybrid.py): fozelix (gated delta rule + chunked attention, beside Llama; the default) or "
+                         "polosun (retention, latent attention, gated recurrence, beside fozelix and Llama)")
     ap.add_argument("--ref-time-budget", type=float, default=float(os.environ.get("TESSERACT_REF_TIME_BUDGET", 780)),
                     help="(--impl reference) seconds the whole reference arm may take; the timed step count shrinks to fit")
     return ap.parse_args()
@@ -296,8 +297,9 @@ def main():
         from bench_hybrid import run
         sampler = ClockSampler(0)
         sampler.start()
-        sizes = run()
-        print(json.dumps({"benchmark": "hybrid decoder serving beside Llama at equal size", "n_gpus": 1, "dtype": "bf16",
+        models = ("hybrid", "llama") if args.hybrid == "fozelix" else ("polosun", "hybrid", "llama")
+        sizes = run(models=models)
+        print(json.dumps({"benchmark": "hybrid decoder serving beside other models at equal size", "models": models, "n_gpus": 1, "dtype": "bf16",
                           "data": "synthetic random token ids; random-init weights", "sizes": sizes, "clocks": sampler.stop()}))
         return 0
 

@@ -1,13 +1,16 @@
 #!/usr/bin/env python
-"""Prefill and decode throughput of hybrid decoders (random weights) beside Llama at equal size, each through its own
+"""Prefill and decode throughput of hybrid decoders (random weights) beside other models at equal size, each through its own
 serving engine on one GPU.
 
     python benchmarks/bench_hybrid.py                      # every size
-    python bench.py --hybrid                               # the same, from the headline benchmark's command line
+    python benchmarks/bench_hybrid.py --models polosun,hybrid,llama
+    python bench.py --hybrid [fozelix | polosun]           # the same, from the headline benchmark's command line
 
-Both models of a size have the same width, feed-forward, layer count, vocabulary and attention heads; the hybrid one has
-three gated-delta layers (16 or 8 key heads, twice as many value heads, 128 x 128) to every chunked-attention layer. bf16
-weights and KV on both sides, greedy. Prefill: ``seqs`` prompts of ``prompt`` tokens in one step; decode: a batch of
+The models of a size have the same width, feed-forward, layer count, vocabulary and attention heads. ``hybrid`` has three
+gated-delta layers (16 or 8 key heads, twice as many value heads, 128 x 128) to every chunked-attention layer; ``polosun``
+cycles through retention (heads of 128 x 128), latent attention (64 + 64 rotated query columns a head, values of 128, a latent
+of 512) and the gated recurrence (as many channels as the width, gate blocks of 256). bf16 weights and KV on all sides,
+greedy. Prefill: ``seqs`` prompts of ``prompt`` tokens in one step; decode: a batch of
 requests after that. Times are wall clock around engine steps with a device synchronise on both sides (inputs from the
 host and the read of the chosen tokens included); ``gpu_ms`` is the captured decode step alone, from CUDA events. Every
 step streams more weight bytes than L2 holds.
@@ -39,6 +42,16 @@ def build(kind, s, device, max_pos):
                           num_key_value_heads=s["kv"], intermediate_size=s["ff"], max_position_embeddings=max_pos,
                           dtype=torch.bfloat16)
         return LlamaModel(cfg, device=device, init_std=0.02, seed=1)
+    if kind == "polosun":
+        from tesseract_b200.models import polosun
+        from tesseract_b200.models.hybrid import LatentSpec, RetentionSpec, RGLRUSpec, Rotary
+        h = s["heads"]
+        layers = polosun.layer_cycle(
+            s["layers"], LatentSpec(h, 64, 64, 128, 512, 128 ** -0.5, Rotary(64, 1e6)),
+            RetentionSpec(h, 128, 128, tuple(1.0 - 2.0 ** (-5 - 7 * i / h) for i in range(h)), Rotary(128, 1e4)),
+            RGLRUSpec(s["width"], s["width"] // 256, 4), s["ff"])
+        return HybridModel(HybridConfig(s["vocab"], s["width"], layers, eps=1e-6, dtype=torch.bfloat16, form="parallel", residual_mult=0.5,
+                                        depth_average=True, tied=False), device=device, init_std=0.02, seed=1)
     att = AttentionSpec(s["heads"], s["kv"], 128, 128, 128 ** -0.5, 4096)
     dlt = DeltaSpec(2 * s["key_heads"], s["key_heads"], 128, 128, 4)
     layers = [LayerSpec(att if i % 4 == 3 else dlt, GLUSpec(s["ff"], 7.0)) for i in range(s["layers"])]
@@ -60,7 +73,7 @@ def measure(kind, s, seqs, prompt, decode_batches, steps, device):
     per = {"prefill": prompt + 1, "decode": 1300 + new + 2}
     blocks = max(seqs * (per["prefill"] // 16 + 2), top * (per["decode"] // 16 + 2)) + 64
     model = build(kind, s, device, max(per.values()) + 16)
-    extra = {"max_step_tokens": seqs * prompt + top} if kind == "hybrid" else {"max_prefill_tokens": seqs * prompt}
+    extra = {"max_step_tokens": seqs * prompt + top} if kind != "llama" else {"max_prefill_tokens": seqs * prompt}
     eng = make_engine(model, EngineConfig(block_size=16, num_blocks=blocks, max_seq_len=max(per.values()), max_batch_size=top), **extra)
     prompts = [[rng.randrange(s["vocab"]) for _ in range(prompt)] for _ in range(seqs)]
     out = {"model": kind, "prefill": {"seqs": seqs, "prompt": prompt}, "decode": []}
@@ -107,14 +120,14 @@ def measure(kind, s, seqs, prompt, decode_batches, steps, device):
     return out
 
 
-def run(sizes=None, seqs=4, prompt=4096, decode_batches=(1, 32, 256), steps=24, device=None):
-    """{size: {"hybrid": ..., "llama": ...}}"""
+def run(sizes=None, seqs=4, prompt=4096, decode_batches=(1, 32, 256), steps=24, device=None, models=("hybrid", "llama")):
+    """{size: {model: ...}}"""
     import torch
     device = device or torch.device("cuda", 0)
     torch.cuda.set_device(device)
     res = {}
     for name in sizes or SIZES:
-        res[name] = {k: measure(k, SIZES[name], seqs, prompt, decode_batches, steps, device) for k in ("hybrid", "llama")}
+        res[name] = {k: measure(k, SIZES[name], seqs, prompt, decode_batches, steps, device) for k in models}
     return res
 
 
@@ -124,9 +137,11 @@ def main():
     ap.add_argument("--seqs", type=int, default=4)
     ap.add_argument("--prompt", type=int, default=4096)
     ap.add_argument("--steps", type=int, default=24)
+    ap.add_argument("--models", default="hybrid,llama", help="comma list of polosun, hybrid, llama")
     a = ap.parse_args()
-    for name, r in run(a.sizes.split(","), a.seqs, a.prompt, steps=a.steps).items():
-        for k in ("hybrid", "llama"):
+    models = a.models.split(",")
+    for name, r in run(a.sizes.split(","), a.seqs, a.prompt, steps=a.steps, models=models).items():
+        for k in models:
             print(json.dumps({"size": name, **r[k]}), flush=True)
 
 

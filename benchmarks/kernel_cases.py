@@ -410,7 +410,7 @@ def case_ag_gemm_emul(b: Bench):
 class _Step:
     """A ragged batch of ``n`` sequences bringing ``rows`` tokens each, after ``past`` tokens."""
 
-    def __init__(self, b, run, n, rows, past=0, chunks=(), block=16):
+    def __init__(self, b, run, n, rows, past=0, chunks=(), block=16, tiles=()):
         from tesseract_b200.nn.ragged import HybridCache, HybridSequence, RaggedBatch
         blocks = n * ((past + rows + block - 1) // block)
         self.cache = HybridCache([run], blocks, block, n, past + rows + block, torch.bfloat16, b.dev)
@@ -419,7 +419,7 @@ class _Step:
             if past:
                 s.reserve(past)
                 s.advance(past)
-        self.batch = RaggedBatch(self.cache, [(s, [0] * rows) for s in seqs], None, chunks)
+        self.batch = RaggedBatch(self.cache, [(s, [0] * rows) for s in seqs], None, chunks, 0, tiles)
 
 
 def _delta_case(b, n, rows, past):
@@ -493,13 +493,80 @@ def case_clamped_glu(b: Bench):
     report("clamped_glu", ms, bytes_=x.numel() * 2 * 1.5, shape=list(x.shape))
 
 
+# ---- the mixers of 4096-wide layers with 32 heads: retention 128 x 128, latent 64 + 64 / 128 / 512, recurrence 4096 in blocks of 256
+def _mixer_case(b, block, n, rows, past=0):
+    """Time of a mixer's core (everything between its two products)."""
+    st = _Step(b, block.run_spec(), n, rows, past, (0,), tiles=[block.tile] if block.tile else [])
+    proj = b.randn(n * rows, block.cols)
+    return b.time(lambda: block.core(proj, st.cache.runs[0], st.batch))
+
+
+def case_retention(b: Bench):
+    """Prompts: bytes of q, k, v, gate and the result; decode: the state read and written once."""
+    from tesseract_b200.nn.hybrid import Retention
+    from tesseract_b200.ops.rotary import Rotary
+    H = 32
+    blk = Retention(64, H, 128, 128, [1.0 - 2.0 ** (-5 - 7 * i / H) for i in range(H)], Rotary(128, 1e4), 1e-6, torch.bfloat16, b.dev)
+    for n, rows in ((4, 4096), (1, 4096), (32, 512)):
+        ms = _mixer_case(b, blk, n, rows)
+        report("retention_prefill", ms, bytes_=n * rows * H * 128 * 5 * 2.0, shape=[n, rows])
+    for n in (256, 32):
+        report("retention_step", _mixer_case(b, blk, n, 1, 7), bytes_=n * 2.0 * H * 128 * 128 * 4, shape=[n])
+
+
+def case_latent(b: Bench):
+    """Prompts: flops of the written-out form (expansion of the latents and causal attention); decode: bytes of the cached rows."""
+    from tesseract_b200.nn.hybrid import LatentAttention
+    from tesseract_b200.ops.rotary import Rotary
+    H = 32
+    blk = LatentAttention(64, H, 64, 64, 128, 512, 128 ** -0.5, Rotary(64, 1e6), 1e-6, torch.bfloat16, b.dev)
+    for n, rows in ((2, 4096), (8, 1024)):
+        ms = _mixer_case(b, blk, n, rows)
+        report("latent_prefill", ms, flops=n * rows * (rows * H * 128 * 2.0 + 2.0 * 512 * H * 192), shape=[n, rows])
+    for n, past in ((256, 1399), (32, 1399), (32, 8191)):
+        ms = _mixer_case(b, blk, n, 1, past)
+        report("latent_decode", ms, bytes_=n * (past + 1) * 576 * 2.0, flops=n * (past + 1.0) * H * 2 * (576 + 512), shape=[n, past + 1])
+
+
+def case_rglru(b: Bench):
+    """Prompts: bytes of x, y and the result; decode: the gate matrices, x, y, the states and the result."""
+    from tesseract_b200.nn.hybrid import RGLRU
+    W = 4096
+    blk = RGLRU(64, W, W // 256, 4, torch.bfloat16, b.dev)
+    blk.w.ra.normal_(std=0.06)
+    blk.w.ri.normal_(std=0.06)
+    blk.w.decay.fill_(0.2)
+    for n, rows in ((4, 4096), (1, 4096), (32, 512)):
+        report("rglru_prefill", _mixer_case(b, blk, n, rows), bytes_=n * rows * W * 3 * 2.0, shape=[n, rows])
+    for n in (256, 32):
+        report("rglru_step", _mixer_case(b, blk, n, 1, 7), bytes_=2.0 * 256 * W * 2 + n * W * (2 * 4 + 5 * 2 + 3 * 2.0), shape=[n])
+
+
+def case_depth_residual(b: Bench):
+    from tesseract_b200 import ops
+    T, W = 16384, 4096
+    hist = torch.randn(5, T, W, device=b.dev, generator=b.gen)
+    x, y, avg = torch.randn(T, W, device=b.dev, generator=b.gen), b.randn(T, W), torch.randn(5, device=b.dev, generator=b.gen)
+    for depth in (1, 4):
+        a = avg[:depth + 1].contiguous()
+        ms = b.time(lambda: ops.depth_residual(x, y, 0.5, history=hist, depth=depth, average=a, eps=1e-6))
+        report("depth_residual", ms, bytes_=T * W * (4 * (depth + 3) + 4), shape=[T, W, depth])
+
+
+def case_silu_glu(b: Bench):
+    from tesseract_b200 import ops
+    x = b.randn(16384, 2 * 14336)
+    report("silu_glu", b.time(lambda: ops.silu_glu(x, 0.9)), bytes_=x.numel() * 2 * 1.5, shape=list(x.shape))
+
+
 CASES = {"gemm": case_gemm, "gemm_fp8": case_gemm_fp8, "gemm_fp8_pertensor": case_gemm_fp8_pertensor, "decode_gemm": case_decode_gemm, "gemm_wgrad": case_gemm_wgrad, "grouped_gemm": case_grouped_gemm,
          "flash_fwd": case_flash_fwd, "flash_bwd": case_flash_bwd, "decode": case_decode,
          "decode_int8": case_decode_int8, "rmsnorm": case_rmsnorm, "swiglu": case_swiglu, "swiglu_bwd": case_swiglu_bwd, "adam": case_adam,
          "ce_stats": case_ce, "selective_scan": case_scan, "gemv_w8": case_gemv, "gemm_rs_emul": case_gemm_rs_emul,
          "ag_gemm_emul": case_ag_gemm_emul, "stream_linear": case_stream_linear, "mx_linear": case_mx_linear, "gemm_mx": case_gemm_mx,
          "delta_prefill": case_delta_prefill, "delta_step": case_delta_step, "chunk_attn": case_chunk_attn,
-         "dyn_tanh": case_dyn_tanh, "clamped_glu": case_clamped_glu}
+         "dyn_tanh": case_dyn_tanh, "clamped_glu": case_clamped_glu, "retention": case_retention, "latent": case_latent, "rglru": case_rglru,
+         "depth_residual": case_depth_residual, "silu_glu": case_silu_glu}
 
 
 def main():

@@ -143,7 +143,7 @@ def save_file(tensors: Dict[str, torch.Tensor], path: str, metadata: Optional[Di
         f.write(hjson)
         for t in blobs:
             if t.numel():
-                f.write(t.view(torch.uint8).numpy().tobytes() if t.dim() else t.reshape(1).view(torch.uint8).numpy().tobytes())
+                f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes())
 
 
 def load_file(path: str, device=None) -> Dict[str, torch.Tensor]:
