@@ -12,7 +12,8 @@ struct HeadTile {
   static constexpr int kThreads = 128, BN = 64;
   static constexpr int kStep = sizeof(T) == 2 ? 64 : 32;                // k columns per stage
   static constexpr int kLd = kStep + 16 / static_cast<int>(sizeof(T));
-  static constexpr int kStages = 3;
+  // few rows: latency decides, most of K is in flight at once; many rows and two matrices: residency decides
+  static constexpr int kStages = BM == 16 ? 5 : NW == 2 ? 2 : 4;
   static constexpr int kStageElems = (BM + NW * BN) * kLd;
   static constexpr int kLdC = BN + 4;
   static constexpr int kRing = kStages * kStageElems * static_cast<int>(sizeof(T));
@@ -61,10 +62,18 @@ struct HeadTile {
       cp_commit();
     }
     for (int s = 0; s < steps; ++s) {
-      cp_wait<kStages - 2>();
-      __syncthreads();
-      if (s + kStages - 1 < steps) issue(s + kStages - 1);
-      cp_commit();
+      if constexpr (kStages > 2) {
+        cp_wait<kStages - 2>();
+        __syncthreads();
+        if (s + kStages - 1 < steps) issue(s + kStages - 1);
+        cp_commit();
+      } else {                            // (with two stages the buffer to fill is the one just read)
+        __syncthreads();
+        if (s + 1 < steps) issue(s + 1);
+        cp_commit();
+        cp_wait<1>();
+        __syncthreads();
+      }
       const T* sx = ring + (s % kStages) * kStageElems;
       if constexpr (sizeof(T) == 2) {
         const uint32_t ax = smem_u32(sx);

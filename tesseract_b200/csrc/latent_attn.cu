@@ -10,8 +10,8 @@
 //                         and, for rows attended in the latent space, the rotated part of `q_cat` [rows, H, cp + rp].
 //   head_linear_kernel    one small product per head: W_uk^T q into q_cat's first cp columns before the attention in the
 //                         latent space, W_uv o after it, times the output gate.
-//   latent_decode_kernel  attention of single rows in the latent space on the tensor cores (bf16), split over keys; the pool
-//                         row serves as key and, its first cp columns, as value, so it is read once for all heads.
+//   latent_decode_kernel  attention of single rows in the latent space on tcgen05 (bf16), split over keys; the pool row serves
+//                         as key and, its first cp columns, as value, so it is read once for 32 heads.
 //   latent_merge_kernel   merges the splits.
 //   latent_rows_kernel    the same attention with one warp per (row, head) in fp32: fp32 models and sizes the other does not take.
 //   latent_gather_kernel  pool rows of earlier portions -> key axis.
@@ -209,162 +209,278 @@ struct LatentAttnParams {
 };
 
 constexpr int kKeys = 64;          // keys of a tile
+constexpr int kHeads = 32;         // heads of a CTA
+constexpr int kBlockBytes = kKeys * 128;      // 64 keys x 64 columns, 128-byte swizzle
 
-// One CTA per (key split, 16 heads, row), eight warps. Per tile: warp w scores keys 8 w .. 8 w + 7 for the 16 heads; the
-// weights go through shared memory; then every warp adds the tile to its own cp / 8 columns of the read-out.
-template <int CT>
-__global__ void __launch_bounds__(256)
-latent_decode_kernel(LatentAttnParams p) {
-  using T = __nv_bfloat16;
+// One CTA per (key split, 32 heads, row); a tile of 64 pool rows is brought in once (TMA, one box per run of rows of a page and
+// 64 columns) and is the B operand of the scores and the A operand of the read-out:
+//   S[head, key]   = q[head, :] . row[key, :]       M = 128 (rows past the heads read whatever lies there and are ignored)
+//   O[col, head]  += row[key, col] P[head, key]     M = 128 columns a time, N = heads: no row of the product is padding
+// Warp 0 turns scores into weights (lane = head) with the lazy reference maximum of flash_attn_fwd.cu: O is rescaled, by all of
+// warps 0 .. 3, only when a head's maximum has grown by more than 2^8. Warp 4 loads, warp 5 issues the products.
+struct LatentSmem {
+  static __host__ __device__ int blocks(int L) { return (L + 63) / 64; }
+  static __host__ __device__ int stages(int L) {
+    const int room = 227 * 1024 - 2048 - blocks(L) * kHeads * 128 - kHeads * 128;
+    const int n = room / (blocks(L) * kBlockBytes);
+    return n < 4 ? n : 4;
+  }
+  static __host__ __device__ int bytes(int L) {
+    return 1024 + blocks(L) * kHeads * 128 + kHeads * 128 + stages(L) * blocks(L) * kBlockBytes;
+  }
+};
+
+__global__ void __launch_bounds__(192, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_pool, LatentAttnParams p) {
   pdl_trigger();
   pdl_grid_wait();
-  extern __shared__ __align__(16) uint8_t smem[];
-  constexpr int kLdP = kKeys + 8;
-  const int L = p.cp + p.rp, ld = L + 8;
-  T* sq = reinterpret_cast<T*>(smem);                 // [16][ld]
-  T* sk = sq + 16 * ld;                               // [2][kKeys][ld]
-  T* sp = sk + 2 * kKeys * ld;                        // [16][kLdP]
-  float* smax = reinterpret_cast<float*>(sp + 16 * kLdP);      // [8][16]
-  float* ssum = smax + 8 * 16;                        // [8][16]
-  const int split = blockIdx.x, h0 = blockIdx.y * 16, row = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int L = p.cp + p.rp, NB = LatentSmem::blocks(L), stages = LatentSmem::stages(L);
+  uint8_t* sq = smem;                                  // [NB][32 heads][128 B]
+  uint8_t* sp = sq + NB * kHeads * 128;                // [32 heads][128 B]
+  uint8_t* sk = sp + kHeads * 128;                     // [stages][NB][64 keys][128 B]
+  __shared__ __align__(8) uint64_t q_full, k_full[4], k_empty[4], s_full[2], s_free[2], p_full, o_full;
+  __shared__ uint32_t tmem_base_smem;
+  __shared__ volatile int cta_abort;
+  __shared__ float corr[kHeads], inv[kHeads];
+  __shared__ volatile int grown;                       // 1: rescale, 0: not, -1: leave
+  const int split = blockIdx.x, h0 = blockIdx.y * kHeads, row = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int len = p.lens ? p.lens[row] : p.pos[row] + 1;
   const int share = ((len + p.splits - 1) / p.splits + kKeys - 1) / kKeys * kKeys;
   const int t_begin = split * share, t_end = min(len, t_begin + share);
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + kKeys - 1) / kKeys : 0;
-  const int* table = p.tables + static_cast<long long>(p.seq_of ? p.seq_of[row] : row) * p.table_ld;
-  const int pieces = L / 8;
+  constexpr uint32_t kColO = 0, kColS = 128;
 
-  auto issue = [&](int j) {
-    T* dst = sk + (j & 1) * kKeys * ld;
-    for (int i = 0; i < 8; ++i) {
-      const int r = warp * 8 + i, t = t_begin + j * kKeys + r;
-      const bool ok = t < t_end;
-      int blk = ok ? table[t / p.bs] : 0;
-      if (blk < 0 || blk >= p.nb) {        // never read outside the pool: block 0 instead, and the host hears of it
-        if (lane == 0 && p.status) atomicCAS(p.status, kStatusOk, kStatusBadIndex);
-        blk = 0;
-      }
-      const T* src = static_cast<const T*>(p.pool) + (static_cast<long long>(blk) * p.bs + (ok ? t % p.bs : 0)) * L;
-      for (int v = lane; v < pieces; v += 32) cp_async_16(smem_u32(dst + r * ld + v * 8), src + v * 8, ok ? 16 : 0);
+  if (threadIdx.x == 0) {
+    cta_abort = 0;
+    mbar_init(&q_full, 1);
+    for (int i = 0; i < 4; ++i) {
+      mbar_init(&k_full[i], 1);
+      mbar_init(&k_empty[i], 1);
     }
-  };
-  for (int i = tid; i < 16 * pieces; i += 256) {
-    const int h = i / pieces, v = i % pieces;
-    const bool ok = h0 + h < p.H;
-    cp_async_16(smem_u32(sq + h * ld + v * 8),
-                static_cast<const T*>(p.q) + (static_cast<long long>(row) * p.H + (ok ? h0 + h : 0)) * L + v * 8, ok ? 16 : 0);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&s_full[i], 1);
+      mbar_init(&s_free[i], 32);
+    }
+    mbar_init(&p_full, 128);
+    mbar_init(&o_full, 1);
+    mbar_fence_init();
+    tma_prefetch_desc(&tm_q);
+    tma_prefetch_desc(&tm_pool);
   }
-  if (n_tiles > 0) issue(0);
-  cp_commit();
+  if (warp == 5) {
+    tmem_alloc(&tmem_base_smem, 256);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_base_smem;
+  const int m_tiles = (p.cp + 127) / 128;
 
-  float o[CT][4];
-#pragma unroll
-  for (int i = 0; i < CT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_part[2] = {0.f, 0.f};      // rows g and g + 8
-  const float scale_log2 = p.scale * 1.4426950408889634f;
-  const uint32_t q_addr = smem_u32(sq), p_addr = smem_u32(sp);
-  for (int j = 0; j < n_tiles; ++j) {
-    if (j + 1 < n_tiles) issue(j + 1);
-    cp_commit();
-    cp_wait<1>();
-    __syncthreads();
-    const uint32_t k_addr = smem_u32(sk + (j & 1) * kKeys * ld);
-    // scores: four independent sums over interleaved slices of the row
-    float s[4][4];
-#pragma unroll
-    for (int e = 0; e < 4; ++e) s[e][0] = s[e][1] = s[e][2] = s[e][3] = 0.f;
-    for (int k0 = 0; k0 < L; k0 += 64) {
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int k = k0 + half * 32;
-        if (k >= L) break;
-        uint32_t b[4], a0[4], a1[4];
-        ldmat_x4(b, k_addr + static_cast<uint32_t>((warp * 8 + (lane & 7)) * ld + k + (lane >> 3) * 8) * 2);
-        ldmat_x4(a0, q_addr + frag_a(lane, 0, k, ld));
-        ldmat_x4(a1, q_addr + frag_a(lane, 0, k + 16, ld));
-        mma_bf16(s[2 * half], a0, b[0], b[1]);
-        mma_bf16(s[2 * half + 1], a1, b[2], b[3]);
+  if (warp == 4) {
+    // ---------------------------------------------------------------- loads: a lane per run of rows inside a page
+    if (n_tiles > 0) {
+      if (lane == 0) mbar_expect_tx(&q_full, NB * kHeads * 128);
+      __syncwarp();
+      for (int b = lane; b < NB; b += 32) tma_load_2d(sq + b * kHeads * 128, &tm_q, &q_full, b * 64, row * p.H + h0);
+      const int* table = p.tables + static_cast<long long>(p.seq_of ? p.seq_of[row] : row) * p.table_ld;
+      int run = 64;
+      while (p.bs % run) run >>= 1;                    // rows that are neighbours in the pool: 64, 32, 16 or 8
+      const int runs = kKeys / run;
+      auto pool_row = [&](int j) {                     // first pool row of this lane's run; past the keys: past the pool (zeros)
+        const int t = t_begin + j * kKeys + lane * run;
+        if (lane >= runs || t >= t_end) return p.nb * p.bs;
+        int blk = table[t / p.bs];
+        if (blk < 0 || blk >= p.nb) {                  // never read another page: zeros instead, and the host hears of it
+          if (p.status) atomicCAS(p.status, kStatusOk, kStatusBadIndex);
+          return p.nb * p.bs;
+        }
+        return blk * p.bs + t % p.bs;
+      };
+      int next = pool_row(0);
+      for (int j = 0; j < n_tiles; ++j) {
+        const int st = j % stages, y = next;
+        if (j + 1 < n_tiles) next = pool_row(j + 1);
+        const bool ok = mbar_wait(&k_empty[st], ((j / stages) & 1) ^ 1u, &cta_abort, p.status);
+        if (!__all_sync(0xffffffffu, ok ? 1 : 0)) break;
+        if (lane == 0) mbar_expect_tx(&k_full[st], NB * kBlockBytes);
+        __syncwarp();
+        if (lane < runs) {
+          uint8_t* dst = sk + st * NB * kBlockBytes + lane * run * 128;
+          for (int b = 0; b < NB; ++b) tma_load_2d(dst + b * kBlockBytes, &tm_pool, &k_full[st], b * 64, y);
+        }
       }
     }
-    const int key = t_begin + j * kKeys + warp * 8 + 2 * t4;
-    float sc[4];
+  } else if (warp == 5) {
+    // ---------------------------------------------------------------- products
+    if (lane == 0 && n_tiles > 0) {
+      constexpr uint32_t idesc_s = umma_idesc(128, kKeys, 1, 1, 0, 0);       // both K-major
+      constexpr uint32_t idesc_o = umma_idesc(128, kHeads, 1, 1, 1, 0);      // pool rows: columns contiguous (M-major)
+      const uint32_t q_base = smem_u32(sq), p_base = smem_u32(sp);
+      bool ok = mbar_wait(&q_full, 0, &cta_abort, p.status);
+      // scores of tile j and the read-out of tile j - 1, whichever can start first: with two stages the next tile's load waits
+      // for the read-out, so a read-out must not wait for a tile that is still on its way
+      for (int j = 0; ok && j <= n_tiles; ++j) {
+        bool score = j < n_tiles, read = j > 0;
+        const long long since = clock64();
+        while (score || read) {
+          const int st = j % stages, sb = j & 1;
+          if (score && mbar_test_wait(&k_full[st], (j / stages) & 1) && mbar_test_wait(&s_free[sb], ((j >> 1) & 1) ^ 1u)) {
+            tc_fence_after();
+            const uint32_t k_base = smem_u32(sk + st * NB * kBlockBytes);
+            for (int b = 0; b < NB; ++b)
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
-      sc[e] = key + (e & 1) < t_end ? (s[0][e] + s[1][e] + s[2][e] + s[3][e]) * scale_log2 : -INFINITY;
-    float mx[2] = {fmaxf(sc[0], sc[1]), fmaxf(sc[2], sc[3])};
+              for (int k = 0; k < 4; ++k)
+                umma_f16(tmem + kColS + sb * 64, umma_smem_desc_sw128(q_base + b * kHeads * 128 + k * 32, 16, 1024),
+                         umma_smem_desc_sw128(k_base + b * kBlockBytes + k * 32, 16, 1024), idesc_s, (b | k) != 0);
+            umma_commit(&s_full[sb]);
+            score = false;
+          }
+          if (read && mbar_test_wait(&p_full, (j - 1) & 1)) {
+            const int sv = (j - 1) % stages;
+            tc_fence_after();
+            const uint32_t v_base = smem_u32(sk + sv * NB * kBlockBytes);
+            for (int m = 0; m < m_tiles; ++m)
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
-      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
-    }
-    if (t4 == 0) {
-      smax[warp * 16 + g] = mx[0];
-      smax[warp * 16 + g + 8] = mx[1];
-    }
-    __syncthreads();
-    float corr[2];
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      float mn = m_run[i];
-#pragma unroll
-      for (int w = 0; w < 8; ++w) mn = fmaxf(mn, smax[w * 16 + g + 8 * i]);     // (every tile has a key in it: finite)
-      corr[i] = m_run[i] == -INFINITY ? 0.f : exp2f(m_run[i] - mn);
-      m_run[i] = mn;
-      const float p0 = exp2f(sc[2 * i] - mn), p1 = exp2f(sc[2 * i + 1] - mn);
-      l_part[i] = l_part[i] * corr[i] + p0 + p1;
-      *reinterpret_cast<uint32_t*>(sp + (g + 8 * i) * kLdP + warp * 8 + 2 * t4) = pack_bf16x2(p0, p1);
-    }
-    __syncthreads();
-    uint32_t pa[4][4];
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk) ldmat_x4(pa[kk], p_addr + frag_a(lane, 0, kk * 16, kLdP));
-#pragma unroll
-    for (int i = 0; i < CT; ++i) {
-      const int col = (warp * CT + i) * 8;
-      o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1];
-#pragma unroll
-      for (int kk = 0; kk < 2; ++kk) {               // 32 keys x 8 columns per load
-        uint32_t b[4];
-        ldmat_x4_trans(b, k_addr + static_cast<uint32_t>((kk * 32 + lane) * ld + col) * 2);
-        mma_bf16(o[i], pa[2 * kk], b[0], b[1]);
-        mma_bf16(o[i], pa[2 * kk + 1], b[2], b[3]);
+              for (int k = 0; k < kKeys / 16; ++k)
+                umma_f16(tmem + kColO + m * kHeads, umma_smem_desc_sw128(v_base + m * 2 * kBlockBytes + k * 2048, kBlockBytes, 1024),
+                         umma_smem_desc_sw128(p_base + k * 32, 16, 1024), idesc_o, ((j - 1) | k) != 0);
+            umma_commit(&o_full);
+            umma_commit(&k_empty[sv]);
+            read = false;
+          }
+          if (cta_abort) ok = false;
+          if (clock64() - since > kWaitCycleLimit) {
+            cta_abort = 1;
+            if (p.status) atomicCAS(p.status, kStatusOk, kStatusMbarTimeout);
+            ok = false;
+          }
+          if (!ok) break;
+        }
       }
     }
-    __syncthreads();
-  }
-  cp_wait<0>();
+  } else {
+    // ---------------------------------------------------------------- weights (warp 0), rescaling and output (warps 0 .. 3)
+    const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
+    const float scale_log2 = p.scale * 1.4426950408889634f;
+    float m_ref = -INFINITY, l = 0.f;
+    bool good = true;
+    for (int j = 0; j < n_tiles; ++j) {
+      const int sb = j & 1;
+      uint32_t s[64];
+      if (warp == 0) {
+        bool ok = mbar_wait(&s_full[sb], (j >> 1) & 1, &cta_abort, p.status);
+        ok = __all_sync(0xffffffffu, ok ? 1 : 0) != 0;
+        float factor = 1.f;
+        bool grow = false;
+        if (ok) {
+          tc_fence_after();
+          tmem_ld_32x32(tmem + kColS + sb * 64, *reinterpret_cast<uint32_t(*)[32]>(&s[0]));
+          tmem_ld_32x32(tmem + kColS + sb * 64 + 32, *reinterpret_cast<uint32_t(*)[32]>(&s[32]));
+          tmem_ld_wait();
+          tc_fence_before();
+          mbar_arrive(&s_free[sb]);
+          const int vis = min(kKeys, t_end - (t_begin + j * kKeys));
+          float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    l_part[i] += __shfl_xor_sync(0xffffffffu, l_part[i], 1);
-    l_part[i] += __shfl_xor_sync(0xffffffffu, l_part[i], 2);
-    if (t4 == 0) ssum[warp * 16 + g + 8 * i] = l_part[i];
+          for (int i = 0; i < kKeys; ++i)
+            if (i < vis) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(s[i]));
+          const float m_tile = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+          if (j == 0) {
+            m_ref = m_tile;
+          } else if ((m_tile - m_ref) * scale_log2 > 8.f) {
+            factor = exp2f((m_ref - m_tile) * scale_log2);
+            m_ref = m_tile;
+            grow = true;
+          }
+          l *= factor;
+          const float mneg = -m_ref * scale_log2;
+          // weights as the tensor core will read them; the denominator sums those
+#pragma unroll
+          for (int i = 0; i < kKeys; i += 2) {
+            const float p0 = i < vis ? exp2f(fmaf(__uint_as_float(s[i]), scale_log2, mneg)) : 0.f;
+            const float p1 = i + 1 < vis ? exp2f(fmaf(__uint_as_float(s[i + 1]), scale_log2, mneg)) : 0.f;
+            const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
+            l += __low2float(pb) + __high2float(pb);
+            s[i >> 1] = *reinterpret_cast<const uint32_t*>(&pb);
+          }
+          // the read-out before must be finished: it reads the weights in shared memory, and rescaling rewrites its result
+          if (j > 0) ok = __all_sync(0xffffffffu, mbar_wait(&o_full, (j - 1) & 1, &cta_abort, p.status) ? 1 : 0) != 0;
+        }
+        corr[lane] = factor;
+        const bool any = __any_sync(0xffffffffu, grow);
+        if (lane == 0) grown = ok ? (any ? 1 : 0) : -1;
+      }
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+      const int what = grown;
+      if (what < 0) {
+        good = false;
+        break;
+      }
+      if (what > 0) {
+        tc_fence_after();
+        for (int m = 0; m < m_tiles; ++m) {
+          uint32_t r[32];
+          tmem_ld_32x32(tmem + lanes + kColO + m * kHeads, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * corr[i]);
+          tmem_st_32x32(tmem + lanes + kColO + m * kHeads, r);
+        }
+        tmem_st_wait();
+      }
+      if (warp == 0) {
+        uint8_t* prow = sp + lane * 128;
+#pragma unroll
+        for (int c = 0; c < 8; ++c)
+          *reinterpret_cast<uint4*>(prow + (c ^ (lane & 7)) * 16) = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
+        fence_proxy_async_smem();
+      }
+      tc_fence_before();
+      mbar_arrive(&p_full);
+    }
+    if (warp == 0) {
+      inv[lane] = p.splits > 1 ? 1.f : l > 0.f ? 1.f / l : 0.f;
+      if (p.splits > 1 && h0 + lane < p.H) {
+        float* ml = p.part_ml + ((static_cast<long long>(row) * p.H + h0 + lane) * p.splits + split) * 2;
+        ml[0] = n_tiles > 0 ? m_ref * scale_log2 : -INFINITY;
+        ml[1] = l;
+      }
+    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    bool have = false;
+    if (good && n_tiles > 0) have = mbar_wait(&o_full, (n_tiles - 1) & 1, &cta_abort, p.status);
+    have = __all_sync(0xffffffffu, have ? 1 : 0) != 0;
+    if (have) tc_fence_after();
+    for (int m = 0; m < m_tiles; ++m) {
+      uint32_t r[32];
+      if (have) {
+        tmem_ld_32x32(tmem + lanes + kColO + m * kHeads, r);
+        tmem_ld_wait();
+      } else {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) r[i] = 0u;
+      }
+      const int c = m * 128 + warp * 32 + lane;
+      if (c >= p.cp) continue;
+      const long long at = static_cast<long long>(row) * p.H + h0;
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        if (h0 + i >= p.H) break;
+        const float v = __uint_as_float(r[i]);
+        if (p.splits == 1) static_cast<__nv_bfloat16*>(p.out)[(at + i) * p.cp + c] = __float2bfloat16_rn(v * inv[i]);
+        else p.part_o[((at + i) * p.splits + split) * p.cp + c] = v;
+      }
+    }
+    tc_fence_before();
   }
   __syncthreads();
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int h = h0 + g + 8 * i;
-    if (h >= p.H) continue;
-    float l = 0.f;
-#pragma unroll
-    for (int w = 0; w < 8; ++w) l += ssum[w * 16 + g + 8 * i];
-    const long long at = static_cast<long long>(row) * p.H + h;
-    if (p.splits == 1) {
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-#pragma unroll
-      for (int c = 0; c < CT; ++c)
-        *reinterpret_cast<uint32_t*>(static_cast<T*>(p.out) + at * p.cp + (warp * CT + c) * 8 + 2 * t4) =
-            pack_bf16x2(o[c][2 * i] * inv, o[c][2 * i + 1] * inv);
-    } else {
-      const long long pi = at * p.splits + split;
-#pragma unroll
-      for (int c = 0; c < CT; ++c)
-        *reinterpret_cast<float2*>(p.part_o + pi * p.cp + (warp * CT + c) * 8 + 2 * t4) = make_float2(o[c][2 * i], o[c][2 * i + 1]);
-      if (warp == 0 && t4 == 0) {
-        p.part_ml[pi * 2] = m_run[i];
-        p.part_ml[pi * 2 + 1] = l;
-      }
-    }
+  if (warp == 5) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 256);
   }
 }
 
@@ -456,19 +572,23 @@ latent_rows_kernel(LatentAttnParams p) {
     if (lane + 32 * i < p.cp) out[lane + 32 * i] = from_f32<T>(o[i] * inv);
 }
 
-template <int CT>
 int launch_latent_decode(const LatentAttnParams& p, cudaStream_t s) {
-  const int ld = p.cp + p.rp + 8;
-  const int smem = (16 * ld + 2 * kKeys * ld + 16 * (kKeys + 8)) * 2 + 2 * 8 * 16 * 4;
-  if (smem > 227 * 1024) return -2;
-  auto kern = latent_decode_kernel<CT>;
+  const int L = p.cp + p.rp;
+  if (LatentSmem::stages(L) < 2) return -2;
   static PerDeviceFlag attr;
   if (attr.unset()) {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 1024);
     if (e != cudaSuccess) return static_cast<int>(e);
     attr.set();
   }
-  launch_pdl(kern, dim3(p.splits, (p.H + 15) / 16, p.rows), dim3(256), smem, s, pdl_all_enabled(), p);
+  int run = 64;
+  while (p.bs % run) run >>= 1;
+  CUtensorMap tm_q, tm_pool;
+  if (!make_tmap_2d(&tm_q, p.q, 2, static_cast<uint64_t>(p.rows) * p.H, L, L * 2ull, kHeads, 64, true) ||
+      !make_tmap_2d(&tm_pool, p.pool, 2, static_cast<uint64_t>(p.nb) * p.bs, L, L * 2ull, run, 64, true))
+    return -3;
+  launch_pdl(latent_decode_kernel, dim3(p.splits, (p.H + kHeads - 1) / kHeads, p.rows), dim3(192), LatentSmem::bytes(L), s,
+             pdl_all_enabled(), tm_q, tm_pool, p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -547,7 +667,7 @@ TSB_EXPORT int tsb_head_linear(const void* x, long long ldx, int xh, const void*
   if (rows <= 0 || H <= 0 || H > 65535 || N <= 0 || N % 2 || K <= 0 || K % 16 || ldx % 8 || xh % 8 || wh % 8 || ldw % 8 || ldw < K || ldo % 2 || oh % 2) return -2;
   HeadLinearParams p{x, ldx, xh, w, wh, ldw, out, ldo, oh, gate, ldg, gate_scale, rows, N, K};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const bool few = rows <= 32;
+  const bool few = rows <= 64 || static_cast<long long>((rows + 63) / 64) * H * ((N + 63) / 64) < 4ll * sm_count();
   if (!few && (rows + 63) / 64 > 65535) return -2;
   if (dtype == 1) return few ? launch_head_linear<__nv_bfloat16, 16>(p, H, s) : launch_head_linear<__nv_bfloat16, 64>(p, H, s);
   if (dtype == 0) return few ? launch_head_linear<float, 16>(p, H, s) : launch_head_linear<float, 64>(p, H, s);
@@ -589,18 +709,8 @@ TSB_EXPORT int tsb_latent_attn(const void* q, const void* pool, const int* table
     if (dtype == 1) return launch_latent_rows<__nv_bfloat16>(p, s);
     return dtype == 0 ? launch_latent_rows<float>(p, s) : -2;
   }
-  if (dtype != 1 || cp % 64 || cp > 512 || rp % 32 || rows > 65535 || (splits > 1 && (!part_o || !part_ml))) return -2;
-  int rc;
-  switch (cp / 64) {
-    case 1: rc = launch_latent_decode<1>(p, s); break;
-    case 2: rc = launch_latent_decode<2>(p, s); break;
-    case 3: rc = launch_latent_decode<3>(p, s); break;
-    case 4: rc = launch_latent_decode<4>(p, s); break;
-    case 5: rc = launch_latent_decode<5>(p, s); break;
-    case 6: rc = launch_latent_decode<6>(p, s); break;
-    case 7: rc = launch_latent_decode<7>(p, s); break;
-    default: rc = launch_latent_decode<8>(p, s); break;
-  }
+  if (dtype != 1 || cp % 64 || cp > 512 || rp % 32 || rp <= 0 || bs % 8 || rows > 65535 || (splits > 1 && (!part_o || !part_ml))) return -2;
+  const int rc = launch_latent_decode(p, s);
   if (rc || splits == 1) return rc;
   launch_pdl(latent_merge_kernel, dim3(static_cast<unsigned>(rows * H)), dim3(128), 0, s, pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());

@@ -12,7 +12,7 @@
 //   retention_span_kernel<.., true>   the read-outs:  o_i = decay^(i+1) q_i S + sum_{j <= i} decay^(i-j) (q_i . k_j) v_j
 //                                     and the update   S <- decay^n S + sum_j decay^(n-1-j) k_j v_j^T  chunk by chunk
 // S lives in fp32 accumulators. Where a factor that must not lose its 32 bits meets the tensor cores (S in the read-out, the
-// decayed values in the update, the decayed scores), it goes in as two bf16 halves whose sum carries 16 bits.
+// decayed keys in the update, the decayed scores), it goes in as two bf16 halves whose sum carries 16 bits.
 // fp32 models take retention_scan_kernel (token by token, state in registers) and retention_norm_kernel.
 // Decoded tokens take retention_step_kernel: the state streams through registers once.
 #include "warp_mma.cuh"
@@ -52,12 +52,15 @@ struct RetParams {
 __device__ __forceinline__ float decay_pow(float log2_decay, int n) { return exp2f(log2_decay * static_cast<float>(n)); }
 
 // ------------------------------------------------------------------ prompts, bf16
-template <int DT, int ET>
+template <int DT, int ET, bool OUT>
 struct SpanCfg {
+  static constexpr int kBuf = DT <= 128 ? 2 : 1;       // chunks in shared memory: the next one arrives while one is worked on
   static constexpr int kLdQ = DT + 8, kLdV = ET + 8;
-  static constexpr int kQ = 0, kK = kQ + kTok * kLdQ, kV = kK + kTok * kLdQ, kVh = kV + kTok * kLdV, kVl = kVh + kTok * kLdV,
-                       kSh = kVl + kTok * kLdV, kSl = kSh + DT * kLdV, kEnd = kSl + DT * kLdV;
-  static constexpr int kSmem = kEnd * 2 + 2 * kTok * 4;
+  // elements of a chunk's buffers (q is only there for read-outs), then what exists once
+  static constexpr int kK = 0, kQ = kK + kTok * kLdQ, kV = kQ + (OUT ? kTok * kLdQ : 0), kChunkElems = kV + kTok * kLdV;
+  static constexpr int kSh = kBuf * kChunkElems, kSl = kSh + (OUT ? DT * kLdV : 0), kElems = kSl + (OUT ? DT * kLdV : 0);
+  static constexpr int kTable = kElems * 2, kRow = kTable + kTok * DT / 2 * 8;
+  static constexpr int kSmem = kRow + 2 * kTok * 4;
   // fragments of S: warp w holds kMT blocks of 16 rows x kNT blocks of 8 columns
   static constexpr int kMT = DT >= 128 ? DT / 128 : 1;
   static constexpr int kNT = DT >= 128 ? ET / 8 : ET / 16;
@@ -68,12 +71,13 @@ template <int DT, int ET, bool OUT>
 __global__ void __launch_bounds__(256)
 retention_span_kernel(RetParams p) {
   using T = __nv_bfloat16;
-  using C = SpanCfg<DT, ET>;
+  using C = SpanCfg<DT, ET, OUT>;
   pdl_trigger();
   pdl_grid_wait();
   extern __shared__ __align__(16) uint8_t smem[];
   T* sm = reinterpret_cast<T*>(smem);
-  float* srow = reinterpret_cast<float*>(smem + C::kEnd * 2);      // [2][kTok]
+  float2* stab = reinterpret_cast<float2*>(smem + C::kTable);      // [kTok][hp] cos, sin
+  float* srow = reinterpret_cast<float*>(smem + C::kRow);          // [2][kTok]
   const int span = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * ET;
   const int seq = p.tile_seq[span], idx = span - p.tile0[seq], n_spans = p.tile0[seq + 1] - p.tile0[seq];
   const int slot = p.slots[seq];
@@ -85,6 +89,31 @@ retention_span_kernel(RetParams p) {
   const long long head_state = static_cast<long long>(p.dp) * p.vp;
   float* st = p.state + (static_cast<long long>(slot) * p.H + h) * head_state;
   float* cr = p.carry ? p.carry + (static_cast<long long>(span) * p.H + h) * head_state : nullptr;
+  const T* proj = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ldp;
+
+  // one chunk as it is in memory; rows and columns that do not exist arrive as zeros
+  auto issue = [&](int t0) {
+    T* buf = sm + (C::kBuf == 2 ? (t0 / kTok & 1) : 0) * C::kChunkElems;
+    const int cnt = min(kTok, n - t0);
+    const T* src = proj + static_cast<long long>(t0) * p.ldp;
+    constexpr int kPQ = DT / 8, kPV = ET / 8;
+    for (int i = tid; i < kTok * kPQ; i += 256) {
+      const int r = i / kPQ, d = (i % kPQ) * 8;
+      const bool ok = r < cnt && d < p.dp;
+      const T* q = ok ? src + r * p.ldp + h * p.dp + d : proj;
+      cp_async_16(smem_u32(buf + C::kK + r * C::kLdQ + d), ok ? q + p.off_k : q, ok ? 16 : 0);
+      if constexpr (OUT) cp_async_16(smem_u32(buf + C::kQ + r * C::kLdQ + d), q, ok ? 16 : 0);
+    }
+    for (int i = tid; i < kTok * kPV; i += 256) {
+      const int r = i / kPV, c = (i % kPV) * 8;
+      const bool ok = r < cnt && e0 + c < p.vp;
+      cp_async_16(smem_u32(buf + C::kV + r * C::kLdV + c), ok ? src + r * p.ldp + p.off_v + h * p.vp + e0 + c : proj, ok ? 16 : 0);
+    }
+    const float2* tab = p.table + static_cast<long long>(pos + t0) * p.hp;     // rows of consecutive positions: one run
+    for (int i = tid * 2; i < cnt * p.hp; i += 512) cp_async_16(smem_u32(stab + i), tab + i, 16);
+    cp_commit();
+  };
+  issue(0);
 
   const int m0 = DT >= 128 ? warp * C::kMT * 16 : (warp & 3) * 16, n0 = DT >= 128 ? 0 : (warp >> 2) * (ET / 2);
   float S[C::kMT][C::kNT][4];
@@ -103,44 +132,45 @@ retention_span_kernel(RetParams p) {
           S[i][j][2 * e + 1] = v.y;
         }
   }
-  const T* proj = static_cast<const T*>(p.proj);
-  const uint32_t aQ = smem_u32(sm + C::kQ), aK = smem_u32(sm + C::kK), aV = smem_u32(sm + C::kV), aVh = smem_u32(sm + C::kVh),
-                 aVl = smem_u32(sm + C::kVl), aSh = smem_u32(sm + C::kSh), aSl = smem_u32(sm + C::kSl);
+  const uint32_t aSh = smem_u32(sm + C::kSh), aSl = smem_u32(sm + C::kSl);
   for (int t0 = 0; t0 < n; t0 += kTok) {
     const int cnt = min(kTok, n - t0);
-    __syncthreads();
-    constexpr int kPQ = DT / 8, kPV = ET / 8;
-    for (int i = tid; i < kTok * kPQ; i += 256) {
-      const int r = i / kPQ, d = (i % kPQ) * 8;
-      float q[8] = {}, k[8] = {};
-      if (r < cnt && d < p.dp) {
-        const T* head = proj + static_cast<long long>(row0 + t0 + r) * p.ldp + h * p.dp;
-        const float2* table = p.table + static_cast<long long>(pos + t0 + r) * p.hp;
-        rotated_piece<T>(head + p.off_k, d, p.hp, table, k);
-        if constexpr (OUT) rotated_piece<T>(head, d, p.hp, table, q);
+    T* buf = sm + (C::kBuf == 2 ? (t0 / kTok & 1) : 0) * C::kChunkElems;
+    cp_wait<0>();
+    __syncthreads();                       // the chunk has arrived, and everyone is done with the one before
+    {
+      // scale, and rotate in place: a thread takes both halves of eight pairs
+      const int np = p.hp / 8, per = np + (p.dp - 2 * p.hp) / 8;
+      for (int i = tid; i < cnt * per; i += 256) {
+        const int r = i / per, w = i % per;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          q[e] *= p.in_scale;
-          k[e] *= p.k_scale;
+        for (int which = 0; which < (OUT ? 2 : 1); ++which) {
+          T* x = buf + (which ? C::kQ : C::kK) + r * C::kLdQ;
+          const float s = which ? p.in_scale : p.k_scale;
+          float u[8];
+          if (w < np) {
+            float v[8], a[8], b[8];
+            ld16<T>(x + w * 8, u);
+            ld16<T>(x + p.hp + w * 8, v);
+#pragma unroll
+            for (int e = 0; e < 8; e += 2) {
+              const float4 cs = *reinterpret_cast<const float4*>(stab + r * p.hp + w * 8 + e);
+              a[e] = (u[e] * cs.x - v[e] * cs.y) * s;
+              b[e] = (v[e] * cs.x + u[e] * cs.y) * s;
+              a[e + 1] = (u[e + 1] * cs.z - v[e + 1] * cs.w) * s;
+              b[e + 1] = (v[e + 1] * cs.z + u[e + 1] * cs.w) * s;
+            }
+            st16<T>(x + w * 8, a);
+            st16<T>(x + p.hp + w * 8, b);
+          } else {
+            const int d = 2 * p.hp + (w - np) * 8;
+            ld16<T>(x + d, u);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) u[e] *= s;
+            st16<T>(x + d, u);
+          }
         }
       }
-      st16<T>(sm + C::kK + r * C::kLdQ + d, k);
-      if constexpr (OUT) st16<T>(sm + C::kQ + r * C::kLdQ + d, q);
-    }
-    for (int i = tid; i < kTok * kPV; i += 256) {
-      const int r = i / kPV, c = (i % kPV) * 8;
-      uint4 raw = make_uint4(0, 0, 0, 0), hi = raw, lo = raw;
-      if (r < cnt && e0 + c < p.vp) {
-        raw = *reinterpret_cast<const uint4*>(proj + static_cast<long long>(row0 + t0 + r) * p.ldp + p.off_v + h * p.vp + e0 + c);
-        const float w = decay_pow(lg, cnt - 1 - r);
-        const T* v = reinterpret_cast<const T*>(&raw);
-        uint32_t *ph = reinterpret_cast<uint32_t*>(&hi), *pl = reinterpret_cast<uint32_t*>(&lo);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) split_bf16x2(to_f32<T>(v[2 * e]) * w, to_f32<T>(v[2 * e + 1]) * w, ph + e, pl + e);
-      }
-      if constexpr (OUT) *reinterpret_cast<uint4*>(sm + C::kV + r * C::kLdV + c) = raw;
-      *reinterpret_cast<uint4*>(sm + C::kVh + r * C::kLdV + c) = hi;
-      *reinterpret_cast<uint4*>(sm + C::kVl + r * C::kLdV + c) = lo;
     }
     if constexpr (OUT) {
 #pragma unroll
@@ -155,6 +185,8 @@ retention_span_kernel(RetParams p) {
           }
     }
     __syncthreads();
+    if (C::kBuf == 2 && t0 + kTok < n) issue(t0 + kTok);
+    const uint32_t aQ = smem_u32(buf + C::kQ), aK = smem_u32(buf + C::kK), aV = smem_u32(buf + C::kV);
     if constexpr (OUT) {
       const int rg = warp & 3, r0 = rg * 16, c0 = (warp >> 2) * (ET / 2);
       float acc[C::kOT][4];
@@ -225,6 +257,14 @@ retention_span_kernel(RetParams p) {
             if (e0 + c0 + j * 8 + 2 * t4 < p.vp) *reinterpret_cast<float2*>(o + j * 8 + 2 * t4) = make_float2(acc[j][2 * e], acc[j][2 * e + 1]);
         }
       } else {
+        __nv_bfloat162 gate[2][C::kOT];            // requested before the norm's barrier
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int r = min(r0 + g + 8 * e, cnt - 1);
+          const T* gr = proj + (t0 + r) * p.ldp + p.off_g + h * p.vp;
+#pragma unroll
+          for (int j = 0; j < C::kOT; ++j) gate[e][j] = *reinterpret_cast<const __nv_bfloat162*>(gr + min(c0 + j * 8 + 2 * t4, p.vp - 2));
+        }
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           float ss = 0.f;
@@ -240,15 +280,12 @@ retention_span_kernel(RetParams p) {
           const int r = r0 + g + 8 * e;
           if (r >= cnt) continue;
           const float rs = rsqrtf((srow[r] + srow[kTok + r]) / static_cast<float>(p.vdim) + p.eps);
-          const long long row = row0 + t0 + r;
-          const T* gate = proj + row * p.ldp + p.off_g + h * p.vp;
-          T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.vp;
+          T* out = static_cast<T*>(p.out) + static_cast<long long>(row0 + t0 + r) * p.ldo + h * p.vp;
 #pragma unroll
           for (int j = 0; j < C::kOT; ++j) {
             const int c = c0 + j * 8 + 2 * t4;
             if (c >= p.vp) continue;
-            const __nv_bfloat162 gg = *reinterpret_cast<const __nv_bfloat162*>(gate + c);
-            const float g0 = p.in_scale * __low2float(gg), g1 = p.in_scale * __high2float(gg);
+            const float g0 = p.in_scale * __low2float(gate[e][j]), g1 = p.in_scale * __high2float(gate[e][j]);
             *reinterpret_cast<uint32_t*>(out + c) =
                 pack_bf16x2(acc[j][2 * e] * rs * __fdividef(g0, 1.f + __expf(-g0)), acc[j][2 * e + 1] * rs * __fdividef(g1, 1.f + __expf(-g1)));
           }
@@ -265,21 +302,39 @@ retention_span_kernel(RetParams p) {
 #pragma unroll
     for (int ks = 0; ks < kTok / 16; ++ks) {
       if (ks * 16 >= cnt) break;
+      float w[4];                          // what is left of tokens 16 ks + 2 t, + 1, + 8, + 9 at the end of the chunk
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int back = cnt - 1 - (ks * 16 + 2 * t4 + (e & 1) + (e >> 1) * 8);
+        w[e] = back < 0 ? 0.f : decay_pow(lg, back);
+      }
+      uint32_t hi[C::kMT][4], lo[C::kMT][4];
 #pragma unroll
       for (int i = 0; i < C::kMT; ++i) {
         uint32_t a[4];
         ldmat_x4_trans(a, aK + frag_a_trans(lane, ks * 16, m0 + i * 16, C::kLdQ));
 #pragma unroll
-        for (int j = 0; j < C::kNT; j += 2) {
-          uint32_t b[4];
-          ldmat_x4_trans(b, aVh + frag_b_trans(lane, ks * 16, n0 + j * 8, C::kLdV));
-          mma_bf16(S[i][j], a, b[0], b[1]);
-          mma_bf16(S[i][j + 1], a, b[2], b[3]);
-          ldmat_x4_trans(b, aVl + frag_b_trans(lane, ks * 16, n0 + j * 8, C::kLdV));
-          mma_bf16(S[i][j], a, b[0], b[1]);
-          mma_bf16(S[i][j + 1], a, b[2], b[3]);
+        for (int e = 0; e < 4; ++e) {
+          const __nv_bfloat162 k = *reinterpret_cast<const __nv_bfloat162*>(&a[e]);
+          split_bf16x2(__low2float(k) * w[e & 2], __high2float(k) * w[(e & 2) + 1], &hi[i][e], &lo[i][e]);
         }
       }
+#pragma unroll
+      for (int j = 0; j < C::kNT; j += 2) {
+        uint32_t b[4];
+        ldmat_x4_trans(b, aV + frag_b_trans(lane, ks * 16, n0 + j * 8, C::kLdV));
+#pragma unroll
+        for (int i = 0; i < C::kMT; ++i) {
+          mma_bf16(S[i][j], hi[i], b[0], b[1]);
+          mma_bf16(S[i][j + 1], hi[i], b[2], b[3]);
+          mma_bf16(S[i][j], lo[i], b[0], b[1]);
+          mma_bf16(S[i][j + 1], lo[i], b[2], b[3]);
+        }
+      }
+    }
+    if (C::kBuf == 1 && t0 + kTok < n) {
+      __syncthreads();
+      issue(t0 + kTok);
     }
   }
   float* dst = !OUT ? cr : idx == n_spans - 1 ? st : nullptr;
@@ -526,8 +581,8 @@ template <int DT, int ET, bool OUT>
 int launch_span(const RetParams& p, cudaStream_t s) {
   auto kern = retention_span_kernel<DT, ET, OUT>;
   static PerDeviceFlag attr;
-  if (const int e = opt_in_smem(kern, &attr, SpanCfg<DT, ET>::kSmem)) return e;
-  launch_pdl(kern, dim3(p.spans, p.H, (p.vp + ET - 1) / ET), dim3(256), SpanCfg<DT, ET>::kSmem, s, pdl_all_enabled(), p);
+  if (const int e = opt_in_smem(kern, &attr, SpanCfg<DT, ET, OUT>::kSmem)) return e;
+  launch_pdl(kern, dim3(p.spans, p.H, (p.vp + ET - 1) / ET), dim3(256), SpanCfg<DT, ET, OUT>::kSmem, s, pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());
 }
 

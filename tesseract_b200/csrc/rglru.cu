@@ -66,66 +66,130 @@ struct RglruParams {
   long long ldo;
 };
 
-__device__ __forceinline__ float gelu_tanh_f32(float z) {
+// FAST (bf16 models): hardware exponentials and divisions, good to a few fp32 roundings; fp32 models take the exact ones.
+template <bool FAST>
+__device__ __forceinline__ float sigmoid_g(float x) {
+  if constexpr (FAST) return __fdividef(1.f, 1.f + __expf(-x));
+  return sigmoid_f32(x);
+}
+template <bool FAST>
+__device__ __forceinline__ float gelu_tanh_g(float z) {
   constexpr float k = 0.79788456080286535588f;     // sqrt(2 / pi)
-  return 0.5f * z * (1.f + tanhf(k * fmaf(0.044715f * z * z, z, z)));
+  const float w = k * fmaf(0.044715f * z * z, z, z);
+  // (1 + tanh w) / 2 = 1 / (1 + exp(-2 w))
+  if constexpr (FAST) return __fdividef(z, 1.f + __expf(-2.f * w));
+  return 0.5f * z * (1.f + tanhf(w));
 }
 struct Gates {
   float a, b;                   // S <- a S + b
 };
+template <bool FAST>
 __device__ __forceinline__ Gates rglru_gates(float r_lin, float i_lin, float decay, float u) {
-  const float log_a = -sigmoid_f32(r_lin) * decay;
-  return {expf(log_a), sqrtf(-expm1f(2.f * log_a)) * sigmoid_f32(i_lin) * u};
+  const float x = -sigmoid_g<FAST>(r_lin) * decay;
+  if constexpr (FAST) {
+    // 1 - a^2 = -(exp(2 x) - 1): by its Taylor series where the difference would cancel (|2 x| < 1/4: the first dropped term
+    // is below 2e-6 of the sum)
+    const float y = 2.f * x, a = __expf(x);
+    const float series = -y * fmaf(y, fmaf(y, fmaf(y, fmaf(y, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+    const float q = y > -0.25f ? series : fmaf(-a, a, 1.f);
+    return {a, sqrtf(q) * sigmoid_g<true>(i_lin) * u};
+  }
+  return {expf(x), sqrtf(-expm1f(2.f * x)) * sigmoid_f32(i_lin) * u};
 }
 
-// A thread takes one 16-byte piece of channels of one row.
-template <typename T>
+// A thread takes one 16-byte piece of channels of kConvRows rows; the inputs before a row stay in registers as a window. TAPS = 0:
+// any number of taps, every input loaded again.
+constexpr int kConvRows = 8;
+
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(256)
 rglru_conv_kernel(RglruParams p) {
   pdl_trigger();
   pdl_grid_wait();
-  constexpr int V = kVec16<T>;
+  constexpr int V = kVec16<T>, W = TAPS > 0 ? TAPS : 1;
   const unsigned per = p.C / V, idx = blockIdx.x * 256u + threadIdx.x;
-  const int row = static_cast<int>(idx / per), c = static_cast<int>(idx % per) * V;
-  if (row >= p.rows) return;
-  const int tail = p.taps - 1;
-  const T* x = static_cast<const T*>(p.proj) + row * p.ldp + c;
-  T* u = static_cast<T*>(p.u) + static_cast<long long>(row) * p.C + c;
-  float acc[V], bias[V];
-  const bool decoded = row < p.n_dec;
-  const int seq = decoded ? row : p.seq_of[row];
-  const int slot = p.slots[seq];
-  if (slot < 0) {
-#pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = 0.f;
-    st16<T>(u, acc);
-    return;
+  const int c = static_cast<int>(idx % per) * V;
+  // decoded rows one by one, then the portions' rows kConvRows at a time
+  int row = static_cast<int>(idx / per), last = row;
+  if (row >= p.n_dec) {
+    row = p.n_dec + (row - p.n_dec) * kConvRows;
+    if (row >= p.rows) return;
+    last = min(row + kConvRows, p.rows) - 1;
   }
-  T* st = static_cast<T*>(p.conv_state) + static_cast<long long>(slot) * tail * p.C + c;
-  const int first = decoded ? row : p.n_dec + p.cu[seq - p.n_dec];      // first row of this sequence in the batch
-  const int pos = p.positions[row];
+  const int tail = p.taps - 1;
+  float bias[V], cb[V], w[W][V];
 #pragma unroll
   for (int i = 0; i < V; ++i) {
-    acc[i] = p.conv_b[c + i];
+    cb[i] = p.conv_b[c + i];
     bias[i] = p.x_bias[c + i];
   }
-  for (int j = 0; j <= tail; ++j) {
-    const int back = tail - j;                     // tokens before this one
-    if (back > pos) continue;                      // before the start of the sequence
-    float v[V];
-    const int at = row - back - first;             // negative: in the slot, which holds the last `tail` inputs
-    if (at >= 0) ld16<T>(x - back * p.ldp, v);
-    else ld16<T>(st + static_cast<long long>(tail + at) * p.C, v);
-    const float* w = p.conv_w + static_cast<long long>(j) * p.C + c;
+  if constexpr (TAPS > 0) {
 #pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = fmaf(w[i], fmaf(v[i], p.in_scale, bias[i]), acc[i]);
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < V; ++i) w[j][i] = p.conv_w[static_cast<long long>(j) * p.C + c + i];
   }
-  st16<T>(u, acc);
-  if (decoded) {
-    for (int j = 0; j < tail; ++j) {
-      uint4 next = *reinterpret_cast<const uint4*>(x);
-      if (j + 1 < tail) next = *reinterpret_cast<const uint4*>(st + static_cast<long long>(j + 1) * p.C);
-      *reinterpret_cast<uint4*>(st + static_cast<long long>(j) * p.C) = next;
+  float win[W][V];
+  for (int first_row = row; row <= last; ++row) {
+    const T* x = static_cast<const T*>(p.proj) + row * p.ldp + c;
+    T* u = static_cast<T*>(p.u) + static_cast<long long>(row) * p.C + c;
+    float acc[V];
+    const bool decoded = row < p.n_dec;
+    const int seq = decoded ? row : p.seq_of[row];
+    const int slot = p.slots[seq];
+    if (slot < 0) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) acc[i] = 0.f;
+      st16<T>(u, acc);
+      continue;
+    }
+    T* st = static_cast<T*>(p.conv_state) + static_cast<long long>(slot) * tail * p.C + c;
+    const int start = decoded ? row : p.n_dec + p.cu[seq - p.n_dec];      // first row of this sequence in the batch
+    const int pos = p.positions[row];
+#pragma unroll
+    for (int i = 0; i < V; ++i) acc[i] = cb[i];
+    auto input = [&](int back, float (&v)[V]) {      // the input `back` tokens ago, with scale and bias
+      const int at = row - back - start;             // negative: in the slot, which holds the last `tail` inputs
+      if (back > pos) {                              // before the start of the sequence
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = 0.f;
+        return;
+      }
+      if (at >= 0) ld16<T>(x - back * p.ldp, v);
+      else ld16<T>(st + static_cast<long long>(tail + at) * p.C, v);
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] = fmaf(v[i], p.in_scale, bias[i]);
+    };
+    if constexpr (TAPS > 0) {
+      if (row == first_row || row == start) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) input(TAPS - 1 - j, win[j]);
+      } else {
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+          for (int i = 0; i < V; ++i) win[j][i] = win[j + 1][i];
+        input(0, win[TAPS - 1]);
+      }
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = fmaf(w[j][i], win[j][i], acc[i]);
+    } else {
+      for (int j = 0; j <= tail; ++j) {
+        input(tail - j, win[0]);
+        const float* wj = p.conv_w + static_cast<long long>(j) * p.C + c;
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = fmaf(wj[i], win[0][i], acc[i]);
+      }
+    }
+    st16<T>(u, acc);
+    if (decoded) {
+      for (int j = 0; j < tail; ++j) {
+        uint4 next = *reinterpret_cast<const uint4*>(x);
+        if (j + 1 < tail) next = *reinterpret_cast<const uint4*>(st + static_cast<long long>(j + 1) * p.C);
+        *reinterpret_cast<uint4*>(st + static_cast<long long>(j) * p.C) = next;
+      }
     }
   }
 }
@@ -153,13 +217,13 @@ rglru_step_kernel(RglruParams p) {
       *out = from_f32<T>(0.f);
       continue;
     }
-    const Gates g = rglru_gates(acc[m * Tile::kLdC + n] + p.ra_b[c], acc[(BM + m) * Tile::kLdC + n] + p.ri_b[c], p.decay[c],
+    const Gates g = rglru_gates<sizeof(T) == 2>(acc[m * Tile::kLdC + n] + p.ra_b[c], acc[(BM + m) * Tile::kLdC + n] + p.ri_b[c], p.decay[c],
                                 to_f32<T>(u[static_cast<long long>(m) * p.C + n0 + n]));
     float* st = p.state + static_cast<long long>(slot) * p.C + c;
     const float s = fmaf(g.a, p.positions[row] > 0 ? *st : 0.f, g.b);
     *st = s;
     const float y = fmaf(to_f32<T>(static_cast<const T*>(p.proj)[row * p.ldp + p.off_y + c]), p.in_scale, p.y_bias[c]);
-    *out = from_f32<T>(s * gelu_tanh_f32(y));
+    *out = from_f32<T>(s * gelu_tanh_g<sizeof(T) == 2>(y));
   }
 }
 
@@ -189,7 +253,7 @@ rglru_chunk_kernel(RglruParams p) {
     for (int m = tid >> 6; m < rows; m += 2) {
       const float uu = ok ? to_f32<T>(u[static_cast<long long>(m) * p.C + n0 + n]) : 0.f;
       const int at = m * Tile::kLdC + n;
-      const Gates g = rglru_gates(sa[at] + rb, sb[at] + ib, dc, uu);
+      const Gates g = rglru_gates<sizeof(T) == 2>(sa[at] + rb, sb[at] + ib, dc, uu);
       sa[at] = g.a;
       sb[at] = g.b;
     }
@@ -278,10 +342,10 @@ rglru_apply_kernel(RglruParams p) {
       const float4 r = *reinterpret_cast<const float4*>(yp);
       y[0] = r.x; y[1] = r.y; y[2] = r.z; y[3] = r.w;
     }
-    const float z0 = fmaf(a.x, in.x, s.x) * gelu_tanh_f32(fmaf(y[0], p.in_scale, yb.x));
-    const float z1 = fmaf(a.y, in.y, s.y) * gelu_tanh_f32(fmaf(y[1], p.in_scale, yb.y));
-    const float z2 = fmaf(a.z, in.z, s.z) * gelu_tanh_f32(fmaf(y[2], p.in_scale, yb.z));
-    const float z3 = fmaf(a.w, in.w, s.w) * gelu_tanh_f32(fmaf(y[3], p.in_scale, yb.w));
+    const float z0 = fmaf(a.x, in.x, s.x) * gelu_tanh_g<sizeof(T) == 2>(fmaf(y[0], p.in_scale, yb.x));
+    const float z1 = fmaf(a.y, in.y, s.y) * gelu_tanh_g<sizeof(T) == 2>(fmaf(y[1], p.in_scale, yb.y));
+    const float z2 = fmaf(a.z, in.z, s.z) * gelu_tanh_g<sizeof(T) == 2>(fmaf(y[2], p.in_scale, yb.z));
+    const float z3 = fmaf(a.w, in.w, s.w) * gelu_tanh_g<sizeof(T) == 2>(fmaf(y[3], p.in_scale, yb.w));
     T* out = static_cast<T*>(p.out) + row * p.ldo + c;
     if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(out) = make_uint2(pack_bf16x2(z0, z1), pack_bf16x2(z2, z3));
     else *reinterpret_cast<float4*>(out) = make_float4(z0, z1, z2, z3);
@@ -312,11 +376,18 @@ int run_rglru(const RglruParams& p, cudaStream_t s) {
   const bool pdl = pdl_all_enabled();
   const long long pieces = static_cast<long long>(p.rows) * (p.C / kVec16<T>);
   if (pieces > 0x7fffff00LL) return -2;
-  launch_pdl(rglru_conv_kernel<T>, dim3(static_cast<unsigned>((pieces + 255) / 256)), dim3(256), 0, s, pdl, p);
+  const long long threads = (p.n_dec + (p.rows - p.n_dec + kConvRows - 1) / kConvRows) * static_cast<long long>(p.C / kVec16<T>);
+  const dim3 cgrid(static_cast<unsigned>((threads + 255) / 256));
+  switch (p.taps) {
+    case 2: launch_pdl(rglru_conv_kernel<T, 2>, cgrid, dim3(256), 0, s, pdl, p); break;
+    case 3: launch_pdl(rglru_conv_kernel<T, 3>, cgrid, dim3(256), 0, s, pdl, p); break;
+    case 4: launch_pdl(rglru_conv_kernel<T, 4>, cgrid, dim3(256), 0, s, pdl, p); break;
+    default: launch_pdl(rglru_conv_kernel<T, 0>, cgrid, dim3(256), 0, s, pdl, p); break;
+  }
   int rc = static_cast<int>(cudaGetLastError());
   if (rc) return rc;
   if (p.n_dec > 0) {
-    rc = p.n_dec <= 32 ? launch_step<T, 16>(p, s) : launch_step<T, 64>(p, s);
+    rc = p.n_dec <= 512 ? launch_step<T, 16>(p, s) : launch_step<T, 64>(p, s);
     if (rc) return rc;
   }
   if (p.rows > p.n_dec) {

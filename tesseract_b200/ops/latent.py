@@ -33,7 +33,6 @@ _native.register_signatures({
 })
 
 MAX_ROW = 1024
-SMEM_LIMIT = 227 * 1024
 
 
 def _up(n: int, m: int) -> int:
@@ -106,9 +105,9 @@ class LatentGeometry:
     def written_out(self, dtype) -> bool:
         return dtype == torch.bfloat16 and self.D <= 128
 
-    def tensor_cores(self, dtype) -> bool:
-        """Whether single rows run on ``latent_decode_kernel`` (its two key tiles and the queries fit in shared memory)."""
-        return dtype == torch.bfloat16 and self.cp <= 512 and (16 + 2 * 64) * (self.row + 8) * 2 + 4096 <= SMEM_LIMIT
+    def tensor_cores(self, dtype, block: int) -> bool:
+        """Whether single rows run on ``latent_decode_kernel`` (two tiles of keys and the queries fit in shared memory)."""
+        return dtype == torch.bfloat16 and self.cp <= 512 and self.row <= 704 and block % 8 == 0
 
 
 @dataclass
@@ -124,12 +123,11 @@ class LatentWeights:
 
 
 def _splits(rows: int, geo: LatentGeometry, max_len: int) -> int:
-    """Key splits of the decode kernel: the number that leaves the fewest idle SM slots, no split shorter than two tiles of
-    the longest sequence."""
-    ctas = rows * ((geo.heads + 15) // 16)
-    slots = 148 * max(1, SMEM_LIMIT // ((16 + 2 * 64) * (geo.row + 8) * 2 + 4096))
-    most = max(1, min((max_len + 127) // 128, 64, (2 * slots + ctas - 1) // ctas))
-    return min(range(1, most + 1), key=lambda s: (-(-ctas * s // slots) / s + 0.004 * s))
+    """Key splits of the decode kernel (one CTA per SM): fewest waves times the tiles of a split, plus what a CTA spends before
+    and after its tiles."""
+    ctas, tiles = rows * ((geo.heads + 31) // 32), (max_len + 63) // 64
+    most = max(1, min((tiles + 1) // 2, 64, 4 * 148 // ctas + 4))
+    return min(range(1, most + 1), key=lambda s: -(-ctas * s // 148) * (-(-tiles // s) + 2))
 
 
 def latent_attention(proj: torch.Tensor, geo: LatentGeometry, w: LatentWeights, pool: torch.Tensor, table: torch.Tensor, batch,
@@ -168,7 +166,7 @@ def latent_attention(proj: torch.Tensor, geo: LatentGeometry, w: LatentWeights, 
         lat = torch.empty((nl, H, geo.cp), **new)
         tables = batch.tables
         single = nl == batch.n_decode                   # row i is sequence i, lengths are at hand
-        fast = geo.tensor_cores(proj.dtype)
+        fast = geo.tensor_cores(proj.dtype, bs)
         splits = _splits(nl, geo, batch.max_len) if fast else 0
         part_o = torch.empty((nl, H, splits, geo.cp), device=dev, dtype=torch.float32) if splits > 1 else None
         part_ml = torch.empty((nl, H, splits, 2), device=dev, dtype=torch.float32) if splits > 1 else None
