@@ -21,30 +21,36 @@ struct HeadTile {
   static constexpr int kSmem = kRing > kOut ? kRing : kOut;
 
   // x: first row of the tile (row stride ldx, `rows` of them exist); w[i]: first matrix row of the tile (row stride ldw,
-  // `cols` of them exist). K is a multiple of 16; all starts and strides are multiples of 16 bytes.
+  // `cols` of them exist); 64 rows of either are less than 2^31 elements apart. K is a multiple of 16; all starts and strides are multiples of 16 bytes.
   static __device__ __forceinline__ float* run(uint8_t* smem, const T* x, long long ldx, int rows, const T* const (&w)[NW],
                                                long long ldw, int cols, int K) {
     constexpr int V = kVec16<T>, kPieces = kStep / V;
     T* ring = reinterpret_cast<T*>(smem);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int steps = (K + kStep - 1) / kStep;
+    // a thread copies the same 16-byte column of every kPass-th row of the input and of the matrices
+    constexpr int kPass = kThreads / kPieces, kRowsX = BM / kPass > 0 ? BM / kPass : 1, kRowsW = BN / kPass;
+    const int pr = tid / kPieces, pk = (tid % kPieces) * V;
+    const int ldx32 = static_cast<int>(ldx), ldw32 = static_cast<int>(ldw);
     auto issue = [&](int s) {
-      T* st = ring + (s % kStages) * kStageElems;
-      const int k0 = s * kStep;
-      for (int i = tid; i < (BM + NW * BN) * kPieces; i += kThreads) {
-        const int r = i / kPieces, k = k0 + (i % kPieces) * V;
-        const T* src;
-        bool ok = k < K;
-        if (r < BM) {
-          ok = ok && r < rows;
-          src = x + (ok ? r * ldx + k : 0);
-        } else {
-          const int n = (r - BM) % BN;
-          ok = ok && n < cols;
-          src = w[(r - BM) / BN] + (ok ? n * ldw + k : 0);
-        }
-        cp_async_16(smem_u32(st + r * kLd + (i % kPieces) * V), src, ok ? 16 : 0);
+      T* st = ring + (s % kStages) * kStageElems + pr * kLd + pk;
+      const int k = s * kStep + pk;
+      const bool in_k = k < K;
+#pragma unroll
+      for (int i = 0; i < kRowsX; ++i) {
+        const int r = pr + i * kPass;
+        if (BM < kPass && r >= BM) break;
+        const bool ok = in_k && r < rows;
+        cp_async_16(smem_u32(st + i * kPass * kLd), ok ? x + r * ldx32 + k : x, ok ? 16 : 0);
       }
+#pragma unroll
+      for (int i = 0; i < NW; ++i)
+#pragma unroll
+        for (int j = 0; j < kRowsW; ++j) {
+          const int n = pr + j * kPass;
+          const bool ok = in_k && n < cols;
+          cp_async_16(smem_u32(st + (BM + i * BN + j * kPass) * kLd), ok ? w[i] + n * ldw32 + k : w[i], ok ? 16 : 0);
+        }
     };
     // bf16: a warp owns 16 rows x 64 columns (BM = 64) or 16 x 16 (BM = 16); fp32: 8 x 16 threads, rows and columns interleaved
     constexpr int kNT = BM == 64 ? 8 : 2;

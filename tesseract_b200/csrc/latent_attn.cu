@@ -158,19 +158,32 @@ head_linear_kernel(HeadLinearParams p) {
   const int rows = min(BM, p.rows - m0), cols = min(64, p.N - n0);
   const T* const w[1] = {static_cast<const T*>(p.w) + h * p.wh + static_cast<long long>(n0) * p.ldw};
   const float* acc = Tile::run(smem, static_cast<const T*>(p.x) + m0 * p.ldx + h * p.xh, p.ldx, rows, w, p.ldw, cols, p.K);
-  for (int i = threadIdx.x; i < rows * 32; i += 128) {
-    const int m = i >> 5, n = (i & 31) * 2;
-    if (n >= cols) continue;                       // (N is even)
-    const long long row = m0 + m;
-    float a = acc[m * Tile::kLdC + n], b = acc[m * Tile::kLdC + n + 1];
-    if (p.gate) {
-      const T* g = static_cast<const T*>(p.gate) + row * p.ldg + h * p.oh + n0 + n;
-      a *= sigmoid_f32(p.gate_scale * to_f32<T>(g[0]));
-      b *= sigmoid_f32(p.gate_scale * to_f32<T>(g[1]));
+  const int n = (threadIdx.x & 31) * 2;
+  if (n >= cols) return;                           // (N is even)
+  const T* gate = p.gate ? static_cast<const T*>(p.gate) + h * p.oh + n0 + n : nullptr;
+  T* out = static_cast<T*>(p.out) + h * p.oh + n0 + n;
+  struct alignas(2 * sizeof(T)) Two { T v[2]; };
+  constexpr int kPer = BM / 4 < 8 ? BM / 4 : 8;    // rows whose gates are requested together
+#pragma unroll
+  for (int r0 = threadIdx.x >> 5; r0 < BM; r0 += 4 * kPer) {
+    Two g[kPer];
+#pragma unroll
+    for (int i = 0; i < kPer; ++i)
+      if (gate) g[i] = *reinterpret_cast<const Two*>(gate + static_cast<long long>(m0 + min(r0 + 4 * i, rows - 1)) * p.ldg);
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      const int m = r0 + 4 * i;
+      if (m >= rows) break;
+      float2 a = *reinterpret_cast<const float2*>(acc + m * Tile::kLdC + n);
+      if (gate) {
+        const float x = p.gate_scale * to_f32<T>(g[i].v[0]), y = p.gate_scale * to_f32<T>(g[i].v[1]);
+        a.x *= sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-x)) : sigmoid_f32(x);
+        a.y *= sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-y)) : sigmoid_f32(y);
+      }
+      T* o = out + static_cast<long long>(m0 + m) * p.ldo;
+      if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(o) = pack_bf16x2(a.x, a.y);
+      else *reinterpret_cast<float2*>(o) = a;
     }
-    T* o = static_cast<T*>(p.out) + row * p.ldo + h * p.oh + n0 + n;
-    if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(o) = pack_bf16x2(a, b);
-    else *reinterpret_cast<float2*>(o) = make_float2(a, b);
   }
 }
 
@@ -214,78 +227,75 @@ constexpr int kBlockBytes = kKeys * 128;      // 64 keys x 64 columns, 128-byte 
 
 // One CTA per (key split, 32 heads, row); a tile of 64 pool rows is brought in once (TMA, one box per run of rows of a page and
 // 64 columns) and is the B operand of the scores and the A operand of the read-out:
-//   S[head, key]   = q[head, :] . row[key, :]       M = 128 (rows past the heads read whatever lies there and are ignored)
+//   S[head, key]   = q[head, :] . row[key, :]       A = q in tensor memory, the 32 heads once in every quarter of the lanes
 //   O[col, head]  += row[key, col] P[head, key]     M = 128 columns a time, N = heads: no row of the product is padding
-// Warp 0 turns scores into weights (lane = head) with the lazy reference maximum of flash_attn_fwd.cu: O is rescaled, by all of
-// warps 0 .. 3, only when a head's maximum has grown by more than 2^8. Warp 4 loads, warp 5 issues the products.
-struct LatentSmem {
-  static __host__ __device__ int blocks(int L) { return (L + 63) / 64; }
-  static __host__ __device__ int stages(int L) {
-    const int room = 227 * 1024 - 2048 - blocks(L) * kHeads * 128 - kHeads * 128;
-    const int n = room / (blocks(L) * kBlockBytes);
-    return n < 4 ? n : 4;
-  }
-  static __host__ __device__ int bytes(int L) {
-    return 1024 + blocks(L) * kHeads * 128 + kHeads * 128 + stages(L) * blocks(L) * kBlockBytes;
+// Warps 0 .. 3 turn scores into weights: lane = head, each warp reads its own quarter of the lanes and takes 16 of the keys. The
+// reference maximum is lazy as in flash_attn_fwd.cu: O is rescaled only when a head's maximum has grown by more than 2^8. Warp 4
+// loads, warp 5 issues the products.
+struct LatentPlan {
+  int blocks, stages, m_tiles, tmem_cols, smem;
+  __host__ __device__ LatentPlan(int cp, int L) {
+    blocks = (L + 63) / 64;
+    m_tiles = (cp + 127) / 128;
+    const int tile = blocks * kBlockBytes, room = 227 * 1024 - 4096 - kHeads * 128;
+    stages = room / tile < 4 ? room / tile : 4;
+    smem = 1024 + kHeads * 128 + stages * tile;
+    const int cols = m_tiles * kHeads + kKeys + blocks * 32;
+    tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;
+    if (cols > 512) stages = 0;
   }
 };
 
 __global__ void __launch_bounds__(192, 1)
-latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_pool, LatentAttnParams p) {
-  pdl_trigger();
+latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnParams p) {
   pdl_grid_wait();
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int L = p.cp + p.rp, NB = LatentSmem::blocks(L), stages = LatentSmem::stages(L);
-  uint8_t* sq = smem;                                  // [NB][32 heads][128 B]
-  uint8_t* sp = sq + NB * kHeads * 128;                // [32 heads][128 B]
+  const int L = p.cp + p.rp;
+  const LatentPlan plan(p.cp, L);
+  const int NB = plan.blocks, stages = plan.stages, m_tiles = plan.m_tiles;
+  uint8_t* sp = smem;                                  // [32 heads][128 B]
   uint8_t* sk = sp + kHeads * 128;                     // [stages][NB][64 keys][128 B]
-  __shared__ __align__(8) uint64_t q_full, k_full[4], k_empty[4], s_full[2], s_free[2], p_full, o_full;
+  __shared__ __align__(8) uint64_t q_full, k_full[4], k_empty[4], s_full, s_free, p_full, o_full;
   __shared__ uint32_t tmem_base_smem;
   __shared__ volatile int cta_abort;
-  __shared__ float corr[kHeads], inv[kHeads];
-  __shared__ volatile int grown;                       // 1: rescale, 0: not, -1: leave
+  __shared__ float smax[2][4][kHeads], lsum[4][kHeads], corr[kHeads];
   const int split = blockIdx.x, h0 = blockIdx.y * kHeads, row = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int len = p.lens ? p.lens[row] : p.pos[row] + 1;
   const int share = ((len + p.splits - 1) / p.splits + kKeys - 1) / kKeys * kKeys;
   const int t_begin = split * share, t_end = min(len, t_begin + share);
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + kKeys - 1) / kKeys : 0;
-  constexpr uint32_t kColO = 0, kColS = 128;
 
   if (threadIdx.x == 0) {
     cta_abort = 0;
-    mbar_init(&q_full, 1);
+    mbar_init(&q_full, 128);
     for (int i = 0; i < 4; ++i) {
       mbar_init(&k_full[i], 1);
       mbar_init(&k_empty[i], 1);
     }
-    for (int i = 0; i < 2; ++i) {
-      mbar_init(&s_full[i], 1);
-      mbar_init(&s_free[i], 32);
-    }
+    mbar_init(&s_full, 1);
+    mbar_init(&s_free, 128);
     mbar_init(&p_full, 128);
     mbar_init(&o_full, 1);
     mbar_fence_init();
-    tma_prefetch_desc(&tm_q);
     tma_prefetch_desc(&tm_pool);
   }
   if (warp == 5) {
-    tmem_alloc(&tmem_base_smem, 256);
+    tmem_alloc(&tmem_base_smem, plan.tmem_cols);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = tmem_base_smem;
-  const int m_tiles = (p.cp + 127) / 128;
+  // Only now may successors start: one that allocates tensor memory ahead of its own wait must not take it from a CTA of this
+  // grid, on whose end it depends.
+  pdl_trigger();
+  const uint32_t tmem = tmem_base_smem, tmem_s = tmem + m_tiles * kHeads, tmem_q = tmem_s + kKeys;
 
   if (warp == 4) {
     // ---------------------------------------------------------------- loads: a lane per run of rows inside a page
     if (n_tiles > 0) {
-      if (lane == 0) mbar_expect_tx(&q_full, NB * kHeads * 128);
-      __syncwarp();
-      for (int b = lane; b < NB; b += 32) tma_load_2d(sq + b * kHeads * 128, &tm_q, &q_full, b * 64, row * p.H + h0);
       const int* table = p.tables + static_cast<long long>(p.seq_of ? p.seq_of[row] : row) * p.table_ld;
       int run = 64;
       while (p.bs % run) run >>= 1;                    // rows that are neighbours in the pool: 64, 32, 16 or 8
@@ -319,24 +329,24 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     if (lane == 0 && n_tiles > 0) {
       constexpr uint32_t idesc_s = umma_idesc(128, kKeys, 1, 1, 0, 0);       // both K-major
       constexpr uint32_t idesc_o = umma_idesc(128, kHeads, 1, 1, 1, 0);      // pool rows: columns contiguous (M-major)
-      const uint32_t q_base = smem_u32(sq), p_base = smem_u32(sp);
+      const uint32_t p_base = smem_u32(sp);
       bool ok = mbar_wait(&q_full, 0, &cta_abort, p.status);
-      // scores of tile j and the read-out of tile j - 1, whichever can start first: with two stages the next tile's load waits
-      // for the read-out, so a read-out must not wait for a tile that is still on its way
+      // scores of tile j and the read-out of tile j - 1, whichever can start first: the load of a later tile waits for the
+      // read-out, so a read-out must not wait for a tile that is still on its way
       for (int j = 0; ok && j <= n_tiles; ++j) {
         bool score = j < n_tiles, read = j > 0;
         const long long since = clock64();
         while (score || read) {
-          const int st = j % stages, sb = j & 1;
-          if (score && mbar_test_wait(&k_full[st], (j / stages) & 1) && mbar_test_wait(&s_free[sb], ((j >> 1) & 1) ^ 1u)) {
+          const int st = j % stages;
+          if (score && mbar_test_wait(&k_full[st], (j / stages) & 1) && mbar_test_wait(&s_free, (j & 1) ^ 1u)) {
             tc_fence_after();
             const uint32_t k_base = smem_u32(sk + st * NB * kBlockBytes);
             for (int b = 0; b < NB; ++b)
 #pragma unroll
               for (int k = 0; k < 4; ++k)
-                umma_f16(tmem + kColS + sb * 64, umma_smem_desc_sw128(q_base + b * kHeads * 128 + k * 32, 16, 1024),
-                         umma_smem_desc_sw128(k_base + b * kBlockBytes + k * 32, 16, 1024), idesc_s, (b | k) != 0);
-            umma_commit(&s_full[sb]);
+                umma_f16_ts(tmem_s, tmem_q + b * 32 + k * 8, umma_smem_desc_sw128(k_base + b * kBlockBytes + k * 32, 16, 1024), idesc_s,
+                            (b | k) != 0);
+            umma_commit(&s_full);
             score = false;
           }
           if (read && mbar_test_wait(&p_full, (j - 1) & 1)) {
@@ -346,7 +356,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
             for (int m = 0; m < m_tiles; ++m)
 #pragma unroll
               for (int k = 0; k < kKeys / 16; ++k)
-                umma_f16(tmem + kColO + m * kHeads, umma_smem_desc_sw128(v_base + m * 2 * kBlockBytes + k * 2048, kBlockBytes, 1024),
+                umma_f16(tmem + m * kHeads, umma_smem_desc_sw128(v_base + m * 2 * kBlockBytes + k * 2048, kBlockBytes, 1024),
                          umma_smem_desc_sw128(p_base + k * 32, 16, 1024), idesc_o, ((j - 1) | k) != 0);
             umma_commit(&o_full);
             umma_commit(&k_empty[sv]);
@@ -363,91 +373,111 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       }
     }
   } else {
-    // ---------------------------------------------------------------- weights (warp 0), rescaling and output (warps 0 .. 3)
+    // ---------------------------------------------------------------- queries, weights, rescaling and output
     const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
     const float scale_log2 = p.scale * 1.4426950408889634f;
+    {
+      const bool there = h0 + lane < p.H;
+      const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) +
+                                                      (static_cast<long long>(row) * p.H + (there ? h0 + lane : 0)) * L);
+      for (int b = 0; b < NB; ++b) {
+        uint32_t r[32];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const uint4 v = there && (b * 8 + i) * 8 < L ? q[b * 8 + i] : make_uint4(0, 0, 0, 0);
+          r[4 * i] = v.x; r[4 * i + 1] = v.y; r[4 * i + 2] = v.z; r[4 * i + 3] = v.w;
+        }
+        tmem_st_32x32(tmem_q + lanes + b * 32, r);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      mbar_arrive(&q_full);
+    }
     float m_ref = -INFINITY, l = 0.f;
     bool good = true;
     for (int j = 0; j < n_tiles; ++j) {
-      const int sb = j & 1;
-      uint32_t s[64];
-      if (warp == 0) {
-        bool ok = mbar_wait(&s_full[sb], (j >> 1) & 1, &cta_abort, p.status);
-        ok = __all_sync(0xffffffffu, ok ? 1 : 0) != 0;
-        float factor = 1.f;
-        bool grow = false;
-        if (ok) {
-          tc_fence_after();
-          tmem_ld_32x32(tmem + kColS + sb * 64, *reinterpret_cast<uint32_t(*)[32]>(&s[0]));
-          tmem_ld_32x32(tmem + kColS + sb * 64 + 32, *reinterpret_cast<uint32_t(*)[32]>(&s[32]));
-          tmem_ld_wait();
-          tc_fence_before();
-          mbar_arrive(&s_free[sb]);
-          const int vis = min(kKeys, t_end - (t_begin + j * kKeys));
-          float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+      // (every warp passes each barrier below once per tile whether its waits succeed or not; a failure is told through smax)
+      bool ok = mbar_wait(&s_full, j & 1, &cta_abort, p.status);
+      ok = __all_sync(0xffffffffu, ok ? 1 : 0) != 0;
+      uint32_t s[16];
+      float m_own = -INFINITY;
+      const int vis = t_end - (t_begin + j * kKeys + warp * 16);
+      if (ok) {
+        tc_fence_after();
+        tmem_ld_32x16(tmem_s + lanes + warp * 16, s);
+        tmem_ld_wait();
+        tc_fence_before();
+        mbar_arrive(&s_free);
 #pragma unroll
-          for (int i = 0; i < kKeys; ++i)
-            if (i < vis) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(s[i]));
-          const float m_tile = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
-          if (j == 0) {
-            m_ref = m_tile;
-          } else if ((m_tile - m_ref) * scale_log2 > 8.f) {
-            factor = exp2f((m_ref - m_tile) * scale_log2);
-            m_ref = m_tile;
-            grow = true;
-          }
-          l *= factor;
-          const float mneg = -m_ref * scale_log2;
-          // weights as the tensor core will read them; the denominator sums those
-#pragma unroll
-          for (int i = 0; i < kKeys; i += 2) {
-            const float p0 = i < vis ? exp2f(fmaf(__uint_as_float(s[i]), scale_log2, mneg)) : 0.f;
-            const float p1 = i + 1 < vis ? exp2f(fmaf(__uint_as_float(s[i + 1]), scale_log2, mneg)) : 0.f;
-            const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
-            l += __low2float(pb) + __high2float(pb);
-            s[i >> 1] = *reinterpret_cast<const uint32_t*>(&pb);
-          }
-          // the read-out before must be finished: it reads the weights in shared memory, and rescaling rewrites its result
-          if (j > 0) ok = __all_sync(0xffffffffu, mbar_wait(&o_full, (j - 1) & 1, &cta_abort, p.status) ? 1 : 0) != 0;
-        }
-        corr[lane] = factor;
-        const bool any = __any_sync(0xffffffffu, grow);
-        if (lane == 0) grown = ok ? (any ? 1 : 0) : -1;
+        for (int i = 0; i < 16; ++i)
+          if (i < vis) m_own = fmaxf(m_own, __uint_as_float(s[i]));
       }
+      smax[j & 1][warp][lane] = ok ? m_own : INFINITY;
       asm volatile("bar.sync 1, 128;" ::: "memory");
-      const int what = grown;
-      if (what < 0) {
+      float m_tile = -INFINITY;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) m_tile = fmaxf(m_tile, smax[j & 1][w][lane]);
+      if (__any_sync(0xffffffffu, m_tile == INFINITY)) {      // the same answer in all four warps
         good = false;
         break;
       }
-      if (what > 0) {
-        tc_fence_after();
-        for (int m = 0; m < m_tiles; ++m) {
-          uint32_t r[32];
-          tmem_ld_32x32(tmem + lanes + kColO + m * kHeads, r);
-          tmem_ld_wait();
+      float factor = 1.f;
+      bool grow = false;
+      if (j == 0) {
+        m_ref = m_tile;
+      } else if ((m_tile - m_ref) * scale_log2 > 8.f) {
+        factor = exp2f((m_ref - m_tile) * scale_log2);
+        m_ref = m_tile;
+        grow = true;
+      }
+      l *= factor;
+      const float mneg = -m_ref * scale_log2;
+      uint32_t w8[8];
+      // weights as the tensor core will read them; the denominator sums those
 #pragma unroll
-          for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * corr[i]);
-          tmem_st_32x32(tmem + lanes + kColO + m * kHeads, r);
+      for (int i = 0; i < 16; i += 2) {
+        const float p0 = i < vis ? exp2f(fmaf(__uint_as_float(s[i]), scale_log2, mneg)) : 0.f;
+        const float p1 = i + 1 < vis ? exp2f(fmaf(__uint_as_float(s[i + 1]), scale_log2, mneg)) : 0.f;
+        const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
+        l += __low2float(pb) + __high2float(pb);
+        w8[i >> 1] = *reinterpret_cast<const uint32_t*>(&pb);
+      }
+      // the read-out before must be finished: it reads the weights in shared memory, and rescaling rewrites its result
+      if (j > 0) {
+        ok = mbar_wait(&o_full, (j - 1) & 1, &cta_abort, p.status);
+        ok = __all_sync(0xffffffffu, ok ? 1 : 0) != 0;
+        if (__any_sync(0xffffffffu, grow)) {           // (the same in all four warps)
+          tc_fence_after();
+          if (warp == 0) corr[lane] = factor;
+          asm volatile("bar.sync 2, 128;" ::: "memory");
+          for (int m = 0; ok && m < m_tiles; ++m) {
+            uint32_t r[32];
+            tmem_ld_32x32(tmem + lanes + m * kHeads, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * corr[i]);
+            tmem_st_32x32(tmem + lanes + m * kHeads, r);
+          }
+          tmem_st_wait();
         }
-        tmem_st_wait();
       }
-      if (warp == 0) {
-        uint8_t* prow = sp + lane * 128;
+      uint8_t* prow = sp + lane * 128;
 #pragma unroll
-        for (int c = 0; c < 8; ++c)
-          *reinterpret_cast<uint4*>(prow + (c ^ (lane & 7)) * 16) = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
-        fence_proxy_async_smem();
-      }
+      for (int c = 0; c < 2; ++c)
+        *reinterpret_cast<uint4*>(prow + ((2 * warp + c) ^ (lane & 7)) * 16) = make_uint4(w8[4 * c], w8[4 * c + 1], w8[4 * c + 2], w8[4 * c + 3]);
+      fence_proxy_async_smem();
       tc_fence_before();
-      mbar_arrive(&p_full);
+      if (ok) mbar_arrive(&p_full);
     }
+    lsum[warp][lane] = l;
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    const float sum = lsum[0][lane] + lsum[1][lane] + lsum[2][lane] + lsum[3][lane];
     if (warp == 0) {
-      inv[lane] = p.splits > 1 ? 1.f : l > 0.f ? 1.f / l : 0.f;
+      corr[lane] = p.splits > 1 ? 1.f : sum > 0.f ? 1.f / sum : 0.f;
       if (p.splits > 1 && h0 + lane < p.H) {
         float* ml = p.part_ml + ((static_cast<long long>(row) * p.H + h0 + lane) * p.splits + split) * 2;
         ml[0] = n_tiles > 0 ? m_ref * scale_log2 : -INFINITY;
-        ml[1] = l;
+        ml[1] = sum;
       }
     }
     asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -458,29 +488,29 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     for (int m = 0; m < m_tiles; ++m) {
       uint32_t r[32];
       if (have) {
-        tmem_ld_32x32(tmem + lanes + kColO + m * kHeads, r);
+        tmem_ld_32x32(tmem + lanes + m * kHeads, r);
         tmem_ld_wait();
       } else {
 #pragma unroll
         for (int i = 0; i < 32; ++i) r[i] = 0u;
       }
       const int c = m * 128 + warp * 32 + lane;
-      if (c >= p.cp) continue;
       const long long at = static_cast<long long>(row) * p.H + h0;
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
-        if (h0 + i >= p.H) break;
+        if (h0 + i >= p.H || c >= p.cp) break;
         const float v = __uint_as_float(r[i]);
-        if (p.splits == 1) static_cast<__nv_bfloat16*>(p.out)[(at + i) * p.cp + c] = __float2bfloat16_rn(v * inv[i]);
+        if (p.splits == 1) static_cast<__nv_bfloat16*>(p.out)[(at + i) * p.cp + c] = __float2bfloat16_rn(v * corr[i]);
         else p.part_o[((at + i) * p.splits + split) * p.cp + c] = v;
       }
+      __syncwarp();
     }
     tc_fence_before();
   }
   __syncthreads();
   if (warp == 5) {
     tc_fence_after();
-    tmem_dealloc(tmem, 256);
+    tmem_dealloc(tmem, plan.tmem_cols);
   }
 }
 
@@ -574,21 +604,20 @@ latent_rows_kernel(LatentAttnParams p) {
 
 int launch_latent_decode(const LatentAttnParams& p, cudaStream_t s) {
   const int L = p.cp + p.rp;
-  if (LatentSmem::stages(L) < 2) return -2;
+  const LatentPlan plan(p.cp, L);
+  if (plan.stages < 2) return -2;
   static PerDeviceFlag attr;
   if (attr.unset()) {
-    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 1024);
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 3072);
     if (e != cudaSuccess) return static_cast<int>(e);
     attr.set();
   }
   int run = 64;
   while (p.bs % run) run >>= 1;
-  CUtensorMap tm_q, tm_pool;
-  if (!make_tmap_2d(&tm_q, p.q, 2, static_cast<uint64_t>(p.rows) * p.H, L, L * 2ull, kHeads, 64, true) ||
-      !make_tmap_2d(&tm_pool, p.pool, 2, static_cast<uint64_t>(p.nb) * p.bs, L, L * 2ull, run, 64, true))
-    return -3;
-  launch_pdl(latent_decode_kernel, dim3(p.splits, (p.H + kHeads - 1) / kHeads, p.rows), dim3(192), LatentSmem::bytes(L), s,
-             pdl_all_enabled(), tm_q, tm_pool, p);
+  CUtensorMap tm_pool;
+  if (!make_tmap_2d(&tm_pool, p.pool, 2, static_cast<uint64_t>(p.nb) * p.bs, L, L * 2ull, run, 64, true)) return -3;
+  launch_pdl(latent_decode_kernel, dim3(p.splits, (p.H + kHeads - 1) / kHeads, p.rows), dim3(192), plan.smem, s, pdl_all_enabled(), tm_pool,
+             p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -664,7 +693,7 @@ TSB_EXPORT int tsb_latent_gather(const void* pool, void* stage, const int* dst_r
 TSB_EXPORT int tsb_head_linear(const void* x, long long ldx, int xh, const void* w, long long wh, int ldw, void* out, long long ldo, int oh,
                                const void* gate, long long ldg, float gate_scale, int rows, int H, int N, int K, int dtype, void* stream) {
   using namespace tsb;
-  if (rows <= 0 || H <= 0 || H > 65535 || N <= 0 || N % 2 || K <= 0 || K % 16 || ldx % 8 || xh % 8 || wh % 8 || ldw % 8 || ldw < K || ldo % 2 || oh % 2) return -2;
+  if (rows <= 0 || H <= 0 || H > 65535 || N <= 0 || N % 2 || K <= 0 || K % 16 || ldx % 8 || xh % 8 || wh % 8 || ldw % 8 || ldw < K || ldo % 2 || oh % 2 || (gate && ldg % 2)) return -2;
   HeadLinearParams p{x, ldx, xh, w, wh, ldw, out, ldo, oh, gate, ldg, gate_scale, rows, N, K};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const bool few = rows <= 64 || static_cast<long long>((rows + 63) / 64) * H * ((N + 63) / 64) < 4ll * sm_count();

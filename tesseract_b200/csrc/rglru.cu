@@ -129,6 +129,41 @@ rglru_conv_kernel(RglruParams p) {
 #pragma unroll
       for (int i = 0; i < V; ++i) w[j][i] = p.conv_w[static_cast<long long>(j) * p.C + c + i];
   }
+  if constexpr (TAPS > 0) {
+    // eight rows in the middle of a portion: every input is requested before the first is used
+    if (row >= p.n_dec && last - row == kConvRows - 1) {
+      const int seq = p.seq_of[row];
+      if (p.seq_of[last] == seq && row - tail >= p.n_dec + p.cu[seq - p.n_dec]) {
+        const T* x = static_cast<const T*>(p.proj) + (row - tail) * p.ldp + c;
+        uint4 raw[kConvRows + TAPS - 1];
+#pragma unroll
+        for (int r = 0; r < kConvRows + TAPS - 1; ++r) raw[r] = *reinterpret_cast<const uint4*>(x + r * p.ldp);
+        // the scale goes into the taps, the biases that they multiply into one
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+          float sum = 0.f;
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) {
+            sum += w[j][i];
+            w[j][i] *= p.in_scale;
+          }
+          cb[i] = fmaf(sum, bias[i], cb[i]);
+        }
+#pragma unroll
+        for (int r = 0; r < kConvRows; ++r) {
+          float acc[V];
+#pragma unroll
+          for (int i = 0; i < V; ++i) {
+            acc[i] = cb[i];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) acc[i] = fmaf(w[j][i], to_f32<T>(reinterpret_cast<const T*>(&raw[r + j])[i]), acc[i]);
+          }
+          st16<T>(static_cast<T*>(p.u) + static_cast<long long>(row + r) * p.C + c, acc);
+        }
+        return;
+      }
+    }
+  }
   float win[W][V];
   for (int first_row = row; row <= last; ++row) {
     const T* x = static_cast<const T*>(p.proj) + row * p.ldp + c;
@@ -207,23 +242,35 @@ rglru_step_kernel(RglruParams p) {
   const long long w0 = (static_cast<long long>(blk) * p.kp + n0) * p.kp;
   const T* const w[2] = {static_cast<const T*>(p.ra) + w0, static_cast<const T*>(p.ri) + w0};
   const float* acc = Tile::run(smem, u, p.C, rows, w, p.kp, cols, p.kp);
-  for (int i = threadIdx.x; i < rows * 64; i += 128) {
-    const int m = i >> 6, n = i & 63;
-    if (n >= cols) continue;
-    const int row = m0 + m, c = blk * p.kp + n0 + n;
-    const int slot = p.slots[row];
-    T* out = static_cast<T*>(p.out) + row * p.ldo + c;
-    if (slot < 0) {
-      *out = from_f32<T>(0.f);
-      continue;
+  const int n = threadIdx.x & 63, c = blk * p.kp + n0 + n;
+  if (n >= cols) return;
+  const float rb = p.ra_b[c], ib = p.ri_b[c], dc = p.decay[c], yb = p.y_bias[c];
+  constexpr int kPer = 8;                          // rows whose inputs are requested together
+#pragma unroll
+  for (int r0 = threadIdx.x >> 6; r0 < BM; r0 += 2 * kPer) {
+    int slot[kPer];
+    float uu[kPer], y[kPer], s[kPer];
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      const int m = min(r0 + 2 * i, rows - 1), row = m0 + m;
+      slot[i] = p.slots[row];
+      uu[i] = to_f32<T>(u[static_cast<long long>(m) * p.C + n0 + n]);
+      y[i] = to_f32<T>(static_cast<const T*>(p.proj)[row * p.ldp + p.off_y + c]);
+      s[i] = slot[i] >= 0 && p.positions[row] > 0 ? p.state[static_cast<long long>(slot[i]) * p.C + c] : 0.f;
     }
-    const Gates g = rglru_gates<sizeof(T) == 2>(acc[m * Tile::kLdC + n] + p.ra_b[c], acc[(BM + m) * Tile::kLdC + n] + p.ri_b[c], p.decay[c],
-                                to_f32<T>(u[static_cast<long long>(m) * p.C + n0 + n]));
-    float* st = p.state + static_cast<long long>(slot) * p.C + c;
-    const float s = fmaf(g.a, p.positions[row] > 0 ? *st : 0.f, g.b);
-    *st = s;
-    const float y = fmaf(to_f32<T>(static_cast<const T*>(p.proj)[row * p.ldp + p.off_y + c]), p.in_scale, p.y_bias[c]);
-    *out = from_f32<T>(s * gelu_tanh_g<sizeof(T) == 2>(y));
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      const int m = r0 + 2 * i;
+      if (m >= rows) break;
+      const Gates g = rglru_gates<sizeof(T) == 2>(acc[m * Tile::kLdC + n] + rb, acc[(BM + m) * Tile::kLdC + n] + ib, dc, uu[i]);
+      const float next = fmaf(g.a, s[i], g.b);
+      float z = 0.f;                               // (a row without a sequence)
+      if (slot[i] >= 0) {
+        p.state[static_cast<long long>(slot[i]) * p.C + c] = next;
+        z = next * gelu_tanh_g<sizeof(T) == 2>(fmaf(y[i], p.in_scale, yb));
+      }
+      static_cast<T*>(p.out)[static_cast<long long>(m0 + m) * p.ldo + c] = from_f32<T>(z);
+    }
   }
 }
 
@@ -249,13 +296,20 @@ rglru_chunk_kernel(RglruParams p) {
   const bool ok = n < cols;
   {
     const float rb = ok ? p.ra_b[c] : 0.f, ib = ok ? p.ri_b[c] : 0.f, dc = ok ? p.decay[c] : 0.f;
-#pragma unroll 4
-    for (int m = tid >> 6; m < rows; m += 2) {
-      const float uu = ok ? to_f32<T>(u[static_cast<long long>(m) * p.C + n0 + n]) : 0.f;
-      const int at = m * Tile::kLdC + n;
-      const Gates g = rglru_gates<sizeof(T) == 2>(sa[at] + rb, sb[at] + ib, dc, uu);
-      sa[at] = g.a;
-      sb[at] = g.b;
+    const T* uc = u + n0 + (ok ? n : 0);
+    constexpr int kPer = 8;                        // tokens whose inputs are requested together
+#pragma unroll 1
+    for (int r0 = tid >> 6; r0 < rows; r0 += 2 * kPer) {
+      float uu[kPer];
+#pragma unroll
+      for (int i = 0; i < kPer; ++i) uu[i] = to_f32<T>(uc[static_cast<long long>(min(r0 + 2 * i, rows - 1)) * p.C]);
+#pragma unroll
+      for (int i = 0; i < kPer; ++i) {             // (rows past the end compute on zeros and are not used)
+        const int at = (r0 + 2 * i) * Tile::kLdC + n;
+        const Gates g = rglru_gates<sizeof(T) == 2>(sa[at] + rb, sb[at] + ib, dc, uu[i]);
+        sa[at] = g.a;
+        sb[at] = g.b;
+      }
     }
   }
   __syncthreads();

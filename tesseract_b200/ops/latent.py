@@ -106,8 +106,8 @@ class LatentGeometry:
         return dtype == torch.bfloat16 and self.D <= 128
 
     def tensor_cores(self, dtype, block: int) -> bool:
-        """Whether single rows run on ``latent_decode_kernel`` (two tiles of keys and the queries fit in shared memory)."""
-        return dtype == torch.bfloat16 and self.cp <= 512 and self.row <= 704 and block % 8 == 0
+        """Whether single rows run on ``latent_decode_kernel`` (its sums, scores and queries fit in tensor memory)."""
+        return dtype == torch.bfloat16 and self.cp <= 512 and self.row <= 640 and block % 8 == 0
 
 
 @dataclass
