@@ -52,15 +52,15 @@ struct HeadTile {
           cp_async_16(smem_u32(st + (BM + i * BN + j * kPass) * kLd), ok ? w[i] + n * ldw32 + k : w[i], ok ? 16 : 0);
         }
     };
-    // bf16: a warp owns 16 rows x 64 columns (BM = 64) or 16 x 16 (BM = 16); fp32: 8 x 16 threads, rows and columns interleaved
-    constexpr int kNT = BM == 64 ? 8 : 2;
+    // bf16: a warp owns 32 rows x 32 columns (BM = 64) or 16 x 16 (BM = 16); fp32: 8 x 16 threads, rows and columns interleaved
+    constexpr int kMB = BM == 64 ? 2 : 1, kNB = BM == 64 ? 4 : 2, kNT = kMB * kNB;      // blocks of 16 rows, of 8 columns
     constexpr int kRowsT = BM / 8;
     float acc[NW][sizeof(T) == 2 ? kNT : kRowsT][4];
 #pragma unroll
     for (int i = 0; i < NW; ++i)
 #pragma unroll
       for (int j = 0; j < (sizeof(T) == 2 ? kNT : kRowsT); ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
-    const int row0 = BM == 64 ? warp * 16 : 0, col0 = BM == 64 ? 0 : warp * 16;
+    const int row0 = BM == 64 ? (warp & 1) * 32 : 0, col0 = BM == 64 ? (warp >> 1) * 32 : warp * 16;
     const int tm = tid >> 4, tn = tid & 15;
 #pragma unroll
     for (int s = 0; s < kStages - 1; ++s) {
@@ -85,17 +85,21 @@ struct HeadTile {
         const uint32_t ax = smem_u32(sx);
 #pragma unroll
         for (int kk = 0; kk < kStep / 16; ++kk) {
-          uint32_t a[4];
-          ldmat_x4(a, ax + frag_a(lane, row0, kk * 16, kLd));
+          uint32_t a[kMB][4];
+#pragma unroll
+          for (int m = 0; m < kMB; ++m) ldmat_x4(a[m], ax + frag_a(lane, row0 + m * 16, kk * 16, kLd));
 #pragma unroll
           for (int i = 0; i < NW; ++i) {
             const uint32_t bx = smem_u32(sx + (BM + i * BN) * kLd);
 #pragma unroll
-            for (int j = 0; j < kNT; j += 2) {
+            for (int j = 0; j < kNB; j += 2) {
               uint32_t b[4];
               ldmat_x4(b, bx + frag_b(lane, col0 + j * 8, kk * 16, kLd));
-              mma_bf16(acc[i][j], a, b[0], b[1]);
-              mma_bf16(acc[i][j + 1], a, b[2], b[3]);
+#pragma unroll
+              for (int m = 0; m < kMB; ++m) {
+                mma_bf16(acc[i][m * kNB + j], a[m], b[0], b[1]);
+                mma_bf16(acc[i][m * kNB + j + 1], a[m], b[2], b[3]);
+              }
             }
           }
         }
@@ -126,7 +130,7 @@ struct HeadTile {
         const int g = lane >> 2, t = lane & 3;
 #pragma unroll
         for (int j = 0; j < kNT; ++j) {
-          float* c = o + (row0 + g) * kLdC + col0 + j * 8 + 2 * t;
+          float* c = o + (row0 + j / kNB * 16 + g) * kLdC + col0 + j % kNB * 8 + 2 * t;
           *reinterpret_cast<float2*>(c) = make_float2(acc[i][j][0], acc[i][j][1]);
           *reinterpret_cast<float2*>(c + 8 * kLdC) = make_float2(acc[i][j][2], acc[i][j][3]);
         }

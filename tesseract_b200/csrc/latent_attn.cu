@@ -247,7 +247,7 @@ struct LatentPlan {
 };
 
 __global__ void __launch_bounds__(192, 1)
-latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnParams p) {
+latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_pool, LatentAttnParams p) {
   pdl_grid_wait();
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -256,7 +256,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnPara
   const int NB = plan.blocks, stages = plan.stages, m_tiles = plan.m_tiles;
   uint8_t* sp = smem;                                  // [32 heads][128 B]
   uint8_t* sk = sp + kHeads * 128;                     // [stages][NB][64 keys][128 B]
-  __shared__ __align__(8) uint64_t q_full, k_full[4], k_empty[4], s_full, s_free, p_full, o_full;
+  __shared__ __align__(8) uint64_t q_in, q_full, k_full[4], k_empty[4], s_full, s_free, p_full, o_full;
   __shared__ uint32_t tmem_base_smem;
   __shared__ volatile int cta_abort;
   __shared__ float smax[2][4][kHeads], lsum[4][kHeads], corr[kHeads];
@@ -269,6 +269,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnPara
 
   if (threadIdx.x == 0) {
     cta_abort = 0;
+    mbar_init(&q_in, 1);
     mbar_init(&q_full, 128);
     for (int i = 0; i < 4; ++i) {
       mbar_init(&k_full[i], 1);
@@ -279,6 +280,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnPara
     mbar_init(&p_full, 128);
     mbar_init(&o_full, 1);
     mbar_fence_init();
+    tma_prefetch_desc(&tm_q);
     tma_prefetch_desc(&tm_pool);
   }
   if (warp == 5) {
@@ -296,6 +298,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnPara
   if (warp == 4) {
     // ---------------------------------------------------------------- loads: a lane per run of rows inside a page
     if (n_tiles > 0) {
+      // the queries land in the last stage on their way to tensor memory
+      if (lane == 0) mbar_expect_tx(&q_in, NB * kHeads * 128);
+      __syncwarp();
+      if (lane < NB) tma_load_2d(sk + (stages - 1) * NB * kBlockBytes + lane * kHeads * 128, &tm_q, &q_in, lane * 64, row * p.H + h0);
       const int* table = p.tables + static_cast<long long>(p.seq_of ? p.seq_of[row] : row) * p.table_ld;
       int run = 64;
       while (p.bs % run) run >>= 1;                    // rows that are neighbours in the pool: 64, 32, 16 or 8
@@ -314,7 +320,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnPara
       for (int j = 0; j < n_tiles; ++j) {
         const int st = j % stages, y = next;
         if (j + 1 < n_tiles) next = pool_row(j + 1);
-        const bool ok = mbar_wait(&k_empty[st], ((j / stages) & 1) ^ 1u, &cta_abort, p.status);
+        bool ok = mbar_wait(&k_empty[st], ((j / stages) & 1) ^ 1u, &cta_abort, p.status);
+        if (j == stages - 1) ok = ok && mbar_wait(&q_full, 0, &cta_abort, p.status);
         if (!__all_sync(0xffffffffu, ok ? 1 : 0)) break;
         if (lane == 0) mbar_expect_tx(&k_full[st], NB * kBlockBytes);
         __syncwarp();
@@ -326,40 +333,56 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnPara
     }
   } else if (warp == 5) {
     // ---------------------------------------------------------------- products
-    if (lane == 0 && n_tiles > 0) {
+    // The products are small (16 - 32 cycles each), so what surrounds them counts: the whole warp walks the loop and works out the
+    // descriptors, which keeps them uniform, and lane 0 alone is predicated on for the instruction itself.
+    if (n_tiles > 0) {
       constexpr uint32_t idesc_s = umma_idesc(128, kKeys, 1, 1, 0, 0);       // both K-major
       constexpr uint32_t idesc_o = umma_idesc(128, kHeads, 1, 1, 1, 0);      // pool rows: columns contiguous (M-major)
-      const uint32_t p_base = smem_u32(sp);
-      bool ok = mbar_wait(&q_full, 0, &cta_abort, p.status);
+      const uint32_t leader = lane == 0;
+      const uint64_t k_desc = umma_smem_desc_sw128(smem_u32(sk), 16, 1024), v_desc = umma_smem_desc_sw128(smem_u32(sk), kBlockBytes, 1024),
+                     p_desc = umma_smem_desc_sw128(smem_u32(sp), 16, 1024);
+      const uint32_t tile16 = NB * kBlockBytes / 16;                         // descriptors count 16-byte units
+      bool ok = __all_sync(0xffffffffu, mbar_wait(&q_full, 0, &cta_abort, p.status) ? 1 : 0) != 0;
       // scores of tile j and the read-out of tile j - 1, whichever can start first: the load of a later tile waits for the
       // read-out, so a read-out must not wait for a tile that is still on its way
+      uint32_t st = 0, sv = 0;                                               // stages of tiles j and j - 1
       for (int j = 0; ok && j <= n_tiles; ++j) {
         bool score = j < n_tiles, read = j > 0;
         const long long since = clock64();
         while (score || read) {
-          const int st = j % stages;
-          if (score && mbar_test_wait(&k_full[st], (j / stages) & 1) && mbar_test_wait(&s_free, (j & 1) ^ 1u)) {
+          if (score && __all_sync(0xffffffffu, mbar_test_wait(&k_full[st], (j / stages) & 1) && mbar_test_wait(&s_free, (j & 1) ^ 1u))) {
             tc_fence_after();
-            const uint32_t k_base = smem_u32(sk + st * NB * kBlockBytes);
-            for (int b = 0; b < NB; ++b)
-#pragma unroll
-              for (int k = 0; k < 4; ++k)
-                umma_f16_ts(tmem_s, tmem_q + b * 32 + k * 8, umma_smem_desc_sw128(k_base + b * kBlockBytes + k * 32, 16, 1024), idesc_s,
-                            (b | k) != 0);
-            umma_commit(&s_full);
+            uint64_t d = k_desc + st * tile16;
+            uint32_t a = tmem_q;
+            umma_f16_ts_if(leader, tmem_s, a, d, idesc_s, 0);
+            umma_f16_ts_if(leader, tmem_s, a + 8, d + 2, idesc_s, 1);
+            umma_f16_ts_if(leader, tmem_s, a + 16, d + 4, idesc_s, 1);
+            umma_f16_ts_if(leader, tmem_s, a + 24, d + 6, idesc_s, 1);
+            for (int b = 1; b < NB; ++b) {
+              a += 32;
+              d += kBlockBytes / 16;
+              umma_f16_ts_if(leader, tmem_s, a, d, idesc_s, 1);
+              umma_f16_ts_if(leader, tmem_s, a + 8, d + 2, idesc_s, 1);
+              umma_f16_ts_if(leader, tmem_s, a + 16, d + 4, idesc_s, 1);
+              umma_f16_ts_if(leader, tmem_s, a + 24, d + 6, idesc_s, 1);
+            }
+            if (leader) umma_commit(&s_full);
             score = false;
           }
-          if (read && mbar_test_wait(&p_full, (j - 1) & 1)) {
-            const int sv = (j - 1) % stages;
+          if (read && __all_sync(0xffffffffu, mbar_test_wait(&p_full, (j - 1) & 1))) {
             tc_fence_after();
-            const uint32_t v_base = smem_u32(sk + sv * NB * kBlockBytes);
-            for (int m = 0; m < m_tiles; ++m)
-#pragma unroll
-              for (int k = 0; k < kKeys / 16; ++k)
-                umma_f16(tmem + m * kHeads, umma_smem_desc_sw128(v_base + m * 2 * kBlockBytes + k * 2048, kBlockBytes, 1024),
-                         umma_smem_desc_sw128(p_base + k * 32, 16, 1024), idesc_o, ((j - 1) | k) != 0);
-            umma_commit(&o_full);
-            umma_commit(&k_empty[sv]);
+            uint64_t d = v_desc + sv * tile16;
+            for (int m = 0; m < m_tiles; ++m) {
+              umma_f16_if(leader, tmem + m * kHeads, d, p_desc, idesc_o, j > 1);
+              umma_f16_if(leader, tmem + m * kHeads, d + 128, p_desc + 2, idesc_o, 1);
+              umma_f16_if(leader, tmem + m * kHeads, d + 256, p_desc + 4, idesc_o, 1);
+              umma_f16_if(leader, tmem + m * kHeads, d + 384, p_desc + 6, idesc_o, 1);
+              d += 2 * kBlockBytes / 16;
+            }
+            if (leader) {
+              umma_commit(&o_full);
+              umma_commit(&k_empty[sv]);
+            }
             read = false;
           }
           if (cta_abort) ok = false;
@@ -368,30 +391,35 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_pool, LatentAttnPara
             if (p.status) atomicCAS(p.status, kStatusOk, kStatusMbarTimeout);
             ok = false;
           }
+          ok = __all_sync(0xffffffffu, ok ? 1 : 0) != 0;
           if (!ok) break;
         }
+        sv = st;
+        st = st + 1 == static_cast<uint32_t>(stages) ? 0 : st + 1;
       }
     }
   } else {
     // ---------------------------------------------------------------- queries, weights, rescaling and output
     const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
     const float scale_log2 = p.scale * 1.4426950408889634f;
-    {
-      const bool there = h0 + lane < p.H;
-      const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) +
-                                                      (static_cast<long long>(row) * p.H + (there ? h0 + lane : 0)) * L);
-      for (int b = 0; b < NB; ++b) {
-        uint32_t r[32];
+    if (n_tiles > 0) {
+      const bool ok = mbar_wait(&q_in, 0, &cta_abort, p.status);
+      if (__all_sync(0xffffffffu, ok ? 1 : 0)) {
+        const uint8_t* sq = sk + (stages - 1) * NB * kBlockBytes + lane * 128;
+        for (int b = 0; b < NB; ++b) {
+          uint32_t r[32];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const uint4 v = there && (b * 8 + i) * 8 < L ? q[b * 8 + i] : make_uint4(0, 0, 0, 0);
-          r[4 * i] = v.x; r[4 * i + 1] = v.y; r[4 * i + 2] = v.z; r[4 * i + 3] = v.w;
+          for (int i = 0; i < 8; ++i) {
+            const uint4 v = *reinterpret_cast<const uint4*>(sq + b * kHeads * 128 + (i ^ (lane & 7)) * 16);
+            r[4 * i] = v.x; r[4 * i + 1] = v.y; r[4 * i + 2] = v.z; r[4 * i + 3] = v.w;
+          }
+          tmem_st_32x32(tmem_q + lanes + b * 32, r);
         }
-        tmem_st_32x32(tmem_q + lanes + b * 32, r);
+        tmem_st_wait();
+        tc_fence_before();
+        fence_proxy_async_smem();                      // (the last stage's next writer is the asynchronous proxy)
+        mbar_arrive(&q_full);
       }
-      tmem_st_wait();
-      tc_fence_before();
-      mbar_arrive(&q_full);
     }
     float m_ref = -INFINITY, l = 0.f;
     bool good = true;
@@ -614,10 +642,11 @@ int launch_latent_decode(const LatentAttnParams& p, cudaStream_t s) {
   }
   int run = 64;
   while (p.bs % run) run >>= 1;
-  CUtensorMap tm_pool;
-  if (!make_tmap_2d(&tm_pool, p.pool, 2, static_cast<uint64_t>(p.nb) * p.bs, L, L * 2ull, run, 64, true)) return -3;
-  launch_pdl(latent_decode_kernel, dim3(p.splits, (p.H + kHeads - 1) / kHeads, p.rows), dim3(192), plan.smem, s, pdl_all_enabled(), tm_pool,
-             p);
+  CUtensorMap tm_q, tm_pool;
+  if (!make_tmap_2d(&tm_q, p.q, 2, static_cast<uint64_t>(p.rows) * p.H, L, L * 2ull, kHeads, 64, true) ||
+      !make_tmap_2d(&tm_pool, p.pool, 2, static_cast<uint64_t>(p.nb) * p.bs, L, L * 2ull, run, 64, true)) return -3;
+  launch_pdl(latent_decode_kernel, dim3(p.splits, (p.H + kHeads - 1) / kHeads, p.rows), dim3(192), plan.smem, s, pdl_all_enabled(), tm_q,
+             tm_pool, p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -696,7 +725,7 @@ TSB_EXPORT int tsb_head_linear(const void* x, long long ldx, int xh, const void*
   if (rows <= 0 || H <= 0 || H > 65535 || N <= 0 || N % 2 || K <= 0 || K % 16 || ldx % 8 || xh % 8 || wh % 8 || ldw % 8 || ldw < K || ldo % 2 || oh % 2 || (gate && ldg % 2)) return -2;
   HeadLinearParams p{x, ldx, xh, w, wh, ldw, out, ldo, oh, gate, ldg, gate_scale, rows, N, K};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const bool few = rows <= 64 || static_cast<long long>((rows + 63) / 64) * H * ((N + 63) / 64) < 4ll * sm_count();
+  const bool few = rows <= 64;
   if (!few && (rows + 63) / 64 > 65535) return -2;
   if (dtype == 1) return few ? launch_head_linear<__nv_bfloat16, 16>(p, H, s) : launch_head_linear<__nv_bfloat16, 64>(p, H, s);
   if (dtype == 0) return few ? launch_head_linear<float, 16>(p, H, s) : launch_head_linear<float, 64>(p, H, s);
