@@ -60,15 +60,17 @@ struct SpanCfg {
   static constexpr int kK = 0, kQ = kK + kTok * kLdQ, kV = kQ + (OUT ? kTok * kLdQ : 0), kChunkElems = kV + kTok * kLdV;
   static constexpr int kSh = kBuf * kChunkElems, kSl = kSh + (OUT ? DT * kLdV : 0), kElems = kSl + (OUT ? DT * kLdV : 0);
   static constexpr int kTable = kElems * 2, kRow = kTable + kTok * DT / 2 * 8;
-  static constexpr int kSmem = kRow + 2 * kTok * 4;
-  // fragments of S: warp w holds kMT blocks of 16 rows x kNT blocks of 8 columns
-  static constexpr int kMT = DT >= 128 ? DT / 128 : 1;
-  static constexpr int kNT = DT >= 128 ? ET / 8 : ET / 16;
-  static constexpr int kOT = ET / 16;      // read-out: 4 groups of 16 tokens x 2 halves of the columns
+  static constexpr int kSmem = kRow + 4 * kTok * 4;
+  static constexpr int kWarps = DT > 128 ? 16 : 8, kThreads = kWarps * 32;
+  // fragments of S: a warp holds kMT blocks of 16 rows x kNT blocks of 8 columns; kSplit warps share a block of rows
+  static constexpr int kBlocks = DT / 16, kMT = kBlocks >= kWarps ? kBlocks / kWarps : 1, kSplit = kBlocks >= kWarps ? 1 : kWarps / kBlocks;
+  static constexpr int kNT = ET / kSplit / 8;
+  // read-out: 4 groups of 16 tokens x kCols groups of columns, kOT blocks of 8 each
+  static constexpr int kCols = kWarps / 4, kOT = ET / kCols / 8;
 };
 
 template <int DT, int ET, bool OUT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(SpanCfg<DT, ET, OUT>::kThreads)
 retention_span_kernel(RetParams p) {
   using T = __nv_bfloat16;
   using C = SpanCfg<DT, ET, OUT>;
@@ -77,7 +79,7 @@ retention_span_kernel(RetParams p) {
   extern __shared__ __align__(16) uint8_t smem[];
   T* sm = reinterpret_cast<T*>(smem);
   float2* stab = reinterpret_cast<float2*>(smem + C::kTable);      // [kTok][hp] cos, sin
-  float* srow = reinterpret_cast<float*>(smem + C::kRow);          // [2][kTok]
+  float* srow = reinterpret_cast<float*>(smem + C::kRow);          // [kCols][kTok]
   const int span = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * ET;
   const int seq = p.tile_seq[span], idx = span - p.tile0[seq], n_spans = p.tile0[seq + 1] - p.tile0[seq];
   const int slot = p.slots[seq];
@@ -97,25 +99,25 @@ retention_span_kernel(RetParams p) {
     const int cnt = min(kTok, n - t0);
     const T* src = proj + static_cast<long long>(t0) * p.ldp;
     constexpr int kPQ = DT / 8, kPV = ET / 8;
-    for (int i = tid; i < kTok * kPQ; i += 256) {
+    for (int i = tid; i < kTok * kPQ; i += C::kThreads) {
       const int r = i / kPQ, d = (i % kPQ) * 8;
       const bool ok = r < cnt && d < p.dp;
       const T* q = ok ? src + r * p.ldp + h * p.dp + d : proj;
       cp_async_16(smem_u32(buf + C::kK + r * C::kLdQ + d), ok ? q + p.off_k : q, ok ? 16 : 0);
       if constexpr (OUT) cp_async_16(smem_u32(buf + C::kQ + r * C::kLdQ + d), q, ok ? 16 : 0);
     }
-    for (int i = tid; i < kTok * kPV; i += 256) {
+    for (int i = tid; i < kTok * kPV; i += C::kThreads) {
       const int r = i / kPV, c = (i % kPV) * 8;
       const bool ok = r < cnt && e0 + c < p.vp;
       cp_async_16(smem_u32(buf + C::kV + r * C::kLdV + c), ok ? src + r * p.ldp + p.off_v + h * p.vp + e0 + c : proj, ok ? 16 : 0);
     }
     const float2* tab = p.table + static_cast<long long>(pos + t0) * p.hp;     // rows of consecutive positions: one run
-    for (int i = tid * 2; i < cnt * p.hp; i += 512) cp_async_16(smem_u32(stab + i), tab + i, 16);
+    for (int i = tid * 2; i < cnt * p.hp; i += 2 * C::kThreads) cp_async_16(smem_u32(stab + i), tab + i, 16);
     cp_commit();
   };
   issue(0);
 
-  const int m0 = DT >= 128 ? warp * C::kMT * 16 : (warp & 3) * 16, n0 = DT >= 128 ? 0 : (warp >> 2) * (ET / 2);
+  const int m0 = warp / C::kSplit * C::kMT * 16, n0 = warp % C::kSplit * (ET / C::kSplit);
   float S[C::kMT][C::kNT][4];
   {
     const float* src = !OUT ? nullptr : n_spans > 1 ? cr : p.pos0[seq] > 0 ? st : nullptr;
@@ -141,7 +143,7 @@ retention_span_kernel(RetParams p) {
     {
       // scale, and rotate in place: a thread takes both halves of eight pairs
       const int np = p.hp / 8, per = np + (p.dp - 2 * p.hp) / 8;
-      for (int i = tid; i < cnt * per; i += 256) {
+      for (int i = tid; i < cnt * per; i += C::kThreads) {
         const int r = i / per, w = i % per;
 #pragma unroll
         for (int which = 0; which < (OUT ? 2 : 1); ++which) {
@@ -188,7 +190,7 @@ retention_span_kernel(RetParams p) {
     if (C::kBuf == 2 && t0 + kTok < n) issue(t0 + kTok);
     const uint32_t aQ = smem_u32(buf + C::kQ), aK = smem_u32(buf + C::kK), aV = smem_u32(buf + C::kV);
     if constexpr (OUT) {
-      const int rg = warp & 3, r0 = rg * 16, c0 = (warp >> 2) * (ET / 2);
+      const int rg = warp & 3, r0 = rg * 16, c0 = (warp >> 2) * (ET / C::kCols);
       float acc[C::kOT][4];
 #pragma unroll
       for (int j = 0; j < C::kOT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
@@ -221,17 +223,27 @@ retention_span_kernel(RetParams p) {
       for (int j = 0; j < C::kOT; ++j) {
         acc[j][0] *= w0; acc[j][1] *= w0; acc[j][2] *= w1; acc[j][3] *= w1;
       }
+      // decay^(i - key) as decay^(i - first key of the block) times decay^-(place in the block); a decay so steep that the second
+      // factor could overflow takes the power itself
+      const bool steep = lg < -8.f;
+      float back_in[2][2];
+#pragma unroll
+      for (int b = 0; b < 2; ++b)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) back_in[b][e] = decay_pow(lg, -(b * 8 + 2 * t4 + e));
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         if (j > rg) break;
         uint32_t hi[4], lo[4];
+        const float from[2] = {decay_pow(lg, r0 + g - 16 * j), decay_pow(lg, r0 + g + 8 - 16 * j)};
 #pragma unroll
         for (int b = 0; b < 2; ++b) {
           float f[4];
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int back = r0 + g + (e >> 1) * 8 - (j * 16 + b * 8 + 2 * t4 + (e & 1));
-            f[e] = back < 0 ? 0.f : sc[2 * j + b][e] * decay_pow(lg, back);
+            const float w = steep ? decay_pow(lg, back) : from[e >> 1] * back_in[b][e & 1];
+            f[e] = back < 0 ? 0.f : sc[2 * j + b][e] * w;
           }
           split_bf16x2(f[0], f[1], &hi[2 * b], &lo[2 * b]);
           split_bf16x2(f[2], f[3], &hi[2 * b + 1], &lo[2 * b + 1]);
@@ -279,7 +291,10 @@ retention_span_kernel(RetParams p) {
         for (int e = 0; e < 2; ++e) {
           const int r = r0 + g + 8 * e;
           if (r >= cnt) continue;
-          const float rs = rsqrtf((srow[r] + srow[kTok + r]) / static_cast<float>(p.vdim) + p.eps);
+          float ss = 0.f;
+#pragma unroll
+          for (int q = 0; q < C::kCols; ++q) ss += srow[q * kTok + r];
+          const float rs = rsqrtf(ss / static_cast<float>(p.vdim) + p.eps);
           T* out = static_cast<T*>(p.out) + static_cast<long long>(row0 + t0 + r) * p.ldo + h * p.vp;
 #pragma unroll
           for (int j = 0; j < C::kOT; ++j) {
@@ -582,7 +597,7 @@ int launch_span(const RetParams& p, cudaStream_t s) {
   auto kern = retention_span_kernel<DT, ET, OUT>;
   static PerDeviceFlag attr;
   if (const int e = opt_in_smem(kern, &attr, SpanCfg<DT, ET, OUT>::kSmem)) return e;
-  launch_pdl(kern, dim3(p.spans, p.H, (p.vp + ET - 1) / ET), dim3(256), SpanCfg<DT, ET, OUT>::kSmem, s, pdl_all_enabled(), p);
+  launch_pdl(kern, dim3(p.spans, p.H, (p.vp + ET - 1) / ET), dim3(SpanCfg<DT, ET, OUT>::kThreads), SpanCfg<DT, ET, OUT>::kSmem, s, pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -289,27 +289,26 @@ rglru_chunk_kernel(RglruParams p) {
   const T* u = static_cast<const T*>(p.u) + static_cast<long long>(p.n_dec + row0) * p.C + blk * p.kp;
   const long long w0 = (static_cast<long long>(blk) * p.kp + n0) * p.kp;
   const T* const w[2] = {static_cast<const T*>(p.ra) + w0, static_cast<const T*>(p.ri) + w0};
+  const int tid = threadIdx.x, n = tid & 63, c = blk * p.kp + n0 + n;
+  const bool ok = n < cols;
+  // this thread's inputs of the gates, requested ahead of the products: rows (tid / 64) + 2 i of one channel
+  T uu[kChunk / 2];
+  {
+    const T* uc = u + n0 + (ok ? n : 0);
+#pragma unroll
+    for (int i = 0; i < kChunk / 2; ++i) uu[i] = uc[static_cast<long long>(min((tid >> 6) + 2 * i, rows - 1)) * p.C];
+  }
   float* acc = Tile::run(smem, u, p.C, rows, w, p.kp, cols, p.kp);
   float* sa = acc;
   float* sb = acc + kChunk * Tile::kLdC;
-  const int tid = threadIdx.x, n = tid & 63, c = blk * p.kp + n0 + n;
-  const bool ok = n < cols;
   {
     const float rb = ok ? p.ra_b[c] : 0.f, ib = ok ? p.ri_b[c] : 0.f, dc = ok ? p.decay[c] : 0.f;
-    const T* uc = u + n0 + (ok ? n : 0);
-    constexpr int kPer = 8;                        // tokens whose inputs are requested together
-#pragma unroll 1
-    for (int r0 = tid >> 6; r0 < rows; r0 += 2 * kPer) {
-      float uu[kPer];
 #pragma unroll
-      for (int i = 0; i < kPer; ++i) uu[i] = to_f32<T>(uc[static_cast<long long>(min(r0 + 2 * i, rows - 1)) * p.C]);
-#pragma unroll
-      for (int i = 0; i < kPer; ++i) {             // (rows past the end compute on zeros and are not used)
-        const int at = (r0 + 2 * i) * Tile::kLdC + n;
-        const Gates g = rglru_gates<sizeof(T) == 2>(sa[at] + rb, sb[at] + ib, dc, uu[i]);
-        sa[at] = g.a;
-        sb[at] = g.b;
-      }
+    for (int i = 0; i < kChunk / 2; ++i) {         // (rows past the end compute on zeros and are not used)
+      const int at = ((tid >> 6) + 2 * i) * Tile::kLdC + n;
+      const Gates g = rglru_gates<sizeof(T) == 2>(sa[at] + rb, sb[at] + ib, dc, to_f32<T>(uu[i]));
+      sa[at] = g.a;
+      sb[at] = g.b;
     }
   }
   __syncthreads();
@@ -441,7 +440,7 @@ int run_rglru(const RglruParams& p, cudaStream_t s) {
   int rc = static_cast<int>(cudaGetLastError());
   if (rc) return rc;
   if (p.n_dec > 0) {
-    rc = p.n_dec <= 512 ? launch_step<T, 16>(p, s) : launch_step<T, 64>(p, s);
+    rc = p.n_dec <= 128 ? launch_step<T, 16>(p, s) : launch_step<T, 64>(p, s);
     if (rc) return rc;
   }
   if (p.rows > p.n_dec) {
