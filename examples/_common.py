@@ -36,13 +36,15 @@ def preset(name: str, dtype: torch.dtype, max_pos: int) -> LlamaConfig:
         cfg = LlamaConfig.llama_3_2_1b()
         cfg.dtype, cfg.max_position_embeddings = dtype, max_pos
         return cfg
-    if name.startswith("fozelix-"):
-        from tesseract_b200.models import fozelix
+    if name.startswith(("fozelix-", "polosun-")):
+        from tesseract_b200 import models
+        family, size = name.split("-", 1)
         try:
-            return fozelix.preset(name[len("fozelix-"):], dtype)
+            return getattr(models, family).preset(size, dtype)
         except ValueError as e:
             raise SystemExit(f"error: --model: {e}") from None
-    raise SystemExit(f"error: unknown --model '{name}' (tiny | small | llama3.2-1b | llama3-8b | fozelix-tiny | fozelix-small)")
+    raise SystemExit(f"error: unknown --model '{name}' (tiny | small | llama3.2-1b | llama3-8b | fozelix-tiny | fozelix-small | "
+                     "polosun-tiny | polosun-small)")
 
 
 def random_model(cfg, device, seed: int):

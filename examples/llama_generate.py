@@ -1,6 +1,6 @@
 #!/usr/bin/env python
 """Text generation from a model directory (config.json + model.safetensors; the model registry picks the family: Hugging
-Face Llama, Fozelix) or a random-weight preset (the reference's examples/llama_generate.cpp, same flags).
+Face Llama, Fozelix, Polosun) or a random-weight preset (the reference's examples/llama_generate.cpp, same flags).
 
     python examples/llama_generate.py --model-dir /path/to/Llama-3.2-1B --prompt "Hello" --max-new-tokens 64
     python examples/llama_generate.py --config c.json --safetensors m.safetensors --tokenizer tokenizer.json --prompt hi
@@ -23,7 +23,7 @@ def main() -> int:
     ap.add_argument("--config", default="")
     ap.add_argument("--safetensors", default="")
     ap.add_argument("--tokenizer", default="")
-    ap.add_argument("--model", default="", help="random-weight preset instead of files: tiny | small | llama3-8b | fozelix-tiny | fozelix-small")
+    ap.add_argument("--model", default="", help="random-weight preset instead of files: tiny | small | llama3-8b | fozelix-tiny | fozelix-small | polosun-tiny | polosun-small")
     ap.add_argument("--prompt", default="Hello")
     ap.add_argument("--device", default="cpu")
     ap.add_argument("--max-new-tokens", type=int, default=32)

@@ -260,7 +260,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   __shared__ uint32_t tmem_base_smem;
   __shared__ volatile int cta_abort;
   __shared__ float smax[2][4][kHeads], lsum[4][kHeads], corr[kHeads];
-  const int split = blockIdx.x, h0 = blockIdx.y * kHeads, row = blockIdx.z;
+  const int split = blockIdx.z, h0 = blockIdx.y * kHeads, row = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int len = p.lens ? p.lens[row] : p.pos[row] + 1;
   const int share = ((len + p.splits - 1) / p.splits + kKeys - 1) / kKeys * kKeys;
@@ -645,7 +645,7 @@ int launch_latent_decode(const LatentAttnParams& p, cudaStream_t s) {
   CUtensorMap tm_q, tm_pool;
   if (!make_tmap_2d(&tm_q, p.q, 2, static_cast<uint64_t>(p.rows) * p.H, L, L * 2ull, kHeads, 64, true) ||
       !make_tmap_2d(&tm_pool, p.pool, 2, static_cast<uint64_t>(p.nb) * p.bs, L, L * 2ull, run, 64, true)) return -3;
-  launch_pdl(latent_decode_kernel, dim3(p.splits, (p.H + kHeads - 1) / kHeads, p.rows), dim3(192), plan.smem, s, pdl_all_enabled(), tm_q,
+  launch_pdl(latent_decode_kernel, dim3(p.rows, (p.H + kHeads - 1) / kHeads, p.splits), dim3(192), plan.smem, s, pdl_all_enabled(), tm_q,
              tm_pool, p);
   return static_cast<int>(cudaGetLastError());
 }
@@ -767,7 +767,7 @@ TSB_EXPORT int tsb_latent_attn(const void* q, const void* pool, const int* table
     if (dtype == 1) return launch_latent_rows<__nv_bfloat16>(p, s);
     return dtype == 0 ? launch_latent_rows<float>(p, s) : -2;
   }
-  if (dtype != 1 || cp % 64 || cp > 512 || rp % 32 || rp <= 0 || bs % 8 || rows > 65535 || (splits > 1 && (!part_o || !part_ml))) return -2;
+  if (dtype != 1 || cp % 64 || cp > 512 || rp % 32 || rp <= 0 || bs % 8 || splits > 65535 || (splits > 1 && (!part_o || !part_ml))) return -2;
   const int rc = launch_latent_decode(p, s);
   if (rc || splits == 1) return rc;
   launch_pdl(latent_merge_kernel, dim3(static_cast<unsigned>(rows * H)), dim3(128), 0, s, pdl_all_enabled(), p);

@@ -4,6 +4,8 @@ import os
 import subprocess
 import sys
 
+import pytest
+
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 
@@ -67,17 +69,20 @@ def test_llama_forward_and_infer():
     assert _run("llama_infer.py").returncode != 0
 
 
-def test_examples_take_every_registered_family(tmp_path):
+@pytest.mark.parametrize("family", ["fozelix", "polosun"])
+def test_examples_take_every_registered_family(tmp_path, family):
     import torch
-    from tesseract_b200.models import HybridModel, fozelix
-    cfg = fozelix.preset("tiny", torch.float32)
+    from tesseract_b200 import models
+    from tesseract_b200.models import HybridModel
+    module, preset = getattr(models, family), family + "-tiny"
+    cfg = module.preset("tiny", torch.float32)
     HybridModel(cfg, init_std=0.05, seed=1).save_safetensors(str(tmp_path / "model.safetensors"))
-    (tmp_path / "config.json").write_text(__import__("json").dumps(fozelix.config_to_dict(cfg)))
+    (tmp_path / "config.json").write_text(__import__("json").dumps(module.config_to_dict(cfg)))
     args = ("llama_generate.py", "--model-dir", str(tmp_path), "--prompt", "hi", "--max-new-tokens", "6", "--no-stream")
     r = _run(*args)
     assert r.returncode == 0 and "6 new tokens" in r.stderr, r.stderr
     assert _run(*args).stdout == r.stdout
-    for extra in (("--model", "fozelix-tiny"), ("--model-dir", str(tmp_path)), ("--model", "fozelix-tiny", "--engine", "batched")):
+    for extra in (("--model", preset), ("--model-dir", str(tmp_path)), ("--model", preset, "--engine", "batched")):
         r = _run("llama_serve.py", *extra, "--prompts", "a|bb|ccc", "--max-new-tokens", "4", "--max-batch", "2")
         assert r.returncode == 0 and "3 requests, 12 tokens" in r.stdout, r.stderr
     r = _run("llama_infer.py", "--model-dir", str(tmp_path), "--batch", "2", "--seq", "9", "--topk", "2")
