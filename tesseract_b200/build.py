@@ -35,6 +35,7 @@ CUDA_LIB = LIB_DIR / "libtesseract_b200_cuda.so"
 _HYBRID = ("runtime", "gemm_tcgen05", "gemm_decode_wq", "gemm_decode_mx", "flash_attn_fwd", "dyn_tanh", "sampling")
 GROUPS = {
     "fozelix": _HYBRID + ("decode_attn", "decode_attn_mma", "ragged_attn", "delta_rule"),
+    "vobotar": _HYBRID + ("attn_prepare", "decode_attn", "decode_attn_mma", "post_norm", "ragged_attn", "ssd", "time_mix"),
     "polosun": _HYBRID + ("depth_residual", "latent_attn", "retention", "rglru"),
 }
 

@@ -1,0 +1,180 @@
+// What happens to a packed projection row [q: H heads | k: Hkv | v: Hkv | ..] before attention: biases, a norm of q and k (per
+// head, or over all heads at once), rotation by position, values mixed with those of an earlier layer; q goes to a buffer of its
+// own, k and v to the token's pool slot and, for prompt rows, to the key axis of the tensor-core kernel.
+//
+// One CTA per row. LPH lanes share a head (16 bytes each, PPL times), so a warp takes 32 / LPH heads at once. Everything between
+// load and store is fp32.
+#include "warp_mma.cuh"
+
+namespace tsb {
+namespace {
+
+struct PrepareParams {
+  int rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, ld;    // norm: 0 none, 1 unit heads, 2 heads with a weight, 3 whole
+  float eps, vmix;
+  const void* proj;
+  const float* bias;          // [off_v + Hkv * D] or null
+  const float* q_norm;
+  const float* k_norm;
+  const float2* table;        // [positions, hp] or null
+  const int* positions;
+  const int* slots;
+  void* q;                    // [rows, H, D]
+  void* k_pool;               // [blocks, Hkv, bs, D]
+  void* v_pool;
+  const void* v_first;        // pool like v_pool, or null
+  void* stage;                // [keys, 2 Hkv, D] or null
+  const int* stage_rows;      // [rows - n_decode]
+};
+
+template <typename T, int LPH, int PPL>
+__global__ void __launch_bounds__(256)
+attn_prepare_kernel(PrepareParams p) {
+  pdl_trigger();
+  pdl_grid_wait();
+  constexpr int V = kVec16<T>;
+  __shared__ float red[2][8];
+  const int row = blockIdx.x, tid = threadIdx.x, gl = tid % LPH, first = tid / LPH, step = blockDim.x / LPH;
+  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(row) * p.ld;
+  const int units = p.H + 2 * p.Hkv, D = p.D;
+  auto load = [&](int col, float (&f)[V]) {         // V columns of the row, with their biases
+    ld16<T>(x + col, f);
+    if (p.bias) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] += p.bias[col + i];
+    }
+  };
+  float whole_q = 0.f, whole_k = 0.f;
+  if (p.norm == 3) {
+    float sq = 0.f, sk = 0.f;
+    for (int c = tid * V; c < (p.H + p.Hkv) * D; c += blockDim.x * V) {
+      const bool is_k = c >= p.H * D;
+      float f[V], s = 0.f;
+      load(is_k ? p.off_k + c - p.H * D : c, f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) s = fmaf(f[i], f[i], s);
+      if (is_k) sk += s;
+      else sq += s;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((tid & 31) == 0) {
+      red[0][tid >> 5] = sq;
+      red[1][tid >> 5] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.f;
+    for (int w = 0; w < static_cast<int>(blockDim.x) / 32; ++w) {
+      sq += red[0][w];
+      sk += red[1][w];
+    }
+    whole_q = 1.f / sqrtf(sq / static_cast<float>(p.H * p.dim) + p.eps);
+    whole_k = 1.f / sqrtf(sk / static_cast<float>(p.Hkv * p.dim) + p.eps);
+  }
+  const int slot = p.slots[row];
+  const long long page = slot >= 0 ? static_cast<long long>(slot / p.bs) * p.Hkv * p.bs + slot % p.bs : 0;
+  const int stage_row = p.stage && row >= p.n_decode ? p.stage_rows[row - p.n_decode] : -1;
+  const float2* turn = p.table && p.hp > 0 ? p.table + static_cast<long long>(max(p.positions[row], 0)) * p.hp : nullptr;
+  for (int u0 = 0; u0 < units; u0 += step) {        // (every lane takes every turn: the sums below are shuffles)
+    const int u = u0 + first;
+    const bool there = u < units;
+    const int kind = u < p.H ? 0 : u < p.H + p.Hkv ? 1 : 2;
+    const int head = kind == 0 ? u : kind == 1 ? u - p.H : u - p.H - p.Hkv;
+    const int col = (kind == 0 ? 0 : kind == 1 ? p.off_k : p.off_v) + head * D;
+    float f[PPL][V], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PPL; ++k) {
+      const int d = (gl + k * LPH) * V;
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[k][i] = 0.f;
+      if (there && d < D) load(col + d, f[k]);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss = fmaf(f[k][i], f[k][i], ss);
+    }
+    float rs = kind == 0 ? whole_q : whole_k;
+    if (p.norm == 1 || p.norm == 2) {
+#pragma unroll
+      for (int o = LPH / 2; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      rs = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+    }
+    if (!there) continue;
+    const float* w = p.norm < 2 ? nullptr : (kind == 0 ? p.q_norm : p.k_norm) + (p.norm == 3 ? head * D : 0);
+#pragma unroll
+    for (int k = 0; k < PPL; ++k) {
+      const int d = (gl + k * LPH) * V;
+      if (d >= D) continue;
+      if (kind == 2) {
+        if (p.v_first) {
+          float v0[V] = {};
+          if (slot >= 0) ld16<T>(static_cast<const T*>(p.v_first) + (page + static_cast<long long>(head) * p.bs) * D + d, v0);
+#pragma unroll
+          for (int i = 0; i < V; ++i) f[k][i] = (1.f - p.vmix) * f[k][i] + p.vmix * v0[i];
+        }
+      } else {
+        if (p.norm) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) f[k][i] *= w ? rs * w[d + i] : rs;
+        }
+        if (turn && d < 2 * p.hp) {
+          const bool second = d >= p.hp;
+          const int i0 = second ? d - p.hp : d, other = second ? i0 : d + p.hp;
+          float g[V];
+          load(col + other, g);
+          if (p.norm) {
+#pragma unroll
+            for (int i = 0; i < V; ++i) g[i] *= w ? rs * w[other + i] : rs;
+          }
+#pragma unroll
+          for (int i = 0; i < V; ++i) {
+            const float2 cs = turn[i0 + i];
+            f[k][i] = second ? f[k][i] * cs.x + g[i] * cs.y : f[k][i] * cs.x - g[i] * cs.y;
+          }
+        }
+      }
+      if (kind == 0) {
+        st16<T>(static_cast<T*>(p.q) + (static_cast<long long>(row) * p.H + head) * D + d, f[k]);
+        continue;
+      }
+      if (slot >= 0) st16<T>(static_cast<T*>(kind == 1 ? p.k_pool : p.v_pool) + (page + static_cast<long long>(head) * p.bs) * D + d, f[k]);
+      if (stage_row >= 0)
+        st16<T>(static_cast<T*>(p.stage) + (static_cast<long long>(stage_row) * 2 * p.Hkv + (kind == 1 ? 0 : p.Hkv) + head) * D + d, f[k]);
+    }
+  }
+}
+
+template <typename T>
+int launch_prepare(const PrepareParams& p, cudaStream_t s) {
+  const int pieces = p.D / kVec16<T>;
+  const int lph = pieces <= 8 ? 8 : pieces <= 16 ? 16 : 32;
+  const int lanes = (p.H + 2 * p.Hkv) * lph;
+  const int nt = lanes >= 256 ? 256 : (lanes + 31) / 32 * 32;
+  const bool pdl = pdl_all_enabled();
+#define TSB_PREP(L, N) launch_pdl(attn_prepare_kernel<T, L, N>, dim3(p.rows), dim3(nt), 0, s, pdl, p)
+  if (lph == 8) TSB_PREP(8, 1);
+  else if (lph == 16) TSB_PREP(16, 1);
+  else if (pieces <= 32) TSB_PREP(32, 1);
+  else TSB_PREP(32, 2);
+#undef TSB_PREP
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace
+}  // namespace tsb
+
+// ints: rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, row stride; floats: eps, vmix; ptrs: proj, bias, q_norm, k_norm,
+// table, positions, slots, q, k_pool, v_pool, v_first, stage, stage_rows (see PrepareParams). dtype: 0 = fp32, 1 = bf16. D is a
+// multiple of 32, up to 256; rows and sections start on 16 bytes.
+TSB_EXPORT int tsb_attn_prepare(const int* v, const float* f, void* const* q, int dtype, void* stream) {
+  using namespace tsb;
+  PrepareParams p{v[0], v[1], v[2], v[3], v[4], v[5], v[6], v[7], v[8], v[9], v[10], v[11], f[0], f[1], q[0], static_cast<const float*>(q[1]),
+                  static_cast<const float*>(q[2]), static_cast<const float*>(q[3]), static_cast<const float2*>(q[4]),
+                  static_cast<const int*>(q[5]), static_cast<const int*>(q[6]), q[7], q[8], q[9], q[10], q[11], static_cast<const int*>(q[12])};
+  if (p.rows <= 0 || p.H <= 0 || p.Hkv <= 0 || p.D <= 0 || p.D % 32 || p.D > 256 || p.dim <= 0 || p.dim > p.D || p.hp % 8 || 2 * p.hp > p.D ||
+      p.off_k % 8 || p.off_v % 8 || p.ld % 8 || p.norm < 0 || p.norm > 3 || (p.norm >= 2 && (!p.q_norm || !p.k_norm)) || p.bs <= 0 ||
+      (p.stage && !p.stage_rows) || (reinterpret_cast<uintptr_t>(p.proj) & 15))
+    return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == 1) return launch_prepare<__nv_bfloat16>(p, s);
+  if (dtype == 0) return launch_prepare<float>(p, s);
+  return -2;
+}

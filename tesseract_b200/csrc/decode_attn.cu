@@ -14,7 +14,7 @@
 //   * 128-bit loads: 8 lanes cover one D = 128 row, 4 tokens per warp per step, two steps in flight.
 // The INT8 path dequantises in registers: s = (q . kq) * k_scale, o += p * v_scale * vq
 // (per-(token, head) symmetric scales, src/cuda/QuantizeKV.cu:51-72).
-#include "common.cuh"
+#include "attn_form.cuh"
 #include "tsb_no_alloc.h"
 
 #include <cuda_fp8.h>
@@ -27,6 +27,9 @@ namespace tsb {
 int paged_decode_mma_dispatch(const void* q, const void* k_pool, const void* v_pool, const float* k_scale,
                               const float* v_scale, const int* tables, const int* lens, void* out, float* part_o, float* part_ml, int A, int H, int Hkv, int D, int bs, int nb,
                               int max_logical, int splits, int gh, float scale_log2, int chunk, int dtype, cudaStream_t s);
+int paged_decode_mma_shaped(const void* q, const void* k_pool, const void* v_pool, const int* tables, const int* lens, void* out,
+                            float* part_o, float* part_ml, int A, int H, int Hkv, int D, int bs, int nb, int max_logical, int splits,
+                            int gh, const AttnForm& form, const AttnGate& gate, cudaStream_t s);
 
 namespace {
 
@@ -555,14 +558,25 @@ TSB_EXPORT int tsb_paged_decode(const void* q, const void* k_pool, const void* v
                       max_len, 0, dtype, stream);
 }
 
-// The same under a chunk mask: the newest token (position lens[a] - 1) sees only the keys of its own run of `chunk`
-// positions. max_len bounds lens as above (the key split is planned for min(max_len, chunk) keys); bf16 / fp16 pools.
-TSB_EXPORT int tsb_paged_decode_chunked(const void* q, const void* k_pool, const void* v_pool, const int* tables,
-                                        const int* lens, void* out, float* scratch, int A, int H, int Hkv, int D, int bs, int nb,
-                                        int max_logical, float scale, int max_len, int chunk, int dtype, void* stream) {
-  if (chunk <= 0) return -2;
-  return paged_decode(q, k_pool, v_pool, nullptr, nullptr, tables, lens, out, scratch, A, H, Hkv, D, bs, nb, max_logical, scale,
-                      max_len < chunk ? max_len : chunk, chunk, dtype, stream);
+// The same for bf16 pools with masks, score forms, gates and a row stride of the result (ints, floats, ptrs: see attn_form.cuh).
+// max_len bounds lens as above; the key split is planned for what the mask leaves of it.
+TSB_EXPORT int tsb_paged_decode_shaped(const void* q, const void* k_pool, const void* v_pool, const int* tables, const int* lens, void* out,
+                                       float* scratch, int A, int H, int Hkv, int D, int bs, int nb, int max_logical, int max_len,
+                                       const long long* ints, const float* floats, const void* const* ptrs, int dtype, void* stream) {
+  using namespace tsb;
+  AttnForm f;
+  AttnGate g;
+  if (A <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || (D != 64 && D != 128) || bs <= 0 || dtype != 1 || !read_attn_form(ints, floats, ptrs, &f, &g))
+    return -2;
+  const int reach = f.chunk > 0 ? f.chunk : f.window > 0 ? f.window : max_len;
+  if (max_len > reach) max_len = reach;
+  if (f.plain() && g.plain() && g.ldo == static_cast<long long>(H) * D)
+    return paged_decode(q, k_pool, v_pool, nullptr, nullptr, tables, lens, out, scratch, A, H, Hkv, D, bs, nb, max_logical, f.scale, max_len,
+                        f.chunk, dtype, stream);
+  int gh = 1, splits = 1;
+  decode_plan(A, H, Hkv, max_len, false, &gh, &splits);
+  return paged_decode_mma_shaped(q, k_pool, v_pool, tables, lens, out, scratch, scratch + static_cast<long long>(A) * H * splits * D, A, H, Hkv,
+                                 D, bs, nb, max_logical, splits, gh, f, g, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" int tsb_quant_act_mx_layout(const void* X, long long ldx, void* Xq, void* sf, int M, int K, int atoms,

@@ -15,7 +15,7 @@
 // when there is one split); the merge of splits is decode_merge_kernel of decode_attn.cu.
 // Same inputs, pool layout and clamping rules as tsb_paged_decode (src/cuda/PagedAttention.cu:88-171 is the
 // reference's one-CTA-per-(request, head) CUDA-core kernel).
-#include "common.cuh"
+#include "attn_form.cuh"
 
 #include <type_traits>
 
@@ -88,7 +88,8 @@ struct MmaDecParams {
   float* part_ml;
   int A, H, Hkv, bs, nb, max_logical, splits, gh;  // gh = query heads per CTA (<= 8)
   float scale_log2;
-  int chunk;             // > 0: the newest token sees only the keys of its own run of `chunk` positions
+  AttnForm form;         // (FORM instances; else only its chunk)
+  AttnGate gate;
   int* status;           // device status word: a block-table entry outside the pool is reported there
 };
 
@@ -96,7 +97,8 @@ struct MmaDecParams {
 // tensor-core path straight from the raw key rows: the queries are quantised once per CTA (one scale per head,
 // |q| / 127), the sums are exact int32, and query scale x key scale multiply S afterwards. The values are widened to
 // fp16 in a per-warp conversion buffer (int8 is exact in fp16) for P V, with the V scales riding on P.
-template <typename T, int D, bool INT8>
+// FORM: windows, score forms, gates and row strides of the result (attn_form.cuh).
+template <typename T, int D, bool INT8, bool FORM>
 __global__ void __launch_bounds__(kWarps * 32)
 paged_decode_mma_kernel(MmaDecParams p) {
   pdl_trigger();
@@ -128,7 +130,7 @@ paged_decode_mma_kernel(MmaDecParams p) {
   const int g = lane >> 2, t4 = lane & 3;
 
   const int len = p.lens[a];
-  const int first = p.chunk > 0 && len > 0 ? (len - 1) / p.chunk * p.chunk : 0;
+  const int first = len > 0 ? p.form.first(len - 1) : 0;
   const int share = ((len - first + p.splits - 1) / p.splits + 15) & ~15;
   const int t_begin = first + split * share;
   const int t_end = min(len, t_begin + share);
@@ -192,6 +194,7 @@ paged_decode_mma_kernel(MmaDecParams p) {
   float o[D / 8][2];  // O[head g][d = nb*8 + 2t, +1]
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = 0.f;
+  const ScoreLog2 score(p.form, FORM && g < p.gh ? h0 + g : 0);
   float m_run = -INFINITY, l_part = 0.f;  // l_part: this lane's share of the row sum (reduced at the end)
 
   // tiles of this warp: warp, warp + 4, ... ; `issue(j)` starts the copies of this warp's j-th tile
@@ -326,7 +329,9 @@ paged_decode_mma_kernel(MmaDecParams p) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int t = tok0 + b * 8 + 2 * t4 + e;
-        float sv = s[b][e] * p.scale_log2;
+        float sv;
+        if constexpr (FORM) sv = score(s[b][e], len - 1 - t);
+        else sv = s[b][e] * p.scale_log2;
         if constexpr (INT8) sv *= sc[b * 8 + 2 * t4 + e];
         s[b][e] = t < t_end ? sv : -INFINITY;
         mx = fmaxf(mx, s[b][e]);
@@ -410,7 +415,10 @@ paged_decode_mma_kernel(MmaDecParams p) {
       ll += sm_l[w * 8 + hh] * c;
     }
     const int h = h0 + hh;
-    if (p.splits == 1) {
+    if (FORM && p.splits == 1) {
+      if (p.form.sink && ll > 0.f) ll += exp2f(p.form.sink[h] * kLog2e - nm);
+      static_cast<T*>(p.out)[a * p.gate.ldo + h * D + d] = from_f32<T>(ll > 0.f ? acc / ll * p.gate.factor<T>(a, h, D, d) : 0.f);
+    } else if (p.splits == 1) {
       static_cast<T*>(p.out)[(static_cast<long long>(a) * p.H + h) * D + d] = from_f32<T>(ll > 0.f ? acc / ll : 0.f);
     } else {
       const long long pi = (static_cast<long long>(a) * p.H + h) * p.splits + split;
@@ -423,7 +431,28 @@ paged_decode_mma_kernel(MmaDecParams p) {
   }
 }
 
-template <typename T, int D, bool INT8>
+// The merge of the key splits with a sink, gates and a row stride of the result.
+template <typename T, int D>
+__global__ void __launch_bounds__(D)
+decode_merge_shaped_kernel(MmaDecParams p) {
+  pdl_trigger();
+  pdl_grid_wait();
+  const int a = blockIdx.x / p.H, h = blockIdx.x % p.H, d = threadIdx.x;
+  const long long at = static_cast<long long>(blockIdx.x) * p.splits;
+  float nm = -INFINITY;
+  for (int s = 0; s < p.splits; ++s) nm = fmaxf(nm, p.part_ml[(at + s) * 2]);
+  float acc = 0.f, ll = 0.f;
+  for (int s = 0; s < p.splits; ++s) {
+    const float ms = p.part_ml[(at + s) * 2];
+    const float c = ms == -INFINITY ? 0.f : exp2f(ms - nm);
+    acc += p.part_o[(at + s) * D + d] * c;
+    ll += p.part_ml[(at + s) * 2 + 1] * c;
+  }
+  if (p.form.sink && ll > 0.f) ll += exp2f(p.form.sink[h] * kLog2e - nm);
+  static_cast<T*>(p.out)[a * p.gate.ldo + h * D + d] = from_f32<T>(ll > 0.f ? acc / ll * p.gate.factor<T>(a, h, D, d) : 0.f);
+}
+
+template <typename T, int D, bool INT8, bool FORM = false>
 int launch_mma(const MmaDecParams& p, cudaStream_t s) {
   constexpr int kRowBytes = D * 2 + 16;
   constexpr int kTileBytes = kTile * kRowBytes;
@@ -432,7 +461,7 @@ int launch_mma(const MmaDecParams& p, cudaStream_t s) {
   constexpr int ring = kWarps * (kStagesD * kStageBytes + (INT8 ? kTileBytes : 0));
   constexpr int merge = (kWarps * 8 * D + 2 * kWarps * 8) * 4;
   constexpr int smem = (ring > merge ? ring : merge) + 128;
-  auto kern = paged_decode_mma_kernel<T, D, INT8>;
+  auto kern = paged_decode_mma_kernel<T, D, INT8, FORM>;
   static PerDeviceFlag attr;
   if (attr.unset()) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -442,6 +471,9 @@ int launch_mma(const MmaDecParams& p, cudaStream_t s) {
   const int G = p.H / p.Hkv;
   dim3 grid(p.splits, p.Hkv * (G / p.gh), p.A);
   launch_pdl(kern, grid, dim3(kWarps * 32), smem, s, pdl_all_enabled(), p);
+  if constexpr (FORM) {
+    if (p.splits > 1) launch_pdl(decode_merge_shaped_kernel<T, D>, dim3(p.A * p.H), dim3(D), 0, s, pdl_all_enabled(), p);
+  }
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -453,13 +485,13 @@ int paged_decode_mma_dispatch(const void* q, const void* k_pool, const void* v_p
                               void* out, float* part_o, float* part_ml, int A, int H, int Hkv, int D, int bs, int nb,
                               int max_logical, int splits, int gh, float scale_log2, int chunk, int dtype, cudaStream_t s) {
   if (gh > 8 || (D != 64 && D != 128)) return -100;
-  MmaDecParams p;
+  MmaDecParams p{};
   p.q = q; p.k_pool = k_pool; p.v_pool = v_pool; p.k_scale = k_scale; p.v_scale = v_scale;
   p.tables = tables; p.lens = lens; p.out = out;
   p.part_o = part_o; p.part_ml = part_ml;
   p.A = A; p.H = H; p.Hkv = Hkv; p.bs = bs; p.nb = nb; p.max_logical = max_logical; p.splits = splits; p.gh = gh;
   p.scale_log2 = scale_log2;
-  p.chunk = chunk;
+  p.form.chunk = chunk;
   p.status = device_status_word();
   const bool i8 = k_scale != nullptr;
   if (dtype == 1) {
@@ -471,6 +503,18 @@ int paged_decode_mma_dispatch(const void* q, const void* k_pool, const void* v_p
     return i8 ? launch_mma<__half, 64, true>(p, s) : launch_mma<__half, 64, false>(p, s);
   }
   return -100;
+}
+
+// The same with the score forms, gates and row stride of attn_form.cuh (bf16 pools; merges the key splits itself).
+int paged_decode_mma_shaped(const void* q, const void* k_pool, const void* v_pool, const int* tables, const int* lens, void* out,
+                            float* part_o, float* part_ml, int A, int H, int Hkv, int D, int bs, int nb, int max_logical, int splits,
+                            int gh, const AttnForm& form, const AttnGate& gate, cudaStream_t s) {
+  if (gh > 8 || (D != 64 && D != 128)) return -2;
+  MmaDecParams p{};
+  p.q = q; p.k_pool = k_pool; p.v_pool = v_pool; p.tables = tables; p.lens = lens; p.out = out; p.part_o = part_o; p.part_ml = part_ml;
+  p.A = A; p.H = H; p.Hkv = Hkv; p.bs = bs; p.nb = nb; p.max_logical = max_logical; p.splits = splits; p.gh = gh;
+  p.form = form; p.gate = gate; p.status = device_status_word();
+  return D == 128 ? launch_mma<__nv_bfloat16, 128, false, true>(p, s) : launch_mma<__nv_bfloat16, 64, false, true>(p, s);
 }
 
 }  // namespace tsb

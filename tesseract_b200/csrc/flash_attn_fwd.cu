@@ -14,7 +14,7 @@
 // row produces zeros; softmax statistics are fp32; scale is folded into the exponent
 // (src/cuda/FusedAttention.cu:69-80,318-331,368-567 is the WMMA kernel this replaces).
 // Also writes the per-row log-sum-exp needed by the backward kernel.
-#include "common.cuh"
+#include "attn_form.cuh"
 
 #include <algorithm>
 
@@ -49,6 +49,8 @@ struct FaParams {
   float scale;
   int causal;
   int* status;
+  AttnForm form;          // (FORM instances)
+  AttnGate gate;
 };
 
 // Descriptor for k-step `ks` (16 elements along K) of a K-major [rows x D] tile made of 64-column halves.
@@ -67,7 +69,9 @@ __device__ __forceinline__ uint64_t mnmajor_desc(uint32_t base, int ks, uint32_t
 // when a row's maximum has grown by more than 2^8 since the reference maximum of its exponents was set; the score
 // row is read from TMEM once per tile and kept in registers for both the maximum and the exponentials.
 // LAZY = false: the output is folded into fp32 registers after every tile (two reads of the score row per tile).
-template <int D, bool LAZY>
+// FORM = true (with LAZY = false): windows, score forms and gates of attn_form.cuh; the scores go back to TMEM in their final
+// form, in units of log 2, between the two reads. Key tiles in front of the window are not visited.
+template <int D, bool LAZY, bool FORM = false>
 __global__ void __launch_bounds__(kFaThreads, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                  const __grid_constant__ CUtensorMap tmV, FaParams p_in) {
@@ -117,6 +121,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const int lim = last_col < 0 ? 0 : last_col / BKV + 1;
     n_tiles = min(n_tiles, lim);
   }
+  int j0 = 0;                  // first key tile
+  if constexpr (FORM) {
+    if (p.form.window > 0) j0 = max(0, q0 + offset - p.form.window + 1) / BKV;
+    n_tiles = max(0, n_tiles - j0);
+  }
 
   if (threadIdx.x == 0) {
     cta_abort = 0;
@@ -158,12 +167,12 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         mbar_expect_tx(&k_full[st], Cfg::kTileBytes);
 #pragma unroll
         for (int hf = 0; hf < Cfg::kHalves; ++hf)
-          tma_load_4d(sK + st * Cfg::kTileBytes + hf * 16384, &tmK, &k_full[st], hf * 64, j * BKV + krow0, hk, bb);
+          tma_load_4d(sK + st * Cfg::kTileBytes + hf * 16384, &tmK, &k_full[st], hf * 64, (FORM ? j0 + j : j) * BKV + krow0, hk, bb);
         if (!mbar_wait(&v_empty[st], par, &cta_abort, p.status)) break;
         mbar_expect_tx(&v_full[st], Cfg::kTileBytes);
 #pragma unroll
         for (int hf = 0; hf < Cfg::kHalves; ++hf)
-          tma_load_4d(sV + st * Cfg::kTileBytes + hf * 16384, &tmV, &v_full[st], hf * 64, j * BKV + krow0, hk, bb);
+          tma_load_4d(sV + st * Cfg::kTileBytes + hf * 16384, &tmV, &v_full[st], hf * 64, (FORM ? j0 + j : j) * BKV + krow0, hk, bb);
       }
     }
   } else if (warp == 5) {
@@ -365,14 +374,16 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     float m_run = -INFINITY, l_run = 0.f, alpha_prev = 1.f;
     bool ok = true;
     const int row_limit = qi + offset;  // last visible key under causal masking
+    const ScoreLog2 score(p.form, FORM ? h : 0);
+    const float mul = FORM ? 1.f : p.scale_log2;
 
     for (int j = 0; j < n_tiles; ++j) {
       const int st = j & 1;
       if (!mbar_wait(&s_full[st], (j >> 1) & 1, &cta_abort, p.status)) { ok = false; break; }
       tc_fence_after();
       const uint32_t s_addr = tmem_base + lane_addr + (st ? Cfg::kColS1 : Cfg::kColS0);
-      const int c0 = j * BKV;
-      const bool need_mask = (p.causal && c0 + BKV - 1 > q0 + offset) || (c0 + BKV > p.Sk);
+      const int c0 = (FORM ? j0 + j : j) * BKV;
+      const bool need_mask = !FORM && ((p.causal && c0 + BKV - 1 > q0 + offset) || (c0 + BKV > p.Sk));
       int vis = BKV;  // number of visible columns of this tile for this row
       if (need_mask) {
         int lim = p.Sk - c0;
@@ -381,7 +392,25 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       }
       // pass 1: row maximum (tiles that need no masking skip the per-element visibility test)
       float m_tile = -INFINITY;
-      if (need_mask) {
+      if constexpr (FORM) {
+        const int hi = min(p.Sk - 1, row_limit) - c0;                                    // visible columns: lo .. hi
+        const int lo = p.form.window > 0 ? row_limit - p.form.window + 1 - c0 : 0;
+#pragma unroll 1
+        for (int c = 0; c < BKV / 32; ++c) {
+          uint32_t r[32];
+          tmem_ld_32x32(s_addr + c * 32, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const int col = c * 32 + i;
+            const float t = col >= lo && col <= hi ? score(__uint_as_float(r[i]), row_limit - c0 - col) : -INFINITY;
+            m_tile = fmaxf(m_tile, t);
+            r[i] = __float_as_uint(t);
+          }
+          tmem_st_32x32(s_addr + c * 32, r);
+        }
+        tmem_st_wait();
+      } else if (need_mask) {
 #pragma unroll 1
         for (int c = 0; c < BKV / 32; ++c) {
           uint32_t r[32];
@@ -409,7 +438,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       }
       const float m_new = fmaxf(m_run, m_tile);
       const float m_use = (m_new == -INFINITY) ? 0.f : m_new;
-      const float alpha = (m_run == -INFINITY) ? 0.f : exp2f((m_run - m_use) * p.scale_log2);
+      const float alpha = (m_run == -INFINITY) ? 0.f : exp2f((m_run - m_use) * mul);
       // fold the previous tile's P V into the running output (this also means sP is free again)
       if (j > 0) {
         if (!mbar_wait(&o_full, (j - 1) & 1, &cta_abort, p.status)) { ok = false; break; }
@@ -431,7 +460,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         tmem_ld_32x32(s_addr + c * 32, r);
         tmem_ld_wait();
         uint32_t packed[16];
-        const float mneg = -m_use * p.scale_log2;
+        const float mneg = -m_use * mul;
         if (need_mask) {
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
@@ -449,8 +478,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           float l0 = 0.f, l1 = 0.f;
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
-            const float p0 = exp2f(fmaf(__uint_as_float(r[i]), p.scale_log2, mneg));
-            const float p1 = exp2f(fmaf(__uint_as_float(r[i + 1]), p.scale_log2, mneg));
+            const float p0 = exp2f(fmaf(__uint_as_float(r[i]), mul, mneg));
+            const float p1 = exp2f(fmaf(__uint_as_float(r[i + 1]), mul, mneg));
             l0 += p0;
             l1 += p1;
             packed[i >> 1] = pack_bf16x2(p0, p1);
@@ -493,7 +522,25 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       }
     }
     if (ok && qi < p.Sq) {
-      const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
+      if constexpr (FORM) {
+        if (p.form.sink && l_run > 0.f) inv_l = 1.f / (l_run + exp2f(p.form.sink[h] * kLog2e - m_run));
+        if (p.gate.kind != 2) inv_l *= p.gate.factor<__nv_bfloat16>(row0 + qi, h, D, 0);
+        else {
+          const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(p.gate.gate) + static_cast<long long>(row0 + qi) * p.gate.ld + h * D;
+          inv_l *= p.gate.scale;
+#pragma unroll
+          for (int c = 0; c < D / 8; ++c) {
+            const uint4 gv = *reinterpret_cast<const uint4*>(gate + c * 8);
+            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              o_acc[c * 8 + 2 * e] = __fdividef(o_acc[c * 8 + 2 * e], 1.f + __expf(-__low2float(g2[e])));
+              o_acc[c * 8 + 2 * e + 1] = __fdividef(o_acc[c * 8 + 2 * e + 1], 1.f + __expf(-__high2float(g2[e])));
+            }
+          }
+        }
+      }
       __nv_bfloat16* orow = p.o + bb * p.o_sb + static_cast<long long>(row0 + qi) * p.o_ss + h * p.o_sh;
 #pragma unroll
       for (int c = 0; c < D / 8; ++c) {
@@ -558,7 +605,7 @@ TSB_EXPORT int tsb_flash_fwd(const void* q, const void* k, const void* v, void* 
   if (!make_bshd_tmap(&tq, q, B, Sq, H, D, q_sb, q_ss, q_sh, 128)) return -3;
   if (!make_bshd_tmap(&tk, k, B, Sk, Hkv, D, k_sb, k_ss, k_sh, 128)) return -3;
   if (!make_bshd_tmap(&tv, v, B, Sk, Hkv, D, v_sb, v_ss, v_sh, 128)) return -3;
-  FaParams p;
+  FaParams p{};
   p.o = static_cast<__nv_bfloat16*>(o);
   p.lse = lse;
   p.cu_seqlens = p.cu_keys = nullptr;
@@ -598,7 +645,8 @@ TSB_EXPORT int tsb_flash_fwd(const void* q, const void* k, const void* v, void* 
 static int flash_fwd_varlen(const void* q, const void* k, const void* v, void* o, const int* cu_seqlens, const int* cu_keys,
                             int n_seqs, int max_len, int T, int TK, int H, int Hkv, int D, long long q_ss, long long q_sh,
                             long long k_ss, long long k_sh, long long v_ss, long long v_sh, long long o_ss,
-                            long long o_sh, float scale, void* stream) {
+                            long long o_sh, float scale, void* stream, const tsb::AttnForm* form = nullptr,
+                            const tsb::AttnGate* gate = nullptr) {
   using namespace tsb;
   if (n_seqs <= 0 || max_len <= 0 || T <= 0 || TK <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || (D != 64 && D != 128) || !cu_seqlens)
     return -2;
@@ -613,7 +661,7 @@ static int flash_fwd_varlen(const void* q, const void* k, const void* v, void* o
   if (!make_bshd_tmap(&tq, q, 1, T, H, D, big, q_ss, q_sh, 128)) return -3;
   if (!make_bshd_tmap(&tk, k, 1, TK, Hkv, D, big, k_ss, k_sh, 128)) return -3;
   if (!make_bshd_tmap(&tv, v, 1, TK, Hkv, D, big, v_ss, v_sh, 128)) return -3;
-  FaParams p;
+  FaParams p{};
   p.o = static_cast<__nv_bfloat16*>(o);
   p.lse = nullptr;
   p.cu_seqlens = cu_seqlens;
@@ -632,6 +680,13 @@ static int flash_fwd_varlen(const void* q, const void* k, const void* v, void* o
     kern<<<grid, kFaThreads, smem_bytes, s>>>(tq, tk, tv, p);
     return 0;
   };
+  if (form) {
+    p.form = *form;
+    p.gate = *gate;
+    const int rc = D == 128 ? launch(flash_fwd_kernel<128, false, true>, FaCfg<128>::kSmemBytes)
+                            : launch(flash_fwd_kernel<64, false, true>, FaCfg<64>::kSmemBytes);
+    return rc ? rc : static_cast<int>(cudaGetLastError());
+  }
   const int rc = (D == 128) ? launch(flash_fwd_kernel<128, false>, FaCfg<128>::kSmemBytes)
                             : launch(flash_fwd_kernel<64, false>, FaCfg<64>::kSmemBytes);
   if (rc) return rc;
@@ -656,4 +711,20 @@ TSB_EXPORT int tsb_flash_fwd_varlen_keys(const void* q, const void* k, const voi
   if (!cu_keys) return -2;
   return flash_fwd_varlen(q, k, v, o, cu_seqlens, cu_keys, n_seqs, max_len, T, TK, H, Hkv, D, q_ss, q_sh, k_ss, k_sh, v_ss,
                           v_sh, o_ss, o_sh, scale, stream);
+}
+
+// The same with the masks, score forms, gates and row stride of attn_form.cuh: q [T, H, D], k / v rows 2 * Hkv heads apart (a key
+// axis [TK, 2 Hkv, D] of keys and values), o rows `ldo` apart. A chunk mask is the caller's: one "sequence" per chunk.
+TSB_EXPORT int tsb_flash_fwd_shaped(const void* q, const void* k, const void* v, void* o, const int* cu_seqlens, const int* cu_keys,
+                                    int n_seqs, int max_len, int T, int TK, int H, int Hkv, int D, const long long* ints,
+                                    const float* floats, const void* const* ptrs, void* stream) {
+  using namespace tsb;
+  AttnForm f;
+  AttnGate g;
+  if (!cu_keys || !read_attn_form(ints, floats, ptrs, &f, &g)) return -2;
+  if (g.kind == 2 && ((reinterpret_cast<uintptr_t>(g.gate) & 15) || g.ld % 8)) return -2;
+  const bool shaped = !f.plain() || !g.plain();
+  const long long kv = 2ll * Hkv * D;
+  return flash_fwd_varlen(q, k, v, o, cu_seqlens, cu_keys, n_seqs, max_len, T, TK, H, Hkv, D, static_cast<long long>(H) * D, D, kv, D, kv,
+                          D, g.ldo, D, f.scale, stream, shaped ? &f : nullptr, &g);
 }

@@ -129,12 +129,20 @@ __device__ __forceinline__ uint32_t mul_bf16x2(uint32_t a, uint32_t b) {
   return d;
 }
 
+// Several inputs of the same batch rows, stacked `rows` apart in X: result columns from first[i] on read the i-th (tiles do not
+// straddle a start). n = 0: one input.
+struct Inputs {
+  int n = 0, rows = 0;
+  int first[8] = {};
+};
+
 template <int S, bool FP8, int RB>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_decode_wq_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW,
                       const uint8_t* __restrict__ w_packed, const float* __restrict__ w_scale,
                       __nv_bfloat16* __restrict__ Y, int M, int N, int K,
-                      long long ldy, int BN, int scale_cols, int scale_rows, const Layout L, int flags, int* status) {
+                      long long ldy, int BN, int scale_cols, int scale_rows, const Layout L, int flags, const Inputs inputs,
+                      int* status) {
   const int CST = L.c_stages;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -197,6 +205,10 @@ gemm_decode_wq_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_cons
       uint64_t* w_full = FP8 ? full_r : full_c;
       uint64_t* w_empty = FP8 ? empty_r : empty_c;
       uint8_t* w_base = FP8 ? sR : sC;
+      int x_row = m0;
+#pragma unroll
+      for (int i = 1; i < 8; ++i)
+        if (i < inputs.n && n0 >= inputs.first[i]) x_row = m0 + i * inputs.rows;
       const uint32_t w_pitch = static_cast<uint32_t>(FP8 ? L.r_pitch : L.c_pitch);
       int w_issued = 0, ws = 0, x_issued = 0, xs = 0;
       uint32_t wphase = 0, xphase = 0;
@@ -231,7 +243,7 @@ gemm_decode_wq_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_cons
           mbar_expect_tx(&full_x[xs], x_bytes);
 #pragma unroll
           for (int rb = 0; rb < RB; ++rb)
-            tma_load_2d(sX + xs * L.x_pitch + rb * kXBlock, &tmX, &full_x[xs], (kb0 + x_issued) * BK, m0 + rb * BM);
+            tma_load_2d(sX + xs * L.x_pitch + rb * kXBlock, &tmX, &full_x[xs], (kb0 + x_issued) * BK, x_row + rb * BM);
           ++x_issued;
           if (++xs == L.x_stages) {
             xs = 0;
@@ -520,7 +532,7 @@ template <int S, bool FP8, int RB>
 int launch_wq(const CUtensorMap& tx, const CUtensorMap& tw, const void* w_packed, const float* w_scale, void* Y, int M,
               int N, int K,
               long long ldy, int BN, int scale_cols, int scale_rows, const Layout& L, int pdl, int flags,
-              cudaStream_t s) {
+              const Inputs& inputs, cudaStream_t s) {
   flags |= (pdl >> 4) & 1;    // pdl bit 4: measurement aid (stages consumed without multiplying)
   pdl &= 1;
   cudaLaunchConfig_t cfg;
@@ -531,7 +543,7 @@ int launch_wq(const CUtensorMap& tx, const CUtensorMap& tw, const void* w_packed
   return static_cast<int>(cudaLaunchKernelEx(&cfg, gemm_decode_wq_kernel<S, FP8, RB>, tx, tw,
                                              static_cast<const uint8_t*>(w_packed), w_scale,
                                              static_cast<__nv_bfloat16*>(Y), M, N, K, ldy, BN, scale_cols, scale_rows, L,
-                                             flags, device_status_word()));
+                                             flags, inputs, device_status_word()));
 }
 
 // CTAs of this kernel that can be resident at once when launched as clusters of S: a GPC takes whole clusters only,
@@ -705,7 +717,7 @@ TSB_EXPORT int tsb_gemm_decode_wq(const void* X, const void* W, const float* w_s
   const int scale_cols = (K + 127) / 128, scale_rows = (N + 127) / 128;
   const int flags = packed ? 2 : 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-#define TSB_WQ_ARGS tx, tw, W, w_scale, Y, M, N, K, ldy, bn, scale_cols, scale_rows, L, pdl, flags, s
+#define TSB_WQ_ARGS tx, tw, W, w_scale, Y, M, N, K, ldy, bn, scale_cols, scale_rows, L, pdl, flags, Inputs{}, s
 #define TSB_WQ(S_)                                                                            \
   return fp8 ? (rb == 2 ? launch_wq<S_, true, 2>(TSB_WQ_ARGS) : launch_wq<S_, true, 1>(TSB_WQ_ARGS))  \
              : (rb == 2 ? launch_wq<S_, false, 2>(TSB_WQ_ARGS) : launch_wq<S_, false, 1>(TSB_WQ_ARGS))
@@ -732,4 +744,54 @@ TSB_EXPORT int tsb_gemm_decode_wq_plan(int M, int N, int K, int w_fp8, int* bn, 
   if (w_stages) *w_stages = (w_fp8 ? L.r_stages : L.c_stages) * (rb == 2 ? -1 : 1);   // negative: two row blocks per CTA
   if (resident) *resident = resident_ctas_for(*split, w_fp8 != 0);   // what the runtime reports for that cluster size
   return 0;
+}
+
+// Y [M, N] whose column ranges read different inputs: columns [starts[i], starts[i + 1]) are X_i [M, K] * W[N, K]^T, X_i starting
+// i * x_rows rows after X (x_rows >= M). Host array `starts` ascends from 0 in multiples of 128; n <= 8. bf16 weights, otherwise as
+// above.
+TSB_EXPORT int tsb_gemm_decode_inputs(const int* starts, const void* X, const void* W, void* Y, int n, int M, int N, int K, long long x_rows,
+                                      long long ldx, long long ldw, long long ldy, int pdl, void* stream) {
+  using namespace tsb;
+  if (n < 1 || n > 8 || M <= 0 || M > 2 * BM || N <= 0 || K <= 0 || K % 16 || x_rows < M || starts[0] != 0) return -2;
+  if ((reinterpret_cast<uintptr_t>(X) & 15) || (reinterpret_cast<uintptr_t>(W) & 15) || (ldx % 8) || (ldw % 8)) return -2;
+  Inputs in;
+  in.n = n;
+  in.rows = static_cast<int>(x_rows);
+  int unit = 256;
+  for (int i = 0; i < n; ++i) {
+    if (starts[i] % 128 || (i && starts[i] <= starts[i - 1]) || starts[i] >= N) return -2;
+    in.first[i] = starts[i];
+    if (starts[i] % 256) unit = 128;
+  }
+  const int kb = (K + BK - 1) / BK;
+  int bn = 0, split = 1;
+  double best = -1.0;
+  const int rb = M > BM ? 2 : 1;
+  for (int b = unit; b >= 32; b /= 2) {            // widths that divide every start
+    int pb = 0, ps = 0;
+    const double sc = plan_family(M, N, kb, false, b, rb, &pb, &ps);
+    if (sc > best) {
+      best = sc;
+      bn = pb;
+      split = ps;
+    }
+  }
+  if (best < 0.0)                                  // several waves of the widest tile that has room
+    for (bn = unit; bn > 32 && !layout_ok(make_layout(M, bn, false, rb), false, bn, rb);) bn /= 2;
+  const Layout L = make_layout(M, bn, false, rb);
+  if (L.c_stages < 2 || rb * BM * (bn * 4 + 16) > kSmemBudget - 1024) return -2;
+  CUtensorMap tx, tw;
+  if (!make_tmap_2d(&tx, X, 2, (n - 1) * x_rows + M, K, ldx * 2, L.x_rows, BK, true) || !make_tmap_2d(&tw, W, 2, N, K, ldw * 2, bn, BK, true))
+    return -3;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+#define TSB_WQ_IN(S_)                                                                                                   \
+  return rb == 2 ? launch_wq<S_, false, 2>(tx, tw, W, nullptr, Y, M, N, K, ldy, bn, 0, 0, L, pdl, 0, in, s)              \
+                 : launch_wq<S_, false, 1>(tx, tw, W, nullptr, Y, M, N, K, ldy, bn, 0, 0, L, pdl, 0, in, s)
+  switch (split) {
+    case 1: TSB_WQ_IN(1);
+    case 2: TSB_WQ_IN(2);
+    case 4: TSB_WQ_IN(4);
+    default: TSB_WQ_IN(8);
+  }
+#undef TSB_WQ_IN
 }

@@ -58,6 +58,8 @@ __device__ __forceinline__ TileCoord tile_coord(int t, int num_m, int num_n) {
 //           each row came from -- row r with tag t >= 0 is stored at peer_out[t >> 24] + (t & 0xFFFFFF) * ldc (peer-mapped
 //           memory of that rank, over NVLink), rows with a negative tag (padding) are dropped. The all-to-all that
 //           returns expert results is the epilogue of the down projection; nothing is written locally.
+// Without offsets, `inputs` > 0: result columns from col_start[i] on read the i-th of several inputs stacked `a_group_rows` rows apart
+// in A (column tiles do not straddle a start).
 struct GroupArgs {
   const int* offsets;
   int groups;
@@ -67,7 +69,18 @@ struct GroupArgs {
   const int* row_tags = nullptr;
   long long peer_rows = 0;
   void* peer_out[8] = {};
+  int inputs = 0;
+  int a_group_rows = 0;
+  int col_start[8] = {};
 };
+
+__device__ __forceinline__ int input_row_offset(const GroupArgs& g, int col) {
+  int off = 0;
+#pragma unroll
+  for (int i = 1; i < 8; ++i)
+    if (i < g.inputs && col >= g.col_start[i]) off = i * g.a_group_rows;
+  return off;
+}
 
 __device__ __forceinline__ int group_of_row(const GroupArgs& g, int row) {
   int e = 0;
@@ -141,6 +154,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         int kb0 = (t % split_k) * kb_per;
         int kb1 = min(total_kb, kb0 + kb_per);
         int b_row_off = 0;  // rows of the stacked B tensor map before this tile's group
+        const int a_row = m0 + input_row_offset(grp, n0);
         if (gmode == 1) {
           if (m0 >= m_limit) continue;
           b_row_off = static_cast<int>(group_of_row(grp, m0) * grp.b_group_rows);
@@ -157,7 +171,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           uint8_t* sB = sA + Cfg::kStageBytesA;
           mbar_expect_tx(&full_bar[stage], Cfg::kStageBytes);
           if (!A_MN) {
-            tma_load_2d(sA, &tmA, &full_bar[stage], kb * BK, m0);
+            tma_load_2d(sA, &tmA, &full_bar[stage], kb * BK, a_row);
           } else {
 #pragma unroll
             for (int i = 0; i < BM / 64; ++i) tma_load_2d(sA + i * 8192, &tmA, &full_bar[stage], m0 + i * 64, kb * BK);
@@ -613,4 +627,30 @@ TSB_EXPORT int tsb_gemm_bf16_splitk(const void* A, const void* B, float* C32, in
                 : launch_cfg<128, false, false, float, false>(ta, tb, C32, M, N, K, ldc, 0, s, split_k);
   return b_mn ? launch_cfg<64, false, true, float, false>(ta, tb, C32, M, N, K, ldc, 0, s, split_k)
               : launch_cfg<64, false, false, float, false>(ta, tb, C32, M, N, K, ldc, 0, s, split_k);
+}
+
+// C[M, N] (bf16) whose column ranges read different inputs: columns [starts[i], starts[i + 1]) are A_i[M, K] * B[N, K]^T, A_i starting
+// i * a_rows rows after A (a_rows >= M). Host array `starts` ascends from 0 in multiples of 128; n <= 8. Alignment as tsb_gemm_bf16.
+TSB_EXPORT int tsb_gemm_bf16_inputs(const int* starts, const void* A, const void* B, void* C, int n, int M, int N, int K, long long a_rows,
+                                    long long lda, long long ldb, long long ldc, void* stream) {
+  using namespace tsb;
+  if (n < 1 || n > 8 || M <= 0 || N <= 0 || K <= 0 || a_rows < M || starts[0] != 0) return -2;
+  if ((reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15) || (lda % 8) || (ldb % 8)) return -2;
+  GroupArgs g{nullptr, 0, 0, 0, 0};
+  g.inputs = n;
+  g.a_group_rows = static_cast<int>(a_rows);
+  bool wide = true;
+  for (int i = 0; i < n; ++i) {
+    if (starts[i] % 128 || (i && starts[i] <= starts[i - 1]) || starts[i] >= N) return -2;
+    g.col_start[i] = starts[i];
+    wide = wide && starts[i] % 256 == 0;
+  }
+  const long long mt = (M + BM - 1) / BM;
+  const int bn = wide && mt * ((N + 255) / 256) >= sm_count() ? 256 : mt * ((N + 127) / 128) >= sm_count() ? 128 : 64;
+  CUtensorMap ta, tb;
+  if (!cached_tmap_2d(&ta, A, (n - 1) * a_rows + M, K, lda * 2, BM, BK) || !cached_tmap_2d(&tb, B, N, K, ldb * 2, bn, BK)) return -3;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (bn == 256) return launch_cfg<256, false, false, __nv_bfloat16, false>(ta, tb, C, M, N, K, ldc, 0, s, 1, g);
+  if (bn == 128) return launch_cfg<128, false, false, __nv_bfloat16, false>(ta, tb, C, M, N, K, ldc, 0, s, 1, g);
+  return launch_cfg<64, false, false, __nv_bfloat16, false>(ta, tb, C, M, N, K, ldc, 0, s, 1, g);
 }

@@ -1,5 +1,5 @@
-// Paged attention pieces for ragged batches: portions of prompts beside single decoded tokens, with an optional chunk
-// mask (token i sees the tokens j <= i of its own run of `chunk` positions, counted from position 0).
+// Paged attention pieces for ragged batches: portions of prompts beside single decoded tokens, with an optional mask (chunks or
+// a window) and the other score forms of attn_form.cuh.
 //
 //   ragged_append_kernel   adds the projection biases to a packed [q | k | v] row, writes q to a buffer of its own, and
 //                          stores k and v in the pool slot of the token and, for prompt rows, in the contiguous key axis
@@ -7,7 +7,7 @@
 //   stage_gather_kernel    copies keys and values that earlier portions left in the pool to the key axis.
 //   ragged_attn_kernel     attention of each row over the pool: one warp per (row, head), fp32 arithmetic. Serves fp32
 //                          models and head sizes that the tensor-core kernels do not take.
-#include "common.cuh"
+#include "attn_form.cuh"
 
 #include <algorithm>
 
@@ -97,10 +97,11 @@ struct RaggedAttnParams {
   const int* tables;      // [sequences, table_ld]
   const int* seq_of;      // [rows] (null: row i is sequence i)
   const int* pos;         // [rows], < 0: no keys (padding)
-  void* o;                // [rows, H, D]
+  void* o;                // [rows, gate.ldo], head h at h * D
   long long ld_q;
-  int rows, H, Hkv, bs, nb, table_ld, chunk;
-  float scale;
+  int rows, H, Hkv, bs, nb, table_ld;
+  AttnForm form;
+  AttnGate gate;
   int* status;
 };
 
@@ -125,7 +126,8 @@ ragged_attn_kernel(RaggedAttnParams p) {
     o[i] = 0.f;
   }
   const int pos = p.pos[row];
-  int t = p.chunk > 0 && pos >= 0 ? pos / p.chunk * p.chunk : 0;
+  int t = pos >= 0 ? p.form.first(pos) : 0;
+  const float slope = p.form.slopes ? p.form.slopes[h] : 0.f;
   float m = -INFINITY, l = 0.f;
   for (; t <= pos; t += 4) {
     float s[4];
@@ -144,7 +146,11 @@ ragged_attn_kernel(RaggedAttnParams p) {
       for (int i = 0; i < EPL; ++i) s[j] = fmaf(q[i], to_f32<T>(static_cast<const T*>(p.k_pool)[base[j] + lane + 32 * i]), s[j]);
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) s[j] = t + j <= pos ? warp_sum(s[j]) * p.scale : -INFINITY;
+    for (int j = 0; j < 4; ++j) {
+      float f = warp_sum(s[j]) * p.form.scale;
+      if (p.form.softcap > 0.f) f = p.form.softcap * tanhf(f / p.form.softcap);
+      s[j] = t + j <= pos ? fmaf(-slope, static_cast<float>(pos - t - j), f) : -INFINITY;
+    }
     const float mn = fmaxf(fmaxf(fmaxf(s[0], s[1]), fmaxf(s[2], s[3])), m);
     const float corr = m == -INFINITY ? 0.f : expf(m - mn);
     l *= corr;
@@ -159,10 +165,11 @@ ragged_attn_kernel(RaggedAttnParams p) {
     }
     m = mn;
   }
+  if (p.form.sink && l > 0.f) l += expf(p.form.sink[h] - m);      // (an overflow leaves nothing of the keys, as it should)
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  T* orow = static_cast<T*>(p.o) + (static_cast<long long>(row) * p.H + h) * D;
+  T* orow = static_cast<T*>(p.o) + row * p.gate.ldo + h * D;
 #pragma unroll
-  for (int i = 0; i < EPL; ++i) orow[lane + 32 * i] = from_f32<T>(o[i] * inv);
+  for (int i = 0; i < EPL; ++i) orow[lane + 32 * i] = from_f32<T>(o[i] * inv * p.gate.factor<T>(row, h, D, lane + 32 * i));
 }
 
 template <typename T>
@@ -219,15 +226,16 @@ TSB_EXPORT int tsb_stage_gather(const void* k_pool, const void* v_pool, void* st
   return static_cast<int>(cudaGetLastError());
 }
 
-// o[row, h, :] = attention of row's query over positions [pos / chunk * chunk, pos] of its sequence (chunk 0: from 0) in
-// the pool, the row's own key included. D is a multiple of 32, up to 256.
+// o[row, h, :] = attention of row's query over the positions it sees of its sequence in the pool, the row's own key included.
+// D is a multiple of 32, up to 256. ints, floats, ptrs: see attn_form.cuh.
 TSB_EXPORT int tsb_ragged_attn(const void* q, long long ld_q, const void* k_pool, const void* v_pool, const int* tables,
                                int table_ld, const int* seq_of, const int* pos, void* o, int rows, int H, int Hkv, int D, int bs,
-                               int nb, int chunk, float scale, int dtype, void* stream) {
+                               int nb, const long long* ints, const float* floats, const void* const* ptrs, int dtype, void* stream) {
   using namespace tsb;
-  if (rows <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || D <= 0 || D % 32 || D > 256 || bs <= 0 || nb <= 0 || chunk < 0) return -2;
-  RaggedAttnParams p{q, k_pool, v_pool, tables, seq_of, pos, o, ld_q, rows, H, Hkv, bs, nb, table_ld, chunk, scale,
-                     device_status_word()};
+  RaggedAttnParams p{q, k_pool, v_pool, tables, seq_of, pos, o, ld_q, rows, H, Hkv, bs, nb, table_ld, {}, {}, device_status_word()};
+  if (rows <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || D <= 0 || D % 32 || D > 256 || bs <= 0 || nb <= 0 ||
+      !read_attn_form(ints, floats, ptrs, &p.form, &p.gate))
+    return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (dtype == 1) return launch_ragged_attn<__nv_bfloat16>(p, D, s);
   if (dtype == 0) return launch_ragged_attn<float>(p, D, s);

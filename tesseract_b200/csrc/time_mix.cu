@@ -1,0 +1,321 @@
+// Time mixing (linear attention with a decay per key channel and token and a bonus for the current token), for ragged batches:
+//
+//   o_t = (S_(t-1) + v_t (u k_t)^T) r_t,  S_t = diag(w_t) S_(t-1) + v_t k_t^T,  w = exp(-exp(d + w0))      per head
+//   out = o / rms(o) * norm * silu(gate)
+//
+// S is [values][keys] in fp32 and stays so. token_shift_kernel makes the inputs of the five projections, mixes of a row and the
+// one before it.
+#include "linear_state.cuh"
+#include "ragged_conv.cuh"
+
+#include <algorithm>
+
+namespace tsb {
+namespace {
+
+// ------------------------------------------------------------------ mixes of a row and the one before it
+struct ShiftParams {
+  const void* h;
+  long long ldh;
+  const float* mu;          // [n, C]
+  void* last;               // [slots, C]
+  void* xs;                 // [n (+ 1), rows, ldx]
+  long long stream, ldx;
+  const int* positions;     // [rows]
+  const int* seq_of;        // [rows]
+  const int* slots;         // [sequences]
+  const int* cu;            // [prompts + 1] rows relative to n_decode
+  const int* pos0;          // [prompts]
+  int n_decode, rows, C, n, keep;
+};
+
+// A thread takes one 16-byte column of kRows rows in a row (the mix factors stay in registers).
+template <typename T, int N, int kRows>
+__global__ void __launch_bounds__(128)
+token_shift_kernel(ShiftParams p) {
+  pdl_trigger();
+  pdl_grid_wait();
+  constexpr int V = kVec16<T>;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V;
+  if (c >= p.C) return;
+  float mu[N][V];
+#pragma unroll
+  for (int s = 0; s < N; ++s)
+#pragma unroll
+    for (int i = 0; i < V; ++i) mu[s][i] = p.mu[s * p.C + c + i];
+  const T* h = static_cast<const T*>(p.h) + c;
+  T* last = static_cast<T*>(p.last) + c;
+  T* xs = static_cast<T*>(p.xs) + c;
+  float prev[V];
+  bool have = false;
+  for (int r = 0; r < kRows; ++r) {
+    const int row = blockIdx.y * kRows + r;
+    if (row >= p.rows) return;
+    float x[V];
+    ld16<T>(h + row * p.ldh, x);
+    const int seq = p.seq_of[row], slot = p.slots[seq];
+    bool start = true, old = false;              // the sequence's first row of this step; there is an earlier token
+    if (row < p.n_decode) {
+      old = p.positions[row] > 0;
+    } else {
+      start = row == p.n_decode + p.cu[seq - p.n_decode];
+      old = p.pos0[seq - p.n_decode] > 0;
+    }
+    if (start) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) prev[i] = 0.f;
+      if (old && slot >= 0) ld16<T>(last + static_cast<long long>(slot) * p.C, prev);
+    } else if (!have) {
+      ld16<T>(h + (row - 1) * p.ldh, prev);
+    }
+    T* out = xs + row * p.ldx;
+    if (p.keep) {
+      st16<T>(out, x);
+      out += p.stream;
+    }
+#pragma unroll
+    for (int s = 0; s < N; ++s) {
+      float y[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[i] = fmaf(prev[i] - x[i], mu[s][i], x[i]);
+      st16<T>(out + s * p.stream, y);
+    }
+    if (row < p.n_decode && slot >= 0) st16<T>(last + static_cast<long long>(slot) * p.C, x);
+#pragma unroll
+    for (int i = 0; i < V; ++i) prev[i] = x[i];
+    have = true;
+  }
+}
+
+// ------------------------------------------------------------------ the recurrence
+struct MixParams {
+  int H, dim, dp, rp, section, rows, n_seq, ld, ldo;
+  const void* proj;          // [rows, ld]: r, k, v, gate `section` columns apart, then the decay's inputs
+  const float* dec;          // [rows, H * dp] (prompts)
+  const void* w2;            // [H * dp, rp] (decoded rows)
+  const float* w0;           // [H * dp]
+  const float* u;
+  const float* norm;
+  float* state;              // [slots, H, dp, dp]
+  const int* slots;
+  const int* positions;      // decoded rows
+  const int* cu;             // prompts
+  const int* pos0;
+  void* out;                 // [rows, ldo]
+  float* o;                  // [rows, H, dp] read-outs of the scan
+  float eps, out_scale;
+};
+
+template <typename T, int RL>
+__global__ void __launch_bounds__(128)
+time_mix_scan_kernel(MixParams p) {
+  pdl_trigger();
+  pdl_grid_wait();
+  __shared__ float sm[ScanShape<RL>::kFloats];
+  const int h = blockIdx.y, seq = blockIdx.z, slot = p.slots[seq];
+  const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
+  if (slot < 0 || n <= 0) return;
+  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ld + h * p.dp;
+  const float* dec = p.dec + static_cast<long long>(row0) * p.H * p.dp + h * p.dp;
+  const float* w0 = p.w0 + h * p.dp;
+  float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp;
+  float* o = p.o + static_cast<long long>(row0) * p.H * p.dp + h * p.dp;
+  state_scan<RL, false>(
+      sm, st, p.dp, p.dp, p.pos0[seq] == 0, n, blockIdx.x * kScanRows,
+      [&](int t, int d, float& q, float& k, float& w) {
+        const T* r = x + static_cast<long long>(t) * p.ld + d;
+        q = to_f32<T>(r[0]);
+        k = to_f32<T>(r[p.section]);
+        w = expf(-expf(dec[static_cast<long long>(t) * p.H * p.dp + d] + w0[d]));
+      },
+      [&](int t, int e) { return to_f32<T>(x[static_cast<long long>(t) * p.ld + 2 * p.section + e]); },
+      [&](int t, int e, const float (&f)[4]) {
+        *reinterpret_cast<float4*>(o + static_cast<long long>(t) * p.H * p.dp + e) = make_float4(f[0], f[1], f[2], f[3]);
+      });
+}
+
+// out = (o + v (u k . r)) / rms * norm * silu(gate): one warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(256)
+time_mix_norm_kernel(MixParams p) {
+  pdl_trigger();
+  pdl_grid_wait();
+  const long long w = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (w >= static_cast<long long>(p.rows) * p.H) return;
+  const long long row = w / p.H;
+  const int h = static_cast<int>(w % p.H);
+  const T* x = static_cast<const T*>(p.proj) + row * p.ld + h * p.dp;
+  const float *o = p.o + w * p.dp, *u = p.u + h * p.dp, *norm = p.norm + h * p.dp;
+  T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.dp;
+  float bonus = 0.f, ss = 0.f;
+  for (int d = lane; d < p.dp; d += 32) bonus = fmaf(u[d] * to_f32<T>(x[p.section + d]), to_f32<T>(x[d]), bonus);
+  bonus = warp_sum(bonus);
+  for (int d = lane; d < p.dp; d += 32) {
+    const float f = fmaf(to_f32<T>(x[2 * p.section + d]), bonus, o[d]);
+    ss = fmaf(f, f, ss);
+  }
+  const float r = p.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(p.dim) + p.eps);
+  for (int d = lane; d < p.dp; d += 32) {
+    const float f = fmaf(to_f32<T>(x[2 * p.section + d]), bonus, o[d]);
+    out[d] = from_f32<T>(f * r * norm[d] * silu_f32(to_f32<T>(x[3 * p.section + d])));
+  }
+}
+
+// Decoded rows: CTA = (row, head).
+template <typename T, int LPR, int PPL, int RPT>
+__global__ void __launch_bounds__(256)
+time_mix_step_kernel(MixParams p) {
+  pdl_trigger();
+  pdl_grid_wait();
+  extern __shared__ __align__(16) float sm[];
+  float *sq = sm, *sk = sq + p.dp, *sv = sk + p.dp, *sw = sv + p.dp, *so = sw + p.dp, *th = so + p.dp, *red = th + p.rp;
+  const int row = blockIdx.x, h = blockIdx.y, slot = p.slots[row];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(row) * p.ld + h * p.dp;
+  T* out = static_cast<T*>(p.out) + static_cast<long long>(row) * p.ldo + h * p.dp;
+  if (slot < 0) {
+    for (int d = tid; d < p.dp; d += 256) out[d] = from_f32<T>(0.f);
+    return;
+  }
+  float bonus = 0.f;
+  for (int d = tid; d < p.dp; d += 256) {
+    sq[d] = to_f32<T>(x[d]);
+    sk[d] = to_f32<T>(x[p.section + d]);
+    sv[d] = to_f32<T>(x[2 * p.section + d]);
+    bonus = fmaf(p.u[h * p.dp + d] * sk[d], sq[d], bonus);
+  }
+  const T* wl = static_cast<const T*>(p.proj) + static_cast<long long>(row) * p.ld + 4 * p.section;
+  for (int j = tid; j < p.rp; j += 256) th[j] = to_f32<T>(from_f32<T>(tanhf(to_f32<T>(wl[j]))));
+  bonus = warp_sum(bonus);
+  if (lane == 0) red[warp] = bonus;
+  __syncthreads();
+  const T* w2 = static_cast<const T*>(p.w2) + static_cast<long long>(h) * p.dp * p.rp;
+  for (int d = warp; d < p.dp; d += 8) {
+    float a = 0.f;
+    for (int j = lane; j < p.rp; j += 32) a = fmaf(to_f32<T>(w2[static_cast<long long>(d) * p.rp + j]), th[j], a);
+    a = warp_sum(a);
+    if (lane == 0) sw[d] = expf(-expf(a + p.w0[h * p.dp + d]));
+  }
+  bonus = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) bonus += red[w];
+  __syncthreads();
+  state_step<LPR, PPL, RPT, false>(p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp, p.dp, p.dp, p.positions[row] <= 0, sq, sk,
+                                   sw, sv, so);
+  __syncthreads();
+  float ss = 0.f;
+  for (int d = tid; d < p.dp; d += 256) {
+    const float f = fmaf(sv[d], bonus, so[d]);
+    ss = fmaf(f, f, ss);
+  }
+  ss = warp_sum(ss);
+  if (lane == 0) red[warp] = ss;
+  __syncthreads();
+  ss = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) ss += red[w];
+  const float r = p.out_scale / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
+  for (int d = tid; d < p.dp; d += 256)
+    out[d] = from_f32<T>(fmaf(sv[d], bonus, so[d]) * r * p.norm[h * p.dp + d] * silu_f32(to_f32<T>(x[3 * p.section + d])));
+}
+
+template <typename T>
+int run_scan(const MixParams& p, cudaStream_t s) {
+  const dim3 grid((p.dp + kScanRows - 1) / kScanRows, p.H, p.n_seq);
+  const bool pdl = pdl_all_enabled();
+  if (p.dp <= 64) launch_pdl(time_mix_scan_kernel<T, 2>, grid, dim3(128), 0, s, pdl, p);
+  else if (p.dp <= 128) launch_pdl(time_mix_scan_kernel<T, 4>, grid, dim3(128), 0, s, pdl, p);
+  else launch_pdl(time_mix_scan_kernel<T, 8>, grid, dim3(128), 0, s, pdl, p);
+  const long long warps = static_cast<long long>(p.rows) * p.H;
+  launch_pdl(time_mix_norm_kernel<T>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, s, pdl, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int run_step(const MixParams& p, cudaStream_t s) {
+  const int smem = (5 * p.dp + p.rp + 8) * 4;
+  if (smem > 48 * 1024) return -2;
+  const dim3 grid(p.rows, p.H);
+  const bool pdl = pdl_all_enabled();
+  if (p.dp <= 32) launch_pdl(time_mix_step_kernel<T, 8, 1, 1>, grid, dim3(256), smem, s, pdl, p);
+  else if (p.dp <= 64) launch_pdl(time_mix_step_kernel<T, 16, 1, 4>, grid, dim3(256), smem, s, pdl, p);
+  else if (p.dp <= 128) launch_pdl(time_mix_step_kernel<T, 32, 1, 16>, grid, dim3(256), smem, s, pdl, p);
+  else launch_pdl(time_mix_step_kernel<T, 32, 2, 8>, grid, dim3(256), smem, s, pdl, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+bool read_mix(const int* v, MixParams* p) {
+  p->H = v[0]; p->dim = v[1]; p->dp = v[2]; p->rp = v[3]; p->section = v[4]; p->rows = v[5]; p->n_seq = v[6]; p->ld = v[7]; p->ldo = v[8];
+  return p->H > 0 && p->H <= 65535 && p->dim > 0 && p->dp >= p->dim && p->dp % 16 == 0 && p->dp <= 256 && p->rp > 0 && p->rp % 16 == 0 &&
+         p->section >= p->H * p->dp && p->section % 8 == 0 && p->rows > 0 && p->ld % 8 == 0 && p->n_seq > 0 && p->n_seq <= 65535;
+}
+
+template <typename T, int N>
+void launch_shift(const ShiftParams& p, cudaStream_t s) {
+  const int cols = (p.C / kVec16<T> + 127) / 128;
+  if (p.rows <= 512) launch_pdl(token_shift_kernel<T, N, 1>, dim3(cols, p.rows), dim3(128), 0, s, pdl_all_enabled(), p);
+  else launch_pdl(token_shift_kernel<T, N, 8>, dim3(cols, (p.rows + 7) / 8), dim3(128), 0, s, pdl_all_enabled(), p);
+}
+
+template <typename T>
+int run_shift(const ShiftParams& p, int n_prompts, cudaStream_t s) {
+  switch (p.n) {
+    case 1: launch_shift<T, 1>(p, s); break;
+    case 5: launch_shift<T, 5>(p, s); break;
+    default: return -2;
+  }
+  if (n_prompts > 0)       // a portion's last row: behind the reads of the one before it
+    launch_pdl(conv_state_kernel<T>, dim3((p.C + 255) / 256, n_prompts), dim3(256), 0, s, pdl_all_enabled(),
+               static_cast<const T*>(p.h) + p.n_decode * p.ldh, p.ldh, p.C, static_cast<T*>(p.last), p.cu, p.slots + p.n_decode, p.pos0, 1);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace
+}  // namespace tsb
+
+// See ShiftParams. Rows below n_decode are single tokens, the others portions. C is a multiple of 8; n is 1 or 5.
+TSB_EXPORT int tsb_token_shift(const void* h, long long ldh, const float* mu, void* last, void* xs, long long stream_elems, long long ldx,
+                               const int* positions, const int* seq_of, const int* slots, const int* cu, const int* pos0, int n_decode, int rows,
+                               int C, int n, int keep, int n_prompts, int dtype, void* stream) {
+  using namespace tsb;
+  if (rows <= 0 || C <= 0 || C % 8 || ldh % 8 || ldx % 8 || stream_elems % 8 || n_prompts < 0 || n_prompts > 65535 || n_decode < 0 ||
+      n_decode > rows || (rows > n_decode && (!cu || !pos0 || n_prompts == 0)))
+    return -2;
+  ShiftParams p{h, ldh, mu, last, xs, stream_elems, ldx, positions, seq_of, slots, cu, pos0, n_decode, rows, C, n, keep};
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == 1) return run_shift<__nv_bfloat16>(p, n_prompts, s);
+  if (dtype == 0) return run_shift<float>(p, n_prompts, s);
+  return -2;
+}
+
+// ints: H, dim, dp, rp, section, rows, sequences, projection row stride, result row stride. ptrs: proj, w2, w0, u, norm, state,
+// slots, positions, out. Row i is the next token of the sequence in slot slots[i] (-1: padding, out = 0).
+TSB_EXPORT int tsb_time_mix_step(const int* ints, void* const* q, float eps, float out_scale, int dtype, void* stream) {
+  using namespace tsb;
+  MixParams p{};
+  if (!read_mix(ints, &p)) return -2;
+  p.proj = q[0]; p.w2 = q[1]; p.w0 = static_cast<const float*>(q[2]); p.u = static_cast<const float*>(q[3]);
+  p.norm = static_cast<const float*>(q[4]); p.state = static_cast<float*>(q[5]); p.slots = static_cast<const int*>(q[6]);
+  p.positions = static_cast<const int*>(q[7]); p.out = q[8]; p.eps = eps; p.out_scale = out_scale;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == 1) return run_step<__nv_bfloat16>(p, s);
+  if (dtype == 0) return run_step<float>(p, s);
+  return -2;
+}
+
+// ptrs: proj, dec, w0, u, norm, state, slots, cu, pos0, out, o ([rows, H, dp] fp32).
+TSB_EXPORT int tsb_time_mix_prefill(const int* ints, void* const* q, float eps, float out_scale, int dtype, void* stream) {
+  using namespace tsb;
+  MixParams p{};
+  if (!read_mix(ints, &p)) return -2;
+  p.proj = q[0]; p.dec = static_cast<const float*>(q[1]); p.w0 = static_cast<const float*>(q[2]); p.u = static_cast<const float*>(q[3]);
+  p.norm = static_cast<const float*>(q[4]); p.state = static_cast<float*>(q[5]); p.slots = static_cast<const int*>(q[6]);
+  p.cu = static_cast<const int*>(q[7]); p.pos0 = static_cast<const int*>(q[8]); p.out = q[9]; p.o = static_cast<float*>(q[10]);
+  p.eps = eps; p.out_scale = out_scale;
+  if (!p.o) return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == 1) return run_scan<__nv_bfloat16>(p, s);
+  if (dtype == 0) return run_scan<float>(p, s);
+  return -2;
+}

@@ -1,12 +1,14 @@
 """Decoders that mix recurrent and attention layers, described by a list: every layer has a mixer and, optionally, a
-feed-forward. Two forms of layer:
+feed-forward. Three forms of layer:
 
 * ``sandwich``: mixer, then feed-forward, each normed before and after by Dynamic Tanh; a range of layers may run several
   times in a row with the same weights and separate caches ("loop");
 * ``parallel``: mixer and feed-forward of the same x side by side, x + m (mixer(norm1 x) + ff(norm2 x)), normed by RMS with one
   gain. The gains ride on the sublayers (``in_scale``), so one normed row feeds one product for both, and one product takes
   both results back. Optionally every layer hands on a weighted sum of the embedding output and all layers' results so far
-  ("depth average").
+  ("depth average");
+* ``post``: mixer, then feed-forward, which read x itself; their results are normed by RMS (gains stored around zero) and added.
+  Optionally every layer then adds a normed side input that depends on the token ("token side").
 
 Embedding and output share one table, or the output has its own.
 
@@ -22,9 +24,11 @@ from typing import Callable, Dict, List, Optional, Union
 import torch
 
 from .. import ops
-from ..nn.hybrid import (RGLRU, ChunkedAttention, ClampedGLU, DynamicTanh, GatedDelta, LatentAttention, Retention, ScalarRMSNorm,
-                         SiluGLU, pad_to)
+from ..nn.hybrid import (RGLRU, SSD, ChunkedAttention, ClampedGLU, DynamicTanh, GatedDelta, LatentAttention, Retention, RMSNorm,
+                         ScalarRMSNorm, ShapedAttention, SideBySide, SiluGLU, TimeMix, TokenSide, pad_to)
 from ..nn.ragged import HybridCache, HybridSequence, RaggedBatch
+from ..ops.masks import Window
+from ..ops.ragged import ScoreForm
 from ..ops.rotary import Rotary, Yarn
 from .llama import GenerateConfig, pick_next_token
 
@@ -76,6 +80,54 @@ class RGLRUSpec:
 
 
 @dataclass(frozen=True)
+class ShapedAttentionSpec:
+    """Attention with chosen parts. ``window`` 0: causal; ``norm`` of q and k: "", "unit" (per head), "head" (per head with a
+    weight), "whole" (all heads at once with a weight); ``distance_bias``: 2^(-8 (h + 1) / heads) per position; ``sink``: "",
+    "learned", "one" (1 more in the denominator); ``gate``: "", "head", "element"; ``v_mix``: values mixed with those of the model's
+    first such layer."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0
+    bias: bool = False
+    keys_as_values: bool = False
+    norm: str = ""
+    rotary: Optional[Rotary] = None
+    softcap: float = 0.0
+    distance_bias: bool = False
+    sink: str = ""
+    gate: str = ""
+    v_mix: bool = False
+
+
+@dataclass(frozen=True)
+class TimeMixSpec:
+    heads: int
+    dim: int
+    rank: int
+
+
+@dataclass(frozen=True)
+class SSDSpec:
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_parts: int = 1
+
+
+@dataclass(frozen=True)
+class SideBySideSpec:
+    left: object
+    right: object
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+@dataclass(frozen=True)
 class GLUSpec:
     ff: int
     limit: float
@@ -88,7 +140,7 @@ class SiluGLUSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, DeltaSpec, LatentSpec, RetentionSpec, RGLRUSpec]
+    mixer: Union[AttentionSpec, DeltaSpec, LatentSpec, RetentionSpec, RGLRUSpec, ShapedAttentionSpec, TimeMixSpec, SSDSpec, SideBySideSpec]
     mlp: Union[GLUSpec, SiluGLUSpec, None] = None
 
 
@@ -112,10 +164,11 @@ class HybridConfig:
     eos_token_id: int = -1
     max_position_embeddings: int = 1 << 20     # a bound for caches only
     architecture: str = ""
-    form: str = "sandwich"                     # or "parallel"
+    form: str = "sandwich"                     # or "parallel" or "post"
     residual_mult: float = 1.0                 # (parallel)
     depth_average: bool = False                # (parallel)
     tied: bool = True                          # the output product uses the embedding table
+    token_side: int = 0                        # (post) columns of the side table per layer, 0: no side input
 
     def __post_init__(self):
         if self.vocab_size < 1 or self.width < 1 or not self.layers:
@@ -125,11 +178,15 @@ class HybridConfig:
             raise ValueError("HybridConfig: loop must name a range of layers and run at least once")
         if self.dtype not in (torch.bfloat16, torch.float32):
             raise ValueError("HybridConfig: dtype is bfloat16 or float32")
-        if self.form not in ("sandwich", "parallel"):
+        if self.form not in ("sandwich", "parallel", "post"):
             raise ValueError(f"HybridConfig: unknown form {self.form!r}")
+        if self.form == "post" and lp is not None:
+            raise ValueError("HybridConfig: post-normed layers take no loop")
+        if self.form != "post" and self.token_side or self.token_side < 0:
+            raise ValueError("HybridConfig: a side input per token belongs to post-normed layers")
         if self.form == "parallel" and (lp is not None or self.embedding_scale != 1.0):
             raise ValueError("HybridConfig: parallel layers take no loop and no embedding scale")
-        if self.form == "sandwich" and (self.residual_mult != 1.0 or self.depth_average):
+        if self.form != "parallel" and (self.residual_mult != 1.0 or self.depth_average):
             raise ValueError("HybridConfig: a residual multiplier and depth averaging belong to parallel layers")
 
     def runs(self):
@@ -142,8 +199,26 @@ class HybridConfig:
                 + [(i, -1) for i in range(lp.stop, n)])
 
 
+def mixers_of(m) -> list:
+    """A mixer's spec, or those of its parts."""
+    return mixers_of(m.left) + mixers_of(m.right) if isinstance(m, SideBySideSpec) else [m]
+
+
 def _make_mixer(m, c: HybridConfig, device):
     W, dt = c.width, c.dtype
+    if isinstance(m, SideBySideSpec):
+        return SideBySide(_make_mixer(m.left, c, device), _make_mixer(m.right, c, device), m.left_scale, m.right_scale, W, dt, device)
+    if isinstance(m, ShapedAttentionSpec):
+        if m.sink not in ("", "learned", "one"):
+            raise ValueError(f"attention: unknown sink {m.sink!r}")
+        slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / m.heads) for h in range(m.heads)]) if m.distance_bias else None
+        form = ScoreForm(m.scale, Window(m.window) if m.window else 0, m.softcap, slopes, torch.zeros(m.heads) if m.sink == "one" else None)
+        return ShapedAttention(W, m.heads, m.kv_heads, m.dim, m.vdim, form, c.eps, dt, device, m.bias, m.keys_as_values, m.norm, m.rotary,
+                               m.sink == "learned", m.v_mix, m.gate)
+    if isinstance(m, TimeMixSpec):
+        return TimeMix(W, m.heads, m.dim, m.rank, c.eps, dt, device)
+    if isinstance(m, SSDSpec):
+        return SSD(W, m.heads, m.vdim, m.state, m.groups, m.conv, m.norm_parts, c.eps, dt, device)
     if isinstance(m, AttentionSpec):
         return ChunkedAttention(W, m.heads, m.kv_heads, m.dim, m.vdim, m.scale, m.chunk, dt, device)
     if isinstance(m, DeltaSpec):
@@ -226,6 +301,30 @@ class _ParallelLayer:
         return ops.project(z, self.w_out)
 
 
+class _PostLayer:
+    def __init__(self, spec: LayerSpec, c: HybridConfig, index: int, device):
+        norm = lambda: RMSNorm(c.width, c.eps, 1.0, c.dtype, device)   # noqa: E731
+        self.mixer, self.mlp = _make_mixer(spec.mixer, c, device), _make_mlp(spec.mlp, c, device)
+        self.norm1, self.norm2 = norm(), norm() if spec.mlp is not None else None
+        self.side = TokenSide(c.width, c.token_side, c.eps, c.dtype, device) if c.token_side else None
+        for s in (self.mixer, self.mlp):
+            if s is not None and s.out_bias is not None:
+                raise ValueError(f"HybridConfig: {type(s).__name__} does not run in post-normed layers")
+
+    def parts(self):
+        out = [("norm1", self.norm1), ("mix.", self.mixer)]
+        if self.mlp is not None:
+            out += [("norm2", self.norm2), ("mlp.", self.mlp)]
+        if self.side is not None:
+            out.append(("side.", self.side))
+        return out
+
+    extra = {}
+
+
+_LAYERS = {"sandwich": _SandwichLayer, "parallel": _ParallelLayer, "post": _PostLayer}
+
+
 class HybridModel:
     def __init__(self, config: HybridConfig, device=None, init_std: Optional[float] = None, seed: int = 0):
         self.config = c = config
@@ -234,17 +333,21 @@ class HybridModel:
         # GEMMs read
         self.embed = torch.zeros(c.vocab_size, pad_to(c.width), dtype=c.dtype, device=self.device)
         self.head = self.embed if c.tied else torch.zeros_like(self.embed)
-        layer = _SandwichLayer if c.form == "sandwich" else _ParallelLayer
-        self.layers = [layer(s, c, i, self.device) for i, s in enumerate(c.layers)]
-        self.final_norm = (DynamicTanh(c.width, c.dtype, self.device) if c.form == "sandwich"
-                           else ScalarRMSNorm(c.eps, c.dtype, self.device))
+        values = {(m.kv_heads, m.vdim) for l in c.layers for m in mixers_of(l.mixer) if getattr(m, "v_mix", False)}
+        if len(values) > 1:
+            raise ValueError("HybridConfig: layers that mix values have the same value heads")
+        self.layers = [_LAYERS[c.form](s, c, i, self.device) for i, s in enumerate(c.layers)]
+        final = {"sandwich": lambda: DynamicTanh(c.width, c.dtype, self.device), "parallel": lambda: ScalarRMSNorm(c.eps, c.dtype, self.device),
+                 "post": lambda: RMSNorm(c.width, c.eps, 1.0, c.dtype, self.device)}
+        self.final_norm = final[c.form]()
+        self.side_table = (torch.zeros(c.vocab_size, c.token_side * len(c.layers), dtype=c.dtype, device=self.device)
+                           if c.token_side else None)
         self.loop_step = (torch.zeros(c.loop.times, c.width, dtype=torch.float32, device=self.device)
                           if c.loop is not None else None)
         self.runs = c.runs()
         # what the mixers ask a batch for: masks of prompt attention, sizes of prompt tiles
-        self.chunks = sorted({s.mixer.chunk if isinstance(s.mixer, AttentionSpec) else 0
-                              for s in c.layers if isinstance(s.mixer, (AttentionSpec, LatentSpec))})
-        self.tiles = sorted({l.mixer.tile for l in self.layers if l.mixer.tile})
+        self.masks = list(dict.fromkeys(m for l in self.layers for m in l.mixer.masks))
+        self.tiles = sorted({t for l in self.layers for t in l.mixer.tiles})
         if init_std is not None:
             self.init_weights(init_std, seed)
 
@@ -280,6 +383,8 @@ class HybridModel:
         yield "embed", self.embed
         if not self.config.tied:
             yield "head", self.head
+        if self.side_table is not None:
+            yield "side.embed", self.side_table
         if self.loop_step is not None:
             yield "loop.step", self.loop_step
         for i, l in enumerate(self.layers):
@@ -287,7 +392,7 @@ class HybridModel:
                 yield f"l{i}.{name}", t
 
     def _logical(self, t: torch.Tensor) -> torch.Tensor:
-        return t[:, :self.config.width] if t.dim() == 2 else t
+        return t[:, :self.config.width] if t.dim() == 2 and t is not self.side_table else t
 
     def logical_shapes(self) -> Dict[str, tuple]:
         out = {name: tuple(self._logical(t).shape) for name, t in self._tables()}
@@ -336,11 +441,22 @@ class HybridModel:
         passes the newest result on."""
         gen = torch.Generator(device=self.device)
         gen.manual_seed(seed)
+        around_zero = {f"l{i}.{n}" for i in range(len(self.layers)) for n in ("norm1", "norm2")} | {"final.norm"}
 
         def draw(name, shape):
             last = name.rsplit(".", 1)[-1]
+            if self.config.form == "post" and name in around_zero or last == "sink":
+                return torch.zeros(shape)
+            if last == "vmix":
+                return torch.tensor(0.5)
             if last == "alpha" or shape == ():
                 return torch.tensor(1.0)
+            if ".mu." in name:
+                return torch.rand(shape, generator=gen, device=self.device)
+            if last == "w0":
+                return torch.rand(shape, generator=gen, device=self.device) * 5.0 - 6.0
+            if last == "u":
+                return torch.rand(shape, generator=gen, device=self.device)
             if last == "dwa":
                 return torch.eye(shape[0])[-1]
             if len(shape) == 3:
@@ -366,13 +482,13 @@ class HybridModel:
         return HybridCache(specs, num_blocks, block_size, max_sequences, max_len, self.config.dtype, self.device)
 
     def make_batch(self, cache: HybridCache, entries, want=None, max_len: int = 0) -> RaggedBatch:
-        return RaggedBatch(cache, entries, want, self.chunks, max_len, self.tiles)
+        return RaggedBatch(cache, entries, want, self.masks, max_len, self.tiles)
 
     @torch.no_grad()
     def forward_ragged(self, batch, cache: HybridCache, on_layer: Optional[Callable] = None) -> Optional[torch.Tensor]:
         """Runs one step over the cache; fp32 logits [wanted rows, vocab] (None when nothing is wanted). ``on_layer`` is
         called with (run, residual) after every layer run, before what comes ahead of the next pass."""
-        run = self._run_sandwich if self.config.form == "sandwich" else self._run_parallel
+        run = {"sandwich": self._run_sandwich, "parallel": self._run_parallel, "post": self._run_post}[self.config.form]
         h = run(batch, cache, on_layer)
         if batch.n_want == 0:
             return None
@@ -430,6 +546,26 @@ class HybridModel:
             last = r == n - 1
             x, h = ops.depth_residual(x, y, c.residual_mult, history=history, depth=r + 1, average=l.average, store=not last,
                                       gain=self.final_norm.gain if last else 1.0, **form)
+            if on_layer is not None:
+                on_layer(r, x)
+        return h
+
+    def _run_post(self, batch, cache: HybridCache, on_layer) -> torch.Tensor:
+        c = self.config
+        x = torch.empty((batch.rows, c.width), device=self.device, dtype=torch.float32)
+        form = dict(out_cols=pad_to(c.width), out_dtype=c.dtype)
+
+        def add(y, norm, last):
+            return ops.post_norm_step(x, y, norm.gain, c.eps, final=self.final_norm.gain if last else None, **form)
+
+        h = ops.post_norm_step(x, tokens=batch.tokens, table=self.embed, scale=c.embedding_scale, eps=c.eps, **form)
+        for r, l in enumerate(self.layers):
+            last = r == len(self.layers) - 1
+            h = add(l.mixer.forward(h, cache.runs[r], batch), l.norm1, last and l.mlp is None and l.side is None)
+            if l.mlp is not None:
+                h = add(l.mlp.forward(h), l.norm2, last and l.side is None)
+            if l.side is not None:
+                h = add(l.side.forward(h, batch.tokens, self.side_table, r * c.token_side), l.side.norm, last)
             if on_layer is not None:
                 on_layer(r, x)
         return h
@@ -496,4 +632,5 @@ class HybridModel:
 
 
 __all__ = ["AttentionSpec", "DeltaSpec", "GLUSpec", "HybridConfig", "HybridModel", "LatentSpec", "LayerSpec", "LoopSpec", "RGLRUSpec",
-           "RetentionSpec", "Rotary", "SiluGLUSpec", "Yarn", "pick_next_token"]
+           "RetentionSpec", "Rotary", "SSDSpec", "ShapedAttentionSpec", "SideBySideSpec", "SiluGLUSpec", "TimeMixSpec", "Yarn",
+           "pick_next_token"]

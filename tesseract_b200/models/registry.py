@@ -18,9 +18,10 @@ import torch
 class Architecture:
     name: str
     matches: Callable[[dict], bool]
-    config: Callable          # (parsed config, dtype) -> configuration object
+    config: Callable          # (parsed config, dtype) -> configuration object; with ``shapes``, (.., name -> shape of the weights)
     build: Callable           # (configuration object, device) -> model with load_safetensors
     kernels: str = ""         # group of translation units that serves it (build.GROUPS); empty: the whole library
+    shapes: bool = False      # some sizes are only in the weights
 
 
 _REGISTRY: List[Architecture] = []
@@ -61,8 +62,16 @@ def load_config(path: str, dtype: torch.dtype):
     return arch, arch.config(obj, dtype)
 
 
+def tensor_shapes(path: str) -> dict:
+    from ..io.safetensors import SafeTensors
+    with SafeTensors.open(path) as st:
+        return {k: st.info(k)[1] for k in st.keys()}
+
+
 def load_model(config_path: str, weights_path: str, dtype: torch.dtype, device=None):
-    arch, cfg = load_config(config_path, dtype)
+    obj = read_config(config_path)
+    arch = resolve(obj)
+    cfg = arch.config(obj, dtype, tensor_shapes(weights_path)) if arch.shapes else arch.config(obj, dtype)
     model = arch.build(cfg, device)
     model.load_safetensors(weights_path)
     return model
@@ -110,8 +119,20 @@ def _polosun_build(cfg, device):
     return polosun.build(cfg, device)
 
 
+def _vobotar_config(obj: dict, dtype: torch.dtype, shapes=None):
+    from . import vobotar
+    return vobotar.config_from_dict(obj, dtype, shapes)
+
+
+def _vobotar_build(cfg, device):
+    from . import vobotar
+    return vobotar.build(cfg, device)
+
+
 register(Architecture("Llama", _is_llama, _llama_config, _llama_build))
 register(Architecture("Fozelix", lambda o: o.get("architecture") == "Fozelix", _fozelix_config, _fozelix_build,
                       kernels="fozelix"))
 register(Architecture("Polosun", lambda o: o.get("architecture") == "Polosun", _polosun_config, _polosun_build,
                       kernels="polosun"))
+register(Architecture("Vobotar", lambda o: o.get("architecture") == "Vobotar", _vobotar_config, _vobotar_build,
+                      kernels="vobotar", shapes=True))

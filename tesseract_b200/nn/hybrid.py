@@ -1,6 +1,7 @@
-"""Building blocks of hybrid decoders for inference over ragged batches: norms (Dynamic Tanh, RMS with one gain), mixers
-(chunked attention, latent attention, the gated delta rule, retention, the real-gated linear recurrence) and gated
-feed-forwards (clamped, SiLU).
+"""Building blocks of hybrid decoders for inference over ragged batches: norms (Dynamic Tanh, RMS with one gain or one per
+channel), mixers (chunked attention, attention with norms, rotations, windows, sinks and gates, latent attention, the gated delta
+rule, retention, the real-gated linear recurrence, time mixing, state-space duality, two of them side by side), gated feed-forwards
+(clamped, SiLU) and a side input per token.
 
 A mixer or feed-forward is two matrix products around a ``core``: rows of ``w_in`` make its packed input, ``w_out`` takes what
 the core leaves. Layers whose sublayers run side by side lay several of them into one matrix (``place``) and call the cores on
@@ -12,18 +13,22 @@ zeros, everything that the kernels use in fp32 already widened) and translates t
 """
 from __future__ import annotations
 
-from typing import Dict
+from typing import Dict, Optional
 
 import torch
 
 from .. import ops
 from ..ops.delta import DeltaGeometry, DeltaWeights, gated_delta
 from ..ops.latent import LatentGeometry, LatentWeights, latent_attention
-from ..ops.ragged import padded_head_dim, ragged_attention
+from ..ops.gemm import INPUT_ALIGN
+from ..ops.masks import Window
+from ..ops.ragged import AttentionGeometry, AttentionWeights, ScoreForm, padded_head_dim, ragged_attention, shaped_attention
 from ..ops.retention import SPAN, RetentionGeometry, log2_decays, retention
 from ..ops.rglru import CHUNK, RGLRUGeometry, RGLRUWeights, rglru
 from ..ops.rotary import Rotary
-from .ragged import LatentRun, PagedRun, StateRun
+from ..ops.ssd import SSDGeometry, SSDWeights, ssd
+from ..ops.timemix import STREAMS, TimeMixGeometry, TimeMixWeights, time_mix, token_shift
+from .ragged import LatentRun, PagedRun, PairRun, StateRun
 
 
 def pad_to(n: int, m: int = 16) -> int:
@@ -53,11 +58,13 @@ class _Packed:
 
 class _Sublayer(_Packed):
     """Two products around a core. ``in_scale`` multiplies the packed input inside the core: the gain of a norm that has only
-    one, where the layer leaves it to the sublayers. ``tile``: size of the prompt tiles that the core asks the batch for."""
+    one, where the layer leaves it to the sublayers. ``tile``: size of the prompt tiles that the core asks the batch for, ``masks``:
+    the attention masks."""
     out_bias = None
     in_scale = 1.0
     takes_in_scale = False
     tile = 0
+    masks = ()
 
     @property
     def cols(self) -> int:
@@ -75,8 +82,19 @@ class _Sublayer(_Packed):
 
 
 class _Mixer(_Sublayer):
+    """``streams``: first packed column of every input that the first product reads (a mixer that makes its own inputs from h has
+    ``mix_inputs``). ``out_scale`` multiplies what the core leaves."""
+    streams = (0,)
+    out_scale = 1.0
+
+    @property
+    def tiles(self) -> tuple:
+        return (self.tile,) if self.tile else ()
+
     def forward(self, h, storage, batch):
-        return ops.project(self.core(ops.project(h, self.w_in), storage, batch), self.w_out)
+        p = ops.project(h, self.w_in) if len(self.streams) == 1 else ops.project_inputs(self.mix_inputs(h, storage, batch), self.w_in,
+                                                                                         self.streams)
+        return ops.project(self.core(p, storage, batch), self.w_out)
 
 
 class _FeedForward(_Sublayer):
@@ -99,6 +117,24 @@ class ScalarRMSNorm(_Packed):
 
     def unpack(self):
         return {"": torch.tensor(self.gain, dtype=self.dtype, device=self.device)}
+
+
+class RMSNorm(_Packed):
+    """x / sqrt(mean(x^2) + eps) times a gain per channel, stored as it is or, with ``offset`` 1, around zero."""
+
+    def __init__(self, width: int, eps: float, offset: float, dtype, device):
+        super().__init__(dtype, device)
+        self.width, self.eps, self.offset = width, float(eps), float(offset)
+        self.gain = self._zeros(width, dtype=torch.float32) + 1.0
+
+    def logical_shapes(self):
+        return {"": (self.width,)}
+
+    def _pack(self, t):
+        self.gain.copy_(t[""].float() + self.offset)
+
+    def unpack(self):
+        return {"": (self.gain - self.offset).to(self.dtype)}
 
 
 class DynamicTanh(_Packed):
@@ -137,6 +173,7 @@ class ChunkedAttention(_Mixer):
             raise ValueError("attention: positive sizes, and heads a multiple of kv_heads")
         self.width, self.heads, self.kv_heads, self.dim, self.vdim = width, heads, kv_heads, dim, vdim
         self.scale, self.chunk = float(scale), int(chunk)
+        self.masks = (self.chunk,)
         self.D = padded_head_dim(dim, vdim, dtype)
         self.w_in = self._zeros((heads + 2 * kv_heads) * self.D, pad_to(width))
         self.b_in = self._zeros((heads + 2 * kv_heads) * self.D, dtype=torch.float32)
@@ -336,6 +373,7 @@ class LatentAttention(_RowPacked):
     """Attention whose keys and values are products of a cached latent, with a rotated key part shared by all heads and a
     sigmoid gate on the heads (see ``ops.latent``)."""
     takes_in_scale = True
+    masks = (0,)
 
     def __init__(self, width: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float, rotary: Rotary, eps: float,
                  dtype, device):
@@ -496,3 +534,281 @@ class RGLRU(_RowPacked):
 
     def core(self, proj, storage, batch, out=None):
         return rglru(proj, self.geo, self.w, storage[0], storage[1], batch, self.in_scale, out)
+
+
+class ShapedAttention(_RowPacked):
+    """Grouped-query attention whose parts can be chosen (see ``ops.ragged``): biases on the projections, values of their own or the
+    keys as projected, a norm of q and k, rotation, a mask, what becomes of the scores, values mixed with those of the model's
+    first such layer, a gate per head or per element."""
+
+    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, form: ScoreForm, eps: float, dtype, device, bias: bool = False,
+                 keys_as_values: bool = False, norm: str = "", rotary: Optional[Rotary] = None, learned_sink: bool = False, v_mix: bool = False,
+                 gate: str = ""):
+        super().__init__(dtype, device)
+        self.width, self.v_mix, self.learned_sink = width, bool(v_mix), bool(learned_sink)
+        self.geo = g = AttentionGeometry(heads, kv_heads, dim, vdim, dtype, rotary, keys_as_values, gate)
+        self.w_in, self.w_out = self._zeros(g.cols, pad_to(width)), self._zeros(width, g.out_cols)
+        vec = lambda n: self._zeros(n, dtype=torch.float32)   # noqa: E731
+        form.slopes, form.sink = (t.to(self.device) if t is not None else None for t in (form.slopes, form.sink))
+        if learned_sink:
+            form.sink = vec(heads)
+        sizes = {"head": (g.D, g.D), "whole": (heads * g.D, kv_heads * g.D)}.get(norm)
+        if norm not in ("", "unit", "head", "whole"):
+            raise ValueError(f"attention: unknown norm {norm!r}")
+        self.w = AttentionWeights(form, vec(g.off_gate) if bias else None, norm, vec(sizes[0]) if sizes else None,
+                                  vec(sizes[1]) if sizes else None, float(eps))
+        self.masks = (form.mask,)
+
+    def tensors(self):
+        w = self.w
+        return super().tensors() + [t for t in (w.bias, w.q_norm, w.k_norm, w.form.slopes, w.form.sink) if t is not None]
+
+    def run_spec(self) -> PagedRun:
+        return PagedRun(self.geo.kv_heads, self.geo.D, self.geo.rotary, self.v_mix)
+
+    def _rows(self):
+        g = self.geo
+        qk, v = g.columns(), torch.arange(g.vdim)
+        out = {"q": _head_rows(0, g.heads, g.D, qk), "k": _head_rows(g.off_k, g.kv_heads, g.D, qk)}
+        if not g.keys_as_values:
+            out["v"] = _head_rows(g.off_v, g.kv_heads, g.D, v)
+        if g.gate:
+            out["g"] = g.off_gate + torch.arange(g.heads) if g.gate == "head" else _head_rows(g.off_gate, g.heads, g.D, v)
+        return out
+
+    def _out_columns(self):
+        return _head_rows(0, self.geo.heads, self.geo.D, torch.arange(self.geo.vdim))
+
+    def _vectors(self):
+        """name -> (fp32 vector, its places)"""
+        g, w, rows, out = self.geo, self.w, self._rows(), {}
+        if w.bias is not None:
+            out.update({n + ".b": (w.bias, rows[n]) for n in "qkv" if n in rows})
+        if w.norm == "head":
+            out.update({"q.norm": (w.q_norm, g.columns()), "k.norm": (w.k_norm, g.columns())})
+        elif w.norm == "whole":
+            out.update({"q.norm": (w.q_norm, rows["q"]), "k.norm": (w.k_norm, rows["k"] - g.off_k)})
+        if self.learned_sink:
+            out["sink"] = (w.form.sink, torch.arange(g.heads))
+        return out
+
+    def logical_shapes(self):
+        out = {**self._row_shapes(), **{n: (len(at),) for n, (_, at) in self._vectors().items()}}
+        if self.v_mix:
+            out["vmix"] = ()
+        return out
+
+    def _pack(self, t):
+        self._pack_rows(t)
+        for n, (vec, at) in self._vectors().items():
+            vec[at.to(self.device)] = t[n].to(self.device).float()
+        if self.v_mix:
+            self.w.vmix = float(t["vmix"])
+
+    def unpack(self):
+        out = {**self._unpack_rows(), **{n: vec[at.to(self.device)].to(self.dtype) for n, (vec, at) in self._vectors().items()}}
+        if self.v_mix:
+            out["vmix"] = torch.tensor(self.w.vmix, dtype=self.dtype, device=self.device)
+        return out
+
+    def core(self, proj, storage, batch, out=None):
+        k, v, angles, first = storage if len(storage) == 4 else (*storage, None, None)
+        return shaped_attention(proj, self.geo, self.w, k, v, angles, first, batch, self.out_scale, out)
+
+
+class TimeMix(_RowPacked):
+    """Linear attention with a decay per channel and token, fed by mixes of a token's input and the one before (see
+    ``ops.timemix``)."""
+
+    def __init__(self, width: int, heads: int, dim: int, rank: int, eps: float, dtype, device):
+        super().__init__(dtype, device)
+        self.width = width
+        self.geo = g = TimeMixGeometry(heads, dim, rank)
+        self.streams = g.starts
+        self.w_in, self.w_out = self._zeros(g.cols, pad_to(width)), self._zeros(width, g.out_cols)
+        f32, n = torch.float32, heads * g.dp
+        self.mu = self._zeros(len(STREAMS), pad_to(width), dtype=f32)
+        self.w = TimeMixWeights(self._zeros(n, g.rp), self._zeros(n, dtype=f32), self._zeros(n, dtype=f32), self._zeros(n, dtype=f32), float(eps))
+
+    def tensors(self):
+        return super().tensors() + [self.w.w2, self.w.w0, self.w.u, self.w.norm]
+
+    def run_spec(self) -> StateRun:
+        g = self.geo
+        return StateRun((g.heads, g.dp, g.dp), (1, pad_to(self.width)))
+
+    def _rows(self):
+        g = self.geo
+        head = lambda i: _head_rows(i * g.section, g.heads, g.dp, torch.arange(g.dim))   # noqa: E731
+        return {"r": head(0), "k": head(1), "v": head(2), "g": head(3), "w1": 4 * g.section + torch.arange(g.rank)}
+
+    def _out_columns(self):
+        return _head_rows(0, self.geo.heads, self.geo.dp, torch.arange(self.geo.dim))
+
+    def logical_shapes(self):
+        g, n = self.geo, self.geo.heads * self.geo.dim
+        return {**{"mu." + s: (self.width,) for s in STREAMS}, **self._row_shapes(), "w2": (n, g.rank), "w0": (n,), "u": (g.heads, g.dim),
+                "norm": (n,)}
+
+    def _pack(self, t):
+        self._pack_rows(t)
+        for i, s in enumerate(STREAMS):
+            self.mu[i, :self.width].copy_(t["mu." + s])
+        at = self._out_columns().to(self.device)
+        self.w.w2[at, :self.geo.rank] = t["w2"].to(self.device, self.dtype)
+        for n in ("w0", "u", "norm"):
+            getattr(self.w, n)[at] = t[n].to(self.device).float().reshape(-1)
+
+    def unpack(self):
+        g, at = self.geo, self._out_columns().to(self.device)
+        out = {**self._unpack_rows(), **{"mu." + s: self.mu[i, :self.width].to(self.dtype) for i, s in enumerate(STREAMS)},
+               "w2": self.w.w2[at, :g.rank]}
+        out.update({n: getattr(self.w, n)[at].to(self.dtype) for n in ("w0", "u", "norm")})
+        out["u"] = out["u"].view(g.heads, g.dim)
+        return out
+
+    def mix_inputs(self, h, storage, batch, keep=False):
+        return token_shift(h, self.mu, storage[0], batch, keep)
+
+    def core(self, proj, storage, batch, out=None):
+        return time_mix(proj, self.geo, self.w, storage[1], batch, self.out_scale, out)
+
+
+class SSD(_RowPacked):
+    """State-space duality with a short convolution, normed in parts after its gate (see ``ops.ssd``)."""
+
+    def __init__(self, width: int, heads: int, vdim: int, state: int, groups: int, conv: int, norm_parts: int, eps: float, dtype, device):
+        super().__init__(dtype, device)
+        self.width = width
+        self.geo = g = SSDGeometry(heads, vdim, state, groups, conv, norm_parts)
+        self.w_in, self.w_out = self._zeros(g.cols, pad_to(width)), self._zeros(width, g.out_cols)
+        vec = lambda *n: self._zeros(*n, dtype=torch.float32)   # noqa: E731
+        self.w = SSDWeights(vec(conv, g.conv_cols), vec(g.conv_cols), vec(heads), vec(heads), vec(heads), vec(heads * g.vp), float(eps))
+
+    def tensors(self):
+        return super().tensors() + [t for t in vars(self.w).values() if isinstance(t, torch.Tensor)]
+
+    def run_spec(self) -> StateRun:
+        g = self.geo
+        return StateRun((g.heads, g.vp, g.np), (g.taps - 1, g.conv_cols))
+
+    def _inner(self, at):
+        return _head_rows(at, self.geo.heads, self.geo.vp, torch.arange(self.geo.vdim))
+
+    def _rows(self):
+        g = self.geo
+        group = lambda at: _head_rows(at, g.groups, g.np, torch.arange(g.state))   # noqa: E731
+        return {"in": torch.cat([self._inner(0), self._inner(g.off_x), group(g.off_b), group(g.off_c), g.off_dt + torch.arange(g.heads)])}
+
+    def _conv_columns(self):
+        g, rows = self.geo, self._rows()["in"]
+        return rows[g.heads * g.vdim:len(rows) - g.heads] - g.off_x
+
+    def _out_columns(self):
+        return self._inner(0)
+
+    def logical_shapes(self):
+        g = self.geo
+        n = len(self._conv_columns())
+        return {**self._row_shapes(), "conv": (n, g.taps), "conv.b": (n,), "dt_bias": (g.heads,), "A_log": (g.heads,), "D": (g.heads,),
+                "norm": (g.heads * g.vdim,)}
+
+    def _pack(self, t):
+        w, c, at = self.w, self._conv_columns().to(self.device), self._out_columns().to(self.device)
+        self._pack_rows(t)
+        w.conv[:, c] = t["conv"].to(self.device).float().t()
+        w.conv_b[c] = t["conv.b"].to(self.device).float()
+        w.norm[at] = t["norm"].to(self.device).float()
+        for vec, n in ((w.dt_bias, "dt_bias"), (w.a_log, "A_log"), (w.d, "D")):
+            vec.copy_(t[n])
+
+    def unpack(self):
+        w, c, at = self.w, self._conv_columns().to(self.device), self._out_columns().to(self.device)
+        return {**self._unpack_rows(), "conv": w.conv[:, c].t().contiguous().to(self.dtype), "conv.b": w.conv_b[c].to(self.dtype),
+                "norm": w.norm[at].to(self.dtype), "dt_bias": w.dt_bias.to(self.dtype), "A_log": w.a_log.to(self.dtype), "D": w.d.to(self.dtype)}
+
+    def core(self, proj, storage, batch, out=None):
+        return ssd(proj, self.geo, self.w, storage[0], storage[1], batch, self.out_scale, out)
+
+
+class SideBySide(_Mixer):
+    """left_scale left(h) + right_scale right(h): one product feeds both cores, one takes both results back and sums them. Tensors
+    are the parts' own, under "left." and "right."."""
+
+    def __init__(self, left: _Mixer, right: _Mixer, left_scale: float, right_scale: float, width: int, dtype, device):
+        super().__init__(dtype, device)
+        if len(left.streams) > 1:
+            raise ValueError("side by side: the mixer that makes its own inputs is the right one")
+        self.left, self.right = left, right
+        left.out_scale, right.out_scale = float(left_scale), float(right_scale)
+        own = len(right.streams) > 1
+        self.cut = pad_to(left.cols, INPUT_ALIGN if own else 8)
+        self.streams = (0,) + tuple(self.cut + s for s in right.streams) if own else (0,)
+        self.w_in, self.w_out = self._zeros(self.cut + right.cols, pad_to(width)), self._zeros(width, left.out_cols + right.out_cols)
+        left.place(self.w_in[:left.cols], self.w_out[:, :left.out_cols])
+        right.place(self.w_in[self.cut:], self.w_out[:, left.out_cols:])
+        self.masks = left.masks + right.masks
+
+    @property
+    def tiles(self) -> tuple:
+        return self.left.tiles + self.right.tiles
+
+    def tensors(self):
+        parts = [t for p in (self.left, self.right) for t in p.tensors() if t is not p.w_in and t is not p.w_out]
+        return super().tensors() + parts
+
+    def run_spec(self) -> PairRun:
+        return PairRun(self.left.run_spec(), self.right.run_spec())
+
+    def _both(self):
+        return (("left.", self.left), ("right.", self.right))
+
+    def logical_shapes(self):
+        return {pre + n: s for pre, p in self._both() for n, s in p.logical_shapes().items()}
+
+    def _pack(self, t):
+        for pre, p in self._both():
+            p._pack({n: t[pre + n] for n in p.logical_shapes()})
+
+    def unpack(self):
+        return {pre + n: v for pre, p in self._both() for n, v in p.unpack().items()}
+
+    def mix_inputs(self, h, storage, batch):
+        return self.right.mix_inputs(h, storage[1], batch, keep=True)
+
+    def core(self, proj, storage, batch, out=None):
+        z = out if out is not None else torch.empty((proj.shape[0], self.out_cols), device=proj.device, dtype=proj.dtype)
+        k = self.left.out_cols
+        self.left.core(proj[:, :self.left.cols], storage[0], batch, out=z[:, :k])
+        self.right.core(proj[:, self.cut:], storage[1], batch, out=z[:, k:])
+        return z
+
+
+class TokenSide(_Packed):
+    """A side input per token and layer: y = W_proj (gelu_tanh(W_gate x) * e), e the token's row of a table; x + y / rms(y) *
+    norm."""
+
+    def __init__(self, width: int, dim: int, eps: float, dtype, device):
+        super().__init__(dtype, device)
+        self.width, self.dim = width, dim
+        self.w_gate, self.w_proj = self._zeros(pad_to(dim), pad_to(width)), self._zeros(width, pad_to(dim))
+        self.norm = RMSNorm(width, eps, 0.0, dtype, device)
+
+    def tensors(self):
+        return super().tensors() + self.norm.tensors()
+
+    def logical_shapes(self):
+        return {"gate": (self.dim, self.width), "proj": (self.width, self.dim), "norm": (self.width,)}
+
+    def _pack(self, t):
+        self.w_gate[:self.dim, :self.width].copy_(t["gate"])
+        self.w_proj[:, :self.dim].copy_(t["proj"])
+        self.norm._pack({"": t["norm"]})
+
+    def unpack(self):
+        return {"gate": self.w_gate[:self.dim, :self.width].contiguous(), "proj": self.w_proj[:, :self.dim].contiguous(),
+                "norm": self.norm.unpack()[""]}
+
+    def forward(self, h, tokens, table, first: int):
+        """What is normed and added; ``table`` [vocab, ..], this layer's part from column ``first`` on."""
+        return ops.project(ops.gelu_lookup(ops.project(h, self.w_gate), tokens, table, first, self.dim), self.w_proj)

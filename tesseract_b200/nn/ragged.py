@@ -14,19 +14,33 @@ from typing import Dict, List, Optional, Sequence
 import numpy as np
 import torch
 
+from ..ops.masks import Mask, Window
 from ..ops.rotary import Rotary
 from .kv_cache import BlockAllocator
 
 
 @dataclass(frozen=True)
 class PagedRun:
-    """Storage of one attention run: K and V pages of ``head_dim`` columns per key head."""
+    """Storage of one attention run: K and V pages of ``head_dim`` columns per key head. A run that rotates also gets the angles of
+    its positions; one of the runs that share their first one's values (``mixes_values``) also gets that run's V pages (None for the
+    first)."""
     kv_heads: int
     head_dim: int
+    rotary: Optional[Rotary] = None
+    mixes_values: bool = False
 
     def allocate(self, c: "HybridCache") -> tuple:
         shape = (c.num_blocks, self.kv_heads, c.block_size, self.head_dim)
-        return tuple(torch.zeros(shape, dtype=c.dtype, device=c.device) for _ in range(2))
+        k, v = (torch.zeros(shape, dtype=c.dtype, device=c.device) for _ in range(2))
+        if self.rotary is None and not self.mixes_values:
+            return k, v
+        first = None
+        if self.mixes_values:
+            if c.first_values is None:
+                c.first_values = v
+            else:
+                first = c.first_values
+        return k, v, c.angles(self.rotary) if self.rotary is not None else None, first
 
 
 @dataclass(frozen=True)
@@ -57,6 +71,16 @@ class StateRun:
         return tuple(out)
 
 
+@dataclass(frozen=True)
+class PairRun:
+    """Storage of two mixers side by side."""
+    left: object
+    right: object
+
+    def allocate(self, c: "HybridCache") -> tuple:
+        return self.left.allocate(c), self.right.allocate(c)
+
+
 class HybridCache:
     quantized = False
 
@@ -70,6 +94,7 @@ class HybridCache:
         self.slot_allocator = BlockAllocator(max_sequences)
         self.tables = np.zeros((max_sequences, self.max_blocks), dtype=np.int32)   # row = the sequence's slot
         self._angles: Dict[Rotary, torch.Tensor] = {}
+        self.first_values: Optional[torch.Tensor] = None      # V pages of the first run that mixes values
         self.runs: List[tuple] = [r.allocate(self) for r in runs]
 
     def angles(self, rotary: Rotary) -> torch.Tensor:
@@ -78,8 +103,14 @@ class HybridCache:
             self._angles[rotary] = rotary.table(self.max_len, self.device)
         return self._angles[rotary]
 
+    def tensors(self, run) -> list:
+        """The tensors of one run's storage."""
+        if isinstance(run, tuple):
+            return [t for part in run for t in self.tensors(part)]
+        return [run] if run is not None else []
+
     def nbytes(self) -> int:
-        unique = {t.data_ptr(): t for r in self.runs for t in r if t.numel()}
+        unique = {t.data_ptr(): t for t in self.tensors(tuple(self.runs)) if t.numel()}
         return sum(t.numel() * t.element_size() for t in unique.values())
 
     def can_admit(self) -> bool:
@@ -147,7 +178,7 @@ class HybridSequence:
 
 @dataclass
 class Segments:
-    """A step's prompt rows cut at the chunk edges, for one chunk size: query and key offsets of every piece, where each
+    """A step's prompt rows for one mask, cut at the chunk edges if it has chunks: query and key offsets of every piece, where each
     row's key goes on the key axis, and which pooled keys are copied in front of it."""
     n: int
     max_q: int
@@ -161,13 +192,16 @@ class Segments:
     gather_src: Optional[torch.Tensor] = None
 
 
-def cut_segments(portions, chunk: int, slot_of) -> Segments:
+def cut_segments(portions, mask: Mask, slot_of) -> Segments:
     """``portions``: (pos0, n) of every prompt portion in row order; ``slot_of(i, positions)`` gives pool slots of portion
-    i's sequence. chunk 0: no mask, one piece per portion with everything before it in front."""
+    i's sequence. Mask 0: one piece per portion with everything before it in front; a window: one piece with what its first
+    row sees in front."""
     cu_q, cu_k, stage, dst, src = [0], [0], [], [], []
     row = key = 0
+    window = mask.size if isinstance(mask, Window) else 0
+    chunk = 0 if window else mask
     for i, (p0, n) in enumerate(portions):
-        first = p0 // chunk * chunk if chunk > 0 else 0
+        first = max(0, p0 - window + 1) if window else p0 // chunk * chunk if chunk > 0 else 0
         before = p0 - first
         if before:
             dst.append(np.arange(key, key + before, dtype=np.int32))
@@ -199,10 +233,10 @@ class Tiles:
 class RaggedBatch:
     """One step. ``entries``: (sequence, token ids); the sequences' pages are reserved here and their lengths advanced by
     ``commit`` once the step has been launched. Rows are ordered with single tokens first; ``row_of[i]`` is the first row
-    of entry i. ``want`` [i]: places among entry i's tokens whose logits are asked for, answered in entry order. ``chunks``:
+    of entry i. ``want`` [i]: places among entry i's tokens whose logits are asked for, answered in entry order. ``masks``:
     attention masks, ``tiles``: tile sizes that the model's mixers ask for (``segments``, ``tiles``)."""
 
-    def __init__(self, cache: HybridCache, entries, want=None, chunks: Sequence[int] = (), max_len: int = 0,
+    def __init__(self, cache: HybridCache, entries, want=None, masks: Sequence[Mask] = (), max_len: int = 0,
                  tiles: Sequence[int] = ()):
         self.cache = cache
         entries = [(s, np.asarray(t, dtype=np.int32)) for s, t in entries]
@@ -249,13 +283,13 @@ class RaggedBatch:
                 rows.append(self.row_of[i] + k)
         self.n_want = len(rows)
         self._spans = list(zip(row0[:-1].tolist(), n.tolist(), slot.tolist(), pos0.tolist()))
-        segs: Dict[int, Segments] = {}
+        segs: Dict[Mask, Segments] = {}
         if self.n_prompts:
             pslots = slot[nd:]
 
             def slot_of(i, p):
                 return cache.tables[pslots[i], p // bs] * bs + p % bs
-            for c in chunks:
+            for c in masks:
                 segs[c] = cut_segments(list(zip(pos0[nd:].tolist(), n[nd:].tolist())), c, slot_of)
         nblk = (n[nd:] + 3) // 4                  # the recurrence takes four tokens of a portion at once
         fields = {
@@ -270,9 +304,10 @@ class RaggedBatch:
                 self._tiles[size] = Tiles(int(per.sum()))
                 fields[f"seq:{size}"] = np.repeat(np.arange(self.n_prompts), per)
                 fields[f"first:{size}"] = np.concatenate([[0], np.cumsum(per)])
-        for c, sg in segs.items():
+        pieces = list(segs.values())
+        for i, sg in enumerate(pieces):
             for name, a in zip(("cu_q", "cu_k", "stage_rows", "gather_dst", "gather_src"), sg.host):
-                fields[f"{name}:{c}"] = a
+                fields[f"{name}:{i}"] = a
         flat = np.concatenate([np.ascontiguousarray(a, dtype=np.int32).reshape(-1) for a in fields.values()])
         host = torch.from_numpy(flat)
         if cache.device.type == "cuda":
@@ -285,13 +320,13 @@ class RaggedBatch:
             at += a.size
             if ":" in name:
                 f, c = name.split(":")
-                setattr(self._tiles[int(c)] if f in ("seq", "first") else segs[int(c)], f, t)
+                setattr(self._tiles[int(c)] if f in ("seq", "first") else pieces[int(c)], f, t)
             else:
                 setattr(self, name, t)
         self._segs = segs
 
-    def segments(self, chunk: int) -> Segments:
-        return self._segs[chunk]
+    def segments(self, mask: Mask) -> Segments:
+        return self._segs[mask]
 
     def tiles(self, size: int) -> Tiles:
         return self._tiles[size]

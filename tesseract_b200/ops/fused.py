@@ -508,3 +508,58 @@ def depth_residual(x_in=None, y=None, mult=1.0, tokens=None, table=None, width=0
         h[:, W:] = 0
         h[:, :W] = new / torch.sqrt((new * new).mean(-1, keepdim=True) + eps) * gain
     return x, h
+
+
+_native.register_signatures({
+    "tsb_post_norm_step": [_P, _P, _L, _P, _P, _F, _P, _P, _L, _I, _F, _P, _L, _I, _I, _I, _I, _P],
+    "tsb_gelu_lookup": [_P, _L, _P, _P, _L, _I, _I, _P, _L, _I, _I, _I, _I, _P],
+})
+
+
+def post_norm_step(x, y=None, gain=None, eps=0.0, tokens=None, table=None, scale=1.0, final=None, out_cols=0, out_dtype=None, out=None):
+    """One step of an fp32 residual stream ``x`` [T, W] (updated in place) whose sublayers are normed on their way in:
+
+        x  = table[tokens] * scale                          (tokens given)
+        x += y / sqrt(mean(y^2) + eps) * gain               (y given; gain fp32 [W])
+        return x, or x / sqrt(mean(x^2) + eps) * final      (final fp32 [W]; [T, out_cols], zero past W, ``out_dtype``)
+
+    ``out``: receives the result when given."""
+    T, W = x.shape
+    h = out if out is not None else torch.empty((T, out_cols or W), device=x.device,
+                                                dtype=out_dtype or (y.dtype if y is not None else table.dtype))
+    if T == 0:
+        return h
+    if x.is_cuda:
+        start = tokens is not None
+        if y is not None and y.dtype != h.dtype or start and table.dtype != h.dtype:
+            raise ValueError("post_norm_step: the inputs and the result share one dtype")
+        check(lib().tsb_post_norm_step(x.data_ptr(), _ptr(y), y.stride(0) if y is not None else 0, _ptr(gain), _ptr(final),
+                                       float(eps), _ptr(tokens), _ptr(table) if start else None, table.stride(0) if start else 0,
+                                       table.shape[0] if start else 0, float(scale), h.data_ptr(), h.stride(0), h.shape[1], T, W,
+                                       dtype_code(h.dtype), stream_ptr(x.device)), "tsb_post_norm_step")
+        return h
+    if tokens is not None:
+        x.copy_(table[tokens.long(), :W].float() * scale)
+    if y is not None:
+        z = y[:, :W].float()
+        x += z / torch.sqrt((z * z).mean(-1, keepdim=True) + eps) * gain
+    h[:, W:] = 0
+    h[:, :W] = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * final if final is not None else x
+    return h
+
+
+def gelu_lookup(g, tokens, table, first, dim):
+    """gelu_tanh(g[:, :dim]) * table[tokens, first:first + dim] as [T, cols of g] (zero past ``dim``)."""
+    T = g.shape[0]
+    out = torch.empty_like(g)
+    if T == 0:
+        return out
+    if g.is_cuda:
+        check(lib().tsb_gelu_lookup(g.data_ptr(), g.stride(0), tokens.data_ptr(), table.data_ptr(), table.stride(0), table.shape[0],
+                                    first, out.data_ptr(), out.stride(0), out.shape[1], T, dim, dtype_code(g.dtype),
+                                    stream_ptr(g.device)), "tsb_gelu_lookup")
+        return out
+    out[:, dim:] = 0
+    e = table[tokens.long(), first:first + dim].float()
+    out[:, :dim] = torch.nn.functional.gelu(g[:, :dim].float(), approximate="tanh") * e
+    return out

@@ -297,3 +297,38 @@ def project(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = No
     if x.is_cuda:
         return (x @ w.t()).to(out_dtype or x.dtype)
     return (x.float() @ w.float().t()).to(out_dtype or x.dtype)
+
+
+_native.register_signatures({
+    "tsb_gemm_bf16_inputs": [_native.P, _native.P, _native.P, _native.P, _native.I, _native.I, _native.I, _native.I, _native.L,
+                             _native.L, _native.L, _native.L, _native.P],
+    "tsb_gemm_decode_inputs": [_native.P, _native.P, _native.P, _native.P, _native.I, _native.I, _native.I, _native.I, _native.L,
+                               _native.L, _native.L, _native.L, _native.I, _native.P],
+})
+INPUT_ALIGN = 128          # first result column of every input
+
+
+def project_inputs(xs: torch.Tensor, w: torch.Tensor, starts) -> torch.Tensor:
+    """One product for several inputs of the same rows: result columns [starts[g], starts[g + 1]) are xs[g] [M, K] times those
+    rows of w [N, K]. The starts are multiples of ``INPUT_ALIGN``; the tiles of either GEMM pick their input by their column."""
+    n, M, K = xs.shape
+    N = w.shape[0]
+    ends = list(starts[1:]) + [N]
+    if len(starts) != n or starts[0] != 0 or any(s % INPUT_ALIGN for s in starts) or any(a >= b for a, b in zip(starts, ends)):
+        raise ValueError("project_inputs: ascending starts, multiples of the alignment, one per input")
+    if n == 1:
+        return project(xs[0], w)
+    if _use_native(xs) and M > 0:
+        import ctypes
+        if xs.stride(2) != 1 or w.stride(1) != 1 or xs.stride(0) % xs.stride(1):
+            raise ValueError("project_inputs: contiguous rows, inputs a whole number of rows apart")
+        out = torch.empty((M, N), device=xs.device, dtype=xs.dtype)
+        first = (ctypes.c_int * n)(*starts)
+        args = (first, xs.data_ptr(), w.data_ptr(), out.data_ptr(), n, M, N, K, xs.stride(0) // xs.stride(1), xs.stride(1),
+                w.stride(0), out.stride(0))
+        if M <= 256:
+            _native.check(_native.lib().tsb_gemm_decode_inputs(*args, 1, _native.stream_ptr(xs.device)), "tsb_gemm_decode_inputs")
+        else:
+            _native.check(_native.lib().tsb_gemm_bf16_inputs(*args, _native.stream_ptr(xs.device)), "tsb_gemm_bf16_inputs")
+        return out
+    return torch.cat([project(xs[g], w[a:b]) for g, (a, b) in enumerate(zip(starts, ends))], dim=1)

@@ -1,4 +1,5 @@
-"""Rotary positions whose pairs are halves of a range: coordinate i of the first ``dims`` turns with coordinate i + dims / 2.
+"""Rotary positions. The pairs are halves of a range (coordinate i of the first ``dims`` turns with coordinate i + dims / 2) or,
+with ``neighbours``, coordinates 2 i and 2 i + 1.
 
 Kernels read a head stored as [u: hp | v: hp | rest], pair i = (u_i, v_i), with hp = dims / 2 rounded up to a multiple of 8
 (a permutation with zero padding, the same for queries and keys, so no score sees it), and a table of (cos, sin) per
@@ -28,6 +29,7 @@ class Rotary:
     dims: int
     base: float
     scaling: Optional[Yarn] = None
+    neighbours: bool = False
 
     def __post_init__(self):
         if self.dims < 0 or self.dims % 2 or self.base <= 0:
@@ -49,6 +51,8 @@ class Rotary:
         if dim < self.dims:
             raise ValueError(f"rotary: {self.dims} rotated dims in a head of {dim}")
         i = torch.arange(dim)
+        if self.neighbours:
+            return torch.where(i < self.dims, i // 2 + i % 2 * self.hp, i - self.dims + 2 * self.hp)
         return torch.where(i < self.half, i, torch.where(i < self.dims, i - self.half + self.hp, i - self.dims + 2 * self.hp))
 
     def stored(self, dim: int, multiple: int = 8) -> int:
