@@ -10,7 +10,7 @@ namespace tsb {
 namespace {
 
 struct PrepareParams {
-  int rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, ld;    // norm: 0 none, 1 unit heads, 2 heads with a weight, 3 whole
+  int rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, ld, D_first;    // norm: 0 none, 1 unit heads, 2 heads with a weight, 3 whole
   float eps, vmix;
   const void* proj;
   const float* bias;          // [off_v + Hkv * D] or null
@@ -22,7 +22,7 @@ struct PrepareParams {
   void* q;                    // [rows, H, D]
   void* k_pool;               // [blocks, Hkv, bs, D]
   void* v_pool;
-  const void* v_first;        // pool like v_pool, or null
+  const void* v_first;        // [blocks, Hkv, bs, D_first] or null
   void* stage;                // [keys, 2 Hkv, D] or null
   const int* stage_rows;      // [rows - n_decode]
 };
@@ -106,7 +106,8 @@ attn_prepare_kernel(PrepareParams p) {
       if (kind == 2) {
         if (p.v_first) {
           float v0[V] = {};
-          if (slot >= 0) ld16<T>(static_cast<const T*>(p.v_first) + (page + static_cast<long long>(head) * p.bs) * D + d, v0);
+          if (slot >= 0 && d < p.D_first)
+            ld16<T>(static_cast<const T*>(p.v_first) + (page + static_cast<long long>(head) * p.bs) * p.D_first + d, v0);
 #pragma unroll
           for (int i = 0; i < V; ++i) f[k][i] = (1.f - p.vmix) * f[k][i] + p.vmix * v0[i];
         }
@@ -161,17 +162,17 @@ int launch_prepare(const PrepareParams& p, cudaStream_t s) {
 }  // namespace
 }  // namespace tsb
 
-// ints: rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, row stride; floats: eps, vmix; ptrs: proj, bias, q_norm, k_norm,
+// ints: rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, row stride, head size of v_first; floats: eps, vmix; ptrs: proj, bias, q_norm, k_norm,
 // table, positions, slots, q, k_pool, v_pool, v_first, stage, stage_rows (see PrepareParams). dtype: 0 = fp32, 1 = bf16. D is a
 // multiple of 32, up to 256; rows and sections start on 16 bytes.
 TSB_EXPORT int tsb_attn_prepare(const int* v, const float* f, void* const* q, int dtype, void* stream) {
   using namespace tsb;
-  PrepareParams p{v[0], v[1], v[2], v[3], v[4], v[5], v[6], v[7], v[8], v[9], v[10], v[11], f[0], f[1], q[0], static_cast<const float*>(q[1]),
+  PrepareParams p{v[0], v[1], v[2], v[3], v[4], v[5], v[6], v[7], v[8], v[9], v[10], v[11], v[12], f[0], f[1], q[0], static_cast<const float*>(q[1]),
                   static_cast<const float*>(q[2]), static_cast<const float*>(q[3]), static_cast<const float2*>(q[4]),
                   static_cast<const int*>(q[5]), static_cast<const int*>(q[6]), q[7], q[8], q[9], q[10], q[11], static_cast<const int*>(q[12])};
   if (p.rows <= 0 || p.H <= 0 || p.Hkv <= 0 || p.D <= 0 || p.D % 32 || p.D > 256 || p.dim <= 0 || p.dim > p.D || p.hp % 8 || 2 * p.hp > p.D ||
       p.off_k % 8 || p.off_v % 8 || p.ld % 8 || p.norm < 0 || p.norm > 3 || (p.norm >= 2 && (!p.q_norm || !p.k_norm)) || p.bs <= 0 ||
-      (p.stage && !p.stage_rows) || (reinterpret_cast<uintptr_t>(p.proj) & 15))
+      (p.stage && !p.stage_rows) || (p.v_first && (p.D_first <= 0 || p.D_first % 8)) || (reinterpret_cast<uintptr_t>(p.proj) & 15))
     return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (dtype == 1) return launch_prepare<__nv_bfloat16>(p, s);

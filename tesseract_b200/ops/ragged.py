@@ -235,7 +235,7 @@ _NORMS = {"": 0, "unit": 1, "head": 2, "whole": 3}
 def shaped_attention(proj: torch.Tensor, geo: AttentionGeometry, w: AttentionWeights, k_pool: torch.Tensor, v_pool: torch.Tensor,
                      angles, first_values, batch, out_scale: float = 1.0, out: torch.Tensor | None = None) -> torch.Tensor:
     """proj [T, geo.cols] -> [T, geo.out_cols] (``out`` may be columns of a wider matrix). ``angles``: the cache's table for
-    ``geo.rotary``; ``first_values``: V pages whose values are mixed in, or None."""
+    ``geo.rotary``; ``first_values``: V pages (of any padded head size) whose values are mixed in, or None."""
     T, H, G, D = proj.shape[0], geo.heads, geo.kv_heads, geo.D
     bs = k_pool.shape[2]
     if out is None:
@@ -250,7 +250,8 @@ def shaped_attention(proj: torch.Tensor, geo: AttentionGeometry, w: AttentionWei
     q = torch.empty((T, H, D), device=proj.device, dtype=proj.dtype)
     seg = batch.segments(w.form.mask) if n and tensor_core_heads(D, proj.dtype) and bs % 8 == 0 else None
     stage = torch.empty((seg.keys, 2 * G, D), device=proj.device, dtype=proj.dtype) if seg is not None else None
-    ints = (ctypes.c_int * 12)(T, H, G, D, geo.dim, geo.hp, geo.off_k, geo.off_v, _NORMS[w.norm], bs, nd, proj.stride(0))
+    ints = (ctypes.c_int * 13)(T, H, G, D, geo.dim, geo.hp, geo.off_k, geo.off_v, _NORMS[w.norm], bs, nd, proj.stride(0),
+                               first_values.shape[3] if first_values is not None else 0)
     floats = (ctypes.c_float * 2)(w.eps, w.vmix)
     ptrs = (ctypes.c_void_p * 13)(proj.data_ptr(), _ptr(w.bias), _ptr(w.q_norm), _ptr(w.k_norm), _ptr(angles), batch.positions.data_ptr(),
                                   batch.slots.data_ptr(), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), _ptr(first_values), _ptr(stage),
@@ -281,7 +282,8 @@ def _shaped_torch(proj, geo, w, k_pool, v_pool, angles, first_values, batch, gat
         q, k = rotate_stored(q, angles, pos), rotate_stored(k, angles, pos)
     if first_values is not None:
         sl = batch.slots.long()
-        v = (1.0 - w.vmix) * v + w.vmix * first_values[sl // bs, :, sl % bs].float()
+        first = torch.nn.functional.pad(first_values[sl // bs, :, sl % bs].float(), (0, max(0, D - first_values.shape[3])))
+        v = (1.0 - w.vmix) * v + w.vmix * first[..., :D]
     return _attend_torch(q.to(proj.dtype), k.to(proj.dtype), v.to(proj.dtype), k_pool, v_pool, batch, w.form, gate, out)
 
 
