@@ -110,10 +110,11 @@ def parse_args():
                     help="auto | dp | tp | tpK (tensor parallel over K ranks, data parallel over the rest) | a comma list: "
                          "every mesh listed is measured and `value` is the fastest")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--hybrid", nargs="?", const="fozelix", default="", choices=["fozelix", "polosun"],
+    ap.add_argument("--hybrid", nargs="?", const="fozelix", default="", choices=["fozelix", "polosun", "vobotar"],
                     help="instead of the headline: prefill and decode throughput of a hybrid decoder at the sizes of real layers, one "
-                         "GPU (benchmarks/bench_hybrid.py): fozelix (gated delta rule + chunked attention, beside Llama; the default) or "
-                         "polosun (retention, latent attention, gated recurrence, beside fozelix and Llama)")
+                         "GPU (benchmarks/bench_hybrid.py): fozelix (gated delta rule + chunked attention, beside Llama; the default), "
+                         "polosun (retention, latent attention, gated recurrence, beside fozelix and Llama) or vobotar (attention, time mixing, "
+                         "state-space duality, beside polosun, fozelix and Llama)")
     ap.add_argument("--ref-time-budget", type=float, default=float(os.environ.get("TESSERACT_REF_TIME_BUDGET", 780)),
                     help="(--impl reference) seconds the whole reference arm may take; the timed step count shrinks to fit")
     return ap.parse_args()
@@ -297,7 +298,8 @@ def main():
         from bench_hybrid import run
         sampler = ClockSampler(0)
         sampler.start()
-        models = ("hybrid", "llama") if args.hybrid == "fozelix" else ("polosun", "hybrid", "llama")
+        models = {"fozelix": ("hybrid", "llama"), "polosun": ("polosun", "hybrid", "llama"),
+                  "vobotar": ("vobotar", "polosun", "hybrid", "llama")}[args.hybrid]
         sizes = run(models=models)
         print(json.dumps({"benchmark": "hybrid decoder serving beside other models at equal size", "models": models, "n_gpus": 1, "dtype": "bf16",
                           "data": "synthetic random token ids; random-init weights", "sizes": sizes, "clocks": sampler.stop()}))

@@ -496,7 +496,7 @@ def case_clamped_glu(b: Bench):
 # ---- the mixers of 4096-wide layers with 32 heads: retention 128 x 128, latent 64 + 64 / 128 / 512, recurrence 4096 in blocks of 256
 def _mixer_case(b, block, n, rows, past=0):
     """Time of a mixer's core (everything between its two products)."""
-    st = _Step(b, block.run_spec(), n, rows, past, (0,), tiles=[block.tile] if block.tile else [])
+    st = _Step(b, block.run_spec(), n, rows, past, block.masks or (0,), tiles=block.tiles)
     proj = b.randn(n * rows, block.cols)
     return b.time(lambda: block.core(proj, st.cache.runs[0], st.batch))
 
@@ -559,6 +559,108 @@ def case_silu_glu(b: Bench):
     report("silu_glu", b.time(lambda: ops.silu_glu(x, 0.9)), bytes_=x.numel() * 2 * 1.5, shape=list(x.shape))
 
 
+# ---- the mixers of 4096-wide post-normed layers: 32 / 8 heads of 128 (attention), 64 heads of 64 (time mixing), 128 heads of 64 with a
+# state of 128 (state-space duality)
+def _shaped(b, window):
+    from tesseract_b200.nn.hybrid import ShapedAttention
+    from tesseract_b200.ops.masks import Window
+    from tesseract_b200.ops.ragged import ScoreForm
+    from tesseract_b200.ops.rotary import Rotary
+    H, G, D, bf = 32, 8, 128, torch.bfloat16
+    if window:
+        form = ScoreForm(D ** -0.5, Window(window), slopes=torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)]))
+        return ShapedAttention(64, H, G, D, D, form, 1e-6, bf, b.dev, bias=True, keys_as_values=True, norm="unit", learned_sink=True, gate="head")
+    form = ScoreForm(D ** -0.5, 0, 30.0, None, torch.zeros(H))
+    blk = ShapedAttention(64, H, G, D, D, form, 1e-6, bf, b.dev, norm="head", rotary=Rotary(D, 1e4, neighbours=True), gate="element")
+    blk.w.q_norm.fill_(1.0)
+    blk.w.k_norm.fill_(1.0)
+    return blk
+
+
+def case_shaped_attn(b: Bench):
+    """Norms, rotation, append, attention and gate; the counts are those of chunk_attn (two sequences of 4096, or as many rows in
+    shorter ones; 256 sequences at 1400 tokens)."""
+    for n, rows, window in ((2, 4096, 0), (8, 1024, 0), (2, 4096, 1024)):
+        seen = rows * (rows + 1) / 2 if not window else window * (rows - window / 2)
+        ms = _mixer_case(b, _shaped(b, window), n, rows)
+        report("shaped_attn_prefill", ms, flops=4.0 * n * seen * 32 * 128, shape=[n, rows, window])
+    for n, window in ((256, 0), (32, 0), (256, 1024)):
+        ms = _mixer_case(b, _shaped(b, window), n, 1, 1399)
+        report("shaped_attn_decode", ms, bytes_=n * (window or 1400) * 8 * 128 * 2 * 2.0, shape=[n, 1400, window])
+
+
+def case_time_mix(b: Bench):
+    """Prompts: bytes of r, k, v, gate and the result; decode: the state read and written once."""
+    from tesseract_b200.nn.hybrid import TimeMix
+    H, D = 64, 64
+    blk = TimeMix(64, H, D, 64, 1e-6, torch.bfloat16, b.dev)
+    blk.w.w0.uniform_(-6.0, -1.0)
+    blk.w.u.uniform_(0.0, 1.0)
+    for n, rows in ((4, 4096), (1, 4096), (32, 512)):
+        report("time_mix_prefill", _mixer_case(b, blk, n, rows), bytes_=n * rows * H * D * 5 * 2.0, shape=[n, rows])
+    for n in (256, 32):
+        report("time_mix_step", _mixer_case(b, blk, n, 1, 7), bytes_=n * 2.0 * H * D * D * 4, shape=[n])
+
+
+def case_ssd(b: Bench):
+    """Prompts: bytes of z, x, B, C and the result (convolution and norm included); decode: the state read and written once."""
+    from tesseract_b200.nn.hybrid import SSD
+    H, E, N = 128, 64, 128
+    blk = SSD(64, H, E, N, 1, 4, 1, 1e-6, torch.bfloat16, b.dev)
+    blk.w.conv.uniform_(-0.5, 0.5)
+    blk.w.dt_bias.uniform_(-4.0, -2.0)
+    for n, rows in ((4, 4096), (1, 4096), (32, 512)):
+        report("ssd_prefill", _mixer_case(b, blk, n, rows), bytes_=n * rows * (3 * H * E + 2 * N) * 2.0, shape=[n, rows])
+    for n in (256, 32):
+        report("ssd_step", _mixer_case(b, blk, n, 1, 7), bytes_=n * 2.0 * H * E * N * 4, shape=[n])
+
+
+def case_post_norm(b: Bench):
+    from tesseract_b200 import ops
+    T, W = 16384, 4096
+    x, y, gain = torch.randn(T, W, device=b.dev, generator=b.gen), b.randn(T, W), torch.ones(W, device=b.dev)
+    report("post_norm_step", b.time(lambda: ops.post_norm_step(x, y, gain, 1e-6)), bytes_=T * W * 12.0, shape=[T, W])
+
+
+def case_token_side(b: Bench):
+    """The side input of 4096-wide layers, 128 columns per layer: bytes of the normed input, the looked-up row, x in and out."""
+    from tesseract_b200 import ops
+    from tesseract_b200.nn.hybrid import TokenSide
+    W, V, dim = 4096, 32768, 128
+    side = TokenSide(W, dim, 1e-6, torch.bfloat16, b.dev)
+    side.w_gate.normal_(std=0.02)
+    side.w_proj.normal_(std=0.02)
+    table = b.randn(V, dim)
+    for T in (16384, 256, 32):
+        toks = torch.randint(0, V, (T,), device=b.dev, generator=b.gen, dtype=torch.int32)
+        x, h = torch.randn(T, W, device=b.dev, generator=b.gen), b.randn(T, W)
+        ms = b.time(lambda: ops.post_norm_step(x, side.forward(h, toks, table, 0), side.norm.gain, 1e-6))
+        report("token_side", ms, bytes_=T * (W * 12.0 + dim * 2) + 2 * W * dim * 2.0, shape=[T, W, dim])
+
+
+def case_token_shift(b: Bench):
+    from tesseract_b200.nn.hybrid import TimeMix
+    from tesseract_b200.ops.timemix import token_shift
+    W = 4096
+    blk = TimeMix(W, 64, 64, 64, 1e-6, torch.bfloat16, b.dev)
+    st = _Step(b, blk.run_spec(), 4, 4096)
+    h = b.randn(4 * 4096, W)
+    ms = b.time(lambda: token_shift(h, blk.mu, st.cache.runs[0][0], st.batch, keep=True))
+    report("token_shift", ms, bytes_=h.numel() * 2.0 * 7, shape=[4, 4096, W])
+
+
+def case_project_inputs(b: Bench):
+    """One product over six inputs (the first of 6272 columns) against the same product over one."""
+    from tesseract_b200 import ops
+    starts = (0, 6400, 10496, 14592, 18688, 22784)
+    w = b.randn(22848, 4096, scale=0.02)
+    for M in (16384, 256, 32):
+        xs = b.randn(6, M, 4096)
+        kw = dict(flops=2.0 * M * w.shape[0] * 4096) if M > 256 else dict(bytes_=w.numel() * 2.0)
+        report("project_inputs", b.time(lambda: ops.project_inputs(xs, w, starts)), shape=[M, w.shape[0], 4096], **kw)
+        report("project_one", b.time(lambda: ops.project(xs[0], w)), shape=[M, w.shape[0], 4096], **kw)
+
+
 CASES = {"gemm": case_gemm, "gemm_fp8": case_gemm_fp8, "gemm_fp8_pertensor": case_gemm_fp8_pertensor, "decode_gemm": case_decode_gemm, "gemm_wgrad": case_gemm_wgrad, "grouped_gemm": case_grouped_gemm,
          "flash_fwd": case_flash_fwd, "flash_bwd": case_flash_bwd, "decode": case_decode,
          "decode_int8": case_decode_int8, "rmsnorm": case_rmsnorm, "swiglu": case_swiglu, "swiglu_bwd": case_swiglu_bwd, "adam": case_adam,
@@ -566,7 +668,9 @@ CASES = {"gemm": case_gemm, "gemm_fp8": case_gemm_fp8, "gemm_fp8_pertensor": cas
          "ag_gemm_emul": case_ag_gemm_emul, "stream_linear": case_stream_linear, "mx_linear": case_mx_linear, "gemm_mx": case_gemm_mx,
          "delta_prefill": case_delta_prefill, "delta_step": case_delta_step, "chunk_attn": case_chunk_attn,
          "dyn_tanh": case_dyn_tanh, "clamped_glu": case_clamped_glu, "retention": case_retention, "latent": case_latent, "rglru": case_rglru,
-         "depth_residual": case_depth_residual, "silu_glu": case_silu_glu}
+         "depth_residual": case_depth_residual, "silu_glu": case_silu_glu, "shaped_attn": case_shaped_attn, "time_mix": case_time_mix,
+         "ssd": case_ssd, "post_norm": case_post_norm, "token_side": case_token_side, "token_shift": case_token_shift,
+         "project_inputs": case_project_inputs}
 
 
 def main():

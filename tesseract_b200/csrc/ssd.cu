@@ -1,10 +1,18 @@
 // State-space duality (a matrix state per head with a scalar decay per token), for ragged batches:
 //
 //   S_t = exp(-exp(A_log) dt) S_(t-1) + (dt x_t) B_t^T,  y_t = S_t C_t + D x_t                      per head, S [vdim][state]
-//   t = y * silu(z), then normed in equal parts (part_norm_kernel)
+//   out = y * silu(z), normed in equal parts (part_norm_kernel)
 //
 // x, B and C pass a short causal convolution with bias and SiLU (ssd_conv_kernel, which also turns the dt projection into dt and
 // the logarithm of the decay); heads share the B and C of their group. The state and what decays it are fp32.
+//
+// Prompts in bf16 run on the tensor cores in the chunked form (ssd_chunk_kernel), 64 tokens at a time, L_i the sum of the
+// logarithms up to token i of the chunk:
+//   y_i = exp(L_i) S C_i + sum_{j <= i} exp(L_i - L_j) dt_j (B_j . C_i) x_j + D x_i
+//   S  <- exp(L_63) S + sum_j (exp(L_63 - L_j) dt_j x_j) B_j^T
+// S stays in the accumulators of the products (values on rows), which is also the layout in which it enters the read-out. S, the
+// decayed scores and the decayed x go in as two bf16 halves (16 bits); B, C and x are bf16 as the convolution leaves them.
+// fp32 models take ssd_scan_kernel (token by token), decoded tokens ssd_step_kernel.
 #include "linear_state.cuh"
 #include "ragged_conv.cuh"
 
@@ -34,7 +42,7 @@ struct SsdParams {
   const int* pos0;
   const int* blk_seq;
   const int* blk0;
-  void* out;                 // [rows, ldo]
+  void* out;                 // [rows, ldo]: y
 };
 
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
@@ -111,7 +119,7 @@ ssd_conv_kernel(SsdParams p) {
   }
 }
 
-// ------------------------------------------------------------------ prompts token by token (fp32 models, wide heads)
+// ------------------------------------------------------------------ prompts token by token (fp32 models)
 template <typename T, int RL>
 __global__ void __launch_bounds__(128)
 ssd_scan_kernel(SsdParams p) {
@@ -124,7 +132,6 @@ ssd_scan_kernel(SsdParams p) {
   const T* xbc = static_cast<const T*>(p.xbc) + static_cast<long long>(row0) * p.conv_c;
   const float2* gates = p.gates + static_cast<long long>(row0) * p.H + h;
   const T *x = xbc + h * p.vp, *B = xbc + p.H * p.vp + grp * p.np, *C = B + p.G * p.np;
-  const T* z = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ld + h * p.vp;
   T* out = static_cast<T*>(p.out) + static_cast<long long>(row0) * p.ldo + h * p.vp;
   const float skip = p.d[h];
   state_scan<RL, true>(
@@ -138,10 +145,8 @@ ssd_scan_kernel(SsdParams p) {
       [&](int t, int e) { return to_f32<T>(x[static_cast<long long>(t) * p.conv_c + e]); },
       [&](int t, int e, const float (&o)[4]) {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const float y = fmaf(skip, to_f32<T>(x[static_cast<long long>(t) * p.conv_c + e + j]), o[j]);
-          out[static_cast<long long>(t) * p.ldo + e + j] = from_f32<T>(y * silu_f32(to_f32<T>(z[static_cast<long long>(t) * p.ld + e + j])));
-        }
+        for (int j = 0; j < 4; ++j)
+          out[static_cast<long long>(t) * p.ldo + e + j] = from_f32<T>(fmaf(skip, to_f32<T>(x[static_cast<long long>(t) * p.conv_c + e + j]), o[j]));
       });
 }
 
@@ -173,32 +178,254 @@ ssd_step_kernel(SsdParams p) {
   state_step<LPR, PPL, RPT, true>(p.state + (static_cast<long long>(slot) * p.H + h) * p.vp * p.np, p.vp, p.np, p.positions[row] <= 0, sq, sk, sw,
                                   sv, so);
   __syncthreads();
-  const T* z = static_cast<const T*>(p.proj) + static_cast<long long>(row) * p.ld + h * p.vp;
-  for (int e = tid; e < p.vp; e += 256) out[e] = from_f32<T>(fmaf(p.d[h], sv[e], so[e]) * silu_f32(to_f32<T>(z[e])));
+  for (int e = tid; e < p.vp; e += 256) out[e] = from_f32<T>(fmaf(p.d[h], sv[e], so[e]));
 }
 
-// In place: every part of a row's logical columns over its root mean square, times weight and scale. CTA = (row, part).
-template <typename T>
-__global__ void __launch_bounds__(256)
-part_norm_kernel(T* t, long long ld, const float* weight, int vdim, int vp, int per, float eps, float scale) {
+// ------------------------------------------------------------------ prompts, bf16
+template <int NT>
+struct SsdChunk {
+  static constexpr int kTok = 64, kCols = 64, kThreads = 128;
+  static constexpr int kLdN = NT + 8, kLdX = kCols + 8;
+  // bytes: C, B, x / y, the decayed scores in two halves, step sizes and logarithms
+  static constexpr int kC = 0, kB = kTok * kLdN * 2, kX = 2 * kB, kPh = kX + kTok * kLdX * 2, kPl = kPh + kTok * kLdX * 2;
+  static constexpr int kG = kPl + kTok * kLdX * 2, kL = kG + kTok * 8, kSmem = kL + 4 * kTok * 4;
+};
+
+// CTA = (head and 64 of its value columns, sequence); warp w owns the state's rows (values) 16 w .. + 15 of them.
+template <int NT>
+__global__ void __launch_bounds__(128, NT <= 128 ? 3 : 1)
+ssd_chunk_kernel(SsdParams p) {
+  using T = __nv_bfloat16;
+  using K = SsdChunk<NT>;
   pdl_trigger();
   pdl_grid_wait();
+  extern __shared__ __align__(16) uint8_t smem[];
+  T *sc = reinterpret_cast<T*>(smem + K::kC), *sb = reinterpret_cast<T*>(smem + K::kB), *sx = reinterpret_cast<T*>(smem + K::kX);
+  T *sph = reinterpret_cast<T*>(smem + K::kPh), *spl = reinterpret_cast<T*>(smem + K::kPl);
+  const float2* sg = reinterpret_cast<const float2*>(smem + K::kG);
+  const int tiles = (p.vp + K::kCols - 1) / K::kCols, h = blockIdx.x / tiles, c0 = blockIdx.x % tiles * K::kCols;
+  const int seq = blockIdx.y, slot = p.slots[seq], grp = h / (p.H / p.G);
+  const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
+  if (slot < 0 || n <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const T* xbc = static_cast<const T*>(p.xbc) + static_cast<long long>(row0) * p.conv_c;
+  const T *x = xbc + h * p.vp + c0, *B = xbc + p.H * p.vp + grp * p.np, *C = B + p.G * p.np;
+  const float2* gates = p.gates + static_cast<long long>(row0) * p.H + h;
+  float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.vp * p.np;
+  float* sl = reinterpret_cast<float*>(smem + K::kL) + warp * K::kTok;      // (every warp has its own copy)
+  const int e0 = warp * 16, cols = min(K::kCols, p.vp - c0);
+  const float skip = p.d[h];
+  float S[NT / 8][4];
+  {
+    const bool old = p.pos0[seq] > 0;
+#pragma unroll
+    for (int j = 0; j < NT / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
+        float2 v = make_float2(0.f, 0.f);
+        if (old && r < cols && c < p.np) v = *reinterpret_cast<const float2*>(st + static_cast<long long>(c0 + r) * p.np + c);
+        S[j][2 * e] = v.x;
+        S[j][2 * e + 1] = v.y;
+      }
+  }
+  const uint32_t aC = smem_u32(sc), aB = smem_u32(sb), aX = smem_u32(sx), aPh = smem_u32(sph), aPl = smem_u32(spl);
+
+  for (int t0 = 0; t0 < n; t0 += K::kTok) {
+    const int cnt = min(K::kTok, n - t0);
+    for (int i = tid; i < K::kTok * (NT / 8); i += K::kThreads) {
+      const int r = i / (NT / 8), d = (i % (NT / 8)) * 8;
+      const bool ok = r < cnt && d < p.np;
+      const long long at = static_cast<long long>(t0 + r) * p.conv_c + d;
+      cp_async_16(aC + (r * K::kLdN + d) * 2, ok ? C + at : C, ok ? 16 : 0);
+      cp_async_16(aB + (r * K::kLdN + d) * 2, ok ? B + at : B, ok ? 16 : 0);
+    }
+    for (int i = tid; i < K::kTok * (K::kCols / 8); i += K::kThreads) {
+      const int r = i / (K::kCols / 8), d = (i % (K::kCols / 8)) * 8;
+      const bool ok = r < cnt && d < cols;
+      cp_async_16(aX + (r * K::kLdX + d) * 2, ok ? x + static_cast<long long>(t0 + r) * p.conv_c + d : x, ok ? 16 : 0);
+    }
+    if (tid < K::kTok) {
+      const bool ok = tid < cnt;
+      cp_async_8(smem_u32(sg + tid), ok ? gates + static_cast<long long>(t0 + tid) * p.H : gates, ok ? 8 : 0);
+    }
+    cp_commit();
+    cp_wait<0>();
+    __syncthreads();
+    float last;                                // L of the chunk's end
+    {
+      const float a = sg[2 * lane].y, b = sg[2 * lane + 1].y;
+      float sum = a + b;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += up;
+      }
+      sl[2 * lane] = sum - b;
+      sl[2 * lane + 1] = sum;
+      last = __shfl_sync(0xffffffffu, sum, 31);
+      __syncwarp();
+    }
+    {
+      // decayed scores: this warp's 16 keys j against the tokens i from their block on
+      float a[8][4];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j][0] = a[j][1] = a[j][2] = a[j][3] = 0.f;
+#pragma unroll 2
+      for (int ks = 0; ks < NT / 16; ++ks) {
+        uint32_t kb[4], q[4];
+        ldmat_x4(kb, aB + frag_a(lane, warp * 16, ks * 16, K::kLdN));
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          if (i < warp) continue;
+          ldmat_x4(q, aC + frag_b(lane, i * 16, ks * 16, K::kLdN));
+          mma_bf16(a[2 * i], kb, q[0], q[1]);
+          mma_bf16(a[2 * i + 1], kb, q[2], q[3]);
+        }
+      }
+      const int j0 = warp * 16 + g, j1 = j0 + 8;
+      const float l0 = sl[j0], l1 = sl[j1], d0 = sg[j0].x, d1 = sg[j1].x;
+#pragma unroll
+      for (int b = 0; b < 8; ++b) {
+        if (b < 2 * warp) continue;
+        const int i = b * 8 + 2 * t4;
+        const float la = sl[i], lb = sl[i + 1];
+        const float f0 = i >= j0 ? a[b][0] * d0 * exp2f(la - l0) : 0.f, f1 = i + 1 >= j0 ? a[b][1] * d0 * exp2f(lb - l0) : 0.f;
+        const float f2 = i >= j1 ? a[b][2] * d1 * exp2f(la - l1) : 0.f, f3 = i + 1 >= j1 ? a[b][3] * d1 * exp2f(lb - l1) : 0.f;
+        split_bf16x2(f0, f1, reinterpret_cast<uint32_t*>(sph + j0 * K::kLdX + i), reinterpret_cast<uint32_t*>(spl + j0 * K::kLdX + i));
+        split_bf16x2(f2, f3, reinterpret_cast<uint32_t*>(sph + j1 * K::kLdX + i), reinterpret_cast<uint32_t*>(spl + j1 * K::kLdX + i));
+      }
+    }
+    __syncthreads();
+    float acc[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < NT / 16; ++ks) {
+      uint32_t hi[4], lo[4];
+      split_bf16x2(S[2 * ks][0], S[2 * ks][1], &hi[0], &lo[0]);
+      split_bf16x2(S[2 * ks][2], S[2 * ks][3], &hi[1], &lo[1]);
+      split_bf16x2(S[2 * ks + 1][0], S[2 * ks + 1][1], &hi[2], &lo[2]);
+      split_bf16x2(S[2 * ks + 1][2], S[2 * ks + 1][3], &hi[3], &lo[3]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        uint32_t q[4];
+        ldmat_x4(q, aC + frag_b(lane, i * 16, ks * 16, K::kLdN));
+        mma_bf16(acc[2 * i], hi, q[0], q[1]);
+        mma_bf16(acc[2 * i + 1], hi, q[2], q[3]);
+        mma_bf16(acc[2 * i], lo, q[0], q[1]);
+        mma_bf16(acc[2 * i + 1], lo, q[2], q[3]);
+      }
+    }
+#pragma unroll
+    for (int b = 0; b < 8; ++b) {
+      const float la = exp2f(sl[b * 8 + 2 * t4]), lb = exp2f(sl[b * 8 + 2 * t4 + 1]);
+      acc[b][0] *= la; acc[b][1] *= lb; acc[b][2] *= la; acc[b][3] *= lb;
+    }
+    const float whole = exp2f(last);
+#pragma unroll
+    for (int j = 0; j < NT / 8; ++j) {
+      S[j][0] *= whole; S[j][1] *= whole; S[j][2] *= whole; S[j][3] *= whole;
+    }
+#pragma unroll
+    for (int jb = 0; jb < 4; ++jb) {
+      if (jb * 16 >= cnt) break;
+      uint32_t xt[4], hi[4], lo[4];
+      ldmat_x4_trans(xt, aX + frag_a_trans(lane, jb * 16, e0, K::kLdX));
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (i < jb) continue;
+        uint32_t ph[4], pl[4];
+        ldmat_x4_trans(ph, aPh + frag_b_trans(lane, jb * 16, i * 16, K::kLdX));
+        ldmat_x4_trans(pl, aPl + frag_b_trans(lane, jb * 16, i * 16, K::kLdX));
+        mma_bf16(acc[2 * i], xt, ph[0], ph[1]);
+        mma_bf16(acc[2 * i + 1], xt, ph[2], ph[3]);
+        mma_bf16(acc[2 * i], xt, pl[0], pl[1]);
+        mma_bf16(acc[2 * i + 1], xt, pl[2], pl[3]);
+      }
+      float w[4];                              // what the chunk's end sees of tokens 16 jb + 2 t, + 1, + 8, + 9
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int j = jb * 16 + 2 * t4 + (e & 1) + (e >> 1) * 8;
+        w[e] = sg[j].x * exp2f(last - sl[j]);
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(&xt[e]);
+        split_bf16x2(__low2float(v) * w[e & 2], __high2float(v) * w[(e & 2) + 1], &hi[e], &lo[e]);
+      }
+#pragma unroll
+      for (int j = 0; j < NT / 8; j += 2) {
+        uint32_t b[4];
+        ldmat_x4_trans(b, aB + frag_b_trans(lane, jb * 16, j * 8, K::kLdN));
+        mma_bf16(S[j], hi, b[0], b[1]);
+        mma_bf16(S[j + 1], hi, b[2], b[3]);
+        mma_bf16(S[j], lo, b[0], b[1]);
+        mma_bf16(S[j + 1], lo, b[2], b[3]);
+      }
+    }
+    // y takes the place of x (a warp's own columns)
+    __syncwarp();
+#pragma unroll
+    for (int b = 0; b < 8; ++b)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        T* at = sx + (b * 8 + 2 * t4 + (e & 1)) * K::kLdX + e0 + g + 8 * (e >> 1);
+        *at = from_f32<T>(fmaf(skip, to_f32<T>(*at), acc[b][e]));
+      }
+    __syncwarp();
+    T* out = static_cast<T*>(p.out) + static_cast<long long>(row0 + t0) * p.ldo + h * p.vp + c0 + e0;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = i * 16 + (lane >> 1), d = (lane & 1) * 8;
+      if (r < cnt && e0 + d < cols)
+        *reinterpret_cast<uint4*>(out + static_cast<long long>(r) * p.ldo + d) = *reinterpret_cast<const uint4*>(sx + r * K::kLdX + e0 + d);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int j = 0; j < NT / 8; ++j)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
+      if (r < cols && c < p.np)
+        *reinterpret_cast<float2*>(st + static_cast<long long>(c0 + r) * p.np + c) = make_float2(S[j][2 * e], S[j][2 * e + 1]);
+    }
+}
+
+// In place: y * silu(z), then every part of a row's logical columns over its root mean square, times weight and scale. CTA = (row,
+// part); a part of up to 256 * KEEP vectors stays in registers (VEC), other layouts go column by column.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+part_norm_kernel(T* t, long long ld, const T* z, long long ldz, const float* weight, int vdim, int vp, int per, float eps, float scale) {
+  pdl_trigger();
+  pdl_grid_wait();
+  constexpr int V = kVec16<T>, kKeep = VEC ? 4 : 1;
   __shared__ float red[8];
   const int row = blockIdx.y, j0 = blockIdx.x * per, tid = threadIdx.x, nt = blockDim.x;
   T* x = t + row * ld;
+  const T* gate = z ? z + row * ldz : nullptr;
   auto column = [&](int j) { return vp == vdim ? j : j / vdim * vp + j % vdim; };
-  float ss = 0.f;
-  const bool vec = vp == vdim && per % 8 == 0 && sizeof(T) == 2;
-  if (vec) {
-    for (int j = tid * 8; j < per; j += nt * 8) {
-      float f[kVec16<T>];
-      ld16<T>(x + j0 + j, f);
+  auto gated = [&](int c) { return to_f32<T>(x[c]) * (gate ? silu_f32(to_f32<T>(gate[c])) : 1.f); };
+  float keep[kKeep][V], ss = 0.f;
+  if constexpr (VEC) {
 #pragma unroll
-      for (int i = 0; i < kVec16<T>; ++i) ss = fmaf(f[i], f[i], ss);
+    for (int k = 0; k < kKeep; ++k) {
+      const int j = (k * nt + tid) * V;
+      if (j >= per) break;
+      ld16<T>(x + j0 + j, keep[k]);
+      if (gate) {
+        float f[V];
+        ld16<T>(gate + j0 + j, f);
+#pragma unroll
+        for (int i = 0; i < V; ++i) keep[k][i] *= sizeof(T) == 2 ? __fdividef(f[i], 1.f + __expf(-f[i])) : silu_f32(f[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss = fmaf(keep[k][i], keep[k][i], ss);
     }
   } else {
     for (int j = tid; j < per; j += nt) {
-      const float f = to_f32<T>(x[column(j0 + j)]);
+      const float f = gated(column(j0 + j));
       ss = fmaf(f, f, ss);
     }
   }
@@ -208,18 +435,22 @@ part_norm_kernel(T* t, long long ld, const float* weight, int vdim, int vp, int 
   ss = 0.f;
   for (int w = 0; w < nt / 32; ++w) ss += red[w];
   const float r = scale / sqrtf(ss / static_cast<float>(per) + eps);
-  if (vec) {
-    for (int j = tid * 8; j < per; j += nt * 8) {
-      float f[kVec16<T>];
-      ld16<T>(x + j0 + j, f);
+  if constexpr (VEC) {
 #pragma unroll
-      for (int i = 0; i < kVec16<T>; ++i) f[i] *= r * weight[j0 + j + i];
-      st16<T>(x + j0 + j, f);
+    for (int k = 0; k < kKeep; ++k) {
+      const int j = (k * nt + tid) * V;
+      if (j >= per) break;
+#pragma unroll
+      for (int i = 0; i < V; i += 4) {
+        const float4 w = *reinterpret_cast<const float4*>(weight + j0 + j + i);
+        keep[k][i] *= r * w.x; keep[k][i + 1] *= r * w.y; keep[k][i + 2] *= r * w.z; keep[k][i + 3] *= r * w.w;
+      }
+      st16<T>(x + j0 + j, keep[k]);
     }
   } else {
     for (int j = tid; j < per; j += nt) {
       const int c = column(j0 + j);
-      x[c] = from_f32<T>(to_f32<T>(x[c]) * r * weight[c]);
+      x[c] = from_f32<T>(gated(c) * r * weight[c]);
     }
   }
 }
@@ -259,6 +490,20 @@ int run_scan(const SsdParams& p, cudaStream_t s) {
   if (p.np <= 64) launch_pdl(ssd_scan_kernel<T, 2>, grid, dim3(128), 0, s, pdl, p);
   else if (p.np <= 128) launch_pdl(ssd_scan_kernel<T, 4>, grid, dim3(128), 0, s, pdl, p);
   else launch_pdl(ssd_scan_kernel<T, 8>, grid, dim3(128), 0, s, pdl, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int NT>
+int run_chunk(const SsdParams& p, cudaStream_t s) {
+  auto kern = ssd_chunk_kernel<NT>;
+  static PerDeviceFlag attr;
+  if (attr.unset()) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SsdChunk<NT>::kSmem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    attr.set();
+  }
+  const int tiles = (p.vp + SsdChunk<NT>::kCols - 1) / SsdChunk<NT>::kCols;
+  launch_pdl(kern, dim3(p.H * tiles, p.n_seq), dim3(SsdChunk<NT>::kThreads), SsdChunk<NT>::kSmem, s, pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -329,29 +574,36 @@ TSB_EXPORT int tsb_ssd_prefill(const int* ints, void* const* q, int dtype, void*
   p.proj = q[0]; p.xbc = q[1]; p.gates = static_cast<float2*>(q[2]); p.d = static_cast<const float*>(q[3]); p.state = static_cast<float*>(q[4]);
   p.slots = static_cast<const int*>(q[5]); p.cu = static_cast<const int*>(q[6]); p.pos0 = static_cast<const int*>(q[7]); p.out = q[8];
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == 1) return run_scan<__nv_bfloat16>(p, s);
+  if (dtype == 1) {
+    if (p.ldo % 8 || (reinterpret_cast<uintptr_t>(p.out) & 15)) return -2;
+    return p.np <= 64 ? run_chunk<64>(p, s) : p.np <= 128 ? run_chunk<128>(p, s) : run_chunk<256>(p, s);
+  }
   if (dtype == 0) return run_scan<float>(p, s);
   return -2;
 }
 
-// t [rows, ld] in place; see part_norm_kernel. dtype: 0 = fp32, 1 = bf16.
-TSB_EXPORT int tsb_part_norm(void* t, long long ld, const float* weight, int rows, int heads, int vdim, int vp, int parts, float eps,
-                             float scale, int dtype, void* stream) {
+// t [rows, ld] in place, z [rows, ldz] or null; see part_norm_kernel. dtype: 0 = fp32, 1 = bf16.
+TSB_EXPORT int tsb_part_norm(void* t, long long ld, const void* z, long long ldz, const float* weight, int rows, int heads, int vdim, int vp,
+                             int parts, float eps, float scale, int dtype, void* stream) {
   using namespace tsb;
-  if (rows <= 0 || heads <= 0 || vdim <= 0 || vp < vdim || parts <= 0 || (heads * vdim) % parts || (dtype != 0 && dtype != 1) ||
-      (dtype == 1 && (ld % 8 || (reinterpret_cast<uintptr_t>(t) & 15))))
-    return -2;
-  const int per = heads * vdim / parts;
-  const int nt = std::min(256, (per / 8 + 31) / 32 * 32 + 32);
+  if (rows <= 0 || heads <= 0 || vdim <= 0 || vp < vdim || parts <= 0 || (heads * vdim) % parts || (dtype != 0 && dtype != 1)) return -2;
+  const int per = heads * vdim / parts, V = dtype == 1 ? 8 : 4;
+  auto off = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) != 0; };
+  const bool vec = vp == vdim && per % V == 0 && per <= 1024 * V && ld % V == 0 && ldz % V == 0 && !off(t) && !off(z) && !off(weight);
+  const int lanes = vec ? (per / V + 3) / 4 : per;
+  const int nt = std::min(256, (std::max(lanes, std::min(per / V, 128)) + 31) / 32 * 32);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  for (int r0 = 0; r0 < rows; r0 += 65535) {
-    const dim3 grid(parts, std::min(rows - r0, 65535));
-    if (dtype == 1)
-      launch_pdl(part_norm_kernel<__nv_bfloat16>, grid, dim3(nt), 0, s, pdl_all_enabled(), static_cast<__nv_bfloat16*>(t) + r0 * ld, ld, weight, vdim,
-                 vp, per, eps, scale);
-    else
-      launch_pdl(part_norm_kernel<float>, grid, dim3(nt), 0, s, pdl_all_enabled(), static_cast<float*>(t) + r0 * ld, ld, weight, vdim, vp, per, eps,
-                 scale);
-  }
+  auto run = [&](auto zero) {
+    using T = decltype(zero);
+    for (int r0 = 0; r0 < rows; r0 += 65535) {
+      const dim3 grid(parts, std::min(rows - r0, 65535));
+      T* x = static_cast<T*>(t) + r0 * ld;
+      const T* gate = z ? static_cast<const T*>(z) + r0 * ldz : nullptr;
+      if (vec) launch_pdl(part_norm_kernel<T, true>, grid, dim3(nt), 0, s, pdl_all_enabled(), x, ld, gate, ldz, weight, vdim, vp, per, eps, scale);
+      else launch_pdl(part_norm_kernel<T, false>, grid, dim3(nt), 0, s, pdl_all_enabled(), x, ld, gate, ldz, weight, vdim, vp, per, eps, scale);
+    }
+  };
+  if (dtype == 1) run(__nv_bfloat16{});
+  else run(0.f);
   return static_cast<int>(cudaGetLastError());
 }

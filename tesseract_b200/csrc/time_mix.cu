@@ -5,6 +5,16 @@
 //
 // S is [values][keys] in fp32 and stays so. token_shift_kernel makes the inputs of the five projections, mixes of a row and the
 // one before it.
+//
+// Prompts in bf16 with heads of up to 128 columns run on the tensor cores (time_mix_chunk_kernel): blocks of 16 tokens, four of
+// them prepared at once. With W_i the product of the decays of the block's tokens up to i,
+//   o_i = S (W_(i-1) r_i) + sum_{j < i} (sum_d r_id k_jd W_(i-1)d / W_jd) v_j + (u k_i . r_i) v_i
+//   S  <- S diag(W_15) + sum_j v_j (k_j W_15 / W_j)^T
+// where every ratio is formed as the product of the decays in between, so nothing overflows however steep they are. S stays in the
+// accumulators of the products (values on rows), which is also the layout in which it enters the read-out. Factors that must not
+// lose their 32 bits meet the tensor cores as two bf16 halves (16 bits).
+// fp32 models and wider heads take time_mix_scan_kernel (token by token) and time_mix_norm_kernel; decoded tokens
+// time_mix_step_kernel.
 #include "linear_state.cuh"
 #include "ragged_conv.cuh"
 
@@ -162,6 +172,247 @@ time_mix_norm_kernel(MixParams p) {
   }
 }
 
+// ------------------------------------------------------------------ prompts, bf16
+template <int DT>
+struct MixChunk {
+  static constexpr int kTok = 64, kBlk = 16, kWarps = DT / 16, kThreads = kWarps * 32, kParts = DT / 64;
+  static constexpr int kLd = DT + 8, kLdO = DT + 4, kLdA = 20;
+  // bytes: r / high half of W r, k / high half of k W, v, the low halves, decay inputs / read-outs, pair sums, block decays
+  static constexpr int kTile = kTok * kLd * 2, kR = 0, kK = kTile, kV = 2 * kTile, kRl = 3 * kTile, kKl = 4 * kTile, kO = 5 * kTile;
+  static constexpr int kA = kO + kTok * kLdO * 4, kTot = kA + kParts * 4 * kBlk * kLdA * 4, kSmem = kTot + 4 * DT * 4;
+};
+
+// Sums of 32 values over the warp: lane l returns the sum of v[l].
+__device__ __forceinline__ float transpose_sum(float (&v)[32], int lane) {
+#pragma unroll
+  for (int o = 16; o; o >>= 1) {
+    const bool up = (lane & o) != 0;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      if (i >= o) break;
+      const float keep = up ? v[i + o] : v[i], give = up ? v[i] : v[i + o];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+    }
+  }
+  return v[0];
+}
+
+// CTA = (head, sequence); warp w owns the state's rows (values) 16 w .. + 15.
+template <int DT>
+__global__ void __launch_bounds__(MixChunk<DT>::kThreads, DT == 64 ? 3 : 1)
+time_mix_chunk_kernel(MixParams p) {
+  using T = __nv_bfloat16;
+  using C = MixChunk<DT>;
+  pdl_trigger();
+  pdl_grid_wait();
+  extern __shared__ __align__(16) uint8_t smem[];
+  T *sr = reinterpret_cast<T*>(smem + C::kR), *sk = reinterpret_cast<T*>(smem + C::kK), *sv = reinterpret_cast<T*>(smem + C::kV);
+  T *srl = reinterpret_cast<T*>(smem + C::kRl), *skl = reinterpret_cast<T*>(smem + C::kKl);
+  float *so = reinterpret_cast<float*>(smem + C::kO), *sa = reinterpret_cast<float*>(smem + C::kA), *stot = reinterpret_cast<float*>(smem + C::kTot);
+  const int h = blockIdx.x, seq = blockIdx.y, slot = p.slots[seq];
+  const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
+  if (slot < 0 || n <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const T* proj = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ld + h * p.dp;
+  const float* dec = p.dec + static_cast<long long>(row0) * p.H * p.dp + h * p.dp;
+  float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp;
+  const int e0 = warp * 16;
+  float S[DT / 8][4];
+  {
+    const bool old = p.pos0[seq] > 0;
+#pragma unroll
+    for (int j = 0; j < DT / 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
+        float2 v = make_float2(0.f, 0.f);
+        if (old && r < p.dp && c < p.dp) v = *reinterpret_cast<const float2*>(st + static_cast<long long>(r) * p.dp + c);
+        S[j][2 * e] = v.x;
+        S[j][2 * e + 1] = v.y;
+      }
+  }
+  // this thread's share of the preparation: two channels of one block of 16 tokens
+  const int blk = warp / C::kParts, part = warp % C::kParts, d0 = part * 64 + lane * 2;
+  float w0[2] = {}, uu[2] = {};
+  if (d0 < p.dp) {
+    w0[0] = p.w0[h * p.dp + d0];
+    w0[1] = p.w0[h * p.dp + d0 + 1];
+    uu[0] = p.u[h * p.dp + d0];
+    uu[1] = p.u[h * p.dp + d0 + 1];
+  }
+  const uint32_t aR = smem_u32(sr), aRl = smem_u32(srl), aK = smem_u32(sk), aKl = smem_u32(skl), aV = smem_u32(sv);
+
+  for (int t0 = 0; t0 < n; t0 += C::kTok) {
+    const int cnt = min(C::kTok, n - t0);
+    for (int i = tid; i < C::kTok * (DT / 8); i += C::kThreads) {
+      const int r = i / (DT / 8), d = (i % (DT / 8)) * 8;
+      const bool ok = r < cnt && d < p.dp;
+      const T* src = ok ? proj + static_cast<long long>(t0 + r) * p.ld + d : proj;
+      const int bytes = ok ? 16 : 0;
+      cp_async_16(aR + (r * C::kLd + d) * 2, src, bytes);
+      cp_async_16(aK + (r * C::kLd + d) * 2, ok ? src + p.section : src, bytes);
+      cp_async_16(aV + (r * C::kLd + d) * 2, ok ? src + 2 * p.section : src, bytes);
+    }
+    for (int i = tid; i < C::kTok * (DT / 4); i += C::kThreads) {
+      const int r = i / (DT / 4), d = (i % (DT / 4)) * 4;
+      const bool ok = r < cnt && d < p.dp;
+      cp_async_16(smem_u32(so + r * C::kLdO + d), ok ? dec + static_cast<long long>(t0 + r) * p.H * p.dp + d : dec, ok ? 16 : 0);
+    }
+    cp_commit();
+    cp_wait<0>();
+    __syncthreads();
+    {
+      float r[16][2], k[16][2], w[16][2];
+      const int row = blk * 16;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const __nv_bfloat162 rv = *reinterpret_cast<const __nv_bfloat162*>(sr + (row + i) * C::kLd + d0);
+        const __nv_bfloat162 kv = *reinterpret_cast<const __nv_bfloat162*>(sk + (row + i) * C::kLd + d0);
+        const float2 dv = *reinterpret_cast<const float2*>(so + (row + i) * C::kLdO + d0);
+        r[i][0] = __low2float(rv); r[i][1] = __high2float(rv);
+        k[i][0] = __low2float(kv); k[i][1] = __high2float(kv);
+        const bool real = row + i < cnt;                     // (a token that is not there decays nothing)
+        w[i][0] = real ? expf(-__expf(dv.x + w0[0])) : 1.f;
+        w[i][1] = real ? expf(-__expf(dv.y + w0[1])) : 1.f;
+      }
+      float f[2] = {1.f, 1.f};
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const int at = (row + i) * C::kLd + d0;
+        split_bf16x2(r[i][0] * f[0], r[i][1] * f[1], reinterpret_cast<uint32_t*>(sr + at), reinterpret_cast<uint32_t*>(srl + at));
+        f[0] *= w[i][0];
+        f[1] *= w[i][1];
+      }
+      *reinterpret_cast<float2*>(stot + blk * DT + d0) = make_float2(f[0], f[1]);
+      f[0] = f[1] = 1.f;
+#pragma unroll
+      for (int i = 15; i >= 0; --i) {
+        const int at = (row + i) * C::kLd + d0;
+        split_bf16x2(k[i][0] * f[0], k[i][1] * f[1], reinterpret_cast<uint32_t*>(sk + at), reinterpret_cast<uint32_t*>(skl + at));
+        f[0] *= w[i][0];
+        f[1] *= w[i][1];
+      }
+      // what token i takes of token j's value, two j at a time
+      float* a = sa + (part * 4 + blk) * C::kBlk * C::kLdA;
+#pragma unroll
+      for (int jj = 0; jj < 16; jj += 2) {
+        float v[32];
+#pragma unroll
+        for (int s = 0; s < 2; ++s) {
+          const int j = jj + s;
+          float x0 = k[j][0], x1 = k[j][1];
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            if (i < j) v[s * 16 + i] = 0.f;
+            else if (i == j) v[s * 16 + i] = fmaf(r[i][0] * uu[0], k[i][0], r[i][1] * uu[1] * k[i][1]);
+            else {
+              v[s * 16 + i] = fmaf(r[i][0], x0, r[i][1] * x1);
+              x0 *= w[i][0];
+              x1 *= w[i][1];
+            }
+          }
+        }
+        a[(jj + (lane >> 4)) * C::kLdA + (lane & 15)] = transpose_sum(v, lane);
+      }
+    }
+    __syncthreads();
+#pragma unroll 1
+    for (int b = 0; b < 4; ++b) {
+      if (b * 16 >= cnt) break;
+      const int row = b * 16;
+      float acc[2][4] = {};
+#pragma unroll
+      for (int ks = 0; ks < DT / 16; ++ks) {
+        uint32_t hi[4], lo[4], q[4];
+        split_bf16x2(S[2 * ks][0], S[2 * ks][1], &hi[0], &lo[0]);
+        split_bf16x2(S[2 * ks][2], S[2 * ks][3], &hi[1], &lo[1]);
+        split_bf16x2(S[2 * ks + 1][0], S[2 * ks + 1][1], &hi[2], &lo[2]);
+        split_bf16x2(S[2 * ks + 1][2], S[2 * ks + 1][3], &hi[3], &lo[3]);
+        ldmat_x4(q, aR + frag_b(lane, row, ks * 16, C::kLd));
+        mma_bf16(acc[0], hi, q[0], q[1]);
+        mma_bf16(acc[1], hi, q[2], q[3]);
+        mma_bf16(acc[0], lo, q[0], q[1]);
+        mma_bf16(acc[1], lo, q[2], q[3]);
+        ldmat_x4(q, aRl + frag_b(lane, row, ks * 16, C::kLd));
+        mma_bf16(acc[0], hi, q[0], q[1]);
+        mma_bf16(acc[1], hi, q[2], q[3]);
+      }
+      uint32_t vt[4];
+      ldmat_x4_trans(vt, aV + frag_a_trans(lane, row, e0, C::kLd));
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        uint32_t hi[2], lo[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          float x[2] = {};
+#pragma unroll
+          for (int q = 0; q < C::kParts; ++q) {
+            const float* a = sa + ((q * 4 + b) * C::kBlk + e * 8 + 2 * t4) * C::kLdA + c * 8 + g;
+            x[0] += a[0];
+            x[1] += a[C::kLdA];
+          }
+          split_bf16x2(x[0], x[1], &hi[e], &lo[e]);
+        }
+        mma_bf16(acc[c], vt, hi[0], hi[1]);
+        mma_bf16(acc[c], vt, lo[0], lo[1]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) so[(row + c * 8 + 2 * t4 + (e & 1)) * C::kLdO + e0 + g + 8 * (e >> 1)] = acc[c][e];
+      }
+#pragma unroll
+      for (int j = 0; j < DT / 8; j += 2) {
+        uint32_t kh[4], kl[4];
+        ldmat_x4_trans(kh, aK + frag_b_trans(lane, row, j * 8, C::kLd));
+        ldmat_x4_trans(kl, aKl + frag_b_trans(lane, row, j * 8, C::kLd));
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          const float2 f = *reinterpret_cast<const float2*>(stot + b * DT + (j + c) * 8 + 2 * t4);
+          S[j + c][0] *= f.x; S[j + c][1] *= f.y; S[j + c][2] *= f.x; S[j + c][3] *= f.y;
+          mma_bf16(S[j + c], vt, kh[2 * c], kh[2 * c + 1]);
+          mma_bf16(S[j + c], vt, kl[2 * c], kl[2 * c + 1]);
+        }
+      }
+    }
+    __syncthreads();
+    // norm and gate: a warp per row, two (four) columns per lane
+    constexpr int kRows = C::kTok / C::kWarps;
+#pragma unroll 4
+    for (int i = 0; i < kRows; ++i) {
+      const int r = i * C::kWarps + warp;
+      if (r >= cnt) break;
+      const T* gate = proj + static_cast<long long>(t0 + r) * p.ld + 3 * p.section;
+      T* out = static_cast<T*>(p.out) + static_cast<long long>(row0 + t0 + r) * p.ldo + h * p.dp;
+      float2 o[C::kParts];
+      __nv_bfloat162 gv[C::kParts];
+      float ss = 0.f;
+#pragma unroll
+      for (int q = 0; q < C::kParts; ++q) {
+        const int d = q * 64 + lane * 2;
+        gv[q] = *reinterpret_cast<const __nv_bfloat162*>(gate + min(d, p.dp - 2));
+        o[q] = *reinterpret_cast<const float2*>(so + r * C::kLdO + d);
+        ss = fmaf(o[q].x, o[q].x, fmaf(o[q].y, o[q].y, ss));
+      }
+      const float rs = p.out_scale * rsqrtf(warp_sum(ss) / static_cast<float>(p.dim) + p.eps);
+#pragma unroll
+      for (int q = 0; q < C::kParts; ++q) {
+        const int d = q * 64 + lane * 2;
+        if (d >= p.dp) continue;
+        const float2 nm = *reinterpret_cast<const float2*>(p.norm + h * p.dp + d);
+        const float g0 = __low2float(gv[q]), g1 = __high2float(gv[q]);
+        *reinterpret_cast<uint32_t*>(out + d) = pack_bf16x2(o[q].x * rs * nm.x * __fdividef(g0, 1.f + __expf(-g0)),
+                                                            o[q].y * rs * nm.y * __fdividef(g1, 1.f + __expf(-g1)));
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int j = 0; j < DT / 8; ++j)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
+      if (r < p.dp && c < p.dp) *reinterpret_cast<float2*>(st + static_cast<long long>(r) * p.dp + c) = make_float2(S[j][2 * e], S[j][2 * e + 1]);
+    }
+}
+
 // Decoded rows: CTA = (row, head).
 template <typename T, int LPR, int PPL, int RPT>
 __global__ void __launch_bounds__(256)
@@ -229,6 +480,19 @@ int run_scan(const MixParams& p, cudaStream_t s) {
   else launch_pdl(time_mix_scan_kernel<T, 8>, grid, dim3(128), 0, s, pdl, p);
   const long long warps = static_cast<long long>(p.rows) * p.H;
   launch_pdl(time_mix_norm_kernel<T>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, s, pdl, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int DT>
+int run_chunk(const MixParams& p, cudaStream_t s) {
+  auto kern = time_mix_chunk_kernel<DT>;
+  static PerDeviceFlag attr;
+  if (attr.unset()) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, MixChunk<DT>::kSmem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    attr.set();
+  }
+  launch_pdl(kern, dim3(p.H, p.n_seq), dim3(MixChunk<DT>::kThreads), MixChunk<DT>::kSmem, s, pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -304,7 +568,7 @@ TSB_EXPORT int tsb_time_mix_step(const int* ints, void* const* q, float eps, flo
   return -2;
 }
 
-// ptrs: proj, dec, w0, u, norm, state, slots, cu, pos0, out, o ([rows, H, dp] fp32).
+// ptrs: proj, dec, w0, u, norm, state, slots, cu, pos0, out, o ([rows, H, dp] fp32; null: bf16 on the tensor cores, dp <= 128).
 TSB_EXPORT int tsb_time_mix_prefill(const int* ints, void* const* q, float eps, float out_scale, int dtype, void* stream) {
   using namespace tsb;
   MixParams p{};
@@ -313,8 +577,11 @@ TSB_EXPORT int tsb_time_mix_prefill(const int* ints, void* const* q, float eps, 
   p.norm = static_cast<const float*>(q[4]); p.state = static_cast<float*>(q[5]); p.slots = static_cast<const int*>(q[6]);
   p.cu = static_cast<const int*>(q[7]); p.pos0 = static_cast<const int*>(q[8]); p.out = q[9]; p.o = static_cast<float*>(q[10]);
   p.eps = eps; p.out_scale = out_scale;
-  if (!p.o) return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (!p.o) {
+    if (dtype != 1 || p.dp > 128 || p.ldo % 2) return -2;
+    return p.dp <= 64 ? run_chunk<64>(p, s) : run_chunk<128>(p, s);
+  }
   if (dtype == 1) return run_scan<__nv_bfloat16>(p, s);
   if (dtype == 0) return run_scan<float>(p, s);
   return -2;

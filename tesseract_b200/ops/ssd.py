@@ -21,7 +21,7 @@ _native.register_signatures({
     "tsb_ssd_conv": [P, P, I, P],
     "tsb_ssd_step": [P, P, I, P],
     "tsb_ssd_prefill": [P, P, I, P],
-    "tsb_part_norm": [P, L, P, I, I, I, I, I, F, F, I, P],
+    "tsb_part_norm": [P, L, P, L, P, I, I, I, I, I, F, F, I, P],
 })
 MAX_STATE = 256
 MAX_TAPS = 8
@@ -104,17 +104,21 @@ class SSDWeights:
     eps: float
 
 
-def part_norm_(t: torch.Tensor, weight: torch.Tensor, heads: int, vdim: int, vp: int, parts: int, eps: float, scale: float) -> torch.Tensor:
-    """In place on t [T, >= heads * vp], heads of ``vdim`` columns stored ``vp`` apart: each of ``parts`` equal runs of the logical
-    columns over its root mean square, times weight [heads * vp] and ``scale``."""
+def part_norm_(t: torch.Tensor, z, weight: torch.Tensor, heads: int, vdim: int, vp: int, parts: int, eps: float, scale: float) -> torch.Tensor:
+    """In place on t [T, >= heads * vp], heads of ``vdim`` columns stored ``vp`` apart: t * silu(z) (z laid out like t, or None), then
+    each of ``parts`` equal runs of the logical columns over its root mean square, times weight [heads * vp] and ``scale``."""
     T = t.shape[0]
     if T == 0:
         return t
     if t.is_cuda:
-        check(lib().tsb_part_norm(t.data_ptr(), t.stride(0), weight.data_ptr(), T, heads, vdim, vp, parts, float(eps), float(scale),
+        check(lib().tsb_part_norm(t.data_ptr(), t.stride(0), z.data_ptr() if z is not None else None,
+                                  z.stride(0) if z is not None else 0, weight.data_ptr(), T, heads, vdim, vp, parts, float(eps), float(scale),
                                   dtype_code(t.dtype), stream_ptr(t.device)), "tsb_part_norm")
         return t
-    x = t[:, :heads * vp].float().clone().view(T, heads, vp)
+    x = t[:, :heads * vp].float().clone()
+    if z is not None:
+        x *= torch.nn.functional.silu(z[:, :heads * vp].float())
+    x = x.view(T, heads, vp)
     flat = x[:, :, :vdim].reshape(T, parts, -1)
     flat = (flat / torch.sqrt((flat * flat).mean(-1, keepdim=True) + eps)).view(T, heads, vdim) * scale
     x[:, :, :vdim] = flat * weight.view(heads, vp)[:, :vdim]
@@ -158,7 +162,7 @@ def ssd(proj: torch.Tensor, geo: SSDGeometry, w: SSDWeights, conv_state: torch.T
                                          out[nd:].data_ptr())
             check(lib().tsb_ssd_prefill(ints, ptrs, dt, st), "tsb_ssd_prefill")
             _native.add_launches(2 if nd and geo.taps > 1 else 1 if nd or geo.taps > 1 else 0)
-    return part_norm_(out, w.norm, H, geo.vdim, geo.vp, geo.norm_parts, w.eps, out_scale)
+    return part_norm_(out, proj, w.norm, H, geo.vdim, geo.vp, geo.norm_parts, w.eps, out_scale)
 
 
 def _ssd_torch(proj, geo, w, conv_state, state, batch, out):
@@ -184,5 +188,4 @@ def _ssd_torch(proj, geo, w, conv_state, state, batch, out):
             S = decay[t][:, None, None] * S + (dt[t][:, None] * xv[t])[:, :, None] * B[t][:, None, :]
             y[t] = (S * C[t][:, None, :]).sum(-1) + w.d[:, None] * xv[t]
         state[slot] = S
-        z = p[:, :X].view(n, H, E)
-        out[row0:row0 + n, :X] = (y * torch.nn.functional.silu(z)).reshape(n, X).to(out.dtype)
+        out[row0:row0 + n, :X] = y.reshape(n, X).to(out.dtype)

@@ -24,6 +24,7 @@ _native.register_signatures({
     "tsb_time_mix_prefill": [P, P, F, F, I, P],
 })
 MAX_DIM = 256
+CHUNK_DIM = 128          # widest heads of the tensor-core kernel
 STREAMS = "rkvgw"
 
 
@@ -141,12 +142,13 @@ def time_mix(proj: torch.Tensor, geo: TimeMixGeometry, w: TimeMixWeights, state:
     if n:
         pr = proj[nd:]
         dec = project(torch.tanh(pr[:, 4 * geo.section:geo.cols].float()).to(proj.dtype), w.w2, out_dtype=torch.float32)
-        o = torch.empty((n, geo.heads, geo.dp), device=proj.device, dtype=torch.float32)
+        chunked = proj.dtype == torch.bfloat16 and geo.dp <= CHUNK_DIM
+        o = None if chunked else torch.empty((n, geo.heads, geo.dp), device=proj.device, dtype=torch.float32)
         ptrs = (ctypes.c_void_p * 11)(pr.data_ptr(), dec.data_ptr(), w.w0.data_ptr(), w.u.data_ptr(), w.norm.data_ptr(), state.data_ptr(),
-                                      batch.state_slots[nd:].data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(), out[nd:].data_ptr(), o.data_ptr())
+                                      batch.state_slots[nd:].data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(), out[nd:].data_ptr(), _ptr(o))
         check(lib().tsb_time_mix_prefill(geo.ints(n, batch.n_prompts, proj.stride(0), out.stride(0)), ptrs, float(w.eps),
                                          float(out_scale), dt, st), "tsb_time_mix_prefill")
-        _native.add_launches(1)
+        _native.add_launches(0 if chunked else 1)
     return out
 
 

