@@ -375,7 +375,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     bool ok = true;
     const int row_limit = qi + offset;  // last visible key under causal masking
     const ScoreLog2 score(p.form, FORM ? h : 0);
-    const float mul = FORM ? 1.f : p.scale_log2;
+    // scores that are only scaled stay as the product leaves them; others go back in units of log 2
+    const bool raw = !FORM || (score.cap == 0.f && score.slope == 0.f);
+    const float mul = raw ? p.scale_log2 : 1.f;
 
     for (int j = 0; j < n_tiles; ++j) {
       const int st = j & 1;
@@ -383,7 +385,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       tc_fence_after();
       const uint32_t s_addr = tmem_base + lane_addr + (st ? Cfg::kColS1 : Cfg::kColS0);
       const int c0 = (FORM ? j0 + j : j) * BKV;
-      const bool need_mask = !FORM && ((p.causal && c0 + BKV - 1 > q0 + offset) || (c0 + BKV > p.Sk));
+      const bool need_mask = raw && ((p.causal && c0 + BKV - 1 > q0 + offset) || (c0 + BKV > p.Sk) ||
+                                     (FORM && p.form.window > 0 && c0 < q0 + BQ + offset - p.form.window));
+      const int lo = FORM && p.form.window > 0 ? row_limit - p.form.window + 1 - c0 : 0;      // first visible column
       int vis = BKV;  // number of visible columns of this tile for this row
       if (need_mask) {
         int lim = p.Sk - c0;
@@ -392,9 +396,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       }
       // pass 1: row maximum (tiles that need no masking skip the per-element visibility test)
       float m_tile = -INFINITY;
-      if constexpr (FORM) {
+      if (FORM && !raw) {
         const int hi = min(p.Sk - 1, row_limit) - c0;                                    // visible columns: lo .. hi
-        const int lo = p.form.window > 0 ? row_limit - p.form.window + 1 - c0 : 0;
 #pragma unroll 1
         for (int c = 0; c < BKV / 32; ++c) {
           uint32_t r[32];
@@ -418,7 +421,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (c * 32 + i < vis) m_tile = fmaxf(m_tile, __uint_as_float(r[i]));
+            if (c * 32 + i < vis && (!FORM || c * 32 + i >= lo)) m_tile = fmaxf(m_tile, __uint_as_float(r[i]));
         }
       } else {
 #pragma unroll 1
@@ -464,8 +467,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         if (need_mask) {
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
-            float p0 = (c * 32 + i < vis) ? exp2f(fmaf(__uint_as_float(r[i]), p.scale_log2, mneg)) : 0.f;
-            float p1 = (c * 32 + i + 1 < vis) ? exp2f(fmaf(__uint_as_float(r[i + 1]), p.scale_log2, mneg)) : 0.f;
+            float p0 = (c * 32 + i < vis && (!FORM || c * 32 + i >= lo)) ? exp2f(fmaf(__uint_as_float(r[i]), p.scale_log2, mneg)) : 0.f;
+            float p1 = (c * 32 + i + 1 < vis && (!FORM || c * 32 + i + 1 >= lo)) ? exp2f(fmaf(__uint_as_float(r[i + 1]), p.scale_log2, mneg)) : 0.f;
             // the denominator sums what the tensor core will actually multiply (bf16-rounded P)
             const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
             const float2 pf = __bfloat1622float2(pb);
@@ -524,7 +527,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     if (ok && qi < p.Sq) {
       float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
       if constexpr (FORM) {
-        if (p.form.sink && l_run > 0.f) inv_l = 1.f / (l_run + exp2f(p.form.sink[h] * kLog2e - m_run));
+        if (p.form.sink && l_run > 0.f) inv_l = 1.f / (l_run + exp2f(p.form.sink[h] * kLog2e - m_run * mul));
         if (p.gate.kind != 2) inv_l *= p.gate.factor<__nv_bfloat16>(row0 + qi, h, D, 0);
         else {
           const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(p.gate.gate) + static_cast<long long>(row0 + qi) * p.gate.ld + h * D;
@@ -562,6 +565,293 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   tc_fence_before();
   __syncthreads();
   if (warp == 5) {
+    if (cta_abort) {
+      for (int i = 0; i < 1000; ++i) __nanosleep(1000);
+    }
+    tc_fence_after();
+    tmem_dealloc(tmem_base, Cfg::kTmemCols);
+  }
+}
+
+// ------------------------------------------------------------------ scores with a known upper bound
+// With a bound M on the scores (capped ones, or products of unit vectors) every exponent refers to M and the softmax needs no
+// maxima: a key tile is read from TMEM once, the output accumulates in TMEM over all tiles, and tiles do not wait for one another.
+// Two groups of four softmax warps take the even and the odd tiles, each with a probability tile of its own.
+//   warps 0-3, 4-7  softmax; at the end each group stores half of the output's columns
+//   warp 8          TMA producer        warp 9   allocates TMEM, issues the MMAs
+// The caller makes sure that exp(score - M) stays far from underflow for a row's largest score.
+constexpr int kBoundedThreads = 320;
+
+template <int D>
+struct BoundedCfg {
+  static constexpr int kHalves = D / 64, kTileBytes = 128 * D * 2, kPBytes = BQ * BKV * 2;
+  static constexpr int kSmemBytes = kTileBytes * 5 + 2 * kPBytes + 1024;
+  static constexpr int kTmemCols = 512, kColO = 256;
+};
+
+__device__ __forceinline__ float2 mul_f32x2(float2 a, float2 b) {
+  float2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(d))
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
+  return d;
+}
+__device__ __forceinline__ float2 fma_f32x2(float2 a, float2 b, float2 c) {
+  float2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<unsigned long long&>(d))
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)),
+        "l"(reinterpret_cast<unsigned long long&>(c)));
+  return d;
+}
+__device__ __forceinline__ float exp2_ftz(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float2 both(float x) { return make_float2(x, x); }
+
+// tanh of both by its Taylor series up to x^11: off by 5e-7 at |x| = 1/2.
+__device__ __forceinline__ float2 tanh_series(float2 x) {
+  const float2 q = mul_f32x2(x, x);
+  float2 t = fma_f32x2(q, both(-1382.f / 155925.f), both(62.f / 2835.f));
+  t = fma_f32x2(q, t, both(-17.f / 315.f));
+  t = fma_f32x2(q, t, both(2.f / 15.f));
+  t = fma_f32x2(q, t, both(-1.f / 3.f));
+  return fma_f32x2(mul_f32x2(q, x), t, x);
+}
+
+template <int D, bool CAP>
+__global__ void __launch_bounds__(kBoundedThreads, 1)
+flash_bounded_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                     const __grid_constant__ CUtensorMap tmV, FaParams p, float bound) {
+  using Cfg = BoundedCfg<D>;
+  const int row0 = p.cu_seqlens[blockIdx.z], krow0 = p.cu_keys[blockIdx.z];
+  const int Sq = p.cu_seqlens[blockIdx.z + 1] - row0, Sk = p.cu_keys[blockIdx.z + 1] - krow0;
+  const int qt = gridDim.x - 1 - blockIdx.x, q0 = qt * BQ;       // heavy (late) query tiles first
+  if (q0 >= Sq) return;
+  const int h = blockIdx.y, hk = h / (p.H / p.Hkv), offset = Sk - Sq;
+  const int window = p.form.window;
+  const int j0 = window > 0 ? max(0, q0 + offset - window + 1) / BKV : 0;
+  const int n_tiles = max(0, min((Sk + BKV - 1) / BKV, (q0 + BQ - 1 + offset) / BKV + 1) - j0);
+
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t *sQ = smem, *sK = sQ + Cfg::kTileBytes, *sV = sK + 2 * Cfg::kTileBytes, *sP = sV + 2 * Cfg::kTileBytes;
+  __shared__ __align__(8) uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], s_free[2], p_full[2], p_free[2], o_done;
+  __shared__ float s_l[2][BQ];
+  __shared__ uint32_t tmem_base_smem;
+  __shared__ volatile int cta_abort;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    cta_abort = 0;
+    mbar_init(&q_full, 1);
+    mbar_init(&o_done, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&k_full[i], 1);
+      mbar_init(&k_empty[i], 1);
+      mbar_init(&v_full[i], 1);
+      mbar_init(&v_empty[i], 1);
+      mbar_init(&s_full[i], 1);
+      mbar_init(&s_free[i], 128);
+      mbar_init(&p_full[i], 128);
+      mbar_init(&p_free[i], 1);
+    }
+    mbar_fence_init();
+    tma_prefetch_desc(&tmQ);
+    tma_prefetch_desc(&tmK);
+    tma_prefetch_desc(&tmV);
+  }
+  if (warp == 9) {
+    tmem_alloc(&tmem_base_smem, Cfg::kTmemCols);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = tmem_base_smem;
+
+  if (warp == 8) {
+    if (lane == 0 && n_tiles > 0) {
+      mbar_expect_tx(&q_full, Cfg::kTileBytes);
+#pragma unroll
+      for (int hf = 0; hf < Cfg::kHalves; ++hf) tma_load_4d(sQ + hf * 16384, &tmQ, &q_full, hf * 64, q0 + row0, h, 0);
+      for (int j = 0; j < n_tiles; ++j) {
+        const int st = j & 1, key = (j0 + j) * BKV + krow0;
+        const uint32_t par = ((j >> 1) & 1) ^ 1u;
+        if (!mbar_wait(&k_empty[st], par, &cta_abort, p.status)) break;
+        mbar_expect_tx(&k_full[st], Cfg::kTileBytes);
+#pragma unroll
+        for (int hf = 0; hf < Cfg::kHalves; ++hf)
+          tma_load_4d(sK + st * Cfg::kTileBytes + hf * 16384, &tmK, &k_full[st], hf * 64, key, hk, 0);
+        if (!mbar_wait(&v_empty[st], par, &cta_abort, p.status)) break;
+        mbar_expect_tx(&v_full[st], Cfg::kTileBytes);
+#pragma unroll
+        for (int hf = 0; hf < Cfg::kHalves; ++hf)
+          tma_load_4d(sV + st * Cfg::kTileBytes + hf * 16384, &tmV, &v_full[st], hf * 64, key, hk, 0);
+      }
+    }
+  } else if (warp == 9) {
+    if (lane == 0 && n_tiles > 0) {
+      constexpr uint32_t idesc_s = umma_idesc(BQ, BKV, 1, 1, 0, 0), idesc_o = umma_idesc(BQ, D, 1, 1, 0, 1);
+      const uint32_t q_base = smem_u32(sQ);
+      bool ok = mbar_wait(&q_full, 0, &cta_abort, p.status);
+      auto issue_s = [&](int j) -> bool {
+        const int st = j & 1;
+        if (!mbar_wait(&k_full[st], (j >> 1) & 1, &cta_abort, p.status)) return false;
+        if (!mbar_wait(&s_free[st], ((j >> 1) & 1) ^ 1u, &cta_abort, p.status)) return false;
+        tc_fence_after();
+        const uint32_t k_base = smem_u32(sK + st * Cfg::kTileBytes), d = tmem_base + st * BKV;
+#pragma unroll
+        for (int ks = 0; ks < D / 16; ++ks)
+          umma_f16(d, kmajor_desc<128>(q_base, ks), kmajor_desc<128>(k_base, ks), idesc_s, ks != 0);
+        umma_commit(&s_full[st]);
+        umma_commit(&k_empty[st]);
+        return true;
+      };
+      if (ok) ok = issue_s(0);
+      for (int j = 0; ok && j < n_tiles; ++j) {
+        if (j + 1 < n_tiles) {
+          ok = issue_s(j + 1);
+          if (!ok) break;
+        }
+        const int st = j & 1;
+        if (!mbar_wait(&p_full[st], (j >> 1) & 1, &cta_abort, p.status)) break;
+        if (!mbar_wait(&v_full[st], (j >> 1) & 1, &cta_abort, p.status)) break;
+        tc_fence_after();
+        const uint32_t p_base = smem_u32(sP + st * Cfg::kPBytes), v_base = smem_u32(sV + st * Cfg::kTileBytes);
+#pragma unroll
+        for (int ks = 0; ks < BKV / 16; ++ks)
+          umma_f16(tmem_base + Cfg::kColO, kmajor_desc<128>(p_base, ks), mnmajor_desc(v_base, ks, 16384), idesc_o, (j | ks) != 0);
+        umma_commit(&p_free[st]);
+        umma_commit(&v_empty[st]);
+        if (j == n_tiles - 1) umma_commit(&o_done);
+      }
+    }
+  } else {
+    const int grp = warp >> 2, row = (warp & 3) * 32 + lane, qi = q0 + row, row_limit = qi + offset;
+    const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
+    const ScoreLog2 score(p.form, h);
+    const float m = bound * kLog2e;
+    // 1/2 in units of the products: the range of the series
+    const float series_to = CAP ? 0.5f / fabsf(score.mul) : 0.f;
+    float2 l2 = make_float2(0.f, 0.f);
+    bool ok = true;
+    for (int j = grp; j < n_tiles; j += 2) {
+      const uint32_t par = (j >> 1) & 1;
+      bool here = mbar_wait(&s_full[grp], par, &cta_abort, p.status);
+      here = here && mbar_wait(&p_free[grp], par ^ 1u, &cta_abort, p.status);
+      if (!__all_sync(0xffffffffu, here ? 1 : 0)) { ok = false; break; }     // (TMEM accesses are warp-collective)
+      tc_fence_after();
+      const int c0 = (j0 + j) * BKV;
+      const bool need_mask = c0 + BKV - 1 > q0 + offset || c0 + BKV > Sk || (window > 0 && c0 < q0 + BQ + offset - window);
+      const int hi = min(Sk - 1, row_limit) - c0, lo = window > 0 ? row_limit - window + 1 - c0 : 0;      // visible columns
+      const uint32_t s_addr = tmem_base + lane_addr + grp * BKV;
+#pragma unroll 1
+      for (int c = 0; c < BKV / 32; ++c) {
+        uint32_t r[32];
+        tmem_ld_32x32(s_addr + c * 32, r);
+        tmem_ld_wait();
+        if (c == BKV / 32 - 1) {
+          tc_fence_before();
+          mbar_arrive(&s_free[grp]);               // the last scores live in registers: the MMA warp may refill the buffer
+        }
+        float2 t[16];
+        const float2 mul = both(score.mul);
+        if constexpr (CAP) {
+          float top = 0.f;
+#pragma unroll
+          for (int i = 0; i < 32; ++i) top = fmaxf(top, fabsf(__uint_as_float(r[i])));
+          const float2 cap = both(score.cap), base = both(-m);
+          if (__any_sync(0xffffffffu, top > series_to)) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+              t[i].x = fmaf(score.cap, tanh_abs(__uint_as_float(r[2 * i]) * score.mul), -m);
+              t[i].y = fmaf(score.cap, tanh_abs(__uint_as_float(r[2 * i + 1]) * score.mul), -m);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 16; ++i)
+              t[i] = fma_f32x2(cap, tanh_series(mul_f32x2(make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), mul)), base);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; ++i)
+            t[i] = fma_f32x2(make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), mul, both(-m));
+        }
+        if (score.slope != 0.f) {
+          const float first = static_cast<float>(row_limit - c0 - c * 32);       // distance of the chunk's first column
+#pragma unroll
+          for (int i = 0; i < 16; ++i)
+            t[i] = fma_f32x2(both(-score.slope), make_float2(first - 2 * i, first - 2 * i - 1), t[i]);
+        }
+        if (need_mask) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const int col = c * 32 + 2 * i;
+            if (col < lo || col > hi) t[i].x = -INFINITY;
+            if (col + 1 < lo || col + 1 > hi) t[i].y = -INFINITY;
+          }
+        }
+        uint32_t packed[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float2 e = make_float2(exp2_ftz(t[i].x), exp2_ftz(t[i].y));
+          l2.x += e.x;
+          l2.y += e.y;
+          packed[i] = pack_bf16x2(e.x, e.y);
+        }
+        uint8_t* prow = sP + grp * Cfg::kPBytes + (c >> 1) * 16384 + row * 128;
+#pragma unroll
+        for (int q4 = 0; q4 < 4; ++q4)
+          *reinterpret_cast<uint4*>(prow + ((((c & 1) * 4 + q4) ^ (row & 7)) << 4)) =
+              make_uint4(packed[q4 * 4], packed[q4 * 4 + 1], packed[q4 * 4 + 2], packed[q4 * 4 + 3]);
+      }
+      fence_proxy_async_smem();
+      mbar_arrive(&p_full[grp]);
+    }
+    s_l[grp][row] = l2.x + l2.y;
+    asm volatile("bar.sync 1, 256;" ::: "memory");           // the softmax warps
+    bool have = ok && n_tiles > 0;
+    if (have) have = mbar_wait(&o_done, 0, &cta_abort, p.status);
+    if (__all_sync(0xffffffffu, have ? 1 : 0)) {
+      tc_fence_after();
+      float l = s_l[0][row] + s_l[1][row];
+      if (p.form.sink && l > 0.f) l += exp2f(fmaf(p.form.sink[h], kLog2e, -m));
+      const int at = row0 + (qi < Sq ? qi : 0);
+      float f = l > 0.f ? 1.f / l : 0.f;
+      if (p.gate.kind != 2) f *= p.gate.factor<__nv_bfloat16>(at, h, D, 0);
+      else f *= p.gate.scale;
+      const __nv_bfloat16* gate = p.gate.kind == 2 ? static_cast<const __nv_bfloat16*>(p.gate.gate) + static_cast<long long>(at) * p.gate.ld + h * D : nullptr;
+      __nv_bfloat16* orow = p.o + static_cast<long long>(at) * p.o_ss + h * p.o_sh;
+#pragma unroll
+      for (int c = grp * (D / 64); c < (grp + 1) * (D / 64); ++c) {
+        uint32_t r[32];
+        tmem_ld_32x32(tmem_base + lane_addr + Cfg::kColO + c * 32, r);
+        tmem_ld_wait();
+        if (qi < Sq) {
+#pragma unroll
+          for (int e = 0; e < 32; e += 8) {
+            float o[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(r[e + i]) * f;
+            if (gate) {
+              const uint4 gv = *reinterpret_cast<const uint4*>(gate + c * 32 + e);
+              const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                o[2 * i] = __fdividef(o[2 * i], 1.f + __expf(-__low2float(g2[i])));
+                o[2 * i + 1] = __fdividef(o[2 * i + 1], 1.f + __expf(-__high2float(g2[i])));
+              }
+            }
+            *reinterpret_cast<uint4*>(orow + c * 32 + e) =
+                make_uint4(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]), pack_bf16x2(o[4], o[5]), pack_bf16x2(o[6], o[7]));
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 9) {
     if (cta_abort) {
       for (int i = 0; i < 1000; ++i) __nanosleep(1000);
     }
@@ -646,7 +936,7 @@ static int flash_fwd_varlen(const void* q, const void* k, const void* v, void* o
                             int n_seqs, int max_len, int T, int TK, int H, int Hkv, int D, long long q_ss, long long q_sh,
                             long long k_ss, long long k_sh, long long v_ss, long long v_sh, long long o_ss,
                             long long o_sh, float scale, void* stream, const tsb::AttnForm* form = nullptr,
-                            const tsb::AttnGate* gate = nullptr) {
+                            const tsb::AttnGate* gate = nullptr, float bound = 0.f) {
   using namespace tsb;
   if (n_seqs <= 0 || max_len <= 0 || T <= 0 || TK <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || (D != 64 && D != 128) || !cu_seqlens)
     return -2;
@@ -683,6 +973,18 @@ static int flash_fwd_varlen(const void* q, const void* k, const void* v, void* o
   if (form) {
     p.form = *form;
     p.gate = *gate;
+    // exp(score - bound) of a row's own key is at least exp(-2 bound): far from underflow up to here
+    if (bound > 0.f && bound <= 40.f) {
+      auto go = [&](auto kern, int smem_bytes) -> int {
+        const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes);
+        if (e != cudaSuccess) return static_cast<int>(e);
+        kern<<<grid, kBoundedThreads, smem_bytes, s>>>(tq, tk, tv, p, bound);
+        return static_cast<int>(cudaGetLastError());
+      };
+      const bool cap = p.form.softcap > 0.f;
+      if (D == 128) return cap ? go(flash_bounded_kernel<128, true>, BoundedCfg<128>::kSmemBytes) : go(flash_bounded_kernel<128, false>, BoundedCfg<128>::kSmemBytes);
+      return cap ? go(flash_bounded_kernel<64, true>, BoundedCfg<64>::kSmemBytes) : go(flash_bounded_kernel<64, false>, BoundedCfg<64>::kSmemBytes);
+    }
     const int rc = D == 128 ? launch(flash_fwd_kernel<128, false, true>, FaCfg<128>::kSmemBytes)
                             : launch(flash_fwd_kernel<64, false, true>, FaCfg<64>::kSmemBytes);
     return rc ? rc : static_cast<int>(cudaGetLastError());
@@ -714,10 +1016,11 @@ TSB_EXPORT int tsb_flash_fwd_varlen_keys(const void* q, const void* k, const voi
 }
 
 // The same with the masks, score forms, gates and row stride of attn_form.cuh: q [T, H, D], k / v rows 2 * Hkv heads apart (a key
-// axis [TK, 2 Hkv, D] of keys and values), o rows `ldo` apart. A chunk mask is the caller's: one "sequence" per chunk.
+// axis [TK, 2 Hkv, D] of keys and values), o rows `ldo` apart. A chunk mask is the caller's: one "sequence" per chunk. bound: no
+// score is larger (before distances are taken off), and none is smaller than -bound; 0: not known.
 TSB_EXPORT int tsb_flash_fwd_shaped(const void* q, const void* k, const void* v, void* o, const int* cu_seqlens, const int* cu_keys,
                                     int n_seqs, int max_len, int T, int TK, int H, int Hkv, int D, const long long* ints,
-                                    const float* floats, const void* const* ptrs, void* stream) {
+                                    const float* floats, const void* const* ptrs, float bound, void* stream) {
   using namespace tsb;
   AttnForm f;
   AttnGate g;
@@ -726,5 +1029,5 @@ TSB_EXPORT int tsb_flash_fwd_shaped(const void* q, const void* k, const void* v,
   const bool shaped = !f.plain() || !g.plain();
   const long long kv = 2ll * Hkv * D;
   return flash_fwd_varlen(q, k, v, o, cu_seqlens, cu_keys, n_seqs, max_len, T, TK, H, Hkv, D, static_cast<long long>(H) * D, D, kv, D, kv,
-                          D, g.ldo, D, f.scale, stream, shaped ? &f : nullptr, &g);
+                          D, g.ldo, D, f.scale, stream, shaped ? &f : nullptr, &g, bound);
 }

@@ -2,7 +2,7 @@
 //
 //   S_t = diag(w_t) S_(t-1) + v_t k_t^T,   o_t = S q_t   with S = S_t (AFTER) or S_(t-1)
 //
-// w is a factor per key column. `state_step` takes one token, `state_scan` walks a portion token by token; both keep everything in
+// w is a factor per key column. `StateStep` takes one token, `state_scan` walks a portion token by token; both keep everything in
 // fp32. The caller brings q, k, w and v.
 #pragma once
 
@@ -10,25 +10,18 @@
 
 namespace tsb {
 
-// One token, 256 threads. LPR lanes share a row of the state (PPL times four columns each), RPT rows are in flight per lane. D is a
-// multiple of 4 up to 4 LPR PPL, E any. sq, sk, sw [D], sv [E] in shared memory, written before the last barrier; so [E] is complete
-// after the next one.
+// One token, 256 threads. LPR lanes share a row of the state (PPL times four columns each), RPT rows are in flight per lane; the
+// first ones are requested by the constructor. D is a multiple of 4 up to 4 LPR PPL, E any. sq, sk, sw [D], sv [E] in shared memory
+// must be complete when `run` is called; so [E] is after the next barrier.
 template <int LPR, int PPL, int RPT, bool AFTER>
-__device__ __forceinline__ void state_step(float* st, int E, int D, bool fresh, const float* sq, const float* sk, const float* sw,
-                                           const float* sv, float* so) {
-  constexpr int kGroups = 256 / LPR;
-  const int grp = threadIdx.x / LPR, gl = threadIdx.x % LPR;
-  float4 q[PPL], k[PPL], w[PPL];
-#pragma unroll
-  for (int i = 0; i < PPL; ++i) {
-    const int d = (gl + i * LPR) * 4;
-    const bool ok = d < D;
-    q[i] = ok ? *reinterpret_cast<const float4*>(sq + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-    k[i] = ok ? *reinterpret_cast<const float4*>(sk + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-    w[i] = ok ? *reinterpret_cast<const float4*>(sw + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-  for (int e0 = grp; e0 - grp < E; e0 += kGroups * RPT) {          // (uniform bounds: the sums are shuffles)
-    float4 S[RPT][PPL];
+struct StateStep {
+  static constexpr int kGroups = 256 / LPR;
+  float* st;
+  int E, D, grp, gl;
+  bool fresh;
+  float4 S[RPT][PPL];
+
+  __device__ __forceinline__ void fetch(int e0) {
 #pragma unroll
     for (int r = 0; r < RPT; ++r)
 #pragma unroll
@@ -37,32 +30,50 @@ __device__ __forceinline__ void state_step(float* st, int E, int D, bool fresh, 
         S[r][i] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (!fresh && e < E && d < D) S[r][i] = __ldcs(reinterpret_cast<const float4*>(st + static_cast<long long>(e) * D + d));
       }
-    float o[RPT];
+  }
+  __device__ __forceinline__ StateStep(float* st_, int E_, int D_, bool fresh_)
+      : st(st_), E(E_), D(D_), grp(threadIdx.x / LPR), gl(threadIdx.x % LPR), fresh(fresh_) {
+    fetch(grp);
+  }
+  __device__ __forceinline__ void run(const float* sq, const float* sk, const float* sw, const float* sv, float* so) {
+    float4 q[PPL], k[PPL], w[PPL];
 #pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-      const int e = e0 + r * kGroups;
-      const float v = e < E ? sv[e] : 0.f;
-      o[r] = 0.f;
+    for (int i = 0; i < PPL; ++i) {
+      const int d = (gl + i * LPR) * 4;
+      const bool ok = d < D;
+      q[i] = ok ? *reinterpret_cast<const float4*>(sq + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+      k[i] = ok ? *reinterpret_cast<const float4*>(sk + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+      w[i] = ok ? *reinterpret_cast<const float4*>(sw + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    for (int e0 = grp; e0 - grp < E; e0 += kGroups * RPT) {          // (uniform bounds: the sums are shuffles)
+      if (e0 != grp) fetch(e0);
+      float o[RPT];
 #pragma unroll
-      for (int i = 0; i < PPL; ++i) {
-        float4 s = S[r][i];
-        if (!AFTER) o[r] = fmaf(s.x, q[i].x, fmaf(s.y, q[i].y, fmaf(s.z, q[i].z, fmaf(s.w, q[i].w, o[r]))));
-        s.x = fmaf(w[i].x, s.x, k[i].x * v); s.y = fmaf(w[i].y, s.y, k[i].y * v);
-        s.z = fmaf(w[i].z, s.z, k[i].z * v); s.w = fmaf(w[i].w, s.w, k[i].w * v);
-        if (AFTER) o[r] = fmaf(s.x, q[i].x, fmaf(s.y, q[i].y, fmaf(s.z, q[i].z, fmaf(s.w, q[i].w, o[r]))));
-        const int d = (gl + i * LPR) * 4;
-        if (e < E && d < D) __stcs(reinterpret_cast<float4*>(st + static_cast<long long>(e) * D + d), s);
+      for (int r = 0; r < RPT; ++r) {
+        const int e = e0 + r * kGroups;
+        const float v = e < E ? sv[e] : 0.f;
+        o[r] = 0.f;
+#pragma unroll
+        for (int i = 0; i < PPL; ++i) {
+          float4 s = S[r][i];
+          if (!AFTER) o[r] = fmaf(s.x, q[i].x, fmaf(s.y, q[i].y, fmaf(s.z, q[i].z, fmaf(s.w, q[i].w, o[r]))));
+          s.x = fmaf(w[i].x, s.x, k[i].x * v); s.y = fmaf(w[i].y, s.y, k[i].y * v);
+          s.z = fmaf(w[i].z, s.z, k[i].z * v); s.w = fmaf(w[i].w, s.w, k[i].w * v);
+          if (AFTER) o[r] = fmaf(s.x, q[i].x, fmaf(s.y, q[i].y, fmaf(s.z, q[i].z, fmaf(s.w, q[i].w, o[r]))));
+          const int d = (gl + i * LPR) * 4;
+          if (e < E && d < D) __stcs(reinterpret_cast<float4*>(st + static_cast<long long>(e) * D + d), s);
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < RPT; ++r) {
+#pragma unroll
+        for (int m = LPR / 2; m; m >>= 1) o[r] += __shfl_xor_sync(0xffffffffu, o[r], m);
+        const int e = e0 + r * kGroups;
+        if (gl == 0 && e < E) so[e] = o[r];
       }
     }
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-#pragma unroll
-      for (int m = LPR / 2; m; m >>= 1) o[r] += __shfl_xor_sync(0xffffffffu, o[r], m);
-      const int e = e0 + r * kGroups;
-      if (gl == 0 && e < E) so[e] = o[r];
-    }
   }
-}
+};
 
 // A portion of n tokens, 128 threads: warp w walks the state's rows e0 + 4 w .. + 3, lane l holds their columns l + 32 i. `fetch(t, d, q,
 // k, w)` gives a token's operands at column d < D, `value(t, e)` its value; `emit(t, e, o[4])` receives the read-out of four rows.

@@ -21,7 +21,7 @@
 namespace tsb {
 namespace {
 
-constexpr int kBlk = 4;            // tokens of a portion that a thread of the convolution takes
+constexpr int kBlk = 16;           // tokens of a portion that a thread of the convolution walks
 
 struct SsdParams {
   int H, vdim, vp, N, np, G, taps, rows, n_decode, n_seq, blocks, ld, ldo;
@@ -47,8 +47,8 @@ struct SsdParams {
 
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
-// A thread takes 16 bytes of columns of one decoded row or of up to kBlk tokens of a portion; the last column blocks take the
-// heads' step sizes.
+// A thread takes 16 bytes of columns of one decoded row or of a tile of up to kBlk tokens of a portion; the last column blocks take
+// the heads' step sizes.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 ssd_conv_kernel(SsdParams p) {
@@ -83,15 +83,6 @@ ssd_conv_kernel(SsdParams p) {
   const int c = (blockIdx.x * 128 + threadIdx.x) * V;
   if (c >= p.conv_c) return;
   T* st = static_cast<T*>(p.conv_state) + static_cast<long long>(max(slot, 0)) * TAIL * p.conv_c + c;
-  uint4 in[TAIL + kBlk];
-#pragma unroll
-  for (int r = 0; r < TAIL + kBlk; ++r) {
-    const int t = r - TAIL;                      // token relative to the first row
-    in[r] = make_uint4(0u, 0u, 0u, 0u);
-    if (t >= cnt) continue;
-    if (before + t >= 0) in[r] = *reinterpret_cast<const uint4*>(proj + static_cast<long long>(t) * p.ld + p.off_x + c);
-    else if (old && slot >= 0) in[r] = *reinterpret_cast<const uint4*>(st + static_cast<long long>(TAIL + before + t) * p.conv_c);
-  }
   float w[TAPS][V], b[V];
 #pragma unroll
   for (int i = 0; i < V; i += 4) {
@@ -99,19 +90,38 @@ ssd_conv_kernel(SsdParams p) {
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) *reinterpret_cast<float4*>(&w[j][i]) = *reinterpret_cast<const float4*>(p.conv_w + j * p.conv_c + c + i);
   }
+  const T* x = proj + p.off_x + c;
   T* out = static_cast<T*>(p.xbc) + static_cast<long long>(row) * p.conv_c + c;
+  constexpr int kStep = 4;                       // tokens whose inputs are requested together
+  uint4 in[TAIL + kStep];                        // the window: the tokens in front, then these
 #pragma unroll
-  for (int t = 0; t < kBlk; ++t) {
-    if (t >= cnt) break;
-    float y[V];
+  for (int r = 0; r < TAIL; ++r) {
+    const int t = r - TAIL;
+    in[r] = make_uint4(0u, 0u, 0u, 0u);
+    if (before + t >= 0) in[r] = *reinterpret_cast<const uint4*>(x + static_cast<long long>(t) * p.ld);
+    else if (old && slot >= 0) in[r] = *reinterpret_cast<const uint4*>(st + static_cast<long long>(TAIL + before + t) * p.conv_c);
+  }
+#pragma unroll 1
+  for (int t0 = 0; t0 < cnt; t0 += kStep) {
 #pragma unroll
-    for (int i = 0; i < V; ++i) {
-      float a = b[i];
+    for (int t = 0; t < kStep; ++t)
+      in[TAIL + t] = t0 + t < cnt ? *reinterpret_cast<const uint4*>(x + static_cast<long long>(t0 + t) * p.ld) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) a = fmaf(w[j][i], to_f32<T>(reinterpret_cast<const T*>(&in[t + j])[i]), a);
-      y[i] = silu_f32(a);
+    for (int t = 0; t < kStep; ++t) {
+      if (t0 + t >= cnt) break;
+      float y[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        float a = b[i];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) a = fmaf(w[j][i], to_f32<T>(reinterpret_cast<const T*>(&in[t + j])[i]), a);
+        y[i] = sizeof(T) == 2 ? __fdividef(a, 1.f + __expf(-a)) : silu_f32(a);
+      }
+      st16<T>(out + static_cast<long long>(t0 + t) * p.conv_c, y);
     }
-    st16<T>(out + static_cast<long long>(t) * p.conv_c, y);
+    if (decode) break;
+#pragma unroll
+    for (int r = 0; r < TAIL; ++r) in[r] = in[r + kStep];
   }
   if (decode && slot >= 0) {
 #pragma unroll
@@ -164,6 +174,7 @@ ssd_step_kernel(SsdParams p) {
     for (int e = tid; e < p.vp; e += 256) out[e] = from_f32<T>(0.f);
     return;
   }
+  StateStep<LPR, PPL, RPT, true> step(p.state + (static_cast<long long>(slot) * p.H + h) * p.vp * p.np, p.vp, p.np, p.positions[row] <= 0);
   const T* xbc = static_cast<const T*>(p.xbc) + static_cast<long long>(row) * p.conv_c;
   const float2 g = p.gates[static_cast<long long>(row) * p.H + h];
   const float w = exp2f(g.y);
@@ -175,8 +186,7 @@ ssd_step_kernel(SsdParams p) {
   }
   for (int e = tid; e < p.vp; e += 256) sv[e] = to_f32<T>(xbc[h * p.vp + e]);
   __syncthreads();
-  state_step<LPR, PPL, RPT, true>(p.state + (static_cast<long long>(slot) * p.H + h) * p.vp * p.np, p.vp, p.np, p.positions[row] <= 0, sq, sk, sw,
-                                  sv, so);
+  step.run(sq, sk, sw, sv, so);
   __syncthreads();
   for (int e = tid; e < p.vp; e += 256) out[e] = from_f32<T>(fmaf(p.d[h], sv[e], so[e]));
 }
@@ -537,7 +547,7 @@ bool read_ssd(const int* v, SsdParams* p) {
 }  // namespace
 }  // namespace tsb
 
-// ints: H, vdim, vp, state, np, groups, taps, rows, n_decode, prompt sequences, blocks of 4 tokens of their portions, projection row
+// ints: H, vdim, vp, state, np, groups, taps, rows, n_decode, prompt sequences, tiles of 16 tokens of their portions, projection row
 // stride, result row stride. ptrs: proj, conv_w, conv_b, a_log, dt_bias, conv_state, xbc, gates, slots, positions, cu, pos0, blk_seq, blk0.
 TSB_EXPORT int tsb_ssd_conv(const int* ints, void* const* q, int dtype, void* stream) {
   using namespace tsb;

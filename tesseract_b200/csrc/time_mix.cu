@@ -7,12 +7,15 @@
 // one before it.
 //
 // Prompts in bf16 with heads of up to 128 columns run on the tensor cores (time_mix_chunk_kernel): blocks of 16 tokens, four of
-// them prepared at once. With W_i the product of the decays of the block's tokens up to i,
-//   o_i = S (W_(i-1) r_i) + sum_{j < i} (sum_d r_id k_jd W_(i-1)d / W_jd) v_j + (u k_i . r_i) v_i
-//   S  <- S diag(W_15) + sum_j v_j (k_j W_15 / W_j)^T
-// where every ratio is formed as the product of the decays in between, so nothing overflows however steep they are. S stays in the
-// accumulators of the products (values on rows), which is also the layout in which it enters the read-out. Factors that must not
-// lose their 32 bits meet the tensor cores as two bf16 halves (16 bits).
+// them prepared at once. With W_i the product of the decays of the block's tokens up to i, R_i = r_i W_(i-1) / W_15 and
+// K_j = k_j W_15 / W_j (the product of the decays behind j),
+//   S  <- S diag(W_15)
+//   o_i = S R_i + sum_{j < i} (R_i . K_j) v_j + (u k_i . r_i) v_i
+//   S  <- S + sum_j v_j K_j^T
+// Where a channel decays by more than 2^60 in a block, 1 / W_15 is not formed: R_i = r_i W_(i-1) meets S before it decays, and the
+// pairs are summed with the decays in between, one by one. S stays in the accumulators of the products (values on rows), which is
+// also the layout in which it enters the read-out. Factors that must not lose their 32 bits meet the tensor cores as two bf16 halves
+// (16 bits).
 // fp32 models and wider heads take time_mix_scan_kernel (token by token) and time_mix_norm_kernel; decoded tokens
 // time_mix_step_kernel.
 #include "linear_state.cuh"
@@ -175,40 +178,46 @@ time_mix_norm_kernel(MixParams p) {
 // ------------------------------------------------------------------ prompts, bf16
 template <int DT>
 struct MixChunk {
-  static constexpr int kTok = 64, kBlk = 16, kWarps = DT / 16, kThreads = kWarps * 32, kParts = DT / 64;
-  static constexpr int kLd = DT + 8, kLdO = DT + 4, kLdA = 20;
-  // bytes: r / high half of W r, k / high half of k W, v, the low halves, decay inputs / read-outs, pair sums, block decays
-  static constexpr int kTile = kTok * kLd * 2, kR = 0, kK = kTile, kV = 2 * kTile, kRl = 3 * kTile, kKl = 4 * kTile, kO = 5 * kTile;
-  static constexpr int kA = kO + kTok * kLdO * 4, kTot = kA + kParts * 4 * kBlk * kLdA * 4, kSmem = kTot + 4 * DT * 4;
+  static constexpr int kTok = 64, kWarps = DT / 16, kThreads = kWarps * 32, kParts = DT / 64;
+  static constexpr int kLd = DT + 8, kLdO = DT + 4;
+  // bytes of a stage: r (its place is taken by the high half of the decayed r), k likewise, v, decay inputs (by the read-outs)
+  static constexpr int kTile = kTok * kLd * 2, kR = 0, kK = kTile, kV = 2 * kTile, kO = 3 * kTile, kStage = kO + kTok * kLdO * 4;
+  // what exists once: the low halves, the pair products, the blocks' decays, the bonus of every token
+  static constexpr int kRl = 2 * kStage, kKl = kRl + kTile, kA = kKl + kTile, kTot = kA + kParts * 4096, kBonus = kTot + 4 * DT * 4;
+  static constexpr int kSmem = kBonus + kParts * kTok * 4;
 };
+constexpr float kSteep = 8.6736174e-19f;       // 2^-60: a block that decays a channel further takes the slow pair products
 
-// Sums of 32 values over the warp: lane l returns the sum of v[l].
-__device__ __forceinline__ float transpose_sum(float (&v)[32], int lane) {
+// Sums of N values over the warp, N a power of two: lane l returns the sum of v[l % N].
+template <int N>
+__device__ __forceinline__ float transpose_sum(float (&v)[N], int lane) {
 #pragma unroll
-  for (int o = 16; o; o >>= 1) {
+  for (int o = N / 2; o; o >>= 1) {
     const bool up = (lane & o) != 0;
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < N / 2; ++i) {
       if (i >= o) break;
       const float keep = up ? v[i + o] : v[i], give = up ? v[i] : v[i + o];
       v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
     }
   }
+#pragma unroll
+  for (int o = N; o < 32; o <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
   return v[0];
 }
 
-// CTA = (head, sequence); warp w owns the state's rows (values) 16 w .. + 15.
+// CTA = (head, sequence); warp w owns the state's rows (values) 16 w .. + 15. The next 64 tokens arrive while some are worked on.
 template <int DT>
-__global__ void __launch_bounds__(MixChunk<DT>::kThreads, DT == 64 ? 3 : 1)
+__global__ void __launch_bounds__(MixChunk<DT>::kThreads, DT == 64 ? 2 : 1)
 time_mix_chunk_kernel(MixParams p) {
   using T = __nv_bfloat16;
   using C = MixChunk<DT>;
   pdl_trigger();
   pdl_grid_wait();
   extern __shared__ __align__(16) uint8_t smem[];
-  T *sr = reinterpret_cast<T*>(smem + C::kR), *sk = reinterpret_cast<T*>(smem + C::kK), *sv = reinterpret_cast<T*>(smem + C::kV);
   T *srl = reinterpret_cast<T*>(smem + C::kRl), *skl = reinterpret_cast<T*>(smem + C::kKl);
-  float *so = reinterpret_cast<float*>(smem + C::kO), *sa = reinterpret_cast<float*>(smem + C::kA), *stot = reinterpret_cast<float*>(smem + C::kTot);
+  float *sa = reinterpret_cast<float*>(smem + C::kA), *stot = reinterpret_cast<float*>(smem + C::kTot);
+  float* sbonus = reinterpret_cast<float*>(smem + C::kBonus);
   const int h = blockIdx.x, seq = blockIdx.y, slot = p.slots[seq];
   const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
   if (slot < 0 || n <= 0) return;
@@ -217,6 +226,28 @@ time_mix_chunk_kernel(MixParams p) {
   const float* dec = p.dec + static_cast<long long>(row0) * p.H * p.dp + h * p.dp;
   float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp;
   const int e0 = warp * 16;
+  auto issue = [&](int t0) {
+    uint8_t* stage = smem + (t0 / C::kTok & 1) * C::kStage;
+    const uint32_t base = smem_u32(stage);
+    const int cnt = min(C::kTok, n - t0);
+    for (int i = tid; i < C::kTok * (DT / 8); i += C::kThreads) {
+      const int r = i / (DT / 8), d = (i % (DT / 8)) * 8;
+      const bool ok = r < cnt && d < p.dp;
+      const T* src = ok ? proj + static_cast<long long>(t0 + r) * p.ld + d : proj;
+      const int bytes = ok ? 16 : 0, sec = ok ? p.section : 0;
+      const uint32_t at = base + (r * C::kLd + d) * 2;
+      cp_async_16(at + C::kR, src, bytes);
+      cp_async_16(at + C::kK, src + sec, bytes);
+      cp_async_16(at + C::kV, src + 2 * sec, bytes);
+    }
+    for (int i = tid; i < C::kTok * (DT / 4); i += C::kThreads) {
+      const int r = i / (DT / 4), d = (i % (DT / 4)) * 4;
+      const bool ok = r < cnt && d < p.dp;
+      cp_async_16(base + C::kO + (r * C::kLdO + d) * 4, ok ? dec + static_cast<long long>(t0 + r) * p.H * p.dp + d : dec, ok ? 16 : 0);
+    }
+    cp_commit();
+  };
+  issue(0);
   float S[DT / 8][4];
   {
     const bool old = p.pos0[seq] > 0;
@@ -240,123 +271,177 @@ time_mix_chunk_kernel(MixParams p) {
     uu[0] = p.u[h * p.dp + d0];
     uu[1] = p.u[h * p.dp + d0 + 1];
   }
-  const uint32_t aR = smem_u32(sr), aRl = smem_u32(srl), aK = smem_u32(sk), aKl = smem_u32(skl), aV = smem_u32(sv);
+  const uint32_t aRl = smem_u32(srl), aKl = smem_u32(skl);
+  // rows of the epilogue: kLanes lanes of four columns share one
+  constexpr int kLanes = DT / 4, kPer = 32 / kLanes, kIter = C::kTok / (C::kWarps * kPer);
+  const int er = warp * kPer + lane / kLanes, ec = lane % kLanes * 4;
 
   for (int t0 = 0; t0 < n; t0 += C::kTok) {
     const int cnt = min(C::kTok, n - t0);
-    for (int i = tid; i < C::kTok * (DT / 8); i += C::kThreads) {
-      const int r = i / (DT / 8), d = (i % (DT / 8)) * 8;
-      const bool ok = r < cnt && d < p.dp;
-      const T* src = ok ? proj + static_cast<long long>(t0 + r) * p.ld + d : proj;
-      const int bytes = ok ? 16 : 0;
-      cp_async_16(aR + (r * C::kLd + d) * 2, src, bytes);
-      cp_async_16(aK + (r * C::kLd + d) * 2, ok ? src + p.section : src, bytes);
-      cp_async_16(aV + (r * C::kLd + d) * 2, ok ? src + 2 * p.section : src, bytes);
-    }
-    for (int i = tid; i < C::kTok * (DT / 4); i += C::kThreads) {
-      const int r = i / (DT / 4), d = (i % (DT / 4)) * 4;
-      const bool ok = r < cnt && d < p.dp;
-      cp_async_16(smem_u32(so + r * C::kLdO + d), ok ? dec + static_cast<long long>(t0 + r) * p.H * p.dp + d : dec, ok ? 16 : 0);
-    }
-    cp_commit();
+    uint8_t* stage = smem + (t0 / C::kTok & 1) * C::kStage;
+    T *sr = reinterpret_cast<T*>(stage + C::kR), *sk = reinterpret_cast<T*>(stage + C::kK), *sv = reinterpret_cast<T*>(stage + C::kV);
+    float* so = reinterpret_cast<float*>(stage + C::kO);
+    const uint32_t aR = smem_u32(sr), aK = smem_u32(sk), aV = smem_u32(sv);
     cp_wait<0>();
     __syncthreads();
+    if (t0 + C::kTok < n) issue(t0 + C::kTok);
+    bool steep;
     {
-      float r[16][2], k[16][2], w[16][2];
+      __nv_bfloat162 r[16], k[16];
+      float w[16][2];
       const int row = blk * 16;
+      float tot[2] = {1.f, 1.f}, bonus[16];
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
-        const __nv_bfloat162 rv = *reinterpret_cast<const __nv_bfloat162*>(sr + (row + i) * C::kLd + d0);
-        const __nv_bfloat162 kv = *reinterpret_cast<const __nv_bfloat162*>(sk + (row + i) * C::kLd + d0);
+        r[i] = *reinterpret_cast<const __nv_bfloat162*>(sr + (row + i) * C::kLd + d0);
+        k[i] = *reinterpret_cast<const __nv_bfloat162*>(sk + (row + i) * C::kLd + d0);
         const float2 dv = *reinterpret_cast<const float2*>(so + (row + i) * C::kLdO + d0);
-        r[i][0] = __low2float(rv); r[i][1] = __high2float(rv);
-        k[i][0] = __low2float(kv); k[i][1] = __high2float(kv);
         const bool real = row + i < cnt;                     // (a token that is not there decays nothing)
         w[i][0] = real ? expf(-__expf(dv.x + w0[0])) : 1.f;
         w[i][1] = real ? expf(-__expf(dv.y + w0[1])) : 1.f;
+        tot[0] *= w[i][0];
+        tot[1] *= w[i][1];
+        bonus[i] = fmaf(__low2float(r[i]) * uu[0], __low2float(k[i]), __high2float(r[i]) * uu[1] * __high2float(k[i]));
       }
-      float f[2] = {1.f, 1.f};
+      const float b = transpose_sum<16>(bonus, lane);
+      if (lane < 16) sbonus[part * C::kTok + row + lane] = b;
+      steep = __syncthreads_or(tot[0] < kSteep || tot[1] < kSteep) != 0;
+      *reinterpret_cast<float2*>(stot + blk * DT + d0) = make_float2(tot[0], tot[1]);
+      float f[2] = {steep ? 1.f : 1.f / tot[0], steep ? 1.f : 1.f / tot[1]};
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         const int at = (row + i) * C::kLd + d0;
-        split_bf16x2(r[i][0] * f[0], r[i][1] * f[1], reinterpret_cast<uint32_t*>(sr + at), reinterpret_cast<uint32_t*>(srl + at));
+        split_bf16x2(__low2float(r[i]) * f[0], __high2float(r[i]) * f[1], reinterpret_cast<uint32_t*>(sr + at), reinterpret_cast<uint32_t*>(srl + at));
         f[0] *= w[i][0];
         f[1] *= w[i][1];
       }
-      *reinterpret_cast<float2*>(stot + blk * DT + d0) = make_float2(f[0], f[1]);
       f[0] = f[1] = 1.f;
 #pragma unroll
       for (int i = 15; i >= 0; --i) {
         const int at = (row + i) * C::kLd + d0;
-        split_bf16x2(k[i][0] * f[0], k[i][1] * f[1], reinterpret_cast<uint32_t*>(sk + at), reinterpret_cast<uint32_t*>(skl + at));
+        split_bf16x2(__low2float(k[i]) * f[0], __high2float(k[i]) * f[1], reinterpret_cast<uint32_t*>(sk + at), reinterpret_cast<uint32_t*>(skl + at));
         f[0] *= w[i][0];
         f[1] *= w[i][1];
       }
-      // what token i takes of token j's value, two j at a time
-      float* a = sa + (part * 4 + blk) * C::kBlk * C::kLdA;
+      if (steep) {
+        // what token i takes of token j's value, two j at a time: the decays in between, one by one
+        float* a = sa + (part * 4 + blk) * 256;
 #pragma unroll
-      for (int jj = 0; jj < 16; jj += 2) {
-        float v[32];
+        for (int jj = 0; jj < 16; jj += 2) {
+          float v[32];
 #pragma unroll
-        for (int s = 0; s < 2; ++s) {
-          const int j = jj + s;
-          float x0 = k[j][0], x1 = k[j][1];
+          for (int q = 0; q < 2; ++q) {
+            const int j = jj + q;
+            float x0 = __low2float(k[j]), x1 = __high2float(k[j]);
 #pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            if (i < j) v[s * 16 + i] = 0.f;
-            else if (i == j) v[s * 16 + i] = fmaf(r[i][0] * uu[0], k[i][0], r[i][1] * uu[1] * k[i][1]);
-            else {
-              v[s * 16 + i] = fmaf(r[i][0], x0, r[i][1] * x1);
+            for (int i = 0; i < 16; ++i) {
+              v[q * 16 + i] = 0.f;
+              if (i <= j) continue;
+              v[q * 16 + i] = fmaf(__low2float(r[i]), x0, __high2float(r[i]) * x1);
               x0 *= w[i][0];
               x1 *= w[i][1];
             }
           }
+          a[(jj + (lane >> 4)) * 16 + (lane & 15)] = transpose_sum<32>(v, lane);
         }
-        a[(jj + (lane >> 4)) * C::kLdA + (lane & 15)] = transpose_sum(v, lane);
       }
     }
+    if (C::kParts > 1) __syncthreads();
+    else __syncwarp();
+    if (!steep && warp < 4) {
+      // the same from the prepared factors: rows i, columns j; this layout is also that of the operand it becomes
+      float c[3][2][4] = {};
+      const int row = warp * 16;
+#pragma unroll
+      for (int ks = 0; ks < DT / 16; ++ks) {
+        uint32_t qh[4], ql[4], kh[4], kl[4];
+        ldmat_x4(qh, aR + frag_a(lane, row, ks * 16, C::kLd));
+        ldmat_x4(ql, aRl + frag_a(lane, row, ks * 16, C::kLd));
+        ldmat_x4(kh, aK + frag_b(lane, row, ks * 16, C::kLd));
+        ldmat_x4(kl, aKl + frag_b(lane, row, ks * 16, C::kLd));
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          mma_bf16(c[0][j], qh, kh[2 * j], kh[2 * j + 1]);
+          mma_bf16(c[1][j], ql, kh[2 * j], kh[2 * j + 1]);
+          mma_bf16(c[2][j], qh, kl[2 * j], kl[2 * j + 1]);
+        }
+      }
+      uint32_t* frag = reinterpret_cast<uint32_t*>(sa) + warp * 256;
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {                        // rows i = g + 8 e, columns j 8 + 2 t, + 1
+          float x[2];
+#pragma unroll
+          for (int q = 0; q < 2; ++q)
+            x[q] = j * 8 + 2 * t4 + q < g + 8 * e ? c[0][j][2 * e + q] + (c[1][j][2 * e + q] + c[2][j][2 * e + q]) : 0.f;
+          uint32_t hi, lo;
+          split_bf16x2(x[0], x[1], &hi, &lo);
+          frag[(e * 4 + j) * 32 + lane] = hi;
+          frag[(e * 4 + 2 + j) * 32 + lane] = lo;
+        }
+    }
     __syncthreads();
+    uint2 gate[kIter];                                       // requested before the products
+#pragma unroll
+    for (int i = 0; i < kIter; ++i) {
+      const int r = min(i * C::kWarps * kPer + er, cnt - 1);
+      gate[i] = *reinterpret_cast<const uint2*>(proj + static_cast<long long>(t0 + r) * p.ld + 3 * p.section + min(ec, p.dp - 4));
+    }
 #pragma unroll 1
     for (int b = 0; b < 4; ++b) {
       if (b * 16 >= cnt) break;
       const int row = b * 16;
-      float acc[2][4] = {};
+      if (!steep) {
+#pragma unroll
+        for (int j = 0; j < DT / 8; ++j) {
+          const float2 f = *reinterpret_cast<const float2*>(stot + b * DT + j * 8 + 2 * t4);
+          S[j][0] *= f.x; S[j][1] *= f.y; S[j][2] *= f.x; S[j][3] *= f.y;
+        }
+      }
+      float acc[3][2][4] = {};
 #pragma unroll
       for (int ks = 0; ks < DT / 16; ++ks) {
-        uint32_t hi[4], lo[4], q[4];
+        uint32_t hi[4], lo[4], qh[4], ql[4];
         split_bf16x2(S[2 * ks][0], S[2 * ks][1], &hi[0], &lo[0]);
         split_bf16x2(S[2 * ks][2], S[2 * ks][3], &hi[1], &lo[1]);
         split_bf16x2(S[2 * ks + 1][0], S[2 * ks + 1][1], &hi[2], &lo[2]);
         split_bf16x2(S[2 * ks + 1][2], S[2 * ks + 1][3], &hi[3], &lo[3]);
-        ldmat_x4(q, aR + frag_b(lane, row, ks * 16, C::kLd));
-        mma_bf16(acc[0], hi, q[0], q[1]);
-        mma_bf16(acc[1], hi, q[2], q[3]);
-        mma_bf16(acc[0], lo, q[0], q[1]);
-        mma_bf16(acc[1], lo, q[2], q[3]);
-        ldmat_x4(q, aRl + frag_b(lane, row, ks * 16, C::kLd));
-        mma_bf16(acc[0], hi, q[0], q[1]);
-        mma_bf16(acc[1], hi, q[2], q[3]);
+        ldmat_x4(qh, aR + frag_b(lane, row, ks * 16, C::kLd));
+        ldmat_x4(ql, aRl + frag_b(lane, row, ks * 16, C::kLd));
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          mma_bf16(acc[0][c], hi, qh[2 * c], qh[2 * c + 1]);
+          mma_bf16(acc[1][c], lo, qh[2 * c], qh[2 * c + 1]);
+          mma_bf16(acc[2][c], hi, ql[2 * c], ql[2 * c + 1]);
+        }
       }
       uint32_t vt[4];
       ldmat_x4_trans(vt, aV + frag_a_trans(lane, row, e0, C::kLd));
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         uint32_t hi[2], lo[2];
+        if (!steep) {
+          const uint32_t* frag = reinterpret_cast<const uint32_t*>(sa) + b * 256 + c * 128 + lane;
+          hi[0] = frag[0]; hi[1] = frag[32]; lo[0] = frag[64]; lo[1] = frag[96];
+        } else {
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          float x[2] = {};
+          for (int e = 0; e < 2; ++e) {
+            float x[2] = {};
 #pragma unroll
-          for (int q = 0; q < C::kParts; ++q) {
-            const float* a = sa + ((q * 4 + b) * C::kBlk + e * 8 + 2 * t4) * C::kLdA + c * 8 + g;
-            x[0] += a[0];
-            x[1] += a[C::kLdA];
+            for (int q = 0; q < C::kParts; ++q) {
+              const float* a = sa + (q * 4 + b) * 256 + (e * 8 + 2 * t4) * 16 + c * 8 + g;
+              x[0] += a[0];
+              x[1] += a[16];
+            }
+            split_bf16x2(x[0], x[1], &hi[e], &lo[e]);
           }
-          split_bf16x2(x[0], x[1], &hi[e], &lo[e]);
         }
-        mma_bf16(acc[c], vt, hi[0], hi[1]);
-        mma_bf16(acc[c], vt, lo[0], lo[1]);
+        mma_bf16(acc[0][c], vt, hi[0], hi[1]);
+        mma_bf16(acc[1][c], vt, lo[0], lo[1]);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) so[(row + c * 8 + 2 * t4 + (e & 1)) * C::kLdO + e0 + g + 8 * (e >> 1)] = acc[c][e];
+        for (int e = 0; e < 4; ++e)
+          so[(row + c * 8 + 2 * t4 + (e & 1)) * C::kLdO + e0 + g + 8 * (e >> 1)] = acc[0][c][e] + (acc[1][c][e] + acc[2][c][e]);
       }
 #pragma unroll
       for (int j = 0; j < DT / 8; j += 2) {
@@ -365,42 +450,39 @@ time_mix_chunk_kernel(MixParams p) {
         ldmat_x4_trans(kl, aKl + frag_b_trans(lane, row, j * 8, C::kLd));
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
-          const float2 f = *reinterpret_cast<const float2*>(stot + b * DT + (j + c) * 8 + 2 * t4);
-          S[j + c][0] *= f.x; S[j + c][1] *= f.y; S[j + c][2] *= f.x; S[j + c][3] *= f.y;
+          if (steep) {
+            const float2 f = *reinterpret_cast<const float2*>(stot + b * DT + (j + c) * 8 + 2 * t4);
+            S[j + c][0] *= f.x; S[j + c][1] *= f.y; S[j + c][2] *= f.x; S[j + c][3] *= f.y;
+          }
           mma_bf16(S[j + c], vt, kh[2 * c], kh[2 * c + 1]);
           mma_bf16(S[j + c], vt, kl[2 * c], kl[2 * c + 1]);
         }
       }
     }
     __syncthreads();
-    // norm and gate: a warp per row, two (four) columns per lane
-    constexpr int kRows = C::kTok / C::kWarps;
-#pragma unroll 4
-    for (int i = 0; i < kRows; ++i) {
-      const int r = i * C::kWarps + warp;
-      if (r >= cnt) break;
-      const T* gate = proj + static_cast<long long>(t0 + r) * p.ld + 3 * p.section;
-      T* out = static_cast<T*>(p.out) + static_cast<long long>(row0 + t0 + r) * p.ldo + h * p.dp;
-      float2 o[C::kParts];
-      __nv_bfloat162 gv[C::kParts];
-      float ss = 0.f;
+    // bonus, norm and gate
+    float4 nm = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (ec < p.dp) nm = *reinterpret_cast<const float4*>(p.norm + h * p.dp + ec);
 #pragma unroll
-      for (int q = 0; q < C::kParts; ++q) {
-        const int d = q * 64 + lane * 2;
-        gv[q] = *reinterpret_cast<const __nv_bfloat162*>(gate + min(d, p.dp - 2));
-        o[q] = *reinterpret_cast<const float2*>(so + r * C::kLdO + d);
-        ss = fmaf(o[q].x, o[q].x, fmaf(o[q].y, o[q].y, ss));
-      }
-      const float rs = p.out_scale * rsqrtf(warp_sum(ss) / static_cast<float>(p.dim) + p.eps);
+    for (int i = 0; i < kIter; ++i) {
+      const int r = i * C::kWarps * kPer + er;
+      float4 o = *reinterpret_cast<const float4*>(so + r * C::kLdO + ec);
+      float bonus = sbonus[r];
+      if (C::kParts > 1) bonus += sbonus[C::kTok + r];
+      const uint2 vv = *reinterpret_cast<const uint2*>(sv + r * C::kLd + ec);
+      const __nv_bfloat162 va = *reinterpret_cast<const __nv_bfloat162*>(&vv.x), vb = *reinterpret_cast<const __nv_bfloat162*>(&vv.y);
+      o.x = fmaf(bonus, __low2float(va), o.x); o.y = fmaf(bonus, __high2float(va), o.y);
+      o.z = fmaf(bonus, __low2float(vb), o.z); o.w = fmaf(bonus, __high2float(vb), o.w);
+      float ss = fmaf(o.x, o.x, fmaf(o.y, o.y, fmaf(o.z, o.z, o.w * o.w)));
 #pragma unroll
-      for (int q = 0; q < C::kParts; ++q) {
-        const int d = q * 64 + lane * 2;
-        if (d >= p.dp) continue;
-        const float2 nm = *reinterpret_cast<const float2*>(p.norm + h * p.dp + d);
-        const float g0 = __low2float(gv[q]), g1 = __high2float(gv[q]);
-        *reinterpret_cast<uint32_t*>(out + d) = pack_bf16x2(o[q].x * rs * nm.x * __fdividef(g0, 1.f + __expf(-g0)),
-                                                            o[q].y * rs * nm.y * __fdividef(g1, 1.f + __expf(-g1)));
-      }
+      for (int m = kLanes / 2; m; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+      if (r >= cnt || ec >= p.dp) continue;
+      const float rs = p.out_scale * rsqrtf(ss / static_cast<float>(p.dim) + p.eps);
+      const __nv_bfloat162 ga = *reinterpret_cast<const __nv_bfloat162*>(&gate[i].x), gb = *reinterpret_cast<const __nv_bfloat162*>(&gate[i].y);
+      auto silu = [](float x) { return __fdividef(x, 1.f + __expf(-x)); };
+      *reinterpret_cast<uint2*>(static_cast<T*>(p.out) + static_cast<long long>(row0 + t0 + r) * p.ldo + h * p.dp + ec) =
+          make_uint2(pack_bf16x2(o.x * rs * nm.x * silu(__low2float(ga)), o.y * rs * nm.y * silu(__high2float(ga))),
+                     pack_bf16x2(o.z * rs * nm.z * silu(__low2float(gb)), o.w * rs * nm.w * silu(__high2float(gb))));
     }
     __syncthreads();
   }
@@ -413,7 +495,7 @@ time_mix_chunk_kernel(MixParams p) {
     }
 }
 
-// Decoded rows: CTA = (row, head).
+// Decoded rows: CTA = (row, head). The state is requested first, the decays are worked out while it arrives.
 template <typename T, int LPR, int PPL, int RPT>
 __global__ void __launch_bounds__(256)
 time_mix_step_kernel(MixParams p) {
@@ -429,6 +511,7 @@ time_mix_step_kernel(MixParams p) {
     for (int d = tid; d < p.dp; d += 256) out[d] = from_f32<T>(0.f);
     return;
   }
+  StateStep<LPR, PPL, RPT, false> step(p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp, p.dp, p.dp, p.positions[row] <= 0);
   float bonus = 0.f;
   for (int d = tid; d < p.dp; d += 256) {
     sq[d] = to_f32<T>(x[d]);
@@ -441,19 +524,26 @@ time_mix_step_kernel(MixParams p) {
   bonus = warp_sum(bonus);
   if (lane == 0) red[warp] = bonus;
   __syncthreads();
+  // four lanes per channel, 16 bytes of its row of the matrix at a time
+  constexpr int V = kVec16<T>;
   const T* w2 = static_cast<const T*>(p.w2) + static_cast<long long>(h) * p.dp * p.rp;
-  for (int d = warp; d < p.dp; d += 8) {
+  for (int d = tid >> 2; d < p.dp; d += 64) {              // (dp is a multiple of 16: a warp's eight channels exist or do not)
     float a = 0.f;
-    for (int j = lane; j < p.rp; j += 32) a = fmaf(to_f32<T>(w2[static_cast<long long>(d) * p.rp + j]), th[j], a);
-    a = warp_sum(a);
-    if (lane == 0) sw[d] = expf(-expf(a + p.w0[h * p.dp + d]));
+    for (int j = (tid & 3) * V; j < p.rp; j += 4 * V) {
+      float f[V];
+      ld16<T>(w2 + static_cast<long long>(d) * p.rp + j, f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) a = fmaf(f[i], th[j + i], a);
+    }
+    a += __shfl_xor_sync(0xffffffffu, a, 1);
+    a += __shfl_xor_sync(0xffffffffu, a, 2);
+    if ((tid & 3) == 0) sw[d] = expf(-expf(a + p.w0[h * p.dp + d]));
   }
   bonus = 0.f;
 #pragma unroll
   for (int w = 0; w < 8; ++w) bonus += red[w];
   __syncthreads();
-  state_step<LPR, PPL, RPT, false>(p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp, p.dp, p.dp, p.positions[row] <= 0, sq, sk,
-                                   sw, sv, so);
+  step.run(sq, sk, sw, sv, so);
   __syncthreads();
   float ss = 0.f;
   for (int d = tid; d < p.dp; d += 256) {
@@ -579,7 +669,7 @@ TSB_EXPORT int tsb_time_mix_prefill(const int* ints, void* const* q, float eps, 
   p.eps = eps; p.out_scale = out_scale;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (!p.o) {
-    if (dtype != 1 || p.dp > 128 || p.ldo % 2) return -2;
+    if (dtype != 1 || p.dp > 128 || p.ldo % 4 || (reinterpret_cast<uintptr_t>(p.out) & 7)) return -2;
     return p.dp <= 64 ? run_chunk<64>(p, s) : run_chunk<128>(p, s);
   }
   if (dtype == 1) return run_scan<__nv_bfloat16>(p, s);

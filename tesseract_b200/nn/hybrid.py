@@ -26,7 +26,7 @@ from ..ops.ragged import AttentionGeometry, AttentionWeights, ScoreForm, padded_
 from ..ops.retention import SPAN, RetentionGeometry, log2_decays, retention
 from ..ops.rglru import CHUNK, RGLRUGeometry, RGLRUWeights, rglru
 from ..ops.rotary import Rotary
-from ..ops.ssd import SSDGeometry, SSDWeights, ssd
+from ..ops.ssd import CONV_TILE, SSDGeometry, SSDWeights, ssd
 from ..ops.timemix import STREAMS, TimeMixGeometry, TimeMixWeights, time_mix, token_shift
 from .ragged import LatentRun, PagedRun, PairRun, StateRun
 
@@ -558,6 +558,8 @@ class ShapedAttention(_RowPacked):
         self.w = AttentionWeights(form, vec(g.off_gate) if bias else None, norm, vec(sizes[0]) if sizes else None,
                                   vec(sizes[1]) if sizes else None, float(eps))
         self.masks = (form.mask,)
+        if norm == "unit":
+            form.product_bound = 1.02 * dim               # (two unit vectors times sqrt(dim), rounded)
 
     def tensors(self):
         w = self.w
@@ -676,6 +678,7 @@ class TimeMix(_RowPacked):
 
 class SSD(_RowPacked):
     """State-space duality with a short convolution, normed in parts after its gate (see ``ops.ssd``)."""
+    tile = CONV_TILE
 
     def __init__(self, width: int, heads: int, vdim: int, state: int, groups: int, conv: int, norm_parts: int, eps: float, dtype, device):
         super().__init__(dtype, device)

@@ -31,7 +31,7 @@ _native.register_signatures({
     "tsb_stage_gather": [P, P, P, P, P, I, I, I, I, P],
     "tsb_ragged_attn": [P, L, P, P, P, I, P, P, P, I, I, I, I, I, I, P, P, P, I, P],
     "tsb_paged_decode_shaped": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, P, P, I, P],
-    "tsb_flash_fwd_shaped": [P, P, P, P, P, P, I, I, I, I, I, I, I, P, P, P, P],
+    "tsb_flash_fwd_shaped": [P, P, P, P, P, P, I, I, I, I, I, I, I, P, P, P, F, P],
     "tsb_attn_prepare": [P, P, P, I, P],
     "tsb_flash_fwd_varlen_keys": [P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, L, L, L, L, L, L, F, P],
 })
@@ -56,16 +56,19 @@ def tensor_core_heads(D: int, dtype: torch.dtype) -> bool:
 class ScoreForm:
     """What becomes of the products q . k before and in the softmax: s = scale (q . k); s = softcap tanh(s / softcap) where a
     softcap is given; s -= slopes[h] (i - j) (``slopes`` fp32 [heads]); exp(sink[h]) joins the denominator (``sink`` fp32
-    [heads])."""
+    [heads]). ``product_bound``: no |q . k| is larger (0: not known)."""
     scale: float
     mask: Mask = 0
     softcap: float = 0.0
     slopes: Optional[torch.Tensor] = None
     sink: Optional[torch.Tensor] = None
+    product_bound: float = 0.0
 
     @property
-    def plain(self) -> bool:
-        return not isinstance(self.mask, Window) and self.softcap == 0.0 and self.slopes is None and self.sink is None
+    def bound(self) -> float:
+        """No |score| is larger before distances are taken off (0: not known)."""
+        known = [b for b in (self.softcap, self.product_bound * abs(self.scale)) if b > 0.0]
+        return min(known) * 1.001 if known else 0.0      # (products of rounded vectors may end slightly above)
 
 
 @dataclass
@@ -74,10 +77,6 @@ class OutputGate:
     gate: Optional[torch.Tensor] = None
     per_element: bool = False
     scale: float = 1.0
-
-    @property
-    def plain(self) -> bool:
-        return self.gate is None and self.scale == 1.0
 
 
 _PLAIN_GATE = OutputGate()
@@ -126,7 +125,7 @@ def _attend(q, stage, k_pool, v_pool, batch, form: ScoreForm, gate: OutputGate, 
         later = OutputGate(gate.gate[nd:] if gate.gate is not None else None, gate.per_element, gate.scale)
         check(lib().tsb_flash_fwd_shaped(q[nd:].data_ptr(), stage.data_ptr(), stage[:, G:].data_ptr(), out[nd:].data_ptr(), seg.cu_q.data_ptr(),
                                          seg.cu_k.data_ptr(), seg.n, seg.max_q, n, seg.keys, H, G, D, *_attention_args(form, later, ldo),
-                                         st), "tsb_flash_fwd_shaped")
+                                         float(form.bound), st), "tsb_flash_fwd_shaped")
 
 
 def ragged_attention(qkv: torch.Tensor, bias, k_pool: torch.Tensor, v_pool: torch.Tensor, batch, heads: int, kv_heads: int,

@@ -25,6 +25,7 @@ _native.register_signatures({
 })
 MAX_STATE = 256
 MAX_TAPS = 8
+CONV_TILE = 16          # tokens of a portion that a thread of the convolution walks
 
 
 def _up(n: int, m: int) -> int:
@@ -145,12 +146,13 @@ def ssd(proj: torch.Tensor, geo: SSDGeometry, w: SSDWeights, conv_state: torch.T
         n = T - nd
         xbc = torch.empty((T, geo.conv_cols), device=proj.device, dtype=proj.dtype)
         gates = torch.empty((T, H, 2), device=proj.device, dtype=torch.float32)       # dt, log2 of the decay
-        blocks = batch.blk_seq.shape[0] if n else 0
-        ints = geo.ints(T, nd, batch.n_prompts, blocks, proj.stride(0), out.stride(0))
+        tiles = batch.tiles(CONV_TILE) if n else None
+        ints = geo.ints(T, nd, batch.n_prompts, tiles.n if n else 0, proj.stride(0), out.stride(0))
         some = lambda name: getattr(batch, name).data_ptr() if n else None   # noqa: E731
         ptrs = (ctypes.c_void_p * 14)(proj.data_ptr(), w.conv.data_ptr(), w.conv_b.data_ptr(), w.a_log.data_ptr(), w.dt_bias.data_ptr(),
                                       conv_state.data_ptr(), xbc.data_ptr(), gates.data_ptr(), batch.state_slots.data_ptr(),
-                                      batch.positions.data_ptr(), some("cu"), some("pos0"), some("blk_seq"), some("blk0"))
+                                      batch.positions.data_ptr(), some("cu"), some("pos0"), tiles.seq.data_ptr() if n else None,
+                                      tiles.first.data_ptr() if n else None)
         check(lib().tsb_ssd_conv(ints, ptrs, dt, st), "tsb_ssd_conv")
         if nd:
             ptrs = (ctypes.c_void_p * 8)(proj.data_ptr(), xbc.data_ptr(), gates.data_ptr(), w.d.data_ptr(), state.data_ptr(),

@@ -297,7 +297,8 @@ ATT = {
     "whole": dict(heads=5, kv=1, dim=9, vdim=22, window=1, bias=True, norm="whole", rotary=Rotary(4, 90.0), gate="head"),
     "whole64": dict(heads=4, kv=4, dim=50, vdim=64, window=129, bias=True, norm="whole", rotary=Rotary(20, 90.0), gate="head"),
     "long": dict(heads=2, kv=1, dim=200, vdim=130, window=40, bias=True, norm="whole", rotary=Rotary(100, 90.0), gate="head"),
-    # parts that the design does not put together
+    # parts that the design does not put together, a cap that bounds nothing
+    "loose": dict(heads=2, kv=1, dim=64, vdim=48, window=140, norm="head", slopes=True, softcap=90.0, sink="learned", gate="head"),
     "bare": dict(heads=2, kv=1, dim=64, vdim=64),
     "sinks": dict(heads=2, kv=2, dim=64, vdim=64, sink="learned", norm="unit", slopes=True, softcap=3.0, window=77, gate="element"),
 }
