@@ -589,6 +589,26 @@ def case_shaped_attn(b: Bench):
         report("shaped_attn_decode", ms, bytes_=n * (window or 1400) * 8 * 128 * 2 * 2.0, shape=[n, 1400, window])
 
 
+def case_attn_prepare(b: Bench):
+    """What comes before attention, alone: biases, norms, rotation, append to the pool and to the key axis (bytes of q, k, v in and out,
+    k and v twice), beside the plain append of chunk_attn."""
+    from tesseract_b200 import ops
+    from tesseract_b200.nn.ragged import PagedRun
+    from tesseract_b200.ops import ragged
+    n, rows, H, G, D = 4, 4096, 32, 8, 128
+    saved, ragged._attend = ragged._attend, lambda *a: None
+    try:
+        for name, window in (("capped", 0), ("window", 1024)):
+            ms = _mixer_case(b, _shaped(b, window), n, rows)
+            report("attn_prepare_" + name, ms, bytes_=n * rows * D * 2.0 * (2 * H + (5 if window else 6) * G), shape=[n, rows])
+        st = _Step(b, PagedRun(G, D), n, rows, 0, (0,))
+        qkv, bias = b.randn(n * rows, (H + 2 * G) * D), torch.zeros((H + 2 * G) * D, device=b.dev)
+        ms = b.time(lambda: ops.ragged_attention(qkv, bias, *st.cache.runs[0], st.batch, H, G, D ** -0.5, 0))
+        report("ragged_append", ms, bytes_=n * rows * D * 2.0 * (2 * H + 6 * G), shape=[n, rows])
+    finally:
+        ragged._attend = saved
+
+
 def case_time_mix(b: Bench):
     """Prompts: bytes of r, k, v, gate and the result; decode: the state read and written once."""
     from tesseract_b200.nn.hybrid import TimeMix
@@ -668,7 +688,7 @@ CASES = {"gemm": case_gemm, "gemm_fp8": case_gemm_fp8, "gemm_fp8_pertensor": cas
          "ag_gemm_emul": case_ag_gemm_emul, "stream_linear": case_stream_linear, "mx_linear": case_mx_linear, "gemm_mx": case_gemm_mx,
          "delta_prefill": case_delta_prefill, "delta_step": case_delta_step, "chunk_attn": case_chunk_attn,
          "dyn_tanh": case_dyn_tanh, "clamped_glu": case_clamped_glu, "retention": case_retention, "latent": case_latent, "rglru": case_rglru,
-         "depth_residual": case_depth_residual, "silu_glu": case_silu_glu, "shaped_attn": case_shaped_attn, "time_mix": case_time_mix,
+         "depth_residual": case_depth_residual, "silu_glu": case_silu_glu, "shaped_attn": case_shaped_attn, "attn_prepare": case_attn_prepare, "time_mix": case_time_mix,
          "ssd": case_ssd, "post_norm": case_post_norm, "token_side": case_token_side, "token_shift": case_token_shift,
          "project_inputs": case_project_inputs}
 

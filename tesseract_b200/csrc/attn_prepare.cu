@@ -27,6 +27,21 @@ struct PrepareParams {
   const int* stage_rows;      // [rows - n_decode]
 };
 
+// V consecutive floats (16-byte aligned), multiplied in.
+template <int V>
+__device__ __forceinline__ void scale_by(float (&f)[V], float r, const float* w) {
+  if (!w) {
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] *= r;
+    return;
+  }
+#pragma unroll
+  for (int i = 0; i < V; i += 4) {
+    const float4 a = *reinterpret_cast<const float4*>(w + i);
+    f[i] *= r * a.x; f[i + 1] *= r * a.y; f[i + 2] *= r * a.z; f[i + 3] *= r * a.w;
+  }
+}
+
 template <typename T, int LPH, int PPL>
 __global__ void __launch_bounds__(256)
 attn_prepare_kernel(PrepareParams p) {
@@ -41,7 +56,10 @@ attn_prepare_kernel(PrepareParams p) {
     ld16<T>(x + col, f);
     if (p.bias) {
 #pragma unroll
-      for (int i = 0; i < V; ++i) f[i] += p.bias[col + i];
+      for (int i = 0; i < V; i += 4) {
+        const float4 b = *reinterpret_cast<const float4*>(p.bias + col + i);
+        f[i] += b.x; f[i + 1] += b.y; f[i + 2] += b.z; f[i + 3] += b.w;
+      }
     }
   };
   float whole_q = 0.f, whole_k = 0.f;
@@ -75,70 +93,79 @@ attn_prepare_kernel(PrepareParams p) {
   const long long page = slot >= 0 ? static_cast<long long>(slot / p.bs) * p.Hkv * p.bs + slot % p.bs : 0;
   const int stage_row = p.stage && row >= p.n_decode ? p.stage_rows[row - p.n_decode] : -1;
   const float2* turn = p.table && p.hp > 0 ? p.table + static_cast<long long>(max(p.positions[row], 0)) * p.hp : nullptr;
-  for (int u0 = 0; u0 < units; u0 += step) {        // (every lane takes every turn: the sums below are shuffles)
-    const int u = u0 + first;
-    const bool there = u < units;
-    const int kind = u < p.H ? 0 : u < p.H + p.Hkv ? 1 : 2;
-    const int head = kind == 0 ? u : kind == 1 ? u - p.H : u - p.H - p.Hkv;
-    const int col = (kind == 0 ? 0 : kind == 1 ? p.off_k : p.off_v) + head * D;
-    float f[PPL][V], ss = 0.f;
+  constexpr int U = PPL == 1 ? 2 : 1;               // heads whose loads are requested together
+  for (int u0 = 0; u0 < units; u0 += U * step) {    // (every lane takes every turn: the sums below are shuffles)
+    float f[U][PPL][V], ss[U];
+    int kind[U], head[U], col[U];
 #pragma unroll
-    for (int k = 0; k < PPL; ++k) {
-      const int d = (gl + k * LPH) * V;
+    for (int q = 0; q < U; ++q) {
+      const int u = u0 + q * step + first;
+      kind[q] = u < p.H ? 0 : u < p.H + p.Hkv ? 1 : u < units ? 2 : 3;      // q, k, v, nothing
+      head[q] = kind[q] == 0 ? u : kind[q] == 1 ? u - p.H : u - p.H - p.Hkv;
+      col[q] = (kind[q] == 0 ? 0 : kind[q] == 1 ? p.off_k : p.off_v) + head[q] * D;
 #pragma unroll
-      for (int i = 0; i < V; ++i) f[k][i] = 0.f;
-      if (there && d < D) load(col + d, f[k]);
+      for (int k = 0; k < PPL; ++k) {
+        const int d = (gl + k * LPH) * V;
 #pragma unroll
-      for (int i = 0; i < V; ++i) ss = fmaf(f[k][i], f[k][i], ss);
-    }
-    float rs = kind == 0 ? whole_q : whole_k;
-    if (p.norm == 1 || p.norm == 2) {
-#pragma unroll
-      for (int o = LPH / 2; o; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      rs = 1.f / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
-    }
-    if (!there) continue;
-    const float* w = p.norm < 2 ? nullptr : (kind == 0 ? p.q_norm : p.k_norm) + (p.norm == 3 ? head * D : 0);
-#pragma unroll
-    for (int k = 0; k < PPL; ++k) {
-      const int d = (gl + k * LPH) * V;
-      if (d >= D) continue;
-      if (kind == 2) {
-        if (p.v_first) {
-          float v0[V] = {};
-          if (slot >= 0 && d < p.D_first)
-            ld16<T>(static_cast<const T*>(p.v_first) + (page + static_cast<long long>(head) * p.bs) * p.D_first + d, v0);
-#pragma unroll
-          for (int i = 0; i < V; ++i) f[k][i] = (1.f - p.vmix) * f[k][i] + p.vmix * v0[i];
-        }
-      } else {
-        if (p.norm) {
-#pragma unroll
-          for (int i = 0; i < V; ++i) f[k][i] *= w ? rs * w[d + i] : rs;
-        }
-        if (turn && d < 2 * p.hp) {
-          const bool second = d >= p.hp;
-          const int i0 = second ? d - p.hp : d, other = second ? i0 : d + p.hp;
-          float g[V];
-          load(col + other, g);
-          if (p.norm) {
-#pragma unroll
-            for (int i = 0; i < V; ++i) g[i] *= w ? rs * w[other + i] : rs;
-          }
-#pragma unroll
-          for (int i = 0; i < V; ++i) {
-            const float2 cs = turn[i0 + i];
-            f[k][i] = second ? f[k][i] * cs.x + g[i] * cs.y : f[k][i] * cs.x - g[i] * cs.y;
-          }
-        }
+        for (int i = 0; i < V; ++i) f[q][k][i] = 0.f;
+        if (kind[q] < 3 && d < D) load(col[q] + d, f[q][k]);
       }
-      if (kind == 0) {
-        st16<T>(static_cast<T*>(p.q) + (static_cast<long long>(row) * p.H + head) * D + d, f[k]);
-        continue;
+    }
+#pragma unroll
+    for (int q = 0; q < U; ++q) {
+      ss[q] = 0.f;
+#pragma unroll
+      for (int k = 0; k < PPL; ++k)
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss[q] = fmaf(f[q][k][i], f[q][k][i], ss[q]);
+      if (p.norm == 1 || p.norm == 2) {
+#pragma unroll
+        for (int o = LPH / 2; o; o >>= 1) ss[q] += __shfl_xor_sync(0xffffffffu, ss[q], o);
       }
-      if (slot >= 0) st16<T>(static_cast<T*>(kind == 1 ? p.k_pool : p.v_pool) + (page + static_cast<long long>(head) * p.bs) * D + d, f[k]);
-      if (stage_row >= 0)
-        st16<T>(static_cast<T*>(p.stage) + (static_cast<long long>(stage_row) * 2 * p.Hkv + (kind == 1 ? 0 : p.Hkv) + head) * D + d, f[k]);
+    }
+#pragma unroll
+    for (int q = 0; q < U; ++q) {
+      if (kind[q] == 3) continue;
+      const float rs = p.norm == 3 ? (kind[q] == 0 ? whole_q : whole_k) : 1.f / sqrtf(ss[q] / static_cast<float>(p.dim) + p.eps);
+      const float* w = p.norm < 2 ? nullptr : (kind[q] == 0 ? p.q_norm : p.k_norm) + (p.norm == 3 ? head[q] * D : 0);
+#pragma unroll
+      for (int k = 0; k < PPL; ++k) {
+        const int d = (gl + k * LPH) * V;
+        if (d >= D) continue;
+        float(&x8)[V] = f[q][k];
+        if (kind[q] == 2) {
+          if (p.v_first) {
+            float v0[V] = {};
+            if (slot >= 0 && d < p.D_first)
+              ld16<T>(static_cast<const T*>(p.v_first) + (page + static_cast<long long>(head[q]) * p.bs) * p.D_first + d, v0);
+#pragma unroll
+            for (int i = 0; i < V; ++i) x8[i] = (1.f - p.vmix) * x8[i] + p.vmix * v0[i];
+          }
+        } else {
+          if (p.norm) scale_by<V>(x8, rs, w ? w + d : nullptr);
+          if (turn && d < 2 * p.hp) {
+            const bool second = d >= p.hp;
+            const int i0 = second ? d - p.hp : d, other = second ? i0 : d + p.hp;
+            float g[V];
+            load(col[q] + other, g);
+            if (p.norm) scale_by<V>(g, rs, w ? w + other : nullptr);
+#pragma unroll
+            for (int i = 0; i < V; i += 2) {
+              const float4 cs = *reinterpret_cast<const float4*>(turn + i0 + i);
+              const float s0 = second ? cs.y : -cs.y, s1 = second ? cs.w : -cs.w;
+              x8[i] = x8[i] * cs.x + g[i] * s0;
+              x8[i + 1] = x8[i + 1] * cs.z + g[i + 1] * s1;
+            }
+          }
+        }
+        if (kind[q] == 0) {
+          st16<T>(static_cast<T*>(p.q) + (static_cast<long long>(row) * p.H + head[q]) * D + d, x8);
+          continue;
+        }
+        if (slot >= 0) st16<T>(static_cast<T*>(kind[q] == 1 ? p.k_pool : p.v_pool) + (page + static_cast<long long>(head[q]) * p.bs) * D + d, x8);
+        if (stage_row >= 0)
+          st16<T>(static_cast<T*>(p.stage) + (static_cast<long long>(stage_row) * 2 * p.Hkv + (kind[q] == 1 ? 0 : p.Hkv) + head[q]) * D + d, x8);
+      }
     }
   }
 }

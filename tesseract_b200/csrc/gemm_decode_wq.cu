@@ -129,11 +129,20 @@ __device__ __forceinline__ uint32_t mul_bf16x2(uint32_t a, uint32_t b) {
   return d;
 }
 
-// Several inputs of the same batch rows, stacked `rows` apart in X: result columns from first[i] on read the i-th (tiles do not
-// straddle a start). n = 0: one input.
+// Several inputs of the same batch rows, stacked `rows` apart in X: result columns [first[i], first[i + 1]) read the i-th and are cut
+// into tiles of their own, the first of which is tile0[i]. n = 0: one input.
 struct Inputs {
   int n = 0, rows = 0;
-  int first[8] = {};
+  int first[9] = {}, tile0[9] = {};
+
+  int count(int bn) const {
+    int t = 0;
+    for (int i = 0; i < n; ++i) t += (first[i + 1] - first[i] + bn - 1) / bn;
+    return t;
+  }
+  void cut(int bn) {
+    for (int i = 0; i < n; ++i) tile0[i + 1] = tile0[i] + (first[i + 1] - first[i] + bn - 1) / bn;
+  }
 };
 
 template <int S, bool FP8, int RB>
@@ -161,7 +170,16 @@ gemm_decode_wq_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_cons
   const int lane = threadIdx.x & 31;
   const int slice = static_cast<int>(cluster_ctarank());
   const int tile = static_cast<int>(blockIdx.x) / S;
-  const int n0 = tile * BN;
+  int n0 = tile * BN, x_off = 0;
+  if (inputs.n) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (i < inputs.n && tile >= inputs.tile0[i]) {
+        n0 = inputs.first[i] + (tile - inputs.tile0[i]) * BN;
+        N = inputs.first[i + 1];
+        x_off = i * inputs.rows;
+      }
+  }
   const int m0 = static_cast<int>(blockIdx.y) * BM * RB;
   constexpr int kXBlock = BM * BK * 2;             // one 128-row activation tile inside a stage
   const int total_kb = (K + BK - 1) / BK;
@@ -205,10 +223,7 @@ gemm_decode_wq_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_cons
       uint64_t* w_full = FP8 ? full_r : full_c;
       uint64_t* w_empty = FP8 ? empty_r : empty_c;
       uint8_t* w_base = FP8 ? sR : sC;
-      int x_row = m0;
-#pragma unroll
-      for (int i = 1; i < 8; ++i)
-        if (i < inputs.n && n0 >= inputs.first[i]) x_row = m0 + i * inputs.rows;
+      const int x_row = m0 + x_off;
       const uint32_t w_pitch = static_cast<uint32_t>(FP8 ? L.r_pitch : L.c_pitch);
       int w_issued = 0, ws = 0, x_issued = 0, xs = 0;
       uint32_t wphase = 0, xphase = 0;
@@ -537,7 +552,7 @@ int launch_wq(const CUtensorMap& tx, const CUtensorMap& tw, const void* w_packed
   pdl &= 1;
   cudaLaunchConfig_t cfg;
   cudaLaunchAttribute at[2];
-  const int tiles = (N + BN - 1) / BN;
+  const int tiles = inputs.n ? inputs.count(BN) : (N + BN - 1) / BN;
   cudaError_t e = config_wq<S, FP8, RB>(&cfg, at, tiles * S, (M + RB * BM - 1) / (RB * BM), pdl, s);
   if (e != cudaSuccess) return static_cast<int>(e);
   return static_cast<int>(cudaLaunchKernelEx(&cfg, gemm_decode_wq_kernel<S, FP8, RB>, tx, tw,
@@ -587,7 +602,7 @@ bool layout_ok(const Layout& L, bool fp8, int bn, int rb) {
 
 // One candidate family: tile widths and K splits for a given number of row blocks per CTA. Returns the score of the
 // best single-wave plan (< 0 if there is none).
-double plan_family(int M, int N, int kb, bool fp8, int fixed_bn, int rb, int* bn_out, int* split_out) {
+double plan_family(int M, int N, int kb, bool fp8, int fixed_bn, int rb, int* bn_out, int* split_out, const Inputs* inputs = nullptr) {
   const int row_ctas = (M + rb * BM - 1) / (rb * BM);
   double best = -1.0;
   for (int s : {1, 2, 4, 8}) {
@@ -600,7 +615,7 @@ double plan_family(int M, int N, int kb, bool fp8, int fixed_bn, int rb, int* bn
       if (fixed_bn > 0 && bn != fixed_bn) continue;
       const Layout L = make_layout(M, bn, fp8, rb);
       if (!layout_ok(L, fp8, bn, rb)) continue;
-      const int tiles = (N + bn - 1) / bn;
+      const int tiles = inputs ? inputs->count(bn) : (N + bn - 1) / bn;
       const int ctas = tiles * s * row_ctas;
       if (ctas > cap) continue;
       const double useful = static_cast<double>(N) / (static_cast<double>(tiles) * bn);
@@ -747,7 +762,7 @@ TSB_EXPORT int tsb_gemm_decode_wq_plan(int M, int N, int K, int w_fp8, int* bn, 
 }
 
 // Y [M, N] whose column ranges read different inputs: columns [starts[i], starts[i + 1]) are X_i [M, K] * W[N, K]^T, X_i starting
-// i * x_rows rows after X (x_rows >= M). Host array `starts` ascends from 0 in multiples of 128; n <= 8. bf16 weights, otherwise as
+// i * x_rows rows after X (x_rows >= M). Host array `starts` ascends from 0 in multiples of 16; n <= 8. bf16 weights, otherwise as
 // above.
 TSB_EXPORT int tsb_gemm_decode_inputs(const int* starts, const void* X, const void* W, void* Y, int n, int M, int N, int K, long long x_rows,
                                       long long ldx, long long ldw, long long ldy, int pdl, void* stream) {
@@ -757,27 +772,16 @@ TSB_EXPORT int tsb_gemm_decode_inputs(const int* starts, const void* X, const vo
   Inputs in;
   in.n = n;
   in.rows = static_cast<int>(x_rows);
-  int unit = 256;
   for (int i = 0; i < n; ++i) {
-    if (starts[i] % 128 || (i && starts[i] <= starts[i - 1]) || starts[i] >= N) return -2;
+    if (starts[i] % 16 || (i && starts[i] <= starts[i - 1]) || starts[i] >= N) return -2;
     in.first[i] = starts[i];
-    if (starts[i] % 256) unit = 128;
   }
-  const int kb = (K + BK - 1) / BK;
+  in.first[n] = N;
+  const int kb = (K + BK - 1) / BK, rb = M > BM ? 2 : 1;
   int bn = 0, split = 1;
-  double best = -1.0;
-  const int rb = M > BM ? 2 : 1;
-  for (int b = unit; b >= 32; b /= 2) {            // widths that divide every start
-    int pb = 0, ps = 0;
-    const double sc = plan_family(M, N, kb, false, b, rb, &pb, &ps);
-    if (sc > best) {
-      best = sc;
-      bn = pb;
-      split = ps;
-    }
-  }
-  if (best < 0.0)                                  // several waves of the widest tile that has room
-    for (bn = unit; bn > 32 && !layout_ok(make_layout(M, bn, false, rb), false, bn, rb);) bn /= 2;
+  if (plan_family(M, N, kb, false, 0, rb, &bn, &split, &in) < 0.0)      // several waves of the widest tile that has room
+    for (bn = kMaxBN; bn > 32 && !layout_ok(make_layout(M, bn, false, rb), false, bn, rb);) bn -= 16;
+  in.cut(bn);
   const Layout L = make_layout(M, bn, false, rb);
   if (L.c_stages < 2 || rb * BM * (bn * 4 + 16) > kSmemBudget - 1024) return -2;
   CUtensorMap tx, tw;

@@ -20,7 +20,7 @@ import torch
 from .. import ops
 from ..ops.delta import DeltaGeometry, DeltaWeights, gated_delta
 from ..ops.latent import LatentGeometry, LatentWeights, latent_attention
-from ..ops.gemm import INPUT_ALIGN
+from ..ops.gemm import input_columns
 from ..ops.masks import Window
 from ..ops.ragged import AttentionGeometry, AttentionWeights, ScoreForm, padded_head_dim, ragged_attention, shaped_attention
 from ..ops.retention import SPAN, RetentionGeometry, log2_decays, retention
@@ -745,7 +745,7 @@ class SideBySide(_Mixer):
         self.left, self.right = left, right
         left.out_scale, right.out_scale = float(left_scale), float(right_scale)
         own = len(right.streams) > 1
-        self.cut = pad_to(left.cols, INPUT_ALIGN if own else 8)
+        self.cut = input_columns(left.cols) if own else pad_to(left.cols, 8)
         self.streams = (0,) + tuple(self.cut + s for s in right.streams) if own else (0,)
         self.w_in, self.w_out = self._zeros(self.cut + right.cols, pad_to(width)), self._zeros(width, left.out_cols + right.out_cols)
         left.place(self.w_in[:left.cols], self.w_out[:, :left.out_cols])

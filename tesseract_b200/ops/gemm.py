@@ -308,6 +308,12 @@ _native.register_signatures({
 INPUT_ALIGN = 128          # first result column of every input
 
 
+def input_columns(n: int) -> int:
+    """Columns to set aside for an input of ``n``: wide ones end where the widest tiles of the GEMM do."""
+    m = 256 if n >= 2048 else INPUT_ALIGN
+    return (n + m - 1) // m * m
+
+
 def project_inputs(xs: torch.Tensor, w: torch.Tensor, starts) -> torch.Tensor:
     """One product for several inputs of the same rows: result columns [starts[g], starts[g + 1]) are xs[g] [M, K] times those
     rows of w [N, K]. The starts are multiples of ``INPUT_ALIGN``; the tiles of either GEMM pick their input by their column."""

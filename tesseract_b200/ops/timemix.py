@@ -15,7 +15,7 @@ import torch
 
 from .. import _native
 from .._native import check, dtype_code, lib, stream_ptr
-from .gemm import INPUT_ALIGN, project
+from .gemm import input_columns, project
 
 P, I, L, F = _native.P, _native.I, _native.L, _native.F
 _native.register_signatures({
@@ -60,7 +60,7 @@ class TimeMixGeometry:
 
     @property
     def section(self) -> int:
-        return _up(self.heads * self.dp, INPUT_ALIGN)
+        return input_columns(self.heads * self.dp)
 
     @property
     def starts(self) -> tuple:
