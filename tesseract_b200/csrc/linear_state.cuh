@@ -139,4 +139,40 @@ __device__ __forceinline__ void state_scan(float* sm, float* st, int E, int D, b
     }
 }
 
+// A few long portions are cut into spans of kStateSpan tokens that are worked on at once: what every span but the last adds to
+// nothing and what it leaves of what was there, then this pass, then the read-outs from the state at the start of every span.
+constexpr int kStateSpan = 512;
+
+struct SpanParams {
+  const int* seq;            // [spans], or null: every portion is one
+  const int* first;          // [sequences + 1] first span of a sequence
+  float* carry;              // [spans, H, E, D]: what a span adds, then the state at its start
+  float* left;               // [spans, H, D or 1]: the factor that a span leaves of every column
+  int n;
+};
+
+static __global__ void __launch_bounds__(256)
+state_carry_kernel(SpanParams p, const float* state, const int* slots, const int* pos0, int E, int D, int per_column) {
+  pdl_trigger();
+  pdl_grid_wait();
+  const int i = (blockIdx.x * 256 + threadIdx.x) * 4, h = blockIdx.y, H = gridDim.y, seq = blockIdx.z;
+  const int first = p.first[seq], n = p.first[seq + 1] - first, slot = slots[seq];
+  if (i >= E * D || n < 2 || slot < 0) return;
+  const long long one = static_cast<long long>(E) * D;
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (pos0[seq] > 0) s = *reinterpret_cast<const float4*>(state + (static_cast<long long>(slot) * H + h) * one + i);
+  for (int k = 0; k < n; ++k) {
+    const long long at = static_cast<long long>(first + k) * H + h;
+    float4* c = reinterpret_cast<float4*>(p.carry + at * one + i);
+    const float4 add = k + 1 < n ? *c : make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 w = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (k + 1 < n) {
+      if (per_column) w = *reinterpret_cast<const float4*>(p.left + at * D + i % D);
+      else w.x = w.y = w.z = w.w = p.left[at];
+    }
+    *c = s;
+    s = make_float4(fmaf(w.x, s.x, add.x), fmaf(w.y, s.y, add.y), fmaf(w.z, s.z, add.z), fmaf(w.w, s.w, add.w));
+  }
+}
+
 }  // namespace tsb

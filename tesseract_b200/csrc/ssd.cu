@@ -43,6 +43,7 @@ struct SsdParams {
   const int* blk_seq;
   const int* blk0;
   void* out;                 // [rows, ldo]: y
+  SpanParams span;
 };
 
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
@@ -201,8 +202,9 @@ struct SsdChunk {
   static constexpr int kG = kPl + kTok * kLdX * 2, kL = kG + kTok * 8, kSmem = kL + 4 * kTok * 4;
 };
 
-// CTA = (head and 64 of its value columns, sequence); warp w owns the state's rows (values) 16 w .. + 15 of them.
-template <int NT>
+// CTA = (head and 64 of its value columns, sequence or span); warp w owns the state's rows (values) 16 w .. + 15 of them. OUT = false:
+// only what a span adds and leaves.
+template <int NT, bool OUT>
 __global__ void __launch_bounds__(128, NT <= 128 ? 3 : 1)
 ssd_chunk_kernel(SsdParams p) {
   using T = __nv_bfloat16;
@@ -214,9 +216,17 @@ ssd_chunk_kernel(SsdParams p) {
   T *sph = reinterpret_cast<T*>(smem + K::kPh), *spl = reinterpret_cast<T*>(smem + K::kPl);
   const float2* sg = reinterpret_cast<const float2*>(smem + K::kG);
   const int tiles = (p.vp + K::kCols - 1) / K::kCols, h = blockIdx.x / tiles, c0 = blockIdx.x % tiles * K::kCols;
-  const int seq = blockIdx.y, slot = p.slots[seq], grp = h / (p.H / p.G);
-  const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
-  if (slot < 0 || n <= 0) return;
+  const int seq = p.span.seq ? p.span.seq[blockIdx.y] : blockIdx.y, slot = p.slots[seq], grp = h / (p.H / p.G);
+  int row0 = p.cu[seq], n = p.cu[seq + 1] - row0, idx = 0, spans = 1;
+  if (p.span.seq) {
+    idx = blockIdx.y - p.span.first[seq];
+    spans = p.span.first[seq + 1] - p.span.first[seq];
+    row0 += idx * kStateSpan;
+    n = min(kStateSpan, n - idx * kStateSpan);
+  }
+  const bool final = idx == spans - 1;
+  if (slot < 0 || n <= 0 || (!OUT && final)) return;
+  float* carry = spans > 1 ? p.span.carry + (static_cast<long long>(blockIdx.y) * p.H + h) * p.vp * p.np : nullptr;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const T* xbc = static_cast<const T*>(p.xbc) + static_cast<long long>(row0) * p.conv_c;
   const T *x = xbc + h * p.vp + c0, *B = xbc + p.H * p.vp + grp * p.np, *C = B + p.G * p.np;
@@ -227,27 +237,28 @@ ssd_chunk_kernel(SsdParams p) {
   const float skip = p.d[h];
   float S[NT / 8][4];
   {
-    const bool old = p.pos0[seq] > 0;
+    const float* from = !OUT ? nullptr : carry ? carry : p.pos0[seq] > 0 ? st : nullptr;
 #pragma unroll
     for (int j = 0; j < NT / 8; ++j)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
         float2 v = make_float2(0.f, 0.f);
-        if (old && r < cols && c < p.np) v = *reinterpret_cast<const float2*>(st + static_cast<long long>(c0 + r) * p.np + c);
+        if (from && r < cols && c < p.np) v = *reinterpret_cast<const float2*>(from + static_cast<long long>(c0 + r) * p.np + c);
         S[j][2 * e] = v.x;
         S[j][2 * e + 1] = v.y;
       }
   }
   const uint32_t aC = smem_u32(sc), aB = smem_u32(sb), aX = smem_u32(sx), aPh = smem_u32(sph), aPl = smem_u32(spl);
 
+  float left = 0.f;                            // (OUT = false) logarithm of what the span leaves
   for (int t0 = 0; t0 < n; t0 += K::kTok) {
     const int cnt = min(K::kTok, n - t0);
     for (int i = tid; i < K::kTok * (NT / 8); i += K::kThreads) {
       const int r = i / (NT / 8), d = (i % (NT / 8)) * 8;
       const bool ok = r < cnt && d < p.np;
       const long long at = static_cast<long long>(t0 + r) * p.conv_c + d;
-      cp_async_16(aC + (r * K::kLdN + d) * 2, ok ? C + at : C, ok ? 16 : 0);
+      if constexpr (OUT) cp_async_16(aC + (r * K::kLdN + d) * 2, ok ? C + at : C, ok ? 16 : 0);
       cp_async_16(aB + (r * K::kLdN + d) * 2, ok ? B + at : B, ok ? 16 : 0);
     }
     for (int i = tid; i < K::kTok * (K::kCols / 8); i += K::kThreads) {
@@ -275,8 +286,9 @@ ssd_chunk_kernel(SsdParams p) {
       sl[2 * lane + 1] = sum;
       last = __shfl_sync(0xffffffffu, sum, 31);
       __syncwarp();
+      left += last;
     }
-    {
+    if constexpr (OUT) {
       // decayed scores: this warp's 16 keys j against the tokens i from their block on
       float a[8][4];
 #pragma unroll
@@ -306,12 +318,13 @@ ssd_chunk_kernel(SsdParams p) {
         split_bf16x2(f2, f3, reinterpret_cast<uint32_t*>(sph + j1 * K::kLdX + i), reinterpret_cast<uint32_t*>(spl + j1 * K::kLdX + i));
       }
     }
-    __syncthreads();
+    if constexpr (OUT) __syncthreads();
     float acc[8][4];
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < NT / 16; ++ks) {
+      if (!OUT) break;
       uint32_t hi[4], lo[4];
       split_bf16x2(S[2 * ks][0], S[2 * ks][1], &hi[0], &lo[0]);
       split_bf16x2(S[2 * ks][2], S[2 * ks][3], &hi[1], &lo[1]);
@@ -329,6 +342,7 @@ ssd_chunk_kernel(SsdParams p) {
     }
 #pragma unroll
     for (int b = 0; b < 8; ++b) {
+      if (!OUT) break;
       const float la = exp2f(sl[b * 8 + 2 * t4]), lb = exp2f(sl[b * 8 + 2 * t4 + 1]);
       acc[b][0] *= la; acc[b][1] *= lb; acc[b][2] *= la; acc[b][3] *= lb;
     }
@@ -344,7 +358,7 @@ ssd_chunk_kernel(SsdParams p) {
       ldmat_x4_trans(xt, aX + frag_a_trans(lane, jb * 16, e0, K::kLdX));
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        if (i < jb) continue;
+        if (!OUT || i < jb) continue;
         uint32_t ph[4], pl[4];
         ldmat_x4_trans(ph, aPh + frag_b_trans(lane, jb * 16, i * 16, K::kLdX));
         ldmat_x4_trans(pl, aPl + frag_b_trans(lane, jb * 16, i * 16, K::kLdX));
@@ -374,6 +388,10 @@ ssd_chunk_kernel(SsdParams p) {
         mma_bf16(S[j + 1], lo, b[2], b[3]);
       }
     }
+    if constexpr (!OUT) {
+      __syncthreads();
+      continue;
+    }
     // y takes the place of x (a warp's own columns)
     __syncwarp();
 #pragma unroll
@@ -393,13 +411,16 @@ ssd_chunk_kernel(SsdParams p) {
     }
     __syncthreads();
   }
+  float* to = !OUT ? carry : final ? st : nullptr;
+  if (!to) return;
+  if (!OUT && tid == 0 && c0 == 0) p.span.left[static_cast<long long>(blockIdx.y) * p.H + h] = exp2f(left);
 #pragma unroll
   for (int j = 0; j < NT / 8; ++j)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
       if (r < cols && c < p.np)
-        *reinterpret_cast<float2*>(st + static_cast<long long>(c0 + r) * p.np + c) = make_float2(S[j][2 * e], S[j][2 * e + 1]);
+        *reinterpret_cast<float2*>(to + static_cast<long long>(c0 + r) * p.np + c) = make_float2(S[j][2 * e], S[j][2 * e + 1]);
     }
 }
 
@@ -503,9 +524,9 @@ int run_scan(const SsdParams& p, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int NT>
-int run_chunk(const SsdParams& p, cudaStream_t s) {
-  auto kern = ssd_chunk_kernel<NT>;
+template <int NT, bool OUT>
+int launch_chunk(const SsdParams& p, cudaStream_t s) {
+  auto kern = ssd_chunk_kernel<NT, OUT>;
   static PerDeviceFlag attr;
   if (attr.unset()) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SsdChunk<NT>::kSmem);
@@ -513,8 +534,19 @@ int run_chunk(const SsdParams& p, cudaStream_t s) {
     attr.set();
   }
   const int tiles = (p.vp + SsdChunk<NT>::kCols - 1) / SsdChunk<NT>::kCols;
-  launch_pdl(kern, dim3(p.H * tiles, p.n_seq), dim3(SsdChunk<NT>::kThreads), SsdChunk<NT>::kSmem, s, pdl_all_enabled(), p);
+  launch_pdl(kern, dim3(p.H * tiles, p.span.seq ? p.span.n : p.n_seq), dim3(SsdChunk<NT>::kThreads), SsdChunk<NT>::kSmem, s,
+             pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <int NT>
+int run_chunk(const SsdParams& p, cudaStream_t s) {
+  if (p.span.seq) {
+    if (const int rc = launch_chunk<NT, false>(p, s)) return rc;
+    launch_pdl(state_carry_kernel, dim3((p.vp * p.np / 4 + 255) / 256, p.H, p.n_seq), dim3(256), 0, s, pdl_all_enabled(), p.span,
+               static_cast<const float*>(p.state), p.slots, p.pos0, p.vp, p.np, 0);
+  }
+  return launch_chunk<NT, true>(p, s);
 }
 
 template <typename T>
@@ -576,8 +608,10 @@ TSB_EXPORT int tsb_ssd_step(const int* ints, void* const* q, int dtype, void* st
   return -2;
 }
 
-// ptrs: proj, xbc, gates, d, state, slots, cu, pos0, out, all from the first prompt row (sequence) on.
-TSB_EXPORT int tsb_ssd_prefill(const int* ints, void* const* q, int dtype, void* stream) {
+// ptrs: proj, xbc, gates, d, state, slots, cu, pos0, out, all from the first prompt row (sequence) on; for `spans` spans of 512 tokens
+// (0, or fp32: every portion is walked in one) their sequences, the first span of every sequence, carry [spans, H, vp, np], left
+// [spans, H].
+TSB_EXPORT int tsb_ssd_prefill(const int* ints, void* const* q, int spans, int dtype, void* stream) {
   using namespace tsb;
   SsdParams p{};
   if (!read_ssd(ints, &p) || p.n_seq <= 0) return -2;
@@ -586,6 +620,10 @@ TSB_EXPORT int tsb_ssd_prefill(const int* ints, void* const* q, int dtype, void*
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (dtype == 1) {
     if (p.ldo % 8 || (reinterpret_cast<uintptr_t>(p.out) & 15)) return -2;
+    if (spans > 0) {
+      p.span = {static_cast<const int*>(q[9]), static_cast<const int*>(q[10]), static_cast<float*>(q[11]), static_cast<float*>(q[12]), spans};
+      if (spans > 65535 || !p.span.seq || !p.span.first || !p.span.carry || !p.span.left) return -2;
+    }
     return p.np <= 64 ? run_chunk<64>(p, s) : p.np <= 128 ? run_chunk<128>(p, s) : run_chunk<256>(p, s);
   }
   if (dtype == 0) return run_scan<float>(p, s);

@@ -116,6 +116,7 @@ struct MixParams {
   const int* pos0;
   void* out;                 // [rows, ldo]
   float* o;                  // [rows, H, dp] read-outs of the scan
+  SpanParams span;
   float eps, out_scale;
 };
 
@@ -206,8 +207,9 @@ __device__ __forceinline__ float transpose_sum(float (&v)[N], int lane) {
   return v[0];
 }
 
-// CTA = (head, sequence); warp w owns the state's rows (values) 16 w .. + 15. The next 64 tokens arrive while some are worked on.
-template <int DT>
+// CTA = (head, sequence or span); warp w owns the state's rows (values) 16 w .. + 15. The next 64 tokens arrive while some are
+// worked on. OUT = false: only what a span adds and leaves.
+template <int DT, bool OUT>
 __global__ void __launch_bounds__(MixChunk<DT>::kThreads, DT == 64 ? 2 : 1)
 time_mix_chunk_kernel(MixParams p) {
   using T = __nv_bfloat16;
@@ -218,11 +220,19 @@ time_mix_chunk_kernel(MixParams p) {
   T *srl = reinterpret_cast<T*>(smem + C::kRl), *skl = reinterpret_cast<T*>(smem + C::kKl);
   float *sa = reinterpret_cast<float*>(smem + C::kA), *stot = reinterpret_cast<float*>(smem + C::kTot);
   float* sbonus = reinterpret_cast<float*>(smem + C::kBonus);
-  const int h = blockIdx.x, seq = blockIdx.y, slot = p.slots[seq];
-  const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
-  if (slot < 0 || n <= 0) return;
+  const int h = blockIdx.x, seq = p.span.seq ? p.span.seq[blockIdx.y] : blockIdx.y, slot = p.slots[seq];
+  int row0 = p.cu[seq], n = p.cu[seq + 1] - row0, idx = 0, spans = 1;
+  if (p.span.seq) {
+    idx = blockIdx.y - p.span.first[seq];
+    spans = p.span.first[seq + 1] - p.span.first[seq];
+    row0 += idx * kStateSpan;
+    n = min(kStateSpan, n - idx * kStateSpan);
+  }
+  const bool last = idx == spans - 1;
+  if (slot < 0 || n <= 0 || (!OUT && last)) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const T* proj = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ld + h * p.dp;
+  float* carry = spans > 1 ? p.span.carry + (static_cast<long long>(blockIdx.y) * p.H + h) * p.dp * p.dp : nullptr;
   const float* dec = p.dec + static_cast<long long>(row0) * p.H * p.dp + h * p.dp;
   float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp;
   const int e0 = warp * 16;
@@ -236,7 +246,7 @@ time_mix_chunk_kernel(MixParams p) {
       const T* src = ok ? proj + static_cast<long long>(t0 + r) * p.ld + d : proj;
       const int bytes = ok ? 16 : 0, sec = ok ? p.section : 0;
       const uint32_t at = base + (r * C::kLd + d) * 2;
-      cp_async_16(at + C::kR, src, bytes);
+      if constexpr (OUT) cp_async_16(at + C::kR, src, bytes);
       cp_async_16(at + C::kK, src + sec, bytes);
       cp_async_16(at + C::kV, src + 2 * sec, bytes);
     }
@@ -250,14 +260,14 @@ time_mix_chunk_kernel(MixParams p) {
   issue(0);
   float S[DT / 8][4];
   {
-    const bool old = p.pos0[seq] > 0;
+    const float* from = !OUT ? nullptr : carry ? carry : p.pos0[seq] > 0 ? st : nullptr;
 #pragma unroll
     for (int j = 0; j < DT / 8; ++j)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
         float2 v = make_float2(0.f, 0.f);
-        if (old && r < p.dp && c < p.dp) v = *reinterpret_cast<const float2*>(st + static_cast<long long>(r) * p.dp + c);
+        if (from && r < p.dp && c < p.dp) v = *reinterpret_cast<const float2*>(from + static_cast<long long>(r) * p.dp + c);
         S[j][2 * e] = v.x;
         S[j][2 * e + 1] = v.y;
       }
@@ -276,6 +286,7 @@ time_mix_chunk_kernel(MixParams p) {
   constexpr int kLanes = DT / 4, kPer = 32 / kLanes, kIter = C::kTok / (C::kWarps * kPer);
   const int er = warp * kPer + lane / kLanes, ec = lane % kLanes * 4;
 
+  float left = 1.f;                                          // (OUT = false) what the span leaves of column tid
   for (int t0 = 0; t0 < n; t0 += C::kTok) {
     const int cnt = min(C::kTok, n - t0);
     uint8_t* stage = smem + (t0 / C::kTok & 1) * C::kStage;
@@ -293,7 +304,7 @@ time_mix_chunk_kernel(MixParams p) {
       float tot[2] = {1.f, 1.f}, bonus[16];
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
-        r[i] = *reinterpret_cast<const __nv_bfloat162*>(sr + (row + i) * C::kLd + d0);
+        if constexpr (OUT) r[i] = *reinterpret_cast<const __nv_bfloat162*>(sr + (row + i) * C::kLd + d0);
         k[i] = *reinterpret_cast<const __nv_bfloat162*>(sk + (row + i) * C::kLd + d0);
         const float2 dv = *reinterpret_cast<const float2*>(so + (row + i) * C::kLdO + d0);
         const bool real = row + i < cnt;                     // (a token that is not there decays nothing)
@@ -301,20 +312,28 @@ time_mix_chunk_kernel(MixParams p) {
         w[i][1] = real ? expf(-__expf(dv.y + w0[1])) : 1.f;
         tot[0] *= w[i][0];
         tot[1] *= w[i][1];
-        bonus[i] = fmaf(__low2float(r[i]) * uu[0], __low2float(k[i]), __high2float(r[i]) * uu[1] * __high2float(k[i]));
+        if constexpr (OUT)
+          bonus[i] = fmaf(__low2float(r[i]) * uu[0], __low2float(k[i]), __high2float(r[i]) * uu[1] * __high2float(k[i]));
       }
-      const float b = transpose_sum<16>(bonus, lane);
-      if (lane < 16) sbonus[part * C::kTok + row + lane] = b;
-      steep = __syncthreads_or(tot[0] < kSteep || tot[1] < kSteep) != 0;
-      *reinterpret_cast<float2*>(stot + blk * DT + d0) = make_float2(tot[0], tot[1]);
-      float f[2] = {steep ? 1.f : 1.f / tot[0], steep ? 1.f : 1.f / tot[1]};
+      float f[2] = {1.f, 1.f};
+      steep = false;
+      if constexpr (OUT) {
+        const float b = transpose_sum<16>(bonus, lane);
+        if (lane < 16) sbonus[part * C::kTok + row + lane] = b;
+        steep = __syncthreads_or(tot[0] < kSteep || tot[1] < kSteep) != 0;
+        if (!steep) {
+          f[0] = 1.f / tot[0];
+          f[1] = 1.f / tot[1];
+        }
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const int at = (row + i) * C::kLd + d0;
-        split_bf16x2(__low2float(r[i]) * f[0], __high2float(r[i]) * f[1], reinterpret_cast<uint32_t*>(sr + at), reinterpret_cast<uint32_t*>(srl + at));
-        f[0] *= w[i][0];
-        f[1] *= w[i][1];
+        for (int i = 0; i < 16; ++i) {
+          const int at = (row + i) * C::kLd + d0;
+          split_bf16x2(__low2float(r[i]) * f[0], __high2float(r[i]) * f[1], reinterpret_cast<uint32_t*>(sr + at), reinterpret_cast<uint32_t*>(srl + at));
+          f[0] *= w[i][0];
+          f[1] *= w[i][1];
+        }
       }
+      *reinterpret_cast<float2*>(stot + blk * DT + d0) = make_float2(tot[0], tot[1]);
       f[0] = f[1] = 1.f;
 #pragma unroll
       for (int i = 15; i >= 0; --i) {
@@ -323,7 +342,7 @@ time_mix_chunk_kernel(MixParams p) {
         f[0] *= w[i][0];
         f[1] *= w[i][1];
       }
-      if (steep) {
+      if (OUT && steep) {
         // what token i takes of token j's value, two j at a time: the decays in between, one by one
         float* a = sa + (part * 4 + blk) * 256;
 #pragma unroll
@@ -346,9 +365,9 @@ time_mix_chunk_kernel(MixParams p) {
         }
       }
     }
-    if (C::kParts > 1) __syncthreads();
+    if (OUT && C::kParts > 1) __syncthreads();
     else __syncwarp();
-    if (!steep && warp < 4) {
+    if (OUT && !steep && warp < 4) {
       // the same from the prepared factors: rows i, columns j; this layout is also that of the operand it becomes
       float c[3][2][4] = {};
       const int row = warp * 16;
@@ -382,9 +401,11 @@ time_mix_chunk_kernel(MixParams p) {
         }
     }
     __syncthreads();
+    if (!OUT && tid < DT) left *= (stot[tid] * stot[DT + tid]) * (stot[2 * DT + tid] * stot[3 * DT + tid]);
     uint2 gate[kIter];                                       // requested before the products
 #pragma unroll
     for (int i = 0; i < kIter; ++i) {
+      if (!OUT) break;
       const int r = min(i * C::kWarps * kPer + er, cnt - 1);
       gate[i] = *reinterpret_cast<const uint2*>(proj + static_cast<long long>(t0 + r) * p.ld + 3 * p.section + min(ec, p.dp - 4));
     }
@@ -402,6 +423,7 @@ time_mix_chunk_kernel(MixParams p) {
       float acc[3][2][4] = {};
 #pragma unroll
       for (int ks = 0; ks < DT / 16; ++ks) {
+        if (!OUT) break;
         uint32_t hi[4], lo[4], qh[4], ql[4];
         split_bf16x2(S[2 * ks][0], S[2 * ks][1], &hi[0], &lo[0]);
         split_bf16x2(S[2 * ks][2], S[2 * ks][3], &hi[1], &lo[1]);
@@ -420,6 +442,7 @@ time_mix_chunk_kernel(MixParams p) {
       ldmat_x4_trans(vt, aV + frag_a_trans(lane, row, e0, C::kLd));
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
+        if (!OUT) break;
         uint32_t hi[2], lo[2];
         if (!steep) {
           const uint32_t* frag = reinterpret_cast<const uint32_t*>(sa) + b * 256 + c * 128 + lane;
@@ -460,6 +483,7 @@ time_mix_chunk_kernel(MixParams p) {
       }
     }
     __syncthreads();
+    if (!OUT) continue;
     // bonus, norm and gate
     float4 nm = make_float4(0.f, 0.f, 0.f, 0.f);
     if (ec < p.dp) nm = *reinterpret_cast<const float4*>(p.norm + h * p.dp + ec);
@@ -486,12 +510,15 @@ time_mix_chunk_kernel(MixParams p) {
     }
     __syncthreads();
   }
+  float* to = !OUT ? carry : last ? st : nullptr;
+  if (!to) return;
+  if (!OUT && tid < p.dp) p.span.left[(static_cast<long long>(blockIdx.y) * p.H + h) * p.dp + tid] = left;
 #pragma unroll
   for (int j = 0; j < DT / 8; ++j)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
-      if (r < p.dp && c < p.dp) *reinterpret_cast<float2*>(st + static_cast<long long>(r) * p.dp + c) = make_float2(S[j][2 * e], S[j][2 * e + 1]);
+      if (r < p.dp && c < p.dp) *reinterpret_cast<float2*>(to + static_cast<long long>(r) * p.dp + c) = make_float2(S[j][2 * e], S[j][2 * e + 1]);
     }
 }
 
@@ -573,17 +600,27 @@ int run_scan(const MixParams& p, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int DT>
-int run_chunk(const MixParams& p, cudaStream_t s) {
-  auto kern = time_mix_chunk_kernel<DT>;
+template <int DT, bool OUT>
+int launch_chunk(const MixParams& p, cudaStream_t s) {
+  auto kern = time_mix_chunk_kernel<DT, OUT>;
   static PerDeviceFlag attr;
   if (attr.unset()) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, MixChunk<DT>::kSmem);
     if (e != cudaSuccess) return static_cast<int>(e);
     attr.set();
   }
-  launch_pdl(kern, dim3(p.H, p.n_seq), dim3(MixChunk<DT>::kThreads), MixChunk<DT>::kSmem, s, pdl_all_enabled(), p);
+  launch_pdl(kern, dim3(p.H, p.span.seq ? p.span.n : p.n_seq), dim3(MixChunk<DT>::kThreads), MixChunk<DT>::kSmem, s, pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <int DT>
+int run_chunk(const MixParams& p, cudaStream_t s) {
+  if (p.span.seq) {
+    if (const int rc = launch_chunk<DT, false>(p, s)) return rc;
+    launch_pdl(state_carry_kernel, dim3((p.dp * p.dp / 4 + 255) / 256, p.H, p.n_seq), dim3(256), 0, s, pdl_all_enabled(), p.span,
+               static_cast<const float*>(p.state), p.slots, p.pos0, p.dp, p.dp, 1);
+  }
+  return launch_chunk<DT, true>(p, s);
 }
 
 template <typename T>
@@ -658,8 +695,10 @@ TSB_EXPORT int tsb_time_mix_step(const int* ints, void* const* q, float eps, flo
   return -2;
 }
 
-// ptrs: proj, dec, w0, u, norm, state, slots, cu, pos0, out, o ([rows, H, dp] fp32; null: bf16 on the tensor cores, dp <= 128).
-TSB_EXPORT int tsb_time_mix_prefill(const int* ints, void* const* q, float eps, float out_scale, int dtype, void* stream) {
+// ptrs: proj, dec, w0, u, norm, state, slots, cu, pos0, out, o ([rows, H, dp] fp32; null: bf16 on the tensor cores, dp <= 128), and for
+// `spans` spans of 512 tokens (0: every portion is walked in one): their sequences, the first span of every sequence, carry [spans, H,
+// dp, dp], left [spans, H, dp].
+TSB_EXPORT int tsb_time_mix_prefill(const int* ints, void* const* q, int spans, float eps, float out_scale, int dtype, void* stream) {
   using namespace tsb;
   MixParams p{};
   if (!read_mix(ints, &p)) return -2;
@@ -669,6 +708,10 @@ TSB_EXPORT int tsb_time_mix_prefill(const int* ints, void* const* q, float eps, 
   p.eps = eps; p.out_scale = out_scale;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (!p.o) {
+    if (spans > 0) {
+      p.span = {static_cast<const int*>(q[11]), static_cast<const int*>(q[12]), static_cast<float*>(q[13]), static_cast<float*>(q[14]), spans};
+      if (spans > 65535 || !p.span.seq || !p.span.first || !p.span.carry || !p.span.left) return -2;
+    }
     if (dtype != 1 || p.dp > 128 || p.ldo % 4 || (reinterpret_cast<uintptr_t>(p.out) & 7)) return -2;
     return p.dp <= 64 ? run_chunk<64>(p, s) : run_chunk<128>(p, s);
   }

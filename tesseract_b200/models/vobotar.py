@@ -26,7 +26,7 @@ def _window(m: dict) -> int:
 def _capped(m: dict) -> ShapedAttentionSpec:
     rot = Rotary(int(m["rot"]["dims"]), float(m["rot"]["base"]), neighbours=True)
     return ShapedAttentionSpec(*_sizes(m), norm="head", rotary=rot, softcap=float(m["softcap"]), sink="one", gate="element",
-                               v_mix=bool(m["v_mix"]))
+                               v_mix=bool(m.get("v_mix", False)))
 
 
 def _biased(m: dict) -> ShapedAttentionSpec:

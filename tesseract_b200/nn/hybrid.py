@@ -27,7 +27,7 @@ from ..ops.retention import SPAN, RetentionGeometry, log2_decays, retention
 from ..ops.rglru import CHUNK, RGLRUGeometry, RGLRUWeights, rglru
 from ..ops.rotary import Rotary
 from ..ops.ssd import CONV_TILE, SSDGeometry, SSDWeights, ssd
-from ..ops.timemix import STREAMS, TimeMixGeometry, TimeMixWeights, time_mix, token_shift
+from ..ops.timemix import SPAN as STATE_SPAN, STREAMS, TimeMixGeometry, TimeMixWeights, time_mix, token_shift
 from .ragged import LatentRun, PagedRun, PairRun, StateRun
 
 
@@ -621,6 +621,7 @@ class ShapedAttention(_RowPacked):
 class TimeMix(_RowPacked):
     """Linear attention with a decay per channel and token, fed by mixes of a token's input and the one before (see
     ``ops.timemix``)."""
+    tile = STATE_SPAN
 
     def __init__(self, width: int, heads: int, dim: int, rank: int, eps: float, dtype, device):
         super().__init__(dtype, device)
@@ -678,7 +679,7 @@ class TimeMix(_RowPacked):
 
 class SSD(_RowPacked):
     """State-space duality with a short convolution, normed in parts after its gate (see ``ops.ssd``)."""
-    tile = CONV_TILE
+    tiles = (CONV_TILE, STATE_SPAN)
 
     def __init__(self, width: int, heads: int, vdim: int, state: int, groups: int, conv: int, norm_parts: int, eps: float, dtype, device):
         super().__init__(dtype, device)

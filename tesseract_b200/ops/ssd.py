@@ -15,12 +15,13 @@ import torch
 
 from .. import _native
 from .._native import check, dtype_code, lib, stream_ptr
+from .timemix import spans_for
 
 P, I, L, F = _native.P, _native.I, _native.L, _native.F
 _native.register_signatures({
     "tsb_ssd_conv": [P, P, I, P],
     "tsb_ssd_step": [P, P, I, P],
-    "tsb_ssd_prefill": [P, P, I, P],
+    "tsb_ssd_prefill": [P, P, I, I, P],
     "tsb_part_norm": [P, L, P, L, P, I, I, I, I, I, F, F, I, P],
 })
 MAX_STATE = 256
@@ -159,10 +160,17 @@ def ssd(proj: torch.Tensor, geo: SSDGeometry, w: SSDWeights, conv_state: torch.T
                                          batch.state_slots.data_ptr(), batch.positions.data_ptr(), out.data_ptr())
             check(lib().tsb_ssd_step(ints, ptrs, dt, st), "tsb_ssd_step")
         if n:
-            ptrs = (ctypes.c_void_p * 9)(proj[nd:].data_ptr(), xbc[nd:].data_ptr(), gates[nd:].data_ptr(), w.d.data_ptr(), state.data_ptr(),
+            spans = spans_for(batch, H * batch.n_prompts * ((geo.vp + 63) // 64)) if proj.dtype == torch.bfloat16 else None
+            extra = (None,) * 4
+            if spans is not None:
+                carry = torch.empty((spans.n, H, geo.vp, geo.np), device=proj.device, dtype=torch.float32)
+                left = torch.empty((spans.n, H), device=proj.device, dtype=torch.float32)
+                extra = tuple(t.data_ptr() for t in (spans.seq, spans.first, carry, left))
+            ptrs = (ctypes.c_void_p * 13)(proj[nd:].data_ptr(), xbc[nd:].data_ptr(), gates[nd:].data_ptr(), w.d.data_ptr(), state.data_ptr(),
                                          batch.state_slots[nd:].data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(),
-                                         out[nd:].data_ptr())
-            check(lib().tsb_ssd_prefill(ints, ptrs, dt, st), "tsb_ssd_prefill")
+                                          out[nd:].data_ptr(), *extra)
+            check(lib().tsb_ssd_prefill(ints, ptrs, spans.n if spans is not None else 0, dt, st), "tsb_ssd_prefill")
+            _native.add_launches(2 if spans is not None else 0)
             _native.add_launches(2 if nd and geo.taps > 1 else 1 if nd or geo.taps > 1 else 0)
     return part_norm_(out, proj, w.norm, H, geo.vdim, geo.vp, geo.norm_parts, w.eps, out_scale)
 

@@ -21,11 +21,19 @@ P, I, L, F = _native.P, _native.I, _native.L, _native.F
 _native.register_signatures({
     "tsb_token_shift": [P, L, P, P, P, L, L, P, P, P, P, P, I, I, I, I, I, I, I, P],
     "tsb_time_mix_step": [P, P, F, F, I, P],
-    "tsb_time_mix_prefill": [P, P, F, F, I, P],
+    "tsb_time_mix_prefill": [P, P, I, F, F, I, P],
 })
 MAX_DIM = 256
 CHUNK_DIM = 128          # widest heads of the tensor-core kernel
 STREAMS = "rkvgw"
+SPAN = 512               # tokens of a portion that one CTA walks where there are few portions
+
+
+def spans_for(batch, ctas: int):
+    """The batch's portions cut into spans, where whole portions would keep at most ``ctas`` CTAs, less than one per SM, busy; else
+    None."""
+    tiles = batch.tiles(SPAN)
+    return tiles if ctas <= 148 and tiles.n > batch.n_prompts else None
 
 
 def _up(n: int, m: int) -> int:
@@ -144,11 +152,18 @@ def time_mix(proj: torch.Tensor, geo: TimeMixGeometry, w: TimeMixWeights, state:
         dec = project(torch.tanh(pr[:, 4 * geo.section:geo.cols].float()).to(proj.dtype), w.w2, out_dtype=torch.float32)
         chunked = proj.dtype == torch.bfloat16 and geo.dp <= CHUNK_DIM
         o = None if chunked else torch.empty((n, geo.heads, geo.dp), device=proj.device, dtype=torch.float32)
-        ptrs = (ctypes.c_void_p * 11)(pr.data_ptr(), dec.data_ptr(), w.w0.data_ptr(), w.u.data_ptr(), w.norm.data_ptr(), state.data_ptr(),
-                                      batch.state_slots[nd:].data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(), out[nd:].data_ptr(), _ptr(o))
-        check(lib().tsb_time_mix_prefill(geo.ints(n, batch.n_prompts, proj.stride(0), out.stride(0)), ptrs, float(w.eps),
-                                         float(out_scale), dt, st), "tsb_time_mix_prefill")
-        _native.add_launches(0 if chunked else 1)
+        spans = spans_for(batch, geo.heads * batch.n_prompts) if chunked else None
+        carry = left = None
+        if spans is not None:
+            carry = torch.empty((spans.n, geo.heads, geo.dp, geo.dp), device=proj.device, dtype=torch.float32)
+            left = torch.empty((spans.n, geo.heads, geo.dp), device=proj.device, dtype=torch.float32)
+        ptrs = (ctypes.c_void_p * 15)(pr.data_ptr(), dec.data_ptr(), w.w0.data_ptr(), w.u.data_ptr(), w.norm.data_ptr(), state.data_ptr(),
+                                      batch.state_slots[nd:].data_ptr(), batch.cu.data_ptr(), batch.pos0.data_ptr(), out[nd:].data_ptr(), _ptr(o),
+                                      *((_ptr(spans.seq), _ptr(spans.first)) if spans is not None else (None, None)), _ptr(carry), _ptr(left))
+        check(lib().tsb_time_mix_prefill(geo.ints(n, batch.n_prompts, proj.stride(0), out.stride(0)), ptrs,
+                                         spans.n if spans is not None else 0, float(w.eps), float(out_scale), dt, st),
+              "tsb_time_mix_prefill")
+        _native.add_launches(2 if spans is not None else 0 if chunked else 1)
     return out
 
 

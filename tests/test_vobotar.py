@@ -625,6 +625,48 @@ def test_ssd_keeps_a_far_token(kind):
                 assert abs(float(st[h, 3, 5]) - want) < 1e-4 * want, (hot, h, cuts)
 
 
+@pytest.mark.parametrize("kind", KINDS[1:])
+@pytest.mark.parametrize("mixer", ["mix", "mix128", "ssd", "ssd_wide"])
+def test_long_portions_are_walked_in_spans(kind, mixer):
+    """Portions longer than a span (and one just as long, one a token longer), from nothing and from what earlier ones left, beside
+    a short one of another sequence."""
+    dt, g = getattr(torch, kind[1]), torch.Generator().manual_seed(2)
+    T, short = 1085, 70
+    if mixer.startswith("mix"):
+        H, D = 2, 128 if mixer == "mix128" else 32
+        blk = TimeMix(32, H, D, 8, 1e-2, dt, kind[0])
+        proj, z, decay, d = mix_case(blk, T, kind, 5, 2.5)
+        o, S = oracle.bonus_recurrence(*(z[n].view(T, H, D) for n in "rkv"), decay, d["u"])
+        want = oracle.over_rms(o, 1e-2).reshape(T, H * D) * d["norm"] * oracle.silu(z["g"])
+    else:
+        H, E, N = (2, 24, 32) if mixer == "ssd" else (1, 136, 16)
+        blk = SSD(32, H, E, N, 1, 1, 1, 1e-2, dt, kind[0])
+        w = {n: torch.zeros(s) for n, s in blk.logical_shapes().items()}
+        w.update({"conv": torch.ones(H * E + 2 * N, 1), "norm": torch.ones(H * E), "D": torch.randn(H, generator=g),
+                  "dt_bias": torch.full((H,), -1.0), "A_log": torch.linspace(-5.0, -2.0, H)})
+        w = {n: t.to(torch.bfloat16) for n, t in w.items()}
+        blk.load(w)
+        d = {n: t.double() for n, t in w.items()}
+        val = torch.randn(T, 2 * H * E + 2 * N + H, generator=g)
+        proj, z = packed(blk, T, {"in": val}, kind), val.to(dt).double()
+        xbc = oracle.silu(z[:, H * E:-H])
+        B, C = (xbc[:, H * E + i * N:H * E + (i + 1) * N][:, None].expand(T, H, N) for i in (0, 1))
+        y, S = oracle.ssd_recurrence(xbc[:, :H * E].view(T, H, E), B, C, oracle.softplus(z[:, -H:] + d["dt_bias"]), d["A_log"], d["D"])
+        want = oracle.gated_group_norm(y.reshape(T, H * E), z[:, :H * E], d["norm"], 1, 1e-2)
+    cols, tol = blk._out_columns(), (3e-4 if dt == torch.float32 else 0.03) * float(want.abs().max())
+    for cuts in ([T], [512, 573], [513, 1, 571], [3, 1082]) if kind[0] == "cuda" else ([T],):
+        got, run, seq = run_core(blk, proj, cuts, kind)
+        err = (got[:, cols] - want).abs().max(1).values
+        assert float(err.max()) < tol, (cuts, int(err.argmax()))
+        state = run[1][seq.slot].cpu().double().transpose(1, 2)[:, :S.shape[1], :S.shape[2]]
+        assert (state - S).abs().max() < (1e-4 if dt == torch.float32 else 0.01) * float(S.abs().max()), cuts
+    cache = HybridCache([blk.run_spec()], 200, 8, 2, 1200, dt, kind[0])
+    b = RaggedBatch(cache, [(HybridSequence(cache), [0] * short), (HybridSequence(cache), [0] * T)], None, list(blk.masks), 0, list(blk.tiles))
+    rows = torch.cat([proj[:short], proj])
+    got = blk.core(rows, cache.runs[0], b).float().cpu().double()[:, cols]
+    assert (got[:short] - want[:short]).abs().max() < tol and (got[short:] - want).abs().max() < tol
+
+
 @pytest.mark.parametrize("kind", KINDS)
 @pytest.mark.parametrize("heads,vdim,vp,parts", [(4, 8, 8, 1), (4, 8, 8, 4), (6, 5, 8, 5), (2, 512, 512, 2), (64, 64, 64, 1), (3, 100, 104, 12)])
 def test_part_norm(kind, heads, vdim, vp, parts):
