@@ -100,6 +100,24 @@ token_shift_kernel(ShiftParams p) {
   }
 }
 
+// tanh of columns of a projection, 16 bytes a thread.
+template <typename T>
+__global__ void __launch_bounds__(256)
+tanh_rows_kernel(const T* x, long long ld, T* out, int cols, long long vecs) {
+  pdl_trigger();
+  pdl_grid_wait();
+  constexpr int V = kVec16<T>;
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i >= vecs) return;
+  const long long row = i / (cols / V);
+  const int c = static_cast<int>(i % (cols / V)) * V;
+  float f[V];
+  ld16<T>(x + row * ld + c, f);
+#pragma unroll
+  for (int k = 0; k < V; ++k) f[k] = tanhf(f[k]);
+  st16<T>(out + row * cols + c, f);
+}
+
 // ------------------------------------------------------------------ the recurrence
 struct MixParams {
   int H, dim, dp, rp, section, rows, n_seq, ld, ldo;
@@ -678,6 +696,21 @@ TSB_EXPORT int tsb_token_shift(const void* h, long long ldh, const float* mu, vo
   if (dtype == 1) return run_shift<__nv_bfloat16>(p, n_prompts, s);
   if (dtype == 0) return run_shift<float>(p, n_prompts, s);
   return -2;
+}
+
+// out [rows, cols] = tanh of x's first `cols` columns (row stride ld); cols and ld are multiples of 8.
+TSB_EXPORT int tsb_tanh_rows(const void* x, long long ld, void* out, int rows, int cols, int dtype, void* stream) {
+  using namespace tsb;
+  if (rows <= 0 || cols <= 0 || cols % 8 || ld % 8 || (dtype != 0 && dtype != 1) || (reinterpret_cast<uintptr_t>(x) & 15)) return -2;
+  const long long vecs = static_cast<long long>(rows) * cols / (dtype == 1 ? 8 : 4);
+  const dim3 grid(static_cast<unsigned>((vecs + 255) / 256));
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == 1)
+    launch_pdl(tanh_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl_all_enabled(), static_cast<const __nv_bfloat16*>(x), ld,
+               static_cast<__nv_bfloat16*>(out), cols, vecs);
+  else
+    launch_pdl(tanh_rows_kernel<float>, grid, dim3(256), 0, s, pdl_all_enabled(), static_cast<const float*>(x), ld, static_cast<float*>(out), cols, vecs);
+  return static_cast<int>(cudaGetLastError());
 }
 
 // ints: H, dim, dp, rp, section, rows, sequences, projection row stride, result row stride. ptrs: proj, w2, w0, u, norm, state,

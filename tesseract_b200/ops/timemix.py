@@ -20,6 +20,7 @@ from .gemm import input_columns, project
 P, I, L, F = _native.P, _native.I, _native.L, _native.F
 _native.register_signatures({
     "tsb_token_shift": [P, L, P, P, P, L, L, P, P, P, P, P, I, I, I, I, I, I, I, P],
+    "tsb_tanh_rows": [P, L, P, I, I, I, P],
     "tsb_time_mix_step": [P, P, F, F, I, P],
     "tsb_time_mix_prefill": [P, P, I, F, F, I, P],
 })
@@ -149,7 +150,9 @@ def time_mix(proj: torch.Tensor, geo: TimeMixGeometry, w: TimeMixWeights, state:
     n = T - nd
     if n:
         pr = proj[nd:]
-        dec = project(torch.tanh(pr[:, 4 * geo.section:geo.cols].float()).to(proj.dtype), w.w2, out_dtype=torch.float32)
+        low = torch.empty((n, geo.rp), device=proj.device, dtype=proj.dtype)
+        check(lib().tsb_tanh_rows(pr[:, 4 * geo.section:].data_ptr(), pr.stride(0), low.data_ptr(), n, geo.rp, dt, st), "tsb_tanh_rows")
+        dec = project(low, w.w2, out_dtype=torch.float32)
         chunked = proj.dtype == torch.bfloat16 and geo.dp <= CHUNK_DIM
         o = None if chunked else torch.empty((n, geo.heads, geo.dp), device=proj.device, dtype=torch.float32)
         spans = spans_for(batch, geo.heads * batch.n_prompts) if chunked else None
