@@ -109,6 +109,7 @@ def build_cuda(force: bool = False, verbose: bool = False, ptxas_info: bool = Fa
         return src.name, out
 
     if jobs:
+        lib.unlink(missing_ok=True)   # a build that fails must not leave a library older than its callers
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             for name, out in ex.map(compile_one, jobs):
                 if ptxas_info and out:

@@ -746,64 +746,70 @@ flash_bounded_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const int hi = min(Sk - 1, row_limit) - c0, lo = window > 0 ? row_limit - window + 1 - c0 : 0;      // visible columns
       const uint32_t s_addr = tmem_base + lane_addr + grp * BKV;
 #pragma unroll 1
-      for (int c = 0; c < BKV / 32; ++c) {
-        uint32_t r[32];
-        tmem_ld_32x32(s_addr + c * 32, r);
+      for (int half = 0; half < 2; ++half) {
+        uint32_t sr[64];
+        tmem_ld_32x32(s_addr + half * 64, *reinterpret_cast<uint32_t(*)[32]>(&sr[0]));
+        tmem_ld_32x32(s_addr + half * 64 + 32, *reinterpret_cast<uint32_t(*)[32]>(&sr[32]));
         tmem_ld_wait();
-        if (c == BKV / 32 - 1) {
+        if (half) {
           tc_fence_before();
-          mbar_arrive(&s_free[grp]);               // the last scores live in registers: the MMA warp may refill the buffer
+          mbar_arrive(&s_free[grp]);                 // the last scores live in registers: the MMA warp may refill the buffer
         }
-        float2 t[16];
-        const float2 mul = both(score.mul);
-        if constexpr (CAP) {
-          float top = 0.f;
 #pragma unroll
-          for (int i = 0; i < 32; ++i) top = fmaxf(top, fabsf(__uint_as_float(r[i])));
-          const float2 cap = both(score.cap), base = both(-m);
-          if (__any_sync(0xffffffffu, top > series_to)) {
+        for (int part = 0; part < 2; ++part) {
+          const int c = half * 2 + part;
+          const uint32_t* r = sr + part * 32;
+          float2 t[16];
+          const float2 mul = both(score.mul);
+          if constexpr (CAP) {
+            float top = 0.f;
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-              t[i].x = fmaf(score.cap, tanh_abs(__uint_as_float(r[2 * i]) * score.mul), -m);
-              t[i].y = fmaf(score.cap, tanh_abs(__uint_as_float(r[2 * i + 1]) * score.mul), -m);
+            for (int i = 0; i < 32; ++i) top = fmaxf(top, fabsf(__uint_as_float(r[i])));
+            const float2 cap = both(score.cap), base = both(-m);
+            if (__any_sync(0xffffffffu, top > series_to)) {
+#pragma unroll
+              for (int i = 0; i < 16; ++i) {
+                t[i].x = fmaf(score.cap, tanh_abs(__uint_as_float(r[2 * i]) * score.mul), -m);
+                t[i].y = fmaf(score.cap, tanh_abs(__uint_as_float(r[2 * i + 1]) * score.mul), -m);
+              }
+            } else {
+#pragma unroll
+              for (int i = 0; i < 16; ++i)
+                t[i] = fma_f32x2(cap, tanh_series(mul_f32x2(make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), mul)), base);
             }
           } else {
 #pragma unroll
             for (int i = 0; i < 16; ++i)
-              t[i] = fma_f32x2(cap, tanh_series(mul_f32x2(make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), mul)), base);
+              t[i] = fma_f32x2(make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), mul, both(-m));
           }
-        } else {
+          if (score.slope != 0.f) {
+            const float first = static_cast<float>(row_limit - c0 - c * 32);       // distance of the chunk's first column
 #pragma unroll
-          for (int i = 0; i < 16; ++i)
-            t[i] = fma_f32x2(make_float2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), mul, both(-m));
-        }
-        if (score.slope != 0.f) {
-          const float first = static_cast<float>(row_limit - c0 - c * 32);       // distance of the chunk's first column
+            for (int i = 0; i < 16; ++i)
+              t[i] = fma_f32x2(both(-score.slope), make_float2(first - 2 * i, first - 2 * i - 1), t[i]);
+          }
+          if (need_mask) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i)
-            t[i] = fma_f32x2(both(-score.slope), make_float2(first - 2 * i, first - 2 * i - 1), t[i]);
-        }
-        if (need_mask) {
+            for (int i = 0; i < 16; ++i) {
+              const int col = c * 32 + 2 * i;
+              if (col < lo || col > hi) t[i].x = -INFINITY;
+              if (col + 1 < lo || col + 1 > hi) t[i].y = -INFINITY;
+            }
+          }
+          uint32_t packed[16];
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
-            const int col = c * 32 + 2 * i;
-            if (col < lo || col > hi) t[i].x = -INFINITY;
-            if (col + 1 < lo || col + 1 > hi) t[i].y = -INFINITY;
+            const float2 e = make_float2(exp2_ftz(t[i].x), exp2_ftz(t[i].y));
+            l2.x += e.x;
+            l2.y += e.y;
+            packed[i] = pack_bf16x2(e.x, e.y);
           }
-        }
-        uint32_t packed[16];
+          uint8_t* prow = sP + grp * Cfg::kPBytes + (c >> 1) * 16384 + row * 128;
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const float2 e = make_float2(exp2_ftz(t[i].x), exp2_ftz(t[i].y));
-          l2.x += e.x;
-          l2.y += e.y;
-          packed[i] = pack_bf16x2(e.x, e.y);
+          for (int q4 = 0; q4 < 4; ++q4)
+            *reinterpret_cast<uint4*>(prow + ((((c & 1) * 4 + q4) ^ (row & 7)) << 4)) =
+                make_uint4(packed[q4 * 4], packed[q4 * 4 + 1], packed[q4 * 4 + 2], packed[q4 * 4 + 3]);
         }
-        uint8_t* prow = sP + grp * Cfg::kPBytes + (c >> 1) * 16384 + row * 128;
-#pragma unroll
-        for (int q4 = 0; q4 < 4; ++q4)
-          *reinterpret_cast<uint4*>(prow + ((((c & 1) * 4 + q4) ^ (row & 7)) << 4)) =
-              make_uint4(packed[q4 * 4], packed[q4 * 4 + 1], packed[q4 * 4 + 2], packed[q4 * 4 + 3]);
       }
       fence_proxy_async_smem();
       mbar_arrive(&p_full[grp]);
