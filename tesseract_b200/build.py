@@ -36,6 +36,7 @@ _HYBRID = ("runtime", "gemm_tcgen05", "gemm_decode_wq", "gemm_decode_mx", "flash
 GROUPS = {
     "fozelix": _HYBRID + ("decode_attn", "decode_attn_mma", "ragged_attn", "delta_rule"),
     "vobotar": _HYBRID + ("attn_prepare", "decode_attn", "decode_attn_mma", "post_norm", "ragged_attn", "ssd", "time_mix"),
+    "tonilix": _HYBRID + ("attn_prepare", "decode_attn", "decode_attn_mma", "delta_rule", "expert_mlp", "pre_norm", "ragged_attn", "time_mix"),
     "polosun": _HYBRID + ("depth_residual", "latent_attn", "retention", "rglru"),
 }
 

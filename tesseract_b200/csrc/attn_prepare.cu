@@ -1,5 +1,5 @@
 // What happens to a packed projection row [q: H heads | k: Hkv | v: Hkv | ..] before attention: biases, a norm of q and k (per
-// head, or over all heads at once), rotation by position, values mixed with those of an earlier layer; q goes to a buffer of its
+// head, or over all heads at once), rotation by position, queries that grow louder with it, values mixed with those of an earlier layer; q goes to a buffer of its
 // own, k and v to the token's pool slot and, for prompt rows, to the key axis of the tensor-core kernel.
 //
 // One CTA per row. LPH lanes share a head (16 bytes each, PPL times), so a warp takes 32 / LPH heads at once. Everything between
@@ -12,6 +12,7 @@ namespace {
 struct PrepareParams {
   int rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, ld, D_first;    // norm: 0 none, 1 unit heads, 2 heads with a weight, 3 whole
   float eps, vmix;
+  float q_coef, q_every;      // q *= 1 + q_coef ln(floor((position + 1) / q_every) + 1); q_coef = 0: not
   const void* proj;
   const float* bias;          // [off_v + Hkv * D] or null
   const float* q_norm;
@@ -93,6 +94,7 @@ attn_prepare_kernel(PrepareParams p) {
   const long long page = slot >= 0 ? static_cast<long long>(slot / p.bs) * p.Hkv * p.bs + slot % p.bs : 0;
   const int stage_row = p.stage && row >= p.n_decode ? p.stage_rows[row - p.n_decode] : -1;
   const float2* turn = p.table && p.hp > 0 ? p.table + static_cast<long long>(max(p.positions[row], 0)) * p.hp : nullptr;
+  const float loud = p.q_coef != 0.f ? 1.f + p.q_coef * logf(floorf(static_cast<float>(max(p.positions[row], 0) + 1) / p.q_every) + 1.f) : 1.f;
   constexpr int U = PPL == 1 ? 2 : 1;               // heads whose loads are requested together
   for (int u0 = 0; u0 < units; u0 += U * step) {    // (every lane takes every turn: the sums below are shuffles)
     float f[U][PPL][V], ss[U];
@@ -159,6 +161,8 @@ attn_prepare_kernel(PrepareParams p) {
           }
         }
         if (kind[q] == 0) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) x8[i] *= loud;
           st16<T>(static_cast<T*>(p.q) + (static_cast<long long>(row) * p.H + head[q]) * D + d, x8);
           continue;
         }
@@ -189,17 +193,17 @@ int launch_prepare(const PrepareParams& p, cudaStream_t s) {
 }  // namespace
 }  // namespace tsb
 
-// ints: rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, row stride, head size of v_first; floats: eps, vmix; ptrs: proj, bias, q_norm, k_norm,
+// ints: rows, H, Hkv, D, dim, hp, off_k, off_v, norm, bs, n_decode, row stride, head size of v_first; floats: eps, vmix, q_coef, q_every; ptrs: proj, bias, q_norm, k_norm,
 // table, positions, slots, q, k_pool, v_pool, v_first, stage, stage_rows (see PrepareParams). dtype: 0 = fp32, 1 = bf16. D is a
 // multiple of 32, up to 256; rows and sections start on 16 bytes.
 TSB_EXPORT int tsb_attn_prepare(const int* v, const float* f, void* const* q, int dtype, void* stream) {
   using namespace tsb;
-  PrepareParams p{v[0], v[1], v[2], v[3], v[4], v[5], v[6], v[7], v[8], v[9], v[10], v[11], v[12], f[0], f[1], q[0], static_cast<const float*>(q[1]),
+  PrepareParams p{v[0], v[1], v[2], v[3], v[4], v[5], v[6], v[7], v[8], v[9], v[10], v[11], v[12], f[0], f[1], f[2], f[3], q[0], static_cast<const float*>(q[1]),
                   static_cast<const float*>(q[2]), static_cast<const float*>(q[3]), static_cast<const float2*>(q[4]),
                   static_cast<const int*>(q[5]), static_cast<const int*>(q[6]), q[7], q[8], q[9], q[10], q[11], static_cast<const int*>(q[12])};
   if (p.rows <= 0 || p.H <= 0 || p.Hkv <= 0 || p.D <= 0 || p.D % 32 || p.D > 256 || p.dim <= 0 || p.dim > p.D || p.hp % 8 || 2 * p.hp > p.D ||
       p.off_k % 8 || p.off_v % 8 || p.ld % 8 || p.norm < 0 || p.norm > 3 || (p.norm >= 2 && (!p.q_norm || !p.k_norm)) || p.bs <= 0 ||
-      (p.stage && !p.stage_rows) || (p.v_first && (p.D_first <= 0 || p.D_first % 8)) || (reinterpret_cast<uintptr_t>(p.proj) & 15))
+      (p.q_coef != 0.f && !(p.q_every > 0.f)) || (p.stage && !p.stage_rows) || (p.v_first && (p.D_first <= 0 || p.D_first % 8)) || (reinterpret_cast<uintptr_t>(p.proj) & 15))
     return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (dtype == 1) return launch_prepare<__nv_bfloat16>(p, s);

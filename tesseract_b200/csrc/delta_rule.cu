@@ -3,8 +3,9 @@
 // Per value head, with a state S [dim, vdim] in fp32:
 //   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 // q, k, v are short causal convolutions (per channel, then SiLU) of a packed projection; q and k are unit vectors per
-// key head (q also times dim^-1/2); g = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b); the read-out is
-// divided by its root mean square over vdim, scaled by a weight and by SiLU of a gate projection.
+// key head (q also times dim^-1/2); g = exp(-exp(A_log) softplus(a + dt_bias)), one per head or, where the caller brings
+// `dec`, one per head and row of S (key channel); beta = sigmoid(b); the read-out is divided by its root mean square over
+// vdim, scaled by a weight and by SiLU or sigmoid of a gate.
 //
 // Prompt rows take four launches: `delta_prepare_kernel` (convolution, unit vectors, gates; every token in parallel),
 // `conv_state_kernel` (the convolution's tail of each sequence goes to its slot), `delta_scan_kernel` (the
@@ -16,11 +17,13 @@
 // state with their k and q are formed from the state before the block, the tokens' influence on one another is a 4 x 4
 // triangle of scalars that the prepare kernel has computed, and the state is updated once. That is 3.25 multiply-adds
 // per element and token instead of 4, and one reduction latency per four tokens; they are issued on register pairs
-// (fma.rn.f32x2). The one-token kernel uses the same identity: S_new^T q = g (S_old^T q) + (k . q) u, so the state is
+// (fma.rn.f32x2). With a decay per channel the products of the decays inside a block are folded into the k and q that meet
+// the old state and into the k that the update writes, so that the same scan runs on three vectors per token and value head
+// instead of two per token and key head. The one-token kernel uses the same identity: S_new^T q = g (S_old^T q) + (k . q) u, so the state is
 // read once. Everything of the recurrence is fp32; nothing here uses the tensor cores.
 //
 // Packed projection row (element offsets, sections padded to multiples of 8):
-//   [ q: Hk * dim | k: Hk * dim | v: H * vdim | gate: H * vdim | b: H | a: H ]
+//   [ q: Hk * dim | k: Hk * dim | v: H * vdim | .. b: H .. | .. a: H (without dec) .. ]
 // A slot's convolution state holds the last taps - 1 rows of the first three sections, in the projection's type.
 #include "ragged_conv.cuh"
 
@@ -34,9 +37,19 @@ namespace {
 struct DeltaGeom {
   int Hk, H, dim, vdim;      // key heads, value heads, row and column extent of a head's state
   int dkp, vp;               // padded extents of the fp32 operands: dkp in {32, 64, 128, 256}, vp = vdim rounded up to 4
-  int off_k, off_v, off_g, off_b, off_a;   // section offsets in a projection row (q starts at 0)
+  int off_k, off_v, off_b, off_a;   // section offsets in a projection row (q starts at 0)
   int conv_c;                // columns of the convolved sections (q | k | v with their padding)
   long long ldp;             // projection row stride
+};
+
+// What the projection row does not hold: gates [rows, ld_gate] (kind 0: SiLU, 1: sigmoid), inputs of the decays [rows, ld_dec] (fp32,
+// H * dim; null: one decay per head, from the row).
+struct DeltaSide {
+  const void* gate;
+  long long ld_gate;
+  int gate_kind;
+  const float* dec;
+  long long ld_dec;
 };
 
 constexpr int kBlk = 4;          // tokens the recurrence takes at once
@@ -49,6 +62,26 @@ __device__ __forceinline__ float silu_f(float x) {
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+template <bool FAST = false>
+__device__ __forceinline__ float gate_f(float x, int kind) {
+  if (kind == 0) return silu_f<FAST>(x);
+  return FAST ? __fdividef(1.f, 1.f + __expf(-x)) : sigmoid_f(x);
+}
+
+// Sums of 16 values over the warp: lane l returns the sum of v[l % 16].
+__device__ __forceinline__ float sums_of_16(float (&v)[16], int lane) {
+#pragma unroll
+  for (int o = 8; o; o >>= 1) {
+    const bool up = (lane & o) != 0;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (i >= o) break;
+      const float keep = up ? v[i + o] : v[i], give = up ? v[i] : v[i + o];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+    }
+  }
+  return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 16);
+}
 
 // N consecutive channels starting at p, of which `valid` exist; vector loads when the caller knows p to be aligned.
 template <typename T, int N>
@@ -97,14 +130,17 @@ struct DeltaPrepParams {
   const void* proj;          // [rows, ldp]
   const float* conv_w;       // [taps, conv_c]
   const float* a_log;        // [H]
-  const float* dt_bias;      // [H]
+  const float* dt_bias;      // [H] or, with dec, [H * dim]
+  const float* dec;          // [rows, ld_dec] or null
+  long long ld_dec;
   const void* conv_state;    // [slots, taps - 1, conv_c]
   const int* cu;             // [nseq + 1] row offsets of the sequences
   const int* slots;          // [nseq]
   const int* pos0;           // [nseq] position of the first row (0: the sequence starts here)
   const int* blk_seq;        // [blocks] sequence of a block of kBlk tokens
   const int* blk0;           // [nseq + 1] first block of a sequence
-  float* kq;                 // [rows, Hk, 2, dkp]: k, then q
+  float* kq;                 // [rows, Hk, 2, dkp]: k, then q; with dec [rows, H, 3, dkp], see delta_prepare_kernel
+  float* g4;                 // with dec: [blocks, H, dkp] the decays of a whole block
   float* v;                  // [rows, H, vp]
   float* coef;               // [blocks, H, kCoef]
   int blocks;
@@ -164,7 +200,11 @@ __device__ __forceinline__ void conv_block(const DeltaPrepParams& p, int row0, i
 //   G_j = g_0 .. g_j,  c_j = g_{j+1} .. g_3,  A_ji = (g_{i+1} .. g_j)(k_i . k_j),  W_ji = (g_{i+1} .. g_j)(k_i . q_j).
 // Coefficients as stored: G (4), beta (4), A (10, 20, 21, 30, 31, 32, 0, 0), c (4), W (4 rows of 4, zero above the
 // diagonal). Tokens past the end of the portion get g = 1, beta = 0, k = q = 0: they change nothing.
-template <typename T, int TAPS, int EPL>
+//
+// CH (a decay per channel): G_j, c_j and the factors in A and W are vectors over the channels. A and W sum them in; G_j goes into
+// the k and q that meet the old state, c_j into the k of the update (kq: k_j G_j, q_j G_j, k_j c_j per value head; the
+// coefficients G and c are 1), and G_3 is kept as it is. All are products of factors up to 1, never quotients.
+template <typename T, int TAPS, int EPL, bool CH>
 __global__ void __launch_bounds__(128, TAPS <= 4 && EPL <= 4 ? 5 : 1)
 delta_prepare_kernel(DeltaPrepParams p) {
   pdl_trigger();
@@ -188,6 +228,8 @@ delta_prepare_kernel(DeltaPrepParams p) {
     conv_block<T, TAPS, EPL>(p, row0, first, cnt, state_row, has_state, unit * g.dim + d0, valid, vec, qv);
     conv_block<T, TAPS, EPL>(p, row0, first, cnt, state_row, has_state, g.off_k + unit * g.dim + d0, valid, vec, kv);
     const float rsqrt_dim = rsqrtf(static_cast<float>(g.dim));
+    const int per = g.H / g.Hk;
+    const T* proj = static_cast<const T*>(p.proj);
     float* out = p.kq + (static_cast<long long>(row0 + first) * g.Hk + unit) * 2 * g.dkp + d0;
 #pragma unroll
     for (int t = 0; t < kBlk; ++t) {
@@ -204,59 +246,125 @@ delta_prepare_kernel(DeltaPrepParams p) {
         qv[t][i] *= rq;
         kv[t][i] *= rk;
       }
-      if (t < cnt) {
+      if (!CH && t < cnt) {
         float* o = out + static_cast<long long>(t) * g.Hk * 2 * g.dkp;
         store_f32<EPL>(o, EPL, true, kv[t]);
         store_f32<EPL>(o + g.dkp, EPL, true, qv[t]);
       }
     }
-    float kk[kBlk][kBlk], kqd[kBlk][kBlk];          // [j][i]: k_i . k_j (i < j) and k_i . q_j (i <= j)
+    if constexpr (CH) {
+      for (int hh = 0; hh < per; ++hh) {
+        const int h = unit * per + hh;
+        float gd[kBlk][EPL], bias[EPL];
+        load_ch<float, EPL>(p.dt_bias + h * g.dim + d0, valid, false, bias);
+        const float rate = expf(p.a_log[h]);
 #pragma unroll
-    for (int j = 0; j < kBlk; ++j)
+        for (int t = 0; t < kBlk; ++t)             // (rows past the end repeat the last one until they are replaced)
+          load_ch<float, EPL>(p.dec + static_cast<long long>(row0 + first + min(t, cnt - 1)) * p.ld_dec + h * g.dim + d0, valid, vec, gd[t]);
 #pragma unroll
-      for (int i = 0; i < kBlk; ++i) {
-        kk[j][i] = kqd[j][i] = 0.f;
-        if (i <= j) {
-          float a = 0.f, b = 0.f;
+        for (int t = 0; t < kBlk; ++t)
+#pragma unroll
+          for (int e = 0; e < EPL; ++e) gd[t][e] = t < cnt && e < valid ? expf(-rate * softplus_f(gd[t][e] + bias[e])) : 1.f;
+        float s[16];                               // A 10, 20, 21, 30, 31, 32, then W 00, 10, 11, 20, .. 33
+#pragma unroll
+        for (int i = 0; i < 16; ++i) s[i] = 0.f;
+#pragma unroll
+        for (int i = 0; i < kBlk; ++i) {           // k_i, decayed further and further
+          float kd[EPL];
+#pragma unroll
+          for (int e = 0; e < EPL; ++e) kd[e] = kv[i][e];
+#pragma unroll
+          for (int j = i; j < kBlk; ++j) {
+#pragma unroll
+            for (int e = 0; e < EPL; ++e) {
+              if (j > i) {
+                kd[e] *= gd[j][e];
+                s[j * (j - 1) / 2 + i] = fmaf(kd[e], kv[j][e], s[j * (j - 1) / 2 + i]);
+              }
+              s[6 + j * (j + 1) / 2 + i] = fmaf(kd[e], qv[j][e], s[6 + j * (j + 1) / 2 + i]);
+            }
+          }
+          if (i < cnt) store_f32<EPL>(p.kq + ((static_cast<long long>(row0 + first + i) * g.H + h) * 3 + 2) * g.dkp + d0, EPL, true, kd);
+        }
+        float G[EPL];
+#pragma unroll
+        for (int e = 0; e < EPL; ++e) G[e] = 1.f;
+#pragma unroll
+        for (int t = 0; t < kBlk; ++t) {
+          float a[EPL], b[EPL];
 #pragma unroll
           for (int e = 0; e < EPL; ++e) {
-            a = fmaf(kv[i][e], kv[j][e], a);
-            b = fmaf(kv[i][e], qv[j][e], b);
+            G[e] *= gd[t][e];
+            a[e] = kv[t][e] * G[e];
+            b[e] = qv[t][e] * G[e];
           }
-          if (i < j) kk[j][i] = warp_sum(a);
-          kqd[j][i] = warp_sum(b);
+          if (t < cnt) {
+            float* o = p.kq + (static_cast<long long>(row0 + first + t) * g.H + h) * 3 * g.dkp + d0;
+            store_f32<EPL>(o, EPL, true, a);
+            store_f32<EPL>(o + g.dkp, EPL, true, b);
+          }
         }
+        store_f32<EPL>(p.g4 + (static_cast<long long>(blk) * g.H + h) * g.dkp + d0, EPL, true, G);
+        const float sum = sums_of_16(s, lane);
+        // coefficients `lane` and, of the last row of W, 32 + lane
+        const int wr = (lane - 20) >> 2, wi = (lane - 20) & 3;
+        const int src = lane >= 20 ? 6 + wr * (wr + 1) / 2 + wi : lane - 8;
+        const float mine = __shfl_sync(0xffffffffu, sum, src & 15), tail = __shfl_sync(0xffffffffu, sum, (12 + lane) & 15);
+        float c = 0.f;
+        if (lane < 4 || (lane >= 16 && lane < 20)) c = 1.f;
+        else if (lane < 8) c = lane - 4 < cnt ? sigmoid_f(to_f32<T>(proj[static_cast<long long>(row0 + first + lane - 4) * g.ldp + g.off_b + h])) : 0.f;
+        else if (lane < 14 || (lane >= 20 && wi <= wr)) c = mine;
+        float* co = p.coef + (static_cast<long long>(blk) * g.H + h) * kCoef;
+        co[lane] = c;
+        if (lane < 4) co[32 + lane] = tail;
       }
-    const int per = g.H / g.Hk;
-    const T* proj = static_cast<const T*>(p.proj);
-    // eight heads at a time: lane = token * 8 + head works out one pair of gates, then lanes 0 .. 7 collect their head's
-    for (int h0 = 0; h0 < per; h0 += 8) {
-      const int hh = h0 + (lane & 7), tok = lane >> 3;
-      const int h = unit * per + min(hh, per - 1);
-      float gate = 1.f, beta = 0.f;
-      if (tok < cnt) {
-        const T* pr = proj + static_cast<long long>(row0 + first + tok) * g.ldp;
-        gate = expf(-expf(p.a_log[h]) * softplus_f(to_f32<T>(pr[g.off_a + h]) + p.dt_bias[h]));
-        beta = sigmoid_f(to_f32<T>(pr[g.off_b + h]));
-      }
-      float gd[kBlk], be[kBlk];
+    } else {
+      float kk[kBlk][kBlk], kqd[kBlk][kBlk];          // [j][i]: k_i . k_j (i < j) and k_i . q_j (i <= j)
 #pragma unroll
-      for (int t = 0; t < kBlk; ++t) {
-        gd[t] = __shfl_sync(0xffffffffu, gate, t * 8 + (lane & 7));
-        be[t] = __shfl_sync(0xffffffffu, beta, t * 8 + (lane & 7));
+      for (int j = 0; j < kBlk; ++j)
+#pragma unroll
+        for (int i = 0; i < kBlk; ++i) {
+          kk[j][i] = kqd[j][i] = 0.f;
+          if (i <= j) {
+            float a = 0.f, b = 0.f;
+#pragma unroll
+            for (int e = 0; e < EPL; ++e) {
+              a = fmaf(kv[i][e], kv[j][e], a);
+              b = fmaf(kv[i][e], qv[j][e], b);
+            }
+            if (i < j) kk[j][i] = warp_sum(a);
+            kqd[j][i] = warp_sum(b);
+          }
+        }
+      // eight heads at a time: lane = token * 8 + head works out one pair of gates, then lanes 0 .. 7 collect their head's
+      for (int h0 = 0; h0 < per; h0 += 8) {
+        const int hh = h0 + (lane & 7), tok = lane >> 3;
+        const int h = unit * per + min(hh, per - 1);
+        float gate = 1.f, beta = 0.f;
+        if (tok < cnt) {
+          const T* pr = proj + static_cast<long long>(row0 + first + tok) * g.ldp;
+          gate = expf(-expf(p.a_log[h]) * softplus_f(to_f32<T>(pr[g.off_a + h]) + p.dt_bias[h]));
+          beta = sigmoid_f(to_f32<T>(pr[g.off_b + h]));
+        }
+        float gd[kBlk], be[kBlk];
+#pragma unroll
+        for (int t = 0; t < kBlk; ++t) {
+          gd[t] = __shfl_sync(0xffffffffu, gate, t * 8 + (lane & 7));
+          be[t] = __shfl_sync(0xffffffffu, beta, t * 8 + (lane & 7));
+        }
+        if (lane >= 8 || hh >= per) continue;
+        float4* o = reinterpret_cast<float4*>(p.coef + (static_cast<long long>(blk) * g.H + h) * kCoef);
+        const float g10 = gd[1], g21 = gd[2], g32 = gd[3], g20 = g10 * g21, g31 = g21 * g32, g30 = g20 * g32;
+        o[0] = make_float4(gd[0], gd[0] * g10, gd[0] * g20, gd[0] * g30);
+        o[1] = make_float4(be[0], be[1], be[2], be[3]);
+        o[2] = make_float4(g10 * kk[1][0], g20 * kk[2][0], g21 * kk[2][1], g30 * kk[3][0]);
+        o[3] = make_float4(g31 * kk[3][1], g32 * kk[3][2], 0.f, 0.f);
+        o[4] = make_float4(g30, g31, g32, 1.f);
+        o[5] = make_float4(kqd[0][0], 0.f, 0.f, 0.f);
+        o[6] = make_float4(g10 * kqd[1][0], kqd[1][1], 0.f, 0.f);
+        o[7] = make_float4(g20 * kqd[2][0], g21 * kqd[2][1], kqd[2][2], 0.f);
+        o[8] = make_float4(g30 * kqd[3][0], g31 * kqd[3][1], g32 * kqd[3][2], kqd[3][3]);
       }
-      if (lane >= 8 || hh >= per) continue;
-      float4* o = reinterpret_cast<float4*>(p.coef + (static_cast<long long>(blk) * g.H + h) * kCoef);
-      const float g10 = gd[1], g21 = gd[2], g32 = gd[3], g20 = g10 * g21, g31 = g21 * g32, g30 = g20 * g32;
-      o[0] = make_float4(gd[0], gd[0] * g10, gd[0] * g20, gd[0] * g30);
-      o[1] = make_float4(be[0], be[1], be[2], be[3]);
-      o[2] = make_float4(g10 * kk[1][0], g20 * kk[2][0], g21 * kk[2][1], g30 * kk[3][0]);
-      o[3] = make_float4(g31 * kk[3][1], g32 * kk[3][2], 0.f, 0.f);
-      o[4] = make_float4(g30, g31, g32, 1.f);
-      o[5] = make_float4(kqd[0][0], 0.f, 0.f, 0.f);
-      o[6] = make_float4(g10 * kqd[1][0], kqd[1][1], 0.f, 0.f);
-      o[7] = make_float4(g20 * kqd[2][0], g21 * kqd[2][1], kqd[2][2], 0.f);
-      o[8] = make_float4(g30 * kqd[3][0], g31 * kqd[3][1], g32 * kqd[3][2], kqd[3][3]);
     }
   } else {
     const int c = (unit - g.Hk) * 256 + lane * 8, total = g.H * g.vdim;
@@ -301,7 +409,8 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src, int bytes) {
 
 struct DeltaScanParams {
   DeltaGeom g;
-  const float* kq;           // [rows, Hk, 2, dkp]
+  const float* kq;           // [rows, Hk, 2, dkp] or [rows, H, 3, dkp]
+  const float* g4;           // [blocks, H, dkp] or null
   const float* v;            // [rows, H, vp]
   const float* coef;         // [blocks, H, kCoef]
   float* state;              // [slots, H, dim, vp]
@@ -315,13 +424,15 @@ struct DeltaScanParams {
 constexpr int kScanWarps = 4;
 constexpr int kScanTile = 16;    // tokens per shared-memory stage
 
-template <int KT, int CT>
+template <int KT, int CT, bool CH>
 struct ScanCfg {
   static constexpr int DK = 8 * KT;
+  static constexpr int kVecs = CH ? 3 : 2;                            // vectors per token
   static constexpr int kCols = kScanWarps * 4 * CT;                   // value columns per CTA
-  static constexpr int kV = kScanTile * 2 * DK;                       // float offsets within a stage
+  static constexpr int kV = kScanTile * kVecs * DK;                   // float offsets within a stage
   static constexpr int kC = kV + kScanTile * kCols;
-  static constexpr int kStageFloats = kC + kScanTile / kBlk * kCoef;
+  static constexpr int kG = kC + kScanTile / kBlk * kCoef;
+  static constexpr int kStageFloats = kG + (CH ? kScanTile / kBlk * DK : 0);
   static constexpr int kSmemBytes = 2 * kStageFloats * 4;
 };
 
@@ -330,12 +441,12 @@ struct ScanCfg {
 // 4 + j with e_j of its columns; every lane then solves for u itself, and lanes 4 .. 7 write the read-outs. A float of k or
 // q loaded from shared memory feeds CT columns: with CT = 2 the kernel is bound by those loads, with CT = 4 by the
 // multiply-adds; small batches take fewer columns per lane and more warps.
-template <int KT, int CT>
+template <int KT, int CT, bool CH>
 __global__ void __launch_bounds__(kScanWarps * 32, 2)
 delta_scan_kernel(DeltaScanParams p) {
   pdl_grid_wait();
-  using Cfg = ScanCfg<KT, CT>;
-  constexpr int DK = Cfg::DK, kScanCols = Cfg::kCols;
+  using Cfg = ScanCfg<KT, CT, CH>;
+  constexpr int DK = Cfg::DK, kScanCols = Cfg::kCols, kVecs = Cfg::kVecs;
   extern __shared__ __align__(16) float sm[];
   const DeltaGeom& g = p.g;
   const int seq = blockIdx.z, head = blockIdx.y;
@@ -343,7 +454,7 @@ delta_scan_kernel(DeltaScanParams p) {
   const int slot = p.slots[seq];
   if (n <= 0 || slot < 0) return;
   const int blk0 = p.blk0[seq], n_blk = (n + kBlk - 1) / kBlk;
-  const int hk = head / (g.H / g.Hk);
+  const int hk = CH ? head : head / (g.H / g.Hk), n_hk = CH ? g.H : g.Hk;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int kl = lane & 7, cg = lane >> 3;
   const int slice0 = blockIdx.x * kScanCols;
@@ -369,12 +480,19 @@ delta_scan_kernel(DeltaScanParams p) {
     const int t0 = tile * kScanTile;
     const int cnt = min(kScanTile, n - t0);
     const int full = (cnt + kBlk - 1) / kBlk * kBlk;     // tokens past the end of the last block are zeros
-    constexpr int kRowVec = 2 * DK / 4;
+    constexpr int kRowVec = kVecs * DK / 4;
     for (int i = threadIdx.x; i < full * kRowVec; i += kScanWarps * 32) {
       const int t = i / kRowVec, w = i % kRowVec;
       const int ts = min(t, cnt - 1);
-      cp16(smem_u32(base + t * 2 * DK + w * 4), p.kq + (static_cast<long long>(row0 + t0 + ts) * g.Hk + hk) * 2 * DK + w * 4,
+      cp16(smem_u32(base + t * kVecs * DK + w * 4), p.kq + (static_cast<long long>(row0 + t0 + ts) * n_hk + hk) * kVecs * DK + w * 4,
            t < cnt ? 16 : 0);
+    }
+    if constexpr (CH) {
+      for (int i = threadIdx.x; i < full / kBlk * (DK / 4); i += kScanWarps * 32) {
+        const int bi = i / (DK / 4), w = i % (DK / 4);
+        cp16(smem_u32(base + Cfg::kG + bi * DK + w * 4),
+             p.g4 + (static_cast<long long>(blk0 + tile * (kScanTile / kBlk) + bi) * g.H + head) * DK + w * 4, 16);
+      }
     }
     constexpr int kColVec = kScanCols / 4;
     for (int i = threadIdx.x; i < full * kColVec; i += kScanWarps * 32) {
@@ -404,13 +522,14 @@ delta_scan_kernel(DeltaScanParams p) {
     const float* base = sm + (tile & 1) * Cfg::kStageFloats;
     const int nb = min(kScanTile / kBlk, n_blk - tile * (kScanTile / kBlk));
     for (int bi = 0; bi < nb; ++bi) {
-      const float* kqb = base + bi * kBlk * 2 * DK;
+      const float* kqb = base + bi * kBlk * kVecs * DK;
       const float4* cf = reinterpret_cast<const float4*>(base + Cfg::kC + bi * kCoef);
-      float2 k2[kBlk][KT / 2];
+      float2 k2[CH ? 1 : kBlk][KT / 2];            // (kept for the update, which has vectors of its own with CH)
       float a[2 * kBlk][CT];                       // d_0 .. d_3, e_0 .. e_3 per column
 #pragma unroll
       for (int j = 0; j < kBlk; ++j) {
-        const float4* kr = reinterpret_cast<const float4*>(kqb + j * 2 * DK);
+        const float4* kr = reinterpret_cast<const float4*>(kqb + j * kVecs * DK);
+        float2(&kj)[KT / 2] = k2[CH ? 0 : j];
         const float4* qr = kr + DK / 4;
         float2 dk[CT], dq[CT];
 #pragma unroll
@@ -418,14 +537,14 @@ delta_scan_kernel(DeltaScanParams p) {
 #pragma unroll
         for (int i = 0; i < KT / 4; ++i) {
           const float4 kk = kr[i * 8 + kl], qq = qr[i * 8 + kl];
-          k2[j][2 * i] = make_float2(kk.x, kk.y);
-          k2[j][2 * i + 1] = make_float2(kk.z, kk.w);
+          kj[2 * i] = make_float2(kk.x, kk.y);
+          kj[2 * i + 1] = make_float2(kk.z, kk.w);
           const float2 q0 = make_float2(qq.x, qq.y), q1 = make_float2(qq.z, qq.w);
 #pragma unroll
           for (int c = 0; c < CT; ++c) {
-            dk[c] = fma2(S[c][2 * i], k2[j][2 * i], dk[c]);
+            dk[c] = fma2(S[c][2 * i], kj[2 * i], dk[c]);
             dq[c] = fma2(S[c][2 * i], q0, dq[c]);
-            dk[c] = fma2(S[c][2 * i + 1], k2[j][2 * i + 1], dk[c]);
+            dk[c] = fma2(S[c][2 * i + 1], kj[2 * i + 1], dk[c]);
             dq[c] = fma2(S[c][2 * i + 1], q1, dq[c]);
           }
         }
@@ -495,19 +614,45 @@ delta_scan_kernel(DeltaScanParams p) {
               orow[c] = fmaf(Gj, r1[c], fmaf(W.x, u[0][c], fmaf(W.y, u[1][c], fmaf(W.z, u[2][c], W.w * u[3][c]))));
         }
       }
-      const float2 g2 = make_float2(G.w, G.w);
-      const float cs[kBlk] = {cc.x, cc.y, cc.z, cc.w};
+      if constexpr (CH) {
+        const float4* gr = reinterpret_cast<const float4*>(base + Cfg::kG + bi * DK);
+        const float4* ur = reinterpret_cast<const float4*>(kqb + 2 * DK);
 #pragma unroll
-      for (int c = 0; c < CT; ++c) {
-        float2 uu[kBlk];
+        for (int i = 0; i < KT / 4; ++i) {
+          const float4 gg = gr[i * 8 + kl];
+          const float2 g0 = make_float2(gg.x, gg.y), g1 = make_float2(gg.z, gg.w);
 #pragma unroll
-        for (int j = 0; j < kBlk; ++j) uu[j] = make_float2(cs[j] * u[j][c], cs[j] * u[j][c]);
+          for (int c = 0; c < CT; ++c) {
+            S[c][2 * i] = mul2(S[c][2 * i], g0);
+            S[c][2 * i + 1] = mul2(S[c][2 * i + 1], g1);
+          }
 #pragma unroll
-        for (int i = 0; i < KT / 2; ++i) {
-          float2 acc = mul2(S[c][i], g2);
+          for (int j = 0; j < kBlk; ++j) {
+            const float4 kk = ur[j * (kVecs * DK / 4) + i * 8 + kl];
+            const float2 k0 = make_float2(kk.x, kk.y), k1 = make_float2(kk.z, kk.w);
 #pragma unroll
-          for (int j = 0; j < kBlk; ++j) acc = fma2(k2[j][i], uu[j], acc);
-          S[c][i] = acc;
+            for (int c = 0; c < CT; ++c) {
+              const float2 uu = make_float2(u[j][c], u[j][c]);
+              S[c][2 * i] = fma2(k0, uu, S[c][2 * i]);
+              S[c][2 * i + 1] = fma2(k1, uu, S[c][2 * i + 1]);
+            }
+          }
+        }
+      } else {
+        const float2 g2 = make_float2(G.w, G.w);
+        const float cs[kBlk] = {cc.x, cc.y, cc.z, cc.w};
+#pragma unroll
+        for (int c = 0; c < CT; ++c) {
+          float2 uu[kBlk];
+#pragma unroll
+          for (int j = 0; j < kBlk; ++j) uu[j] = make_float2(cs[j] * u[j][c], cs[j] * u[j][c]);
+#pragma unroll
+          for (int i = 0; i < KT / 2; ++i) {
+            float2 acc = mul2(S[c][i], g2);
+#pragma unroll
+            for (int j = 0; j < kBlk; ++j) acc = fma2(k2[j][i], uu[j], acc);
+            S[c][i] = acc;
+          }
         }
       }
     }
@@ -524,25 +669,25 @@ delta_scan_kernel(DeltaScanParams p) {
 }
 
 // ------------------------------------------------------------------ read-out norm and gate
-// y = o / rms(o) * weight * silu(gate) per (row, head), in the projection's type; columns past H * vdim of the output row
+// y = o / rms(o) * weight * gate per (row, head), in the projection's type; columns past H * vdim of the output row
 // are zeroed by the last head's warp. A warp takes one head of kNormRows rows; heads of up to 128 columns are read once,
 // all rows at a time, wider ones are read twice.
 constexpr int kNormRows = 4;
 
 template <typename T, bool NARROW>
 __global__ void __launch_bounds__(256)
-delta_gate_norm_kernel(DeltaGeom g, const float* o, const T* proj, const float* weight, T* y, long long ldy, int y_cols,
-                       int rows, float eps) {
+delta_gate_norm_kernel(DeltaGeom g, const float* o, const T* gate, long long ldg, int kind, const float* weight, T* y, long long ldy,
+                       int y_cols, int rows, float eps) {
   pdl_trigger();
   pdl_grid_wait();
   const int h = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (h >= g.H) return;
   constexpr bool kFast = sizeof(T) == 2;
-  const bool vec = g.vdim % 4 == 0 && ldy % 4 == 0;
+  const bool vec = g.vdim % 4 == 0 && ldy % 4 == 0 && ldg % 4 == 0;
   const int row_a = blockIdx.y * kNormRows, cnt = min(kNormRows, rows - row_a);
   const float inv_n = 1.f / static_cast<float>(g.vdim);
   const float* o0 = o + (static_cast<long long>(row_a) * g.H + h) * g.vp;
-  const T* g0 = proj + static_cast<long long>(row_a) * g.ldp + g.off_g + h * g.vdim;
+  const T* g0 = gate + static_cast<long long>(row_a) * ldg + h * g.vdim;
   T* y0 = y + row_a * ldy + h * g.vdim;
   const long long so = static_cast<long long>(g.H) * g.vp;
   auto store = [&](T* dst, int c, const float (&f)[4]) {
@@ -562,7 +707,7 @@ delta_gate_norm_kernel(DeltaGeom g, const float* o, const T* proj, const float* 
     for (int r = 0; r < kNormRows; ++r) {
       const int rr = min(r, cnt - 1);
       load_ch<float, 4>(o0 + rr * so + c, valid, true, f[r]);
-      load_ch<T, 4>(g0 + rr * g.ldp + c, valid, vec, gt[r]);
+      load_ch<T, 4>(g0 + rr * ldg + c, valid, vec, gt[r]);
     }
     load_ch<float, 4>(weight + c, valid, true, wt);
 #pragma unroll
@@ -570,7 +715,7 @@ delta_gate_norm_kernel(DeltaGeom g, const float* o, const T* proj, const float* 
       const float ss = warp_sum(f[r][0] * f[r][0] + f[r][1] * f[r][1] + f[r][2] * f[r][2] + f[r][3] * f[r][3]);
       const float rs = rsqrtf(fmaf(ss, inv_n, eps));
 #pragma unroll
-      for (int e = 0; e < 4; ++e) f[r][e] *= rs * wt[e] * silu_f<kFast>(gt[r][e]);
+      for (int e = 0; e < 4; ++e) f[r][e] *= rs * wt[e] * gate_f<kFast>(gt[r][e], kind);
       if (r < cnt && valid > 0) store(y0 + r * ldy, c, f[r]);
     }
   } else {
@@ -585,10 +730,10 @@ delta_gate_norm_kernel(DeltaGeom g, const float* o, const T* proj, const float* 
       for (int c = lane * 4; c < g.vdim; c += 128) {
         float f[4], gt[4], wt[4];
         load_ch<float, 4>(o0 + r * so + c, g.vdim - c, true, f);
-        load_ch<T, 4>(g0 + r * g.ldp + c, g.vdim - c, vec, gt);
+        load_ch<T, 4>(g0 + r * ldg + c, g.vdim - c, vec, gt);
         load_ch<float, 4>(weight + c, g.vdim - c, true, wt);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) f[e] *= rs * wt[e] * silu_f<kFast>(gt[e]);
+        for (int e = 0; e < 4; ++e) f[e] *= rs * wt[e] * gate_f<kFast>(gt[e], kind);
         store(y0 + r * ldy, c, f);
       }
     }
@@ -601,6 +746,7 @@ delta_gate_norm_kernel(DeltaGeom g, const float* o, const T* proj, const float* 
 // ------------------------------------------------------------------ decoded rows: one token per sequence, one launch
 struct DeltaStepParams {
   DeltaGeom g;
+  DeltaSide side;
   const void* proj;
   const float* conv_w;
   const float* a_log;
@@ -621,7 +767,7 @@ constexpr int kStepWarps = kStepThreads / 32;
 
 // CTA = (sequence, key head): it owns the head's q / k channels and all value heads that read them. A warp holds RPW
 // rows of a 128-column block of S: dim / 8 rounded up.
-template <typename T, int RPW>
+template <typename T, int RPW, bool CH>
 __global__ void __launch_bounds__(kStepThreads, RPW <= 16 ? 2 : 1)
 delta_step_kernel(DeltaStepParams p) {
   pdl_trigger();
@@ -635,6 +781,7 @@ delta_step_kernel(DeltaStepParams p) {
   float* so = sv + per * g.vp;             // [per * vp]
   float* part = so + per * g.vp;           // [8 warps][2][128]
   float* red = part + kStepWarps * 256;    // [8 warps][3]
+  float* sd = red + kStepWarps * 3 + 8;    // CH: [per * dkp] decays
   const int row = blockIdx.x, hk = blockIdx.y;
   const int slot = p.slots[row];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -713,6 +860,13 @@ delta_step_kernel(DeltaStepParams p) {
       *dst[h] = silu_f<sizeof(T) == 2>(acc);
     }
   }
+  if constexpr (CH) {
+    for (int i = tid; i < per * g.dim; i += kStepThreads) {
+      const int h = hk * per + i / g.dim, d = i % g.dim;
+      sd[(i / g.dim) * g.dkp + d] =
+          expf(-expf(p.a_log[h]) * softplus_f(p.side.dec[row * p.side.ld_dec + h * g.dim + d] + p.dt_bias[h * g.dim + d]));
+    }
+  }
   __syncthreads();
   float sqq = 0.f, skk = 0.f, sqk = 0.f;
   for (int d = tid; d < g.dim; d += kStepThreads) {
@@ -744,7 +898,8 @@ delta_step_kernel(DeltaStepParams p) {
   for (int it = 0; it < steps; ++it) {
     const int hh = it / col_blocks, h = hk * per + hh;
     if (it % col_blocks == 0) {
-      decay = expf(-expf(p.a_log[h]) * softplus_f(to_f32<T>(proj[g.off_a + h]) + p.dt_bias[h]));
+      decay = 1.f;                        // (CH: the products with the state take their channel's decay along)
+      if constexpr (!CH) decay = expf(-expf(p.a_log[h]) * softplus_f(to_f32<T>(proj[g.off_a + h]) + p.dt_bias[h]));
       beta = sigmoid_f(to_f32<T>(proj[g.off_b + h]));
     }
     float* st = state_at(it);
@@ -755,7 +910,12 @@ delta_step_kernel(DeltaStepParams p) {
 #pragma unroll
       for (int i = 0; i < RPW; ++i) {
         const int k = warp + kStepWarps * i;
-        const float kk = k < g.dim ? sk[k] * rk : 0.f, qq = k < g.dim ? sq[k] * rq : 0.f;
+        float kk = k < g.dim ? sk[k] * rk : 0.f, qq = k < g.dim ? sq[k] * rq : 0.f;
+        if constexpr (CH) {
+          const float dd = k < g.dim ? sd[hh * g.dkp + k] : 0.f;
+          kk *= dd;
+          qq *= dd;
+        }
         dk.x = fmaf(S[i].x, kk, dk.x); dk.y = fmaf(S[i].y, kk, dk.y);
         dk.z = fmaf(S[i].z, kk, dk.z); dk.w = fmaf(S[i].w, kk, dk.w);
         dq.x = fmaf(S[i].x, qq, dq.x); dq.y = fmaf(S[i].y, qq, dq.y);
@@ -794,12 +954,12 @@ delta_step_kernel(DeltaStepParams p) {
         for (int i = 0; i < RPW; ++i) {
           const int k = warp + kStepWarps * i;
           if (k < g.dim) {
-            const float kk = sk[k] * rk;
+            const float kk = sk[k] * rk, dd = CH ? sd[hh * g.dkp + k] : decay;
             float4 s = S[i];
-            s.x = fmaf(s.x, decay, kk * u.x);
-            s.y = fmaf(s.y, decay, kk * u.y);
-            s.z = fmaf(s.z, decay, kk * u.z);
-            s.w = fmaf(s.w, decay, kk * u.w);
+            s.x = fmaf(s.x, dd, kk * u.x);
+            s.y = fmaf(s.y, dd, kk * u.y);
+            s.z = fmaf(s.z, dd, kk * u.z);
+            s.w = fmaf(s.w, dd, kk * u.w);
             __stcs(reinterpret_cast<float4*>(st + static_cast<long long>(k) * g.vp), s);
           }
         }
@@ -809,6 +969,7 @@ delta_step_kernel(DeltaStepParams p) {
     }
   }
   // read-out norm and gate: one warp per value head
+  const T* gate = static_cast<const T*>(p.side.gate) + row * p.side.ld_gate;
   for (int hh = warp; hh < per; hh += kStepWarps) {
     const float* orow = so + hh * g.vp;
     const int c0 = (hk * per + hh) * g.vdim;
@@ -817,54 +978,57 @@ delta_step_kernel(DeltaStepParams p) {
     ss = warp_sum(ss);
     const float r = 1.f / sqrtf(ss / static_cast<float>(g.vdim) + p.eps);
     for (int c = lane; c < g.vdim; c += 32)
-      y[c0 + c] = from_f32<T>(orow[c] * r * p.norm_w[c] * silu_f(to_f32<T>(proj[g.off_g + c0 + c])));
+      y[c0 + c] = from_f32<T>(orow[c] * r * p.norm_w[c] * gate_f(to_f32<T>(gate[c0 + c]), p.side.gate_kind));
   }
 }
 
-// geom: 12 ints in the order of DeltaGeom (without ldp)
-bool read_geom(const int* v, long long ldp, DeltaGeom* g) {
+// geom: 11 ints in the order of DeltaGeom (without ldp), then the gate's kind; off_a is not used with dec
+bool read_geom(const int* v, long long ldp, const void* gate, long long ld_gate, const float* dec, long long ld_dec, DeltaGeom* g, DeltaSide* side) {
   g->Hk = v[0]; g->H = v[1]; g->dim = v[2]; g->vdim = v[3]; g->dkp = v[4]; g->vp = v[5];
-  g->off_k = v[6]; g->off_v = v[7]; g->off_g = v[8]; g->off_b = v[9]; g->off_a = v[10]; g->conv_c = v[11];
+  g->off_k = v[6]; g->off_v = v[7]; g->off_b = v[8]; g->off_a = v[9]; g->conv_c = v[10];
   g->ldp = ldp;
+  *side = {gate, ld_gate, v[11], dec, ld_dec};
+  if (!gate || ld_gate < g->H * g->vdim || v[11] < 0 || v[11] > 1 || ldp < g->off_b + g->H || (!dec && ldp < g->off_a + g->H) ||
+      (dec && (ld_dec < g->H * g->dim || ld_dec % 4 || (reinterpret_cast<uintptr_t>(dec) & 15))))
+    return false;
   const bool dk_ok = g->dkp == 32 || g->dkp == 64 || g->dkp == 128 || g->dkp == 256;
   return g->Hk > 0 && g->H > 0 && g->H % g->Hk == 0 && g->dim > 0 && g->vdim > 0 && dk_ok && g->dim <= g->dkp &&
-         g->vp >= g->vdim && g->vp % 4 == 0 && g->conv_c > 0 && ldp >= g->off_a + g->H && ldp % 8 == 0 && g->off_k % 8 == 0 &&
-         g->off_v % 8 == 0 && g->off_g % 8 == 0 && g->conv_c % 8 == 0;
+         g->vp >= g->vdim && g->vp % 4 == 0 && g->conv_c > 0 && ldp % 8 == 0 && g->off_k % 8 == 0 && g->off_v % 8 == 0 && g->conv_c % 8 == 0;
 }
 
-template <typename T, int TAPS>
+template <typename T, int TAPS, bool CH>
 int launch_prepare_taps(const DeltaPrepParams& p, cudaStream_t s) {
   const DeltaGeom& g = p.g;
   const dim3 grid(g.Hk + (g.H * g.vdim + 255) / 256, (p.blocks + 3) / 4);
   const bool pdl = pdl_all_enabled();
   switch (g.dkp) {
-    case 32: launch_pdl(delta_prepare_kernel<T, TAPS, 1>, grid, dim3(128), 0, s, pdl, p); break;
-    case 64: launch_pdl(delta_prepare_kernel<T, TAPS, 2>, grid, dim3(128), 0, s, pdl, p); break;
-    case 128: launch_pdl(delta_prepare_kernel<T, TAPS, 4>, grid, dim3(128), 0, s, pdl, p); break;
-    default: launch_pdl(delta_prepare_kernel<T, TAPS, 8>, grid, dim3(128), 0, s, pdl, p); break;
+    case 32: launch_pdl(delta_prepare_kernel<T, TAPS, 1, CH>, grid, dim3(128), 0, s, pdl, p); break;
+    case 64: launch_pdl(delta_prepare_kernel<T, TAPS, 2, CH>, grid, dim3(128), 0, s, pdl, p); break;
+    case 128: launch_pdl(delta_prepare_kernel<T, TAPS, 4, CH>, grid, dim3(128), 0, s, pdl, p); break;
+    default: launch_pdl(delta_prepare_kernel<T, TAPS, 8, CH>, grid, dim3(128), 0, s, pdl, p); break;
   }
   return static_cast<int>(cudaGetLastError());
 }
 
-template <typename T>
+template <typename T, bool CH>
 int launch_prepare(const DeltaPrepParams& p, int taps, cudaStream_t s) {
   switch (taps) {
-    case 1: return launch_prepare_taps<T, 1>(p, s);
-    case 2: return launch_prepare_taps<T, 2>(p, s);
-    case 3: return launch_prepare_taps<T, 3>(p, s);
-    case 4: return launch_prepare_taps<T, 4>(p, s);
-    case 5: return launch_prepare_taps<T, 5>(p, s);
-    case 6: return launch_prepare_taps<T, 6>(p, s);
-    case 7: return launch_prepare_taps<T, 7>(p, s);
-    case 8: return launch_prepare_taps<T, 8>(p, s);
+    case 1: return launch_prepare_taps<T, 1, CH>(p, s);
+    case 2: return launch_prepare_taps<T, 2, CH>(p, s);
+    case 3: return launch_prepare_taps<T, 3, CH>(p, s);
+    case 4: return launch_prepare_taps<T, 4, CH>(p, s);
+    case 5: return launch_prepare_taps<T, 5, CH>(p, s);
+    case 6: return launch_prepare_taps<T, 6, CH>(p, s);
+    case 7: return launch_prepare_taps<T, 7, CH>(p, s);
+    case 8: return launch_prepare_taps<T, 8, CH>(p, s);
     default: return -2;
   }
 }
 
-template <int KT, int CT>
+template <int KT, int CT, bool CH>
 int launch_scan_cols(const DeltaScanParams& p, int nseq, cudaStream_t s) {
-  using Cfg = ScanCfg<KT, CT>;
-  auto kern = delta_scan_kernel<KT, CT>;
+  using Cfg = ScanCfg<KT, CT, CH>;
+  auto kern = delta_scan_kernel<KT, CT, CH>;
   static PerDeviceFlag attr;
   if (attr.unset()) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes);
@@ -878,7 +1042,7 @@ int launch_scan_cols(const DeltaScanParams& p, int nseq, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int KT>
+template <int KT, bool CH>
 int launch_scan(const DeltaScanParams& p, int nseq, cudaStream_t s) {
   static const int forced = [] { const char* e = getenv("TESSERACT_DELTA_COLS"); return e ? atoi(e) : 0; }();
   // columns of the whole launch against what one warp per scheduler covers
@@ -886,16 +1050,26 @@ int launch_scan(const DeltaScanParams& p, int nseq, cudaStream_t s) {
   int ct = forced ? forced : (cols >= 5 * one ? 4 : (cols >= one ? 2 : 1));
   if (KT > 16 && ct > 2) ct = 2;
   if constexpr (KT <= 16)
-    if (ct == 4) return launch_scan_cols<KT, 4>(p, nseq, s);
-  return ct >= 2 ? launch_scan_cols<KT, 2>(p, nseq, s) : launch_scan_cols<KT, 1>(p, nseq, s);
+    if (ct == 4) return launch_scan_cols<KT, 4, CH>(p, nseq, s);
+  return ct >= 2 ? launch_scan_cols<KT, 2, CH>(p, nseq, s) : launch_scan_cols<KT, 1, CH>(p, nseq, s);
 }
 
-template <typename T, int RPW>
+template <bool CH>
+int launch_scan_dim(const DeltaScanParams& p, int nseq, cudaStream_t s) {
+  switch (p.g.dkp) {
+    case 32: return launch_scan<4, CH>(p, nseq, s);
+    case 64: return launch_scan<8, CH>(p, nseq, s);
+    case 128: return launch_scan<16, CH>(p, nseq, s);
+    default: return launch_scan<32, CH>(p, nseq, s);
+  }
+}
+
+template <typename T, int RPW, bool CH>
 int launch_step(const DeltaStepParams& p, int rows, cudaStream_t s) {
   const int per = p.g.H / p.g.Hk;
-  const int smem = (2 * p.g.dkp + 2 * per * p.g.vp + kStepWarps * 256 + kStepWarps * 3 + 8) * 4;
+  const int smem = (2 * p.g.dkp + 2 * per * p.g.vp + kStepWarps * 256 + kStepWarps * 3 + 8 + (CH ? per * p.g.dkp : 0)) * 4;
   if (smem > 200 * 1024) return -2;
-  auto kern = delta_step_kernel<T, RPW>;
+  auto kern = delta_step_kernel<T, RPW, CH>;
   static PerDeviceFlag attr;
   if (attr.unset()) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
@@ -910,22 +1084,26 @@ int launch_step(const DeltaStepParams& p, int rows, cudaStream_t s) {
 }  // namespace tsb
 
 // Prompt rows [rows, ldp] of nseq sequences, cut into blocks of 4 tokens from each sequence's first row (blk_seq [blocks],
-// blk0 [nseq + 1]). dtype: 0 = fp32, 1 = bf16 (projection, convolution state, y). `kq`, `v`, `coef`, `o` are fp32 scratch
-// of rows * Hk * 2 * dkp, rows * H * vp, blocks * H * 36 and rows * H * vp elements (16-byte aligned). See the
-// structures above for the rest.
-TSB_EXPORT int tsb_delta_prefill(const void* proj, long long ldp, const int* geom, const float* conv_w, const float* a_log,
-                                 const float* dt_bias, const float* norm_w, void* conv_state, float* state, const int* cu,
-                                 const int* slots, const int* pos0, const int* blk_seq, const int* blk0, float* kq, float* v,
-                                 float* coef, float* o, void* y, long long ldy, int y_cols, int rows, int blocks, int nseq,
-                                 int taps, float eps, int dtype, void* stream) {
+// blk0 [nseq + 1]). dtype: 0 = fp32, 1 = bf16 (projection, gate, convolution state, y). `kq`, `v`, `coef`, `o` are fp32 scratch
+// of rows * Hk * 2 * dkp, rows * H * vp, blocks * H * 36 and rows * H * vp elements (16-byte aligned). With `dec` [rows, ld_dec]
+// (dt_bias then is [H * dim]) kq has rows * H * 3 * dkp elements and `g4` is scratch of blocks * H * dkp. See the structures above
+// for the rest.
+TSB_EXPORT int tsb_delta_prefill(const void* proj, long long ldp, const int* geom, const void* gate, long long ld_gate, const float* dec,
+                                 long long ld_dec, const float* conv_w, const float* a_log, const float* dt_bias, const float* norm_w,
+                                 void* conv_state, float* state, const int* cu, const int* slots, const int* pos0, const int* blk_seq,
+                                 const int* blk0, float* kq, float* g4, float* v, float* coef, float* o, void* y, long long ldy, int y_cols,
+                                 int rows, int blocks, int nseq, int taps, float eps, int dtype, void* stream) {
   using namespace tsb;
   DeltaGeom g;
-  if (!read_geom(geom, ldp, &g) || rows <= 0 || blocks <= 0 || nseq <= 0 || nseq > 65535 || taps < 1 || taps > 8 ||
-      (blocks + 3) / 4 > 65535 || (rows + kNormRows - 1) / kNormRows > 65535 || (dtype != 0 && dtype != 1) || y_cols < g.H * g.vdim)
+  DeltaSide side;
+  if (!read_geom(geom, ldp, gate, ld_gate, dec, ld_dec, &g, &side) || rows <= 0 || blocks <= 0 || nseq <= 0 || nseq > 65535 || taps < 1 ||
+      taps > 8 || (blocks + 3) / 4 > 65535 || (rows + kNormRows - 1) / kNormRows > 65535 || (dtype != 0 && dtype != 1) ||
+      y_cols < g.H * g.vdim || (dec && !g4))
     return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  DeltaPrepParams pp{g, proj, conv_w, a_log, dt_bias, conv_state, cu, slots, pos0, blk_seq, blk0, kq, v, coef, blocks};
-  int rc = dtype == 1 ? launch_prepare<__nv_bfloat16>(pp, taps, s) : launch_prepare<float>(pp, taps, s);
+  DeltaPrepParams pp{g, proj, conv_w, a_log, dt_bias, dec, ld_dec, conv_state, cu, slots, pos0, blk_seq, blk0, kq, g4, v, coef, blocks};
+  int rc = dec ? (dtype == 1 ? launch_prepare<__nv_bfloat16, true>(pp, taps, s) : launch_prepare<float, true>(pp, taps, s))
+               : (dtype == 1 ? launch_prepare<__nv_bfloat16, false>(pp, taps, s) : launch_prepare<float, false>(pp, taps, s));
   if (rc) return rc;
   const bool pdl = pdl_all_enabled();
   if (taps > 1) {
@@ -939,19 +1117,14 @@ TSB_EXPORT int tsb_delta_prefill(const void* proj, long long ldp, const int* geo
     rc = static_cast<int>(cudaGetLastError());
     if (rc) return rc;
   }
-  DeltaScanParams sp{g, kq, v, coef, state, o, cu, slots, pos0, blk0};
-  switch (g.dkp) {
-    case 32: rc = launch_scan<4>(sp, nseq, s); break;
-    case 64: rc = launch_scan<8>(sp, nseq, s); break;
-    case 128: rc = launch_scan<16>(sp, nseq, s); break;
-    default: rc = launch_scan<32>(sp, nseq, s); break;
-  }
+  DeltaScanParams sp{g, kq, g4, v, coef, state, o, cu, slots, pos0, blk0};
+  rc = dec ? launch_scan_dim<true>(sp, nseq, s) : launch_scan_dim<false>(sp, nseq, s);
   if (rc) return rc;
   const dim3 ngrid((g.H + 7) / 8, (rows + kNormRows - 1) / kNormRows);
   auto norm = [&](auto tag, auto narrow) {
     using T = decltype(tag);
-    launch_pdl(delta_gate_norm_kernel<T, decltype(narrow)::value>, ngrid, dim3(256), 0, s, pdl, g, o, static_cast<const T*>(proj),
-               norm_w, static_cast<T*>(y), ldy, y_cols, rows, eps);
+    launch_pdl(delta_gate_norm_kernel<T, decltype(narrow)::value>, ngrid, dim3(256), 0, s, pdl, g, o, static_cast<const T*>(gate), ld_gate,
+               side.gate_kind, norm_w, static_cast<T*>(y), ldy, y_cols, rows, eps);
   };
   const bool narrow = g.vdim <= 128;
   if (dtype == 1) narrow ? norm(__nv_bfloat16{}, std::true_type{}) : norm(__nv_bfloat16{}, std::false_type{});
@@ -960,18 +1133,21 @@ TSB_EXPORT int tsb_delta_prefill(const void* proj, long long ldp, const int* geo
 }
 
 // Decoded rows: row i is the next token of the sequence in slot slots[i] (-1: padding, y = 0) at position pos[i].
-TSB_EXPORT int tsb_delta_step(const void* proj, long long ldp, const int* geom, const float* conv_w, const float* a_log,
-                              const float* dt_bias, const float* norm_w, void* conv_state, float* state, const int* slots,
-                              const int* pos, void* y, long long ldy, int y_cols, int rows, int taps, float eps, int dtype,
-                              void* stream) {
+TSB_EXPORT int tsb_delta_step(const void* proj, long long ldp, const int* geom, const void* gate, long long ld_gate, const float* dec,
+                              long long ld_dec, const float* conv_w, const float* a_log, const float* dt_bias, const float* norm_w,
+                              void* conv_state, float* state, const int* slots, const int* pos, void* y, long long ldy, int y_cols, int rows,
+                              int taps, float eps, int dtype, void* stream) {
   using namespace tsb;
   DeltaGeom g;
-  if (!read_geom(geom, ldp, &g) || rows <= 0 || g.Hk > 65535 || taps < 1 || taps > 8 || (dtype != 0 && dtype != 1) ||
-      y_cols < g.H * g.vdim)
+  DeltaSide side;
+  if (!read_geom(geom, ldp, gate, ld_gate, dec, ld_dec, &g, &side) || rows <= 0 || g.Hk > 65535 || taps < 1 || taps > 8 ||
+      (dtype != 0 && dtype != 1) || y_cols < g.H * g.vdim)
     return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  DeltaStepParams p{g, proj, conv_w, a_log, dt_bias, norm_w, conv_state, state, slots, pos, y, ldy, y_cols, taps, eps};
-#define TSB_STEP(R) return dtype == 1 ? launch_step<__nv_bfloat16, R>(p, rows, s) : launch_step<float, R>(p, rows, s)
+  DeltaStepParams p{g, side, proj, conv_w, a_log, dt_bias, norm_w, conv_state, state, slots, pos, y, ldy, y_cols, taps, eps};
+#define TSB_STEP(R)                                                                                                       \
+  if (dec) return dtype == 1 ? launch_step<__nv_bfloat16, R, true>(p, rows, s) : launch_step<float, R, true>(p, rows, s); \
+  return dtype == 1 ? launch_step<__nv_bfloat16, R, false>(p, rows, s) : launch_step<float, R, false>(p, rows, s)
   switch (g.dkp) {
     case 32: TSB_STEP(4);
     case 64: TSB_STEP(8);

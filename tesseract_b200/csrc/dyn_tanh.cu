@@ -179,11 +179,12 @@ void launch_residual(const DynTanhParams& p, dim3 grid, cudaStream_t s) {
 }
 
 // out[r, c] = g sigmoid(slope g) (u + shift), g = min(scale * gate + bias, limit), u = clamp(scale * up + bias, -limit, limit);
-// gate and up are the two halves of a row. (limit = infinity, slope 1, shift 0: SiLU(g) u.)
+// gate and up are the two halves of a row; sigmoid(slope (g + cubic g^3)) with a cubic. (limit = infinity, shift 0: SiLU(g) u for
+// slope 1, the tanh form of GELU(g) u for slope 2 sqrt(2 / pi) and cubic 0.044715.)
 template <typename T>
 __global__ void __launch_bounds__(256)
 clamped_glu_kernel(const T* gu, long long ldg, const float* bias, T* out, long long ldo, int rows, int F, float limit, float slope,
-                   float shift, float scale) {
+                   float shift, float scale, float cubic) {
   pdl_trigger();
   pdl_grid_wait();
   constexpr int V = 16 / sizeof(T);
@@ -227,7 +228,8 @@ clamped_glu_kernel(const T* gu, long long ldg, const float* bias, T* out, long l
       for (int i = 0; i < V; ++i) {
         const float gg = fminf(fmaf(to_f32<T>(g[k].v[i]), scale, gb[i]), limit);
         const float uu = fminf(fmaxf(fmaf(to_f32<T>(u[k].v[i]), scale, ub[i]), -limit), limit);
-        const float q = sizeof(T) == 2 ? __fdividef(gg, 1.f + __expf(-slope * gg)) : gg / (1.f + expf(-slope * gg));
+        const float a = -slope * fmaf(cubic * gg * gg, gg, gg);
+        const float q = sizeof(T) == 2 ? __fdividef(gg, 1.f + __expf(a)) : gg / (1.f + expf(a));
         y.v[i] = from_f32<T>(q * (uu + shift));
       }
       *reinterpret_cast<Vec*>(out + static_cast<long long>(r0 + k) * ldo + c) = y;
@@ -279,7 +281,7 @@ TSB_EXPORT int tsb_dyn_tanh_residual(float* x, int rows, int W, const void* y, l
 // gate_up [rows, 2 F] (row stride ldg), bias fp32 [2 F] or null, out [rows, F] (row stride ldo); F and the strides are
 // multiples of 8 and the bases 16-byte aligned.
 TSB_EXPORT int tsb_clamped_glu(const void* gate_up, long long ldg, const float* bias, void* out, long long ldo, int rows, int F,
-                               float limit, float slope, float shift, float scale, int dtype, void* stream) {
+                               float limit, float slope, float shift, float scale, float cubic, int dtype, void* stream) {
   using namespace tsb;
   if (rows <= 0 || F <= 0 || F % 8 || ldg % 8 || ldo % 8 || (dtype != 0 && dtype != 1)) return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -287,9 +289,9 @@ TSB_EXPORT int tsb_clamped_glu(const void* gate_up, long long ldg, const float* 
   if (dtype == 1)
     launch_pdl(clamped_glu_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl_all_enabled(),
                static_cast<const __nv_bfloat16*>(gate_up), ldg, bias, static_cast<__nv_bfloat16*>(out), ldo, rows, F, limit, slope,
-               shift, scale);
+               shift, scale, cubic);
   else
     launch_pdl(clamped_glu_kernel<float>, grid, dim3(256), 0, s, pdl_all_enabled(), static_cast<const float*>(gate_up), ldg, bias,
-               static_cast<float*>(out), ldo, rows, F, limit, slope, shift, scale);
+               static_cast<float*>(out), ldo, rows, F, limit, slope, shift, scale, cubic);
   return static_cast<int>(cudaGetLastError());
 }

@@ -69,6 +69,7 @@ struct GroupArgs {
   const int* row_tags = nullptr;
   long long peer_rows = 0;
   void* peer_out[8] = {};
+  int act = 0;             // mode 1: 1 = relu(result)^2
   int inputs = 0;
   int a_group_rows = 0;
   int col_start[8] = {};
@@ -285,6 +286,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         if (gmode == 2 && empty_slice) {  // a group without rows: nothing was accumulated
 #pragma unroll
           for (int j = 0; j < 32; ++j) r[j] = 0u;
+        }
+        if (gmode == 1 && grp.act) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float f = fmaxf(__uint_as_float(r[j]), 0.f);
+            r[j] = __float_as_uint(f * f);
+          }
         }
         const int col0 = n0 + c * 32;
         if (row_ok && col0 < N) {
@@ -504,16 +512,17 @@ TSB_EXPORT int tsb_gemm_bf16(const void* A, const void* B, void* C, int M, int N
 //   mode 1 (rows grouped):  C[r, :] = A[r, :] * op(B[g(r)])  for the row blocks below offsets[groups].
 //       A [rows_cap, K] bf16 (lda), C [rows_cap, N] bf16 (ldc); rows_cap >= offsets[groups] is the allocated height.
 //       b_mn = 0: B[g] is [N, K];  b_mn = 1: B[g] is [K, N]  (row stride ldb); B[g] starts b_group_stride elements
-//       after B[g - 1] (a multiple of ldb: the groups need not be packed, e.g. expert weights in a flat arena).
+//       after B[g - 1] (a multiple of ldb: the groups need not be packed, e.g. expert weights in a flat arena). act = 1: relu(C)^2.
 //   mode 2 (reduction grouped, expert weight gradient):  C[g] (+)= A[rows of g, :]^T * B[rows of g, :]
 //       A [rows_cap, M] bf16 (lda), B [rows_cap, N] bf16 (ldb), C[g] [M, N] fp32 or bf16 (ldc), C[g] starting
 //       c_group_stride elements after C[g - 1].
 // Returns 0, a cudaError_t, -2 (bad argument) or -3 (tensor map encoding failed).
 TSB_EXPORT int tsb_gemm_grouped(const void* A, const void* B, void* C, const int* offsets, int groups, int mode,
                                 int rows_cap, int M, int N, int K, long long lda, long long ldb, long long ldc, int b_mn,
-                                long long b_group_stride, long long c_group_stride, int out_f32, int accumulate,
+                                long long b_group_stride, long long c_group_stride, int out_f32, int accumulate, int act,
                                 void* stream) {
   using namespace tsb;
+  if (act < 0 || act > 1 || (act && mode != 1)) return -2;
   if (!offsets || groups < 1 || groups > 1024 || rows_cap <= 0 || rows_cap % BM || N <= 0) return -2;
   if ((reinterpret_cast<uintptr_t>(A) & 15) || (reinterpret_cast<uintptr_t>(B) & 15) || (lda % 8) || (ldb % 8)) return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -531,6 +540,7 @@ TSB_EXPORT int tsb_gemm_grouped(const void* A, const void* B, void* C, const int
                          : cached_tmap_2d(&tb, B, map_rows, K, ldb * 2, bn, BK);
     if (!ok) return -3;
     GroupArgs g{offsets, groups, 1, grows, 0};
+    g.act = act;
     auto go = [&](auto bn_tag, auto bmn_tag) {
       return launch_cfg<decltype(bn_tag)::value, false, decltype(bmn_tag)::value, __nv_bfloat16, false>(
           ta, tb, C, rows_cap, N, K, ldc, 0, s, 1, g);

@@ -24,6 +24,12 @@ struct HeadTile {
   // `cols` of them exist); 64 rows of either are less than 2^31 elements apart. K is a multiple of 16; all starts and strides are multiples of 16 bytes.
   static __device__ __forceinline__ float* run(uint8_t* smem, const T* x, long long ldx, int rows, const T* const (&w)[NW],
                                                long long ldw, int cols, int K) {
+    const int ldx32 = static_cast<int>(ldx);
+    return run_rows(smem, [&](int r) -> const T* { return r < rows ? x + r * ldx32 : nullptr; }, w, ldw, cols, K);
+  }
+  // The same with rows anywhere: x_row(r) is row r of the tile, or null for zeros.
+  template <typename Row>
+  static __device__ __forceinline__ float* run_rows(uint8_t* smem, Row x_row, const T* const (&w)[NW], long long ldw, int cols, int K) {
     constexpr int V = kVec16<T>, kPieces = kStep / V;
     T* ring = reinterpret_cast<T*>(smem);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -31,17 +37,19 @@ struct HeadTile {
     // a thread copies the same 16-byte column of every kPass-th row of the input and of the matrices
     constexpr int kPass = kThreads / kPieces, kRowsX = BM / kPass > 0 ? BM / kPass : 1, kRowsW = BN / kPass;
     const int pr = tid / kPieces, pk = (tid % kPieces) * V;
-    const int ldx32 = static_cast<int>(ldx), ldw32 = static_cast<int>(ldw);
+    const int ldw32 = static_cast<int>(ldw);
+    const T* xr[kRowsX];
+#pragma unroll
+    for (int i = 0; i < kRowsX; ++i) xr[i] = BM >= kPass || pr < BM ? x_row(pr + i * kPass) : nullptr;
     auto issue = [&](int s) {
       T* st = ring + (s % kStages) * kStageElems + pr * kLd + pk;
       const int k = s * kStep + pk;
       const bool in_k = k < K;
 #pragma unroll
       for (int i = 0; i < kRowsX; ++i) {
-        const int r = pr + i * kPass;
-        if (BM < kPass && r >= BM) break;
-        const bool ok = in_k && r < rows;
-        cp_async_16(smem_u32(st + i * kPass * kLd), ok ? x + r * ldx32 + k : x, ok ? 16 : 0);
+        if (BM < kPass && pr >= BM) break;
+        const bool ok = in_k && xr[i] != nullptr;
+        cp_async_16(smem_u32(st + i * kPass * kLd), ok ? xr[i] + k : w[0], ok ? 16 : 0);
       }
 #pragma unroll
       for (int i = 0; i < NW; ++i)

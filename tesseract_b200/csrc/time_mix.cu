@@ -1,6 +1,12 @@
-// Time mixing (linear attention with a decay per key channel and token and a bonus for the current token), for ragged batches:
+// Linear attention with a decay per key channel and token, for ragged batches of sequences, in two forms. Time mixing (a bonus for
+// the current token, which the read-out sees otherwise):
 //
 //   o_t = (S_(t-1) + v_t (u k_t)^T) r_t,  S_t = diag(w_t) S_(t-1) + v_t k_t^T,  w = exp(-exp(d + w0))      per head
+//
+// and gated linear attention (the read-out sees the state with the current token in it):
+//
+//   S_t = diag(w_t) S_(t-1) + v_t k_t^T,  o_t = S_t r_t,  w = sigmoid(d + w0)^(1 / tau)
+//
 //   out = o / rms(o) * norm * silu(gate)
 //
 // S is [values][keys] in fp32 and stays so. token_shift_kernel makes the inputs of the five projections, mixes of a row and the
@@ -12,7 +18,7 @@
 //   S  <- S diag(W_15)
 //   o_i = S R_i + sum_{j < i} (R_i . K_j) v_j + (u k_i . r_i) v_i
 //   S  <- S + sum_j v_j K_j^T
-// Where a channel decays by more than 2^60 in a block, 1 / W_15 is not formed: R_i = r_i W_(i-1) meets S before it decays, and the
+// (gated: R_i = r_i W_i / W_15, and the sum takes j = i along instead of the bonus). Where a channel decays by more than 2^60 in a block, 1 / W_15 is not formed: R_i = r_i W_(i-1) (gated: W_i) meets S before it decays, and the
 // pairs are summed with the decays in between, one by one. S stays in the accumulators of the products (values on rows), which is
 // also the layout in which it enters the read-out. Factors that must not lose their 32 bits meet the tensor cores as two bf16 halves
 // (16 bits).
@@ -119,26 +125,35 @@ tanh_rows_kernel(const T* x, long long ld, T* out, int cols, long long vecs) {
 }
 
 // ------------------------------------------------------------------ the recurrence
+enum MixKind { kTime, kGated };
+
 struct MixParams {
-  int H, dim, dp, rp, section, rows, n_seq, ld, ldo;
-  const void* proj;          // [rows, ld]: r, k, v, gate `section` columns apart, then the decay's inputs
-  const float* dec;          // [rows, H * dp] (prompts)
-  const void* w2;            // [H * dp, rp] (decoded rows)
+  int H, dim, dp, ep, rp, off_k, off_v, off_g, off_low, rows, n_seq, ld, ldo;    // dim: columns of a value head, ep: as stored; dp: of a key
+  const void* proj;          // [rows, ld]: r, k (heads of dp columns), v, gate (of ep), time mixing: the decay's inputs
+  const float* dec;          // [rows, ld_dec] (time mixing: prompts)
+  long long ld_dec;
+  const void* w2;            // [H * dp, rp] (time mixing, decoded rows)
   const float* w0;           // [H * dp]
-  const float* u;
-  const float* norm;
-  float* state;              // [slots, H, dp, dp]
+  const float* u;            // [H * dp] (time mixing)
+  const float* norm;         // [H * ep]
+  float* state;              // [slots, H, ep, dp]
   const int* slots;
   const int* positions;      // decoded rows
   const int* cu;             // prompts
   const int* pos0;
   void* out;                 // [rows, ldo]
-  float* o;                  // [rows, H, dp] read-outs of the scan
+  float* o;                  // [rows, H, ep] read-outs of the scan
   SpanParams span;
-  float eps, out_scale;
+  float eps, out_scale, r_scale, inv_tau;
 };
 
-template <typename T, int RL>
+template <int KIND, bool FAST = false>
+__device__ __forceinline__ float decay_of(float x, float inv_tau) {
+  if constexpr (KIND == kTime) return expf(-(FAST ? __expf(x) : expf(x)));
+  return expf(-inv_tau * (fmaxf(-x, 0.f) + log1pf(FAST ? __expf(-fabsf(x)) : expf(-fabsf(x)))));
+}
+
+template <typename T, int RL, int KIND>
 __global__ void __launch_bounds__(128)
 time_mix_scan_kernel(MixParams p) {
   pdl_trigger();
@@ -147,27 +162,27 @@ time_mix_scan_kernel(MixParams p) {
   const int h = blockIdx.y, seq = blockIdx.z, slot = p.slots[seq];
   const int row0 = p.cu[seq], n = p.cu[seq + 1] - row0;
   if (slot < 0 || n <= 0) return;
-  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ld + h * p.dp;
-  const float* dec = p.dec + static_cast<long long>(row0) * p.H * p.dp + h * p.dp;
+  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ld;
+  const float* dec = p.dec + static_cast<long long>(row0) * p.ld_dec + h * p.dp;
   const float* w0 = p.w0 + h * p.dp;
-  float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp;
-  float* o = p.o + static_cast<long long>(row0) * p.H * p.dp + h * p.dp;
-  state_scan<RL, false>(
-      sm, st, p.dp, p.dp, p.pos0[seq] == 0, n, blockIdx.x * kScanRows,
+  float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.ep * p.dp;
+  float* o = p.o + static_cast<long long>(row0) * p.H * p.ep + h * p.ep;
+  state_scan<RL, KIND == kGated>(
+      sm, st, p.ep, p.dp, p.pos0[seq] == 0, n, blockIdx.x * kScanRows,
       [&](int t, int d, float& q, float& k, float& w) {
-        const T* r = x + static_cast<long long>(t) * p.ld + d;
-        q = to_f32<T>(r[0]);
-        k = to_f32<T>(r[p.section]);
-        w = expf(-expf(dec[static_cast<long long>(t) * p.H * p.dp + d] + w0[d]));
+        const T* r = x + static_cast<long long>(t) * p.ld + h * p.dp + d;
+        q = p.r_scale * to_f32<T>(r[0]);
+        k = to_f32<T>(r[p.off_k]);
+        w = decay_of<KIND>(dec[t * p.ld_dec + d] + w0[d], p.inv_tau);
       },
-      [&](int t, int e) { return to_f32<T>(x[static_cast<long long>(t) * p.ld + 2 * p.section + e]); },
+      [&](int t, int e) { return to_f32<T>(x[static_cast<long long>(t) * p.ld + p.off_v + h * p.ep + e]); },
       [&](int t, int e, const float (&f)[4]) {
-        *reinterpret_cast<float4*>(o + static_cast<long long>(t) * p.H * p.dp + e) = make_float4(f[0], f[1], f[2], f[3]);
+        *reinterpret_cast<float4*>(o + static_cast<long long>(t) * p.H * p.ep + e) = make_float4(f[0], f[1], f[2], f[3]);
       });
 }
 
-// out = (o + v (u k . r)) / rms * norm * silu(gate): one warp per (row, head).
-template <typename T>
+// out = (o + v (u k . r)) / rms * norm * silu(gate): one warp per (row, head). Gated: without the bonus.
+template <typename T, int KIND>
 __global__ void __launch_bounds__(256)
 time_mix_norm_kernel(MixParams p) {
   pdl_trigger();
@@ -177,20 +192,24 @@ time_mix_norm_kernel(MixParams p) {
   if (w >= static_cast<long long>(p.rows) * p.H) return;
   const long long row = w / p.H;
   const int h = static_cast<int>(w % p.H);
-  const T* x = static_cast<const T*>(p.proj) + row * p.ld + h * p.dp;
-  const float *o = p.o + w * p.dp, *u = p.u + h * p.dp, *norm = p.norm + h * p.dp;
-  T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.dp;
+  const T *x = static_cast<const T*>(p.proj) + row * p.ld, *v = x + p.off_v + h * p.ep, *gate = x + p.off_g + h * p.ep;
+  const float *o = p.o + w * p.ep, *norm = p.norm + h * p.ep;
+  T* out = static_cast<T*>(p.out) + row * p.ldo + h * p.ep;
   float bonus = 0.f, ss = 0.f;
-  for (int d = lane; d < p.dp; d += 32) bonus = fmaf(u[d] * to_f32<T>(x[p.section + d]), to_f32<T>(x[d]), bonus);
-  bonus = warp_sum(bonus);
-  for (int d = lane; d < p.dp; d += 32) {
-    const float f = fmaf(to_f32<T>(x[2 * p.section + d]), bonus, o[d]);
+  if constexpr (KIND == kTime) {
+    const T* r = x + h * p.dp;
+    const float* u = p.u + h * p.dp;
+    for (int d = lane; d < p.dp; d += 32) bonus = fmaf(u[d] * to_f32<T>(r[p.off_k + d]), to_f32<T>(r[d]), bonus);
+    bonus = warp_sum(bonus);
+  }
+  for (int d = lane; d < p.ep; d += 32) {
+    const float f = fmaf(to_f32<T>(v[d]), bonus, o[d]);
     ss = fmaf(f, f, ss);
   }
   const float r = p.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(p.dim) + p.eps);
-  for (int d = lane; d < p.dp; d += 32) {
-    const float f = fmaf(to_f32<T>(x[2 * p.section + d]), bonus, o[d]);
-    out[d] = from_f32<T>(f * r * norm[d] * silu_f32(to_f32<T>(x[3 * p.section + d])));
+  for (int d = lane; d < p.ep; d += 32) {
+    const float f = fmaf(to_f32<T>(v[d]), bonus, o[d]);
+    out[d] = from_f32<T>(f * r * norm[d] * silu_f32(to_f32<T>(gate[d])));
   }
 }
 
@@ -227,7 +246,7 @@ __device__ __forceinline__ float transpose_sum(float (&v)[N], int lane) {
 
 // CTA = (head, sequence or span); warp w owns the state's rows (values) 16 w .. + 15. The next 64 tokens arrive while some are
 // worked on. OUT = false: only what a span adds and leaves.
-template <int DT, bool OUT>
+template <int DT, bool OUT, int KIND>
 __global__ void __launch_bounds__(MixChunk<DT>::kThreads, DT == 64 ? 2 : 1)
 time_mix_chunk_kernel(MixParams p) {
   using T = __nv_bfloat16;
@@ -249,10 +268,10 @@ time_mix_chunk_kernel(MixParams p) {
   const bool last = idx == spans - 1;
   if (slot < 0 || n <= 0 || (!OUT && last)) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const T* proj = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ld + h * p.dp;
-  float* carry = spans > 1 ? p.span.carry + (static_cast<long long>(blockIdx.y) * p.H + h) * p.dp * p.dp : nullptr;
-  const float* dec = p.dec + static_cast<long long>(row0) * p.H * p.dp + h * p.dp;
-  float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp;
+  const T* proj = static_cast<const T*>(p.proj) + static_cast<long long>(row0) * p.ld;
+  float* carry = spans > 1 ? p.span.carry + (static_cast<long long>(blockIdx.y) * p.H + h) * p.ep * p.dp : nullptr;
+  const float* dec = p.dec + static_cast<long long>(row0) * p.ld_dec + h * p.dp;
+  float* st = p.state + (static_cast<long long>(slot) * p.H + h) * p.ep * p.dp;
   const int e0 = warp * 16;
   auto issue = [&](int t0) {
     uint8_t* stage = smem + (t0 / C::kTok & 1) * C::kStage;
@@ -260,18 +279,17 @@ time_mix_chunk_kernel(MixParams p) {
     const int cnt = min(C::kTok, n - t0);
     for (int i = tid; i < C::kTok * (DT / 8); i += C::kThreads) {
       const int r = i / (DT / 8), d = (i % (DT / 8)) * 8;
-      const bool ok = r < cnt && d < p.dp;
-      const T* src = ok ? proj + static_cast<long long>(t0 + r) * p.ld + d : proj;
-      const int bytes = ok ? 16 : 0, sec = ok ? p.section : 0;
+      const bool key = r < cnt && d < p.dp, val = r < cnt && d < p.ep;
+      const T* src = proj + static_cast<long long>(r < cnt ? t0 + r : 0) * p.ld + d;
       const uint32_t at = base + (r * C::kLd + d) * 2;
-      if constexpr (OUT) cp_async_16(at + C::kR, src, bytes);
-      cp_async_16(at + C::kK, src + sec, bytes);
-      cp_async_16(at + C::kV, src + 2 * sec, bytes);
+      if constexpr (OUT) cp_async_16(at + C::kR, key ? src + h * p.dp : proj, key ? 16 : 0);
+      cp_async_16(at + C::kK, key ? src + p.off_k + h * p.dp : proj, key ? 16 : 0);
+      cp_async_16(at + C::kV, val ? src + p.off_v + h * p.ep : proj, val ? 16 : 0);
     }
     for (int i = tid; i < C::kTok * (DT / 4); i += C::kThreads) {
       const int r = i / (DT / 4), d = (i % (DT / 4)) * 4;
       const bool ok = r < cnt && d < p.dp;
-      cp_async_16(base + C::kO + (r * C::kLdO + d) * 4, ok ? dec + static_cast<long long>(t0 + r) * p.H * p.dp + d : dec, ok ? 16 : 0);
+      cp_async_16(base + C::kO + (r * C::kLdO + d) * 4, ok ? dec + (t0 + r) * p.ld_dec + d : dec, ok ? 16 : 0);
     }
     cp_commit();
   };
@@ -285,19 +303,22 @@ time_mix_chunk_kernel(MixParams p) {
       for (int e = 0; e < 2; ++e) {
         const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
         float2 v = make_float2(0.f, 0.f);
-        if (from && r < p.dp && c < p.dp) v = *reinterpret_cast<const float2*>(from + static_cast<long long>(r) * p.dp + c);
+        if (from && r < p.ep && c < p.dp) v = *reinterpret_cast<const float2*>(from + static_cast<long long>(r) * p.dp + c);
         S[j][2 * e] = v.x;
         S[j][2 * e + 1] = v.y;
       }
   }
   // this thread's share of the preparation: two channels of one block of 16 tokens
   const int blk = warp / C::kParts, part = warp % C::kParts, d0 = part * 64 + lane * 2;
+  constexpr bool kOwn = KIND == kGated;                      // token i sees its own key and value like the others
   float w0[2] = {}, uu[2] = {};
   if (d0 < p.dp) {
     w0[0] = p.w0[h * p.dp + d0];
     w0[1] = p.w0[h * p.dp + d0 + 1];
-    uu[0] = p.u[h * p.dp + d0];
-    uu[1] = p.u[h * p.dp + d0 + 1];
+    if constexpr (KIND == kTime) {
+      uu[0] = p.u[h * p.dp + d0];
+      uu[1] = p.u[h * p.dp + d0 + 1];
+    }
   }
   const uint32_t aRl = smem_u32(srl), aKl = smem_u32(skl);
   // rows of the epilogue: kLanes lanes of four columns share one
@@ -326,29 +347,37 @@ time_mix_chunk_kernel(MixParams p) {
         k[i] = *reinterpret_cast<const __nv_bfloat162*>(sk + (row + i) * C::kLd + d0);
         const float2 dv = *reinterpret_cast<const float2*>(so + (row + i) * C::kLdO + d0);
         const bool real = row + i < cnt;                     // (a token that is not there decays nothing)
-        w[i][0] = real ? expf(-__expf(dv.x + w0[0])) : 1.f;
-        w[i][1] = real ? expf(-__expf(dv.y + w0[1])) : 1.f;
+        w[i][0] = real ? decay_of<KIND, true>(dv.x + w0[0], p.inv_tau) : 1.f;
+        w[i][1] = real ? decay_of<KIND, true>(dv.y + w0[1], p.inv_tau) : 1.f;
         tot[0] *= w[i][0];
         tot[1] *= w[i][1];
-        if constexpr (OUT)
+        if constexpr (OUT && !kOwn)
           bonus[i] = fmaf(__low2float(r[i]) * uu[0], __low2float(k[i]), __high2float(r[i]) * uu[1] * __high2float(k[i]));
       }
-      float f[2] = {1.f, 1.f};
+      float f[2] = {p.r_scale, p.r_scale};
       steep = false;
       if constexpr (OUT) {
-        const float b = transpose_sum<16>(bonus, lane);
-        if (lane < 16) sbonus[part * C::kTok + row + lane] = b;
+        if constexpr (!kOwn) {
+          const float b = transpose_sum<16>(bonus, lane);
+          if (lane < 16) sbonus[part * C::kTok + row + lane] = b;
+        }
         steep = __syncthreads_or(tot[0] < kSteep || tot[1] < kSteep) != 0;
         if (!steep) {
-          f[0] = 1.f / tot[0];
-          f[1] = 1.f / tot[1];
+          f[0] /= tot[0];
+          f[1] /= tot[1];
         }
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           const int at = (row + i) * C::kLd + d0;
+          if constexpr (kOwn) {
+            f[0] *= w[i][0];
+            f[1] *= w[i][1];
+          }
           split_bf16x2(__low2float(r[i]) * f[0], __high2float(r[i]) * f[1], reinterpret_cast<uint32_t*>(sr + at), reinterpret_cast<uint32_t*>(srl + at));
-          f[0] *= w[i][0];
-          f[1] *= w[i][1];
+          if constexpr (!kOwn) {
+            f[0] *= w[i][0];
+            f[1] *= w[i][1];
+          }
         }
       }
       *reinterpret_cast<float2*>(stot + blk * DT + d0) = make_float2(tot[0], tot[1]);
@@ -369,14 +398,20 @@ time_mix_chunk_kernel(MixParams p) {
 #pragma unroll
           for (int q = 0; q < 2; ++q) {
             const int j = jj + q;
-            float x0 = __low2float(k[j]), x1 = __high2float(k[j]);
+            float x0 = __low2float(k[j]) * p.r_scale, x1 = __high2float(k[j]) * p.r_scale;
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
               v[q * 16 + i] = 0.f;
-              if (i <= j) continue;
+              if (i < j + !kOwn) continue;
+              if (kOwn && i > j) {
+                x0 *= w[i][0];
+                x1 *= w[i][1];
+              }
               v[q * 16 + i] = fmaf(__low2float(r[i]), x0, __high2float(r[i]) * x1);
-              x0 *= w[i][0];
-              x1 *= w[i][1];
+              if (!kOwn) {
+                x0 *= w[i][0];
+                x1 *= w[i][1];
+              }
             }
           }
           a[(jj + (lane >> 4)) * 16 + (lane & 15)] = transpose_sum<32>(v, lane);
@@ -411,7 +446,7 @@ time_mix_chunk_kernel(MixParams p) {
           float x[2];
 #pragma unroll
           for (int q = 0; q < 2; ++q)
-            x[q] = j * 8 + 2 * t4 + q < g + 8 * e ? c[0][j][2 * e + q] + (c[1][j][2 * e + q] + c[2][j][2 * e + q]) : 0.f;
+            x[q] = j * 8 + 2 * t4 + q < g + 8 * e + kOwn ? c[0][j][2 * e + q] + (c[1][j][2 * e + q] + c[2][j][2 * e + q]) : 0.f;
           uint32_t hi, lo;
           split_bf16x2(x[0], x[1], &hi, &lo);
           frag[(e * 4 + j) * 32 + lane] = hi;
@@ -425,7 +460,7 @@ time_mix_chunk_kernel(MixParams p) {
     for (int i = 0; i < kIter; ++i) {
       if (!OUT) break;
       const int r = min(i * C::kWarps * kPer + er, cnt - 1);
-      gate[i] = *reinterpret_cast<const uint2*>(proj + static_cast<long long>(t0 + r) * p.ld + 3 * p.section + min(ec, p.dp - 4));
+      gate[i] = *reinterpret_cast<const uint2*>(proj + static_cast<long long>(t0 + r) * p.ld + p.off_g + h * p.ep + min(ec, p.ep - 4));
     }
 #pragma unroll 1
     for (int b = 0; b < 4; ++b) {
@@ -504,25 +539,27 @@ time_mix_chunk_kernel(MixParams p) {
     if (!OUT) continue;
     // bonus, norm and gate
     float4 nm = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (ec < p.dp) nm = *reinterpret_cast<const float4*>(p.norm + h * p.dp + ec);
+    if (ec < p.ep) nm = *reinterpret_cast<const float4*>(p.norm + h * p.ep + ec);
 #pragma unroll
     for (int i = 0; i < kIter; ++i) {
       const int r = i * C::kWarps * kPer + er;
       float4 o = *reinterpret_cast<const float4*>(so + r * C::kLdO + ec);
-      float bonus = sbonus[r];
-      if (C::kParts > 1) bonus += sbonus[C::kTok + r];
-      const uint2 vv = *reinterpret_cast<const uint2*>(sv + r * C::kLd + ec);
-      const __nv_bfloat162 va = *reinterpret_cast<const __nv_bfloat162*>(&vv.x), vb = *reinterpret_cast<const __nv_bfloat162*>(&vv.y);
-      o.x = fmaf(bonus, __low2float(va), o.x); o.y = fmaf(bonus, __high2float(va), o.y);
-      o.z = fmaf(bonus, __low2float(vb), o.z); o.w = fmaf(bonus, __high2float(vb), o.w);
+      if constexpr (!kOwn) {
+        float bonus = sbonus[r];
+        if (C::kParts > 1) bonus += sbonus[C::kTok + r];
+        const uint2 vv = *reinterpret_cast<const uint2*>(sv + r * C::kLd + ec);
+        const __nv_bfloat162 va = *reinterpret_cast<const __nv_bfloat162*>(&vv.x), vb = *reinterpret_cast<const __nv_bfloat162*>(&vv.y);
+        o.x = fmaf(bonus, __low2float(va), o.x); o.y = fmaf(bonus, __high2float(va), o.y);
+        o.z = fmaf(bonus, __low2float(vb), o.z); o.w = fmaf(bonus, __high2float(vb), o.w);
+      }
       float ss = fmaf(o.x, o.x, fmaf(o.y, o.y, fmaf(o.z, o.z, o.w * o.w)));
 #pragma unroll
       for (int m = kLanes / 2; m; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
-      if (r >= cnt || ec >= p.dp) continue;
+      if (r >= cnt || ec >= p.ep) continue;
       const float rs = p.out_scale * rsqrtf(ss / static_cast<float>(p.dim) + p.eps);
       const __nv_bfloat162 ga = *reinterpret_cast<const __nv_bfloat162*>(&gate[i].x), gb = *reinterpret_cast<const __nv_bfloat162*>(&gate[i].y);
       auto silu = [](float x) { return __fdividef(x, 1.f + __expf(-x)); };
-      *reinterpret_cast<uint2*>(static_cast<T*>(p.out) + static_cast<long long>(row0 + t0 + r) * p.ldo + h * p.dp + ec) =
+      *reinterpret_cast<uint2*>(static_cast<T*>(p.out) + static_cast<long long>(row0 + t0 + r) * p.ldo + h * p.ep + ec) =
           make_uint2(pack_bf16x2(o.x * rs * nm.x * silu(__low2float(ga)), o.y * rs * nm.y * silu(__high2float(ga))),
                      pack_bf16x2(o.z * rs * nm.z * silu(__low2float(gb)), o.w * rs * nm.w * silu(__high2float(gb))));
     }
@@ -536,62 +573,65 @@ time_mix_chunk_kernel(MixParams p) {
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int r = e0 + g + 8 * e, c = j * 8 + 2 * t4;
-      if (r < p.dp && c < p.dp) *reinterpret_cast<float2*>(to + static_cast<long long>(r) * p.dp + c) = make_float2(S[j][2 * e], S[j][2 * e + 1]);
+      if (r < p.ep && c < p.dp) *reinterpret_cast<float2*>(to + static_cast<long long>(r) * p.dp + c) = make_float2(S[j][2 * e], S[j][2 * e + 1]);
     }
 }
 
 // Decoded rows: CTA = (row, head). The state is requested first, the decays are worked out while it arrives.
-template <typename T, int LPR, int PPL, int RPT>
+template <typename T, int LPR, int PPL, int RPT, int KIND>
 __global__ void __launch_bounds__(256)
 time_mix_step_kernel(MixParams p) {
   pdl_trigger();
   pdl_grid_wait();
   extern __shared__ __align__(16) float sm[];
-  float *sq = sm, *sk = sq + p.dp, *sv = sk + p.dp, *sw = sv + p.dp, *so = sw + p.dp, *th = so + p.dp, *red = th + p.rp;
+  float *sq = sm, *sk = sq + p.dp, *sw = sk + p.dp, *sv = sw + p.dp, *so = sv + p.ep, *th = so + p.ep, *red = th + p.rp;
   const int row = blockIdx.x, h = blockIdx.y, slot = p.slots[row];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(row) * p.ld + h * p.dp;
-  T* out = static_cast<T*>(p.out) + static_cast<long long>(row) * p.ldo + h * p.dp;
+  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(row) * p.ld;
+  T* out = static_cast<T*>(p.out) + static_cast<long long>(row) * p.ldo + h * p.ep;
   if (slot < 0) {
-    for (int d = tid; d < p.dp; d += 256) out[d] = from_f32<T>(0.f);
+    for (int d = tid; d < p.ep; d += 256) out[d] = from_f32<T>(0.f);
     return;
   }
-  StateStep<LPR, PPL, RPT, false> step(p.state + (static_cast<long long>(slot) * p.H + h) * p.dp * p.dp, p.dp, p.dp, p.positions[row] <= 0);
+  StateStep<LPR, PPL, RPT, KIND == kGated> step(p.state + (static_cast<long long>(slot) * p.H + h) * p.ep * p.dp, p.ep, p.dp, p.positions[row] <= 0);
   float bonus = 0.f;
   for (int d = tid; d < p.dp; d += 256) {
-    sq[d] = to_f32<T>(x[d]);
-    sk[d] = to_f32<T>(x[p.section + d]);
-    sv[d] = to_f32<T>(x[2 * p.section + d]);
-    bonus = fmaf(p.u[h * p.dp + d] * sk[d], sq[d], bonus);
+    sq[d] = p.r_scale * to_f32<T>(x[h * p.dp + d]);
+    sk[d] = to_f32<T>(x[p.off_k + h * p.dp + d]);
+    if constexpr (KIND == kTime) bonus = fmaf(p.u[h * p.dp + d] * sk[d], sq[d], bonus);
+    else sw[d] = decay_of<KIND>(p.dec[row * p.ld_dec + h * p.dp + d] + p.w0[h * p.dp + d], p.inv_tau);
   }
-  const T* wl = static_cast<const T*>(p.proj) + static_cast<long long>(row) * p.ld + 4 * p.section;
-  for (int j = tid; j < p.rp; j += 256) th[j] = to_f32<T>(from_f32<T>(tanhf(to_f32<T>(wl[j]))));
-  bonus = warp_sum(bonus);
-  if (lane == 0) red[warp] = bonus;
-  __syncthreads();
-  // four lanes per channel, 16 bytes of its row of the matrix at a time
-  constexpr int V = kVec16<T>;
-  const T* w2 = static_cast<const T*>(p.w2) + static_cast<long long>(h) * p.dp * p.rp;
-  for (int d = tid >> 2; d < p.dp; d += 64) {              // (dp is a multiple of 16: a warp's eight channels exist or do not)
-    float a = 0.f;
-    for (int j = (tid & 3) * V; j < p.rp; j += 4 * V) {
-      float f[V];
-      ld16<T>(w2 + static_cast<long long>(d) * p.rp + j, f);
+  for (int e = tid; e < p.ep; e += 256) sv[e] = to_f32<T>(x[p.off_v + h * p.ep + e]);
+  if constexpr (KIND == kTime) {
+    const T* wl = x + p.off_low;
+    for (int j = tid; j < p.rp; j += 256) th[j] = to_f32<T>(from_f32<T>(tanhf(to_f32<T>(wl[j]))));
+    bonus = warp_sum(bonus);
+    if (lane == 0) red[warp] = bonus;
+    __syncthreads();
+    // four lanes per channel, 16 bytes of its row of the matrix at a time
+    constexpr int V = kVec16<T>;
+    const T* w2 = static_cast<const T*>(p.w2) + static_cast<long long>(h) * p.dp * p.rp;
+    for (int d = tid >> 2; d < p.dp; d += 64) {            // (dp is a multiple of 16: a warp's eight channels exist or do not)
+      float a = 0.f;
+      for (int j = (tid & 3) * V; j < p.rp; j += 4 * V) {
+        float f[V];
+        ld16<T>(w2 + static_cast<long long>(d) * p.rp + j, f);
 #pragma unroll
-      for (int i = 0; i < V; ++i) a = fmaf(f[i], th[j + i], a);
+        for (int i = 0; i < V; ++i) a = fmaf(f[i], th[j + i], a);
+      }
+      a += __shfl_xor_sync(0xffffffffu, a, 1);
+      a += __shfl_xor_sync(0xffffffffu, a, 2);
+      if ((tid & 3) == 0) sw[d] = decay_of<KIND>(a + p.w0[h * p.dp + d], 1.f);
     }
-    a += __shfl_xor_sync(0xffffffffu, a, 1);
-    a += __shfl_xor_sync(0xffffffffu, a, 2);
-    if ((tid & 3) == 0) sw[d] = expf(-expf(a + p.w0[h * p.dp + d]));
-  }
-  bonus = 0.f;
+    bonus = 0.f;
 #pragma unroll
-  for (int w = 0; w < 8; ++w) bonus += red[w];
+    for (int w = 0; w < 8; ++w) bonus += red[w];
+  }
   __syncthreads();
   step.run(sq, sk, sw, sv, so);
   __syncthreads();
   float ss = 0.f;
-  for (int d = tid; d < p.dp; d += 256) {
+  for (int d = tid; d < p.ep; d += 256) {
     const float f = fmaf(sv[d], bonus, so[d]);
     ss = fmaf(f, f, ss);
   }
@@ -602,25 +642,25 @@ time_mix_step_kernel(MixParams p) {
 #pragma unroll
   for (int w = 0; w < 8; ++w) ss += red[w];
   const float r = p.out_scale / sqrtf(ss / static_cast<float>(p.dim) + p.eps);
-  for (int d = tid; d < p.dp; d += 256)
-    out[d] = from_f32<T>(fmaf(sv[d], bonus, so[d]) * r * p.norm[h * p.dp + d] * silu_f32(to_f32<T>(x[3 * p.section + d])));
+  for (int d = tid; d < p.ep; d += 256)
+    out[d] = from_f32<T>(fmaf(sv[d], bonus, so[d]) * r * p.norm[h * p.ep + d] * silu_f32(to_f32<T>(x[p.off_g + h * p.ep + d])));
 }
 
-template <typename T>
+template <typename T, int KIND>
 int run_scan(const MixParams& p, cudaStream_t s) {
-  const dim3 grid((p.dp + kScanRows - 1) / kScanRows, p.H, p.n_seq);
+  const dim3 grid((p.ep + kScanRows - 1) / kScanRows, p.H, p.n_seq);
   const bool pdl = pdl_all_enabled();
-  if (p.dp <= 64) launch_pdl(time_mix_scan_kernel<T, 2>, grid, dim3(128), 0, s, pdl, p);
-  else if (p.dp <= 128) launch_pdl(time_mix_scan_kernel<T, 4>, grid, dim3(128), 0, s, pdl, p);
-  else launch_pdl(time_mix_scan_kernel<T, 8>, grid, dim3(128), 0, s, pdl, p);
+  if (p.dp <= 64) launch_pdl(time_mix_scan_kernel<T, 2, KIND>, grid, dim3(128), 0, s, pdl, p);
+  else if (p.dp <= 128) launch_pdl(time_mix_scan_kernel<T, 4, KIND>, grid, dim3(128), 0, s, pdl, p);
+  else launch_pdl(time_mix_scan_kernel<T, 8, KIND>, grid, dim3(128), 0, s, pdl, p);
   const long long warps = static_cast<long long>(p.rows) * p.H;
-  launch_pdl(time_mix_norm_kernel<T>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, s, pdl, p);
+  launch_pdl(time_mix_norm_kernel<T, KIND>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, s, pdl, p);
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int DT, bool OUT>
+template <int DT, bool OUT, int KIND>
 int launch_chunk(const MixParams& p, cudaStream_t s) {
-  auto kern = time_mix_chunk_kernel<DT, OUT>;
+  auto kern = time_mix_chunk_kernel<DT, OUT, KIND>;
   static PerDeviceFlag attr;
   if (attr.unset()) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, MixChunk<DT>::kSmem);
@@ -631,33 +671,39 @@ int launch_chunk(const MixParams& p, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int DT>
+template <int DT, int KIND>
 int run_chunk(const MixParams& p, cudaStream_t s) {
   if (p.span.seq) {
-    if (const int rc = launch_chunk<DT, false>(p, s)) return rc;
-    launch_pdl(state_carry_kernel, dim3((p.dp * p.dp / 4 + 255) / 256, p.H, p.n_seq), dim3(256), 0, s, pdl_all_enabled(), p.span,
-               static_cast<const float*>(p.state), p.slots, p.pos0, p.dp, p.dp, 1);
+    if (const int rc = launch_chunk<DT, false, KIND>(p, s)) return rc;
+    launch_pdl(state_carry_kernel, dim3((p.ep * p.dp / 4 + 255) / 256, p.H, p.n_seq), dim3(256), 0, s, pdl_all_enabled(), p.span,
+               static_cast<const float*>(p.state), p.slots, p.pos0, p.ep, p.dp, 1);
   }
-  return launch_chunk<DT, true>(p, s);
+  return launch_chunk<DT, true, KIND>(p, s);
 }
 
-template <typename T>
+template <typename T, int KIND>
 int run_step(const MixParams& p, cudaStream_t s) {
-  const int smem = (5 * p.dp + p.rp + 8) * 4;
+  const int smem = (3 * p.dp + 2 * p.ep + p.rp + 8) * 4;
   if (smem > 48 * 1024) return -2;
   const dim3 grid(p.rows, p.H);
   const bool pdl = pdl_all_enabled();
-  if (p.dp <= 32) launch_pdl(time_mix_step_kernel<T, 8, 1, 1>, grid, dim3(256), smem, s, pdl, p);
-  else if (p.dp <= 64) launch_pdl(time_mix_step_kernel<T, 16, 1, 4>, grid, dim3(256), smem, s, pdl, p);
-  else if (p.dp <= 128) launch_pdl(time_mix_step_kernel<T, 32, 1, 16>, grid, dim3(256), smem, s, pdl, p);
-  else launch_pdl(time_mix_step_kernel<T, 32, 2, 8>, grid, dim3(256), smem, s, pdl, p);
+  if (p.dp <= 32) launch_pdl(time_mix_step_kernel<T, 8, 1, 1, KIND>, grid, dim3(256), smem, s, pdl, p);
+  else if (p.dp <= 64) launch_pdl(time_mix_step_kernel<T, 16, 1, 4, KIND>, grid, dim3(256), smem, s, pdl, p);
+  else if (p.dp <= 128) launch_pdl(time_mix_step_kernel<T, 32, 1, 16, KIND>, grid, dim3(256), smem, s, pdl, p);
+  else launch_pdl(time_mix_step_kernel<T, 32, 2, 8, KIND>, grid, dim3(256), smem, s, pdl, p);
   return static_cast<int>(cudaGetLastError());
 }
 
-bool read_mix(const int* v, MixParams* p) {
-  p->H = v[0]; p->dim = v[1]; p->dp = v[2]; p->rp = v[3]; p->section = v[4]; p->rows = v[5]; p->n_seq = v[6]; p->ld = v[7]; p->ldo = v[8];
-  return p->H > 0 && p->H <= 65535 && p->dim > 0 && p->dp >= p->dim && p->dp % 16 == 0 && p->dp <= 256 && p->rp > 0 && p->rp % 16 == 0 &&
-         p->section >= p->H * p->dp && p->section % 8 == 0 && p->rows > 0 && p->ld % 8 == 0 && p->n_seq > 0 && p->n_seq <= 65535;
+// ints: H, dim, dp, ep, rp, off_k, off_v, off_g, off_low, rows, sequences, row strides of the projection, the result and the decays, kind
+// (0 time mixing, 1 gated linear attention); floats: eps, out_scale, r_scale, 1 / tau
+bool read_mix(const int* v, const float* f, MixParams* p, int* kind) {
+  p->H = v[0]; p->dim = v[1]; p->dp = v[2]; p->ep = v[3]; p->rp = v[4]; p->off_k = v[5]; p->off_v = v[6]; p->off_g = v[7]; p->off_low = v[8];
+  p->rows = v[9]; p->n_seq = v[10]; p->ld = v[11]; p->ldo = v[12]; p->ld_dec = v[13];
+  *kind = v[14];
+  p->eps = f[0]; p->out_scale = f[1]; p->r_scale = f[2]; p->inv_tau = f[3];
+  return p->H > 0 && p->H <= 65535 && p->dim > 0 && p->ep >= p->dim && p->ep % 16 == 0 && p->dp > 0 && p->dp % 16 == 0 && p->dp <= 256 && p->rp >= 0 &&
+         p->rp % 16 == 0 && p->off_k % 8 == 0 && p->off_v % 8 == 0 && p->off_g % 8 == 0 && p->off_low % 8 == 0 && p->rows > 0 && p->ld % 8 == 0 &&
+         p->ld_dec % 4 == 0 && p->n_seq > 0 && p->n_seq <= 65535 && (*kind == kTime || *kind == kGated);
 }
 
 template <typename T, int N>
@@ -713,42 +759,47 @@ TSB_EXPORT int tsb_tanh_rows(const void* x, long long ld, void* out, int rows, i
   return static_cast<int>(cudaGetLastError());
 }
 
-// ints: H, dim, dp, rp, section, rows, sequences, projection row stride, result row stride. ptrs: proj, w2, w0, u, norm, state,
-// slots, positions, out. Row i is the next token of the sequence in slot slots[i] (-1: padding, out = 0).
-TSB_EXPORT int tsb_time_mix_step(const int* ints, void* const* q, float eps, float out_scale, int dtype, void* stream) {
+// ints and floats: see read_mix. ptrs: proj, w2, w0, u, norm, state, slots, positions, out, dec (time mixing: w2 and u, gated: dec). Row i is
+// the next token of the sequence in slot slots[i] (-1: padding, out = 0).
+TSB_EXPORT int tsb_time_mix_step(const int* ints, const float* floats, void* const* q, int dtype, void* stream) {
   using namespace tsb;
   MixParams p{};
-  if (!read_mix(ints, &p)) return -2;
+  int kind;
+  if (!read_mix(ints, floats, &p, &kind)) return -2;
   p.proj = q[0]; p.w2 = q[1]; p.w0 = static_cast<const float*>(q[2]); p.u = static_cast<const float*>(q[3]);
   p.norm = static_cast<const float*>(q[4]); p.state = static_cast<float*>(q[5]); p.slots = static_cast<const int*>(q[6]);
-  p.positions = static_cast<const int*>(q[7]); p.out = q[8]; p.eps = eps; p.out_scale = out_scale;
+  p.positions = static_cast<const int*>(q[7]); p.out = q[8]; p.dec = static_cast<const float*>(q[9]);
+  if (kind == kTime ? (!p.w2 || !p.u || p.rp <= 0) : !p.dec) return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == 1) return run_step<__nv_bfloat16>(p, s);
-  if (dtype == 0) return run_step<float>(p, s);
+  if (dtype == 1) return kind == kTime ? run_step<__nv_bfloat16, kTime>(p, s) : run_step<__nv_bfloat16, kGated>(p, s);
+  if (dtype == 0) return kind == kTime ? run_step<float, kTime>(p, s) : run_step<float, kGated>(p, s);
   return -2;
 }
 
-// ptrs: proj, dec, w0, u, norm, state, slots, cu, pos0, out, o ([rows, H, dp] fp32; null: bf16 on the tensor cores, dp <= 128), and for
+// ptrs: proj, dec, w0, u, norm, state, slots, cu, pos0, out, o ([rows, H, ep] fp32; null: bf16 on the tensor cores, dp and ep <= 128), and for
 // `spans` spans of 512 tokens (0: every portion is walked in one): their sequences, the first span of every sequence, carry [spans, H,
-// dp, dp], left [spans, H, dp].
-TSB_EXPORT int tsb_time_mix_prefill(const int* ints, void* const* q, int spans, float eps, float out_scale, int dtype, void* stream) {
+// ep, dp], left [spans, H, dp].
+TSB_EXPORT int tsb_time_mix_prefill(const int* ints, const float* floats, void* const* q, int spans, int dtype, void* stream) {
   using namespace tsb;
   MixParams p{};
-  if (!read_mix(ints, &p)) return -2;
+  int kind;
+  if (!read_mix(ints, floats, &p, &kind)) return -2;
   p.proj = q[0]; p.dec = static_cast<const float*>(q[1]); p.w0 = static_cast<const float*>(q[2]); p.u = static_cast<const float*>(q[3]);
   p.norm = static_cast<const float*>(q[4]); p.state = static_cast<float*>(q[5]); p.slots = static_cast<const int*>(q[6]);
   p.cu = static_cast<const int*>(q[7]); p.pos0 = static_cast<const int*>(q[8]); p.out = q[9]; p.o = static_cast<float*>(q[10]);
-  p.eps = eps; p.out_scale = out_scale;
+  if (!p.dec || (kind == kTime && !p.u)) return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (!p.o) {
     if (spans > 0) {
       p.span = {static_cast<const int*>(q[11]), static_cast<const int*>(q[12]), static_cast<float*>(q[13]), static_cast<float*>(q[14]), spans};
       if (spans > 65535 || !p.span.seq || !p.span.first || !p.span.carry || !p.span.left) return -2;
     }
-    if (dtype != 1 || p.dp > 128 || p.ldo % 4 || (reinterpret_cast<uintptr_t>(p.out) & 7)) return -2;
-    return p.dp <= 64 ? run_chunk<64>(p, s) : run_chunk<128>(p, s);
+    const int wide = std::max(p.dp, p.ep);
+    if (dtype != 1 || wide > 128 || p.ldo % 4 || (reinterpret_cast<uintptr_t>(p.out) & 7)) return -2;
+    if (kind == kTime) return wide <= 64 ? run_chunk<64, kTime>(p, s) : run_chunk<128, kTime>(p, s);
+    return wide <= 64 ? run_chunk<64, kGated>(p, s) : run_chunk<128, kGated>(p, s);
   }
-  if (dtype == 1) return run_scan<__nv_bfloat16>(p, s);
-  if (dtype == 0) return run_scan<float>(p, s);
+  if (dtype == 1) return kind == kTime ? run_scan<__nv_bfloat16, kTime>(p, s) : run_scan<__nv_bfloat16, kGated>(p, s);
+  if (dtype == 0) return kind == kTime ? run_scan<float, kTime>(p, s) : run_scan<float, kGated>(p, s);
   return -2;
 }

@@ -1,4 +1,4 @@
-from . import fozelix, polosun, vobotar
+from . import fozelix, polosun, tonilix, vobotar
 from .hybrid import HybridConfig, HybridModel
 from .llama import GenerateConfig, LlamaConfig, LlamaModel, llama_local_to_hf_name
 from .registry import architectures, load_config, load_model, load_pretrained

@@ -1,5 +1,5 @@
 """Decoders that mix recurrent and attention layers, described by a list: every layer has a mixer and, optionally, a
-feed-forward. Three forms of layer:
+feed-forward. Four forms of layer:
 
 * ``sandwich``: mixer, then feed-forward, each normed before and after by Dynamic Tanh; a range of layers may run several
   times in a row with the same weights and separate caches ("loop");
@@ -8,7 +8,10 @@ feed-forward. Three forms of layer:
   both results back. Optionally every layer hands on a weighted sum of the embedding output and all layers' results so far
   ("depth average");
 * ``post``: mixer, then feed-forward, which read x itself; their results are normed by RMS (gains stored around zero) and added.
-  Optionally every layer then adds a normed side input that depends on the token ("token side").
+  Optionally every layer then adds a normed side input that depends on the token ("token side");
+* ``pre``: mixer, then feed-forward, each of its own norm of x, an RMS norm in equal parts of the row. Optionally a scale per channel on
+  what they add ("layer scale"), a mixer input that is mixed with the one of the token before ("token shift"), and a sinusoid of the
+  position and a norm at the embedding.
 
 Embedding and output share one table, or the output has its own.
 
@@ -24,10 +27,12 @@ from typing import Callable, Dict, List, Optional, Union
 import torch
 
 from .. import ops
-from ..nn.hybrid import (RGLRU, SSD, ChunkedAttention, ClampedGLU, DynamicTanh, GatedDelta, LatentAttention, Retention, RMSNorm,
-                         ScalarRMSNorm, ShapedAttention, SideBySide, SiluGLU, TimeMix, TokenSide, pad_to)
-from ..nn.ragged import HybridCache, HybridSequence, RaggedBatch
+from ..nn.hybrid import (RGLRU, SSD, ChunkedAttention, ClampedGLU, DynamicTanh, ExpertMLP, GatedDelta, GatedLinear, GeluGLU, LatentAttention,
+                         PartRMSNorm, Retention, RMSNorm, ScalarRMSNorm, ShapedAttention, SideBySide, SiluGLU, TimeMix, TokenSide, pad_to)
+from ..nn.ragged import HybridCache, HybridSequence, PairRun, RaggedBatch, StateRun
 from ..ops.masks import Window
+from ..ops.moe import Choice
+from ..ops.pre_norm import Shift, sinusoid_frequencies
 from ..ops.ragged import ScoreForm
 from ..ops.rotary import Rotary, Yarn
 from .llama import GenerateConfig, pick_next_token
@@ -45,11 +50,14 @@ class AttentionSpec:
 
 @dataclass(frozen=True)
 class DeltaSpec:
+    """``decay_rank`` and ``gate_rank`` (both or neither): a decay per key channel, which like the gate is a product of that rank."""
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     conv: int
+    decay_rank: int = 0
+    gate_rank: int = 0
 
 
 @dataclass(frozen=True)
@@ -84,7 +92,8 @@ class ShapedAttentionSpec:
     """Attention with chosen parts. ``window`` 0: causal; ``norm`` of q and k: "", "unit" (per head), "head" (per head with a
     weight), "whole" (all heads at once with a weight); ``distance_bias``: 2^(-8 (h + 1) / heads) per position; ``sink``: "",
     "learned", "one" (1 more in the denominator); ``gate``: "", "head", "element"; ``v_mix``: values mixed with those of the model's
-    first such layer."""
+    first such layer; ``q_temp`` (coef, every): queries times 1 + coef ln(floor((position + 1) / every) + 1); ``out_bias``: a bias on the
+    output product."""
     heads: int
     kv_heads: int
     dim: int
@@ -100,12 +109,23 @@ class ShapedAttentionSpec:
     sink: str = ""
     gate: str = ""
     v_mix: bool = False
+    q_temp: Optional[tuple] = None
+    out_bias: bool = False
 
 
 @dataclass(frozen=True)
 class TimeMixSpec:
     heads: int
     dim: int
+    rank: int
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
     rank: int
 
 
@@ -139,9 +159,22 @@ class SiluGLUSpec:
 
 
 @dataclass(frozen=True)
+class GeluGLUSpec:
+    ff: int
+
+
+@dataclass(frozen=True)
+class ExpertSpec:
+    """Squared-ReLU experts of ``ff`` channels."""
+    ff: int
+    choice: Choice
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, DeltaSpec, LatentSpec, RetentionSpec, RGLRUSpec, ShapedAttentionSpec, TimeMixSpec, SSDSpec, SideBySideSpec]
-    mlp: Union[GLUSpec, SiluGLUSpec, None] = None
+    mixer: Union[AttentionSpec, DeltaSpec, LatentSpec, RetentionSpec, RGLRUSpec, ShapedAttentionSpec, TimeMixSpec, GatedLinearSpec, SSDSpec,
+                 SideBySideSpec]
+    mlp: Union[GLUSpec, SiluGLUSpec, GeluGLUSpec, ExpertSpec, None] = None
 
 
 @dataclass(frozen=True)
@@ -164,11 +197,16 @@ class HybridConfig:
     eos_token_id: int = -1
     max_position_embeddings: int = 1 << 20     # a bound for caches only
     architecture: str = ""
-    form: str = "sandwich"                     # or "parallel" or "post"
+    form: str = "sandwich"                     # or "parallel", "post" or "pre"
     residual_mult: float = 1.0                 # (parallel)
     depth_average: bool = False                # (parallel)
     tied: bool = True                          # the output product uses the embedding table
     token_side: int = 0                        # (post) columns of the side table per layer, 0: no side input
+    norm_parts: int = 1                        # (pre)
+    layer_scale: bool = False                  # (pre)
+    token_shift: bool = False                  # (pre)
+    sinusoid: bool = False                     # (pre) positions are added to the embedding
+    embed_norm: bool = False                   # (pre)
 
     def __post_init__(self):
         if self.vocab_size < 1 or self.width < 1 or not self.layers:
@@ -178,10 +216,17 @@ class HybridConfig:
             raise ValueError("HybridConfig: loop must name a range of layers and run at least once")
         if self.dtype not in (torch.bfloat16, torch.float32):
             raise ValueError("HybridConfig: dtype is bfloat16 or float32")
-        if self.form not in ("sandwich", "parallel", "post"):
+        if self.form not in ("sandwich", "parallel", "post", "pre"):
             raise ValueError(f"HybridConfig: unknown form {self.form!r}")
-        if self.form == "post" and lp is not None:
-            raise ValueError("HybridConfig: post-normed layers take no loop")
+        if self.form in ("post", "pre") and lp is not None:
+            raise ValueError(f"HybridConfig: {self.form}-normed layers take no loop")
+        if self.form == "pre" and self.embedding_scale != 1.0:
+            raise ValueError("HybridConfig: pre-normed layers take no embedding scale")
+        if self.form != "pre" and (self.norm_parts != 1 or self.layer_scale or self.token_shift or self.sinusoid or self.embed_norm):
+            raise ValueError("HybridConfig: norms in parts, layer scales, a token shift, a sinusoid and a norm of the embedding belong to "
+                             "pre-normed layers")
+        if self.form != "pre" and any(isinstance(l.mlp, ExpertSpec) for l in self.layers):
+            raise ValueError("HybridConfig: mixtures of experts run in pre-normed layers")
         if self.form != "post" and self.token_side or self.token_side < 0:
             raise ValueError("HybridConfig: a side input per token belongs to post-normed layers")
         if self.form == "parallel" and (lp is not None or self.embedding_scale != 1.0):
@@ -214,7 +259,9 @@ def _make_mixer(m, c: HybridConfig, device):
         slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / m.heads) for h in range(m.heads)]) if m.distance_bias else None
         form = ScoreForm(m.scale, Window(m.window) if m.window else 0, m.softcap, slopes, torch.zeros(m.heads) if m.sink == "one" else None)
         return ShapedAttention(W, m.heads, m.kv_heads, m.dim, m.vdim, form, c.eps, dt, device, m.bias, m.keys_as_values, m.norm, m.rotary,
-                               m.sink == "learned", m.v_mix, m.gate)
+                               m.sink == "learned", m.v_mix, m.gate, m.q_temp, m.out_bias)
+    if isinstance(m, GatedLinearSpec):
+        return GatedLinear(W, m.heads, m.dim, m.vdim, m.rank, m.tau, c.eps, dt, device)
     if isinstance(m, TimeMixSpec):
         return TimeMix(W, m.heads, m.dim, m.rank, c.eps, dt, device)
     if isinstance(m, SSDSpec):
@@ -222,7 +269,7 @@ def _make_mixer(m, c: HybridConfig, device):
     if isinstance(m, AttentionSpec):
         return ChunkedAttention(W, m.heads, m.kv_heads, m.dim, m.vdim, m.scale, m.chunk, dt, device)
     if isinstance(m, DeltaSpec):
-        return GatedDelta(W, m.heads, m.kv_heads, m.dim, m.vdim, m.conv, c.eps, dt, device)
+        return GatedDelta(W, m.heads, m.kv_heads, m.dim, m.vdim, m.conv, c.eps, dt, device, m.decay_rank, m.gate_rank)
     if isinstance(m, LatentSpec):
         return LatentAttention(W, m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.scale, m.rotary, c.eps, dt, device)
     if isinstance(m, RetentionSpec):
@@ -237,10 +284,21 @@ def _make_mlp(m, c: HybridConfig, device):
         return None
     if isinstance(m, SiluGLUSpec):
         return SiluGLU(c.width, m.ff, c.dtype, device)
+    if isinstance(m, GeluGLUSpec):
+        return GeluGLU(c.width, m.ff, c.dtype, device)
+    if isinstance(m, ExpertSpec):
+        return ExpertMLP(c.width, m.ff, m.choice, c.dtype, device)
     return ClampedGLU(c.width, m.ff, m.limit, c.dtype, device)
 
 
-class _SandwichLayer:
+class _Layer:
+    extra: dict = {}                  # vectors of the layer itself: name -> tensor
+
+    def run_spec(self):
+        return self.mixer.run_spec()
+
+
+class _SandwichLayer(_Layer):
     def __init__(self, spec: LayerSpec, c: HybridConfig, index: int, device):
         norm = lambda: DynamicTanh(c.width, c.dtype, device)   # noqa: E731
         self.mixer, self.mlp = _make_mixer(spec.mixer, c, device), _make_mlp(spec.mlp, c, device)
@@ -253,10 +311,8 @@ class _SandwichLayer:
             out += [("norm2", self.norm2), ("norm2b", self.norm2b), ("mlp.", self.mlp)]
         return out
 
-    extra = {}
 
-
-class _ParallelLayer:
+class _ParallelLayer(_Layer):
     """One input matrix (rows of the mixer, then of the feed-forward) and one output matrix (columns likewise)."""
 
     def __init__(self, spec: LayerSpec, c: HybridConfig, index: int, device):
@@ -301,7 +357,7 @@ class _ParallelLayer:
         return ops.project(z, self.w_out)
 
 
-class _PostLayer:
+class _PostLayer(_Layer):
     def __init__(self, spec: LayerSpec, c: HybridConfig, index: int, device):
         norm = lambda: RMSNorm(c.width, c.eps, 1.0, c.dtype, device)   # noqa: E731
         self.mixer, self.mlp = _make_mixer(spec.mixer, c, device), _make_mlp(spec.mlp, c, device)
@@ -319,10 +375,34 @@ class _PostLayer:
             out.append(("side.", self.side))
         return out
 
-    extra = {}
+
+class _PreLayer(_Layer):
+    def __init__(self, spec: LayerSpec, c: HybridConfig, index: int, device):
+        norm = lambda: PartRMSNorm(c.width, c.norm_parts, c.eps, c.dtype, device)   # noqa: E731
+        vec = lambda on: torch.zeros(c.width, dtype=torch.float32, device=device) if on else None   # noqa: E731
+        self.mixer, self.mlp = _make_mixer(spec.mixer, c, device), _make_mlp(spec.mlp, c, device)
+        self.norm1, self.norm2 = norm(), norm() if spec.mlp is not None else None
+        self.ls1, self.ls2, self.shift = vec(c.layer_scale), vec(c.layer_scale and spec.mlp is not None), vec(c.token_shift)
+        self.extra = {n: t for n, t in (("ls1", self.ls1), ("ls2", self.ls2), ("shift", self.shift)) if t is not None}
+        self.width = c.width
+
+    def parts(self):
+        out = [("norm1", self.norm1), ("mix.", self.mixer)]
+        if self.mlp is not None:
+            out += [("norm2", self.norm2), ("mlp.", self.mlp)]
+        return out
+
+    def run_spec(self):
+        """With a token shift: the mixer's storage, and the last input of every sequence."""
+        spec = self.mixer.run_spec()
+        return PairRun(spec, StateRun((self.width,))) if self.shift is not None else spec
+
+    def storage(self, run):
+        """(the mixer's storage, what the norm takes for the shift)"""
+        return (run[0], Shift(self.shift, run[1][0])) if self.shift is not None else (run, None)
 
 
-_LAYERS = {"sandwich": _SandwichLayer, "parallel": _ParallelLayer, "post": _PostLayer}
+_LAYERS = {"sandwich": _SandwichLayer, "parallel": _ParallelLayer, "post": _PostLayer, "pre": _PreLayer}
 
 
 class HybridModel:
@@ -338,8 +418,11 @@ class HybridModel:
             raise ValueError("HybridConfig: layers that mix values have the same value heads")
         self.layers = [_LAYERS[c.form](s, c, i, self.device) for i, s in enumerate(c.layers)]
         final = {"sandwich": lambda: DynamicTanh(c.width, c.dtype, self.device), "parallel": lambda: ScalarRMSNorm(c.eps, c.dtype, self.device),
-                 "post": lambda: RMSNorm(c.width, c.eps, 1.0, c.dtype, self.device)}
+                 "post": lambda: RMSNorm(c.width, c.eps, 1.0, c.dtype, self.device),
+                 "pre": lambda: PartRMSNorm(c.width, c.norm_parts, c.eps, c.dtype, self.device)}
         self.final_norm = final[c.form]()
+        self.embed_norm = final["pre"]() if c.embed_norm else None
+        self.frequencies = sinusoid_frequencies(c.width).to(self.device) if c.sinusoid else None
         self.side_table = (torch.zeros(c.vocab_size, c.token_side * len(c.layers), dtype=c.dtype, device=self.device)
                            if c.token_side else None)
         self.loop_step = (torch.zeros(c.loop.times, c.width, dtype=torch.float32, device=self.device)
@@ -376,6 +459,8 @@ class HybridModel:
         for i, l in enumerate(self.layers):
             for name, part in l.parts():
                 yield f"l{i}.{name}", part
+        if self.embed_norm is not None:
+            yield "embed.norm", self.embed_norm
         yield "final.norm", self.final_norm
 
     def _tables(self):
@@ -451,8 +536,10 @@ class HybridModel:
                 return torch.tensor(0.5)
             if last == "alpha" or shape == ():
                 return torch.tensor(1.0)
-            if ".mu." in name:
+            if ".mu." in name or last == "shift":
                 return torch.rand(shape, generator=gen, device=self.device)
+            if last == "correction":
+                return 0.05 * torch.randn(shape, generator=gen, device=self.device)
             if last == "w0":
                 return torch.rand(shape, generator=gen, device=self.device) * 5.0 - 6.0
             if last == "u":
@@ -478,7 +565,7 @@ class HybridModel:
     # ------------------------------------------------------------------ the step
     def make_cache(self, num_blocks: int, block_size: int, max_sequences: int, max_len: int) -> HybridCache:
         """K / V pages and recurrent slots of every layer run (a looped layer has one store per pass)."""
-        specs = [self.layers[i].mixer.run_spec() for i, _ in self.runs]
+        specs = [self.layers[i].run_spec() for i, _ in self.runs]
         return HybridCache(specs, num_blocks, block_size, max_sequences, max_len, self.config.dtype, self.device)
 
     def make_batch(self, cache: HybridCache, entries, want=None, max_len: int = 0) -> RaggedBatch:
@@ -488,7 +575,7 @@ class HybridModel:
     def forward_ragged(self, batch, cache: HybridCache, on_layer: Optional[Callable] = None) -> Optional[torch.Tensor]:
         """Runs one step over the cache; fp32 logits [wanted rows, vocab] (None when nothing is wanted). ``on_layer`` is
         called with (run, residual) after every layer run, before what comes ahead of the next pass."""
-        run = {"sandwich": self._run_sandwich, "parallel": self._run_parallel, "post": self._run_post}[self.config.form]
+        run = {"sandwich": self._run_sandwich, "parallel": self._run_parallel, "post": self._run_post, "pre": self._run_pre}[self.config.form]
         h = run(batch, cache, on_layer)
         if batch.n_want == 0:
             return None
@@ -570,6 +657,30 @@ class HybridModel:
                 on_layer(r, x)
         return h
 
+    def _run_pre(self, batch, cache: HybridCache, on_layer) -> torch.Tensor:
+        c = self.config
+        x = moved = None
+
+        def step(norm, shift=None, **kw):
+            nonlocal x, moved
+            x, h, moved = ops.pre_norm_step(batch, c.width, norm.gain, c.norm_parts, c.eps, x, shift=shift, moved=moved, out_cols=pad_to(c.width),
+                                            out_dtype=c.dtype, **kw)
+            return h
+
+        kept = [l.storage(run) for l, run in zip(self.layers, cache.runs)]
+        h = step(self.layers[0].norm1, kept[0][1], table=self.embed, freq=self.frequencies,
+                 embed_gain=self.embed_norm.gain if self.embed_norm is not None else None)
+        for r, l in enumerate(self.layers):
+            add = dict(y=l.mixer.forward(h, kept[r][0], batch), bias=l.mixer.out_bias, scale=l.ls1)
+            if l.mlp is not None:
+                h = step(l.norm2, **add)
+                add = dict(y=l.mlp.forward(h), bias=l.mlp.out_bias, scale=l.ls2)
+            last = r == len(self.layers) - 1
+            h = step(self.final_norm if last else self.layers[r + 1].norm1, None if last else kept[r + 1][1], **add)
+            if on_layer is not None:
+                on_layer(r, x)
+        return h
+
     # ------------------------------------------------------------------ interface of the per-request schedulers
     def make_layer_pools(self, num_blocks: int, block_size: int, max_sequences: int = 16, max_len: int = 0) -> list:
         return [self.make_cache(num_blocks, block_size, max_sequences, max_len or num_blocks * block_size)]
@@ -631,6 +742,6 @@ class HybridModel:
         return eng.result(rid)
 
 
-__all__ = ["AttentionSpec", "DeltaSpec", "GLUSpec", "HybridConfig", "HybridModel", "LatentSpec", "LayerSpec", "LoopSpec", "RGLRUSpec",
+__all__ = ["AttentionSpec", "Choice", "DeltaSpec", "ExpertSpec", "GLUSpec", "GatedLinearSpec", "GeluGLUSpec", "HybridConfig", "HybridModel", "LatentSpec", "LayerSpec", "LoopSpec", "RGLRUSpec",
            "RetentionSpec", "Rotary", "SSDSpec", "ShapedAttentionSpec", "SideBySideSpec", "SiluGLUSpec", "TimeMixSpec", "Yarn",
            "pick_next_token"]

@@ -129,6 +129,16 @@ def _vobotar_build(cfg, device):
     return vobotar.build(cfg, device)
 
 
+def _tonilix_config(obj: dict, dtype: torch.dtype, shapes=None):
+    from . import tonilix
+    return tonilix.config_from_dict(obj, dtype, shapes)
+
+
+def _tonilix_build(cfg, device):
+    from . import tonilix
+    return tonilix.build(cfg, device)
+
+
 register(Architecture("Llama", _is_llama, _llama_config, _llama_build))
 register(Architecture("Fozelix", lambda o: o.get("architecture") == "Fozelix", _fozelix_config, _fozelix_build,
                       kernels="fozelix"))
@@ -136,3 +146,5 @@ register(Architecture("Polosun", lambda o: o.get("architecture") == "Polosun", _
                       kernels="polosun"))
 register(Architecture("Vobotar", lambda o: o.get("architecture") == "Vobotar", _vobotar_config, _vobotar_build,
                       kernels="vobotar", shapes=True))
+register(Architecture("Tonilix", lambda o: o.get("architecture") == "Tonilix", _tonilix_config, _tonilix_build,
+                      kernels="tonilix", shapes=True))

@@ -1,7 +1,8 @@
 """Building blocks of hybrid decoders for inference over ragged batches: norms (Dynamic Tanh, RMS with one gain or one per
-channel), mixers (chunked attention, attention with norms, rotations, windows, sinks and gates, latent attention, the gated delta
-rule, retention, the real-gated linear recurrence, time mixing, state-space duality, two of them side by side), gated feed-forwards
-(clamped, SiLU) and a side input per token.
+channel, over the row or equal parts of it), mixers (chunked attention, attention with norms, rotations, windows, sinks and gates, latent
+attention, the gated delta rule with decays per head or per channel, retention, the real-gated linear recurrence, time mixing, gated linear
+attention, state-space duality, two of them side by side), feed-forwards (gated: clamped, SiLU, GELU; a mixture of squared-ReLU experts)
+and a side input per token.
 
 A mixer or feed-forward is two matrix products around a ``core``: rows of ``w_in`` make its packed input, ``w_out`` takes what
 the core leaves. Layers whose sublayers run side by side lay several of them into one matrix (``place``) and call the cores on
@@ -27,7 +28,9 @@ from ..ops.retention import SPAN, RetentionGeometry, log2_decays, retention
 from ..ops.rglru import CHUNK, RGLRUGeometry, RGLRUWeights, rglru
 from ..ops.rotary import Rotary
 from ..ops.ssd import CONV_TILE, SSDGeometry, SSDWeights, ssd
-from ..ops.timemix import SPAN as STATE_SPAN, STREAMS, TimeMixGeometry, TimeMixWeights, time_mix, token_shift
+from ..ops.moe import Choice, relu2_experts
+from ..ops.timemix import (SPAN as STATE_SPAN, STREAMS, GatedLinearGeometry, GatedLinearWeights, TimeMixGeometry, TimeMixWeights, gated_linear,
+                           time_mix, token_shift)
 from .ragged import LatentRun, PagedRun, PairRun, StateRun
 
 
@@ -137,6 +140,16 @@ class RMSNorm(_Packed):
         return {"": (self.gain - self.offset).to(self.dtype)}
 
 
+class PartRMSNorm(RMSNorm):
+    """The row in ``parts`` equal runs of channels, every one over its own root mean square, times a gain per channel."""
+
+    def __init__(self, width: int, parts: int, eps: float, dtype, device):
+        if parts < 1 or width % parts:
+            raise ValueError("norm: the width is a multiple of its parts")
+        super().__init__(width, eps, 0.0, dtype, device)
+        self.parts = parts
+
+
 class DynamicTanh(_Packed):
     """tanh(alpha x) * weight + bias per channel; computes no statistics."""
 
@@ -220,20 +233,25 @@ class ChunkedAttention(_Mixer):
 
 
 class GatedDelta(_Mixer):
-    """The gated delta rule with short convolutions (see ``ops.delta``)."""
+    """The gated delta rule with short convolutions (see ``ops.delta``). With ``decay_rank`` and ``gate_rank``: decays per key channel, and
+    these and a sigmoid gate from products of that rank."""
 
-    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, conv: int, eps: float, dtype, device):
+    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, conv: int, eps: float, dtype, device,
+                 decay_rank: int = 0, gate_rank: int = 0):
         super().__init__(dtype, device)
         self.width = width
-        self.geo = g = DeltaGeometry(kv_heads, heads, dim, vdim, conv)
+        self.geo = g = DeltaGeometry(kv_heads, heads, dim, vdim, conv, decay_rank, gate_rank)
         self.w_in = self._zeros(g.cols, pad_to(width))
         self.w_out = self._zeros(width, g.out_cols)
         f32 = torch.float32
         self.w = DeltaWeights(self._zeros(conv, g.conv_cols, dtype=f32), self._zeros(heads, dtype=f32),
-                              self._zeros(heads, dtype=f32), self._zeros(vdim, dtype=f32), float(eps))
+                              self._zeros(heads * dim if g.channels else heads, dtype=f32), self._zeros(vdim, dtype=f32), float(eps))
+        if g.channels:
+            self.w.w_decay = self._zeros(pad_to(heads * dim, 8), pad_to(decay_rank))
+            self.w.w_gate = self._zeros(pad_to(heads * vdim, 8), pad_to(gate_rank))
 
     def tensors(self):
-        return super().tensors() + [self.w.conv, self.w.a_log, self.w.dt_bias, self.w.norm]
+        return super().tensors() + [t for t in vars(self.w).values() if isinstance(t, torch.Tensor)]
 
     def run_spec(self) -> StateRun:
         g = self.geo
@@ -242,8 +260,16 @@ class GatedDelta(_Mixer):
     def _sections(self):
         g = self.geo
         qk, hv = g.kv_heads * g.dim, g.heads * g.vdim
-        return (("q", 0, qk), ("k", g.off_k, qk), ("v", g.off_v, hv), ("g", g.off_gate, hv), ("b", g.off_b, g.heads),
-                ("a", g.off_a, g.heads))
+        own = (("q", 0, qk), ("k", g.off_k, qk), ("v", g.off_v, hv))
+        if g.channels:
+            return own + (("b", g.off_b, g.heads), ("a1", g.off_a, g.decay_rank), ("g1", g.off_low_gate, g.gate_rank))
+        return own + (("g", g.off_gate, hv), ("b", g.off_b, g.heads), ("a", g.off_a, g.heads))
+
+    def _second(self):
+        """name -> (matrix, rows, columns) of the products that follow the first."""
+        g = self.geo
+        return {"a2": (self.w.w_decay, g.heads * g.dim, g.decay_rank),
+                "g2": (self.w.w_gate, g.heads * g.vdim, g.gate_rank)} if g.channels else {}
 
     def logical_shapes(self):
         g = self.geo
@@ -252,7 +278,8 @@ class GatedDelta(_Mixer):
             out[name] = (n, self.width)
             if name in "qkv":
                 out[name + ".conv"] = (n, g.taps)
-        out.update({"A_log": (g.heads,), "dt_bias": (g.heads,), "norm": (g.vdim,), "o": (self.width, g.heads * g.vdim)})
+        out.update({"A_log": (g.heads,), "dt_bias": tuple(self.w.dt_bias.shape), "norm": (g.vdim,), "o": (self.width, g.heads * g.vdim)})
+        out.update({name: (n, k) for name, (_, n, k) in self._second().items()})
         return out
 
     def _pack(self, t):
@@ -264,6 +291,8 @@ class GatedDelta(_Mixer):
         self.w.dt_bias.copy_(t["dt_bias"])
         self.w.norm.copy_(t["norm"])
         self.w_out[:, :t["o"].shape[1]].copy_(t["o"])
+        for name, (w, n, k) in self._second().items():
+            w[:n, :k].copy_(t[name])
 
     def unpack(self):
         out = {}
@@ -273,10 +302,11 @@ class GatedDelta(_Mixer):
                 out[name + ".conv"] = self.w.conv[:, at:at + n].t().contiguous().to(self.dtype)
         out.update({"A_log": self.w.a_log.to(self.dtype), "dt_bias": self.w.dt_bias.to(self.dtype),
                     "norm": self.w.norm.to(self.dtype), "o": self.w_out[:, :self.geo.heads * self.geo.vdim].contiguous()})
+        out.update({name: w[:n, :k].contiguous() for name, (w, n, k) in self._second().items()})
         return out
 
-    def core(self, proj, storage, batch):
-        return gated_delta(proj, self.geo, self.w, storage[0], storage[1], batch)
+    def core(self, proj, storage, batch, out=None):
+        return gated_delta(proj, self.geo, self.w, storage[0], storage[1], batch, out)
 
 
 class ClampedGLU(_FeedForward):
@@ -342,6 +372,51 @@ class SiluGLU(_FeedForward):
 
     def core(self, gate_up, out=None):
         return ops.silu_glu(gate_up, self.in_scale, out)
+
+
+class GeluGLU(SiluGLU):
+    """W_down (gelu(W_gate h) * (W_up h)), the tanh form of GELU, without biases."""
+
+    def core(self, gate_up, out=None):
+        return ops.gelu_glu(gate_up, self.in_scale, out)
+
+
+class ExpertMLP(_Packed):
+    """A mixture of experts W_down relu(W_up h)^2 (see ``ops.moe.relu2_experts``); their weighted sum is left to the residual step."""
+    out_bias = None
+
+    def __init__(self, width: int, ff: int, choice: Choice, dtype, device):
+        super().__init__(dtype, device)
+        if ff < 1:
+            raise ValueError("feed-forward: ff must be positive")
+        self.width, self.ff, self.choice = width, ff, choice
+        E, F, K = choice.experts, pad_to(ff), pad_to(width)
+        self.w_router, self.correction = self._zeros(pad_to(E, 8), K), self._zeros(E, dtype=torch.float32)
+        self.w_up, self.w_down = self._zeros(E, F, K), self._zeros(E, width, F)
+
+    def logical_shapes(self):
+        E = self.choice.experts
+        out = {"router": (E, self.width), "correction": (E,)}
+        for e in range(E):
+            out[f"e{e}.up"], out[f"e{e}.down"] = (self.ff, self.width), (self.width, self.ff)
+        return out
+
+    def _pack(self, t):
+        self.w_router[:self.choice.experts, :self.width].copy_(t["router"])
+        self.correction.copy_(t["correction"])
+        for e in range(self.choice.experts):
+            self.w_up[e, :self.ff, :self.width].copy_(t[f"e{e}.up"])
+            self.w_down[e, :, :self.ff].copy_(t[f"e{e}.down"])
+
+    def unpack(self):
+        out = {"router": self.w_router[:self.choice.experts, :self.width].contiguous(), "correction": self.correction.to(self.dtype)}
+        for e in range(self.choice.experts):
+            out[f"e{e}.up"] = self.w_up[e, :self.ff, :self.width].contiguous()
+            out[f"e{e}.down"] = self.w_down[e, :, :self.ff].contiguous()
+        return out
+
+    def forward(self, h):
+        return relu2_experts(h, ops.project(h, self.w_router, out_dtype=torch.float32), self.correction, self.choice, self.w_up, self.w_down)
 
 
 def _head_rows(at: int, heads: int, stride: int, columns: torch.Tensor) -> torch.Tensor:
@@ -538,12 +613,12 @@ class RGLRU(_RowPacked):
 
 class ShapedAttention(_RowPacked):
     """Grouped-query attention whose parts can be chosen (see ``ops.ragged``): biases on the projections, values of their own or the
-    keys as projected, a norm of q and k, rotation, a mask, what becomes of the scores, values mixed with those of the model's
-    first such layer, a gate per head or per element."""
+    keys as projected, a norm of q and k, rotation, queries that grow with the position, a mask, what becomes of the scores, values mixed
+    with those of the model's first such layer, a gate per head or per element, a bias on the result."""
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, form: ScoreForm, eps: float, dtype, device, bias: bool = False,
                  keys_as_values: bool = False, norm: str = "", rotary: Optional[Rotary] = None, learned_sink: bool = False, v_mix: bool = False,
-                 gate: str = ""):
+                 gate: str = "", q_temp: Optional[tuple] = None, out_bias: bool = False):
         super().__init__(dtype, device)
         self.width, self.v_mix, self.learned_sink = width, bool(v_mix), bool(learned_sink)
         self.geo = g = AttentionGeometry(heads, kv_heads, dim, vdim, dtype, rotary, keys_as_values, gate)
@@ -556,7 +631,9 @@ class ShapedAttention(_RowPacked):
         if norm not in ("", "unit", "head", "whole"):
             raise ValueError(f"attention: unknown norm {norm!r}")
         self.w = AttentionWeights(form, vec(g.off_gate) if bias else None, norm, vec(sizes[0]) if sizes else None,
-                                  vec(sizes[1]) if sizes else None, float(eps))
+                                  vec(sizes[1]) if sizes else None, float(eps), q_temp=q_temp)
+        if out_bias:
+            self.out_bias = vec(width)
         self.masks = (form.mask,)
         if norm == "unit":
             form.product_bound = 1.02 * dim               # (two unit vectors times sqrt(dim), rounded)
@@ -592,6 +669,8 @@ class ShapedAttention(_RowPacked):
             out.update({"q.norm": (w.q_norm, rows["q"]), "k.norm": (w.k_norm, rows["k"] - g.off_k)})
         if self.learned_sink:
             out["sink"] = (w.form.sink, torch.arange(g.heads))
+        if self.out_bias is not None:
+            out["o.b"] = (self.out_bias, torch.arange(self.width))
         return out
 
     def logical_shapes(self):
@@ -677,6 +756,61 @@ class TimeMix(_RowPacked):
         return time_mix(proj, self.geo, self.w, storage[1], batch, self.out_scale, out)
 
 
+class GatedLinear(_RowPacked):
+    """Gated linear attention: a decay per key channel from a product of low rank (see ``ops.timemix.gated_linear``)."""
+    tile = STATE_SPAN
+
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, rank: int, tau: float, eps: float, dtype, device):
+        super().__init__(dtype, device)
+        if tau <= 0:
+            raise ValueError("gated linear attention: tau must be positive")
+        self.width = width
+        self.geo = g = GatedLinearGeometry(heads, dim, vdim, rank)
+        self.w_in, self.w_out = self._zeros(g.cols, pad_to(width)), self._zeros(width, g.out_cols)
+        f32 = torch.float32
+        self.w = GatedLinearWeights(self._zeros(heads * g.dp, g.rp), self._zeros(heads * g.dp, dtype=f32), self._zeros(heads * g.ep, dtype=f32),
+                                    float(tau), float(eps))
+
+    def tensors(self):
+        return super().tensors() + [self.w.w2, self.w.w0, self.w.norm]
+
+    def run_spec(self) -> StateRun:
+        g = self.geo
+        return StateRun((g.heads, g.ep, g.dp))
+
+    def _keys(self, at=0):
+        return _head_rows(at, self.geo.heads, self.geo.dp, torch.arange(self.geo.dim))
+
+    def _values(self, at=0):
+        return _head_rows(at, self.geo.heads, self.geo.ep, torch.arange(self.geo.vdim))
+
+    def _rows(self):
+        g = self.geo
+        return {"q": self._keys(), "k": self._keys(g.off_k), "v": self._values(g.off_v), "g": self._values(g.off_gate),
+                "a1": g.off_low + torch.arange(g.rank)}
+
+    def _out_columns(self):
+        return self._values()
+
+    def logical_shapes(self):
+        g = self.geo
+        return {**self._row_shapes(), "norm": (g.vdim,), "a2": (g.heads * g.dim, g.rank), "a2.b": (g.heads * g.dim,)}
+
+    def _pack(self, t):
+        g, at = self.geo, self._keys().to(self.device)
+        self._pack_rows(t)
+        self.w.w2[at, :g.rank] = t["a2"].to(self.device, self.dtype)
+        self.w.w0[at] = t["a2.b"].to(self.device).float()
+        self.w.norm.view(g.heads, g.ep)[:, :g.vdim] = t["norm"].to(self.device).float()
+
+    def unpack(self):
+        g, at = self.geo, self._keys().to(self.device)
+        return {**self._unpack_rows(), "norm": self.w.norm[:g.vdim].to(self.dtype), "a2": self.w.w2[at, :g.rank], "a2.b": self.w.w0[at].to(self.dtype)}
+
+    def core(self, proj, storage, batch, out=None):
+        return gated_linear(proj, self.geo, self.w, storage[0], batch, self.out_scale, out)
+
+
 class SSD(_RowPacked):
     """State-space duality with a short convolution, normed in parts after its gate (see ``ops.ssd``)."""
     tiles = (CONV_TILE, STATE_SPAN)
@@ -752,6 +886,8 @@ class SideBySide(_Mixer):
         left.place(self.w_in[:left.cols], self.w_out[:, :left.out_cols])
         right.place(self.w_in[self.cut:], self.w_out[:, left.out_cols:])
         self.masks = left.masks + right.masks
+        if any(p.out_bias is not None for p in (left, right)):
+            self.out_bias = self._zeros(width, dtype=torch.float32)
 
     @property
     def tiles(self) -> tuple:
@@ -773,6 +909,11 @@ class SideBySide(_Mixer):
     def _pack(self, t):
         for pre, p in self._both():
             p._pack({n: t[pre + n] for n in p.logical_shapes()})
+        if self.out_bias is not None:
+            self.out_bias.zero_()
+            for _, p in self._both():
+                if p.out_bias is not None:
+                    self.out_bias += p.out_scale * p.out_bias
 
     def unpack(self):
         return {pre + n: v for pre, p in self._both() for n, v in p.unpack().items()}

@@ -382,7 +382,7 @@ def cross_entropy(logits: torch.Tensor, targets: torch.Tensor) -> torch.Tensor:
 _P, _I, _L, _F = _native.P, _native.I, _native.L, _native.F
 _native.register_signatures({
     "tsb_dyn_tanh_residual": [_P, _I, _I, _P, _L, _P, _F, _P, _P, _P, _P, _L, _F, _I, _I, _P, _F, _P, _P, _P, _L, _I, _I, _P],
-    "tsb_clamped_glu": [_P, _L, _P, _P, _L, _I, _I, _F, _F, _F, _F, _I, _P],
+    "tsb_clamped_glu": [_P, _L, _P, _P, _L, _I, _I, _F, _F, _F, _F, _F, _I, _P],
     "tsb_depth_residual": [_P, _P, _P, _L, _P, _I, _I, _P, _L, _F, _P, _P, _L, _I, _P, _L, _I, _I, _I, _F, _F, _I, _P],
 })
 _EMBED_MODES = {None: 0, "set": 1, "add": 2}
@@ -441,9 +441,9 @@ def dyn_tanh_residual(x, y=None, y_bias=None, post=None, tokens=None, table=None
     return h
 
 
-def clamped_glu(gate_up, bias, limit, slope=1.702, shift=1.0, in_scale=1.0, out=None):
-    """gate_up [T, 2 F] (gate, then up; times ``in_scale``, plus ``bias`` fp32 [2 F] if given) -> g sigmoid(slope g) (u + shift)
-    with g = min(gate, limit), u = clamp(up, -limit, limit). ``out`` may be columns of a wider matrix."""
+def clamped_glu(gate_up, bias, limit, slope=1.702, shift=1.0, in_scale=1.0, out=None, cubic=0.0):
+    """gate_up [T, 2 F] (gate, then up; times ``in_scale``, plus ``bias`` fp32 [2 F] if given) ->
+    g sigmoid(slope (g + cubic g^3)) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit). ``out`` may be columns of a wider matrix."""
     T, F2 = gate_up.shape
     F = F2 // 2
     if out is None:
@@ -452,19 +452,24 @@ def clamped_glu(gate_up, bias, limit, slope=1.702, shift=1.0, in_scale=1.0, out=
         return out
     if gate_up.is_cuda:
         check(lib().tsb_clamped_glu(gate_up.data_ptr(), gate_up.stride(0), _ptr(bias), out.data_ptr(), out.stride(0), T, F,
-                                    float(limit), float(slope), float(shift), float(in_scale), dtype_code(gate_up.dtype),
+                                    float(limit), float(slope), float(shift), float(in_scale), float(cubic), dtype_code(gate_up.dtype),
                                     stream_ptr(gate_up.device)), "tsb_clamped_glu")
         return out
     z = gate_up.float() * in_scale
     if bias is not None:
         z = z + bias
     g, u = z[:, :F].clamp(max=limit), z[:, F:].clamp(-limit, limit)
-    return out.copy_(g * torch.sigmoid(slope * g) * (u + shift))
+    return out.copy_(g * torch.sigmoid(slope * (g + cubic * g ** 3)) * (u + shift))
 
 
 def silu_glu(gate_up, in_scale=1.0, out=None):
     """SiLU(gate) * up of the two halves of a row, both times ``in_scale`` first."""
     return clamped_glu(gate_up, None, math.inf, 1.0, 0.0, in_scale, out)
+
+
+def gelu_glu(gate_up, in_scale=1.0, out=None):
+    """The tanh form of GELU(gate) * up: (1 + tanh z) / 2 = sigmoid(2 z)."""
+    return clamped_glu(gate_up, None, math.inf, 2.0 * math.sqrt(2.0 / math.pi), 0.0, in_scale, out, 0.044715)
 
 
 def depth_residual(x_in=None, y=None, mult=1.0, tokens=None, table=None, width=0, history=None, depth=0, average=None, store=True,

@@ -8,8 +8,14 @@ grouped kernel for the input gradients and its reduction-grouped mode for all ex
 routing math itself (softmax, top-k, renormalisation) stays in ``nn.moe.route_topk`` so that every path shares it.
 Replaces the reference's host-synchronised count -> permute -> cublasGemmGroupedBatchedEx pipeline
 (src/cuda/MoeForward.cu:139-298).
+
+``relu2_experts`` is the serving form of another mixture (``csrc/expert_mlp.cu``): sigmoid scores, a choice corrected and limited to
+groups, squared-ReLU experts; its weighted sum is left to the residual step.
 """
 from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
 
 import torch
 
@@ -26,7 +32,7 @@ _native.register_signatures({
     "tsb_moe_gather_rows": [P, P, P, P, I, I, I, P],
     "tsb_moe_combine": [P, P, P, P, I, I, I, P],
     "tsb_moe_gate_grad": [P, P, P, P, I, I, I, P],
-    "tsb_gemm_grouped": [P, P, P, P, I, I, I, I, I, I, L, L, L, I, L, L, I, I, P],
+    "tsb_gemm_grouped": [P, P, P, P, I, I, I, I, I, I, L, L, L, I, L, L, I, I, I, P],
     "tsb_gemm_grouped_scatter": [P, P, P, I, I, I, I, L, L, I, L, P, _native.ctypes.POINTER(_native.ctypes.c_void_p), I, L,
                                  L, P],
     "tsb_ep_publish_counts": [_native.ctypes.POINTER(_native.ctypes.c_void_p), P, I, I, I, P],
@@ -108,14 +114,14 @@ def combine_rows(ys: torch.Tensor, pos: torch.Tensor, T: int, k: int, gates: tor
 
 
 def grouped_gemm_rows(a: torch.Tensor, w0: torch.Tensor, group_stride: int, offsets: torch.Tensor, groups: int,
-                      b_mn: bool = False) -> torch.Tensor:
+                      b_mn: bool = False, act: int = 0) -> torch.Tensor:
     """Row-grouped GEMM: out[r] = a[r] @ op(W[g(r)]). ``w0`` is group 0's weight ([N, K], or used as [K, N] when
-    ``b_mn``); group g's weight starts ``g * group_stride`` elements later in the same allocation."""
+    ``b_mn``); group g's weight starts ``g * group_stride`` elements later in the same allocation. ``act`` 1: relu(out)^2."""
     rows_cap, K = a.shape
     N = w0.shape[1] if b_mn else w0.shape[0]
     out = torch.empty((rows_cap, N), dtype=torch.bfloat16, device=a.device)
     check(lib().tsb_gemm_grouped(a.data_ptr(), w0.data_ptr(), out.data_ptr(), offsets.data_ptr(), groups, 1, rows_cap,
-                                 0, N, K, a.stride(0), w0.stride(0), out.stride(0), int(b_mn), group_stride, 0, 0, 0,
+                                 0, N, K, a.stride(0), w0.stride(0), out.stride(0), int(b_mn), group_stride, 0, 0, 0, act,
                                  stream_ptr(a.device)), "tsb_gemm_grouped")
     return out
 
@@ -141,7 +147,7 @@ def grouped_gemm_wgrad(dy: torch.Tensor, x: torch.Tensor, offsets: torch.Tensor,
     N = x.shape[1]
     check(lib().tsb_gemm_grouped(dy.data_ptr(), x.data_ptr(), out.data_ptr(), offsets.data_ptr(), groups, 2, rows_cap,
                                  M, N, 0, dy.stride(0), x.stride(0), ldc, 1, 0, group_stride,
-                                 int(out.dtype == torch.float32), int(accumulate), stream_ptr(dy.device)),
+                                 int(out.dtype == torch.float32), int(accumulate), 0, stream_ptr(dy.device)),
           "tsb_gemm_grouped")
 
 
@@ -297,3 +303,101 @@ def moe_ffn_grouped(x2: torch.Tensor, idx: torch.Tensor, gates: torch.Tensor, mo
     if counts is None:
         counts = torch.bincount(idx32.view(-1), minlength=E).to(torch.int32)
     return _GroupedExpertsFn.apply(x2.contiguous(), gates, idx32, counts, per, E, k, w_gu0, w_dn0, *ws)
+
+
+# ------------------------------------------------------------------------------ serving: grouped choice, squared-ReLU experts
+_native.register_signatures({
+    "tsb_expert_route": [P, L, P, _native.F, P],
+    "tsb_expert_gather": [P, L, P, P, P, I, I, I, P],
+    "tsb_expert_tiles": [P, P, P, I, P],
+})
+MAX_EXPERTS, MAX_TOP = 256, 32
+TILE_ROWS = 256              # up to so many tokens the experts' rows go through tiles of 16 (bf16)
+
+
+@dataclass(frozen=True)
+class Choice:
+    """``top`` of ``experts`` by score + correction, out of the ``keep`` best of ``groups`` groups of neighbours; weights are scores over
+    their sum, times ``scale``."""
+    experts: int
+    top: int
+    groups: int
+    keep: int
+    scale: float
+
+    def __post_init__(self):
+        if min(self.experts, self.top, self.groups, self.keep) < 1 or self.experts % self.groups or self.keep > self.groups:
+            raise ValueError("experts: positive sizes, equal groups, and at most all of them kept")
+        if self.top > self.experts // self.groups * self.keep:
+            raise ValueError("experts: the kept groups have fewer experts than are taken")
+        if self.experts > MAX_EXPERTS or self.top > MAX_TOP:
+            raise ValueError(f"experts: at most {MAX_EXPERTS}, of which {MAX_TOP} are taken")
+
+
+@dataclass
+class Mixed:
+    """Experts' results that are yet to be summed: token t's result is sum_j weight[t, j] rows[pos[t, j]]."""
+    rows: torch.Tensor
+    pos: torch.Tensor
+    weight: torch.Tensor
+
+    def sum(self) -> torch.Tensor:
+        """fp32 [T, columns]."""
+        return (self.rows[self.pos.long()].float() * self.weight[..., None]).sum(1)
+
+
+def choose_experts_torch(logits: torch.Tensor, correction: torch.Tensor, c: Choice):
+    """(expert ids [T, top], weights [T, top]) from fp32 logits [T, experts]."""
+    s = torch.sigmoid(logits)
+    choice = s + correction
+    if c.keep < c.groups:
+        g = choice.view(-1, c.groups, c.experts // c.groups)
+        worth = g.topk(min(2, g.shape[2]), dim=2).values.sum(2)
+        kept = torch.zeros_like(worth, dtype=torch.bool).scatter_(1, worth.topk(c.keep, dim=1).indices, True)
+        choice = g.masked_fill(~kept[:, :, None], float("-inf")).view(-1, c.experts)
+    idx = choice.topk(c.top, dim=1).indices
+    w = s.gather(1, idx)
+    return idx, w / (w.sum(1, keepdim=True) + 1e-20) * c.scale
+
+
+def relu2_experts(h: torch.Tensor, logits: torch.Tensor, correction: torch.Tensor, c: Choice, w_up: torch.Tensor,
+                  w_down: torch.Tensor) -> Mixed:
+    """Every token's chosen experts W_down relu(W_up h)^2. h [T, K] and ``logits`` [T, >= experts] (fp32) of the same rows, ``w_up``
+    [experts, F, K], ``w_down`` [experts, W, F] in the type of h, F and K multiples of 16; ``correction`` fp32 [experts]."""
+    T, K = h.shape
+    E, F, top, dev = c.experts, w_up.shape[1], c.top, h.device
+    W = w_down.shape[1]
+    if not h.is_cuda:
+        idx, weight = choose_experts_torch(logits[:, :E], correction, c)
+        rows = torch.empty((T * top, W), dtype=h.dtype)
+        for e in range(E):
+            t, j = (idx == e).nonzero(as_tuple=True)
+            a = torch.relu(h[t].float() @ w_up[e].float().t()) ** 2
+            rows[t * top + j] = (a.to(h.dtype).float() @ w_down[e].float().t()).to(h.dtype)
+        return Mixed(rows, torch.arange(T * top).view(T, top), weight)
+    grouped = h.dtype == torch.bfloat16 and T > TILE_ROWS
+    pad = 128 if grouped else 16 if T <= TILE_ROWS else 64
+    tiles = min(E, T * top) + T * top // pad          # (an expert without rows has no tile)
+    i32 = lambda *s: torch.empty(s, device=dev, dtype=torch.int32)   # noqa: E731
+    idx, pos, offsets, assign, counts = i32(T, top), i32(T, top), i32(E + 1), i32(tiles * pad), i32(2 * E)
+    weight = torch.empty((T, top), device=dev, dtype=torch.float32)
+    st = stream_ptr(dev)
+    ptrs = (ctypes.c_void_p * 8)(logits.data_ptr(), correction.data_ptr(), idx.data_ptr(), weight.data_ptr(), counts.data_ptr(),
+                                 offsets.data_ptr(), pos.data_ptr(), assign.data_ptr())
+    check(lib().tsb_expert_route((ctypes.c_int * 6)(T, E, top, c.groups, c.keep, pad), logits.stride(0), ptrs, float(c.scale), st),
+          "tsb_expert_route")
+    if grouped:
+        _native.add_launches(1)
+        xs = torch.empty((tiles * pad, K), device=dev, dtype=h.dtype)
+        check(lib().tsb_expert_gather(h.data_ptr(), h.stride(0), assign.data_ptr(), offsets[E:].data_ptr(), xs.data_ptr(), tiles * pad, K, top,
+                                      st), "tsb_expert_gather")
+        a = grouped_gemm_rows(xs, w_up[0], w_up.stride(0), offsets, E, act=1)
+        return Mixed(grouped_gemm_rows(a, w_down[0], w_down.stride(0), offsets, E), pos, weight)
+    act = torch.empty((tiles * pad, F), device=dev, dtype=h.dtype)
+    rows = torch.empty((tiles * pad, W), device=dev, dtype=h.dtype)
+    for x, w, y, up in ((h, w_up, act, 1), (act, w_down, rows, 0)):
+        ints = (ctypes.c_int * 7)(E, w.shape[1], w.shape[2], top, tiles, pad, up)
+        lds = (ctypes.c_longlong * 3)(x.stride(0), w.stride(1), y.stride(0))
+        ptrs = (ctypes.c_void_p * 5)(x.data_ptr(), w.data_ptr(), y.data_ptr(), offsets.data_ptr(), assign.data_ptr())
+        check(lib().tsb_expert_tiles(ints, lds, ptrs, _native.dtype_code(h.dtype), st), "tsb_expert_tiles")
+    return Mixed(rows, pos, weight)

@@ -218,7 +218,8 @@ class AttentionGeometry:
 class AttentionWeights:
     """fp32 parameters besides the projections. ``bias`` [off_gate] or None. ``norm``: "" (none), "unit" (every q and k head over its
     root mean square), "head" (times q_norm, k_norm [D]), "whole" (all heads together, times q_norm [heads * D], k_norm). Values:
-    (1 - vmix) v + vmix v_first where a first layer's values are given."""
+    (1 - vmix) v + vmix v_first where a first layer's values are given. Queries at position p times 1 + coef ln(floor((p + 1) / every) + 1)
+    for ``q_temp`` = (coef, every)."""
     form: ScoreForm
     bias: Optional[torch.Tensor] = None
     norm: str = ""
@@ -226,6 +227,7 @@ class AttentionWeights:
     k_norm: Optional[torch.Tensor] = None
     eps: float = 0.0
     vmix: float = 0.0
+    q_temp: Optional[tuple] = None
 
 
 _NORMS = {"": 0, "unit": 1, "head": 2, "whole": 3}
@@ -251,7 +253,7 @@ def shaped_attention(proj: torch.Tensor, geo: AttentionGeometry, w: AttentionWei
     stage = torch.empty((seg.keys, 2 * G, D), device=proj.device, dtype=proj.dtype) if seg is not None else None
     ints = (ctypes.c_int * 13)(T, H, G, D, geo.dim, geo.hp, geo.off_k, geo.off_v, _NORMS[w.norm], bs, nd, proj.stride(0),
                                first_values.shape[3] if first_values is not None else 0)
-    floats = (ctypes.c_float * 2)(w.eps, w.vmix)
+    floats = (ctypes.c_float * 4)(w.eps, w.vmix, *(w.q_temp or (0.0, 1.0)))
     ptrs = (ctypes.c_void_p * 13)(proj.data_ptr(), _ptr(w.bias), _ptr(w.q_norm), _ptr(w.k_norm), _ptr(angles), batch.positions.data_ptr(),
                                   batch.slots.data_ptr(), q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), _ptr(first_values), _ptr(stage),
                                   _ptr(seg.stage_rows) if seg is not None else None)
@@ -279,6 +281,9 @@ def _shaped_torch(proj, geo, w, k_pool, v_pool, angles, first_values, batch, gat
     if angles is not None:
         pos = batch.positions.long()
         q, k = rotate_stored(q, angles, pos), rotate_stored(k, angles, pos)
+    if w.q_temp is not None:
+        coef, every = w.q_temp
+        q = q * (1.0 + coef * torch.log(torch.floor((batch.positions + 1).float() / every) + 1.0))[:, None, None]
     if first_values is not None:
         sl = batch.slots.long()
         first = torch.nn.functional.pad(first_values[sl // bs, :, sl % bs].float(), (0, max(0, D - first_values.shape[3])))
