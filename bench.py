@@ -110,11 +110,12 @@ def parse_args():
                     help="auto | dp | tp | tpK (tensor parallel over K ranks, data parallel over the rest) | a comma list: "
                          "every mesh listed is measured and `value` is the fastest")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--hybrid", nargs="?", const="fozelix", default="", choices=["fozelix", "polosun", "vobotar"],
+    ap.add_argument("--hybrid", nargs="?", const="fozelix", default="", choices=["fozelix", "polosun", "vobotar", "tonilix"],
                     help="instead of the headline: prefill and decode throughput of a hybrid decoder at the sizes of real layers, one "
                          "GPU (benchmarks/bench_hybrid.py): fozelix (gated delta rule + chunked attention, beside Llama; the default), "
-                         "polosun (retention, latent attention, gated recurrence, beside fozelix and Llama) or vobotar (attention, time mixing, "
-                         "state-space duality, beside polosun, fozelix and Llama)")
+                         "polosun (retention, latent attention, gated recurrence, beside fozelix and Llama), vobotar (attention, time mixing, "
+                         "state-space duality, beside polosun, fozelix and Llama) or tonilix (delta rule with channel decays, gated linear "
+                         "attention, experts, beside vobotar, fozelix and Llama)")
     ap.add_argument("--ref-time-budget", type=float, default=float(os.environ.get("TESSERACT_REF_TIME_BUDGET", 780)),
                     help="(--impl reference) seconds the whole reference arm may take; the timed step count shrinks to fit")
     return ap.parse_args()
@@ -299,7 +300,7 @@ def main():
         sampler = ClockSampler(0)
         sampler.start()
         models = {"fozelix": ("hybrid", "llama"), "polosun": ("polosun", "hybrid", "llama"),
-                  "vobotar": ("vobotar", "polosun", "hybrid", "llama")}[args.hybrid]
+                  "vobotar": ("vobotar", "polosun", "hybrid", "llama"), "tonilix": ("tonilix", "vobotar", "hybrid", "llama")}[args.hybrid]
         sizes = run(models=models)
         print(json.dumps({"benchmark": "hybrid decoder serving beside other models at equal size", "models": models, "n_gpus": 1, "dtype": "bf16",
                           "data": "synthetic random token ids; random-init weights", "sizes": sizes, "clocks": sampler.stop()}))

@@ -3,15 +3,17 @@
 serving engine on one GPU.
 
     python benchmarks/bench_hybrid.py                      # every size
-    python benchmarks/bench_hybrid.py --models vobotar,polosun,hybrid,llama
-    python bench.py --hybrid [fozelix | polosun | vobotar] # the same, from the headline benchmark's command line
+    python benchmarks/bench_hybrid.py --models tonilix,vobotar,polosun,hybrid,llama
+    python bench.py --hybrid [fozelix | polosun | vobotar | tonilix]    # the same, from the headline benchmark's command line
 
 The models of a size have the same width, feed-forward, layer count, vocabulary and attention heads. ``hybrid`` has three
 gated-delta layers (16 or 8 key heads, twice as many value heads, 128 x 128) to every chunked-attention layer; ``polosun``
 cycles through retention (heads of 128 x 128), latent attention (64 + 64 rotated query columns a head, values of 128, a latent
 of 512) and the gated recurrence (as many channels as the width, gate blocks of 256); ``vobotar`` through capped attention, attention
 in a window of 1024 beside time mixing (heads of 64, as wide as the model) and beside state-space duality (heads of 64, twice as wide as
-the model, a state of 128), with a side input of 128 columns per layer. bf16 weights and KV on all sides,
+the model, a state of 128), with a side input of 128 columns per layer; ``tonilix`` has two layers of the delta rule with decays per channel
+(heads of 128 x 128, as wide as the model) to every one of attention beside gated linear attention (heads of 64, as wide as the model), a
+dense first feed-forward and then 6 of 32 experts, which together do the work of the dense one. bf16 weights and KV on all sides,
 greedy. Prefill: ``seqs`` prompts of ``prompt`` tokens in one step; decode: a batch of
 requests after that. Times are wall clock around engine steps with a device synchronise on both sides (inputs from the
 host and the read of the chosen tokens included); ``gpu_ms`` is the captured decode step alone, from CUDA events. Every
@@ -60,6 +62,14 @@ def build(kind, s, device, max_pos):
         layers = vobotar.standard_layers(s["layers"], s["heads"], s["kv"], 128, 1024, W // 64, 64, 64, 2 * W // 64, 64, 128, s["ff"])
         return HybridModel(HybridConfig(s["vocab"], W, layers, eps=1e-6, dtype=torch.bfloat16, form="post", token_side=128), device=device,
                            init_std=0.02, seed=1)
+    if kind == "tonilix":
+        from tesseract_b200.models import tonilix
+        from tesseract_b200.models.hybrid import Choice
+        W = s["width"]
+        layers = tonilix.standard_layers(s["layers"], s["heads"], s["kv"], 128, W // 128, 128, 128, W // 64, 64, s["ff"], s["ff"] // 4,
+                                         Choice(32, 6, 4, 2, 1.0))
+        return HybridModel(HybridConfig(s["vocab"], W, layers, eps=1e-6, dtype=torch.bfloat16, form="pre", tied=False, norm_parts=2,
+                                        layer_scale=True, token_shift=True, sinusoid=True, embed_norm=True), device=device, init_std=0.02, seed=1)
     att = AttentionSpec(s["heads"], s["kv"], 128, 128, 128 ** -0.5, 4096)
     dlt = DeltaSpec(2 * s["key_heads"], s["key_heads"], 128, 128, 4)
     layers = [LayerSpec(att if i % 4 == 3 else dlt, GLUSpec(s["ff"], 7.0)) for i in range(s["layers"])]
@@ -145,7 +155,7 @@ def main():
     ap.add_argument("--seqs", type=int, default=4)
     ap.add_argument("--prompt", type=int, default=4096)
     ap.add_argument("--steps", type=int, default=24)
-    ap.add_argument("--models", default="hybrid,llama", help="comma list of vobotar, polosun, hybrid, llama")
+    ap.add_argument("--models", default="hybrid,llama", help="comma list of tonilix, vobotar, polosun, hybrid, llama")
     a = ap.parse_args()
     models = a.models.split(",")
     for name, r in run(a.sizes.split(","), a.seqs, a.prompt, steps=a.steps, models=models).items():

@@ -681,6 +681,90 @@ def case_project_inputs(b: Bench):
         report("project_one", b.time(lambda: ops.project(xs[0], w)), shape=[M, w.shape[0], 4096], **kw)
 
 
+# ---- 4096-wide pre-normed layers: 32 heads of 128 x 128 (delta rule, decays per channel), 64 heads of 64 (gated linear attention), 32 / 8
+# heads of 128 (attention), 6 of 32 experts of 3584
+def case_channel_delta(b: Bench):
+    """All launches, the two products of low rank included; counted like delta_prefill and delta_step."""
+    from tesseract_b200.nn.hybrid import GatedDelta
+    H, D = 32, 128
+    blk = GatedDelta(64, H, H, D, D, 4, 1e-6, torch.bfloat16, b.dev, 128, 128)
+    blk.w.conv.uniform_(-0.5, 0.5)
+    blk.w.dt_bias.uniform_(-6.0, -1.0)
+    blk.w.w_decay.normal_(std=0.05)
+    blk.w.w_gate.normal_(std=0.05)
+    peak = 148 * 128 * 2 * 1.965e9 / 1e12
+    for n, rows in ((4, 4096), (1, 4096), (32, 512)):
+        ms = _mixer_case(b, blk, n, rows)
+        fl = 8.0 * H * D * D * n * rows
+        print(json.dumps({"case": "channel_delta_prefill", "ms": round(ms, 4), "fp32_tflops": round(fl / ms / 1e9, 2),
+                          "frac_of_nominal_fp32": round(fl / ms / 1e9 / peak, 3), "ns_per_token": round(ms * 1e6 / (n * rows), 1),
+                          "shape": [n, rows]}), flush=True)
+    for n in (256, 32):
+        report("channel_delta_step", _mixer_case(b, blk, n, 1, 7), bytes_=n * 2.0 * H * D * D * 4, shape=[n])
+
+
+def case_gated_linear(b: Bench):
+    """Prompts: bytes of q, k, v, gate and the result; decode: the state read and written once."""
+    from tesseract_b200.nn.hybrid import GatedLinear
+    for H, D in ((64, 64), (32, 128)):
+        blk = GatedLinear(64, H, D, D, 64, 16.0, 1e-6, torch.bfloat16, b.dev)
+        blk.w.w2.normal_(std=0.1)
+        for n, rows in ((4, 4096), (1, 4096), (32, 512)):
+            report("gated_linear_prefill", _mixer_case(b, blk, n, rows), bytes_=n * rows * H * D * 5 * 2.0, shape=[n, rows, H, D])
+        for n in (256, 32):
+            report("gated_linear_step", _mixer_case(b, blk, n, 1, 7), bytes_=n * 2.0 * H * D * D * 4, shape=[n, H, D])
+
+
+def case_growing_attn(b: Bench):
+    """Counts of shaped_attn."""
+    from tesseract_b200.nn.hybrid import ShapedAttention
+    from tesseract_b200.ops.ragged import ScoreForm
+    blk = ShapedAttention(64, 32, 8, 128, 128, ScoreForm(128 ** -0.5), 1e-6, torch.bfloat16, b.dev, bias=True, gate="element", q_temp=(0.1, 512.0))
+    for n, rows in ((2, 4096), (8, 1024)):
+        report("growing_attn_prefill", _mixer_case(b, blk, n, rows), flops=4.0 * n * rows * (rows + 1) / 2 * 32 * 128, shape=[n, rows])
+    for n in (256, 32):
+        report("growing_attn_decode", _mixer_case(b, blk, n, 1, 1399), bytes_=n * 1400 * 8 * 128 * 2 * 2.0, shape=[n, 1400])
+
+
+def case_pre_norm(b: Bench):
+    """The step between two products: bytes of x and y in, x and h out (mixed: the chosen rows)."""
+    from tesseract_b200.nn.ragged import StateRun
+    from tesseract_b200.ops.moe import Mixed
+    from tesseract_b200.ops.pre_norm import Shift, pre_norm_step
+    W = 4096
+    for n, rows in ((4, 4096), (256, 1), (32, 1)):
+        T = n * rows
+        st = _Step(b, StateRun((W,)), n, rows, 7 if rows == 1 else 0)
+        x, y, one = torch.randn(T, W, device=b.dev, generator=b.gen), b.randn(T, W), torch.ones(W, device=b.dev)
+        mixed = Mixed(b.randn(T * 6, W), torch.randperm(T * 6, device=b.dev).int().view(T, 6), torch.rand(T, 6, device=b.dev))
+        shift = Shift(0.5 * one, st.cache.runs[0][0])
+        for name, yy, sh, by in (("plain", y, None, 12), ("shift", y, shift, 12), ("mixed_shift", mixed, shift, 22)):
+            ms = b.time(lambda: pre_norm_step(st.batch, W, one, 2, 1e-6, x, yy, one, one, shift=sh, out_dtype=torch.bfloat16))
+            report("pre_norm_" + name, ms, bytes_=T * W * float(by), shape=[n, rows, W])
+
+
+def case_experts(b: Bench):
+    """Choice, layout, gather and both products (router and weighted sum not included): prompts by FLOPs, decoded tokens by the bytes
+    of the experts that are taken."""
+    from tesseract_b200.ops.moe import Choice, relu2_experts
+    W, F, c = 4096, 3584, Choice(32, 6, 4, 2, 1.0)
+    up, down = b.randn(32, F, W, scale=0.02), b.randn(32, W, F, scale=0.02)
+    corr = torch.zeros(32, device=b.dev)
+    for T in (16384, 2048, 256, 32, 1):
+        h, z = b.randn(T, W), torch.randn(T, 32, device=b.dev, generator=b.gen)
+        ms = b.time(lambda: relu2_experts(h, z, corr, c, up, down))
+        from tesseract_b200.ops.moe import choose_experts_torch
+        taken = choose_experts_torch(z, corr, c)[0].unique().numel()
+        kw = dict(flops=4.0 * T * 6 * W * F) if T > 256 else dict(bytes_=taken * 2 * W * F * 2.0)
+        report("experts", ms, shape=[T, 32, 6, W, F], **kw)
+
+
+def case_gelu_glu(b: Bench):
+    from tesseract_b200 import ops
+    x = b.randn(16384, 2 * 14336)
+    report("gelu_glu", b.time(lambda: ops.gelu_glu(x)), bytes_=x.numel() * 2 * 1.5, shape=list(x.shape))
+
+
 CASES = {"gemm": case_gemm, "gemm_fp8": case_gemm_fp8, "gemm_fp8_pertensor": case_gemm_fp8_pertensor, "decode_gemm": case_decode_gemm, "gemm_wgrad": case_gemm_wgrad, "grouped_gemm": case_grouped_gemm,
          "flash_fwd": case_flash_fwd, "flash_bwd": case_flash_bwd, "decode": case_decode,
          "decode_int8": case_decode_int8, "rmsnorm": case_rmsnorm, "swiglu": case_swiglu, "swiglu_bwd": case_swiglu_bwd, "adam": case_adam,
@@ -690,7 +774,8 @@ CASES = {"gemm": case_gemm, "gemm_fp8": case_gemm_fp8, "gemm_fp8_pertensor": cas
          "dyn_tanh": case_dyn_tanh, "clamped_glu": case_clamped_glu, "retention": case_retention, "latent": case_latent, "rglru": case_rglru,
          "depth_residual": case_depth_residual, "silu_glu": case_silu_glu, "shaped_attn": case_shaped_attn, "attn_prepare": case_attn_prepare, "time_mix": case_time_mix,
          "ssd": case_ssd, "post_norm": case_post_norm, "token_side": case_token_side, "token_shift": case_token_shift,
-         "project_inputs": case_project_inputs}
+         "project_inputs": case_project_inputs, "channel_delta": case_channel_delta, "gated_linear": case_gated_linear,
+         "growing_attn": case_growing_attn, "pre_norm": case_pre_norm, "experts": case_experts, "gelu_glu": case_gelu_glu}
 
 
 def main():

@@ -36,7 +36,7 @@ def preset(name: str, dtype: torch.dtype, max_pos: int) -> LlamaConfig:
         cfg = LlamaConfig.llama_3_2_1b()
         cfg.dtype, cfg.max_position_embeddings = dtype, max_pos
         return cfg
-    if name.startswith(("fozelix-", "polosun-", "vobotar-")):
+    if name.startswith(("fozelix-", "polosun-", "tonilix-", "vobotar-")):
         from tesseract_b200 import models
         family, size = name.split("-", 1)
         try:
@@ -44,7 +44,7 @@ def preset(name: str, dtype: torch.dtype, max_pos: int) -> LlamaConfig:
         except ValueError as e:
             raise SystemExit(f"error: --model: {e}") from None
     raise SystemExit(f"error: unknown --model '{name}' (tiny | small | llama3.2-1b | llama3-8b | fozelix-tiny | fozelix-small | "
-                     "polosun-tiny | polosun-small | vobotar-tiny | vobotar-small)")
+                     "polosun-tiny | polosun-small | vobotar-tiny | vobotar-small | tonilix-tiny | tonilix-small)")
 
 
 def random_model(cfg, device, seed: int):

@@ -23,7 +23,7 @@ def main() -> int:
     ap.add_argument("--config", default="")
     ap.add_argument("--safetensors", default="")
     ap.add_argument("--tokenizer", default="")
-    ap.add_argument("--model", default="", help="random-weight preset instead of files: tiny | small | llama3-8b | fozelix-tiny | fozelix-small | polosun-tiny | polosun-small | vobotar-tiny | vobotar-small")
+    ap.add_argument("--model", default="", help="random-weight preset instead of files: tiny | small | llama3-8b | fozelix-tiny | fozelix-small | polosun-tiny | polosun-small | vobotar-tiny | vobotar-small | tonilix-tiny | tonilix-small")
     ap.add_argument("--prompt", default="Hello")
     ap.add_argument("--device", default="cpu")
     ap.add_argument("--max-new-tokens", type=int, default=32)

@@ -69,7 +69,7 @@ def test_llama_forward_and_infer():
     assert _run("llama_infer.py").returncode != 0
 
 
-@pytest.mark.parametrize("family", ["fozelix", "polosun", "vobotar"])
+@pytest.mark.parametrize("family", ["fozelix", "polosun", "vobotar", "tonilix"])
 def test_examples_take_every_registered_family(tmp_path, family):
     import torch
     from tesseract_b200 import models
