@@ -734,7 +734,7 @@ def case_pre_norm(b: Bench):
     W = 4096
     for n, rows in ((4, 4096), (256, 1), (32, 1)):
         T = n * rows
-        st = _Step(b, StateRun((W,)), n, rows, 7 if rows == 1 else 0)
+        st = _Step(b, StateRun((0,), (1, W)), n, rows, 7 if rows == 1 else 0)
         x, y, one = torch.randn(T, W, device=b.dev, generator=b.gen), b.randn(T, W), torch.ones(W, device=b.dev)
         mixed = Mixed(b.randn(T * 6, W), torch.randperm(T * 6, device=b.dev).int().view(T, 6), torch.rand(T, 6, device=b.dev))
         shift = Shift(0.5 * one, st.cache.runs[0][0])
@@ -751,10 +751,10 @@ def case_experts(b: Bench):
     up, down = b.randn(32, F, W, scale=0.02), b.randn(32, W, F, scale=0.02)
     corr = torch.zeros(32, device=b.dev)
     for T in (16384, 2048, 256, 32, 1):
-        h, z = b.randn(T, W), torch.randn(T, 32, device=b.dev, generator=b.gen)
+        h, z = b.randn(T, W), torch.randn(1, T, 32, device=b.dev, generator=b.gen)
         ms = b.time(lambda: relu2_experts(h, z, corr, c, up, down))
         from tesseract_b200.ops.moe import choose_experts_torch
-        taken = choose_experts_torch(z, corr, c)[0].unique().numel()
+        taken = choose_experts_torch(z[0], corr, c)[0].unique().numel()
         kw = dict(flops=4.0 * T * 6 * W * F) if T > 256 else dict(bytes_=taken * 2 * W * F * 2.0)
         report("experts", ms, shape=[T, 32, 6, W, F], **kw)
 

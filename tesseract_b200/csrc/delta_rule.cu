@@ -62,6 +62,14 @@ __device__ __forceinline__ float silu_f(float x) {
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// exp(-rate softplus(x)); the short form has 5e-6 of the softplus.
+template <bool FAST = false>
+__device__ __forceinline__ float decay_f(float x, float rate) {
+  if constexpr (!FAST) return expf(-rate * softplus_f(x));
+  const float e = __expf(-fabsf(x));
+  const float l = e < 0.0625f ? e * (1.f - e * (0.5f - e * (0.33333333f - 0.25f * e))) : __logf(1.f + e);
+  return __expf(-rate * (fmaxf(x, 0.f) + l));
+}
 template <bool FAST = false>
 __device__ __forceinline__ float gate_f(float x, int kind) {
   if (kind == 0) return silu_f<FAST>(x);
@@ -225,6 +233,13 @@ delta_prepare_kernel(DeltaPrepParams p) {
     const int valid = min(EPL, g.dim - d0);
     const bool vec = g.dim % EPL == 0;
     float qv[kBlk][EPL], kv[kBlk][EPL];
+    float gd[CH ? kBlk : 1][EPL];                  // CH: the inputs of a head's decays, requested ahead of the convolution
+    auto fetch = [&](int h) {                      // (rows past the end repeat the last one until they are replaced)
+#pragma unroll
+      for (int t = 0; t < (CH ? kBlk : 0); ++t)
+        load_ch<float, EPL>(p.dec + static_cast<long long>(row0 + first + min(t, cnt - 1)) * p.ld_dec + h * g.dim + d0, valid, vec, gd[t]);
+    };
+    if constexpr (CH) fetch(unit * (g.H / g.Hk));
     conv_block<T, TAPS, EPL>(p, row0, first, cnt, state_row, has_state, unit * g.dim + d0, valid, vec, qv);
     conv_block<T, TAPS, EPL>(p, row0, first, cnt, state_row, has_state, g.off_k + unit * g.dim + d0, valid, vec, kv);
     const float rsqrt_dim = rsqrtf(static_cast<float>(g.dim));
@@ -255,16 +270,14 @@ delta_prepare_kernel(DeltaPrepParams p) {
     if constexpr (CH) {
       for (int hh = 0; hh < per; ++hh) {
         const int h = unit * per + hh;
-        float gd[kBlk][EPL], bias[EPL];
-        load_ch<float, EPL>(p.dt_bias + h * g.dim + d0, valid, false, bias);
+        if (hh > 0) fetch(h);
+        float bias[EPL];
+        load_ch<float, EPL>(p.dt_bias + h * g.dim + d0, valid, vec, bias);
         const float rate = expf(p.a_log[h]);
-#pragma unroll
-        for (int t = 0; t < kBlk; ++t)             // (rows past the end repeat the last one until they are replaced)
-          load_ch<float, EPL>(p.dec + static_cast<long long>(row0 + first + min(t, cnt - 1)) * p.ld_dec + h * g.dim + d0, valid, vec, gd[t]);
 #pragma unroll
         for (int t = 0; t < kBlk; ++t)
 #pragma unroll
-          for (int e = 0; e < EPL; ++e) gd[t][e] = t < cnt && e < valid ? expf(-rate * softplus_f(gd[t][e] + bias[e])) : 1.f;
+          for (int e = 0; e < EPL; ++e) gd[t][e] = t < cnt && e < valid ? decay_f<sizeof(T) == 2>(gd[t][e] + bias[e], rate) : 1.f;
         float s[16];                               // A 10, 20, 21, 30, 31, 32, then W 00, 10, 11, 20, .. 33
 #pragma unroll
         for (int i = 0; i < 16; ++i) s[i] = 0.f;
@@ -760,12 +773,13 @@ struct DeltaStepParams {
   long long ldy;
   int y_cols, taps;
   float eps;
+  int kh;                    // key heads per CTA
 };
 
 constexpr int kStepThreads = 256;
 constexpr int kStepWarps = kStepThreads / 32;
 
-// CTA = (sequence, key head): it owns the head's q / k channels and all value heads that read them. A warp holds RPW
+// CTA = (sequence, KH key heads): it owns the heads' q / k channels and all value heads that read them. A warp holds RPW
 // rows of a 128-column block of S: dim / 8 rounded up.
 template <typename T, int RPW, bool CH>
 __global__ void __launch_bounds__(kStepThreads, RPW <= 16 ? 2 : 1)
@@ -774,22 +788,22 @@ delta_step_kernel(DeltaStepParams p) {
   pdl_grid_wait();
   const DeltaGeom& g = p.g;
   extern __shared__ __align__(16) float sm[];
-  const int per = g.H / g.Hk;
-  float* sq = sm;                          // [dkp]
-  float* sk = sq + g.dkp;                  // [dkp]
-  float* sv = sk + g.dkp;                  // [per * vp]
+  const int per1 = g.H / g.Hk, KH = p.kh, per = KH * per1, hk = blockIdx.y * KH;    // value heads per key head and of this CTA
+  float* sq = sm;                          // [KH * dkp]
+  float* sk = sq + KH * g.dkp;             // [KH * dkp]
+  float* sv = sk + KH * g.dkp;             // [per * vp]
   float* so = sv + per * g.vp;             // [per * vp]
   float* part = so + per * g.vp;           // [8 warps][2][128]
-  float* red = part + kStepWarps * 256;    // [8 warps][3]
-  float* sd = red + kStepWarps * 3 + 8;    // CH: [per * dkp] decays
-  const int row = blockIdx.x, hk = blockIdx.y;
+  float* red = part + kStepWarps * 256;    // [KH][4]: factors of q and k, k . q of the unit vectors
+  float* sd = red + KH * 4;                // CH: [per * dkp] decays
+  const int row = blockIdx.x;
   const int slot = p.slots[row];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   T* y = static_cast<T*>(p.y) + row * p.ldy;
-  if (hk == g.Hk - 1)
+  if (hk + KH == g.Hk)
     for (int c = g.H * g.vdim + tid; c < p.y_cols; c += kStepThreads) y[c] = from_f32<T>(0.f);
   if (slot < 0) {
-    for (int c = tid; c < per * g.vdim; c += kStepThreads) y[hk * per * g.vdim + c] = from_f32<T>(0.f);
+    for (int c = tid; c < per * g.vdim; c += kStepThreads) y[hk * per1 * g.vdim + c] = from_f32<T>(0.f);
     return;
   }
   const bool has_state = p.pos[row] > 0;
@@ -801,7 +815,7 @@ delta_step_kernel(DeltaStepParams p) {
   const int col_blocks = (g.vp + 127) / 128, steps = per * col_blocks;
   float4 S[RPW];
   auto state_at = [&](int it) {
-    return p.state + (static_cast<long long>(slot) * g.H + hk * per + it / col_blocks) * g.dim * g.vp + (it % col_blocks) * 128 +
+    return p.state + (static_cast<long long>(slot) * g.H + hk * per1 + it / col_blocks) * g.dim * g.vp + (it % col_blocks) * 128 +
            lane * 4;
   };
   auto fetch = [&](int it) {
@@ -816,18 +830,16 @@ delta_step_kernel(DeltaStepParams p) {
   };
   fetch(0);
   // channel i of this CTA (its q, its k, then the v of its heads): column in the projection, place in shared memory
-  const int n_ch = 2 * g.dim + per * g.vdim;
+  const int n_q = KH * g.dim, n_ch = 2 * n_q + per * g.vdim;
   auto channel = [&](int i, int* c) -> float* {
-    if (i < g.dim) {
-      *c = hk * g.dim + i;
-      return sq + i;
+    if (i < 2 * n_q) {
+      const bool is_k = i >= n_q;
+      const int j = is_k ? i - n_q : i;
+      *c = (is_k ? g.off_k : 0) + hk * g.dim + j;
+      return (is_k ? sk : sq) + (j / g.dim) * g.dkp + j % g.dim;
     }
-    if (i < 2 * g.dim) {
-      *c = g.off_k + hk * g.dim + i - g.dim;
-      return sk + i - g.dim;
-    }
-    const int v = i - 2 * g.dim;
-    *c = g.off_v + hk * per * g.vdim + v;
+    const int v = i - 2 * n_q;
+    *c = g.off_v + hk * per1 * g.vdim + v;
     return sv + (v / g.vdim) * g.vp + v % g.vdim;
   };
   for (int i0 = tid; i0 < n_ch; i0 += 2 * kStepThreads) {
@@ -862,41 +874,37 @@ delta_step_kernel(DeltaStepParams p) {
   }
   if constexpr (CH) {
     for (int i = tid; i < per * g.dim; i += kStepThreads) {
-      const int h = hk * per + i / g.dim, d = i % g.dim;
+      const int h = hk * per1 + i / g.dim, d = i % g.dim;
       sd[(i / g.dim) * g.dkp + d] =
-          expf(-expf(p.a_log[h]) * softplus_f(p.side.dec[row * p.side.ld_dec + h * g.dim + d] + p.dt_bias[h * g.dim + d]));
+          decay_f<sizeof(T) == 2>(p.side.dec[row * p.side.ld_dec + h * g.dim + d] + p.dt_bias[h * g.dim + d], expf(p.a_log[h]));
     }
   }
   __syncthreads();
-  float sqq = 0.f, skk = 0.f, sqk = 0.f;
-  for (int d = tid; d < g.dim; d += kStepThreads) {
-    sqq = fmaf(sq[d], sq[d], sqq);
-    skk = fmaf(sk[d], sk[d], skk);
-    sqk = fmaf(sq[d], sk[d], sqk);
-  }
-  sqq = warp_sum(sqq);
-  skk = warp_sum(skk);
-  sqk = warp_sum(sqk);
-  if (lane == 0) {
-    red[warp * 3] = sqq;
-    red[warp * 3 + 1] = skk;
-    red[warp * 3 + 2] = sqk;
+  for (int kh = warp; kh < KH; kh += kStepWarps) {
+    float sqq = 0.f, skk = 0.f, sqk = 0.f;
+    for (int d = lane; d < g.dim; d += 32) {
+      const float a = sq[kh * g.dkp + d], b = sk[kh * g.dkp + d];
+      sqq = fmaf(a, a, sqq);
+      skk = fmaf(b, b, skk);
+      sqk = fmaf(a, b, sqk);
+    }
+    sqq = warp_sum(sqq);
+    skk = warp_sum(skk);
+    sqk = warp_sum(sqk);
+    if (lane == 0) {
+      const float rq = 1.f / (sqrtf(sqq + 1e-6f) * sqrtf(static_cast<float>(g.dim))), rk = 1.f / sqrtf(skk + 1e-6f);
+      red[kh * 4] = rq;
+      red[kh * 4 + 1] = rk;
+      red[kh * 4 + 2] = sqk * rq * rk;
+    }
   }
   __syncthreads();
-  sqq = skk = sqk = 0.f;
-#pragma unroll
-  for (int w = 0; w < kStepWarps; ++w) {
-    sqq += red[w * 3];
-    skk += red[w * 3 + 1];
-    sqk += red[w * 3 + 2];
-  }
-  const float rq = 1.f / (sqrtf(sqq + 1e-6f) * sqrtf(static_cast<float>(g.dim)));
-  const float rk = 1.f / sqrtf(skk + 1e-6f);
-  const float kq = sqk * rq * rk;
 
   float decay = 0.f, beta = 0.f;
   for (int it = 0; it < steps; ++it) {
-    const int hh = it / col_blocks, h = hk * per + hh;
+    const int hh = it / col_blocks, h = hk * per1 + hh, kh = hh / per1;
+    const float rq = red[kh * 4], rk = red[kh * 4 + 1], kq = red[kh * 4 + 2];
+    const float *hq = sq + kh * g.dkp, *hkk = sk + kh * g.dkp;
     if (it % col_blocks == 0) {
       decay = 1.f;                        // (CH: the products with the state take their channel's decay along)
       if constexpr (!CH) decay = expf(-expf(p.a_log[h]) * softplus_f(to_f32<T>(proj[g.off_a + h]) + p.dt_bias[h]));
@@ -910,7 +918,7 @@ delta_step_kernel(DeltaStepParams p) {
 #pragma unroll
       for (int i = 0; i < RPW; ++i) {
         const int k = warp + kStepWarps * i;
-        float kk = k < g.dim ? sk[k] * rk : 0.f, qq = k < g.dim ? sq[k] * rq : 0.f;
+        float kk = k < g.dim ? hkk[k] * rk : 0.f, qq = k < g.dim ? hq[k] * rq : 0.f;
         if constexpr (CH) {
           const float dd = k < g.dim ? sd[hh * g.dkp + k] : 0.f;
           kk *= dd;
@@ -954,7 +962,7 @@ delta_step_kernel(DeltaStepParams p) {
         for (int i = 0; i < RPW; ++i) {
           const int k = warp + kStepWarps * i;
           if (k < g.dim) {
-            const float kk = sk[k] * rk, dd = CH ? sd[hh * g.dkp + k] : decay;
+            const float kk = hkk[k] * rk, dd = CH ? sd[hh * g.dkp + k] : decay;
             float4 s = S[i];
             s.x = fmaf(s.x, dd, kk * u.x);
             s.y = fmaf(s.y, dd, kk * u.y);
@@ -972,7 +980,7 @@ delta_step_kernel(DeltaStepParams p) {
   const T* gate = static_cast<const T*>(p.side.gate) + row * p.side.ld_gate;
   for (int hh = warp; hh < per; hh += kStepWarps) {
     const float* orow = so + hh * g.vp;
-    const int c0 = (hk * per + hh) * g.vdim;
+    const int c0 = (hk * per1 + hh) * g.vdim;
     float ss = 0.f;
     for (int c = lane; c < g.vdim; c += 32) ss = fmaf(orow[c], orow[c], ss);
     ss = warp_sum(ss);
@@ -1065,9 +1073,13 @@ int launch_scan_dim(const DeltaScanParams& p, int nseq, cudaStream_t s) {
 }
 
 template <typename T, int RPW, bool CH>
-int launch_step(const DeltaStepParams& p, int rows, cudaStream_t s) {
-  const int per = p.g.H / p.g.Hk;
-  const int smem = (2 * p.g.dkp + 2 * per * p.g.vp + kStepWarps * 256 + kStepWarps * 3 + 8 + (CH ? per * p.g.dkp : 0)) * 4;
+int launch_step(DeltaStepParams p, int rows, cudaStream_t s) {
+  // several key heads per CTA where that leaves every SM its CTAs: the state of the next one is under way early
+  const int per1 = p.g.H / p.g.Hk;
+  p.kh = 1;
+  while (p.kh * per1 < 4 && p.g.Hk % (2 * p.kh) == 0 && static_cast<long long>(rows) * (p.g.Hk / (2 * p.kh)) >= 3 * sm_count()) p.kh *= 2;
+  const int per = p.kh * per1;
+  const int smem = (2 * p.kh * p.g.dkp + 2 * per * p.g.vp + kStepWarps * 256 + p.kh * 4 + (CH ? per * p.g.dkp : 0)) * 4;
   if (smem > 200 * 1024) return -2;
   auto kern = delta_step_kernel<T, RPW, CH>;
   static PerDeviceFlag attr;
@@ -1076,7 +1088,7 @@ int launch_step(const DeltaStepParams& p, int rows, cudaStream_t s) {
     if (e != cudaSuccess) return static_cast<int>(e);
     attr.set();
   }
-  launch_pdl(kern, dim3(rows, p.g.Hk), dim3(kStepThreads), smem, s, pdl_all_enabled(), p);
+  launch_pdl(kern, dim3(rows, p.g.Hk / p.kh), dim3(kStepThreads), smem, s, pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -1144,7 +1156,7 @@ TSB_EXPORT int tsb_delta_step(const void* proj, long long ldp, const int* geom, 
       (dtype != 0 && dtype != 1) || y_cols < g.H * g.vdim)
     return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  DeltaStepParams p{g, side, proj, conv_w, a_log, dt_bias, norm_w, conv_state, state, slots, pos, y, ldy, y_cols, taps, eps};
+  DeltaStepParams p{g, side, proj, conv_w, a_log, dt_bias, norm_w, conv_state, state, slots, pos, y, ldy, y_cols, taps, eps, 1};
 #define TSB_STEP(R)                                                                                                       \
   if (dec) return dtype == 1 ? launch_step<__nv_bfloat16, R, true>(p, rows, s) : launch_step<float, R, true>(p, rows, s); \
   return dtype == 1 ? launch_step<__nv_bfloat16, R, false>(p, rows, s) : launch_step<float, R, false>(p, rows, s)

@@ -16,11 +16,12 @@
 namespace tsb {
 namespace {
 
-constexpr int kMaxExperts = 256, kMaxTop = 32, kPlanTokens = 256, kPlanWarps = 32, kRouteWarps = 8;
+constexpr int kMaxExperts = 256, kMaxTop = 32, kPlanTokens = 64, kPlanWarps = 32, kRouteWarps = 8;
 
 struct RouteParams {
-  const float* logits;       // [T, ld]
+  const float* logits;       // [slices, T, ld]: the sum over slices
   long long ld;
+  int slices;
   const float* correction;   // [E]
   int T, E, top, groups, keep, pad;
   float scale;
@@ -32,17 +33,22 @@ struct RouteParams {
   int* assign;               // [rows]
 };
 
-// The warp's choice for one token: lane r < top returns its r-th expert and weight. sm: 2 E floats of the warp's own.
+// The warp's choice for one token: lane r < top returns its r-th expert and weight. SL experts a lane; sm: 3 E floats of the warp's own.
+template <int SL>
 __device__ __forceinline__ void choose(const RouteParams& p, int token, float* sm, int* expert, float* weight) {
   const int lane = threadIdx.x & 31, size = p.E / p.groups;
   const float* z = p.logits + token * p.ld;
-  float *choice = sm, *worth = sm + p.E;
-  float c[kMaxExperts / 32];
+  float *choice = sm, *worth = sm + p.E, *score = worth + p.E;
+  float c[SL];
 #pragma unroll
-  for (int i = 0; i < kMaxExperts / 32; ++i) {
+  for (int i = 0; i < SL; ++i) {
     const int e = lane + 32 * i;
     c[i] = -INFINITY;
-    if (e < p.E) choice[e] = c[i] = sigmoid_f32(z[e]) + p.correction[e];
+    if (e >= p.E) continue;
+    float sum = 0.f;
+    for (int k = 0; k < p.slices; ++k) sum += z[k * p.T * p.ld + e];
+    score[e] = sigmoid_f32(sum);
+    choice[e] = c[i] = score[e] + p.correction[e];
   }
   __syncwarp();
   if (p.keep < p.groups) {
@@ -57,7 +63,7 @@ __device__ __forceinline__ void choose(const RouteParams& p, int token, float* s
     }
     __syncwarp();
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i) {
+    for (int i = 0; i < SL; ++i) {
       const int e = lane + 32 * i;
       if (e >= p.E) continue;
       const int g = e / size;
@@ -71,7 +77,7 @@ __device__ __forceinline__ void choose(const RouteParams& p, int token, float* s
     float bv = -INFINITY;
     int bi = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i)
+    for (int i = 0; i < SL; ++i)
       if (c[i] > bv) {
         bv = c[i];
         bi = lane + 32 * i;
@@ -88,10 +94,10 @@ __device__ __forceinline__ void choose(const RouteParams& p, int token, float* s
     bi = min(bi, p.E - 1);                             // (nothing compares with a NaN)
     if (lane == r) mine = bi;
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i)
+    for (int i = 0; i < SL; ++i)
       if (lane + 32 * i == bi) c[i] = -INFINITY;
   }
-  const float s = lane < p.top ? sigmoid_f32(z[mine]) : 0.f;
+  const float s = lane < p.top ? score[mine] : 0.f;
   *weight = s / (warp_sum(s) + 1e-20f) * p.scale;
   *expert = mine;
   __syncwarp();
@@ -120,6 +126,7 @@ __device__ __forceinline__ void padded_offsets(const int* counts, int E, int pad
 }
 
 // Up to kPlanTokens tokens: choice, counts, layout.
+template <int SL>
 __global__ void __launch_bounds__(kPlanWarps * 32)
 expert_plan_kernel(RouteParams p) {
   pdl_trigger();
@@ -132,7 +139,7 @@ expert_plan_kernel(RouteParams p) {
   for (int t = warp; t < p.T; t += kPlanWarps) {
     int e;
     float w;
-    choose(p, t, choice_sm + warp * 2 * p.E, &e, &w);
+    choose<SL>(p, t, choice_sm + warp * 3 * p.E, &e, &w);
     if (lane < p.top) {
       p.idx[t * p.top + lane] = e;
       p.weight[t * p.top + lane] = w;
@@ -151,6 +158,7 @@ expert_plan_kernel(RouteParams p) {
   }
 }
 
+template <int SL>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 expert_route_kernel(RouteParams p) {
   pdl_trigger();
@@ -163,7 +171,7 @@ expert_route_kernel(RouteParams p) {
   for (int t = blockIdx.x * kRouteWarps + warp; t < p.T; t += gridDim.x * kRouteWarps) {
     int e;
     float w;
-    choose(p, t, choice_sm + warp * 2 * p.E, &e, &w);
+    choose<SL>(p, t, choice_sm + warp * 3 * p.E, &e, &w);
     if (lane < p.top) {
       p.idx[static_cast<long long>(t) * p.top + lane] = e;
       p.weight[static_cast<long long>(t) * p.top + lane] = w;
@@ -231,6 +239,64 @@ expert_gather_kernel(const uint4* src, long long lds, const int* assign, const i
     for (int k = 0; k < 4; ++k)
       if (i + k * step < n) dst[i + k * step] = v[k];
   }
+}
+
+// logits[slice] [T, ld] = x W^T over the slice's columns: one tile of 16 tokens and 64 experts a CTA. Few tokens against a narrow matrix:
+// the columns are cut so that the whole is not one CTA's walk; whoever reads the logits sums the slices.
+template <typename T>
+__global__ void __launch_bounds__(128)
+expert_logits_kernel(const T* x, long long ldx, const T* w, long long ldw, float* out, long long ld, int rows, int N, int K, int step) {
+  pdl_trigger();
+  pdl_grid_wait();
+  using Tile = HeadTile<T, 16, 1>;
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int n0 = blockIdx.x * 64, row0 = blockIdx.y * 16, k0 = blockIdx.z * step, cols = min(64, N - n0);
+  const T* const wp[1] = {w + n0 * ldw + k0};
+  auto row = [&](int r) -> const T* { return row0 + r < rows ? x + (row0 + r) * ldx + k0 : nullptr; };
+  const float* c = Tile::run_rows(smem, row, wp, ldw, cols, min(step, K - k0));
+  for (int i = threadIdx.x; i < 16 * 64; i += 128) {
+    const int r = i >> 6, n = i & 63;
+    if (row0 + r < rows && n < cols) out[(static_cast<long long>(blockIdx.z) * rows + row0 + r) * ld + n0 + n] = c[r * Tile::kLdC + n];
+  }
+}
+
+template <typename T>
+int run_logits(const T* x, long long ldx, const T* w, long long ldw, float* out, long long ld, int rows, int N, int K, int slices, cudaStream_t s) {
+  auto kern = expert_logits_kernel<T>;
+  constexpr int smem = HeadTile<T, 16, 1>::kSmem;
+  static PerDeviceFlag attr;
+  if (attr.unset()) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    attr.set();
+  }
+  const int step = ((K + slices - 1) / slices + 15) / 16 * 16;
+  if ((slices - 1) * step >= K) return -2;                   // (a slice without columns)
+  launch_pdl(kern, dim3((N + 63) / 64, (rows + 15) / 16, slices), dim3(128), smem, s, pdl_all_enabled(), x, ldx, w, ldw, out, ld, rows, N, K, step);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int SL>
+int run_route(const RouteParams& p, cudaStream_t s) {
+  const bool pdl = pdl_all_enabled();
+  if (p.T <= kPlanTokens) {
+    static PerDeviceFlag attr;
+    auto kern = expert_plan_kernel<SL>;
+    if (attr.unset()) {
+      const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kPlanWarps * 3 * 32 * SL * 4);
+      if (e != cudaSuccess) return static_cast<int>(e);
+      attr.set();
+    }
+    launch_pdl(kern, dim3(1), dim3(kPlanWarps * 32), kPlanWarps * 3 * p.E * 4, s, pdl, p);
+    return static_cast<int>(cudaGetLastError());
+  }
+  const cudaError_t e = cudaMemsetAsync(p.counts, 0, 2 * p.E * sizeof(int), s);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  const int ctas = std::min((p.T + kRouteWarps - 1) / kRouteWarps, sm_count() * 8);
+  launch_pdl(expert_route_kernel<SL>, dim3(ctas), dim3(kRouteWarps * 32), kRouteWarps * 3 * p.E * 4, s, false, p);
+  const long long n = static_cast<long long>(p.T) * p.top;
+  launch_pdl(expert_place_kernel, dim3(static_cast<unsigned>((n + 1023) / 1024)), dim3(256), 0, s, pdl, p);
+  return static_cast<int>(cudaGetLastError());
 }
 
 struct ExpertParams {
@@ -316,36 +382,37 @@ int run_tile(const ExpertParams& p, int tiles, int bm, int up, cudaStream_t s) {
 }  // namespace
 }  // namespace tsb
 
-// ints: T, E, top, groups, keep, pad; ptrs: logits, correction, idx, weight, counts, offsets, pos, assign (see RouteParams). counts has 2 E
-// places; assign as many as T * top assignments of E experts may take with padding. Returns in offsets[E] (on the device) the rows in use.
+// out [slices, rows, ld] fp32, summed over slices: x [rows, K] times w [N, K]^T. K is a multiple of 16, rows start on 16 bytes.
+TSB_EXPORT int tsb_expert_logits(const void* x, long long ldx, const void* w, long long ldw, float* out, long long ld, int rows, int N, int K,
+                                 int slices, int dtype, void* stream) {
+  using namespace tsb;
+  if (rows <= 0 || N <= 0 || K <= 0 || K % 16 || ld < N || slices < 1 || slices > 64 || ldx % 8 || ldw % 8 || (reinterpret_cast<uintptr_t>(x) & 15) ||
+      (reinterpret_cast<uintptr_t>(w) & 15))
+    return -2;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == 1)
+    return run_logits(static_cast<const __nv_bfloat16*>(x), ldx, static_cast<const __nv_bfloat16*>(w), ldw, out, ld, rows, N, K, slices, s);
+  if (dtype == 0) return run_logits(static_cast<const float*>(x), ldx, static_cast<const float*>(w), ldw, out, ld, rows, N, K, slices, s);
+  return -2;
+}
+
+// ints: T, E, top, groups, keep, pad, slices; ptrs: logits, correction, idx, weight, counts, offsets, pos, assign (see RouteParams). counts
+// has 2 E places; assign as many as T * top assignments of E experts may take with padding. Returns in offsets[E] (on the device) the rows
+// in use.
 TSB_EXPORT int tsb_expert_route(const int* v, long long ld, void* const* q, float scale, void* stream) {
   using namespace tsb;
-  RouteParams p{static_cast<const float*>(q[0]), ld, static_cast<const float*>(q[1]), v[0], v[1], v[2], v[3], v[4], v[5], scale,
+  RouteParams p{static_cast<const float*>(q[0]), ld, v[6], static_cast<const float*>(q[1]), v[0], v[1], v[2], v[3], v[4], v[5], scale,
                 static_cast<int*>(q[2]), static_cast<float*>(q[3]), static_cast<int*>(q[4]), static_cast<int*>(q[5]), static_cast<int*>(q[6]),
                 static_cast<int*>(q[7])};
   if (p.T <= 0 || p.E <= 0 || p.E > kMaxExperts || p.top <= 0 || p.top > kMaxTop || p.groups <= 0 || p.E % p.groups || p.keep <= 0 ||
-      p.keep > p.groups || p.top > p.E / p.groups * p.keep || p.pad <= 0 || p.ld < p.E || static_cast<long long>(p.T) * p.top > 0x3fffffff)
+      p.keep > p.groups || p.top > p.E / p.groups * p.keep || p.pad <= 0 || p.ld < p.E || p.slices < 1 ||
+      static_cast<long long>(p.T) * p.top > 0x3fffffff)
     return -2;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const bool pdl = pdl_all_enabled();
-  if (p.T <= kPlanTokens) {
-    static PerDeviceFlag attr;
-    constexpr int most = kPlanWarps * 2 * kMaxExperts * 4;
-    if (attr.unset()) {
-      const cudaError_t e = cudaFuncSetAttribute(expert_plan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
-      if (e != cudaSuccess) return static_cast<int>(e);
-      attr.set();
-    }
-    launch_pdl(expert_plan_kernel, dim3(1), dim3(kPlanWarps * 32), kPlanWarps * 2 * p.E * 4, s, pdl, p);
-    return static_cast<int>(cudaGetLastError());
-  }
-  const cudaError_t e = cudaMemsetAsync(p.counts, 0, 2 * p.E * sizeof(int), s);
-  if (e != cudaSuccess) return static_cast<int>(e);
-  const int ctas = std::min((p.T + kRouteWarps - 1) / kRouteWarps, sm_count() * 8);
-  launch_pdl(expert_route_kernel, dim3(ctas), dim3(kRouteWarps * 32), kRouteWarps * 2 * p.E * 4, s, false, p);
-  const long long n = static_cast<long long>(p.T) * p.top;
-  launch_pdl(expert_place_kernel, dim3(static_cast<unsigned>((n + 1023) / 1024)), dim3(256), 0, s, pdl, p);
-  return static_cast<int>(cudaGetLastError());
+  if (p.E <= 32) return run_route<1>(p, s);
+  if (p.E <= 64) return run_route<2>(p, s);
+  if (p.E <= 128) return run_route<4>(p, s);
+  return run_route<8>(p, s);
 }
 
 // dst [rows_cap, cols] bf16: the first offsets[E] rows (`total` points at that number) are gathered. cols, lds: multiples of 8.

@@ -8,10 +8,11 @@
 //
 // pnorm splits a row into equal parts, each over its own root mean square. Stream, norms and shift are fp32.
 //
-// A CTA walks kRows rows; a warp owns units of 32 V columns that lie inside one part, and keeps them in registers, also those of the
-// row before. The row in front of the CTA's first is worked out once more (x is not updated in place, so it still can be). What the
-// next step of a sequence needs of its last row goes to the slot at once for single tokens, and for portions to `tail`: another CTA
-// may still have to read the slot. The next launch moves `tail` into the slots.
+// A CTA takes a row; a warp owns units of 32 V columns that lie inside one part, and keeps them in registers. With a shift the row of the
+// token before is worked out once more where it is part of the launch (x is not updated in place, so it still can be), which suits few
+// rows; many are shifted by a pass of their own (token_shift_kernel). What the next step of a sequence needs of its last row goes to the
+// slot at once for single tokens, and for portions to `tail`: another CTA may still have to read the slot. The next launch moves `tail`
+// into the slots. n' is rounded to h's type wherever it comes from.
 #include "warp_mma.cuh"
 
 #include <algorithm>
@@ -42,17 +43,17 @@ struct PreParams {
   int parts;
   float eps;
   const float* mu;          // [W] or null: no shift
-  float* last;              // [slots, W]
-  float* tail;              // [prompts, W]
+  void* last;               // [slots, h_cols]
+  void* tail;               // [prompts, h_cols]
   const int *seq_of, *slots, *cu, *pos0;
   int n_decode;
-  const float* moved;       // [n_moved, W]: what the launch before left in its tail
-  float* moved_to;          // [slots, W]
+  const void* moved;        // [n_moved, h_cols]: what the launch before left in its tail
+  void* moved_to;           // [slots, h_cols]
   const int* moved_slots;
   int n_moved;
   void* h;                  // [rows, ldh]
   long long ldh;
-  int h_cols, rows, W, blocks;
+  int h_cols, rows, W;
   int* status;
 };
 
@@ -89,17 +90,22 @@ __device__ __forceinline__ float2 sin_cos(float p, float2 f) {
   return make_float2(fmaf(c, e, s), fmaf(-s, e, c));
 }
 
-template <typename T, int V, int KEEP, bool SHIFT>
+enum StepMode { kStart, kAdd, kMixed };      // where x comes from: the embedding, x + y, x + a weighted sum of rows
+
+template <typename T, int V, int KEEP, int MODE, bool SHIFT>
 __global__ void __launch_bounds__(kMaxWarps * 32)
-pre_norm_kernel(PreParams p, int rows_per) {
+pre_norm_kernel(PreParams p) {
   pdl_trigger();
   pdl_grid_wait();
-  extern __shared__ float red[];                       // two turns of a sum per unit
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
-  if (static_cast<int>(blockIdx.x) >= p.blocks) {
-    const int i = blockIdx.x - p.blocks, slot = p.moved_slots[i];
+  constexpr int N = SHIFT ? 2 : 1;                     // rows held: the one before, then the CTA's own
+  extern __shared__ float red[];                       // two turns of a sum per row and unit
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5, row = blockIdx.x;
+  if (row >= p.rows) {
+    const int i = row - p.rows, slot = p.moved_slots[i];
     if (slot < 0) return;
-    for (int c = tid; c < p.W; c += blockDim.x) p.moved_to[static_cast<long long>(slot) * p.W + c] = p.moved[static_cast<long long>(i) * p.W + c];
+    const T* from = static_cast<const T*>(p.moved) + static_cast<long long>(i) * p.h_cols;
+    T* to = static_cast<T*>(p.moved_to) + static_cast<long long>(slot) * p.h_cols;
+    for (int c = tid; c < p.h_cols; c += blockDim.x) to[c] = from[c];
     return;
   }
   const int gs = p.W / p.parts, pieces = (gs + 32 * V - 1) / (32 * V), units = p.parts * pieces;
@@ -108,197 +114,214 @@ pre_norm_kernel(PreParams p, int rows_per) {
   for (int k = 0; k < KEEP; ++k) {
     const int u = warp + k * nw;
     part[k] = u / pieces;
-    const int c = (u % pieces) * 32 * V + lane * V;
+    const int c = (u - part[k] * pieces) * 32 * V + lane * V;
     col[k] = u < units && c < gs ? part[k] * gs + c : -1;
   }
+  // (whether the row in front belongs to the sequence is only known later; its loads do not wait)
+  const bool look_back = SHIFT && row > p.n_decode;
+  auto used = [&](int n) { return n == N - 1 || look_back; };
+  float a[N][KEEP][V];
   int turn = 0;
   // a -> a / rms of its part * w
-  auto norm = [&](float (&a)[KEEP][V], const float* w) {
-    float* r = red + (turn ^= 1) * units;
+  auto norm = [&](const float* w) {
+    float* r = red + (turn ^= 1) * N * units;
 #pragma unroll
-    for (int k = 0; k < KEEP; ++k) {
-      float ss = 0.f;
-      if (col[k] >= 0) {
+    for (int n = 0; n < N; ++n)
 #pragma unroll
-        for (int i = 0; i < V; ++i) ss = fmaf(a[k][i], a[k][i], ss);
+      for (int k = 0; k < KEEP; ++k) {
+        float ss = 0.f;
+        if (col[k] >= 0 && used(n)) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) ss = fmaf(a[n][k][i], a[n][k][i], ss);
+        }
+        ss = warp_sum(ss);
+        if (lane == 0 && warp + k * nw < units) r[n * units + warp + k * nw] = ss;
       }
-      ss = warp_sum(ss);
-      if (lane == 0 && warp + k * nw < units) r[warp + k * nw] = ss;
-    }
     __syncthreads();
+    float sums[N][KEEP];                               // of the parts that this warp's units lie in
+#pragma unroll
+    for (int n = 0; n < N; ++n)
+#pragma unroll
+      for (int k = 0; k < KEEP; ++k) {
+        const float* z = r + n * units + min(part[k], p.parts - 1) * pieces;
+        float ss = 0.f;
+        if (pieces <= 2) {
+          ss = z[0] + (pieces > 1 ? z[1] : 0.f);
+        } else {
+          for (int j = lane; j < pieces; j += 32) ss += z[j];
+          ss = warp_sum(ss);
+        }
+        sums[n][k] = ss;
+      }
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
       if (col[k] < 0) continue;
-      float ss = 0.f, g[V];
-      for (int j = 0; j < pieces; ++j) ss += r[part[k] * pieces + j];
-      const float rs = 1.f / sqrtf(ss / static_cast<float>(gs) + p.eps);
+      float g[V];
       ld_v<float, V>(w + col[k], g);
 #pragma unroll
-      for (int i = 0; i < V; ++i) a[k][i] *= rs * g[i];
+      for (int n = 0; n < N; ++n) {
+        const float rs = 1.f / sqrtf(sums[n][k] / static_cast<float>(gs) + p.eps);
+#pragma unroll
+        for (int i = 0; i < V; ++i) a[n][k][i] *= rs * g[i];
+      }
     }
   };
-  // the normed row; `store`: x goes out
-  auto work = [&](int row, bool store, float (&a)[KEEP][V]) {
-    if (p.tokens) {
-      int tok = p.tokens[row];
+  if constexpr (MODE == kStart) {
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      if (!used(n)) continue;
+      const int at = row - (N - 1) + n;
+      int tok = p.tokens[at];
       if (tok < 0 || tok >= p.vocab) {
         if (tid == 0 && p.status) atomicCAS(p.status, kStatusOk, kStatusBadIndex);
         tok = 0;
       }
       const T* emb = static_cast<const T*>(p.table) + tok * p.ld_table;
-      const float at = static_cast<float>(max(p.positions[row], 0));
+      const float pos = static_cast<float>(max(p.positions[at], 0));
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         if (col[k] < 0) continue;
-        ld_v<T, V>(emb + col[k], a[k]);
+        ld_v<T, V>(emb + col[k], a[n][k]);
         if (!p.freq) continue;
         if constexpr (V == 1) {
-          const float2 sc = sin_cos(at, p.freq[col[k] >> 1]);
-          a[k][0] += col[k] & 1 ? sc.y : sc.x;
+          const float2 sc = sin_cos(pos, p.freq[col[k] >> 1]);
+          a[n][k][0] += col[k] & 1 ? sc.y : sc.x;
         } else {
 #pragma unroll
           for (int i = 0; i < V; i += 2) {
-            const float2 sc = sin_cos(at, p.freq[(col[k] + i) >> 1]);
-            a[k][i] += sc.x;
-            a[k][i + 1] += sc.y;
+            const float2 sc = sin_cos(pos, p.freq[(col[k] + i) >> 1]);
+            a[n][k][i] += sc.x;
+            a[n][k][i + 1] += sc.y;
           }
         }
       }
-      if (p.embed_gain) norm(a, p.embed_gain);
-    } else {
-      const float* x = p.x + static_cast<long long>(row) * p.W;
-      float b[KEEP][V];
+    }
+    if (p.embed_gain) norm(p.embed_gain);
+  } else {
+    float b[N][KEEP][V];
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const long long at = row - (N - 1) + n;
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
-        if (col[k] < 0) continue;
-        ld_v<float, V>(x + col[k], a[k]);
-        if (p.y && !p.pos) ld_v<T, V>(static_cast<const T*>(p.y) + row * p.ldy + col[k], b[k]);
+#pragma unroll
+        for (int i = 0; i < V; ++i) b[n][k][i] = 0.f;
+        if (col[k] < 0 || !used(n)) continue;
+        ld_v<float, V>(p.x + at * p.W + col[k], a[n][k]);
+        if (MODE == kAdd && p.y) ld_v<T, V>(static_cast<const T*>(p.y) + at * p.ldy + col[k], b[n][k]);
       }
-      if (p.y && p.pos) {
+    }
+    if constexpr (MODE == kMixed) {
+      for (int j = 0; j < p.top; ++j) {
 #pragma unroll
-        for (int k = 0; k < KEEP; ++k)
-#pragma unroll
-          for (int i = 0; i < V; ++i) b[k][i] = 0.f;
-        for (int j = 0; j < p.top; ++j) {
-          const long long at = static_cast<long long>(row) * p.top + j;
-          const T* e = static_cast<const T*>(p.y) + p.pos[at] * p.ldy;
-          const float w = p.weight[at];
+        for (int n = 0; n < N; ++n) {
+          if (!used(n)) continue;
+          const long long i = static_cast<long long>(row - (N - 1) + n) * p.top + j;
+          const T* e = static_cast<const T*>(p.y) + p.pos[i] * p.ldy;
+          const float w = p.weight[i];
 #pragma unroll
           for (int k = 0; k < KEEP; ++k) {
             if (col[k] < 0) continue;
             float f[V];
             ld_v<T, V>(e + col[k], f);
 #pragma unroll
-            for (int i = 0; i < V; ++i) b[k][i] = fmaf(w, f[i], b[k][i]);
-          }
-        }
-      }
-      if (p.y) {
-#pragma unroll
-        for (int k = 0; k < KEEP; ++k) {
-          if (col[k] < 0) continue;
-          float f[V];
-          if (p.bias) {
-            ld_v<float, V>(p.bias + col[k], f);
-#pragma unroll
-            for (int i = 0; i < V; ++i) b[k][i] += f[i];
-          }
-          if (p.scale) {
-            ld_v<float, V>(p.scale + col[k], f);
-#pragma unroll
-            for (int i = 0; i < V; ++i) a[k][i] = fmaf(b[k][i], f[i], a[k][i]);
-          } else {
-#pragma unroll
-            for (int i = 0; i < V; ++i) a[k][i] += b[k][i];
+            for (int i = 0; i < V; ++i) b[n][k][i] = fmaf(w, f[i], b[n][k][i]);
           }
         }
       }
     }
-    if (store && p.x_out) {
-#pragma unroll
-      for (int k = 0; k < KEEP; ++k)
-        if (col[k] >= 0) st_v<float, V>(p.x_out + static_cast<long long>(row) * p.W + col[k], a[k]);
-    }
-    norm(a, p.gain);
-  };
-  float cur[KEEP][V], prev[SHIFT ? KEEP : 1][V];
-  bool have = false;                                   // prev holds the row before
-  for (int r = 0; r < rows_per; ++r) {
-    const int row = blockIdx.x * rows_per + r;
-    if (row >= p.rows) return;
-    if constexpr (SHIFT) {
-      const int seq = p.seq_of[row], slot = p.slots[seq];
-      bool start = true, old = false, ends = false;
-      if (row < p.n_decode) {
-        old = p.positions[row] > 0;
-      } else {
-        const int i = seq - p.n_decode;
-        start = row == p.n_decode + p.cu[i];
-        ends = row + 1 == p.n_decode + p.cu[i + 1];
-        old = p.pos0[i] > 0;
-      }
-      if (start) {
-#pragma unroll
-        for (int k = 0; k < KEEP; ++k) {
-#pragma unroll
-          for (int i = 0; i < V; ++i) prev[k][i] = 0.f;
-          if (old && slot >= 0 && col[k] >= 0) ld_v<float, V>(p.last + static_cast<long long>(slot) * p.W + col[k], prev[k]);
-        }
-      } else if (!have) {
-        work(row - 1, false, prev);
-      }
-      work(row, true, cur);
-      have = true;
-      float* keep = row < p.n_decode ? (slot >= 0 ? p.last + static_cast<long long>(slot) * p.W : nullptr)
-                                     : (ends ? p.tail + static_cast<long long>(seq - p.n_decode) * p.W : nullptr);
-      if (keep) {
-#pragma unroll
-        for (int k = 0; k < KEEP; ++k)
-          if (col[k] >= 0) st_v<float, V>(keep + col[k], cur[k]);
-      }
+    if (MODE == kMixed || p.y) {
 #pragma unroll
       for (int k = 0; k < KEEP; ++k) {
         if (col[k] < 0) continue;
-        float m[V], o[V];
-        ld_v<float, V>(p.mu + col[k], m);
+        float bias[V], scale[V];
 #pragma unroll
         for (int i = 0; i < V; ++i) {
-          o[i] = fmaf(prev[k][i] - cur[k][i], m[i], cur[k][i]);
-          prev[k][i] = cur[k][i];
+          bias[i] = 0.f;
+          scale[i] = 1.f;
         }
-        st_v<T, V>(static_cast<T*>(p.h) + row * p.ldh + col[k], o);
-      }
-    } else {
-      work(row, true, cur);
+        if (p.bias) ld_v<float, V>(p.bias + col[k], bias);
+        if (p.scale) ld_v<float, V>(p.scale + col[k], scale);
 #pragma unroll
-      for (int k = 0; k < KEEP; ++k)
-        if (col[k] >= 0) st_v<T, V>(static_cast<T*>(p.h) + row * p.ldh + col[k], cur[k]);
+        for (int n = 0; n < N; ++n)
+#pragma unroll
+          for (int i = 0; i < V; ++i) a[n][k][i] = fmaf(b[n][k][i] + bias[i], scale[i], a[n][k][i]);
+      }
     }
-    for (int c = p.W + tid; c < p.h_cols; c += blockDim.x) static_cast<T*>(p.h)[row * p.ldh + c] = from_f32<T>(0.f);
+  }
+  if (p.x_out) {
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k)
+      if (col[k] >= 0) st_v<float, V>(p.x_out + static_cast<long long>(row) * p.W + col[k], a[N - 1][k]);
+  }
+  bool joined = false;                                 // the row above is the token before
+  const T* before = nullptr;                           // the token before is in a slot
+  T* keep = nullptr;                                   // where the next step of the sequence finds this row
+  if constexpr (SHIFT) {
+    const int seq = p.seq_of[row], slot = p.slots[seq];
+    T* mine = slot >= 0 ? static_cast<T*>(p.last) + static_cast<long long>(slot) * p.h_cols : nullptr;
+    bool old;
+    if (row < p.n_decode) {
+      old = p.positions[row] > 0;
+      keep = mine;
+    } else {
+      const int i = seq - p.n_decode;
+      joined = row > p.n_decode + p.cu[i];
+      if (row + 1 == p.n_decode + p.cu[i + 1]) keep = static_cast<T*>(p.tail) + static_cast<long long>(i) * p.h_cols;
+      old = p.pos0[i] > 0;
+    }
+    if (!joined && old) before = mine;
+  }
+  norm(p.gain);
+  T* h = static_cast<T*>(p.h) + row * p.ldh;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    if (col[k] < 0) continue;
+    const float(&cur)[V] = a[N - 1][k];
+    if constexpr (SHIFT) {
+      float m[V], prev[V], o[V];
+      ld_v<float, V>(p.mu + col[k], m);
+#pragma unroll
+      for (int i = 0; i < V; ++i) prev[i] = joined ? to_f32<T>(from_f32<T>(a[0][k][i])) : 0.f;
+      if (before) ld_v<T, V>(before + col[k], prev);
+#pragma unroll
+      for (int i = 0; i < V; ++i) o[i] = fmaf(prev[i] - cur[i], m[i], cur[i]);
+      st_v<T, V>(h + col[k], o);
+      if (keep) st_v<T, V>(keep + col[k], cur);
+    } else {
+      st_v<T, V>(h + col[k], cur);
+    }
+  }
+  for (int c = p.W + tid; c < p.h_cols; c += blockDim.x) {
+    h[c] = from_f32<T>(0.f);
+    if (keep) keep[c] = from_f32<T>(0.f);
   }
 }
 
-template <typename T, int V>
-int launch_pre(PreParams& p, cudaStream_t s) {
-  const int gs = p.W / p.parts, units = p.parts * ((gs + 32 * V - 1) / (32 * V));
-  const int nw = std::min(kMaxWarps, std::max(1, (units + 1) / 2)), keep = (units + nw - 1) / nw;
-  const int per = p.rows > 2048 ? 8 : 1;
-  p.blocks = (p.rows + per - 1) / per;
-  const dim3 grid(p.blocks + p.n_moved), block(nw * 32);
-  const size_t smem = 2 * units * sizeof(float);
-  if (keep > 8 || smem > 48 * 1024) return -2;
-  const bool pdl = pdl_all_enabled();
-#define TSB_PRE(K)                                                                              \
-  do {                                                                                          \
-    if (p.mu) launch_pdl(pre_norm_kernel<T, V, K, true>, grid, block, smem, s, pdl, p, per);    \
-    else launch_pdl(pre_norm_kernel<T, V, K, false>, grid, block, smem, s, pdl, p, per);        \
-  } while (0)
-  if (keep == 1) TSB_PRE(1);
-  else if (keep == 2) TSB_PRE(2);
-  else if (keep <= 4) TSB_PRE(4);
-  else TSB_PRE(8);
-#undef TSB_PRE
+template <typename T, int V, int KEEP, int MODE>
+int launch_mode(const PreParams& p, int nw, int units, cudaStream_t s) {
+  const dim3 grid(p.rows + p.n_moved), block(nw * 32);
+  const size_t smem = 4 * units * sizeof(float);
+  if (p.mu) launch_pdl(pre_norm_kernel<T, V, KEEP, MODE, true>, grid, block, smem, s, pdl_all_enabled(), p);
+  else launch_pdl(pre_norm_kernel<T, V, KEEP, MODE, false>, grid, block, smem, s, pdl_all_enabled(), p);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int V, int KEEP>
+int launch_keep(const PreParams& p, int nw, int units, cudaStream_t s) {
+  if (p.tokens) return launch_mode<T, V, KEEP, kStart>(p, nw, units, s);
+  if (p.pos) return launch_mode<T, V, KEEP, kMixed>(p, nw, units, s);
+  return launch_mode<T, V, KEEP, kAdd>(p, nw, units, s);
+}
+
+template <typename T, int V>
+int launch_pre(const PreParams& p, cudaStream_t s) {
+  const int gs = p.W / p.parts, units = p.parts * ((gs + 32 * V - 1) / (32 * V));
+  const int nw = std::min(kMaxWarps, (units + 1) / 2), keep = (units + nw - 1) / nw;
+  if (keep <= 2) return launch_keep<T, V, 2>(p, nw, units, s);
+  if constexpr (V == 4)
+    if (keep <= 4) return launch_keep<T, V, 4>(p, nw, units, s);
+  return keep <= 8 ? launch_keep<T, V, 8>(p, nw, units, s) : -2;
 }
 
 }  // namespace
@@ -315,8 +338,8 @@ TSB_EXPORT int tsb_pre_norm_step(const int* v, const long long* ld, void* const*
   auto f = [&](int i) { return static_cast<float*>(q[i]); };
   auto n = [&](int i) { return static_cast<const int*>(q[i]); };
   p.x = f(0); p.x_out = f(1); p.y = q[2]; p.pos = n(3); p.weight = f(4); p.bias = f(5); p.scale = f(6); p.tokens = n(7); p.table = q[8];
-  p.freq = static_cast<const float2*>(q[9]); p.embed_gain = f(10); p.positions = n(11); p.gain = f(12); p.mu = f(13); p.last = f(14);
-  p.tail = f(15); p.seq_of = n(16); p.slots = n(17); p.cu = n(18); p.pos0 = n(19); p.moved = f(20); p.moved_to = f(21);
+  p.freq = static_cast<const float2*>(q[9]); p.embed_gain = f(10); p.positions = n(11); p.gain = f(12); p.mu = f(13); p.last = q[14];
+  p.tail = q[15]; p.seq_of = n(16); p.slots = n(17); p.cu = n(18); p.pos0 = n(19); p.moved = q[20]; p.moved_to = q[21];
   p.moved_slots = n(22); p.h = q[23];
   if (p.rows <= 0 || p.W <= 0 || p.parts <= 0 || p.W % p.parts || p.h_cols < p.W || !p.h || !p.gain || (dtype != 0 && dtype != 1) ||
       (p.tokens ? (!p.table || !p.x_out || !p.positions || p.y) : !p.x) || (p.y && !p.x_out) || p.x == p.x_out ||

@@ -382,9 +382,11 @@ class _PreLayer(_Layer):
         vec = lambda on: torch.zeros(c.width, dtype=torch.float32, device=device) if on else None   # noqa: E731
         self.mixer, self.mlp = _make_mixer(spec.mixer, c, device), _make_mlp(spec.mlp, c, device)
         self.norm1, self.norm2 = norm(), norm() if spec.mlp is not None else None
-        self.ls1, self.ls2, self.shift = vec(c.layer_scale), vec(c.layer_scale and spec.mlp is not None), vec(c.token_shift)
-        self.extra = {n: t for n, t in (("ls1", self.ls1), ("ls2", self.ls2), ("shift", self.shift)) if t is not None}
-        self.width = c.width
+        self.ls1, self.ls2, self.shift = vec(c.layer_scale), vec(c.layer_scale and spec.mlp is not None), None
+        self.extra = {n: t for n, t in (("ls1", self.ls1), ("ls2", self.ls2)) if t is not None}
+        if c.token_shift:
+            self.shift = torch.zeros(pad_to(c.width), dtype=torch.float32, device=device)
+            self.extra["shift"] = self.shift[:c.width]
 
     def parts(self):
         out = [("norm1", self.norm1), ("mix.", self.mixer)]
@@ -395,7 +397,7 @@ class _PreLayer(_Layer):
     def run_spec(self):
         """With a token shift: the mixer's storage, and the last input of every sequence."""
         spec = self.mixer.run_spec()
-        return PairRun(spec, StateRun((self.width,))) if self.shift is not None else spec
+        return PairRun(spec, StateRun((0,), (1, self.shift.shape[0]))) if self.shift is not None else spec
 
     def storage(self, run):
         """(the mixer's storage, what the norm takes for the shift)"""

@@ -28,7 +28,7 @@ from ..ops.retention import SPAN, RetentionGeometry, log2_decays, retention
 from ..ops.rglru import CHUNK, RGLRUGeometry, RGLRUWeights, rglru
 from ..ops.rotary import Rotary
 from ..ops.ssd import CONV_TILE, SSDGeometry, SSDWeights, ssd
-from ..ops.moe import Choice, relu2_experts
+from ..ops.moe import Choice, relu2_experts, router_logits
 from ..ops.timemix import (SPAN as STATE_SPAN, STREAMS, GatedLinearGeometry, GatedLinearWeights, TimeMixGeometry, TimeMixWeights, gated_linear,
                            time_mix, token_shift)
 from .ragged import LatentRun, PagedRun, PairRun, StateRun
@@ -416,7 +416,7 @@ class ExpertMLP(_Packed):
         return out
 
     def forward(self, h):
-        return relu2_experts(h, ops.project(h, self.w_router, out_dtype=torch.float32), self.correction, self.choice, self.w_up, self.w_down)
+        return relu2_experts(h, router_logits(h, self.w_router), self.correction, self.choice, self.w_up, self.w_down)
 
 
 def _head_rows(at: int, heads: int, stride: int, columns: torch.Tensor) -> torch.Tensor:

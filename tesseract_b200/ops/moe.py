@@ -21,7 +21,7 @@ import torch
 
 from .. import _native
 from .._native import check, lib, stream_ptr
-from .gemm import gemm_bf16, linear
+from .gemm import gemm_bf16, linear, project
 from .fused import swiglu
 
 P, I, L = _native.P, _native.I, _native.L
@@ -307,12 +307,15 @@ def moe_ffn_grouped(x2: torch.Tensor, idx: torch.Tensor, gates: torch.Tensor, mo
 
 # ------------------------------------------------------------------------------ serving: grouped choice, squared-ReLU experts
 _native.register_signatures({
+    "tsb_expert_logits": [P, L, P, L, P, L, I, I, I, I, I, P],
     "tsb_expert_route": [P, L, P, _native.F, P],
     "tsb_expert_gather": [P, L, P, P, P, I, I, I, P],
     "tsb_expert_tiles": [P, P, P, I, P],
 })
 MAX_EXPERTS, MAX_TOP = 256, 32
-TILE_ROWS = 256              # up to so many tokens the experts' rows go through tiles of 16 (bf16)
+FEW_TOKENS = 256             # router products of so many share the columns among CTAs
+PLAN_TOKENS = 64             # one CTA chooses for so many and lays them out
+TILE_ROWS = 16               # up to so many rows per expert on average they go through tiles of 16 (bf16)
 
 
 @dataclass(frozen=True)
@@ -360,23 +363,36 @@ def choose_experts_torch(logits: torch.Tensor, correction: torch.Tensor, c: Choi
     return idx, w / (w.sum(1, keepdim=True) + 1e-20) * c.scale
 
 
+def router_logits(h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """h [T, K] times w [N, K]^T in fp32: [slices, T, N], to be summed over slices (few tokens: K is cut, so that several CTAs share it)."""
+    T, K = h.shape
+    if not h.is_cuda or T > FEW_TOKENS:
+        return project(h, w, out_dtype=torch.float32)[None]
+    slices = max(1, min(8, K // 256))
+    out = torch.empty((slices, T, w.shape[0]), device=h.device, dtype=torch.float32)
+    check(lib().tsb_expert_logits(h.data_ptr(), h.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), w.shape[0], T, w.shape[0], K, slices,
+                                  _native.dtype_code(h.dtype), stream_ptr(h.device)), "tsb_expert_logits")
+    return out
+
+
 def relu2_experts(h: torch.Tensor, logits: torch.Tensor, correction: torch.Tensor, c: Choice, w_up: torch.Tensor,
                   w_down: torch.Tensor) -> Mixed:
-    """Every token's chosen experts W_down relu(W_up h)^2. h [T, K] and ``logits`` [T, >= experts] (fp32) of the same rows, ``w_up``
+    """Every token's chosen experts W_down relu(W_up h)^2. h [T, K] and ``logits`` [slices, T, >= experts] (fp32, summed over
+    slices) of the same rows, ``w_up``
     [experts, F, K], ``w_down`` [experts, W, F] in the type of h, F and K multiples of 16; ``correction`` fp32 [experts]."""
     T, K = h.shape
     E, F, top, dev = c.experts, w_up.shape[1], c.top, h.device
     W = w_down.shape[1]
     if not h.is_cuda:
-        idx, weight = choose_experts_torch(logits[:, :E], correction, c)
+        idx, weight = choose_experts_torch(logits.sum(0)[:, :E], correction, c)
         rows = torch.empty((T * top, W), dtype=h.dtype)
         for e in range(E):
             t, j = (idx == e).nonzero(as_tuple=True)
             a = torch.relu(h[t].float() @ w_up[e].float().t()) ** 2
             rows[t * top + j] = (a.to(h.dtype).float() @ w_down[e].float().t()).to(h.dtype)
         return Mixed(rows, torch.arange(T * top).view(T, top), weight)
-    grouped = h.dtype == torch.bfloat16 and T > TILE_ROWS
-    pad = 128 if grouped else 16 if T <= TILE_ROWS else 64
+    grouped = h.dtype == torch.bfloat16 and T * top > TILE_ROWS * E
+    pad = 128 if grouped else 16 if T * top <= TILE_ROWS * E else 64
     tiles = min(E, T * top) + T * top // pad          # (an expert without rows has no tile)
     i32 = lambda *s: torch.empty(s, device=dev, dtype=torch.int32)   # noqa: E731
     idx, pos, offsets, assign, counts = i32(T, top), i32(T, top), i32(E + 1), i32(tiles * pad), i32(2 * E)
@@ -384,10 +400,11 @@ def relu2_experts(h: torch.Tensor, logits: torch.Tensor, correction: torch.Tenso
     st = stream_ptr(dev)
     ptrs = (ctypes.c_void_p * 8)(logits.data_ptr(), correction.data_ptr(), idx.data_ptr(), weight.data_ptr(), counts.data_ptr(),
                                  offsets.data_ptr(), pos.data_ptr(), assign.data_ptr())
-    check(lib().tsb_expert_route((ctypes.c_int * 6)(T, E, top, c.groups, c.keep, pad), logits.stride(0), ptrs, float(c.scale), st),
+    check(lib().tsb_expert_route((ctypes.c_int * 7)(T, E, top, c.groups, c.keep, pad, logits.shape[0]), logits.stride(1), ptrs, float(c.scale), st),
           "tsb_expert_route")
-    if grouped:
+    if T > PLAN_TOKENS:
         _native.add_launches(1)
+    if grouped:
         xs = torch.empty((tiles * pad, K), device=dev, dtype=h.dtype)
         check(lib().tsb_expert_gather(h.data_ptr(), h.stride(0), assign.data_ptr(), offsets[E:].data_ptr(), xs.data_ptr(), tiles * pad, K, top,
                                       st), "tsb_expert_gather")

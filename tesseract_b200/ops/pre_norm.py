@@ -10,9 +10,11 @@ import torch
 from .. import _native
 from .._native import check, dtype_code, lib, stream_ptr
 from .moe import Mixed
+from .timemix import token_shift
 
 P, I, F = _native.P, _native.I, _native.F
 _native.register_signatures({"tsb_pre_norm_step": [P, P, P, F, I, P]})
+SHIFT_ROWS = 1024            # prompt rows of a step up to which the shift is part of it
 
 
 def _ptr(t):
@@ -29,7 +31,8 @@ class Moved:
 
 @dataclass
 class Shift:
-    """h + (h' - h) mu with h' of the token before: ``mu`` fp32 [W]; ``last`` [slots, W] (fp32) carries the last row of every sequence."""
+    """h + (h' - h) mu with h' of the token before, rounded to the type of h: ``mu`` fp32 [columns of h]; ``last`` [slots, 1, columns of h]
+    carries the last row of every sequence."""
     mu: torch.Tensor
     last: torch.Tensor
 
@@ -61,9 +64,12 @@ def pre_norm_step(batch, width, gain, parts, eps, x=None, y=None, bias=None, sca
     start = table is not None
     dev = table.device if start else x.device
     h = torch.empty((T, out_cols or W), device=dev, dtype=out_dtype or (table.dtype if start else torch.float32))
+    if shift is not None and h.is_cuda and T - batch.n_decode > SHIFT_ROWS:      # (many rows: cheaper than to work out most of them twice)
+        new, h, _ = pre_norm_step(batch, W, gain, parts, eps, x, y, bias, scale, table, freq, embed_gain, None, moved, out_cols, out_dtype)
+        return new, token_shift(h, shift.mu[None], shift.last, batch)[0], None
     new = torch.empty((T, W), device=dev, dtype=torch.float32)
     prompts = shift is not None and batch.n_prompts > 0
-    after = (Moved(torch.empty((batch.n_prompts, W), device=dev, dtype=torch.float32), shift.last, batch.state_slots[batch.n_decode:])
+    after = (Moved(torch.empty((batch.n_prompts, h.shape[1]), device=dev, dtype=h.dtype), shift.last, batch.state_slots[batch.n_decode:])
              if prompts else None)
     if T == 0:
         return new, h, after
@@ -90,7 +96,7 @@ def pre_norm_step(batch, width, gain, parts, eps, x=None, y=None, bias=None, sca
 
 def _pre_norm_torch(batch, W, gain, parts, eps, x, y, bias, scale, table, freq, embed_gain, shift, moved, new, h, after):
     if moved is not None:
-        moved.last[moved.slots.long()] = moved.tail
+        moved.last[moved.slots.long(), 0] = moved.tail
     if table is not None:
         new.copy_(table[batch.tokens.long(), :W])
         if freq is not None:
@@ -108,13 +114,14 @@ def _pre_norm_torch(batch, W, gain, parts, eps, x, y, bias, scale, table, freq, 
     if shift is not None:
         out = n.clone()
         for i, (row0, rows, slot, pos0) in enumerate(batch.spans()):
-            first = shift.last[slot][None] if pos0 > 0 and slot >= 0 else torch.zeros(1, W)
             z = n[row0:row0 + rows]
-            out[row0:row0 + rows] = z + (torch.cat([first, z[:-1]]) - z) * shift.mu
+            kept = torch.nn.functional.pad(z, (0, h.shape[1] - W)).to(h.dtype)
+            first = shift.last[slot] if pos0 > 0 and slot >= 0 else torch.zeros(1, h.shape[1])
+            out[row0:row0 + rows] = z + (torch.cat([first, kept[:-1]])[:, :W].float() - z) * shift.mu[:W]
             if i >= batch.n_decode:
-                after.tail[i - batch.n_decode] = z[-1]
+                after.tail[i - batch.n_decode] = kept[-1]
             elif slot >= 0:
-                shift.last[slot] = z[-1]
+                shift.last[slot] = kept[-1]
         n = out
     h[:, W:] = 0
     h[:, :W] = n

@@ -20,7 +20,7 @@ from tesseract_b200.models.scheduler import ContinuousBatchingScheduler, EngineC
 from tesseract_b200.nn.hybrid import ExpertMLP, GatedDelta, GatedLinear, ShapedAttention
 from tesseract_b200.nn.ragged import HybridCache, HybridSequence, RaggedBatch
 from tesseract_b200.ops.delta import DeltaGeometry
-from tesseract_b200.ops.moe import Mixed, choose_experts_torch, relu2_experts
+from tesseract_b200.ops.moe import Mixed, choose_experts_torch, relu2_experts, router_logits
 from tesseract_b200.ops.pre_norm import Moved, Shift, pre_norm_step, sinusoid_frequencies
 from tesseract_b200.ops.ragged import ScoreForm
 from tesseract_b200.ops.timemix import GatedLinearGeometry
@@ -178,7 +178,8 @@ class Rows:
         g = torch.Generator().manual_seed(seed)
         self.cache = HybridCache([], 64, 8, 6, 512, getattr(torch, kind[1]), kind[0])
         self.cache.slot_allocator.allocate()
-        self.last = torch.randn(6, W, generator=g).to(kind[0])
+        C = (W + 15) // 16 * 16
+        self.last = torch.randn(6, 1, C, generator=g).to(kind[0], getattr(torch, kind[1]))
         self.toks = {}
         self.g, self.vocab = g, vocab
 
@@ -241,27 +242,29 @@ def test_token_shift_across_rows_steps_and_slots(kind, W, parts):
     dev, dt = kind[0], getattr(torch, kind[1])
     r = Rows(kind, W, parts, seed=W)
     rnd = lambda *s: torch.randn(*s, generator=r.g)   # noqa: E731
-    gain, mu, eps = (1 + 0.3 * rnd(W)).to(dev), rnd(W).to(dev), 1e-3
+    cols = r.last.shape[2]
+    gain, mu, eps = (1 + 0.3 * rnd(W)).to(dev), torch.nn.functional.pad(rnd(W), (0, cols - W)).to(dev), 1e-3
     big = 2100 if dev == "cuda" and W == 40 else 20           # (more rows than a launch takes one by one)
     r.cache = HybridCache([], 800, 8, 6, 6000, dt, dev)
     r.cache.slot_allocator.allocate()
     seqs = [HybridSequence(r.cache) for _ in range(4)]
     plan = [[(0, 5), (1, 1)], [(1, 1), (0, 1), (2, 2)], [(2, 9), (0, big), (1, 1), (3, 1)], [(0, 1), (1, 3), (2, 17), (3, 2)], [(0, 1), (1, 1), (2, 1)]]
     moved, stream = None, {i: rnd(sum(dict(p).get(i, 0) for p in plan), W) for i in range(4)}
-    want = {i: oracle.shifted_mix(oracle.part_rms_norm(s.double(), gain.double().cpu(), parts, eps), mu.double().cpu()) for i, s in stream.items()}
+    want = {i: oracle.shifted_mix(oracle.part_rms_norm(s.double(), gain.double().cpu(), parts, eps), mu[:W].double().cpu()) for i, s in stream.items()}
     at = dict.fromkeys(stream, 0)
     for p in plan:
         batch = RaggedBatch(r.cache, [(seqs[i], [0] * n) for i, n in p])
         x = torch.empty(batch.rows, W)
         for e, (i, n) in enumerate(p):
             x[batch.row_of[e]:batch.row_of[e] + n] = stream[i][at[i]:at[i] + n]
-        _, h, moved = pre_norm_step(batch, W, gain, parts, eps, x.to(dev), shift=Shift(mu, r.last), out_dtype=dt)
+        _, h, moved = pre_norm_step(batch, W, gain, parts, eps, x.to(dev), shift=Shift(mu, r.last), out_cols=cols, out_dtype=dt)
         if moved is not None:
             assert isinstance(moved, Moved)
-            _, _, none = pre_norm_step(batch, W, gain, parts, eps, x.to(dev), moved=moved, out_dtype=dt)
+            _, _, none = pre_norm_step(batch, W, gain, parts, eps, x.to(dev), moved=moved, out_cols=cols, out_dtype=dt)
             assert none is None
         for e, (i, n) in enumerate(p):
-            got = h[batch.row_of[e]:batch.row_of[e] + n].double().cpu()
+            got = h[batch.row_of[e]:batch.row_of[e] + n, :W].double().cpu()
+            assert float(h[:, W:].abs().sum()) == 0.0
             assert (got - want[i][at[i]:at[i] + n]).abs().max() < (2e-5 if dt == torch.float32 else 0.1), (p, i)
             at[i] += n
         batch.commit()
@@ -559,7 +562,8 @@ def test_choice_of_experts(kind, E, top, groups, keep, T):
     corr = (w["correction"].double() * 0).float()
     corr += torch.linspace(-0.9, -0.95, E)          # (scores are at least 8 / E apart in the middle, the correction moves them little)
     s = oracle.sigmoid(logits[:, :E].double())
-    got = relu2_experts(hp.to(dev), logits.to(dev), corr.to(dev), c, blk.w_up, blk.w_down)
+    parts = torch.stack([0.25 * logits, 0.75 * logits]) if T < 100 else logits[None]
+    got = relu2_experts(hp.to(dev), parts.to(dev), corr.to(dev), c, blk.w_up, blk.w_down)
     d = {n: t.double() for n, t in w.items()}
     weights = got.weight.cpu().double()
     summed = got.sum().cpu().double()
@@ -572,6 +576,15 @@ def test_choice_of_experts(kind, E, top, groups, keep, T):
         assert torch.allclose(weights[t].sort().values, torch.stack([s[t, e] / total * 1.7 for e in ids]).sort().values, atol=1e-6)
         want = sum(s[t, e] / total * 1.7 * (torch.clamp(h[t].double() @ d[f"e{e}.up"].t(), min=0) ** 2 @ d[f"e{e}.down"].t()) for e in ids)
         assert (summed[t] - want).abs().max() < (1e-4 if dt == torch.float32 else 0.03) * max(1.0, float(want.abs().max())), t
+
+
+@pytest.mark.parametrize("kind", KINDS)
+@pytest.mark.parametrize("T,K,N", [(1, 16, 8), (5, 2048, 72), (40, 304, 16), (256, 784, 128), (300, 528, 8)])
+def test_router_logits(kind, T, K, N):
+    g, dt = torch.Generator().manual_seed(K), getattr(torch, kind[1])
+    h, w = torch.randn(T, K, generator=g).to(dt), (torch.randn(N, K, generator=g) * K ** -0.5).to(dt)
+    got = router_logits(h.to(kind[0]), w.to(kind[0]))
+    assert got.dtype == torch.float32 and (got.sum(0).cpu().double() - h.double() @ w.double().t()).abs().max() < 2e-5      # in either type
 
 
 def test_masked_experts_stay_out_although_all_scores_are_negative():
@@ -601,7 +614,7 @@ def test_experts_of_long_prompts(kind, T, E, W, F):
     logits = torch.randn(T, (E + 7) // 8 * 8, generator=g)
     logits[:, 0] += 6.0
     logits[:, E - 1] -= 12.0
-    got = relu2_experts(h.to(kind[0]), logits.to(kind[0]), torch.zeros(E, device=kind[0]), c, blk.w_up, blk.w_down).sum().cpu().double()
+    got = relu2_experts(h.to(kind[0]), logits[None].to(kind[0]), torch.zeros(E, device=kind[0]), c, blk.w_up, blk.w_down).sum().cpu().double()
     idx, weight = choose_experts_torch(logits[:, :E], torch.zeros(E), c)
     want = torch.zeros(T, W, dtype=torch.float64)
     for e in range(E):
