@@ -20,6 +20,7 @@ import torch
 
 from .. import ops
 from ..ops.delta import DeltaGeometry, DeltaWeights, gated_delta
+from ..ops.pre_norm import NORM_UNIT, NORM_UNITS
 from ..ops.latent import LatentGeometry, LatentWeights, latent_attention
 from ..ops.gemm import input_columns
 from ..ops.masks import Window
@@ -146,6 +147,8 @@ class PartRMSNorm(RMSNorm):
     def __init__(self, width: int, parts: int, eps: float, dtype, device):
         if parts < 1 or width % parts:
             raise ValueError("norm: the width is a multiple of its parts")
+        if parts * -(-(width // parts) // NORM_UNIT[width // parts % 4 == 0]) > NORM_UNITS:
+            raise ValueError("norm: the row has too many parts or columns")
         super().__init__(width, eps, 0.0, dtype, device)
         self.parts = parts
 

@@ -14,6 +14,7 @@ from .timemix import token_shift
 
 P, I, F = _native.P, _native.I, _native.F
 _native.register_signatures({"tsb_pre_norm_step": [P, P, P, F, I, P]})
+NORM_UNITS, NORM_UNIT = 128, (32, 128)      # a row is at most so many runs of 32 columns (128 where parts are multiples of 4) inside parts
 SHIFT_ROWS = 1024            # prompt rows of a step up to which the shift is part of it
 
 

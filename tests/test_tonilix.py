@@ -831,7 +831,7 @@ def test_size_errors():
     d = DeltaSpec(1, 1, 8, 8, 2, 4, 4)
     experts = ExpertSpec(8, Choice(4, 2, 1, 1, 1.0))
     for kw in (dict(layers=[LayerSpec(d, experts)]), dict(layers=[LayerSpec(d)], norm_parts=2), dict(layers=[LayerSpec(d)], token_shift=True),
-               dict(layers=[LayerSpec(d)], form="pre", norm_parts=3), dict(layers=[LayerSpec(d)], form="pre", embedding_scale=2.0)):
+               dict(layers=[LayerSpec(d)], form="pre", norm_parts=3), dict(layers=[LayerSpec(d)], form="pre", norm_parts=0), dict(layers=[LayerSpec(d)], form="pre", embedding_scale=2.0)):
         with pytest.raises(ValueError):
             HybridModel(HybridConfig(8, 8, **kw))
 
